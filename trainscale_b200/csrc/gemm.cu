@@ -41,7 +41,13 @@ struct GemmParams {
   const int* seg_start;     // MODE 2: [E + 1] first row of every expert's (128-aligned) segment along the K axis
   int group_rows;           // MODE 1: rows (K-major B) or K extent (MN-major B) of one expert inside the stacked B
   int num_groups;           // MODE 2: E; C is [E][M][ldc]
+  int act;                  // MODE 1 epilogue activation: 0 none, 1 squared ReLU
 };
+
+__device__ __forceinline__ float relu_squared(float v) {
+  v = fmaxf(v, 0.f);
+  return v * v;
+}
 
 // 32 consecutive fp32 accumulator columns of one output row: scale, optionally add to C, convert, store.
 __device__ __forceinline__ void gemm_store_chunk(const GemmParams& p, const uint32_t* r, size_t row, int col0) {
@@ -317,6 +323,10 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
         uint32_t r[32];
         tmem_ld_32x32b_x32(t_row + c * 32, r);
         tc_wait_ld();
+        if (MODE == 1 && p.act == 1) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(relu_squared(__uint_as_float(r[j])));
+        }
         const int col0 = n0 + c * 32;
         if (row < p.M && col0 < p.N) gemm_store_chunk(p, r, ti.c_row0 + row, col0);
       }
@@ -580,7 +590,7 @@ extern "C" int ts_gemm_bf16(const void* A, const void* B, void* C, int M, int N,
   p.num_m_tiles = (M + GEMM_BM - 1) / GEMM_BM;
   p.num_n_tiles = (N + bn - 1) / bn;
   p.k_blocks = (K + GEMM_BK - 1) / GEMM_BK;
-  p.tile_expert = nullptr; p.seg_start = nullptr; p.group_rows = 0; p.num_groups = 1;
+  p.tile_expert = nullptr; p.seg_start = nullptr; p.group_rows = 0; p.num_groups = 1; p.act = 0;
   p.c_bytes = (static_cast<size_t>(M - 1) * ldc + N) * (out_fp32 ? 4 : 2);
 #ifdef TS_DEBUG
   // test hook of the debug build: pretend C ends `TS_DEBUG_SHRINK_C_ROWS` rows early, so that the bounds check (and
@@ -603,13 +613,16 @@ extern "C" int ts_gemm_bf16(const void* A, const void* B, void* C, int M, int N,
 //   mode 2 (wgrad): C[e][M][N] = sum over rows r in [seg_start[e], seg_start[e+1]) of A[r][m] * B[r][n]; both operands
 //     MN-major (a_mn = b_mn = 1), K = P.  An empty segment gives a zero slab (or leaves C alone when accumulating).
 // `groups` is the device int32 array tile_expert (mode 1, ceil(P/128) entries) or seg_start (mode 2, E + 1 entries).
+// `act` (mode 1): 1 applies max(v, 0)^2 to the product in the epilogue (C must not accumulate then).
 // Serves the grouped expert GEMMs of data_pipeline/trainer/kernels/moe_kernels.py:219-785.
-extern "C" int ts_gemm_grouped_bf16(const void* A, const void* B, void* C, int mode, int M, int N, int K, int lda,
-                                    int ldb, int ldc, int a_mn, int b_mn, int out_fp32, int accumulate, float alpha,
-                                    const int* groups, int num_groups, void* stream) {
+extern "C" int ts_gemm_grouped_bf16_act(const void* A, const void* B, void* C, int mode, int M, int N, int K, int lda,
+                                        int ldb, int ldc, int a_mn, int b_mn, int out_fp32, int accumulate, float alpha,
+                                        const int* groups, int num_groups, int act, void* stream) {
   using namespace ts;
   if (M <= 0 || N <= 0 || K <= 0 || num_groups <= 0 || groups == nullptr) return -10;
-  if (mode == 1 && (a_mn != 0 || K % GEMM_BK != 0)) return -12;
+  // experts stacked along K (b_mn) need whole K blocks; with K-major B the tail of K is zero-filled by the loads
+  if (mode == 1 && (a_mn != 0 || (b_mn && K % GEMM_BK != 0))) return -12;
+  if (act != 0 && (mode != 1 || act != 1 || accumulate || alpha != 1.f)) return -13;
   if (mode == 2 && (a_mn != 1 || b_mn != 1)) return -12;
   if (mode != 1 && mode != 2) return -11;
   const int bn = (N >= 256) ? 256 : (N >= 128 ? 128 : 64);
@@ -636,6 +649,7 @@ extern "C" int ts_gemm_grouped_bf16(const void* A, const void* B, void* C, int m
   p.seg_start = (mode == 2) ? groups : nullptr;
   p.group_rows = b_mn ? K : N;
   p.num_groups = num_groups;
+  p.act = act;
   p.c_bytes = (static_cast<size_t>((mode == 2 ? num_groups : 1)) * M - 1) * ldc * (out_fp32 ? 4 : 2) +
               static_cast<size_t>(N) * (out_fp32 ? 4 : 2);
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
@@ -647,4 +661,11 @@ extern "C" int ts_gemm_grouped_bf16(const void* A, const void* B, void* C, int m
   if (bn == 256) return launch_gemm<256, 2>(tmA, tmB, p, st);
   if (bn == 128) return launch_gemm<128, 2>(tmA, tmB, p, st);
   return launch_gemm<64, 2>(tmA, tmB, p, st);
+}
+
+extern "C" int ts_gemm_grouped_bf16(const void* A, const void* B, void* C, int mode, int M, int N, int K, int lda,
+                                    int ldb, int ldc, int a_mn, int b_mn, int out_fp32, int accumulate, float alpha,
+                                    const int* groups, int num_groups, void* stream) {
+  return ts_gemm_grouped_bf16_act(A, B, C, mode, M, N, K, lda, ldb, ldc, a_mn, b_mn, out_fp32, accumulate, alpha, groups,
+                                  num_groups, 0, stream);
 }

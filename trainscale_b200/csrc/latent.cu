@@ -1,0 +1,488 @@
+// Latent attention over a paged cache: every token caches ONE row [latent c (rank) | rotated key part (rot)] that all
+// heads share, instead of keys and values per head.
+//
+//   ts_latent_prep    split of the q | down projection: RMS norm of the latent, rotary embedding of the shared key part
+//                     and of every head's rotated query part (in place), cache write - one launch
+//   ts_latent_gather  cache rows of a list of slots -> contiguous rows (the keys a portion of a prompt needs again)
+//   ts_latent_attend  attention in latent space for single query rows against the paged cache.  The query's unrotated
+//                     part has been carried into latent space (q_lat = W_uk^T q), so scores are dot products with the
+//                     cached row, and the weighted sum of latents is returned (W_uv is applied afterwards):
+//                       s_j = (q_lat . c_j + q_rot . r_j) * scale,   o = sum_j softmax(s)_j c_j
+//                     for the keys max(0, len - window) <= j < len of the row's sequence.  Reads each cached row once
+//                     for all heads; long windows are split over CTAs and merged by log-sum-exp.
+//
+// Two attention kernels: `latent_attend_mma_kernel` (bf16; 16 heads are the rows of warp MMAs, the CTA's tile of cached
+// rows is both K and V) and `latent_attend_simt_kernel` (fp32, or bf16 sizes the tiles do not fit).
+#include "common.cuh"
+#include "host_common.h"
+
+namespace ts {
+
+template <typename T> __device__ __forceinline__ T from_f32(float v);
+template <> __device__ __forceinline__ float from_f32<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
+__device__ __forceinline__ float to_f32(float v) { return v; }
+__device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
+
+// One CTA per token.  proj row: [H heads x (dim | rot)] [latent rank | rot].
+template <typename T>
+__global__ void __launch_bounds__(128)
+latent_prep_kernel(T* __restrict__ proj, long long ld, int H, int dim, int rot, int rank, const float* __restrict__ norm_w,
+                   float eps, const float* __restrict__ inv_freq, const int* __restrict__ pos,
+                   const long long* __restrict__ slots, T* __restrict__ cache, T* __restrict__ flat, int row_width) {
+  extern __shared__ float cs[];     // cos | sin of the token's rot / 2 angles
+  __shared__ float scratch[32];
+  const int t = blockIdx.x, half = rot / 2;
+  T* q = proj + static_cast<long long>(t) * ld;
+  const T* down = q + H * (dim + rot);
+  const float p = static_cast<float>(pos[t]);
+  for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(p * inv_freq[i], &cs[half + i], &cs[i]);
+  float ss = 0.f;
+  for (int r = threadIdx.x; r < rank; r += blockDim.x) {
+    const float v = to_f32(down[r]);
+    ss += v * v;
+  }
+  ss = block_sum(ss, scratch);      // also orders the angles
+  const float inv = 1.f / sqrtf(ss / static_cast<float>(rank) + eps);
+  T* crow = cache + slots[t] * row_width;
+  T* frow = flat ? flat + static_cast<long long>(t) * row_width : nullptr;
+  for (int r = threadIdx.x; r < row_width; r += blockDim.x) {
+    float v = 0.f;                  // columns past rank + rot pad the row
+    if (r < rank) {
+      v = to_f32(down[r]) * inv * norm_w[r];
+    } else if (r < rank + rot) {
+      const int i = r - rank;
+      const float a = to_f32(down[r]);
+      v = i < half ? a * cs[i] - to_f32(down[r + half]) * cs[half + i]
+                   : a * cs[i - half] + to_f32(down[r - half]) * cs[i];
+    }
+    crow[r] = from_f32<T>(v);
+    if (frow) frow[r] = from_f32<T>(v);
+  }
+  for (int i = threadIdx.x; i < H * half; i += blockDim.x) {
+    const int h = i / half, j = i - h * half;
+    T* a = q + h * (dim + rot) + dim + j;
+    const float u = to_f32(a[0]), v = to_f32(a[half]), c = cs[j], s = cs[half + j];
+    a[0] = from_f32<T>(u * c - v * s);
+    a[half] = from_f32<T>(v * c + u * s);
+  }
+}
+
+__global__ void latent_gather_kernel(const uint4* __restrict__ cache, const long long* __restrict__ slots,
+                                     uint4* __restrict__ out, long long rows, int vec) {
+  const long long total = rows * vec;
+  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < total;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long r = i / vec;
+    out[i] = cache[slots[r] * vec + (i - r * vec)];
+  }
+}
+
+struct LatentAttendParams {
+  const void* q_lat;          // [rows][H][rank]
+  const void* q;              // projection rows; rotated part of head h at column h * (dim + rot) + dim
+  long long q_ld;
+  const void* cache;          // [slots][row_width]
+  const int* block_table;     // [sequences][max_blocks]
+  const int* row_seq;         // [rows] sequence of a row (nullptr: the row itself)
+  const int* row_len;         // [rows] keys visible before the window is applied (position + 1)
+  void* out;                  // [rows][H][rank]
+  float* part_out;            // [rows][H][splits][rank]
+  float* part_lse;            // [rows][H][splits]
+  int rows, H, dim, rot, rank, row_width, max_blocks, block_size, window, chunk, splits;
+  float scale;
+};
+
+__device__ __forceinline__ void attend_range(const LatentAttendParams& p, int row, int split, int& j0, int& j1) {
+  const int len = p.row_len[row];
+  const int lo = max(0, len - p.window);
+  j0 = lo + split * p.chunk;
+  j1 = min(len, j0 + p.chunk);
+}
+
+// grid (rows, H, splits).  Scores of the chunk go to shared memory, then threads own latent columns.
+template <typename T>
+__global__ void __launch_bounds__(128) latent_attend_simt_kernel(LatentAttendParams p) {
+  extern __shared__ float sm[];
+  __shared__ float scratch[32];
+  const int row = blockIdx.x, h = blockIdx.y, split = blockIdx.z;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  float* qs = sm;                          // [rank + rot]
+  float* sc = sm + p.rank + p.rot;         // [chunk]
+  int j0, j1;
+  attend_range(p, row, split, j0, j1);
+  const int seq = p.row_seq ? p.row_seq[row] : row;
+  const int* bt = p.block_table + static_cast<long long>(seq) * p.max_blocks;
+  const T* cache = reinterpret_cast<const T*>(p.cache);
+  const T* ql = reinterpret_cast<const T*>(p.q_lat) + (static_cast<long long>(row) * p.H + h) * p.rank;
+  const T* qr = reinterpret_cast<const T*>(p.q) + row * p.q_ld + h * (p.dim + p.rot) + p.dim;
+  for (int i = threadIdx.x; i < p.rank + p.rot; i += blockDim.x) qs[i] = to_f32(i < p.rank ? ql[i] : qr[i - p.rank]);
+  __syncthreads();
+  float mx = -INFINITY;
+  for (int j = j0 + warp; j < j1; j += nw) {
+    const T* c = cache + (static_cast<long long>(bt[j / p.block_size]) * p.block_size + j % p.block_size) * p.row_width;
+    float s = 0.f;
+    for (int i = lane; i < p.rank + p.rot; i += 32) s += qs[i] * to_f32(c[i]);
+    s = warp_sum(s) * p.scale;
+    if (lane == 0) sc[j - j0] = s;
+    mx = fmaxf(mx, s);
+  }
+  mx = block_max(mx, scratch);
+  float l = 0.f;
+  for (int j = j0 + threadIdx.x; j < j1; j += blockDim.x) {
+    const float w = expf(sc[j - j0] - mx);
+    sc[j - j0] = w;
+    l += w;
+  }
+  l = block_sum(l, scratch);               // also orders the weights
+  const float inv = l > 0.f ? 1.f / l : 0.f;
+  const long long o = (static_cast<long long>(row) * p.H + h);
+  for (int r = threadIdx.x; r < p.rank; r += blockDim.x) {
+    float acc = 0.f;
+    for (int j = j0; j < j1; ++j)
+      acc += sc[j - j0] *
+             to_f32(cache[(static_cast<long long>(bt[j / p.block_size]) * p.block_size + j % p.block_size) * p.row_width + r]);
+    if (p.splits == 1) reinterpret_cast<T*>(p.out)[o * p.rank + r] = from_f32<T>(acc * inv);
+    else p.part_out[(o * p.splits + split) * p.rank + r] = acc * inv;
+  }
+  if (p.splits > 1 && threadIdx.x == 0) p.part_lse[o * p.splits + split] = l > 0.f ? mx + logf(l) : -INFINITY;
+}
+
+template <typename T>
+__global__ void latent_merge_kernel(LatentAttendParams p) {
+  const long long o = static_cast<long long>(blockIdx.x) * p.H + blockIdx.y;
+  const float* lse = p.part_lse + o * p.splits;
+  float mx = -INFINITY, den = 0.f;
+  for (int s = 0; s < p.splits; ++s) mx = fmaxf(mx, lse[s]);
+  for (int s = 0; s < p.splits; ++s) den += lse[s] == -INFINITY ? 0.f : expf(lse[s] - mx);
+  for (int r = threadIdx.x; r < p.rank; r += blockDim.x) {
+    float acc = 0.f;
+    for (int s = 0; s < p.splits; ++s)
+      if (lse[s] != -INFINITY) acc += expf(lse[s] - mx) * p.part_out[(o * p.splits + s) * p.rank + r];
+    reinterpret_cast<T*>(p.out)[o * p.rank + r] = from_f32<T>(acc / den);
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------
+// bf16 decode kernel.  grid (rows, ceil(H / 16), splits), 8 warps.  Tiles of KT cached rows stream through two
+// shared-memory buffers (cp.async); a tile serves as K (all row_width columns) and as V (the first rank columns).
+//   scores   warp w: the 16 heads x keys [8w, 8w + 8) of the tile, over all columns
+//   softmax  warp w: heads 2w, 2w + 1 (running max and sum in registers, fp32)
+//   output   warp w: latent columns [16 NP w, 16 NP (w + 1)) of the 16 heads, fp32 accumulators in registers
+// ---------------------------------------------------------------------------------------------------------
+constexpr int LD_WARPS = 8;
+constexpr int LD_KT = 64;
+
+__device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(addr));
+}
+__device__ __forceinline__ void ldsm_x4_t(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(addr));
+}
+__device__ __forceinline__ void mma_16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src));
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;"); }
+template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N)); }
+
+// shared-memory row stride in elements: an odd number of 16-byte units, so that ldmatrix rows hit different banks
+__host__ __device__ inline int latent_stride(int width) { return (width / 8 + 1 - (width / 8) % 2) * 8; }
+static size_t latent_smem_bytes(int row_width) {
+  const size_t st = latent_stride(row_width);
+  return (2 * LD_KT + 16) * st * 2 + 16 * (LD_KT + 8) * 2 + 16 * (LD_KT + 4) * 4 + 16 * 4 * 2;
+}
+
+template <int NP>   // pairs of 8-wide column tiles per warp: rank <= 128 * NP
+__global__ void __launch_bounds__(LD_WARPS * 32) latent_attend_mma_kernel(LatentAttendParams p) {
+  extern __shared__ __align__(16) uint8_t raw[];
+  const int st = latent_stride(p.row_width), cols = p.row_width;
+  __nv_bfloat16* kv = reinterpret_cast<__nv_bfloat16*>(raw);             // [2][KT][st]
+  __nv_bfloat16* qs = kv + 2 * LD_KT * st;                               // [16][st]
+  __nv_bfloat16* ps = qs + 16 * st;                                      // [16][KT + 8]
+  float* ss = reinterpret_cast<float*>(ps + 16 * (LD_KT + 8));           // [16][KT + 4]
+  float* s_alpha = ss + 16 * (LD_KT + 4);                                // [16]
+  float* s_l = s_alpha + 16;                                             // [16]
+  const int row = blockIdx.x, h0 = blockIdx.y * 16, split = blockIdx.z;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  int j0, j1;
+  attend_range(p, row, split, j0, j1);
+  const int seq = p.row_seq ? p.row_seq[row] : row;
+  const int* bt = p.block_table + static_cast<long long>(seq) * p.max_blocks;
+  const __nv_bfloat16* cache = reinterpret_cast<const __nv_bfloat16*>(p.cache);
+  const __nv_bfloat16* ql = reinterpret_cast<const __nv_bfloat16*>(p.q_lat) + static_cast<long long>(row) * p.H * p.rank;
+  const __nv_bfloat16* qr = reinterpret_cast<const __nv_bfloat16*>(p.q) + row * p.q_ld;
+  const int vec = cols / 8;
+  const int tiles = j1 > j0 ? (j1 - j0 + LD_KT - 1) / LD_KT : 0;
+
+  auto load_tile = [&](int i) {
+    __nv_bfloat16* dst = kv + (i & 1) * LD_KT * st;
+    const int base = j0 + i * LD_KT, n = min(LD_KT, j1 - base);
+    for (int x = threadIdx.x; x < LD_KT * vec; x += LD_WARPS * 32) {
+      const int r = x / vec, c = x - r * vec;
+      const int j = base + r;
+      if (r < n) {
+        const long long slot = static_cast<long long>(bt[j / p.block_size]) * p.block_size + j % p.block_size;
+        cp_async16(smem_u32(dst + r * st + c * 8), cache + slot * cols + c * 8);
+      } else {
+        *reinterpret_cast<uint4*>(dst + r * st + c * 8) = make_uint4(0u, 0u, 0u, 0u);   // keeps 0 * x finite
+      }
+    }
+    cp_async_commit();
+  };
+  if (tiles > 0) load_tile(0);
+  // the 16 query rows: [q_lat | q_rot | 0]
+  for (int x = threadIdx.x; x < 16 * cols; x += LD_WARPS * 32) {
+    const int r = x / cols, c = x - r * cols, h = h0 + r;
+    __nv_bfloat16 v = __float2bfloat16(0.f);
+    if (h < p.H) {
+      if (c < p.rank) v = ql[h * p.rank + c];
+      else if (c < p.rank + p.rot) v = qr[h * (p.dim + p.rot) + p.dim + c - p.rank];
+    }
+    qs[r * st + c] = v;
+  }
+  float o[2 * NP][4];
+#pragma unroll
+  for (int i = 0; i < 2 * NP; ++i)
+#pragma unroll
+    for (int q = 0; q < 4; ++q) o[i][q] = 0.f;
+  float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+  const float sl = p.scale * 1.4426950408889634f;
+  const int gid = lane >> 2, tig = lane & 3;
+
+  for (int i = 0; i < tiles; ++i) {
+    const __nv_bfloat16* tile = kv + (i & 1) * LD_KT * st;
+    if (i + 1 < tiles) {
+      load_tile(i + 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    const int n = min(LD_KT, j1 - (j0 + i * LD_KT));
+    {   // scores: four independent accumulators over the columns
+      float c[4][4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u)
+#pragma unroll
+        for (int q = 0; q < 4; ++q) c[u][q] = 0.f;
+      const uint32_t qa = smem_u32(qs + (lane & 15) * st + (lane >> 4) * 8);
+      const uint32_t ka = smem_u32(tile + (warp * 8 + (lane & 7)) * st + (lane >> 3) * 8);
+      int k = 0;
+      for (; k + 64 <= cols; k += 64) {
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          uint32_t a0[4], a1[4], b[4];
+          ldsm_x4(a0, qa + (k + u * 32) * 2);
+          ldsm_x4(a1, qa + (k + u * 32 + 16) * 2);
+          ldsm_x4(b, ka + (k + u * 32) * 2);       // 8 keys x 32 columns
+          mma_16816(c[2 * u], a0, b[0], b[1]);
+          mma_16816(c[2 * u + 1], a1, b[2], b[3]);
+        }
+      }
+      for (; k < cols; k += 16) {
+        uint32_t a0[4], b0, b1;
+        ldsm_x4(a0, qa + k * 2);
+        asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];"
+                     : "=r"(b0), "=r"(b1)
+                     : "r"(smem_u32(tile + (warp * 8 + (lane & 7)) * st + ((lane >> 3) & 1) * 8 + k)));
+        mma_16816(c[0], a0, b0, b1);
+      }
+      float* d = ss + gid * (LD_KT + 4) + warp * 8 + tig * 2;
+      d[0] = (c[0][0] + c[1][0]) + (c[2][0] + c[3][0]);
+      d[1] = (c[0][1] + c[1][1]) + (c[2][1] + c[3][1]);
+      d[8 * (LD_KT + 4)] = (c[0][2] + c[1][2]) + (c[2][2] + c[3][2]);
+      d[8 * (LD_KT + 4) + 1] = (c[0][3] + c[1][3]) + (c[2][3] + c[3][3]);
+    }
+    __syncthreads();
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {   // softmax of heads 2 warp, 2 warp + 1; two keys per lane
+      const int r = warp * 2 + u;
+      const float s0 = lane < n ? ss[r * (LD_KT + 4) + lane] * sl : -INFINITY;
+      const float s1 = lane + 32 < n ? ss[r * (LD_KT + 4) + lane + 32] * sl : -INFINITY;
+      const float m_new = fmaxf(m_run[u], warp_max(fmaxf(s0, s1)));   // n >= 1: finite
+      const float alpha = exp2f(m_run[u] - m_new);
+      const float p0 = exp2f(s0 - m_new), p1 = exp2f(s1 - m_new);
+      m_run[u] = m_new;
+      l_run[u] = l_run[u] * alpha + warp_sum(p0 + p1);
+      ps[r * (LD_KT + 8) + lane] = __float2bfloat16(p0);
+      ps[r * (LD_KT + 8) + lane + 32] = __float2bfloat16(p1);
+      if (lane == 0) s_alpha[r] = alpha;
+    }
+    __syncthreads();
+    {
+      const float al0 = s_alpha[gid], al1 = s_alpha[gid + 8];
+      if (i > 0) {
+#pragma unroll
+        for (int x = 0; x < 2 * NP; ++x) {
+          o[x][0] *= al0; o[x][1] *= al0; o[x][2] *= al1; o[x][3] *= al1;
+        }
+      }
+      const uint32_t pa = smem_u32(ps + (lane & 15) * (LD_KT + 8) + (lane >> 4) * 8);
+#pragma unroll
+      for (int kk = 0; kk < LD_KT / 16; ++kk) {
+        if (kk * 16 >= n) break;
+        uint32_t a[4];
+        ldsm_x4(a, pa + kk * 32);
+#pragma unroll
+        for (int x = 0; x < NP; ++x) {
+          const int c0 = (warp * NP + x) * 16;
+          if (c0 < p.rank) {
+            uint32_t b[4];    // keys kk*16 .. +16 (two 8-row matrices) x columns c0 .. +16 (two), transposed
+            ldsm_x4_t(b, smem_u32(tile + (kk * 16 + (lane & 15)) * st + c0 + (lane >> 4) * 8));
+            mma_16816(o[2 * x], a, b[0], b[1]);
+            mma_16816(o[2 * x + 1], a, b[2], b[3]);
+          }
+        }
+      }
+    }
+    __syncthreads();   // the tile's buffer, ps and ss are free again
+  }
+  if (lane == 0) {
+    s_l[warp * 2] = l_run[0];
+    s_l[warp * 2 + 1] = l_run[1];
+    if (p.splits > 1) {
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        const int h = h0 + warp * 2 + u;
+        if (h < p.H)
+          p.part_lse[(static_cast<long long>(row) * p.H + h) * p.splits + split] =
+              l_run[u] > 0.f ? (m_run[u] + log2f(l_run[u])) * 0.6931471805599453f : -INFINITY;
+      }
+    }
+  }
+  __syncthreads();
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {
+    const int r = gid + half * 8, h = h0 + r;
+    if (h >= p.H) continue;
+    const float inv = s_l[r] > 0.f ? 1.f / s_l[r] : 0.f;
+    const long long base = static_cast<long long>(row) * p.H + h;
+#pragma unroll
+    for (int x = 0; x < 2 * NP; ++x) {
+      const int c = (warp * NP + (x >> 1)) * 16 + (x & 1) * 8 + tig * 2;
+      if (c < p.rank) {
+        const float v0 = o[x][2 * half] * inv, v1 = o[x][2 * half + 1] * inv;
+        if (p.splits == 1)
+          *reinterpret_cast<uint32_t*>(reinterpret_cast<__nv_bfloat16*>(p.out) + base * p.rank + c) = pack_bf16x2(v0, v1);
+        else
+          *reinterpret_cast<float2*>(p.part_out + (base * p.splits + split) * p.rank + c) = make_float2(v0, v1);
+      }
+    }
+  }
+}
+
+}  // namespace ts
+
+TS_DEFINE_ERROR_API(ts_latent)
+using namespace ts;
+#define ST(s) reinterpret_cast<cudaStream_t>(s)
+
+// Width of a cache row: rank + rot rounded up to whole 16-column MMA steps.
+extern "C" int ts_latent_row_width(int rank, int rot) { return (rank + rot + 15) / 16 * 16; }
+
+extern "C" int ts_latent_prep(void* proj, long long ld, int H, int dim, int rot, int rank, const float* norm_w, float eps,
+                              const float* inv_freq, const int* pos, const long long* slots, void* cache, void* flat,
+                              int row_width, int rows, int fp32, void* stream) {
+  if (rows <= 0) return 0;
+  if (H <= 0 || rank <= 0 || rot < 0 || rot % 2 || row_width < rank + rot) return -10;
+  const size_t sm = sizeof(float) * (rot > 0 ? rot : 2);
+  if (fp32)
+    latent_prep_kernel<float><<<rows, 128, sm, ST(stream)>>>((float*)proj, ld, H, dim, rot, rank, norm_w, eps, inv_freq,
+                                                             pos, slots, (float*)cache, (float*)flat, row_width);
+  else
+    latent_prep_kernel<__nv_bfloat16><<<rows, 128, sm, ST(stream)>>>(
+        (__nv_bfloat16*)proj, ld, H, dim, rot, rank, norm_w, eps, inv_freq, pos, slots, (__nv_bfloat16*)cache,
+        (__nv_bfloat16*)flat, row_width);
+  return (int)cudaGetLastError();
+}
+
+extern "C" int ts_latent_gather(const void* cache, const long long* slots, void* out, long long rows, int row_bytes,
+                                void* stream) {
+  if (rows <= 0) return 0;
+  if (row_bytes <= 0 || row_bytes % 16) return -10;
+  const int vec = row_bytes / 16;
+  long long blocks = (rows * vec + 255) / 256;
+  const long long cap = static_cast<long long>(sm_count()) * 16;
+  if (blocks > cap) blocks = cap;
+  latent_gather_kernel<<<(unsigned)blocks, 256, 0, ST(stream)>>>((const uint4*)cache, slots, (uint4*)out, rows, vec);
+  return (int)cudaGetLastError();
+}
+
+static int latent_mma_fits(int rank, int row_width, int fp32) {
+  return !fp32 && rank % 16 == 0 && rank <= 512 && row_width % 16 == 0 && latent_smem_bytes(row_width) <= 227 * 1024;
+}
+
+// Number of CTAs a window is split over: enough to fill the GPU, no more than there are tiles.
+extern "C" int ts_latent_splits(int rows, int H, int rank, int row_width, int max_keys, int fp32) {
+  const int mma = latent_mma_fits(rank, row_width, fp32);
+  const long long units = static_cast<long long>(rows) * (mma ? (H + 15) / 16 : H);
+  const int unit_keys = mma ? LD_KT : 256;
+  const int most = (max_keys + unit_keys - 1) / unit_keys;
+  long long s = (2ll * sm_count() + units - 1) / units;
+  if (s > most) s = most;
+  if (!mma && s < (max_keys + 2047) / 2048) s = (max_keys + 2047) / 2048;   // the chunk's scores sit in shared memory
+  return (int)(s < 1 ? 1 : s);
+}
+
+// max_keys: upper bound of the visible keys of any row (min of window and longest length).  part_out / part_lse:
+// workspaces when splits > 1.
+extern "C" int ts_latent_attend(const void* q_lat, const void* q, long long q_ld, const void* cache,
+                                const int* block_table, int max_blocks, const int* row_seq, const int* row_len, void* out,
+                                float* part_out, float* part_lse, int rows, int H, int dim, int rot, int rank,
+                                int row_width, int block_size, int window, int max_keys, int splits, float scale, int fp32,
+                                void* stream) {
+  if (rows <= 0) return 0;
+  if (H <= 0 || rank <= 0 || block_size <= 0 || window <= 0 || splits <= 0 || splits > 65535) return -10;
+  LatentAttendParams p;
+  p.q_lat = q_lat; p.q = q; p.q_ld = q_ld; p.cache = cache; p.block_table = block_table; p.row_seq = row_seq;
+  p.row_len = row_len; p.out = out; p.part_out = part_out; p.part_lse = part_lse; p.rows = rows; p.H = H; p.dim = dim;
+  p.rot = rot; p.rank = rank; p.row_width = row_width; p.max_blocks = max_blocks; p.block_size = block_size;
+  p.window = window; p.splits = splits; p.scale = scale;
+  cudaStream_t st = ST(stream);
+  if (latent_mma_fits(rank, row_width, fp32)) {
+    const int tiles = (max_keys + LD_KT - 1) / LD_KT;
+    p.chunk = (tiles + splits - 1) / splits * LD_KT;
+    const size_t sm = latent_smem_bytes(row_width);
+    const dim3 grid(rows, (H + 15) / 16, splits);
+    const int np = (rank + 127) / 128;
+#define TS_LATENT(N)                                                                                             \
+  {                                                                                                              \
+    static bool configured = false;                                                                              \
+    if (!configured) {                                                                                           \
+      cudaError_t e = cudaFuncSetAttribute(latent_attend_mma_kernel<N>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+                                           227 * 1024);                                                          \
+      if (e != cudaSuccess) return (int)e;                                                                       \
+      configured = true;                                                                                         \
+    }                                                                                                            \
+    latent_attend_mma_kernel<N><<<grid, LD_WARPS * 32, sm, st>>>(p);                                             \
+  }
+    if (np == 1) TS_LATENT(1)
+    else if (np == 2) TS_LATENT(2)
+    else if (np == 3) TS_LATENT(3)
+    else TS_LATENT(4)
+#undef TS_LATENT
+  } else {
+    p.chunk = (max_keys + splits - 1) / splits;
+    const size_t sm = sizeof(float) * (rank + rot + p.chunk);
+    if (sm > 48 * 1024) return -12;
+    const dim3 grid(rows, H, splits);
+    if (fp32) latent_attend_simt_kernel<float><<<grid, 128, sm, st>>>(p);
+    else latent_attend_simt_kernel<__nv_bfloat16><<<grid, 128, sm, st>>>(p);
+  }
+  if (splits > 1) {
+    const dim3 grid(rows, H);
+    if (fp32) latent_merge_kernel<float><<<grid, 128, 0, st>>>(p);
+    else latent_merge_kernel<__nv_bfloat16><<<grid, 128, 0, st>>>(p);
+  }
+  return (int)cudaGetLastError();
+}

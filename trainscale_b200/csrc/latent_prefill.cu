@@ -1,0 +1,360 @@
+// Windowed causal attention for portions of prompts whose keys come from a latent cache (tcgen05 / TMEM / TMA).
+//
+// The latents a portion needs (its own tokens and the window before them) have been expanded to per-head keys and values
+// by one GEMM; the rotated key part is shared by all heads and read from the latent rows.  Scores are therefore a sum of
+// two products with operands of different origin:  S = Qn Kn^T (per head) + Qr Kr^T (shared),  O = softmax(S) V.
+//
+// Per CTA: one 256-row query block of one head of one sequence, as two 128-row tiles that ping-pong:
+//   warp 0       TMA loader: Q tiles once, then rings of 128-row key and value tiles.  Every operand is cut into
+//                64-column blocks (128-byte swizzle); 3-D maps (column, head, token) zero-fill columns past the head's
+//                size, so heads of any multiple of eight columns use the same code
+//   warp 1       MMA issuer: S_t = Q_t K^T over the unrotated, then the rotated columns; O_t += P_t V, P_t from TMEM
+//   warps 2..9   softmax: one thread per query row; scores, running max and sum in fp32
+// Key tiles outside every row's window are never loaded.  Queries are the LAST Lq of the sequence's Lk keys.
+#include "common.cuh"
+#include "host_common.h"
+
+namespace ts {
+
+constexpr int LP_THREADS = 320;
+constexpr int LP_BLOCK = 16384;          // 128 rows x 64 bf16 columns
+
+struct LatentPrefillParams {
+  const int* cu_q;                       // [sequences + 1] query rows
+  const int* cu_k;                       // [sequences + 1] key rows
+  int H;
+  int nb_n, nb_r, nb_v;                  // 64-column blocks of the unrotated part, the rotated part, the value
+  int ks_n, ks_r;                        // 16-column MMA steps
+  int vdim, v_cols;                      // value size; rounded up to 16
+  int k_stages, v_stages;
+  int window;
+  float scale_log2;
+  __nv_bfloat16* o;                      // [rows][o_stride], head h at column h * vdim
+  long long o_stride;
+};
+
+__global__ void __launch_bounds__(LP_THREADS, 1)
+latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_constant__ CUtensorMap tmQr,
+                      const __grid_constant__ CUtensorMap tmKn, const __grid_constant__ CUtensorMap tmKr,
+                      const __grid_constant__ CUtensorMap tmV, LatentPrefillParams p) {
+  constexpr uint32_t TMEM_COLS = 512;
+  constexpr uint32_t O_COL0 = 256;       // O_t at O_COL0 + 128 t
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  const int nb_k = p.nb_n + p.nb_r;
+  const int q_bytes = nb_k * LP_BLOCK, k_bytes = nb_k * LP_BLOCK, v_bytes = p.nb_v * LP_BLOCK;
+  uint8_t* k_base = smem + 2 * q_bytes;
+  uint8_t* v_base = k_base + p.k_stages * k_bytes;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(v_base + p.v_stages * v_bytes);
+  uint64_t* q_full = bars;          // [2]
+  uint64_t* k_full = bars + 2;      // [2]
+  uint64_t* k_empty = bars + 4;     // [2]
+  uint64_t* v_full = bars + 6;      // [2]
+  uint64_t* v_empty = bars + 8;     // [2]
+  uint64_t* s_full = bars + 10;     // [2]
+  uint64_t* p_full = bars + 12;     // [2]
+  uint64_t* o_full = bars + 14;     // [2]
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 16);
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int h = blockIdx.x % p.H, b = blockIdx.x / p.H;
+  const int q_start = p.cu_q[b], Lq = p.cu_q[b + 1] - q_start;
+  const int k_start = p.cu_k[b], Lk = p.cu_k[b + 1] - k_start;
+  const int n_qblocks = (Lq + 255) / 256;
+  if ((int)blockIdx.y >= n_qblocks) return;
+  const int qb = n_qblocks - 1 - blockIdx.y;
+  const int off = Lk - Lq;
+  int r0[2], nkv[2];
+  // key tiles entirely left of the first row's window are never loaded
+  const int kb_lo = max(0, qb * 256 + off - p.window + 1) / 128;
+#pragma unroll
+  for (int t = 0; t < 2; ++t) {
+    r0[t] = qb * 256 + t * 128;
+    nkv[t] = r0[t] >= Lq ? 0 : max(0, (min(Lk, r0[t] + 128 + off) + 127) / 128 - kb_lo);
+  }
+  const int n = max(nkv[0], nkv[1]);
+
+  if (threadIdx.x == 0) {
+    tma_prefetch_desc(&tmQn);
+    tma_prefetch_desc(&tmKn);
+    tma_prefetch_desc(&tmKr);
+    tma_prefetch_desc(&tmV);
+    for (int i = 0; i < 16; ++i) mbar_init(&bars[i], (i == 12 || i == 13) ? 4 : 1);
+    fence_barrier_init();
+  }
+  if (warp == 1) {
+    tmem_alloc(tmem_slot, TMEM_COLS);
+    tmem_relinquish();
+    tc_fence_before_sync();
+  }
+  __syncthreads();
+  tc_fence_after_sync();
+  const uint32_t tmem_base = *tmem_slot;
+  bool alive = true;
+
+  if (warp == 0) {
+    if (elect_one_sync()) {
+      for (int t = 0; t < 2; ++t) {
+        if (nkv[t] == 0) continue;
+        mbar_expect_tx(&q_full[t], q_bytes);
+        for (int j = 0; j < p.nb_n; ++j)
+          tma_load_3d(smem + t * q_bytes + j * LP_BLOCK, &tmQn, &q_full[t], j * 64, h, q_start + r0[t]);
+        for (int j = 0; j < p.nb_r; ++j)
+          tma_load_3d(smem + t * q_bytes + (p.nb_n + j) * LP_BLOCK, &tmQr, &q_full[t], j * 64, h, q_start + r0[t]);
+      }
+      uint32_t ki = 0, vi = 0;
+      for (int i = 0; i < n && alive; ++i, ++ki, ++vi) {
+        const int ks = ki % p.k_stages, vs = vi % p.v_stages, row = k_start + (kb_lo + i) * 128;
+        if (!mbar_wait(&k_empty[ks], ((ki / p.k_stages) & 1u) ^ 1u, alive, 400)) break;
+        mbar_expect_tx(&k_full[ks], k_bytes);
+        for (int j = 0; j < p.nb_n; ++j)
+          tma_load_3d(k_base + ks * k_bytes + j * LP_BLOCK, &tmKn, &k_full[ks], j * 64, h, row);
+        for (int j = 0; j < p.nb_r; ++j)
+          tma_load_2d(k_base + ks * k_bytes + (p.nb_n + j) * LP_BLOCK, &tmKr, &k_full[ks], j * 64, row);
+        if (!mbar_wait(&v_empty[vs], ((vi / p.v_stages) & 1u) ^ 1u, alive, 401)) break;
+        mbar_expect_tx(&v_full[vs], v_bytes);
+        for (int j = 0; j < p.nb_v; ++j)
+          tma_load_3d(v_base + vs * v_bytes + j * LP_BLOCK, &tmV, &v_full[vs], j * 64, h, row);
+      }
+    }
+  } else if (warp == 1) {
+    if (elect_one_sync()) {
+      const uint32_t idesc_s = make_idesc(128, 128, 1, 1, 0, 0);
+      const uint32_t idesc_o = make_idesc(128, p.v_cols, 1, 1, 0, 1);
+      auto issue_s = [&](int t, int stage) {
+        const uint32_t qa = smem_u32(smem + t * q_bytes), ka = smem_u32(k_base + stage * k_bytes);
+        for (int k = 0; k < p.ks_n; ++k) {
+          const uint32_t o = (k >> 2) * LP_BLOCK + (k & 3) * 32;
+          umma_f16_ss(tmem_base + t * 128, make_smem_desc_sw128(qa + o, 16, 1024),
+                      make_smem_desc_sw128(ka + o, 16, 1024), idesc_s, k != 0);
+        }
+        for (int k = 0; k < p.ks_r; ++k) {
+          const uint32_t o = (p.nb_n + (k >> 2)) * LP_BLOCK + (k & 3) * 32;
+          umma_f16_ss(tmem_base + t * 128, make_smem_desc_sw128(qa + o, 16, 1024),
+                      make_smem_desc_sw128(ka + o, 16, 1024), idesc_s, 1u);
+        }
+        umma_commit(&s_full[t]);
+      };
+      for (int t = 0; t < 2; ++t)
+        if (nkv[t] > 0) mbar_wait(&q_full[t], 0, alive, 500);
+      if (n > 0 && mbar_wait(&k_full[0], 0, alive, 501)) {
+        tc_fence_after_sync();
+        for (int t = 0; t < 2; ++t)
+          if (nkv[t] > 0) issue_s(t, 0);
+        umma_commit(&k_empty[0]);
+      }
+      for (int i = 0; i < n && alive; ++i) {
+        const int vs = i % p.v_stages, kn = (i + 1) % p.k_stages;
+        if (!mbar_wait(&v_full[vs], (i / p.v_stages) & 1u, alive, 502)) break;
+        bool k_waited = false;
+        for (int t = 0; t < 2 && alive; ++t) {
+          if (i < nkv[t]) {
+            if (!mbar_wait(&p_full[t], i & 1u, alive, 503)) break;
+            tc_fence_after_sync();
+            const uint32_t va = smem_u32(v_base + vs * v_bytes);
+#pragma unroll
+            for (int kk = 0; kk < 8; ++kk)
+              umma_f16_ts(tmem_base + O_COL0 + t * 128, tmem_base + t * 128 + kk * 8,
+                          make_smem_desc_sw128(va + kk * 2048, LP_BLOCK, 1024), idesc_o, (i | kk) != 0);
+            if (i == nkv[t] - 1) umma_commit(&o_full[t]);
+          }
+          if (i + 1 < nkv[t]) {
+            if (!k_waited) {
+              if (!mbar_wait(&k_full[kn], ((i + 1) / p.k_stages) & 1u, alive, 504)) break;
+              tc_fence_after_sync();
+              k_waited = true;
+            }
+            issue_s(t, kn);
+          }
+        }
+        if (!alive) break;
+        if (i + 1 < n) umma_commit(&k_empty[kn]);
+        umma_commit(&v_empty[vs]);
+      }
+    }
+  } else {
+    const int t = (warp - 2) >> 2;
+    const int q4 = warp & 3;
+    const int r = q4 * 32 + lane;
+    const int row = r0[t] + r;
+    const uint32_t t_lane = tmem_base + (static_cast<uint32_t>(q4 * 32) << 16);
+    const uint32_t t_s = t_lane + t * 128;
+    const uint32_t t_o = t_lane + O_COL0 + t * 128;
+    float m_used = -INFINITY, l = 0.f;
+    const int nt = nkv[t];
+    const float sc = p.scale_log2;
+    for (int i = 0; i < nt && alive; ++i) {
+      if (!mbar_wait(&s_full[t], i & 1u, alive, 600)) break;
+      tc_fence_after_sync();
+      const int c0 = (kb_lo + i) * 128;
+      const bool need_mask = (c0 + 127 > r0[t] + off) || (c0 + 128 > Lk) || (c0 <= r0[t] + 127 + off - p.window);
+      const int limit = min(Lk - 1, row + off);        // last visible key
+      const int lo = row + off - p.window + 1;         // first visible key
+      uint32_t v[128];
+#pragma unroll
+      for (int c = 0; c < 4; ++c) tmem_ld_32x32b_x32(t_s + c * 32, v + c * 32);
+      tc_wait_ld();
+      if (need_mask) {
+#pragma unroll
+        for (int j = 0; j < 128; ++j)
+          if (c0 + j > limit || c0 + j < lo) v[j] = 0xff800000u;
+      }
+      float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
+#pragma unroll
+      for (int j = 0; j < 128; j += 4) {
+        mx0 = fmaxf(mx0, __uint_as_float(v[j]));
+        mx1 = fmaxf(mx1, __uint_as_float(v[j + 1]));
+        mx2 = fmaxf(mx2, __uint_as_float(v[j + 2]));
+        mx3 = fmaxf(mx3, __uint_as_float(v[j + 3]));
+      }
+      const float mx = fmaxf(fmaxf(mx0, mx1), fmaxf(mx2, mx3));
+      const float m_new = fmaxf(m_used, mx * sc);
+      const bool grow = (m_new - m_used > 8.0f);       // also true on the first tile with a visible key
+      if (__any_sync(0xffffffffu, grow)) {
+        const float alpha = (m_used == -INFINITY) ? 0.f : fast_ex2(m_used - m_new);
+        m_used = m_new;
+        l *= alpha;
+        if (i > 0) {
+#pragma unroll 1
+          for (int c = 0; c < p.v_cols / 16; ++c) {
+            uint32_t o[16];
+            tmem_ld_32x32b_x16(t_o + c * 16, o);
+            tc_wait_ld();
+#pragma unroll
+            for (int j = 0; j < 16; ++j) o[j] = __float_as_uint(__uint_as_float(o[j]) * alpha);
+            tmem_st_32x32b_x16(t_o + c * 16, o);
+          }
+        }
+      }
+      const float m_sub = (m_used == -INFINITY) ? 0.f : m_used;
+      float l0 = 0.f, l1 = 0.f;
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        uint32_t pk[16];
+#pragma unroll
+        for (int j = 0; j < 32; j += 2) {
+          const float p0 = fast_ex2(fmaf(__uint_as_float(v[c * 32 + j]), sc, -m_sub));
+          const float p1 = fast_ex2(fmaf(__uint_as_float(v[c * 32 + j + 1]), sc, -m_sub));
+          l0 += p0;
+          l1 += p1;
+          pk[j >> 1] = pack_bf16x2(p0, p1);
+        }
+        tmem_st_32x32b_x16(t_s + c * 16, pk);
+      }
+      l += l0 + l1;
+      tc_wait_st();
+      tc_fence_before_sync();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&p_full[t]);
+    }
+    if (nt > 0 && alive && mbar_wait(&o_full[t], 0, alive, 601)) {
+      tc_fence_after_sync();
+      const float inv = l > 0.f ? 1.f / l : 0.f;
+      const bool valid = row < Lq;
+      __nv_bfloat16* dst = p.o + (q_start + row) * p.o_stride + h * p.vdim;
+#pragma unroll 1
+      for (int c = 0; c < p.v_cols / 16; ++c) {
+        uint32_t v[16];
+        tmem_ld_32x32b_x16(t_o + c * 16, v);
+        tc_wait_ld();
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          if (valid && c * 16 + j * 8 < p.vdim) {
+            uint4 o4;
+            o4.x = pack_bf16x2(__uint_as_float(v[8 * j]) * inv, __uint_as_float(v[8 * j + 1]) * inv);
+            o4.y = pack_bf16x2(__uint_as_float(v[8 * j + 2]) * inv, __uint_as_float(v[8 * j + 3]) * inv);
+            o4.z = pack_bf16x2(__uint_as_float(v[8 * j + 4]) * inv, __uint_as_float(v[8 * j + 5]) * inv);
+            o4.w = pack_bf16x2(__uint_as_float(v[8 * j + 6]) * inv, __uint_as_float(v[8 * j + 7]) * inv);
+            *reinterpret_cast<uint4*>(dst + c * 16 + j * 8) = o4;
+          }
+        }
+      }
+    }
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after_sync();
+    tmem_dealloc(tmem_base, TMEM_COLS);
+  }
+}
+
+struct LatentPrefillPlan {
+  int nb_n, nb_r, nb_v, k_stages, v_stages;
+  size_t smem;
+};
+
+static bool plan_prefill(int dim, int rot, int vdim, LatentPrefillPlan& pl) {
+  if (dim <= 0 || rot < 0 || vdim <= 0 || dim % 8 || rot % 8 || vdim % 8 || vdim > 128) return false;
+  pl.nb_n = (dim + 63) / 64;
+  pl.nb_r = (rot + 63) / 64;
+  pl.nb_v = (vdim + 63) / 64;
+  const size_t limit = 227 * 1024, fixed = 256 + 1024;
+  const int nb_k = pl.nb_n + pl.nb_r;
+  const int order[3][2] = {{2, 2}, {2, 1}, {1, 1}};
+  for (auto& o : order) {
+    pl.smem = static_cast<size_t>(2 * nb_k + o[0] * nb_k + o[1] * pl.nb_v) * LP_BLOCK + fixed;
+    if (pl.smem <= limit) {
+      pl.k_stages = o[0];
+      pl.v_stages = o[1];
+      return true;
+    }
+  }
+  return false;
+}
+
+}  // namespace ts
+
+TS_DEFINE_ERROR_API(ts_latent_prefill)
+using namespace ts;
+
+// 1 when the head sizes fit this kernel (multiples of eight, values up to 128 wide, tiles within shared memory).
+extern "C" int ts_latent_prefill_supported(int dim, int rot, int vdim) {
+  LatentPrefillPlan pl;
+  return plan_prefill(dim, rot, vdim, pl) ? 1 : 0;
+}
+
+// q: projection rows [q_rows][q_ld], head h at column h * (dim + rot).  kv: expanded rows [k_rows][kv_ld], unrotated key
+// of head h at column h * dim, value at column v_col0 + h * vdim.  k_rot: [k_rows][kr_ld] shared rotated key part.
+// cu_q / cu_k: [sequences + 1].  out: [q_rows][o_stride].
+extern "C" int ts_latent_prefill(const void* q, long long q_ld, long long q_rows, const void* kv, long long kv_ld,
+                                 int v_col0, const void* k_rot, long long kr_ld, long long k_rows, const int* cu_q,
+                                 const int* cu_k, int sequences, int max_q, int H, int dim, int rot, int vdim, int window,
+                                 float scale, void* out, long long o_stride, void* stream) {
+  if (sequences <= 0 || max_q <= 0) return 0;
+  LatentPrefillPlan pl;
+  if (H <= 0 || window <= 0 || !(scale > 0.f) || !plan_prefill(dim, rot, vdim, pl)) return -10;
+  if (q_ld % 8 || kv_ld % 8 || kr_ld % 8 || o_stride % 8 || (reinterpret_cast<uintptr_t>(out) & 15u)) return -11;
+  const __nv_bfloat16* qp = reinterpret_cast<const __nv_bfloat16*>(q);
+  const __nv_bfloat16* kvp = reinterpret_cast<const __nv_bfloat16*>(kv);
+  CUtensorMap tQn, tQr, tKn, tKr, tV;
+  const CUtensorMapDataType dt = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
+  int rc = make_tmap_3d(&tQn, qp, dt, 2, dim, H, q_rows, dim + rot, q_ld, 64, 1, 128);
+  if (rc) return rc * 100 - 1;
+  rc = make_tmap_3d(&tKn, kvp, dt, 2, dim, H, k_rows, dim, kv_ld, 64, 1, 128);
+  if (rc) return rc * 100 - 2;
+  rc = make_tmap_3d(&tV, kvp + v_col0, dt, 2, vdim, H, k_rows, vdim, kv_ld, 64, 1, 128);
+  if (rc) return rc * 100 - 3;
+  tQr = tQn;
+  tKr = tKn;
+  if (rot > 0) {
+    rc = make_tmap_3d(&tQr, qp + dim, dt, 2, rot, H, q_rows, dim + rot, q_ld, 64, 1, 128);
+    if (rc) return rc * 100 - 4;
+    rc = make_tmap_2d(&tKr, k_rot, dt, 2, k_rows, rot, kr_ld, 128, 64);
+    if (rc) return rc * 100 - 5;
+  }
+  LatentPrefillParams p;
+  p.cu_q = cu_q; p.cu_k = cu_k; p.H = H; p.nb_n = pl.nb_n; p.nb_r = pl.nb_r; p.nb_v = pl.nb_v;
+  p.ks_n = (dim + 15) / 16; p.ks_r = (rot + 15) / 16; p.vdim = vdim; p.v_cols = (vdim + 15) / 16 * 16;
+  p.k_stages = pl.k_stages; p.v_stages = pl.v_stages; p.window = window; p.scale_log2 = scale * 1.4426950408889634f;
+  p.o = reinterpret_cast<__nv_bfloat16*>(out); p.o_stride = o_stride;
+  static bool configured = false;
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(latent_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+    if (e != cudaSuccess) return (int)e;
+    configured = true;
+  }
+  const dim3 grid((unsigned)(H * sequences), (unsigned)((max_q + 255) / 256));
+  latent_prefill_kernel<<<grid, LP_THREADS, pl.smem, reinterpret_cast<cudaStream_t>(stream)>>>(tQn, tQr, tKn, tKr, tV, p);
+  return (int)cudaGetLastError();
+}

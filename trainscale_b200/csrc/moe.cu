@@ -152,69 +152,127 @@ __global__ void moe_combine_dw_kernel(const __nv_bfloat16* __restrict__ dout, co
   }
 }
 
-// Router: softmax over E experts and top-k selection, one warp per token (E <= 1024).  probs [T][E] fp32 is written for
-// the auxiliary losses and the backward; weights are the selected probabilities, optionally renormalised to sum to 1.
-// Ties resolve to the lower expert index, as torch.topk does on equal values in practice for distinct logits.
+// Router: softmax over E experts and top-k selection, one warp per token (E <= 1024).  probs [E] fp32 (may be null) is
+// written for the auxiliary losses and the backward; weights are the selected probabilities, optionally renormalised to
+// sum to 1.  Ties resolve to the lower expert index, as torch.topk does on equal values in practice for distinct logits.
 constexpr int ROUTER_MAX_PER_LANE = 32;
+__device__ __forceinline__ void warp_topk_softmax(const float* __restrict__ logits, float* probs, float* weights, int* idx,
+                                                  int E, int k, int normalize) {
+  const int lane = threadIdx.x & 31;
+  const int per = (E + 31) / 32;
+  float v[ROUTER_MAX_PER_LANE];
+  float mx = -INFINITY;
+#pragma unroll 4
+  for (int j = 0; j < per; ++j) {
+    const int e = lane + j * 32;
+    v[j] = e < E ? logits[e] : -INFINITY;
+    mx = fmaxf(mx, v[j]);
+  }
+  mx = warp_max(mx);
+  float sum = 0.f;
+#pragma unroll 4
+  for (int j = 0; j < per; ++j) {
+    v[j] = (lane + j * 32 < E) ? expf(v[j] - mx) : 0.f;
+    sum += v[j];
+  }
+  sum = warp_sum(sum);
+  const float inv = 1.f / sum;
+#pragma unroll 4
+  for (int j = 0; j < per; ++j) {
+    v[j] *= inv;
+    const int e = lane + j * 32;
+    if (probs && e < E) probs[e] = v[j];
+  }
+  float wsum = 0.f;
+  for (int s = 0; s < k; ++s) {
+    // arg-max over what is left: (value, lowest index) reduced across the warp
+    float best = -1.f;
+    int best_e = 0x7fffffff;
+#pragma unroll 4
+    for (int j = 0; j < per; ++j) {
+      const int e = lane + j * 32;
+      if (e < E && v[j] > best) {
+        best = v[j];
+        best_e = e;
+      }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oe = __shfl_xor_sync(0xffffffffu, best_e, o);
+      if (ob > best || (ob == best && oe < best_e)) {
+        best = ob;
+        best_e = oe;
+      }
+    }
+    if (lane == 0) {
+      weights[s] = best;
+      idx[s] = best_e;
+    }
+    wsum += best;
+    if ((best_e & 31) == lane) v[best_e >> 5] = -1.f;   // taken
+  }
+  __syncwarp();
+  if (normalize && lane < k) weights[lane] /= fmaxf(wsum, 1e-9f);
+}
+
 __global__ void __launch_bounds__(128) moe_topk_softmax_kernel(const float* __restrict__ logits, float* __restrict__ probs,
                                                               float* __restrict__ weights, int* __restrict__ idx, int T,
                                                               int E, int k, int normalize) {
-  const int lane = threadIdx.x & 31;
-  const int per = (E + 31) / 32;
-  for (int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5); t < T; t += gridDim.x * (blockDim.x >> 5)) {
-    float v[ROUTER_MAX_PER_LANE];
-    float mx = -INFINITY;
-#pragma unroll 4
-    for (int j = 0; j < per; ++j) {
-      const int e = lane + j * 32;
-      v[j] = e < E ? logits[static_cast<size_t>(t) * E + e] : -INFINITY;
-      mx = fmaxf(mx, v[j]);
-    }
-    mx = warp_max(mx);
-    float sum = 0.f;
-#pragma unroll 4
-    for (int j = 0; j < per; ++j) {
-      v[j] = (lane + j * 32 < E) ? __expf(v[j] - mx) : 0.f;
-      sum += v[j];
-    }
-    sum = warp_sum(sum);
-    const float inv = 1.f / sum;
-#pragma unroll 4
-    for (int j = 0; j < per; ++j) {
-      v[j] *= inv;
-      const int e = lane + j * 32;
-      if (e < E) probs[static_cast<size_t>(t) * E + e] = v[j];
-    }
-    float wsum = 0.f;
-    for (int s = 0; s < k; ++s) {
-      // arg-max over what is left: (value, lowest index) reduced across the warp
-      float best = -1.f;
-      int best_e = 0x7fffffff;
-#pragma unroll 4
-      for (int j = 0; j < per; ++j) {
-        const int e = lane + j * 32;
-        if (e < E && v[j] > best) {
-          best = v[j];
-          best_e = e;
-        }
-      }
+  for (int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5); t < T; t += gridDim.x * (blockDim.x >> 5))
+    warp_topk_softmax(logits + static_cast<size_t>(t) * E, probs ? probs + static_cast<size_t>(t) * E : nullptr,
+                      weights + static_cast<size_t>(t) * k, idx + static_cast<size_t>(t) * k, E, k, normalize);
+}
+
+// Router of a decode batch in one launch (one CTA): softmax, top-k and the expert-sorted slot list.
+//   order [T * k]: slots sorted by expert, stable;  start / count [E]: every expert's run inside `order`
+constexpr int ROUTE_THREADS = 1024;
+constexpr int ROUTE_MAX_SLOTS = 2048;
+__global__ void __launch_bounds__(ROUTE_THREADS) moe_route_kernel(const float* __restrict__ logits,
+                                                                  float* __restrict__ weights, int* __restrict__ order,
+                                                                  int* __restrict__ start, int* __restrict__ count, int T,
+                                                                  int E, int k, int normalize) {
+  __shared__ int ids[ROUTE_MAX_SLOTS];
+  __shared__ int first[1024 + 1];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = ROUTE_THREADS / 32;
+  const int n = T * k;
+  for (int t = warp; t < T; t += nw)
+    warp_topk_softmax(logits + static_cast<size_t>(t) * E, nullptr, weights + static_cast<size_t>(t) * k, ids + t * k, E, k,
+                      normalize);
+  __syncthreads();
+  for (int e = warp; e < E; e += nw) {
+    int c = 0;
+    for (int b = 0; b < n; b += 32) c += __popc(__ballot_sync(0xffffffffu, b + lane < n && ids[b + lane] == e));
+    if (lane == 0) first[e] = c;
+  }
+  __syncthreads();
+  if (warp == 0) {   // exclusive scan of the counts
+    int base = 0;
+    for (int b = 0; b < E; b += 32) {
+      const int c = b + lane < E ? first[b + lane] : 0;
+      int inc = c;
 #pragma unroll
-      for (int o = 16; o > 0; o >>= 1) {
-        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-        const int oe = __shfl_xor_sync(0xffffffffu, best_e, o);
-        if (ob > best || (ob == best && oe < best_e)) {
-          best = ob;
-          best_e = oe;
-        }
+      for (int o = 1; o < 32; o <<= 1) {
+        const int up = __shfl_up_sync(0xffffffffu, inc, o);
+        if (lane >= o) inc += up;
       }
-      if (lane == 0) {
-        weights[static_cast<size_t>(t) * k + s] = best;
-        idx[static_cast<size_t>(t) * k + s] = best_e;
+      if (b + lane < E) {
+        start[b + lane] = base + inc - c;
+        count[b + lane] = c;
+        first[b + lane] = base + inc - c;
       }
-      wsum += best;
-      if ((best_e & 31) == lane) v[best_e >> 5] = -1.f;   // taken
+      base += __shfl_sync(0xffffffffu, inc, 31);
     }
-    if (normalize && lane < k) weights[static_cast<size_t>(t) * k + lane] /= fmaxf(wsum, 1e-9f);
+  }
+  __syncthreads();
+  for (int e = warp; e < E; e += nw) {
+    int at = first[e];
+    for (int b = 0; b < n; b += 32) {
+      const bool hit = b + lane < n && ids[b + lane] == e;
+      const unsigned m = __ballot_sync(0xffffffffu, hit);
+      if (hit) order[at + __popc(m & ((1u << lane) - 1u))] = b + lane;
+      at += __popc(m);
+    }
   }
 }
 
@@ -278,5 +336,14 @@ extern "C" int ts_moe_topk_softmax(const float* logits, float* probs, float* wei
   const long long cap = static_cast<long long>(sm_count()) * 16;
   if (blocks > cap) blocks = cap;
   moe_topk_softmax_kernel<<<(unsigned)blocks, 128, 0, ST(stream)>>>(logits, probs, weights, idx, T, E, k, normalize);
+  return (int)cudaGetLastError();
+}
+
+// Decode-sized router: logits fp32 [T][E] -> weights [T][k], order [T * k], start [E], count [E].
+extern "C" int ts_moe_route_max_slots() { return ROUTE_MAX_SLOTS; }
+extern "C" int ts_moe_route(const float* logits, float* weights, int* order, int* start, int* count, int T, int E, int k,
+                            int normalize, void* stream) {
+  if (T <= 0 || E <= 0 || E > 32 * ROUTER_MAX_PER_LANE || k <= 0 || k > 32 || k > E || T * k > ROUTE_MAX_SLOTS) return -10;
+  moe_route_kernel<<<1, ROUTE_THREADS, 0, ST(stream)>>>(logits, weights, order, start, count, T, E, k, normalize);
   return (int)cudaGetLastError();
 }

@@ -243,13 +243,11 @@ class ModelDeserializer:
 
 
 def load_pretrained(path: str | os.PathLike, dtype=torch.bfloat16, device=None):
-    """Build the framework decoder from a local HF-format directory (config.json + safetensors)."""
-    from ..models.llama import LlamaConfig, build_model
+    """Build a framework model from a local directory (config.json + safetensors); config.json says which class."""
+    from ..models import architecture_of
     p = Path(path)
-    cfg = LlamaConfig.from_dict(json.loads((p / "config.json").read_text()))
-    model = build_model(cfg, dtype=dtype, device=device)
-    model.load_hf_state_dict(ModelDeserializer().load(p), strict=True)
-    return model
+    raw = json.loads((p / "config.json").read_text())
+    return architecture_of(raw).load(raw, ModelDeserializer().load(p), dtype, device)
 
 
 def generate_model_card(model_name, base_model: str = "", config: dict | None = None, metrics: dict | None = None,

@@ -6,8 +6,9 @@ speculative / LoRA / observability sub-configs, `GenerationParams`, `RequestMetr
 `MetricsAggregator`, `EngineBuilder`, `SOTAInferenceEngine.generate`, `SOTAAsyncStreamEngine.generate_stream /
 abort_request`, `EnginePresets`, `create_openai_server` with /v1/completions, /v1/chat/completions, /health,
 /metrics, CLI sub-commands probe | batch | stream | serve | bench).  The reference wraps vLLM; this engine runs
-the framework's own decoder on its own kernels: flash attention with packed prompts (cu_seqlens) for prefill,
-paged split-KV decode attention, tcgen05 GEMMs, fused norms.
+the framework's own decoders on its own kernels: flash attention with packed prompts (cu_seqlens) for prefill,
+paged split-KV decode attention, tcgen05 GEMMs, fused norms.  A model class that defines `serve` and `cache_spec` (latent
+caches, state per sequence, its own layers) is batched, scheduled and sampled by the same code.
 """
 from __future__ import annotations
 
@@ -28,7 +29,8 @@ from ..utils.refargs import ANY, reference_kwargs
 
 from ..core.types import Err, Ok, Result
 from ..ops import _lib, activation, attention, gemm, norm, rope
-from .kv_cache import PagedKVCache
+from .batch import HostBatch, StepBatch, StepEntry
+from .kv_cache import CacheSpec, PagedKVCache
 from .sampling import apply_penalties, sample
 
 
@@ -249,7 +251,8 @@ class StreamChunk:
 
 # ------------------------------------------------------------------------------------------------ model runner
 class ModelRunner:
-    """Runs the framework decoder over a flattened token batch with a paged KV cache."""
+    """Runs a decoder over a flattened token batch with the paged cache.  A model that defines `serve(batch, cache)` brings
+    its own layers (models/mezilix.py); for `LlamaForCausalLM` they are here."""
 
     def __init__(self, model, cache: PagedKVCache, device, tp=None, use_graphs: bool = False):
         """`tp`: tensor-parallel context of a model sharded with `shard_model_for_tensor_parallel` (every rank runs
@@ -257,13 +260,17 @@ class ModelRunner:
         graph per (padded batch size, block-table width) instead of launching ~12 kernels per layer from Python."""
         self.model, self.cache, self.device = model.eval(), cache, torch.device(device)
         self.cfg = model.config
-        self.cuda = self.device.type == "cuda" and next(model.parameters()).dtype == torch.bfloat16
-        self.cos, self.sin = model.model.rope_tables(self.device, min(self.cfg.max_position_embeddings, 1 << 16))
+        self.own_layers = hasattr(model, "serve")
         self.lora = None                 # multi_lora.BatchedLoRA when adapters are loaded
         self.tp = tp if (tp is not None and tp.active) else None
-        ws = self.tp.size if self.tp is not None else 1
-        self.Hq, self.Hkv = self.cfg.num_attention_heads // ws, self.cfg.num_key_value_heads // ws
-        self.use_graphs = bool(use_graphs) and self.cuda
+        if self.own_layers:
+            self.use_graphs = bool(use_graphs) and self.device.type == "cuda"
+        else:
+            self.cuda = self.device.type == "cuda" and next(model.parameters()).dtype == torch.bfloat16
+            self.cos, self.sin = model.model.rope_tables(self.device, min(self.cfg.max_position_embeddings, 1 << 16))
+            ws = self.tp.size if self.tp is not None else 1
+            self.Hq, self.Hkv = self.cfg.num_attention_heads // ws, self.cfg.num_key_value_heads // ws
+            self.use_graphs = bool(use_graphs) and self.cuda
         self.graphs: dict = {}
         self.graph_replays = 0
 
@@ -304,9 +311,10 @@ class ModelRunner:
         v = self.cache.v[layer][idx].reshape(-1, self.Hkv, c.head_dim)[:s.num_tokens]
         return k, v
 
-    def _attend(self, layer: int, qkv2d: torch.Tensor, seq_ids: list[int], q_lens: list[int], fresh: bool,
-                block_table, seq_lens, splits: int | None = None) -> torch.Tensor:
+    def _attend(self, layer: int, qkv2d: torch.Tensor, batch: StepBatch) -> torch.Tensor:
         c = self.cfg
+        q_lens, fresh, splits = batch.q_lens, batch.fresh, batch.splits
+        block_table, seq_lens = batch.block_table, batch.seq_lens
         Hq, Hkv, D = self.Hq, self.Hkv, c.head_dim
         scale = 1.0 / math.sqrt(D)
         T = qkv2d.shape[0]
@@ -334,7 +342,7 @@ class ModelRunner:
             return out
         # general path (chunked prefill continuation, CPU): per sequence against the gathered cache
         outs, off = [], 0
-        for sid, n in zip(seq_ids, q_lens):
+        for sid, n in zip(batch.seq_ids, q_lens):
             q = qkv2d[off:off + n, :Hq * D].view(1, n, Hq, D)
             k, v = self._gathered_kv(layer, sid)
             o = attention.attention_reference(q, k.unsqueeze(0), v.unsqueeze(0), True, scale)
@@ -342,11 +350,13 @@ class ModelRunner:
             off += n
         return torch.cat(outs)
 
-    def _layers(self, token_ids, pos32, slots, seq_ids, q_lens, fresh, adapter_ids, block_table, seq_lens,
-                splits: int | None = None) -> torch.Tensor:
-        """The decoder over a flattened token batch; returns the final-norm hidden state of every token."""
+    def _layers(self, batch: StepBatch) -> torch.Tensor:
+        """The decoder over a flattened token batch; returns the final-norm hidden state of the wanted rows."""
+        if self.own_layers:
+            return self.model.serve(batch, self.cache)
+        pos32, adapter_ids = batch.positions, batch.adapter_ids
         m, c = self.model.model, self.cfg
-        x = m.embed_tokens(token_ids)
+        x = m.embed_tokens(batch.token_ids)
         if getattr(c, "scale_embeddings", False):
             x = x * torch.tensor(c.hidden_size ** 0.5, dtype=x.dtype)
         res = None
@@ -358,8 +368,8 @@ class ModelRunner:
                 qkv = qkv + attn.bqkv
             qkv = rope.apply_rope_qkv(qkv.unsqueeze(0), self.Hq + self.Hkv, c.head_dim, self.cos, self.sin,
                                       pos32.unsqueeze(0), qkv.shape[0], 0, c.rope_interleaved)[0]
-            self._write_cache(li, qkv, slots)
-            a = self._attend(li, qkv, seq_ids, q_lens, fresh, block_table, seq_lens, splits)
+            self._write_cache(li, qkv, batch.slots)
+            a = self._attend(li, qkv, batch)
             a = self._reduce(self._lin(li, "wo", attn.wo, a, adapter_ids))
             h, res = layer.post_attention_layernorm(a, res)
             if hasattr(mlp, "router"):            # mixture of experts: the block routes by itself
@@ -369,53 +379,53 @@ class ModelRunner:
                                            activation.glu(self._lin(li, "w_gate_up", mlp.w_gate_up, h, adapter_ids),
                                                           mlp.act), adapter_ids))
         x, _ = m.norm(x, res)
-        return x
+        return x[batch.out_rows]
 
     @torch.no_grad()
-    def forward(self, token_ids: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, seq_ids: list[int],
-                q_lens: list[int], fresh: bool, adapter_ids: torch.Tensor | None = None) -> torch.Tensor:
-        """token_ids / positions / slots: [T]; returns the hidden state of each sequence's LAST token [n_seq, H].
-        `adapter_ids` [T]: LoRA adapter index of every token (requests with different adapters share the batch)."""
-        block_table, seq_lens = self.cache.block_table(seq_ids, self.device)
-        x = self._layers(token_ids, positions.to(torch.int32), slots, seq_ids, q_lens, fresh, adapter_ids, block_table,
-                         seq_lens)
-        last = torch.tensor(q_lens, device=self.device).cumsum(0) - 1
-        return x[last]
+    def forward(self, batch: StepBatch) -> torch.Tensor:
+        """Hidden state of every wanted row [wanted, H]."""
+        return self._layers(batch)
 
     # ---------------------------------------------------------------- CUDA-graph decode
-    def can_graph(self, q_lens: list[int]) -> bool:
+    def can_graph(self, host: HostBatch) -> bool:
+        """Decode steps (one token per sequence, logits of every row) replay a captured graph."""
         c = self.cfg
-        return (self.use_graphs and self.lora is None and all(n == 1 for n in q_lens) and c.head_dim in (64, 128)
-                and getattr(c, "num_local_experts", 0) == 0 and len(q_lens) <= 256)
+        return (self.use_graphs and self.lora is None and host.all_single and len(host.q_lens) <= 256
+                and host.out_rows == list(range(len(host.q_lens)))
+                and (self.own_layers or (c.head_dim in (64, 128) and getattr(c, "num_local_experts", 0) == 0)))
+
+    # index tensors of a captured step: name -> (dtype, value of a padding row)
+    def _static_fields(self) -> dict:
+        bs, trash = self.cache.block_size, self.cache.trash_block
+        return {"token_ids": (torch.long, 0), "prev_tokens": (torch.int32, -1), "positions": (torch.int32, 0),
+                "slots": (torch.long, trash * bs), "seq_lens": (torch.int32, 1), "row_prev": (torch.int32, -1),
+                "row_next": (torch.int32, self.cache.trash_state if self.cache.spec.has_state else -1)}
 
     @torch.no_grad()
-    def decode_graphed(self, toks: list[int], pos: list[int], slots: list[int], seq_ids: list[int]) -> torch.Tensor:
+    def decode_graphed(self, host: HostBatch) -> torch.Tensor:
         """One decode step (one new token per sequence) replayed from a CUDA graph; returns fp32 logits [n, V].
         The batch is padded to a power of two with rows that write to / read from the cache's spare block."""
-        n = len(seq_ids)
+        n = len(host.seq_ids)
         n_pad = 1
         while n_pad < n:
             n_pad *= 2
-        bt, sl = self.cache.block_table(seq_ids, None)
+        bt, sl = self.cache.block_table(host.seq_ids, None)
         width = -(-bt.shape[1] // 32) * 32
         key = (n_pad, width)
         st = self.graphs.get(key)
         if st is None:
             st = self.graphs[key] = self._capture(n_pad, width)
-        bs, trash = self.cache.block_size, self.cache.trash_block
         h = st["host"]
-        h["tok"].zero_()
-        h["pos"].zero_()
-        h["slots"].fill_(trash * bs)
-        h["sl"].fill_(1)
-        h["bt"].fill_(trash)
-        h["tok"][:n] = torch.tensor(toks)
-        h["pos"][:n] = torch.tensor(pos, dtype=torch.int32)
-        h["slots"][:n] = torch.tensor(slots)
-        h["sl"][:n] = sl
-        h["bt"][:n, :bt.shape[1]] = bt
-        for k in ("tok", "pos", "slots", "sl", "bt"):
-            st[k].copy_(h[k], non_blocking=True)
+        for name, (dtype, pad) in self._static_fields().items():
+            h[name].fill_(pad)
+        h["block_table"].fill_(self.cache.trash_block)
+        for name, values in (("token_ids", host.tok), ("prev_tokens", host.prev), ("positions", host.pos),
+                             ("slots", host.slots), ("row_prev", host.row_prev), ("row_next", host.row_next)):
+            h[name][:n] = torch.tensor(values, dtype=h[name].dtype)
+        h["seq_lens"][:n] = sl
+        h["block_table"][:n, :bt.shape[1]] = bt
+        for name, buf in h.items():
+            getattr(st["batch"], name).copy_(buf, non_blocking=True)
         st["graph"].replay()
         self.graph_replays += 1
         return st["logits"][:n]
@@ -423,18 +433,15 @@ class ModelRunner:
     def _capture(self, n_pad: int, width: int) -> dict:
         dev = self.device
         bs, trash = self.cache.block_size, self.cache.trash_block
-        st = {"tok": torch.zeros(n_pad, dtype=torch.long, device=dev),
-              "pos": torch.zeros(n_pad, dtype=torch.int32, device=dev),
-              "slots": torch.full((n_pad,), trash * bs, dtype=torch.long, device=dev),
-              "sl": torch.ones(n_pad, dtype=torch.int32, device=dev),
-              "bt": torch.full((n_pad, width), trash, dtype=torch.int32, device=dev)}
-        st["host"] = {k: torch.empty_like(v, device="cpu").pin_memory() for k, v in st.items()}
-        splits = max(1, -(-(width * bs) // 512))
-        ids = list(range(n_pad))
+        buf = {k: torch.full((n_pad,), pad, dtype=dt, device=dev) for k, (dt, pad) in self._static_fields().items()}
+        buf["block_table"] = torch.full((n_pad, width), trash, dtype=torch.int32, device=dev)
+        rows = torch.arange(n_pad, dtype=torch.int32, device=dev)
+        batch = StepBatch(None, row_seq=rows, out_rows=rows, n_single=n_pad, max_len=width * bs, fresh=False,
+                          splits=max(1, -(-(width * bs) // 512)), **buf)
+        st = {"batch": batch, "host": {k: torch.empty_like(v, device="cpu").pin_memory() for k, v in buf.items()}}
 
         def body():
-            x = self._layers(st["tok"], st["pos"], st["slots"], ids, [1] * n_pad, False, None, st["bt"], st["sl"], splits)
-            return self.model.logits(x).float()
+            return self.model.logits(self._layers(batch)).float()
 
         side = torch.cuda.Stream(device=dev)
         side.wait_stream(torch.cuda.current_stream())
@@ -465,10 +472,16 @@ class _Request:
     output_ids: list[int] = field(default_factory=list)
     logprobs: list[float] = field(default_factory=list)
     prefilled: int = 0
+    context_ids: list[int] | None = None     # after a preemption: prompt and output so far, to be prefilled again
     generator: torch.Generator | None = None
     finished: bool = False
     finish_reason: str | None = None
     emitted_text_len: int = 0
+
+    @property
+    def prefill_ids(self) -> list[int]:
+        """Tokens that have to be in the cache before the next one can be sampled."""
+        return self.prompt_ids if self.context_ids is None else self.context_ids
 
 
 class EngineCore:
@@ -477,7 +490,7 @@ class EngineCore:
 
     def __init__(self, config: EngineConfig, model=None, tokenizer=None):
         from ..data.tokenization import TokenizerWrapper, create_tokenizer
-        from ..models.llama import PRESETS, build_model
+        from ..models import build_preset, is_preset
         self.config = config
         self.adapter_states: dict[str, dict[str, torch.Tensor]] = {}   # registry behind `load_adapters`
         dev = config.device
@@ -488,8 +501,8 @@ class EngineCore:
         if self.device.type == "cpu":
             dtype = torch.float32
         if model is None:
-            if config.model in PRESETS:
-                model = build_model(config.model, dtype=dtype, device=self.device, seed=config.seed)
+            if is_preset(config.model):
+                model = build_preset(config.model, dtype=dtype, device=self.device, seed=config.seed)
             else:
                 from ..hub import load_pretrained
                 model = load_pretrained(config.model, dtype=dtype, device=self.device)
@@ -498,6 +511,8 @@ class EngineCore:
         # requests with its slice of every projection; sampling uses the same seeds, so all ranks emit the same tokens
         self.tp = None
         tps = int(config.parallel.tensor_parallel_size or 1)
+        if tps > 1 and hasattr(self.model, "serve"):
+            raise ValueError(f"{type(self.model).__name__} is served on one GPU: tensor_parallel_size must be 1")
         if tps > 1:
             import torch.distributed as dist
             from ..parallel import tp as TP
@@ -509,23 +524,25 @@ class EngineCore:
                 TP.shard_model_for_tensor_parallel(self.model, ctx)
             self.tp = self.model.tp
         if tokenizer is None:
-            tokenizer = create_tokenizer(name_or_path=config.tokenizer or ("byte" if config.model in PRESETS else config.model),
-                                         padding=False, truncation=False)
+            tokenizer = create_tokenizer(name_or_path=config.tokenizer or default_tokenizer(config.model), padding=False,
+                                         truncation=False)
         self.tokenizer = tokenizer if isinstance(tokenizer, TokenizerWrapper) else TokenizerWrapper(tokenizer, padding=False)
         c = self.model.config
         cc = config.cache
         nb = cc.num_gpu_blocks
+        spec = self.model.cache_spec() if hasattr(self.model, "cache_spec") else \
+            CacheSpec.kv(c.num_hidden_layers, c.num_key_value_heads // tps, c.head_dim)
         if nb is None:
-            per_block = 2 * c.num_hidden_layers * cc.block_size * (c.num_key_value_heads // tps) * c.head_dim * \
-                (2 if dtype != torch.float32 else 4)
+            per_block = cc.block_size * spec.bytes_per_token(2 if dtype != torch.float32 else 4)
             if self.device.type == "cuda":
                 free, _ = torch.cuda.mem_get_info(self.device)
                 nb = max(64, int(free * cc.gpu_memory_utilization * 0.5) // per_block)
             else:
                 nb = 512
             nb = min(nb, max(64, cc.max_model_len * config.scheduler.max_num_seqs // cc.block_size + 64))
-        self.cache = PagedKVCache(c.num_hidden_layers, nb, cc.block_size, c.num_key_value_heads // tps, c.head_dim, dtype,
-                                  self.device, cc.enable_prefix_caching)
+        self.cache = PagedKVCache(c.num_hidden_layers, nb, cc.block_size, dtype=dtype, device=self.device,
+                                  enable_prefix_caching=cc.enable_prefix_caching, spec=spec,
+                                  state_slots=config.scheduler.max_num_seqs)
         self.runner = ModelRunner(self.model, self.cache, self.device, tp=self.tp, use_graphs=not config.enforce_eager)
         self.waiting: deque[_Request] = deque()
         self.running: list[_Request] = []
@@ -545,6 +562,7 @@ class EngineCore:
         max_len = self.config.cache.max_model_len
         if len(ids) >= max_len:
             ids = ids[-(max_len - 1):]
+        self._check_tokens(ids)
         rid = request_id or f"req-{self._next_seq}"
         gen = None
         if params.seed is not None:
@@ -555,11 +573,18 @@ class EngineCore:
         self.waiting.append(r)
         return r
 
+    def _check_tokens(self, ids: list[int]) -> None:
+        vocab = self.model.config.vocab_size
+        if any(not 0 <= t < vocab for t in ids):
+            raise ValueError(f"token ids must lie in [0, {vocab})")
+
     def load_adapters(self, adapters: dict[str, dict[str, torch.Tensor]]) -> None:
         """Make named LoRA adapters available to requests (`GenerationParams.lora_name`).  The model must carry LoRA
         modules of matching shapes (`lora.get_peft_model`); requests that use different adapters, or none, are batched
         together (`multi_lora.BatchedLoRA`)."""
         from .multi_lora import BatchedLoRA
+        if self.runner.own_layers:
+            raise ValueError(f"LoRA adapters are not supported for {type(self.model).__name__}")
         limit = getattr(getattr(self.config, "lora", None), "max_loras", None)
         if limit and len(adapters) > limit:
             raise ValueError(f"{len(adapters)} adapters exceed lora.max_loras = {limit}")
@@ -593,89 +618,125 @@ class EngineCore:
             self.metrics.add(r.metrics)
 
     # -------------------------------------------------------------- one engine step
-    def step(self) -> list[tuple[_Request, int]]:
-        """Runs one forward over the scheduled tokens; returns (request, new token) for every request that sampled."""
+    @torch.no_grad()
+    def execute(self, entries: list[StepEntry]) -> torch.Tensor | None:
+        """Run the entries as ONE batch from what earlier steps left in the cache; fp32 logits of the wanted places, in the
+        order of the entries (None when nothing is wanted).  `step` is this plus scheduling and sampling."""
+        for e in entries:
+            if not e.tokens or any(not 0 <= w < len(e.tokens) for w in e.wanted):
+                raise ValueError("an entry needs tokens, and the wanted places lie among them")
+            self._check_tokens(e.tokens)
+        if len({e.seq_id for e in entries}) != len(entries):
+            raise ValueError("a sequence may appear once in a step")
+        need = sum(self.cache.blocks_needed(e.seq_id, len(e.tokens)) for e in entries)
+        if need > self.cache.alloc.num_free:
+            raise MemoryError(f"the step needs {need} cache blocks, {self.cache.alloc.num_free} are free")
+        host = HostBatch(self.cache, entries)
+        self.steps += 1
+        if self.runner.can_graph(host):
+            logits = self.runner.decode_graphed(host)
+        else:
+            hidden = self.runner.forward(host.to_device(self.device, self.runner.lora is not None))
+            if not host.out_rows:
+                return None
+            logits = self.runner.logits(hidden)
+        if host.out_entry != sorted(host.out_entry):
+            logits = logits[torch.tensor(sorted(range(len(host.out_entry)), key=lambda i: host.out_entry[i]),
+                                         device=self.device)]
+        return logits
+
+    def release(self, seq_id: int) -> None:
+        """Give back everything a sequence holds in the cache."""
+        self.cache.free_sequence(seq_id)
+
+    def _preempt(self, r: _Request) -> None:
+        """Out of blocks: drop what the request holds and compute it again later."""
+        self.running.remove(r)
+        self.release(r.seq_id)
+        r.prefilled = 0
+        r.context_ids = r.prompt_ids + r.output_ids
+        self.waiting.appendleft(r)
+
+    def _schedule(self) -> list[tuple[_Request, list[int]]]:
+        """(request, tokens fed this step) within the token budget and the free cache blocks: decode tokens of running
+        requests first, then (chunked) prefill."""
         sc = self.config.scheduler
-        budget = sc.max_num_batched_tokens
-        batch: list[tuple[_Request, list[int], int]] = []   # (request, tokens fed this step, start position)
-        # 1) decode tokens of running requests
+        budget, free = sc.max_num_batched_tokens, self.cache.alloc.num_free
+        batch: list[tuple[_Request, list[int]]] = []
+
+        def fits(r, n):
+            nonlocal free
+            need = self.cache.blocks_needed(r.seq_id, n)
+            if need > free:
+                return False
+            free -= need
+            return True
+
         for r in list(self.running):
             if budget <= 0:
                 break
-            if not self.cache.can_append(r.seq_id, 1):
-                # out of blocks: preempt the most recent request (recompute later)
-                self.running.remove(r)
-                self.cache.free_sequence(r.seq_id)
-                r.prefilled = 0
-                r.prompt_ids = r.prompt_ids + r.output_ids
-                self.waiting.appendleft(r)
+            if r.prefilled < len(r.prefill_ids):
                 continue
-            if r.prefilled < len(r.prompt_ids):
+            if not fits(r, 1):
+                self._preempt(r)
+                free = self.cache.alloc.num_free - sum(self.cache.blocks_needed(x.seq_id, len(t)) for x, t in batch)
                 continue
-            batch.append((r, [r.output_ids[-1]], len(r.prompt_ids) + len(r.output_ids) - 1))
+            batch.append((r, [r.output_ids[-1]]))
             budget -= 1
-        # 2) (chunked) prefill
-        candidates = [r for r in self.running if r.prefilled < len(r.prompt_ids)]
+        candidates = [r for r in self.running if r.prefilled < len(r.prefill_ids)]
         while self.waiting and len(self.running) < sc.max_num_seqs:
             r = self.waiting.popleft()
             if r.prefilled == 0:
-                covered = self.cache.match_prefix(r.seq_id, r.prompt_ids, self._salt(r))
+                covered = self.cache.match_prefix(r.seq_id, r.prefill_ids, self._salt(r))
                 r.prefilled = covered
                 r.metrics.cached_prompt_tokens = covered
             self.running.append(r)
             candidates.append(r)
+        free = self.cache.alloc.num_free - sum(self.cache.blocks_needed(x.seq_id, len(t)) for x, t in batch)
         for r in candidates:
             if budget <= 0:
                 break
-            remaining = len(r.prompt_ids) - r.prefilled
+            remaining = len(r.prefill_ids) - r.prefilled
             n = min(remaining, budget) if sc.enable_chunked_prefill else remaining
             if n <= 0 or (not sc.enable_chunked_prefill and n > budget and batch):
                 continue
-            if not self.cache.can_append(r.seq_id, n):
+            if not fits(r, n):
                 continue
-            batch.append((r, r.prompt_ids[r.prefilled:r.prefilled + n], r.prefilled))
+            batch.append((r, r.prefill_ids[r.prefilled:r.prefilled + n]))
             budget -= n
+        return batch
+
+    def step(self) -> list[tuple[_Request, int]]:
+        """Runs one forward over the scheduled tokens; returns (request, new token) for every request that sampled."""
+        batch = self._schedule()
+        while not batch and self.running:
+            # nothing fits: the most recent request gives its blocks to the others
+            if len(self.running) == 1 and not self.waiting:
+                raise MemoryError("the KV cache is too small for the request")
+            self._preempt(self.running[-1])
+            held = self.waiting.popleft()
+            batch = self._schedule() if self.running else []
+            self.waiting.appendleft(held)
+            if not self.running:
+                raise MemoryError("the KV cache is too small for the request")
         if not batch:
             return []
-        # 3) build the flattened inputs
-        toks, pos, slots, seq_ids, q_lens, ad = [], [], [], [], [], []
-        fresh = True
         lora = self.runner.lora
-        for r, feed, start in batch:
-            s = self.cache.append_slots(r.seq_id, len(feed))
-            toks += feed
-            if lora is not None:
-                ad += lora.ids_for([r.params.lora_name]) * len(feed)
-            pos += list(range(start, start + len(feed)))
-            slots += s
-            seq_ids.append(r.seq_id)
-            q_lens.append(len(feed))
-            fresh &= (start == 0)
-        dev = self.device
-        graphed = self.runner.can_graph(q_lens)
-        if graphed:
-            all_logits = self.runner.decode_graphed(toks, pos, slots, seq_ids)     # [n, V] of every decode row
-            hidden = None
-        else:
-            hidden = self.runner.forward(torch.tensor(toks, device=dev), torch.tensor(pos, device=dev),
-                                         torch.tensor(slots, device=dev, dtype=torch.long), seq_ids, q_lens, fresh,
-                                         torch.tensor(ad, device=dev) if lora is not None else None)
-        self.steps += 1
-        # 4) sample for every request whose prompt is now complete
-        sample_rows, sample_reqs = [], []
-        for i, (r, feed, start) in enumerate(batch):
-            if start + len(feed) >= len(r.prompt_ids):
-                if r.prefilled < len(r.prompt_ids):
-                    r.prefilled = len(r.prompt_ids)
-                    self.cache.register_full_blocks(r.seq_id, r.prompt_ids, self._salt(r))
-                sample_rows.append(i)
+        entries, sample_reqs = [], []
+        for r, feed in batch:
+            done = r.prefilled + len(feed) >= len(r.prefill_ids)         # decode steps are past it already
+            entries.append(StepEntry(r.seq_id, feed, None if done else [],
+                                     lora.ids_for([r.params.lora_name])[0] if lora is not None else 0))
+            if done:
                 sample_reqs.append(r)
-            else:
-                r.prefilled = start + len(feed)
+        logits = self.execute(entries)
+        for r, feed in batch:
+            if r.prefilled < len(r.prefill_ids):
+                r.prefilled += len(feed)
+                if r.prefilled >= len(r.prefill_ids):
+                    self.cache.register_full_blocks(r.seq_id, r.prefill_ids, self._salt(r))
         if not sample_reqs:
             return []
-        rows = torch.tensor(sample_rows, device=dev)
-        logits = all_logits[rows] if graphed else self.runner.logits(hidden[rows])
         ps = [r.params for r in sample_reqs]
         logits = apply_penalties(logits, [r.output_ids for r in sample_reqs], [p.repetition_penalty for p in ps],
                                  [p.presence_penalty for p in ps], [p.frequency_penalty for p in ps])
@@ -715,6 +776,16 @@ class EngineCore:
             if s in text:
                 text = text[:text.index(s)]
         return text
+
+
+def default_tokenizer(model: str) -> str:
+    """A preset, or a directory that holds weights but no tokenizer, is read and written as bytes."""
+    import os
+    from ..models import is_preset
+    names = ("tokenizer.json", "tokenizer.model", "tokenizer_config.json", "vocab.json", "vocab.txt")
+    if is_preset(model) or (os.path.isdir(model) and not any(os.path.exists(os.path.join(model, n)) for n in names)):
+        return "byte"
+    return model
 
 
 def _lora_request_parts(req) -> tuple[str, str | None]:
@@ -1172,6 +1243,7 @@ def run_hf_generate_baseline(model_cfg, num_prompts: int, input_len: int, output
 def main(argv: list[str] | None = None) -> int:
     ap = argparse.ArgumentParser(prog="python -m trainscale_b200.inference")
     sub = ap.add_subparsers(dest="cmd", required=True)
+    sub.add_parser("trace", help="replay a trace of token ids (bin/trace_run)", add_help=False)
     for name in ("probe", "batch", "stream", "serve", "bench"):
         p = sub.add_parser(name)
         p.add_argument("--model", default="tiny")
@@ -1190,6 +1262,10 @@ def main(argv: list[str] | None = None) -> int:
         p.add_argument("--tensor-parallel-size", type=int, default=1, help="launch under torchrun with this many ranks")
         p.add_argument("--eager", action="store_true", help="no CUDA graphs in the decode loop")
         p.add_argument("--max-num-seqs", type=int, default=64)
+    argv = sys.argv[1:] if argv is None else argv
+    if argv[:1] == ["trace"]:
+        from .trace import main as trace_main
+        return trace_main(argv[1:])
     a = ap.parse_args(argv)
     cfg = EngineConfig(model=a.model, enforce_eager=a.eager)
     cfg.parallel.tensor_parallel_size = a.tensor_parallel_size

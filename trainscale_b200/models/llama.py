@@ -679,3 +679,10 @@ def build_model(cfg: LlamaConfig | str | dict, dtype=torch.bfloat16, device=None
     if seed is not None:
         m.reset_parameters(seed, on_device=init_on_device)
     return m
+
+
+def load_model(config: dict, state_dict: dict[str, torch.Tensor], dtype=torch.bfloat16, device=None) -> LlamaForCausalLM:
+    """Decoder of a HuggingFace-style config.json with the weights of a checkpoint in that naming."""
+    model = build_model(LlamaConfig.from_dict(config), dtype=dtype, device=device)
+    model.load_hf_state_dict(state_dict, strict=True)
+    return model

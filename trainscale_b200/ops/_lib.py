@@ -10,7 +10,7 @@ import functools
 
 import torch
 
-from .build import build_all, lib_path
+from .build import build_libraries, lib_path
 
 _ERR_NAMES = {0: "none", 1: "mbarrier wait timed out", 2: "flag wait timed out", 3: "bad argument", 4: "tmem",
               5: "access outside its tensor (debug build: skipped)"}
@@ -24,14 +24,26 @@ def cuda_available() -> bool:
     return torch.cuda.is_available()
 
 
+LOADED: list[str] = []
+
+
 @functools.lru_cache(maxsize=None)
 def load(name: str) -> ctypes.CDLL:
     path = lib_path(name)
     if not path.exists():
-        build_all()
+        build_libraries([name])
     if not path.exists():
         raise KernelError(f"CUDA library {path} is missing; run `python -m trainscale_b200.ops.build`")
-    return ctypes.CDLL(str(path))
+    lib = ctypes.CDLL(str(path))
+    LOADED.append(name)
+    return lib
+
+
+def prepare(names: list[str]) -> None:
+    """Compile whichever of these libraries are missing (in parallel) before the first of them is needed."""
+    missing = [n for n in names if not lib_path(n).exists()]
+    if missing:
+        build_libraries(missing)
 
 
 def stream_ptr() -> ctypes.c_void_p:
@@ -91,3 +103,9 @@ def raise_on_any_device_error() -> None:
     for src in sources():
         if lib_path(src.stem).exists():
             raise_on_device_error(src.stem)
+
+
+def raise_on_loaded_device_error() -> None:
+    """Check the error word of every library this process has loaded."""
+    for name in LOADED:
+        raise_on_device_error(name)

@@ -52,34 +52,47 @@ def _stale(src: Path, out: Path) -> bool:
     return out.stat().st_mtime < newest
 
 
-def build_all(force: bool = False, verbose: bool = False, debug: bool | None = None) -> list[Path]:
-    """Compile every stale library; returns the list of library paths. Raises on a compile error.
-    `debug`: build the checked variant into lib_debug/ (default: what TS_DEBUG selected for this process)."""
+def build_libraries(names: list[str], force: bool = False, verbose: bool = False, debug: bool | None = None) -> list[Path]:
+    """Compile the stale ones of the named libraries, in parallel; returns their paths. Raises on a compile error.
+    Every library is written under a temporary name and moved into place, so that processes that build at the same time
+    never load half a file.  `debug`: the checked variant in lib_debug/ (default: what TS_DEBUG selected)."""
     nvcc = find_nvcc()
     debug = DEBUG if debug is None else debug
     lib_dir = PKG_DIR / ("lib_debug" if debug else "lib")
     lib_dir.mkdir(exist_ok=True)
     outs = []
     procs = []
-    for src in sources():
-        out = lib_dir / f"libts_{src.stem}.so"
+    for name in names:
+        src, out = CSRC_DIR / f"{name}.cu", lib_dir / f"libts_{name}.so"
         outs.append(out)
         if not force and not _stale(src, out):
             continue
         if nvcc is None:
             raise RuntimeError(f"nvcc not found and {out.name} is missing or stale")
-        cmd = [nvcc, *NVCC_FLAGS, *(["-DTS_DEBUG=1"] if debug else []), "-o", str(out), str(src)]
+        tmp = lib_dir / f".{out.name}.{os.getpid()}"
+        cmd = [nvcc, *NVCC_FLAGS, *(["-DTS_DEBUG=1"] if debug else []), "-o", str(tmp), str(src)]
         if verbose:
             cmd.insert(1, "-Xptxas=-v")
             print(" ".join(cmd), file=sys.stderr)
-        procs.append((src, subprocess.Popen(cmd, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)))
-    for src, p in procs:
+        procs.append((src, tmp, out, subprocess.Popen(cmd, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)))
+    failed = None
+    for src, tmp, out, p in procs:
         log, _ = p.communicate()
         if p.returncode != 0:
-            raise RuntimeError(f"nvcc failed for {src.name}:\n{log}")
+            tmp.unlink(missing_ok=True)
+            failed = failed or f"nvcc failed for {src.name}:\n{log}"
+            continue
+        os.replace(tmp, out)
         if verbose and log:
             print(log, file=sys.stderr)
+    if failed:
+        raise RuntimeError(failed)
     return outs
+
+
+def build_all(force: bool = False, verbose: bool = False, debug: bool | None = None) -> list[Path]:
+    """`build_libraries` for every library of csrc/."""
+    return build_libraries([s.stem for s in sources()], force, verbose, debug)
 
 
 if __name__ == "__main__":

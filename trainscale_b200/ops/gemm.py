@@ -203,3 +203,22 @@ class _SplitLinearCPU(torch.autograd.Function):
             WgradQueue._active.push(dy2, x, w)
             return dx, None
         return dx, (dy2.t() @ x.reshape(-1, x.shape[-1])).to(w.dtype)
+
+
+FEW_ROWS = 64        # up to this many rows a product is one pass over the weight (ops/grouped.rows_linear)
+
+
+@torch.no_grad()
+def serve_linear(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None = None) -> torch.Tensor:
+    """x [M, K] @ w [N, K]^T for serving (no autograd), optionally with an fp32 result.  bf16 on the GPU: few rows go to
+    the few-row kernel, more to the tcgen05 GEMM; rows that are not whole 16-byte vectors, and fp32, to the library."""
+    out_dtype = out_dtype or x.dtype
+    vec = x.is_cuda and x.dtype == torch.bfloat16 and w.shape[1] % 8 == 0 and x.stride(0) % 8 == 0 and x.stride(1) == 1
+    if vec and x.shape[0] <= FEW_ROWS:
+        from . import grouped
+        return grouped.rows_linear(x, w, out_dtype)
+    if vec:
+        return matmul_nt(x, w, out_dtype=out_dtype)
+    if out_dtype != x.dtype:
+        x, w = x.to(out_dtype), w.to(out_dtype)
+    return torch.nn.functional.linear(x, w)

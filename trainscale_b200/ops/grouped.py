@@ -1,0 +1,56 @@
+"""Products of few rows with groups of weight matrices (csrc/skinny.cu): per-head projections, the experts of a decode
+batch, and the fp32 form of both.  Tensors on the CPU take PyTorch math."""
+from __future__ import annotations
+
+import ctypes
+
+import torch
+
+from . import _lib
+
+_ll = ctypes.c_longlong
+ACT_NONE, ACT_RELU_SQUARED = 0, 1
+
+
+def activate(x: torch.Tensor, act: int) -> torch.Tensor:
+    return torch.relu(x).square() if act == ACT_RELU_SQUARED else x
+
+
+def _launch(A, W, out, lda, ldw, ldo, a_group, w_group, o_group, order, start, count, a_div, groups, M, N, K, act):
+    rc = _lib.load("skinny").ts_skinny_gemm(
+        _lib.ptr(A), _lib.ptr(W), _lib.ptr(out), _ll(lda), _ll(ldw), _ll(ldo), _ll(a_group), _ll(w_group), _ll(o_group),
+        _lib.ptr(order), _lib.ptr(start), _lib.ptr(count), a_div, groups, M, N, K, act, int(A.dtype == torch.float32),
+        int(out.dtype == torch.float32), _lib.stream_ptr())
+    _lib.check(rc, "ts_skinny_gemm")
+
+
+def rows_linear(x: torch.Tensor, w: torch.Tensor, out_dtype=None) -> torch.Tensor:
+    """x [M, K] @ w [N, K]^T for a handful of rows: the cost is one pass over w, spread over N / 16 CTAs."""
+    out = torch.empty(x.shape[0], w.shape[0], dtype=out_dtype or x.dtype, device=x.device)
+    _launch(x, w, out, x.stride(0), w.stride(0), out.stride(0), 0, 0, 0, None, None, None, 1, 1, x.shape[0], w.shape[0],
+            w.shape[1], ACT_NONE)
+    return out
+
+
+def head_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
+    """x [T, H, K] (last dimension contiguous), w [H, N, K] -> [T, H, N]: every head has its own matrix."""
+    T, H, K = x.shape
+    N = w.shape[1]
+    if out is None:
+        out = torch.empty(T, H, N, dtype=x.dtype, device=x.device)
+    if not x.is_cuda:
+        return out.copy_(torch.einsum("thk,hnk->thn", x, w))
+    _launch(x, w, out, x.stride(0), w.stride(1), out.stride(0), x.stride(1), w.stride(0), out.stride(1), None, None, None, 1,
+            H, T, N, K, ACT_NONE)
+    return out
+
+
+def expert_linear(x: torch.Tensor, w: torch.Tensor, order, start, count, slots: int, max_rows: int, per_row: int,
+                  act: int = ACT_NONE) -> torch.Tensor:
+    """out[s] = act(w[e(s)] @ x[s // per_row]) for every routed slot s; slots of expert e are
+    order[start[e] : start[e] + count[e]].  w [E, N, K]; `max_rows` bounds count."""
+    E, N, K = w.shape
+    out = torch.empty(slots, N, dtype=x.dtype, device=x.device)
+    _launch(x, w, out, x.stride(0), w.stride(1), out.stride(0), 0, w.stride(0), 0, order, start, count, per_row, E, max_rows,
+            N, K, act)
+    return out

@@ -226,3 +226,69 @@ def topk_softmax(logits: torch.Tensor, k: int, normalize: bool = True):
     if normalize:
         w = w / w.sum(-1, keepdim=True).clamp(min=1e-9)
     return w, idx, probs
+
+
+# ---------------------------------------------------------------------------------------------- serving (no autograd)
+DECODE_ROWS = 64     # up to this many tokens the experts are read by the few-row kernels instead of 128-row tiles
+
+
+def _topk_raw(logits: torch.Tensor, k: int, normalize: bool):
+    T, E = logits.shape
+    w = torch.empty(T, k, dtype=torch.float32, device=logits.device)
+    idx = torch.empty(T, k, dtype=torch.int32, device=logits.device)
+    rc = _lib.load("moe").ts_moe_topk_softmax(_lib.ptr(logits), _lib.ptr(None), _lib.ptr(w), _lib.ptr(idx), T, E, int(k),
+                                              int(normalize), _lib.stream_ptr())
+    _lib.check(rc, "ts_moe_topk_softmax")
+    return w, idx
+
+
+def _route_decode(logits: torch.Tensor, k: int, normalize: bool):
+    T, E = logits.shape
+    i32 = dict(dtype=torch.int32, device=logits.device)
+    w = torch.empty(T, k, dtype=torch.float32, device=logits.device)
+    order, start, count = torch.empty(T * k, **i32), torch.empty(E, **i32), torch.empty(E, **i32)
+    rc = _lib.load("moe").ts_moe_route(_lib.ptr(logits), _lib.ptr(w), _lib.ptr(order), _lib.ptr(start), _lib.ptr(count), T, E,
+                                       int(k), int(normalize), _lib.stream_ptr())
+    _lib.check(rc, "ts_moe_route")
+    return w, order, start, count
+
+
+def _grouped_act(x, W, plan: MoEPlan, act: int):
+    E, N, K = W.shape
+    y = torch.empty(plan.P, N, dtype=x.dtype, device=x.device)
+    rc = _lib.load("gemm").ts_gemm_grouped_bf16_act(
+        _lib.ptr(x), _lib.ptr(W), _lib.ptr(y), 1, plan.P, N, K, K, K, N, 0, 0, 0, 0, _c.c_float(1.0),
+        _lib.ptr(plan.tile_expert), E, act, _lib.stream_ptr())
+    _lib.check(rc, "ts_gemm_grouped_bf16_act")
+    return y
+
+
+def routed_experts(x: torch.Tensor, logits: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, k: int, act: int,
+                   normalize: bool = False):
+    """Ungated experts down(act(up x)) of every token's top-k of softmax(logits), NOT combined: the layer boundary sums
+    them into the fp32 stream.  x [T, H], logits [T, E] fp32, w_up [E, F, H], w_down [E, H, F], act of ops/grouped.
+    Returns (outputs, dest, weights [T, k]): slot t * k + j is row dest[slot] of the outputs (dest None: row slot).
+
+    Few tokens: router, top-k and sort in one kernel, then one pass over the visited experts' weights.  Many (bf16):
+    128-row expert segments on the grouped tcgen05 GEMM, the activation in its epilogue."""
+    from . import grouped
+    T, E = logits.shape
+    if not x.is_cuda:
+        w, idx, _ = topk_softmax(logits, k, normalize)
+        y = torch.zeros(T * k, x.shape[1], dtype=x.dtype)
+        for e in range(E):
+            slots = (idx.reshape(-1) == e).nonzero().squeeze(1)
+            y[slots] = grouped.activate(x[slots // k] @ w_up[e].t(), act) @ w_down[e].t()
+        return y, None, w
+    H, F = x.shape[1], w_up.shape[1]
+    if T <= DECODE_ROWS and T * k <= _lib.load("moe").ts_moe_route_max_slots():
+        w, order, start, count = _route_decode(logits, k, normalize)
+    else:
+        w, idx = _topk_raw(logits, k, normalize)
+        plan = make_plan(idx, E)
+        if x.dtype == torch.bfloat16 and H % 8 == 0 and F % 8 == 0:
+            h = _grouped_act(_permute_raw(x, plan), w_up, plan, act)
+            return _grouped_act(h, w_down, plan, grouped.ACT_NONE), plan.dest, w
+        order, start, count = plan.src_of_row, plan.seg_start, plan.counts
+    h = grouped.expert_linear(x, w_up, order, start, count, T * k, T, k, act)
+    return grouped.expert_linear(h, w_down, order, start, count, T * k, T, 1), None, w
