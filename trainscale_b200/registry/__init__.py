@@ -409,6 +409,8 @@ register_models_from_meta([
     ModelInfo("mixtral", "mistralai", ("8x7B", "8x22B"), "MixtralForCausalLM", mlp="moe"),
     ModelInfo("qwen_moe", "Qwen", ("A2.7B", "A14B"), "Qwen2MoeForCausalLM", mlp="moe", supported=False,
               notes="shared expert + per-layer dense/sparse mix not covered"),
+    ModelInfo("mezilix", "trainscale", ("4B",), "MezilixForCausalLM", attention="latent", mlp="moe (squared ReLU)",
+              norm="scalar rmsnorm", notes="serving only: models/mezilix.py; windowed latent cache, state per sequence"),
     ModelInfo("llava", "llava-hf", ("7B", "13B"), "LlavaForConditionalGeneration", supported=False, notes="vision tower not covered"),
 ])
 
