@@ -403,7 +403,8 @@ class ModelRunner:
 
     @torch.no_grad()
     def decode_graphed(self, host: HostBatch) -> torch.Tensor:
-        """One decode step (one new token per sequence) replayed from a CUDA graph; returns fp32 logits [n, V].
+        """One decode step (one new token per sequence) replayed from a CUDA graph; returns fp32 logits [n, V], valid until
+        the next replay.
         The batch is padded to a power of two with rows that write to / read from the cache's spare block."""
         n = len(host.seq_ids)
         n_pad = 1
@@ -416,6 +417,7 @@ class ModelRunner:
         if st is None:
             st = self.graphs[key] = self._capture(n_pad, width)
         h = st["host"]
+        st["copied"].synchronize()           # the copies of the step before may still be reading the pinned buffers
         for name, (dtype, pad) in self._static_fields().items():
             h[name].fill_(pad)
         h["block_table"].fill_(self.cache.trash_block)
@@ -426,6 +428,7 @@ class ModelRunner:
         h["block_table"][:n, :bt.shape[1]] = bt
         for name, buf in h.items():
             getattr(st["batch"], name).copy_(buf, non_blocking=True)
+        st["copied"].record()
         st["graph"].replay()
         self.graph_replays += 1
         return st["logits"][:n]
@@ -438,7 +441,8 @@ class ModelRunner:
         rows = torch.arange(n_pad, dtype=torch.int32, device=dev)
         batch = StepBatch(None, row_seq=rows, out_rows=rows, n_single=n_pad, max_len=width * bs, fresh=False,
                           splits=max(1, -(-(width * bs) // 512)), **buf)
-        st = {"batch": batch, "host": {k: torch.empty_like(v, device="cpu").pin_memory() for k, v in buf.items()}}
+        st = {"batch": batch, "host": {k: torch.empty_like(v, device="cpu").pin_memory() for k, v in buf.items()},
+              "copied": torch.cuda.Event()}
 
         def body():
             return self.model.logits(self._layers(batch)).float()
