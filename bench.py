@@ -287,6 +287,18 @@ def measure(args, sharding: str, steps: int, warmup: int, e2e: bool = True) -> d
                                   "config": {}}
 
 
+def run_serving(args) -> None:
+    """One JSON line per size; device-timed, L2 flushed between steps, random weights and tokens."""
+    from trainscale_b200.inference import bench_serving
+    sampler = ClockSampler(0)
+    for size in args.serve or list(bench_serving.SIZES):
+        sampler.samples.clear()
+        sampler.start()
+        res = bench_serving.run([size], ROOT / "MEASURED_PEAKS.json", max(args.steps, 5))[size]
+        print(json.dumps({"size": size, "dtype": "bf16", "data": "random weights and tokens", **res,
+                          "clocks": sampler.stop()}), flush=True)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -301,7 +313,12 @@ def main():
     ap.add_argument("--comm", default="auto", choices=["auto", "fused", "nccl"])
     ap.add_argument("--no-secondary", action="store_true", help="skip the measurement of the other sharding mode")
     ap.add_argument("--secondary-timeout", type=float, default=300.0)
+    ap.add_argument("--serve", nargs="*", default=None, metavar="SIZE",
+                    help="instead: prefill / decode throughput of the Mezilix decoder beside the closest model at these "
+                         "sizes (default all), with per-op roofline fractions; one GPU")
     args = ap.parse_args()
+    if args.serve is not None:
+        return run_serving(args)
     args.warmup = max(args.warmup, 3)
     world = int(os.environ.get("WORLD_SIZE", "1"))
     if args.gpus > 1 and world == 1:

@@ -2,8 +2,9 @@
 //
 // Decode multiplies a handful of rows with every weight of the layer, so the cost is reading the weights once.  A
 // tcgen05 tile would be 128 rows high with almost all of them empty and gives too few CTAs to pull from every memory
-// channel; here the WEIGHTS are the 16-row operand of a warp MMA, tokens are its 8 columns, a CTA owns 16 weight rows
-// and its eight warps split the reduction, so a projection of N rows spreads over N / 16 CTAs.  Both operands are read
+// channel; here the WEIGHTS are the 16-row operand of a warp MMA, tokens are its 8 columns, and the eight warps of a CTA
+// split the reduction of one 16-row tile (or of several, when it is short), so a projection of N rows spreads over up to
+// N / 16 CTAs.  Both operands are read
 // straight from global memory as 16-byte vectors: the reduction index is permuted the same way on both sides (a lane's
 // eight consecutive values feed two MMA steps), so no shared-memory staging or transposition is needed.
 //
@@ -56,18 +57,24 @@ __device__ __forceinline__ uint4 ld_stream(const void* p) {   // weights: read o
   return v;
 }
 
-// NT: token tiles of 8 per pass.  grid (ceil(N / 16), groups).
-template <int NT>
+// 32-wide reduction steps a warp has in flight
+__host__ __device__ constexpr int skinny_unroll(int nt) { return nt == 1 ? 8 : (nt <= 4 ? 4 : 2); }
+
+// NT: token tiles of 8 per pass.  KW: warps that share a row tile and split its reduction; the CTA's 8 / KW row tiles are
+// neighbours.  grid (ceil(N / (16 * 8 / KW)), groups).
+template <int NT, int KW>
 __global__ void __launch_bounds__(SK_WARPS * 32)
 skinny_gemm_kernel(SkinnyParams p) {
-  constexpr int UN = NT <= 2 ? 4 : (NT == 4 ? 2 : 1);     // 32-wide reduction steps in flight
+  constexpr int UN = skinny_unroll(NT);
   __shared__ float red[SK_WARPS][16][NT * 8 + 1];
-  const int g = blockIdx.y, n0 = blockIdx.x * 16;
+  constexpr int TILES = SK_WARPS / KW;
+  const int g = blockIdx.y;
   const int m_total = p.count ? p.count[g] : p.M;
   const int first = p.start ? p.start[g] : 0;
   if (m_total == 0) return;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int gid = lane >> 2, tig = lane & 3;
+  const int n0 = (blockIdx.x * TILES + warp / KW) * 16, wk = warp % KW;
   const __nv_bfloat16* A = reinterpret_cast<const __nv_bfloat16*>(p.A) + g * p.a_group;
   const __nv_bfloat16* W = reinterpret_cast<const __nv_bfloat16*>(p.W) + g * p.w_group;
   const bool row0 = n0 + gid < p.N, row1 = n0 + gid + 8 < p.N;
@@ -92,7 +99,7 @@ skinny_gemm_kernel(SkinnyParams p) {
       for (int q = 0; q < 4; ++q) acc[t][q] = 0.f;
 
     const int steps = (p.K + 31) / 32;
-    for (int s = warp * UN; s < steps; s += SK_WARPS * UN) {
+    for (int s = wk * UN; s < steps; s += KW * UN) {       // UN steps in a row: 64 * UN bytes of a weight row at once
       uint4 a0[UN], a1[UN], b[UN][NT];
 #pragma unroll
       for (int u = 0; u < UN; ++u) {
@@ -121,15 +128,16 @@ skinny_gemm_kernel(SkinnyParams p) {
       red[warp][gid + 8][t * 8 + tig * 2 + 1] = acc[t][3];
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < m * 16; i += SK_WARPS * 32) {
-      const int tk = i >> 4, n = i & 15;
-      if (n0 + n < p.N) {
+    for (int i = threadIdx.x; i < TILES * m * 16; i += SK_WARPS * 32) {
+      const int tile = TILES == 1 ? 0 : i / (m * 16), r = i - tile * m * 16;
+      const int tk = r >> 4, n = r & 15, nn = (blockIdx.x * TILES + tile) * 16 + n;
+      if (nn < p.N) {
         float v = 0.f;
 #pragma unroll
-        for (int w = 0; w < SK_WARPS; ++w) v += red[w][n][tk];
+        for (int w = 0; w < KW; ++w) v += red[tile * KW + w][n][tk];
         v = skinny_act(v, p.act);
         const int slot = p.order ? p.order[first + base + tk] : base + tk;
-        const long long at = g * p.o_group + static_cast<long long>(slot) * p.ldo + n0 + n;
+        const long long at = g * p.o_group + static_cast<long long>(slot) * p.ldo + nn;
         if (p.out_fp32) reinterpret_cast<float*>(p.out)[at] = v;
         else reinterpret_cast<__nv_bfloat16*>(p.out)[at] = __float2bfloat16(v);
       }
@@ -179,6 +187,14 @@ __global__ void __launch_bounds__(256) grouped_simt_kernel(SkinnyParams p) {
   }
 }
 
+template <int NT>
+static void launch_skinny(int kw, dim3 grid, cudaStream_t st, const SkinnyParams& p) {
+  if (kw == 8) skinny_gemm_kernel<NT, 8><<<grid, SK_WARPS * 32, 0, st>>>(p);
+  else if (kw == 4) skinny_gemm_kernel<NT, 4><<<grid, SK_WARPS * 32, 0, st>>>(p);
+  else if (kw == 2) skinny_gemm_kernel<NT, 2><<<grid, SK_WARPS * 32, 0, st>>>(p);
+  else skinny_gemm_kernel<NT, 1><<<grid, SK_WARPS * 32, 0, st>>>(p);
+}
+
 static bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; }
 
 }  // namespace ts
@@ -186,11 +202,12 @@ static bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 
 TS_DEFINE_ERROR_API(ts_skinny)
 using namespace ts;
 
-// M: rows of every group, or an upper bound of them when `count` is given.  fp32: A and W are fp32 (else bf16).
+// M: rows of every group, or an upper bound of them when `count` is given (`typical`: how many a group usually has; more
+// take further passes over the weights, which then come from L2).  fp32: A and W are fp32 (else bf16).
 extern "C" int ts_skinny_gemm(const void* A, const void* W, void* out, long long lda, long long ldw, long long ldo,
                               long long a_group, long long w_group, long long o_group, const int* order,
                               const int* start, const int* count, int a_div, int groups, int M, int N, int K, int act,
-                              int fp32, int out_fp32, void* stream) {
+                              int fp32, int out_fp32, int typical, void* stream) {
   if (M <= 0 || groups <= 0) return 0;
   if (N <= 0 || K <= 0 || a_div <= 0 || act < 0 || act > 1 || groups > 65535) return -10;
   if (fp32 && !out_fp32) return -11;
@@ -209,10 +226,15 @@ extern "C" int ts_skinny_gemm(const void* A, const void* W, void* out, long long
     else grouped_simt_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>(p);
     return (int)cudaGetLastError();
   }
-  const dim3 grid((N + 15) / 16, groups);
-  if (M <= 8) skinny_gemm_kernel<1><<<grid, SK_WARPS * 32, 0, st>>>(p);
-  else if (M <= 16) skinny_gemm_kernel<2><<<grid, SK_WARPS * 32, 0, st>>>(p);
-  else if (M <= 32) skinny_gemm_kernel<4><<<grid, SK_WARPS * 32, 0, st>>>(p);
-  else skinny_gemm_kernel<8><<<grid, SK_WARPS * 32, 0, st>>>(p);
+  const int per_pass = count && typical > 0 && typical < M ? typical : M;
+  const int nt = per_pass <= 8 ? 1 : (per_pass <= 16 ? 2 : (per_pass <= 32 ? 4 : 8));
+  int kw = 1;
+  while (kw < SK_WARPS && kw * skinny_unroll(nt) * 32 < K) kw *= 2;
+  const int rows = 16 * SK_WARPS / kw;
+  const dim3 grid((N + rows - 1) / rows, groups);
+  if (nt == 1) launch_skinny<1>(kw, grid, st, p);
+  else if (nt == 2) launch_skinny<2>(kw, grid, st, p);
+  else if (nt == 4) launch_skinny<4>(kw, grid, st, p);
+  else launch_skinny<8>(kw, grid, st, p);
   return (int)cudaGetLastError();
 }

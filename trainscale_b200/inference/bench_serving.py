@@ -1,0 +1,293 @@
+"""Prefill and decode throughput of a served design beside the framework's closest existing model at equal size, with the
+device time of every op and its distance from the roofline (`bench.py --serve`).
+
+Both models run through `ModelRunner` on the engine's cache with random weights and random tokens.  Step times are CUDA
+events around whole steps; for the per-op table the host first queues a spin kernel, so that a whole step is enqueued
+before the device starts it and the events around each op see no launch gaps.
+"""
+from __future__ import annotations
+
+import json
+import math
+import statistics
+from pathlib import Path
+
+import torch
+
+from .batch import HostBatch, StepEntry
+from .engine import EngineConfig, EngineCore
+
+# name -> sizes shared by both models; Mezilix experts have two matrices of `ff`, the gated ones three of 2/3 ff
+SIZES = {
+    "1k": dict(layers=12, width=1024, heads=8, dim=64, rot=32, vdim=64, rank=256, window=512, experts=16, top=2, ff=1536),
+    "2k": dict(layers=16, width=2048, heads=16, dim=128, rot=64, vdim=128, rank=512, window=1024, experts=32, top=4, ff=1536),
+    "4k": dict(layers=8, width=4096, heads=32, dim=128, rot=64, vdim=128, rank=512, window=4096, experts=64, top=6, ff=1536),
+}
+VOCAB = 32000
+
+
+def build_mezilix(z: dict):
+    from ..models.mezilix import build_model, uniform_config
+    return build_model(uniform_config(layers=z["layers"], vocab=VOCAB, width=z["width"], heads=z["heads"], dim=z["dim"],
+                                      rot_dim=z["rot"], vdim=z["vdim"], kv_rank=z["rank"], window=z["window"],
+                                      experts=z["experts"], top=z["top"], ff=z["ff"], buckets=65521),
+                       torch.bfloat16, "cuda", seed=0)
+
+
+def build_closest(z: dict):
+    """Llama decoder with a mixture of gated experts: same width, depth, heads, experts and expert weights."""
+    from ..models.llama import LlamaConfig, build_model
+    cfg = LlamaConfig(vocab_size=VOCAB, hidden_size=z["width"], intermediate_size=z["ff"] * 2 // 3,
+                      num_hidden_layers=z["layers"], num_attention_heads=z["heads"], num_key_value_heads=max(1, z["heads"] // 4),
+                      head_dim=z["vdim"], num_local_experts=z["experts"], num_experts_per_tok=z["top"],
+                      model_type="mixtral", max_position_embeddings=16384)
+    return build_model(cfg, torch.bfloat16, "cuda", seed=0, init_on_device=True)
+
+
+def make_core(model, tokens: int, seqs: int) -> EngineCore:
+    cfg = EngineConfig(model="custom", tokenizer="byte", device="cuda", enforce_eager=False)
+    cfg.cache.num_gpu_blocks = tokens // cfg.cache.block_size + seqs
+    cfg.cache.enable_prefix_caching = False
+    cfg.scheduler.max_num_seqs = seqs
+    return EngineCore(cfg, model=model)
+
+
+def _tokens(n: int, seed: int) -> list[int]:
+    return torch.randint(0, VOCAB, (n,), generator=torch.Generator().manual_seed(seed)).tolist()
+
+
+def _timed(fn, n: int, warm: int = 3) -> float:
+    """Median device time (ms) of `fn`, the L2 flushed between calls."""
+    flush = torch.empty(64 << 20, dtype=torch.float32, device="cuda")
+    out = []
+    for i in range(warm + n):
+        flush.zero_()
+        torch.cuda._sleep(20_000_000)       # the step is enqueued while the device spins
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        a.record()
+        fn()
+        b.record()
+        b.synchronize()
+        if i >= warm:
+            out.append(a.elapsed_time(b))
+    return statistics.median(out)
+
+
+# ---------------------------------------------------------------------------------------------- per-op costs
+def _bytes(*ts) -> int:
+    return sum(t.numel() * t.element_size() for t in ts if isinstance(t, torch.Tensor))
+
+
+class OpTimer:
+    """Events around every call of the wrapped op functions; `cost(args, kwargs, result) -> (bytes, flops)`."""
+
+    def __init__(self, table: list[tuple]):
+        self.table, self.records, self.saved, self.depth = table, [], [], 0
+
+    def __enter__(self):
+        for owner, attr, name, cost in self.table:
+            fn = getattr(owner, attr)
+            self.saved.append((owner, attr, fn))
+            setattr(owner, attr, self._wrap(fn, name, cost))
+        return self
+
+    def __exit__(self, *exc):
+        for owner, attr, fn in reversed(self.saved):
+            setattr(owner, attr, fn)
+        self.saved.clear()
+
+    def _wrap(self, fn, name, cost):
+        def call(*a, **k):
+            if self.depth:
+                return fn(*a, **k)
+            self.depth += 1
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            out = fn(*a, **k)
+            e1.record()
+            self.depth -= 1
+            label = name(a, out) if callable(name) else name
+            self.records.append((label, e0, e1, *cost(a, k, out)))
+            return out
+        return call
+
+    def summary(self, peaks: dict) -> dict:
+        torch.cuda.synchronize()
+        acc: dict = {}
+        for name, e0, e1, nbytes, flops in self.records:
+            r = acc.setdefault(name, [0, 0.0, 0.0, 0.0])
+            floor = max(nbytes / (peaks["hbm_gbs"] * 1e9), flops / (peaks["bf16_tflops"] * 1e12)) * 1e3
+            r[0] += 1
+            r[1] += e0.elapsed_time(e1)
+            r[2] += floor
+        return {n: {"calls": c, "ms": round(ms, 4), "of_roofline": round(fl / ms, 3) if ms else None}
+                for n, (c, ms, fl, _) in sorted(acc.items(), key=lambda kv: -kv[1][1])}
+
+
+def _linear_cost(a, k, out):
+    x, w = a[0], a[1]
+    return _bytes(x, w, out), 2.0 * (x.numel() // x.shape[-1]) * w.shape[0] * w.shape[1]
+
+
+def _linear_name(prefix):
+    return lambda a, out: f"{prefix} {a[1].shape[0]}x{a[1].shape[1]}"
+
+
+def _visited(top: int, experts: int, rows: int) -> float:
+    """Expected number of distinct experts of `rows` tokens."""
+    return experts * (1.0 - (1.0 - top / experts) ** rows)
+
+
+def mezilix_table(z: dict, rows: int, keys: float, pairs: float) -> list[tuple]:
+    """`keys`: cached rows a step must read per layer; `pairs`: visible (query, key) pairs per layer and head."""
+    from ..ops import gemm, grouped, latent_attention as latent, moe, stream
+    W, H = z["width"], z["heads"]
+    ew = _visited(z["top"], z["experts"], rows) * z["ff"] * W * 2
+
+    def boundary(a, k, out):
+        x, mixer, experts, hist, n = a[0], a[1], a[2], a[3], a[5]
+        T = out.shape[0] if isinstance(out, torch.Tensor) else x.shape[0]
+        per = 4 + 2 + (0 if experts is None else 2 * experts[2].shape[1]) + 4 * n
+        per += 2 if isinstance(out, torch.Tensor) else 4 + 4 + 2 + 2
+        return per * T * W, 0.0
+
+    def experts(a, k, out):
+        x, w = a[0], a[1]
+        return ew + _bytes(x, out), 2.0 * rows * z["top"] * w.shape[1] * w.shape[2]
+
+    return [
+        (stream, "embed", "embedding, norm, shift", lambda a, k, o: (a[0].shape[0] * W * (2 + 2 + 4 + 2 + 2), 0.0)),
+        (stream, "boundary", "layer boundary", boundary),
+        (stream, "final", "final norm", boundary),
+        (gemm, "serve_linear", _linear_name("gemm"), _linear_cost),
+        (gemm, "matmul_nt", _linear_name("gemm"), _linear_cost),
+        (latent, "prepare", "latent norm, rotary, cache write",
+         lambda a, k, o: (_bytes(a[0]) * (1 + z["heads"] * z["rot"] / a[0].shape[1]) +
+                          a[0].shape[0] * a[1].row_width * 2 * (2 if o is not None else 1), 0.0)),
+        (latent, "gather_rows", "latent gather", lambda a, k, o: (2 * _bytes(o), 0.0)),
+        (latent, "attend_latent", "attention (latent space)",
+         lambda a, k, o: (keys * a[2].row_width * 2 + 2 * _bytes(a[0]), 2.0 * pairs * H * (2 * z["rank"] + z["rot"]))),
+        (latent, "attend_expanded", "attention (expanded)",
+         lambda a, k, o: (_bytes(a[1], a[2]) + a[0].shape[0] * a[3].q_width * 2 + _bytes(a[7]),
+                          2.0 * pairs * H * (z["dim"] + z["rot"] + z["vdim"]))),
+        (grouped, "head_linear", lambda a, o: f"per-head projection {a[1].shape[1]}x{a[1].shape[2]}",
+         lambda a, k, o: (_bytes(a[0], a[1], o), 2.0 * a[0].shape[0] * a[1].numel())),
+        (grouped, "expert_linear", lambda a, o: f"experts {a[1].shape[1]}x{a[1].shape[2]}", experts),
+        (moe, "_route_decode", "router top-k, sort", lambda a, k, o: (_bytes(a[0], *o), 0.0)),
+        (moe, "_topk_raw", "router top-k", lambda a, k, o: (_bytes(a[0], *o), 0.0)),
+        (moe, "make_plan", "routing plan", lambda a, k, o: (_bytes(a[0], o.dest, o.src_of_row), 0.0)),
+        (moe, "_permute_raw", "permute", lambda a, k, o: (_bytes(a[0]) + a[1].n * W * 2, 0.0)),
+        (moe, "_grouped_act", lambda a, o: f"experts {a[1].shape[1]}x{a[1].shape[2]}",
+         lambda a, k, o: (ew + rows * z["top"] * (a[1].shape[1] + a[1].shape[2]) * 2,
+                          2.0 * rows * z["top"] * a[1].shape[1] * a[1].shape[2])),
+    ]
+
+
+def closest_table(z: dict, rows: int, keys: float, pairs: float, runner) -> list[tuple]:
+    from ..ops import activation, gemm, moe, norm, rope
+    W, H, D = z["width"], z["heads"], z["vdim"]
+    hkv = max(1, H // 4)
+
+    def grouped_cost(a, k, out):
+        E, N, K = a[1].shape
+        return (_visited(z["top"], E, rows) * N * K * 2 + rows * z["top"] * (N + K) * 2, 2.0 * rows * z["top"] * N * K)
+
+    return [
+        (norm, "rmsnorm", "rms norm", lambda a, k, o: (_bytes(a[0], *[t for t in o if t is not None]) + _bytes(*a[3:4]), 0.0)),
+        (gemm, "linear", _linear_name("gemm"), _linear_cost),
+        (rope, "apply_rope_qkv", "rotary", lambda a, k, o: (2 * _bytes(a[0]) * (H + hkv) / (H + 2 * hkv), 0.0)),
+        (runner, "_write_cache", "cache write", lambda a, k, o: (2 * a[1].shape[0] * 2 * hkv * D * 2, 0.0)),
+        (runner, "_attend", "attention", lambda a, k, o: (keys * 2 * hkv * D * 2 + 2 * _bytes(o), 4.0 * pairs * H * D)),
+        (moe, "topk_softmax", "router top-k", lambda a, k, o: (_bytes(a[0], *o), 0.0)),
+        (moe, "make_plan", "routing plan", lambda a, k, o: (_bytes(a[0], o.dest, o.src_of_row), 0.0)),
+        (moe, "_permute_raw", "permute", lambda a, k, o: (_bytes(a[0]) + a[1].n * W * 2, 0.0)),
+        (moe, "grouped_linear", lambda a, o: f"experts {a[1].shape[1]}x{a[1].shape[2]}", grouped_cost),
+        (activation, "glu", "gated activation", lambda a, k, o: (rows * z["top"] * 3 * o.shape[1] * 2, 0.0)),
+        (moe, "_combine_raw", "combine", lambda a, k, o: (rows * z["top"] * W * 2 + _bytes(o), 0.0)),
+    ]
+
+
+# ---------------------------------------------------------------------------------------------- measurement
+def _visible_pairs(lengths: list[tuple[int, int]], window: int) -> float:
+    """Sum over (first position, tokens) of the keys each position sees."""
+    return float(sum(min(p + 1, window) for start, n in lengths for p in range(start, start + n)))
+
+
+def measure(name: str, z: dict, peaks: dict, prompts: int = 2, prompt_len: int = 4096, batches=(8, 64), context: int = 2048,
+            iters: int = 5) -> dict:
+    out: dict = {"sizes": z, "models": {}}
+    for kind, build in (("mezilix", build_mezilix), ("closest", build_closest)):
+        model = build(z)
+        core = make_core(model, max(prompts * prompt_len, max(batches) * (context + 64)), max(max(batches), prompts))
+        window = z["window"] if kind == "mezilix" else 1 << 30
+        res: dict = {"parameters": sum(p.numel() for p in model.parameters())}
+
+        def table(rows, keys, pairs):
+            return mezilix_table(z, rows, keys, pairs) if kind == "mezilix" else \
+                closest_table(z, rows, keys, pairs, core.runner)
+
+        def profile(step, rows, keys, pairs):
+            with OpTimer(table(rows, keys, pairs)) as t:
+                torch.cuda._sleep(200_000_000)
+                step()
+            return t.summary(peaks)
+
+        # prefill: whole prompts in one step
+        entries = [StepEntry(i, _tokens(prompt_len, i)) for i in range(prompts)]
+        host = HostBatch(core.cache, entries)
+        batch = host.to_device("cuda")
+        step = lambda: core.runner.forward(batch)   # noqa: E731
+        ms = _timed(step, iters)
+        T = prompts * prompt_len
+        res["prefill"] = {"tokens": T, "ms": ms, "tokens_per_s": T / ms * 1e3,
+                          "ops": profile(step, T, T, _visible_pairs([(0, prompt_len)] * prompts, window))}
+        # portions that continue cached prompts
+        if kind == "mezilix":
+            for i in range(prompts):
+                core.release(i)
+            half = prompt_len // 2
+            with torch.no_grad():
+                core.execute([StepEntry(i, e.tokens[:half], []) for i, e in enumerate(entries)])
+            b2 = HostBatch(core.cache, [StepEntry(i, e.tokens[half:]) for i, e in enumerate(entries)]).to_device("cuda")
+            ms = _timed(lambda: core.runner.forward(b2), iters)
+            res["prefill_continued"] = {"tokens": T - prompts * half, "ms": ms, "tokens_per_s": (T - prompts * half) / ms * 1e3}
+        for i in range(prompts):
+            core.release(i)
+        # decode: one token per sequence on top of `context` cached tokens
+        res["decode"] = {}
+        for n in batches:
+            for i in range(0, n, 4):
+                core.execute([StepEntry(j, _tokens(context, 100 + j), []) for j in range(i, min(n, i + 4))])
+            host = HostBatch(core.cache, [StepEntry(j, [j + 1]) for j in range(n)])
+            batch = host.to_device("cuda")
+            step = lambda: core.runner.logits(core.runner.forward(batch))   # noqa: E731
+            keys = float(n * min(window, context + 1))
+            d = {"ms": _timed(step, iters), "ops": profile(step, n, keys, keys)}
+            if core.runner.can_graph(host):
+                core.runner.decode_graphed(host)
+                d["graph_ms"] = _timed(lambda: core.runner.decode_graphed(host), iters)
+            d["tokens_per_s"] = n / min(d["ms"], d.get("graph_ms", math.inf)) * 1e3
+            res["decode"][str(n)] = d
+            for j in range(n):
+                core.release(j)
+        out["models"][kind] = res
+        del core, model, batch, host, step
+        torch.cuda.empty_cache()
+    m = out["models"]
+    out["mezilix_over_closest"] = {
+        "prefill": m["mezilix"]["prefill"]["tokens_per_s"] / m["closest"]["prefill"]["tokens_per_s"],
+        **{f"decode_{n}": m["mezilix"]["decode"][n]["tokens_per_s"] / m["closest"]["decode"][n]["tokens_per_s"]
+           for n in m["mezilix"]["decode"]}}
+    return out
+
+
+def run(sizes: list[str], peaks_file: Path, iters: int = 5) -> dict:
+    peaks = {"hbm_gbs": 6538.9, "bf16_tflops": 1608.3}
+    try:
+        peaks.update(json.loads(peaks_file.read_text()))
+    except OSError:
+        pass
+    from ..ops import _lib
+    out = {n: measure(n, SIZES[n], peaks, iters=iters) for n in sizes}
+    _lib.raise_on_loaded_device_error()
+    return out

@@ -205,7 +205,10 @@ class _SplitLinearCPU(torch.autograd.Function):
         return dx, (dy2.t() @ x.reshape(-1, x.shape[-1])).to(w.dtype)
 
 
-FEW_ROWS = 64        # up to this many rows a product is one pass over the weight (ops/grouped.rows_linear)
+def few_rows(M: int, N: int, K: int) -> bool:
+    """Whether one pass over the weight by warps (ops/grouped.rows_linear) beats 128-row tcgen05 tiles: measured crossover,
+    later for small weights, whose few tiles leave most of the GPU idle."""
+    return M <= 16 or (M <= 32 and N * K <= 1 << 23)
 
 
 @torch.no_grad()
@@ -214,7 +217,7 @@ def serve_linear(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None
     the few-row kernel, more to the tcgen05 GEMM; rows that are not whole 16-byte vectors, and fp32, to the library."""
     out_dtype = out_dtype or x.dtype
     vec = x.is_cuda and x.dtype == torch.bfloat16 and w.shape[1] % 8 == 0 and x.stride(0) % 8 == 0 and x.stride(1) == 1
-    if vec and x.shape[0] <= FEW_ROWS:
+    if vec and few_rows(x.shape[0], *w.shape):
         from . import grouped
         return grouped.rows_linear(x, w, out_dtype)
     if vec:

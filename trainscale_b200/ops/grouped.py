@@ -16,11 +16,12 @@ def activate(x: torch.Tensor, act: int) -> torch.Tensor:
     return torch.relu(x).square() if act == ACT_RELU_SQUARED else x
 
 
-def _launch(A, W, out, lda, ldw, ldo, a_group, w_group, o_group, order, start, count, a_div, groups, M, N, K, act):
+def _launch(A, W, out, lda, ldw, ldo, a_group, w_group, o_group, order, start, count, a_div, groups, M, N, K, act,
+            typical=0):
     rc = _lib.load("skinny").ts_skinny_gemm(
         _lib.ptr(A), _lib.ptr(W), _lib.ptr(out), _ll(lda), _ll(ldw), _ll(ldo), _ll(a_group), _ll(w_group), _ll(o_group),
         _lib.ptr(order), _lib.ptr(start), _lib.ptr(count), a_div, groups, M, N, K, act, int(A.dtype == torch.float32),
-        int(out.dtype == torch.float32), _lib.stream_ptr())
+        int(out.dtype == torch.float32), typical, _lib.stream_ptr())
     _lib.check(rc, "ts_skinny_gemm")
 
 
@@ -52,5 +53,5 @@ def expert_linear(x: torch.Tensor, w: torch.Tensor, order, start, count, slots: 
     E, N, K = w.shape
     out = torch.empty(slots, N, dtype=x.dtype, device=x.device)
     _launch(x, w, out, x.stride(0), w.stride(1), out.stride(0), 0, w.stride(0), 0, order, start, count, per_row, E, max_rows,
-            N, K, act)
+            N, K, act, -(-2 * slots // E))
     return out

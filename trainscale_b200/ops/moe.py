@@ -229,7 +229,7 @@ def topk_softmax(logits: torch.Tensor, k: int, normalize: bool = True):
 
 
 # ---------------------------------------------------------------------------------------------- serving (no autograd)
-DECODE_ROWS = 64     # up to this many tokens the experts are read by the few-row kernels instead of 128-row tiles
+DECODE_ROWS = 32     # up to this many tokens the experts are read by the few-row kernels instead of 128-row tiles
 
 
 def _topk_raw(logits: torch.Tensor, k: int, normalize: bool):
