@@ -164,13 +164,14 @@ __global__ void latent_merge_kernel(LatentAttendParams p) {
 }
 
 // ---------------------------------------------------------------------------------------------------------
-// bf16 decode kernel.  grid (rows, ceil(H / 16), splits), 8 warps.  Tiles of KT cached rows stream through two
+// bf16 decode kernel.  grid (rows, ceil(H / 16), splits), 16 warps.  Tiles of KT cached rows stream through two
 // shared-memory buffers (cp.async); a tile serves as K (all row_width columns) and as V (the first rank columns).
-//   scores   warp w: the 16 heads x keys [8w, 8w + 8) of the tile, over all columns
-//   softmax  warp w: heads 2w, 2w + 1 (running max and sum in registers, fp32)
-//   output   warp w: latent columns [16 NP w, 16 NP (w + 1)) of the 16 heads, fp32 accumulators in registers
+//   scores   warp w: the 16 heads x keys [8 (w % 8), + 8) of the tile, over half w / 8 of the columns; the query fragments
+//            of that half stay in registers for the whole kernel
+//   softmax  warp w: head w (running max and sum in registers, fp32)
+//   output   warp w: latent columns [8 NP w, 8 NP (w + 1)) of the 16 heads, fp32 accumulators in registers
 // ---------------------------------------------------------------------------------------------------------
-constexpr int LD_WARPS = 8;
+constexpr int LD_WARPS = 16;
 constexpr int LD_KT = 64;
 
 __device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], uint32_t addr) {
@@ -199,18 +200,20 @@ template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile(
 __host__ __device__ inline int latent_stride(int width) { return (width / 8 + 1 - (width / 8) % 2) * 8; }
 static size_t latent_smem_bytes(int row_width) {
   const size_t st = latent_stride(row_width);
-  return (2 * LD_KT + 16) * st * 2 + 16 * (LD_KT + 8) * 2 + 16 * (LD_KT + 4) * 4 + 16 * 4 * 2;
+  return (2 * LD_KT + 16) * st * 2 + 16 * (LD_KT + 8) * 2 + 2 * 16 * (LD_KT + 4) * 4 + 16 * 4 * 2;
 }
 
-template <int NP>   // pairs of 8-wide column tiles per warp: rank <= 128 * NP
-__global__ void __launch_bounds__(LD_WARPS * 32) latent_attend_mma_kernel(LatentAttendParams p) {
+template <int NP>   // rank <= 128 NP, row_width <= 128 NP + 64
+__global__ void __launch_bounds__(LD_WARPS * 32, 1) latent_attend_mma_kernel(LatentAttendParams p) {
+  constexpr int KS = 4 * NP + 2;           // 16-column steps of half a row
+  constexpr int SW = LD_KT + 4;
   extern __shared__ __align__(16) uint8_t raw[];
   const int st = latent_stride(p.row_width), cols = p.row_width;
   __nv_bfloat16* kv = reinterpret_cast<__nv_bfloat16*>(raw);             // [2][KT][st]
   __nv_bfloat16* qs = kv + 2 * LD_KT * st;                               // [16][st]
   __nv_bfloat16* ps = qs + 16 * st;                                      // [16][KT + 8]
-  float* ss = reinterpret_cast<float*>(ps + 16 * (LD_KT + 8));           // [16][KT + 4]
-  float* s_alpha = ss + 16 * (LD_KT + 4);                                // [16]
+  float* ss = reinterpret_cast<float*>(ps + 16 * (LD_KT + 8));           // [2 halves][16][SW]
+  float* s_alpha = ss + 2 * 16 * SW;                                     // [16]
   float* s_l = s_alpha + 16;                                             // [16]
   const int row = blockIdx.x, h0 = blockIdx.y * 16, split = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -224,38 +227,51 @@ __global__ void __launch_bounds__(LD_WARPS * 32) latent_attend_mma_kernel(Latent
   const int vec = cols / 8;
   const int tiles = j1 > j0 ? (j1 - j0 + LD_KT - 1) / LD_KT : 0;
 
-  auto load_tile = [&](int i) {
+  auto load_tile = [&](int i) {   // warp w: rows w, w + 16, ...
     __nv_bfloat16* dst = kv + (i & 1) * LD_KT * st;
     const int base = j0 + i * LD_KT, n = min(LD_KT, j1 - base);
-    for (int x = threadIdx.x; x < LD_KT * vec; x += LD_WARPS * 32) {
-      const int r = x / vec, c = x - r * vec;
-      const int j = base + r;
+#pragma unroll
+    for (int u = 0; u < LD_KT / LD_WARPS; ++u) {
+      const int r = warp + u * LD_WARPS, j = base + r;
       if (r < n) {
         const long long slot = static_cast<long long>(bt[j / p.block_size]) * p.block_size + j % p.block_size;
-        cp_async16(smem_u32(dst + r * st + c * 8), cache + slot * cols + c * 8);
+        const __nv_bfloat16* src = cache + slot * cols;
+        for (int c = lane; c < vec; c += 32) cp_async16(smem_u32(dst + r * st + c * 8), src + c * 8);
       } else {
-        *reinterpret_cast<uint4*>(dst + r * st + c * 8) = make_uint4(0u, 0u, 0u, 0u);   // keeps 0 * x finite
+        for (int c = lane; c < vec; c += 32)       // zero rows keep 0 * x finite
+          *reinterpret_cast<uint4*>(dst + r * st + c * 8) = make_uint4(0u, 0u, 0u, 0u);
       }
     }
     cp_async_commit();
   };
   if (tiles > 0) load_tile(0);
-  // the 16 query rows: [q_lat | q_rot | 0]
-  for (int x = threadIdx.x; x < 16 * cols; x += LD_WARPS * 32) {
-    const int r = x / cols, c = x - r * cols, h = h0 + r;
-    __nv_bfloat16 v = __float2bfloat16(0.f);
-    if (h < p.H) {
-      if (c < p.rank) v = ql[h * p.rank + c];
-      else if (c < p.rank + p.rot) v = qr[h * (p.dim + p.rot) + p.dim + c - p.rank];
+  {   // the 16 query rows, one per warp: [q_lat | q_rot | 0]
+    const int h = h0 + warp;
+    for (int c = lane; c < cols; c += 32) {
+      __nv_bfloat16 v = __float2bfloat16(0.f);
+      if (h < p.H) {
+        if (c < p.rank) v = ql[h * p.rank + c];
+        else if (c < p.rank + p.rot) v = qr[h * (p.dim + p.rot) + p.dim + c - p.rank];
+      }
+      qs[warp * st + c] = v;
     }
-    qs[r * st + c] = v;
   }
-  float o[2 * NP][4];
+  __syncthreads();
+  // columns in 16-wide steps: this warp's half
+  const int steps = cols / 16, half0 = (steps + 1) / 2;
+  const int k_first = (warp >> 3) ? half0 : 0, k_count = (warp >> 3) ? steps - half0 : half0;
+  uint32_t qf[KS][4];
 #pragma unroll
-  for (int i = 0; i < 2 * NP; ++i)
+  for (int k = 0; k < KS; ++k) {
+    qf[k][0] = qf[k][1] = qf[k][2] = qf[k][3] = 0u;
+    if (k < k_count) ldsm_x4(qf[k], smem_u32(qs + (lane & 15) * st + (lane >> 4) * 8 + (k_first + k) * 16));
+  }
+  float o[NP][4];
+#pragma unroll
+  for (int i = 0; i < NP; ++i)
 #pragma unroll
     for (int q = 0; q < 4; ++q) o[i][q] = 0.f;
-  float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+  float m_run = -INFINITY, l_run = 0.f;
   const float sl = p.scale * 1.4426950408889634f;
   const int gid = lane >> 2, tig = lane & 3;
 
@@ -269,78 +285,68 @@ __global__ void __launch_bounds__(LD_WARPS * 32) latent_attend_mma_kernel(Latent
     }
     __syncthreads();
     const int n = min(LD_KT, j1 - (j0 + i * LD_KT));
-    {   // scores: four independent accumulators over the columns
-      float c[4][4];
+    {
+      float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
+      // 8 keys x 32 columns per load
+      const uint32_t ka = smem_u32(tile + ((warp & 7) * 8 + (lane & 7)) * st + (k_first * 16) + (lane >> 3) * 8);
 #pragma unroll
-      for (int u = 0; u < 4; ++u)
-#pragma unroll
-        for (int q = 0; q < 4; ++q) c[u][q] = 0.f;
-      const uint32_t qa = smem_u32(qs + (lane & 15) * st + (lane >> 4) * 8);
-      const uint32_t ka = smem_u32(tile + (warp * 8 + (lane & 7)) * st + (lane >> 3) * 8);
-      int k = 0;
-      for (; k + 64 <= cols; k += 64) {
-#pragma unroll
-        for (int u = 0; u < 2; ++u) {
-          uint32_t a0[4], a1[4], b[4];
-          ldsm_x4(a0, qa + (k + u * 32) * 2);
-          ldsm_x4(a1, qa + (k + u * 32 + 16) * 2);
-          ldsm_x4(b, ka + (k + u * 32) * 2);       // 8 keys x 32 columns
-          mma_16816(c[2 * u], a0, b[0], b[1]);
-          mma_16816(c[2 * u + 1], a1, b[2], b[3]);
+      for (int k = 0; k < KS; k += 2) {
+        if (k + 1 < k_count) {
+          uint32_t b[4];
+          ldsm_x4(b, ka + k * 32);
+          mma_16816(c0, qf[k], b[0], b[1]);
+          mma_16816(c1, qf[k + 1], b[2], b[3]);
+        } else if (k < k_count) {
+          uint32_t b0, b1;
+          asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];"
+                       : "=r"(b0), "=r"(b1)
+                       : "r"(smem_u32(tile + ((warp & 7) * 8 + (lane & 7)) * st + (k_first + k) * 16 + ((lane >> 3) & 1) * 8)));
+          mma_16816(c0, qf[k], b0, b1);
         }
       }
-      for (; k < cols; k += 16) {
-        uint32_t a0[4], b0, b1;
-        ldsm_x4(a0, qa + k * 2);
-        asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];"
-                     : "=r"(b0), "=r"(b1)
-                     : "r"(smem_u32(tile + (warp * 8 + (lane & 7)) * st + ((lane >> 3) & 1) * 8 + k)));
-        mma_16816(c[0], a0, b0, b1);
-      }
-      float* d = ss + gid * (LD_KT + 4) + warp * 8 + tig * 2;
-      d[0] = (c[0][0] + c[1][0]) + (c[2][0] + c[3][0]);
-      d[1] = (c[0][1] + c[1][1]) + (c[2][1] + c[3][1]);
-      d[8 * (LD_KT + 4)] = (c[0][2] + c[1][2]) + (c[2][2] + c[3][2]);
-      d[8 * (LD_KT + 4) + 1] = (c[0][3] + c[1][3]) + (c[2][3] + c[3][3]);
+      float* d = ss + (warp >> 3) * 16 * SW + gid * SW + (warp & 7) * 8 + tig * 2;
+      *reinterpret_cast<float2*>(d) = make_float2(c0[0] + c1[0], c0[1] + c1[1]);
+      *reinterpret_cast<float2*>(d + 8 * SW) = make_float2(c0[2] + c1[2], c0[3] + c1[3]);
     }
     __syncthreads();
-#pragma unroll
-    for (int u = 0; u < 2; ++u) {   // softmax of heads 2 warp, 2 warp + 1; two keys per lane
-      const int r = warp * 2 + u;
-      const float s0 = lane < n ? ss[r * (LD_KT + 4) + lane] * sl : -INFINITY;
-      const float s1 = lane + 32 < n ? ss[r * (LD_KT + 4) + lane + 32] * sl : -INFINITY;
-      const float m_new = fmaxf(m_run[u], warp_max(fmaxf(s0, s1)));   // n >= 1: finite
-      const float alpha = exp2f(m_run[u] - m_new);
+    {   // softmax of head `warp`; two keys per lane
+      const float* a = ss + warp * SW;
+      const float* b = a + 16 * SW;
+      const float s0 = lane < n ? (a[lane] + b[lane]) * sl : -INFINITY;
+      const float s1 = lane + 32 < n ? (a[lane + 32] + b[lane + 32]) * sl : -INFINITY;
+      const float m_new = fmaxf(m_run, warp_max(fmaxf(s0, s1)));   // n >= 1: finite
+      const float alpha = exp2f(m_run - m_new);
       const float p0 = exp2f(s0 - m_new), p1 = exp2f(s1 - m_new);
-      m_run[u] = m_new;
-      l_run[u] = l_run[u] * alpha + warp_sum(p0 + p1);
-      ps[r * (LD_KT + 8) + lane] = __float2bfloat16(p0);
-      ps[r * (LD_KT + 8) + lane + 32] = __float2bfloat16(p1);
-      if (lane == 0) s_alpha[r] = alpha;
+      m_run = m_new;
+      l_run = l_run * alpha + warp_sum(p0 + p1);
+      ps[warp * (LD_KT + 8) + lane] = __float2bfloat16(p0);
+      ps[warp * (LD_KT + 8) + lane + 32] = __float2bfloat16(p1);
+      if (lane == 0) s_alpha[warp] = alpha;
     }
     __syncthreads();
     {
-      const float al0 = s_alpha[gid], al1 = s_alpha[gid + 8];
       if (i > 0) {
+        const float al0 = s_alpha[gid], al1 = s_alpha[gid + 8];
 #pragma unroll
-        for (int x = 0; x < 2 * NP; ++x) {
+        for (int x = 0; x < NP; ++x) {
           o[x][0] *= al0; o[x][1] *= al0; o[x][2] *= al1; o[x][3] *= al1;
         }
       }
       const uint32_t pa = smem_u32(ps + (lane & 15) * (LD_KT + 8) + (lane >> 4) * 8);
 #pragma unroll
-      for (int kk = 0; kk < LD_KT / 16; ++kk) {
-        if (kk * 16 >= n) break;
-        uint32_t a[4];
-        ldsm_x4(a, pa + kk * 32);
+      for (int kk = 0; kk < LD_KT / 32; ++kk) {
+        if (kk * 32 >= n) break;
+        uint32_t a0[4], a1[4];
+        ldsm_x4(a0, pa + kk * 64);
+        ldsm_x4(a1, pa + kk * 64 + 32);
 #pragma unroll
         for (int x = 0; x < NP; ++x) {
-          const int c0 = (warp * NP + x) * 16;
-          if (c0 < p.rank) {
-            uint32_t b[4];    // keys kk*16 .. +16 (two 8-row matrices) x columns c0 .. +16 (two), transposed
-            ldsm_x4_t(b, smem_u32(tile + (kk * 16 + (lane & 15)) * st + c0 + (lane >> 4) * 8));
-            mma_16816(o[2 * x], a, b[0], b[1]);
-            mma_16816(o[2 * x + 1], a, b[2], b[3]);
+          const int c = (warp * NP + x) * 8;
+          if (c < p.rank) {
+            uint32_t b[4];    // keys kk*32 .. +32 (four 8-row matrices) x columns c .. +8, transposed
+            ldsm_x4_t(b, smem_u32(tile + (kk * 32 + lane) * st + c));
+            mma_16816(o[x], a0, b[0], b[1]);
+            mma_16816(o[x], a1, b[2], b[3]);
           }
         }
       }
@@ -348,17 +354,11 @@ __global__ void __launch_bounds__(LD_WARPS * 32) latent_attend_mma_kernel(Latent
     __syncthreads();   // the tile's buffer, ps and ss are free again
   }
   if (lane == 0) {
-    s_l[warp * 2] = l_run[0];
-    s_l[warp * 2 + 1] = l_run[1];
-    if (p.splits > 1) {
-#pragma unroll
-      for (int u = 0; u < 2; ++u) {
-        const int h = h0 + warp * 2 + u;
-        if (h < p.H)
-          p.part_lse[(static_cast<long long>(row) * p.H + h) * p.splits + split] =
-              l_run[u] > 0.f ? (m_run[u] + log2f(l_run[u])) * 0.6931471805599453f : -INFINITY;
-      }
-    }
+    s_l[warp] = l_run;
+    const int h = h0 + warp;
+    if (p.splits > 1 && h < p.H)
+      p.part_lse[(static_cast<long long>(row) * p.H + h) * p.splits + split] =
+          l_run > 0.f ? (m_run + log2f(l_run)) * 0.6931471805599453f : -INFINITY;
   }
   __syncthreads();
 #pragma unroll
@@ -368,8 +368,8 @@ __global__ void __launch_bounds__(LD_WARPS * 32) latent_attend_mma_kernel(Latent
     const float inv = s_l[r] > 0.f ? 1.f / s_l[r] : 0.f;
     const long long base = static_cast<long long>(row) * p.H + h;
 #pragma unroll
-    for (int x = 0; x < 2 * NP; ++x) {
-      const int c = (warp * NP + (x >> 1)) * 16 + (x & 1) * 8 + tig * 2;
+    for (int x = 0; x < NP; ++x) {
+      const int c = (warp * NP + x) * 8 + tig * 2;
       if (c < p.rank) {
         const float v0 = o[x][2 * half] * inv, v1 = o[x][2 * half + 1] * inv;
         if (p.splits == 1)
@@ -418,19 +418,39 @@ extern "C" int ts_latent_gather(const void* cache, const long long* slots, void*
   return (int)cudaGetLastError();
 }
 
+static int latent_mma_np(int rank, int row_width) {
+  const int by_rank = (rank + 127) / 128, by_row = (row_width - 64 + 127) / 128;
+  return by_rank > by_row ? by_rank : by_row;
+}
 static int latent_mma_fits(int rank, int row_width, int fp32) {
-  return !fp32 && rank % 16 == 0 && rank <= 512 && row_width % 16 == 0 && latent_smem_bytes(row_width) <= 227 * 1024;
+  return !fp32 && rank % 16 == 0 && row_width % 16 == 0 && latent_mma_np(rank, row_width) <= 4 &&
+         latent_smem_bytes(row_width) <= 227 * 1024;
 }
 
-// Number of CTAs a window is split over: enough to fill the GPU, no more than there are tiles.
+// Number of CTAs a row's window is split over.
 extern "C" int ts_latent_splits(int rows, int H, int rank, int row_width, int max_keys, int fp32) {
-  const int mma = latent_mma_fits(rank, row_width, fp32);
-  const long long units = static_cast<long long>(rows) * (mma ? (H + 15) / 16 : H);
-  const int unit_keys = mma ? LD_KT : 256;
-  const int most = (max_keys + unit_keys - 1) / unit_keys;
+  if (latent_mma_fits(rank, row_width, fp32)) {
+    // one CTA per SM at a time: rounds x (tiles of a CTA + a fixed start-up cost of about one tile), and a merge
+    const long long units = static_cast<long long>(rows) * ((H + 15) / 16);
+    const int tiles = (max_keys + LD_KT - 1) / LD_KT;
+    int best = 1;
+    long long cost = -1;
+    for (int s = 1; s <= tiles && s <= 64; ++s) {
+      const int per = (tiles + s - 1) / s;
+      if (s > 1 && (tiles + per - 1) / per != s) continue;     // some CTAs would get no tile
+      const long long c = (units * s + sm_count() - 1) / sm_count() * (per + 1) + (s > 1 ? 1 : 0);
+      if (cost < 0 || c < cost) {
+        cost = c;
+        best = s;
+      }
+    }
+    return best;
+  }
+  const long long units = static_cast<long long>(rows) * H;
+  const int most = (max_keys + 255) / 256;
   long long s = (2ll * sm_count() + units - 1) / units;
   if (s > most) s = most;
-  if (!mma && s < (max_keys + 2047) / 2048) s = (max_keys + 2047) / 2048;   // the chunk's scores sit in shared memory
+  if (s < (max_keys + 2047) / 2048) s = (max_keys + 2047) / 2048;   // the chunk's scores sit in shared memory
   return (int)(s < 1 ? 1 : s);
 }
 
@@ -454,7 +474,7 @@ extern "C" int ts_latent_attend(const void* q_lat, const void* q, long long q_ld
     p.chunk = (tiles + splits - 1) / splits * LD_KT;
     const size_t sm = latent_smem_bytes(row_width);
     const dim3 grid(rows, (H + 15) / 16, splits);
-    const int np = (rank + 127) / 128;
+    const int np = latent_mma_np(rank, row_width);
 #define TS_LATENT(N)                                                                                             \
   {                                                                                                              \
     static bool configured = false;                                                                              \
@@ -466,7 +486,7 @@ extern "C" int ts_latent_attend(const void* q_lat, const void* q, long long q_ld
     }                                                                                                            \
     latent_attend_mma_kernel<N><<<grid, LD_WARPS * 32, sm, st>>>(p);                                             \
   }
-    if (np == 1) TS_LATENT(1)
+    if (np <= 1) TS_LATENT(1)
     else if (np == 2) TS_LATENT(2)
     else if (np == 3) TS_LATENT(3)
     else TS_LATENT(4)

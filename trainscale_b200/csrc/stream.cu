@@ -85,7 +85,7 @@ template <> struct VecIO<__nv_bfloat16> {
 };
 
 template <typename T, int MODE, int V, int NV>
-__global__ void __launch_bounds__(V == 4 ? 256 : 1024)
+__global__ void __launch_bounds__(V == 4 ? 512 : 1024)
 stream_kernel(StreamParams p) {
   __shared__ float scratch[32];
   const int W = p.W, nvec = W / V;
@@ -150,18 +150,15 @@ stream_kernel(StreamParams p) {
         }
       }
     }
+    // every load of the history is issued before the first store of the row
+    constexpr int UN = NV == 1 ? 8 : (NV == 2 ? 4 : 2);
+    float acc[NV][V];
     const float an = p.dwa[p.n_hist];
 #pragma unroll
-    for (int i = 0; i < NV; ++i) {
-      const int c = threadIdx.x + i * blockDim.x;
-      if (c < nvec) {
-        if (keep && MODE == STREAM_LAYER)
-          VecIO<float>::store<V>(p.hist + p.n_hist * p.hist_stride + base + c * V, v[i]);
+    for (int i = 0; i < NV; ++i)
 #pragma unroll
-        for (int q = 0; q < V; ++q) v[i][q] *= an;
-      }
-    }
-#pragma unroll 4
+      for (int q = 0; q < V; ++q) acc[i][q] = an * v[i][q];
+#pragma unroll UN
     for (int j = 0; j < p.n_hist; ++j) {
       const float aj = p.dwa[j];
       const float* src = p.hist + j * p.hist_stride + base;
@@ -172,16 +169,19 @@ stream_kernel(StreamParams p) {
           float a[V];
           VecIO<float>::load<V>(src + c * V, a);
 #pragma unroll
-          for (int q = 0; q < V; ++q) v[i][q] += aj * a[q];
+          for (int q = 0; q < V; ++q) acc[i][q] += aj * a[q];
         }
       }
     }
-    if (keep && MODE == STREAM_LAYER) {
 #pragma unroll
-      for (int i = 0; i < NV; ++i) {
-        const int c = threadIdx.x + i * blockDim.x;
-        if (c < nvec) VecIO<float>::store<V>(p.x_out + base + c * V, v[i]);
+    for (int i = 0; i < NV; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c < nvec && keep && MODE == STREAM_LAYER) {
+        VecIO<float>::store<V>(p.hist + p.n_hist * p.hist_stride + base + c * V, v[i]);
+        VecIO<float>::store<V>(p.x_out + base + c * V, acc[i]);
       }
+#pragma unroll
+      for (int q = 0; q < V; ++q) v[i][q] = acc[i][q];
     }
   };
 
@@ -254,7 +254,7 @@ stream_kernel(StreamParams p) {
 template <typename T, int MODE>
 static int launch_stream(StreamParams p, cudaStream_t st) {
   const bool vec = p.W % 4 == 0 && p.mixer_ld % 4 == 0;
-  const int nvec = vec ? p.W / 4 : p.W, cap = vec ? 256 : 1024;
+  const int nvec = vec ? p.W / 4 : p.W, cap = vec ? 512 : 1024;
   int threads = (nvec + 31) / 32 * 32;
   if (threads > cap) threads = cap;
   const int nv = (nvec + threads - 1) / threads;
@@ -262,7 +262,7 @@ static int launch_stream(StreamParams p, cudaStream_t st) {
   p.rows_per_cta = 1;
   if (MODE != STREAM_FINAL) {
     // runs of rows amortise the halo once the grid fills the GPU anyway
-    int r = p.n_rows / (sm_count() * 6);
+    int r = p.n_rows / (sm_count() * 4);
     p.rows_per_cta = r < 1 ? 1 : (r > 16 ? 16 : r);
     grid = (p.n_rows + p.rows_per_cta - 1) / p.rows_per_cta;
   }
