@@ -251,35 +251,43 @@ stream_kernel(StreamParams p) {
   }
 }
 
+template <typename T, int MODE, int V, int NV>
+static int launch_stream_nv(StreamParams p, int threads, cudaStream_t st) {
+  int grid = p.n_rows;
+  p.rows_per_cta = 1;
+  if (MODE != STREAM_FINAL) {
+    // one wave: every resident CTA walks an equal run of rows (longer runs, fewer halo rows)
+    static int per_sm[33] = {};
+    int& occ = per_sm[threads / 32];
+    if (occ == 0 && (cudaOccupancyMaxActiveBlocksPerMultiprocessor(&occ, stream_kernel<T, MODE, V, NV>, threads, 0) !=
+                         cudaSuccess || occ < 1))
+      occ = 1;
+    const int slots = occ * sm_count();
+    p.rows_per_cta = (p.n_rows + slots - 1) / slots;
+    if (p.rows_per_cta > 32) p.rows_per_cta = 32;
+    grid = (p.n_rows + p.rows_per_cta - 1) / p.rows_per_cta;
+  }
+  stream_kernel<T, MODE, V, NV><<<grid, threads, 0, st>>>(p);
+  return (int)cudaGetLastError();
+}
+
 template <typename T, int MODE>
-static int launch_stream(StreamParams p, cudaStream_t st) {
+static int launch_stream(const StreamParams& p, cudaStream_t st) {
   const bool vec = p.W % 4 == 0 && p.mixer_ld % 4 == 0;
   const int nvec = vec ? p.W / 4 : p.W, cap = vec ? 512 : 1024;
   int threads = (nvec + 31) / 32 * 32;
   if (threads > cap) threads = cap;
   const int nv = (nvec + threads - 1) / threads;
-  int grid = p.n_rows;
-  p.rows_per_cta = 1;
-  if (MODE != STREAM_FINAL) {
-    // runs of rows amortise the halo once the grid fills the GPU anyway
-    int r = p.n_rows / (sm_count() * 4);
-    p.rows_per_cta = r < 1 ? 1 : (r > 16 ? 16 : r);
-    grid = (p.n_rows + p.rows_per_cta - 1) / p.rows_per_cta;
-  }
-#define TS_STREAM(V, NV) stream_kernel<T, MODE, V, NV><<<grid, threads, 0, st>>>(p)
   if (vec) {
-    if (nv <= 1) TS_STREAM(4, 1);
-    else if (nv <= 2) TS_STREAM(4, 2);
-    else if (nv <= 4) TS_STREAM(4, 4);
-    else if (nv <= 8) TS_STREAM(4, 8);
-    else return -11;
-  } else {
-    if (nv <= 1) TS_STREAM(1, 1);
-    else if (nv <= 8) TS_STREAM(1, 8);
-    else return -11;
+    if (nv <= 1) return launch_stream_nv<T, MODE, 4, 1>(p, threads, st);
+    if (nv <= 2) return launch_stream_nv<T, MODE, 4, 2>(p, threads, st);
+    if (nv <= 4) return launch_stream_nv<T, MODE, 4, 4>(p, threads, st);
+    if (nv <= 8) return launch_stream_nv<T, MODE, 4, 8>(p, threads, st);
+    return -11;
   }
-#undef TS_STREAM
-  return (int)cudaGetLastError();
+  if (nv <= 1) return launch_stream_nv<T, MODE, 1, 1>(p, threads, st);
+  if (nv <= 8) return launch_stream_nv<T, MODE, 1, 8>(p, threads, st);
+  return -11;
 }
 
 }  // namespace ts
