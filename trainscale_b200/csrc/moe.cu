@@ -13,35 +13,43 @@ namespace ts {
 
 constexpr int MOE_THREADS = 256;
 
-// grid = E.  Block e walks ids in order and gives the i-th occurrence of e rank i: a stable, deterministic order.
+// grid = E.  Block e walks ids in order and gives the i-th occurrence of e rank i: a stable, deterministic order.  Every
+// thread takes MOE_ITEMS consecutive slots per pass, so a pass costs two barriers for thousands of slots.
+constexpr int MOE_ITEMS = 16;
 __global__ void __launch_bounds__(MOE_THREADS) moe_rank_kernel(const int* __restrict__ ids, int n, int* __restrict__ rank,
                                                                int* __restrict__ counts) {
-  __shared__ int warp_tot[MOE_THREADS / 32];
-  __shared__ int running_s;
+  __shared__ int warp_tot[2][MOE_THREADS / 32];
   const int e = blockIdx.x;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  if (threadIdx.x == 0) running_s = 0;
-  __syncthreads();
-  for (int base = 0; base < n; base += MOE_THREADS) {
-    const int i = base + threadIdx.x;
-    const bool hit = (i < n) && (ids[i] == e);
-    const unsigned m = __ballot_sync(0xffffffffu, hit);
-    const int pre = __popc(m & ((1u << lane) - 1u));
-    if (lane == 0) warp_tot[warp] = __popc(m);
+  int run = 0, buf = 0;
+  for (int base = 0; base < n; base += MOE_THREADS * MOE_ITEMS, buf ^= 1) {
+    const int i0 = base + threadIdx.x * MOE_ITEMS;
+    unsigned hits = 0;
+#pragma unroll
+    for (int j = 0; j < MOE_ITEMS; ++j)
+      if (i0 + j < n && ids[i0 + j] == e) hits |= 1u << j;
+    const int mine = __popc(hits);
+    int inc = mine;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int up = __shfl_up_sync(0xffffffffu, inc, o);
+      if (lane >= o) inc += up;
+    }
+    if (lane == 31) warp_tot[buf][warp] = inc;
     __syncthreads();
-    int woff = 0, tot = 0;
+    int at = run + inc - mine;
 #pragma unroll
     for (int w = 0; w < MOE_THREADS / 32; ++w) {
-      if (w < warp) woff += warp_tot[w];
-      tot += warp_tot[w];
+      if (w < warp) at += warp_tot[buf][w];
+      run += warp_tot[buf][w];
     }
-    const int run = running_s;
-    if (hit) rank[i] = run + woff + pre;
-    __syncthreads();
-    if (threadIdx.x == 0) running_s = run + tot;
-    __syncthreads();
+    while (hits) {
+      const int j = __ffs(hits) - 1;
+      hits &= hits - 1;
+      rank[i0 + j] = at++;
+    }
   }
-  if (threadIdx.x == 0) counts[e] = running_s;
+  if (threadIdx.x == 0) counts[e] = run;
 }
 
 // one block: seg_start[e] = 128-aligned exclusive scan of counts; tile_expert[t] = expert owning rows [128t, 128t+128)

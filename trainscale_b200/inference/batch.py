@@ -107,6 +107,11 @@ class StepBatch:
     _contexts: dict = field(default_factory=dict)
 
     @property
+    def captured(self) -> bool:
+        """A decode step that is (being) recorded as a CUDA graph over static buffers."""
+        return self.host is None
+
+    @property
     def num_tokens(self) -> int:
         return self.token_ids.shape[0]
 

@@ -180,6 +180,7 @@ class MezilixForCausalLM(nn.Module):
         self.layers = nn.ModuleList(MezilixLayer(cfg, i) for i in range(cfg.num_hidden_layers))
         self.final_norm = nn.Parameter(torch.empty((), dtype=torch.float32), requires_grad=False)
         self.head = nn.Parameter(torch.empty(cfg.vocab_size, W), requires_grad=False)
+        self._side = None                 # stream of the experts in captured decode steps
 
     # ---------------------------------------------------------------- weights
     @torch.no_grad()
@@ -245,6 +246,11 @@ class MezilixForCausalLM(nn.Module):
         return CacheSpec([{"latent": (l.mixer.row_width,)} for l in self.layers],
                          [self.config.hidden_size] * len(self.layers))
 
+    def _side_stream(self) -> "torch.cuda.Stream":
+        if self._side is None:
+            self._side = torch.cuda.Stream(device=self.embed.device)
+        return self._side
+
     @torch.no_grad()
     def serve(self, batch, cache, observe=None) -> torch.Tensor:
         """Final-norm hidden state of the batch's wanted rows.  `observe(n, x)`: called with the stream after layer n."""
@@ -258,8 +264,17 @@ class MezilixForCausalLM(nn.Module):
                              first.norm1, cfg.eps, first.shift, rows, cache.state[0])
         x = hist[0]
         for i, layer in enumerate(self.layers):
-            mixer = layer.mix(hs, batch, cache.entries[i]["latent"], row_len, cfg.eps)
-            experts = layer.feed_forward(h)
+            if batch.captured and layer.mlp is not None:
+                # a decode step is a chain of short kernels: mixer and experts of the parallel block run side by side
+                main, side = torch.cuda.current_stream(), self._side_stream()
+                side.wait_stream(main)
+                with torch.cuda.stream(side):
+                    experts = layer.feed_forward(h)
+                mixer = layer.mix(hs, batch, cache.entries[i]["latent"], row_len, cfg.eps)
+                main.wait_stream(side)
+            else:
+                mixer = layer.mix(hs, batch, cache.entries[i]["latent"], row_len, cfg.eps)
+                experts = layer.feed_forward(h)
             if i + 1 == L:
                 break
             nxt = self.layers[i + 1]
