@@ -89,7 +89,7 @@ struct LatentAttendParams {
   void* out;                  // [rows][H][rank]
   float* part_out;            // [rows][H][splits][rank]
   float* part_lse;            // [rows][H][splits]
-  int rows, H, dim, rot, rank, row_width, max_blocks, block_size, window, chunk, splits;
+  int rows, H, dim, rot, rank, row_width, max_blocks, block_size, block_shift, window, chunk, splits;
   float scale;
 };
 
@@ -164,15 +164,18 @@ __global__ void latent_merge_kernel(LatentAttendParams p) {
 }
 
 // ---------------------------------------------------------------------------------------------------------
-// bf16 decode kernel.  grid (rows, ceil(H / 16), splits), 16 warps.  Tiles of KT cached rows stream through two
-// shared-memory buffers (cp.async); a tile serves as K (all row_width columns) and as V (the first rank columns).
-//   scores   warp w: the 16 heads x keys [8 (w % 8), + 8) of the tile, over half w / 8 of the columns; the query fragments
-//            of that half stay in registers for the whole kernel
-//   softmax  warp w: head w (running max and sum in registers, fp32)
+// bf16 decode kernel.  grid (rows, ceil(H / 16), splits), 16 warps.  Tiles of 32 cached rows stream through a ring of
+// shared-memory stages (cp.async, one group per tile); a tile serves as K (all row_width columns) and as V (the first rank
+// columns).
+//   scores   warp w: the 16 heads x keys [8 (w % 4), + 8) of the tile, over quarter w / 4 of the columns; the query
+//            fragments of that quarter stay in registers for the whole kernel
+//   softmax  warp w: head w, one key per lane (running max and sum in registers, fp32)
 //   output   warp w: latent columns [8 NP w, 8 NP (w + 1)) of the 16 heads, fp32 accumulators in registers
+// Three barriers per tile; a stage is refilled after the first barrier of the next tile, when every warp is past its use.
 // ---------------------------------------------------------------------------------------------------------
 constexpr int LD_WARPS = 16;
-constexpr int LD_KT = 64;
+constexpr int LD_KT = 32;
+constexpr int LD_STAGES = 4;
 
 __device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], uint32_t addr) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
@@ -191,29 +194,29 @@ __device__ __forceinline__ void mma_16816(float (&c)[4], const uint32_t (&a)[4],
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src));
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
 }
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;"); }
-template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N)); }
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
 // shared-memory row stride in elements: an odd number of 16-byte units, so that ldmatrix rows hit different banks
 __host__ __device__ inline int latent_stride(int width) { return (width / 8 + 1 - (width / 8) % 2) * 8; }
 static size_t latent_smem_bytes(int row_width) {
   const size_t st = latent_stride(row_width);
-  return (2 * LD_KT + 16) * st * 2 + 16 * (LD_KT + 8) * 2 + 2 * 16 * (LD_KT + 4) * 4 + 16 * 4 * 2;
+  return (LD_STAGES * LD_KT + 16) * st * 2 + 16 * (LD_KT + 8) * 2 + 4 * 16 * (LD_KT + 4) * 4 + 16 * 4 * 2;
 }
 
 template <int NP>   // rank <= 128 NP, row_width <= 128 NP + 64
 __global__ void __launch_bounds__(LD_WARPS * 32, 1) latent_attend_mma_kernel(LatentAttendParams p) {
-  constexpr int KS = 4 * NP + 2;           // 16-column steps of half a row
+  constexpr int KS = 2 * NP + 1;           // 16-column steps of a quarter of a row
   constexpr int SW = LD_KT + 4;
   extern __shared__ __align__(16) uint8_t raw[];
   const int st = latent_stride(p.row_width), cols = p.row_width;
-  __nv_bfloat16* kv = reinterpret_cast<__nv_bfloat16*>(raw);             // [2][KT][st]
-  __nv_bfloat16* qs = kv + 2 * LD_KT * st;                               // [16][st]
+  __nv_bfloat16* kv = reinterpret_cast<__nv_bfloat16*>(raw);             // [STAGES][KT][st]
+  __nv_bfloat16* qs = kv + LD_STAGES * LD_KT * st;                       // [16][st]
   __nv_bfloat16* ps = qs + 16 * st;                                      // [16][KT + 8]
-  float* ss = reinterpret_cast<float*>(ps + 16 * (LD_KT + 8));           // [2 halves][16][SW]
-  float* s_alpha = ss + 2 * 16 * SW;                                     // [16]
+  float* ss = reinterpret_cast<float*>(ps + 16 * (LD_KT + 8));           // [4 quarters][16][SW]
+  float* s_alpha = ss + 4 * 16 * SW;                                     // [16]
   float* s_l = s_alpha + 16;                                             // [16]
   const int row = blockIdx.x, h0 = blockIdx.y * 16, split = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -224,27 +227,7 @@ __global__ void __launch_bounds__(LD_WARPS * 32, 1) latent_attend_mma_kernel(Lat
   const __nv_bfloat16* cache = reinterpret_cast<const __nv_bfloat16*>(p.cache);
   const __nv_bfloat16* ql = reinterpret_cast<const __nv_bfloat16*>(p.q_lat) + static_cast<long long>(row) * p.H * p.rank;
   const __nv_bfloat16* qr = reinterpret_cast<const __nv_bfloat16*>(p.q) + row * p.q_ld;
-  const int vec = cols / 8;
   const int tiles = j1 > j0 ? (j1 - j0 + LD_KT - 1) / LD_KT : 0;
-
-  auto load_tile = [&](int i) {   // warp w: rows w, w + 16, ...
-    __nv_bfloat16* dst = kv + (i & 1) * LD_KT * st;
-    const int base = j0 + i * LD_KT, n = min(LD_KT, j1 - base);
-#pragma unroll
-    for (int u = 0; u < LD_KT / LD_WARPS; ++u) {
-      const int r = warp + u * LD_WARPS, j = base + r;
-      if (r < n) {
-        const long long slot = static_cast<long long>(bt[j / p.block_size]) * p.block_size + j % p.block_size;
-        const __nv_bfloat16* src = cache + slot * cols;
-        for (int c = lane; c < vec; c += 32) cp_async16(smem_u32(dst + r * st + c * 8), src + c * 8);
-      } else {
-        for (int c = lane; c < vec; c += 32)       // zero rows keep 0 * x finite
-          *reinterpret_cast<uint4*>(dst + r * st + c * 8) = make_uint4(0u, 0u, 0u, 0u);
-      }
-    }
-    cp_async_commit();
-  };
-  if (tiles > 0) load_tile(0);
   {   // the 16 query rows, one per warp: [q_lat | q_rot | 0]
     const int h = h0 + warp;
     for (int c = lane; c < cols; c += 32) {
@@ -257,9 +240,46 @@ __global__ void __launch_bounds__(LD_WARPS * 32, 1) latent_attend_mma_kernel(Lat
     }
   }
   __syncthreads();
-  // columns in 16-wide steps: this warp's half
-  const int steps = cols / 16, half0 = (steps + 1) / 2;
-  const int k_first = (warp >> 3) ? half0 : 0, k_count = (warp >> 3) ? steps - half0 : half0;
+  // warp w loads rows w, w + 16 of a tile; the pages of its next rows (lane u: row u) are looked up one tile ahead and used
+  // no earlier, so the table's latency is off the path
+  constexpr int RPW = LD_KT / LD_WARPS;
+  constexpr int NC = (128 * NP + 64 + 255) / 256;      // 16-byte columns per lane
+  const int shift = p.block_shift, mask = p.block_size - 1;
+  int page = 0, j_look = j0 + warp + lane * LD_WARPS, j_load = j0 + warp;
+  const __nv_bfloat16* src0 = cache + lane * 8;
+  const uint32_t dst0 = smem_u32(kv + warp * st + lane * 8);
+  const uint32_t row_step = LD_WARPS * st * 2, tile_step = LD_KT * st * 2;
+  auto look_up = [&]() {
+    if (lane < RPW && j_look < j1) page = bt[j_look >> shift];
+    j_look += LD_KT;
+  };
+  auto load_tile = [&](int i) {
+    const uint32_t dst_t = dst0 + (i % LD_STAGES) * tile_step;
+#pragma unroll
+    for (int u = 0; u < RPW; ++u) {
+      const int j = j_load + u * LD_WARPS;
+      const int slot = (__shfl_sync(0xffffffffu, page, u) << shift) + (j & mask);
+      const __nv_bfloat16* src = src0 + static_cast<long long>(slot) * cols;
+      const uint32_t dst = dst_t + u * row_step;
+#pragma unroll
+      for (int k = 0; k < NC; ++k) {
+        if (lane + k * 32 < cols / 8) {
+          if (j < j1) cp_async16(dst + k * 512, src + k * 256);
+          else asm volatile("st.shared.v4.u32 [%0], {%1, %1, %1, %1};" ::"r"(dst + k * 512), "r"(0u) : "memory");
+        }                              // (zero rows past the range keep 0 * x finite)
+      }
+    }
+    j_load += LD_KT;
+    look_up();
+  };
+  look_up();
+  for (int i = 0; i < LD_STAGES - 1; ++i) {
+    if (i < tiles) load_tile(i);
+    cp_async_commit();
+  }
+  // columns in 16-wide steps: this warp's quarter
+  const int steps = cols / 16, per = (steps + 3) / 4;
+  const int k_first = (warp >> 2) * per, k_count = min(per, steps - k_first);      // may be <= 0 for narrow rows
   uint32_t qf[KS][4];
 #pragma unroll
   for (int k = 0; k < KS; ++k) {
@@ -271,59 +291,52 @@ __global__ void __launch_bounds__(LD_WARPS * 32, 1) latent_attend_mma_kernel(Lat
   for (int i = 0; i < NP; ++i)
 #pragma unroll
     for (int q = 0; q < 4; ++q) o[i][q] = 0.f;
-  float m_run = -INFINITY, l_run = 0.f;
+  float m_run = -INFINITY, l_lane = 0.f;
   const float sl = p.scale * 1.4426950408889634f;
   const int gid = lane >> 2, tig = lane & 3;
 
   for (int i = 0; i < tiles; ++i) {
-    const __nv_bfloat16* tile = kv + (i & 1) * LD_KT * st;
-    if (i + 1 < tiles) {
-      load_tile(i + 1);
-      cp_async_wait<1>();
-    } else {
-      cp_async_wait<0>();
-    }
-    __syncthreads();
+    const int s = i % LD_STAGES;
+    const __nv_bfloat16* tile = kv + s * LD_KT * st;
     const int n = min(LD_KT, j1 - (j0 + i * LD_KT));
+    cp_async_wait<LD_STAGES - 2>();
+    __syncthreads();                               // tile i is in; every warp is past tile i - 1
+    if (i + LD_STAGES - 1 < tiles) load_tile(i + LD_STAGES - 1);
+    cp_async_commit();
     {
       float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
-      // 8 keys x 32 columns per load
-      const uint32_t ka = smem_u32(tile + ((warp & 7) * 8 + (lane & 7)) * st + (k_first * 16) + (lane >> 3) * 8);
+      const uint32_t ka = smem_u32(tile + ((warp & 3) * 8 + (lane & 7)) * st + k_first * 16 + (lane >> 3) * 8);
 #pragma unroll
       for (int k = 0; k < KS; k += 2) {
-        if (k + 1 < k_count) {
+        if (k + 1 < KS && k + 1 < k_count) {
           uint32_t b[4];
-          ldsm_x4(b, ka + k * 32);
+          ldsm_x4(b, ka + k * 32);                 // 8 keys x 32 columns
           mma_16816(c0, qf[k], b[0], b[1]);
-          mma_16816(c1, qf[k + 1], b[2], b[3]);
+          mma_16816(c1, qf[k + 1 < KS ? k + 1 : k], b[2], b[3]);
         } else if (k < k_count) {
           uint32_t b0, b1;
           asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];"
                        : "=r"(b0), "=r"(b1)
-                       : "r"(smem_u32(tile + ((warp & 7) * 8 + (lane & 7)) * st + (k_first + k) * 16 + ((lane >> 3) & 1) * 8)));
+                       : "r"(smem_u32(tile + ((warp & 3) * 8 + (lane & 7)) * st + (k_first + k) * 16 + ((lane >> 3) & 1) * 8)));
           mma_16816(c0, qf[k], b0, b1);
         }
       }
-      float* d = ss + (warp >> 3) * 16 * SW + gid * SW + (warp & 7) * 8 + tig * 2;
+      float* d = ss + ((warp >> 2) * 16 + gid) * SW + (warp & 3) * 8 + tig * 2;
       *reinterpret_cast<float2*>(d) = make_float2(c0[0] + c1[0], c0[1] + c1[1]);
       *reinterpret_cast<float2*>(d + 8 * SW) = make_float2(c0[2] + c1[2], c0[3] + c1[3]);
     }
-    __syncthreads();
-    {   // softmax of head `warp`; two keys per lane
-      const float* a = ss + warp * SW;
-      const float* b = a + 16 * SW;
-      const float s0 = lane < n ? (a[lane] + b[lane]) * sl : -INFINITY;
-      const float s1 = lane + 32 < n ? (a[lane + 32] + b[lane + 32]) * sl : -INFINITY;
-      const float m_new = fmaxf(m_run, warp_max(fmaxf(s0, s1)));   // n >= 1: finite
-      const float alpha = exp2f(m_run - m_new);
-      const float p0 = exp2f(s0 - m_new), p1 = exp2f(s1 - m_new);
+    __syncthreads();                               // scores complete
+    {   // softmax of head `warp`, one key per lane
+      const float* a = ss + warp * SW + lane;
+      const float v = lane < n ? ((a[0] + a[16 * SW]) + (a[32 * SW] + a[48 * SW])) * sl : -INFINITY;
+      const float m_new = fmaxf(m_run, warp_max(v));   // n >= 1: finite
+      const float alpha = fast_ex2(m_run - m_new), w = fast_ex2(v - m_new);
       m_run = m_new;
-      l_run = l_run * alpha + warp_sum(p0 + p1);
-      ps[warp * (LD_KT + 8) + lane] = __float2bfloat16(p0);
-      ps[warp * (LD_KT + 8) + lane + 32] = __float2bfloat16(p1);
+      l_lane = l_lane * alpha + w;
+      ps[warp * (LD_KT + 8) + lane] = __float2bfloat16(w);
       if (lane == 0) s_alpha[warp] = alpha;
     }
-    __syncthreads();
+    __syncthreads();                               // weights complete
     {
       if (i > 0) {
         const float al0 = s_alpha[gid], al1 = s_alpha[gid + 8];
@@ -333,26 +346,22 @@ __global__ void __launch_bounds__(LD_WARPS * 32, 1) latent_attend_mma_kernel(Lat
         }
       }
       const uint32_t pa = smem_u32(ps + (lane & 15) * (LD_KT + 8) + (lane >> 4) * 8);
+      uint32_t a0[4], a1[4];
+      ldsm_x4(a0, pa);
+      ldsm_x4(a1, pa + 32);
 #pragma unroll
-      for (int kk = 0; kk < LD_KT / 32; ++kk) {
-        if (kk * 32 >= n) break;
-        uint32_t a0[4], a1[4];
-        ldsm_x4(a0, pa + kk * 64);
-        ldsm_x4(a1, pa + kk * 64 + 32);
-#pragma unroll
-        for (int x = 0; x < NP; ++x) {
-          const int c = (warp * NP + x) * 8;
-          if (c < p.rank) {
-            uint32_t b[4];    // keys kk*32 .. +32 (four 8-row matrices) x columns c .. +8, transposed
-            ldsm_x4_t(b, smem_u32(tile + (kk * 32 + lane) * st + c));
-            mma_16816(o[x], a0, b[0], b[1]);
-            mma_16816(o[x], a1, b[2], b[3]);
-          }
+      for (int x = 0; x < NP; ++x) {
+        const int c = (warp * NP + x) * 8;
+        if (c < p.rank) {
+          uint32_t b[4];    // 32 keys (four 8-row matrices) x columns c .. +8, transposed
+          ldsm_x4_t(b, smem_u32(tile + lane * st + c));
+          mma_16816(o[x], a0, b[0], b[1]);
+          mma_16816(o[x], a1, b[2], b[3]);
         }
       }
     }
-    __syncthreads();   // the tile's buffer, ps and ss are free again
   }
+  const float l_run = warp_sum(l_lane);
   if (lane == 0) {
     s_l[warp] = l_run;
     const int h = h0 + warp;
@@ -422,15 +431,16 @@ static int latent_mma_np(int rank, int row_width) {
   const int by_rank = (rank + 127) / 128, by_row = (row_width - 64 + 127) / 128;
   return by_rank > by_row ? by_rank : by_row;
 }
-static int latent_mma_fits(int rank, int row_width, int fp32) {
-  return !fp32 && rank % 16 == 0 && row_width % 16 == 0 && latent_mma_np(rank, row_width) <= 4 &&
+static int latent_mma_fits(int rank, int row_width, int block_size, int fp32) {
+  return !fp32 && (block_size & (block_size - 1)) == 0 && rank % 16 == 0 && row_width % 16 == 0 && latent_mma_np(rank, row_width) <= 4 &&
          latent_smem_bytes(row_width) <= 227 * 1024;
 }
 
 // Number of CTAs a row's window is split over.
-extern "C" int ts_latent_splits(int rows, int H, int rank, int row_width, int max_keys, int fp32) {
-  if (latent_mma_fits(rank, row_width, fp32)) {
-    // one CTA per SM at a time: rounds x (tiles of a CTA + a fixed start-up cost of about one tile), and a merge
+extern "C" int ts_latent_splits(int rows, int H, int rank, int row_width, int block_size, int max_keys,
+                                int fp32) {
+  if (latent_mma_fits(rank, row_width, block_size, fp32)) {
+    // one CTA per SM at a time: rounds x (tiles of a CTA + a start-up cost of about four tiles), and a merge
     const long long units = static_cast<long long>(rows) * ((H + 15) / 16);
     const int tiles = (max_keys + LD_KT - 1) / LD_KT;
     int best = 1;
@@ -438,7 +448,7 @@ extern "C" int ts_latent_splits(int rows, int H, int rank, int row_width, int ma
     for (int s = 1; s <= tiles && s <= 64; ++s) {
       const int per = (tiles + s - 1) / s;
       if (s > 1 && (tiles + per - 1) / per != s) continue;     // some CTAs would get no tile
-      const long long c = (units * s + sm_count() - 1) / sm_count() * (per + 1) + (s > 1 ? 1 : 0);
+      const long long c = (units * s + sm_count() - 1) / sm_count() * (per + 4) + (s > 1 ? 4 : 0);
       if (cost < 0 || c < cost) {
         cost = c;
         best = s;
@@ -468,8 +478,10 @@ extern "C" int ts_latent_attend(const void* q_lat, const void* q, long long q_ld
   p.row_len = row_len; p.out = out; p.part_out = part_out; p.part_lse = part_lse; p.rows = rows; p.H = H; p.dim = dim;
   p.rot = rot; p.rank = rank; p.row_width = row_width; p.max_blocks = max_blocks; p.block_size = block_size;
   p.window = window; p.splits = splits; p.scale = scale;
+  p.block_shift = 0;
+  while ((1 << p.block_shift) < block_size) ++p.block_shift;
   cudaStream_t st = ST(stream);
-  if (latent_mma_fits(rank, row_width, fp32)) {
+  if (latent_mma_fits(rank, row_width, block_size, fp32)) {
     const int tiles = (max_keys + LD_KT - 1) / LD_KT;
     p.chunk = (tiles + splits - 1) / splits * LD_KT;
     const size_t sm = latent_smem_bytes(row_width);

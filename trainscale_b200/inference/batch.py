@@ -123,6 +123,16 @@ class StepBatch:
     def q_lens(self) -> list[int]:
         return self.host.q_lens if self.host is not None else [1] * self.num_tokens
 
+    @property
+    def cu_q(self) -> torch.Tensor:
+        """int32 [sequences + 1]: first row of every sequence (uploaded once per step)."""
+        if "cu_q" not in self._contexts:
+            cu = [0]
+            for n in self.q_lens:
+                cu.append(cu[-1] + n)
+            self._contexts["cu_q"] = torch.tensor(cu, dtype=torch.int32).to(self.token_ids.device)
+        return self._contexts["cu_q"]
+
     def prompt_context(self, window: int) -> PromptContext | None:
         """Key rows of the multi-token entries when a position sees `window` keys (None: no such entries)."""
         if self.host is None or self.host.all_single:

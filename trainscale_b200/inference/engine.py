@@ -321,15 +321,14 @@ class ModelRunner:
         if self.cuda and fresh and D in (64, 128):
             # every sequence starts at position 0: packed-prompt flash attention
             from ..ops import flash
-            cu = torch.tensor([0] + list(torch.tensor(q_lens).cumsum(0).tolist()), dtype=torch.int32, device=self.device)
-            o, _ = flash.flash_forward_only(qkv2d.unsqueeze(0), Hq, Hkv, D, True, scale, cu, max(q_lens))
+            o, _ = flash.flash_forward_only(qkv2d.unsqueeze(0), Hq, Hkv, D, True, scale, batch.cu_q, max(q_lens))
             return o.view(T, Hq * D)
         if self.cuda and all(n == 1 for n in q_lens) and D in (64, 128):
             lib = _lib.load("decode")
             n = qkv2d.shape[0]
             chunk = 512
             if splits is None:       # (a captured decode passes the split count of its block-table width)
-                splits = max(1, -(-int(seq_lens.max().item()) // chunk))
+                splits = max(1, -(-batch.max_len // chunk))
             out = torch.empty(n, Hq * D, dtype=qkv2d.dtype, device=self.device)
             po = torch.empty(n, Hq, splits, D, dtype=torch.float32, device=self.device)
             pl = torch.empty(n, Hq, splits, dtype=torch.float32, device=self.device)

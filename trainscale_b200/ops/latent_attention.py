@@ -108,7 +108,7 @@ def attend_latent(q_lat: torch.Tensor, proj: torch.Tensor, s: LatentShape, cache
     lib = _lib.load("latent")
     fp32 = int(q_lat.dtype == torch.float32)
     keys = min(s.window, max_len)
-    splits = lib.ts_latent_splits(T, H, rank, s.row_width, keys, fp32)
+    splits = lib.ts_latent_splits(T, H, rank, s.row_width, bs, keys, fp32)
     out = torch.empty_like(q_lat)
     po = pl = None
     if splits > 1:
