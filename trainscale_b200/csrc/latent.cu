@@ -148,34 +148,45 @@ __global__ void __launch_bounds__(128) latent_attend_simt_kernel(LatentAttendPar
   if (p.splits > 1 && threadIdx.x == 0) p.part_lse[o * p.splits + split] = l > 0.f ? mx + logf(l) : -INFINITY;
 }
 
+constexpr int MERGE_MAX_SPLITS = 256;
 template <typename T>
-__global__ void latent_merge_kernel(LatentAttendParams p) {
+__global__ void __launch_bounds__(128) latent_merge_kernel(LatentAttendParams p) {
+  __shared__ float w[MERGE_MAX_SPLITS];
+  __shared__ float scratch[32];
   const long long o = static_cast<long long>(blockIdx.x) * p.H + blockIdx.y;
   const float* lse = p.part_lse + o * p.splits;
   float mx = -INFINITY, den = 0.f;
-  for (int s = 0; s < p.splits; ++s) mx = fmaxf(mx, lse[s]);
-  for (int s = 0; s < p.splits; ++s) den += lse[s] == -INFINITY ? 0.f : expf(lse[s] - mx);
+  for (int s = threadIdx.x; s < p.splits; s += blockDim.x) mx = fmaxf(mx, lse[s]);
+  mx = block_max(mx, scratch);
+  for (int s = threadIdx.x; s < p.splits; s += blockDim.x) {
+    w[s] = lse[s] == -INFINITY ? 0.f : expf(lse[s] - mx);
+    den += w[s];
+  }
+  den = block_sum(den, scratch);           // also orders the weights
+  const float inv = 1.f / den;
   for (int r = threadIdx.x; r < p.rank; r += blockDim.x) {
+    const float* part = p.part_out + o * p.splits * p.rank + r;
     float acc = 0.f;
-    for (int s = 0; s < p.splits; ++s)
-      if (lse[s] != -INFINITY) acc += expf(lse[s] - mx) * p.part_out[(o * p.splits + s) * p.rank + r];
-    reinterpret_cast<T*>(p.out)[o * p.rank + r] = from_f32<T>(acc / den);
+#pragma unroll 8
+    for (int s = 0; s < p.splits; ++s) acc += w[s] * part[static_cast<long long>(s) * p.rank];
+    reinterpret_cast<T*>(p.out)[o * p.rank + r] = from_f32<T>(acc * inv);
   }
 }
 
 // ---------------------------------------------------------------------------------------------------------
-// bf16 decode kernel.  grid (rows, ceil(H / 16), splits), 16 warps.  Tiles of 32 cached rows stream through a ring of
-// shared-memory stages (cp.async, one group per tile); a tile serves as K (all row_width columns) and as V (the first rank
-// columns).
+// bf16 decode kernel.  grid (rows, ceil(H / 16), splits), 16 compute warps and 4 loader warps.  Tiles of 32 cached rows
+// stream through a ring of shared-memory stages (one bulk copy per row, full / empty mbarriers per stage); a tile serves as
+// K (all row_width columns) and as V (the first rank columns).
 //   scores   warp w: the 16 heads x keys [8 (w % 4), + 8) of the tile, over quarter w / 4 of the columns; the query
 //            fragments of that quarter stay in registers for the whole kernel
 //   softmax  warp w: head w, one key per lane (running max and sum in registers, fp32)
 //   output   warp w: latent columns [8 NP w, 8 NP (w + 1)) of the 16 heads, fp32 accumulators in registers
-// Three barriers per tile; a stage is refilled after the first barrier of the next tile, when every warp is past its use.
+// Two barriers among the compute warps per tile.
 // ---------------------------------------------------------------------------------------------------------
 constexpr int LD_WARPS = 16;
 constexpr int LD_KT = 32;
 constexpr int LD_STAGES = 4;
+constexpr int LD_LOADERS = 4;
 
 __device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], uint32_t addr) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
@@ -193,21 +204,25 @@ __device__ __forceinline__ void mma_16816(float (&c)[4], const uint32_t (&a)[4],
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+// one contiguous row, global -> shared; both 16-byte aligned, size a multiple of 16
+__device__ __forceinline__ void bulk_load(uint32_t dst, const void* src, uint32_t bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst),
+               "l"(src), "r"(bytes), "r"(smem_u32(bar))
+               : "memory");
 }
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+__device__ __forceinline__ void compute_barrier() {
+  asm volatile("bar.sync 1, %0;" ::"n"(LD_WARPS * 32) : "memory");
+}
 
 // shared-memory row stride in elements: an odd number of 16-byte units, so that ldmatrix rows hit different banks
 __host__ __device__ inline int latent_stride(int width) { return (width / 8 + 1 - (width / 8) % 2) * 8; }
 static size_t latent_smem_bytes(int row_width) {
   const size_t st = latent_stride(row_width);
-  return (LD_STAGES * LD_KT + 16) * st * 2 + 16 * (LD_KT + 8) * 2 + 4 * 16 * (LD_KT + 4) * 4 + 16 * 4 * 2;
+  return (LD_STAGES * LD_KT + 16) * st * 2 + 16 * (LD_KT + 8) * 2 + 4 * 16 * (LD_KT + 4) * 4 + 16 * 4 * 2 + 2 * LD_STAGES * 8;
 }
 
 template <int NP>   // rank <= 128 NP, row_width <= 128 NP + 64
-__global__ void __launch_bounds__(LD_WARPS * 32, 1) latent_attend_mma_kernel(LatentAttendParams p) {
+__global__ void __launch_bounds__((LD_WARPS + LD_LOADERS) * 32, 1) latent_attend_mma_kernel(LatentAttendParams p) {
   constexpr int KS = 2 * NP + 1;           // 16-column steps of a quarter of a row
   constexpr int SW = LD_KT + 4;
   extern __shared__ __align__(16) uint8_t raw[];
@@ -218,6 +233,8 @@ __global__ void __launch_bounds__(LD_WARPS * 32, 1) latent_attend_mma_kernel(Lat
   float* ss = reinterpret_cast<float*>(ps + 16 * (LD_KT + 8));           // [4 quarters][16][SW]
   float* s_alpha = ss + 4 * 16 * SW;                                     // [16]
   float* s_l = s_alpha + 16;                                             // [16]
+  uint64_t* full = reinterpret_cast<uint64_t*>(s_l + 16);                // [STAGES]
+  uint64_t* empty = full + LD_STAGES;                                    // [STAGES]
   const int row = blockIdx.x, h0 = blockIdx.y * 16, split = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   int j0, j1;
@@ -228,54 +245,57 @@ __global__ void __launch_bounds__(LD_WARPS * 32, 1) latent_attend_mma_kernel(Lat
   const __nv_bfloat16* ql = reinterpret_cast<const __nv_bfloat16*>(p.q_lat) + static_cast<long long>(row) * p.H * p.rank;
   const __nv_bfloat16* qr = reinterpret_cast<const __nv_bfloat16*>(p.q) + row * p.q_ld;
   const int tiles = j1 > j0 ? (j1 - j0 + LD_KT - 1) / LD_KT : 0;
-  {   // the 16 query rows, one per warp: [q_lat | q_rot | 0]
-    const int h = h0 + warp;
-    for (int c = lane; c < cols; c += 32) {
-      __nv_bfloat16 v = __float2bfloat16(0.f);
-      if (h < p.H) {
-        if (c < p.rank) v = ql[h * p.rank + c];
-        else if (c < p.rank + p.rot) v = qr[h * (p.dim + p.rot) + p.dim + c - p.rank];
-      }
-      qs[warp * st + c] = v;
+  bool alive = true;
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < LD_STAGES; ++i) {
+      mbar_init(&full[i], LD_LOADERS);
+      mbar_init(&empty[i], LD_WARPS);
     }
+    fence_barrier_init();
+  }
+  if (warp < LD_WARPS) {   // the 16 query rows, one per warp: [q_lat | q_rot | 0]
+    const int h = h0 + warp;
+    __nv_bfloat16* dst = qs + warp * st;
+    const uint4* lat = reinterpret_cast<const uint4*>(ql + static_cast<long long>(h) * p.rank);
+#pragma unroll
+    for (int k = 0; k < (128 * NP + 255) / 256; ++k) {
+      const int c = lane + k * 32;
+      if (c < p.rank / 8) *reinterpret_cast<uint4*>(dst + c * 8) = h < p.H ? lat[c] : make_uint4(0u, 0u, 0u, 0u);
+    }
+    const __nv_bfloat16* rotated = qr + h * (p.dim + p.rot) + p.dim;
+    for (int c = lane; c < cols - p.rank; c += 32)
+      dst[p.rank + c] = h < p.H && c < p.rot ? rotated[c] : __float2bfloat16(0.f);
   }
   __syncthreads();
-  // warp w loads rows w, w + 16 of a tile; the pages of its next rows (lane u: row u) are looked up one tile ahead and used
-  // no earlier, so the table's latency is off the path
-  constexpr int RPW = LD_KT / LD_WARPS;
-  constexpr int NC = (128 * NP + 64 + 255) / 256;      // 16-byte columns per lane
-  const int shift = p.block_shift, mask = p.block_size - 1;
-  int page = 0, j_look = j0 + warp + lane * LD_WARPS, j_load = j0 + warp;
-  const __nv_bfloat16* src0 = cache + lane * 8;
-  const uint32_t dst0 = smem_u32(kv + warp * st + lane * 8);
-  const uint32_t row_step = LD_WARPS * st * 2, tile_step = LD_KT * st * 2;
-  auto look_up = [&]() {
-    if (lane < RPW && j_look < j1) page = bt[j_look >> shift];
-    j_look += LD_KT;
-  };
-  auto load_tile = [&](int i) {
-    const uint32_t dst_t = dst0 + (i % LD_STAGES) * tile_step;
-#pragma unroll
-    for (int u = 0; u < RPW; ++u) {
-      const int j = j_load + u * LD_WARPS;
-      const int slot = (__shfl_sync(0xffffffffu, page, u) << shift) + (j & mask);
-      const __nv_bfloat16* src = src0 + static_cast<long long>(slot) * cols;
-      const uint32_t dst = dst_t + u * row_step;
-#pragma unroll
-      for (int k = 0; k < NC; ++k) {
-        if (lane + k * 32 < cols / 8) {
-          if (j < j1) cp_async16(dst + k * 512, src + k * 256);
-          else asm volatile("st.shared.v4.u32 [%0], {%1, %1, %1, %1};" ::"r"(dst + k * 512), "r"(0u) : "memory");
-        }                              // (zero rows past the range keep 0 * x finite)
+
+  if (warp >= LD_WARPS) {
+    // loader warp w: rows 8 w .. 8 w + 7 of a tile, one per lane; the page of the lane's next row is looked up one tile ahead
+    // and used no earlier, so the table's latency is off the path
+    constexpr int RPW = LD_KT / LD_LOADERS;
+    const int r = (warp - LD_WARPS) * RPW + lane, shift = p.block_shift;
+    int page = 0;
+    if (lane < RPW && j0 + r < j1) page = bt[(j0 + r) >> shift];
+    for (int i = 0; i < tiles; ++i) {
+      const int s = i % LD_STAGES, j = j0 + i * LD_KT + r;
+      const int mine = max(0, min(RPW, j1 - (j - lane)));            // rows of this warp inside the range
+      if (!__all_sync(0xffffffffu, mbar_wait(&empty[s], ((i / LD_STAGES) & 1u) ^ 1u, alive, 901))) break;
+      for (int z = mine; z < RPW; ++z)                               // zero rows past the range keep 0 * x finite
+        for (int c = lane; c < cols / 8; c += 32)
+          *reinterpret_cast<uint4*>(kv + (s * LD_KT + r - lane + z) * st + c * 8) = make_uint4(0u, 0u, 0u, 0u);
+      __syncwarp();
+      if (lane == 0) mbar_expect_tx(&full[s], mine * cols * 2);
+      __syncwarp();
+      if (lane < mine)
+        bulk_load(smem_u32(kv + (s * LD_KT + r) * st),
+                  cache + ((static_cast<long long>(page) << shift) + (j & (p.block_size - 1))) * cols, cols * 2, &full[s]);
+      if (lane < RPW && j + LD_KT < j1) page = bt[(j + LD_KT) >> shift];
+    }
+    if (!alive) {                        // a wait ran out: give the copies in flight a bounded time to land
+      const long long t0 = clock64();
+      while (clock64() - t0 < 2000000ll) {
       }
     }
-    j_load += LD_KT;
-    look_up();
-  };
-  look_up();
-  for (int i = 0; i < LD_STAGES - 1; ++i) {
-    if (i < tiles) load_tile(i);
-    cp_async_commit();
+    return;
   }
   // columns in 16-wide steps: this warp's quarter
   const int steps = cols / 16, per = (steps + 3) / 4;
@@ -299,10 +319,7 @@ __global__ void __launch_bounds__(LD_WARPS * 32, 1) latent_attend_mma_kernel(Lat
     const int s = i % LD_STAGES;
     const __nv_bfloat16* tile = kv + s * LD_KT * st;
     const int n = min(LD_KT, j1 - (j0 + i * LD_KT));
-    cp_async_wait<LD_STAGES - 2>();
-    __syncthreads();                               // tile i is in; every warp is past tile i - 1
-    if (i + LD_STAGES - 1 < tiles) load_tile(i + LD_STAGES - 1);
-    cp_async_commit();
+    mbar_wait(&full[s], (i / LD_STAGES) & 1u, alive, 900);
     {
       float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
       const uint32_t ka = smem_u32(tile + ((warp & 3) * 8 + (lane & 7)) * st + k_first * 16 + (lane >> 3) * 8);
@@ -325,7 +342,7 @@ __global__ void __launch_bounds__(LD_WARPS * 32, 1) latent_attend_mma_kernel(Lat
       *reinterpret_cast<float2*>(d) = make_float2(c0[0] + c1[0], c0[1] + c1[1]);
       *reinterpret_cast<float2*>(d + 8 * SW) = make_float2(c0[2] + c1[2], c0[3] + c1[3]);
     }
-    __syncthreads();                               // scores complete
+    compute_barrier();                             // scores complete
     {   // softmax of head `warp`, one key per lane
       const float* a = ss + warp * SW + lane;
       const float v = lane < n ? ((a[0] + a[16 * SW]) + (a[32 * SW] + a[48 * SW])) * sl : -INFINITY;
@@ -336,7 +353,7 @@ __global__ void __launch_bounds__(LD_WARPS * 32, 1) latent_attend_mma_kernel(Lat
       ps[warp * (LD_KT + 8) + lane] = __float2bfloat16(w);
       if (lane == 0) s_alpha[warp] = alpha;
     }
-    __syncthreads();                               // weights complete
+    compute_barrier();                             // weights complete
     {
       if (i > 0) {
         const float al0 = s_alpha[gid], al1 = s_alpha[gid + 8];
@@ -359,6 +376,8 @@ __global__ void __launch_bounds__(LD_WARPS * 32, 1) latent_attend_mma_kernel(Lat
           mma_16816(o[x], a1, b[2], b[3]);
         }
       }
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&empty[s]);
     }
   }
   const float l_run = warp_sum(l_lane);
@@ -369,7 +388,7 @@ __global__ void __launch_bounds__(LD_WARPS * 32, 1) latent_attend_mma_kernel(Lat
       p.part_lse[(static_cast<long long>(row) * p.H + h) * p.splits + split] =
           l_run > 0.f ? (m_run + log2f(l_run)) * 0.6931471805599453f : -INFINITY;
   }
-  __syncthreads();
+  compute_barrier();
 #pragma unroll
   for (int half = 0; half < 2; ++half) {
     const int r = gid + half * 8, h = h0 + r;
@@ -461,6 +480,7 @@ extern "C" int ts_latent_splits(int rows, int H, int rank, int row_width, int bl
   long long s = (2ll * sm_count() + units - 1) / units;
   if (s > most) s = most;
   if (s < (max_keys + 2047) / 2048) s = (max_keys + 2047) / 2048;   // the chunk's scores sit in shared memory
+  if (s > MERGE_MAX_SPLITS) s = MERGE_MAX_SPLITS;
   return (int)(s < 1 ? 1 : s);
 }
 
@@ -472,7 +492,7 @@ extern "C" int ts_latent_attend(const void* q_lat, const void* q, long long q_ld
                                 int row_width, int block_size, int window, int max_keys, int splits, float scale, int fp32,
                                 void* stream) {
   if (rows <= 0) return 0;
-  if (H <= 0 || rank <= 0 || block_size <= 0 || window <= 0 || splits <= 0 || splits > 65535) return -10;
+  if (H <= 0 || rank <= 0 || block_size <= 0 || window <= 0 || splits <= 0 || splits > MERGE_MAX_SPLITS) return -10;
   LatentAttendParams p;
   p.q_lat = q_lat; p.q = q; p.q_ld = q_ld; p.cache = cache; p.block_table = block_table; p.row_seq = row_seq;
   p.row_len = row_len; p.out = out; p.part_out = part_out; p.part_lse = part_lse; p.rows = rows; p.H = H; p.dim = dim;
@@ -496,7 +516,7 @@ extern "C" int ts_latent_attend(const void* q_lat, const void* q, long long q_ld
       if (e != cudaSuccess) return (int)e;                                                                       \
       configured = true;                                                                                         \
     }                                                                                                            \
-    latent_attend_mma_kernel<N><<<grid, LD_WARPS * 32, sm, st>>>(p);                                             \
+    latent_attend_mma_kernel<N><<<grid, (LD_WARPS + LD_LOADERS) * 32, sm, st>>>(p);                                             \
   }
     if (np <= 1) TS_LATENT(1)
     else if (np == 2) TS_LATENT(2)
