@@ -64,12 +64,13 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
   if ((int)blockIdx.y >= n_qblocks) return;
   const int qb = n_qblocks - 1 - blockIdx.y;
   const int off = Lk - Lq;
-  int r0[2], nkv[2];
-  // key tiles entirely left of the first row's window are never loaded
+  // key tiles entirely left of the first row's window are never loaded; query tile t works on tiles [first[t], nkv[t])
+  int r0[2], first[2], nkv[2];
   const int kb_lo = max(0, qb * 256 + off - p.window + 1) / 128;
 #pragma unroll
   for (int t = 0; t < 2; ++t) {
     r0[t] = qb * 256 + t * 128;
+    first[t] = max(0, r0[t] + off - p.window + 1) / 128 - kb_lo;
     nkv[t] = r0[t] >= Lq ? 0 : max(0, (min(Lk, r0[t] + 128 + off) + 127) / 128 - kb_lo);
   }
   const int n = max(nkv[0], nkv[1]);
@@ -140,7 +141,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
       if (n > 0 && mbar_wait(&k_full[0], 0, alive, 501)) {
         tc_fence_after_sync();
         for (int t = 0; t < 2; ++t)
-          if (nkv[t] > 0) issue_s(t, 0);
+          if (nkv[t] > 0 && first[t] == 0) issue_s(t, 0);
         umma_commit(&k_empty[0]);
       }
       for (int i = 0; i < n && alive; ++i) {
@@ -148,17 +149,17 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
         if (!mbar_wait(&v_full[vs], (i / p.v_stages) & 1u, alive, 502)) break;
         bool k_waited = false;
         for (int t = 0; t < 2 && alive; ++t) {
-          if (i < nkv[t]) {
-            if (!mbar_wait(&p_full[t], i & 1u, alive, 503)) break;
+          if (i >= first[t] && i < nkv[t]) {
+            if (!mbar_wait(&p_full[t], (i - first[t]) & 1u, alive, 503)) break;
             tc_fence_after_sync();
             const uint32_t va = smem_u32(v_base + vs * v_bytes);
 #pragma unroll
             for (int kk = 0; kk < 8; ++kk)
               umma_f16_ts(tmem_base + O_COL0 + t * 128, tmem_base + t * 128 + kk * 8,
-                          make_smem_desc_sw128(va + kk * 2048, LP_BLOCK, 1024), idesc_o, (i | kk) != 0);
+                          make_smem_desc_sw128(va + kk * 2048, LP_BLOCK, 1024), idesc_o, (i - first[t]) != 0 || kk != 0);
             if (i == nkv[t] - 1) umma_commit(&o_full[t]);
           }
-          if (i + 1 < nkv[t]) {
+          if (i + 1 >= first[t] && i + 1 < nkv[t]) {
             if (!k_waited) {
               if (!mbar_wait(&k_full[kn], ((i + 1) / p.k_stages) & 1u, alive, 504)) break;
               tc_fence_after_sync();
@@ -181,10 +182,10 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
     const uint32_t t_s = t_lane + t * 128;
     const uint32_t t_o = t_lane + O_COL0 + t * 128;
     float m_used = -INFINITY, l = 0.f;
-    const int nt = nkv[t];
+    const int nt = nkv[t], i0 = first[t];
     const float sc = p.scale_log2;
-    for (int i = 0; i < nt && alive; ++i) {
-      if (!mbar_wait(&s_full[t], i & 1u, alive, 600)) break;
+    for (int i = i0; i < nt && alive; ++i) {
+      if (!mbar_wait(&s_full[t], (i - i0) & 1u, alive, 600)) break;
       tc_fence_after_sync();
       const int c0 = (kb_lo + i) * 128;
       const bool need_mask = (c0 + 127 > r0[t] + off) || (c0 + 128 > Lk) || (c0 <= r0[t] + 127 + off - p.window);
@@ -214,7 +215,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
         const float alpha = (m_used == -INFINITY) ? 0.f : fast_ex2(m_used - m_new);
         m_used = m_new;
         l *= alpha;
-        if (i > 0) {
+        if (i > i0) {
 #pragma unroll 1
           for (int c = 0; c < p.v_cols / 16; ++c) {
             uint32_t o[16];
