@@ -19,6 +19,33 @@ namespace ts {
 constexpr int LP_THREADS = 320;
 constexpr int LP_BLOCK = 16384;          // 128 rows x 64 bf16 columns
 
+__device__ __forceinline__ float max3(float a, float b, float c) {
+  float d;
+  asm("max.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c));
+  return d;
+}
+// two fp32 lanes in one instruction
+__device__ __forceinline__ uint64_t pack_f32x2(float lo, float hi) {
+  uint64_t d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+  return d;
+}
+__device__ __forceinline__ float2 unpack_f32x2(uint64_t v) {
+  float2 d;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(d.x), "=f"(d.y) : "l"(v));
+  return d;
+}
+__device__ __forceinline__ uint64_t fma_f32x2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ uint64_t add_f32x2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+
 struct LatentPrefillParams {
   const int* cu_q;                       // [sequences + 1] query rows
   const int* cu_k;                       // [sequences + 1] key rows
@@ -196,19 +223,30 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
       for (int c = 0; c < 4; ++c) tmem_ld_32x32b_x32(t_s + c * 32, v + c * 32);
       tc_wait_ld();
       if (need_mask) {
+        // visible columns of the tile are [lo - c0, limit - c0]: one bit per column, a word per 32
+        const int a = max(lo - c0, 0), e = min(limit - c0, 127);
 #pragma unroll
-        for (int j = 0; j < 128; ++j)
-          if (c0 + j > limit || c0 + j < lo) v[j] = 0xff800000u;
-      }
-      float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
+        for (int c = 0; c < 4; ++c) {
+          const int s0 = a - c * 32, s1 = e - c * 32;      // first and last visible bit of this word
+          uint32_t bits = s1 < 0 || s0 > 31 ? 0u : 0xffffffffu;
+          if (s0 > 0) bits &= 0xffffffffu << (s0 & 31);
+          if (s1 < 31) bits &= 0xffffffffu >> (31 - (s1 & 31));
 #pragma unroll
-      for (int j = 0; j < 128; j += 4) {
-        mx0 = fmaxf(mx0, __uint_as_float(v[j]));
-        mx1 = fmaxf(mx1, __uint_as_float(v[j + 1]));
-        mx2 = fmaxf(mx2, __uint_as_float(v[j + 2]));
-        mx3 = fmaxf(mx3, __uint_as_float(v[j + 3]));
+          for (int j = 0; j < 32; ++j)
+            if (!(bits & (1u << j))) v[c * 32 + j] = 0xff800000u;
+        }
       }
-      const float mx = fmaxf(fmaxf(mx0, mx1), fmaxf(mx2, mx3));
+      float mx0 = __uint_as_float(v[0]), mx1 = __uint_as_float(v[1]), mx2 = __uint_as_float(v[2]), mx3 = __uint_as_float(v[3]);
+#pragma unroll
+      for (int j = 4; j + 7 < 128; j += 8) {
+        mx0 = max3(mx0, __uint_as_float(v[j]), __uint_as_float(v[j + 1]));
+        mx1 = max3(mx1, __uint_as_float(v[j + 2]), __uint_as_float(v[j + 3]));
+        mx2 = max3(mx2, __uint_as_float(v[j + 4]), __uint_as_float(v[j + 5]));
+        mx3 = max3(mx3, __uint_as_float(v[j + 6]), __uint_as_float(v[j + 7]));
+      }
+      mx0 = max3(mx0, __uint_as_float(v[124]), __uint_as_float(v[125]));
+      mx1 = max3(mx1, __uint_as_float(v[126]), __uint_as_float(v[127]));
+      const float mx = fmaxf(max3(mx0, mx1, mx2), mx3);
       const float m_new = fmaxf(m_used, mx * sc);
       const bool grow = (m_new - m_used > 8.0f);       // also true on the first tile with a visible key
       if (__any_sync(0xffffffffu, grow)) {
@@ -228,21 +266,24 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
         }
       }
       const float m_sub = (m_used == -INFINITY) ? 0.f : m_used;
-      float l0 = 0.f, l1 = 0.f;
+      uint64_t sum0 = 0ull, sum1 = 0ull;
+      const uint64_t sc2 = pack_f32x2(sc, sc), m2 = pack_f32x2(-m_sub, -m_sub);
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
         uint32_t pk[16];
 #pragma unroll
         for (int j = 0; j < 32; j += 2) {
-          const float p0 = fast_ex2(fmaf(__uint_as_float(v[c * 32 + j]), sc, -m_sub));
-          const float p1 = fast_ex2(fmaf(__uint_as_float(v[c * 32 + j + 1]), sc, -m_sub));
-          l0 += p0;
-          l1 += p1;
+          const float2 e = unpack_f32x2(fma_f32x2(
+              pack_f32x2(__uint_as_float(v[c * 32 + j]), __uint_as_float(v[c * 32 + j + 1])), sc2, m2));
+          const float p0 = fast_ex2(e.x), p1 = fast_ex2(e.y);
+          if (j & 2) sum1 = add_f32x2(sum1, pack_f32x2(p0, p1));
+          else sum0 = add_f32x2(sum0, pack_f32x2(p0, p1));
           pk[j >> 1] = pack_bf16x2(p0, p1);
         }
         tmem_st_32x32b_x16(t_s + c * 16, pk);
       }
-      l += l0 + l1;
+      const float2 sums = unpack_f32x2(add_f32x2(sum0, sum1));
+      l += sums.x + sums.y;
       tc_wait_st();
       tc_fence_before_sync();
       __syncwarp();
