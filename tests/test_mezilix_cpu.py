@@ -255,6 +255,32 @@ def test_configurations_the_class_cannot_run_are_refused():
     assert architecture_of({"model_type": "llama"}).name == "Llama"
 
 
+def test_features_of_the_llama_path_are_refused_with_a_reason():
+    _, _, core = make()
+    with pytest.raises(ValueError, match="LoRA"):
+        core.load_adapters({"a": {}})
+    cfg = EngineConfig(model="custom", tokenizer="byte", device="cpu")
+    cfg.speculative.enabled = True
+    eng = SOTAInferenceEngine(cfg, model=core.model, draft_model=core.model)
+    assert eng.generate("ab", GenerationParams(max_tokens=2)).is_err()
+    cfg = EngineConfig(model="custom", tokenizer="byte", device="cpu")
+    cfg.parallel.tensor_parallel_size = 2
+    with pytest.raises(ValueError, match="one GPU"):
+        EngineCore(cfg, model=core.model)
+
+
+def test_prefix_sharing_is_off_for_models_with_state():
+    cfg, w, core = make()
+    ids = tokens(24, 3)
+    outs = []
+    for _ in range(2):
+        r = core.add_request(ids, GenerationParams(max_tokens=4, temperature=0.0, ignore_eos=True))
+        while core.has_unfinished():
+            core.step()
+        outs.append(r.output_ids)
+    assert outs[0] == outs[1] == O.greedy(w, cfg, ids, 4) and core.cache.prefix_hits == 0
+
+
 def test_presets_and_registry():
     from trainscale_b200.models import is_preset
     from trainscale_b200.registry import MODEL_REGISTRY

@@ -125,7 +125,7 @@ def test_head_linear(dtype, T, H, K, N):
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("T,W,E,k,F", [(1, 64, 4, 2, 24), (7, 96, 12, 3, 40), (33, 64, 5, 5, 136), (64, 64, 40, 4, 64),
                                        (65, 64, 4, 2, 24), (300, 96, 12, 3, 40), (500, 128, 3, 1, 200), (90, 50, 6, 2, 17),
-                                       (9, 50, 6, 2, 17)])
+                                       (9, 50, 6, 2, 17), (20, 64, 1, 1, 24), (200, 64, 1, 1, 24)])
 def test_routed_experts(dtype, T, W, E, k, F):
     """Router, top-k, plan and both expert products against a loop over tokens; decode-sized and prompt-sized batches."""
     from trainscale_b200.ops import gemm, grouped, moe
@@ -451,3 +451,52 @@ def test_bf16_rejects_nothing_it_should_run():
     assert L.expanded_supported(ok)
     assert not L.expanded_supported(L.LatentShape(4, 12, 4, 20, 24, 40, 0.1, 1e4))
     assert not L.expanded_supported(L.LatentShape(4, 64, 16, 256, 128, 40, 0.1, 1e4))
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_wide_decode_batch(dtype):
+    """More sequences than the few-row kernels take: tensor-core products, grouped experts and a padded captured batch."""
+    from trainscale_b200.inference.batch import StepEntry
+    cfg = O.make_config(**CASES["tiles"])
+    w = O.make_weights(cfg, 8, 1.5)
+    core = engine(cfg, w, dtype, seqs=45, blocks=45 * 8)
+    ids = [tokens(20 + 2 * i, 200 + i) for i in range(45)]
+    for a in range(0, 45, 15):
+        core.execute([StepEntry(i, ids[i][:-3], []) for i in range(a, a + 15)])
+    for k in (3, 2, 1):
+        got = core.execute([StepEntry(i, [t[-k]], None) for i, t in enumerate(ids)]).clone()
+    assert core.runner.graph_replays == 3
+    for i in range(0, 45, 6):
+        assert rel(got[i], oracle64(w, cfg, ids[i])[-1]) < model_tol(dtype), i
+
+
+def test_trace_program(tmp_path):
+    """bin/trace_run as a process of its own: a directory with config.json and weights, steps on stdin, logits in files."""
+    import json
+    import subprocess
+    from pathlib import Path
+
+    import numpy as np
+    from trainscale_b200.hub import ModelSerializer
+    cfg = O.make_config(**CASES["unlike"])
+    w = O.make_weights(cfg, 9, 1.5)
+    (tmp_path / "model").mkdir()
+    (tmp_path / "model" / "config.json").write_text(json.dumps(cfg))
+    ModelSerializer().save({k: v.to(torch.bfloat16) for k, v in w.items()}, tmp_path / "model")
+    a, b = tokens(40, 1), tokens(9, 2)
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": a[:30], "want": []}], "end": []},
+             {"step": 1, "entries": [{"id": "b", "tokens": b, "want": [8, 0]}, {"id": "a", "tokens": a[30:31], "want": [0]}],
+              "end": ["b"]},
+             {"step": 2, "entries": [{"id": "a", "tokens": a[31:], "want": [2, 8]}], "end": ["a"]}]
+    for dtype in ("float32", "bfloat16"):
+        out = tmp_path / dtype
+        out.mkdir()
+        r = subprocess.run([str(Path(__file__).resolve().parent.parent / "bin" / "trace_run"), "--model", str(tmp_path / "model"),
+                            "--dtype", dtype, "--out", str(out), "--max-tokens", "128"],
+                           input="".join(json.dumps(s) + "\n" for s in steps), capture_output=True, text=True, timeout=240)
+        assert r.returncode == 0, r.stderr[-2000:]
+        assert r.stdout.split("\n")[:3] == ["done 0", "done 1", "done 2"] and not (out / "0.f32").exists()
+        la, lb = oracle64(w, cfg, a), oracle64(w, cfg, b)
+        for step, want in ((1, torch.stack([lb[8], lb[0], la[30]])), (2, torch.stack([la[33], la[39]]))):
+            got = torch.from_numpy(np.fromfile(out / f"{step}.f32", dtype="<f4").copy()).view(want.shape)
+            assert rel(got, want) < model_tol(dtype)

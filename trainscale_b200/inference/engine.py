@@ -825,6 +825,9 @@ class SOTAInferenceEngine:
     def _generate_speculative(self, prompts: list[str], params: GenerationParams) -> list["InferenceResponse"]:
         """One request at a time through draft-and-verify decoding (inference/speculative.py)."""
         from .speculative import speculative_generate
+        if self.core.runner.own_layers or hasattr(self.draft_model, "serve"):
+            raise ValueError("speculative decoding rolls a key/value cache back; models with their own layers and "
+                             "sequence state do not support it")
         out = []
         for p in prompts:
             r = self.core.add_request(p, params)
