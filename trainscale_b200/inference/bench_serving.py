@@ -115,13 +115,13 @@ class OpTimer:
         torch.cuda.synchronize()
         acc: dict = {}
         for name, e0, e1, nbytes, flops in self.records:
-            r = acc.setdefault(name, [0, 0.0, 0.0, 0.0])
+            r = acc.setdefault(name, [0, 0.0, 0.0])
             floor = max(nbytes / (peaks["hbm_gbs"] * 1e9), flops / (peaks["bf16_tflops"] * 1e12)) * 1e3
             r[0] += 1
             r[1] += e0.elapsed_time(e1)
             r[2] += floor
         return {n: {"calls": c, "ms": round(ms, 4), "of_roofline": round(fl / ms, 3) if ms else None}
-                for n, (c, ms, fl, _) in sorted(acc.items(), key=lambda kv: -kv[1][1])}
+                for n, (c, ms, fl) in sorted(acc.items(), key=lambda kv: -kv[1][1])}
 
 
 def _linear_cost(a, k, out):
