@@ -94,6 +94,17 @@ __device__ __forceinline__ float2 unpack_bf16x2(uint32_t v) {
   return __bfloat1622float2(b);
 }
 
+// Activations that a product may apply to its result: 1 squared ReLU, 2 tanh, 3 soft cap c * tanh(v / c)
+__device__ __forceinline__ float product_act(float v, int act, float cap) {
+  if (act == 1) {
+    v = fmaxf(v, 0.f);
+    return v * v;
+  }
+  if (act == 2) return tanhf(v);
+  if (act == 3) return cap * tanhf(v / cap);
+  return v;
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

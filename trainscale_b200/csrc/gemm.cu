@@ -41,12 +41,23 @@ struct GemmParams {
   const int* seg_start;     // MODE 2: [E + 1] first row of every expert's (128-aligned) segment along the K axis
   int group_rows;           // MODE 1: rows (K-major B) or K extent (MN-major B) of one expert inside the stacked B
   int num_groups;           // MODE 2: E; C is [E][M][ldc]
-  int act;                  // MODE 1 epilogue activation: 0 none, 1 squared ReLU
+  int act;                  // epilogue activation of common.cuh product_act (modes 0 and 1; 0: none)
+  float act_cap;
 };
 
-__device__ __forceinline__ float relu_squared(float v) {
-  v = fmaxf(v, 0.f);
-  return v * v;
+// product_act of 32 accumulators; one uniform branch per kind, so that the common kinds stay short
+__device__ __forceinline__ void gemm_activate(uint32_t* r, int act, float cap) {
+  if (act == 1) {
+#pragma unroll
+    for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(product_act(__uint_as_float(r[j]), 1, cap));
+  } else {
+#pragma unroll
+    for (int j = 0; j < 32; ++j) {
+      const float v = __uint_as_float(r[j]);
+      const float t = tanhf(act == 3 ? v / cap : v);
+      r[j] = __float_as_uint(act == 3 ? cap * t : t);
+    }
+  }
 }
 
 // 32 consecutive fp32 accumulator columns of one output row: scale, optionally add to C, convert, store.
@@ -323,10 +334,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
         uint32_t r[32];
         tmem_ld_32x32b_x32(t_row + c * 32, r);
         tc_wait_ld();
-        if (MODE == 1 && p.act == 1) {
-#pragma unroll
-          for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(relu_squared(__uint_as_float(r[j])));
-        }
+        if (MODE != 2 && p.act != 0) gemm_activate(r, p.act, p.act_cap);
         const int col0 = n0 + c * 32;
         if (row < p.M && col0 < p.N) gemm_store_chunk(p, r, ti.c_row0 + row, col0);
       }
@@ -489,6 +497,7 @@ gemm_bf16_2cta_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_cons
         uint32_t r[32];
         tmem_ld_32x32b_x32(t_row + c * 32, r);
         tc_wait_ld();
+        if (p.act != 0) gemm_activate(r, p.act, p.act_cap);
         const int col0 = n0 + c * 32;
         if (row < p.M && col0 < p.N) gemm_store_chunk(p, r, static_cast<size_t>(row), col0);
       }
@@ -557,10 +566,13 @@ TS_DEFINE_ERROR_API(ts_gemm)
 //   out_fp32: C is fp32 (else bf16); accumulate: add into the existing C.
 //   bn: N tile (256, 128 or 64; 0 = choose).
 // Leading dimensions are in elements and must keep rows 16-byte aligned. Returns 0 on success.
-extern "C" int ts_gemm_bf16(const void* A, const void* B, void* C, int M, int N, int K, int lda, int ldb, int ldc,
-                            int a_mn, int b_mn, int out_fp32, int accumulate, float alpha, int bn, void* stream) {
+//   act: activation of the result (common.cuh product_act; C must not accumulate then).
+extern "C" int ts_gemm_bf16_act(const void* A, const void* B, void* C, int M, int N, int K, int lda, int ldb, int ldc,
+                                int a_mn, int b_mn, int out_fp32, int accumulate, float alpha, int bn, int act,
+                                float act_cap, void* stream) {
   using namespace ts;
   if (M <= 0 || N <= 0 || K <= 0) return -10;
+  if (act != 0 && (act < 0 || act > 3 || accumulate || alpha != 1.f || (act == 3 && !(act_cap > 0.f)))) return -13;
   if (bn == 0) {
     // prefer the widest tile that still gives every SM work
     const int tiles256 = ((M + 127) / 128) * ((N + 255) / 256);
@@ -590,7 +602,8 @@ extern "C" int ts_gemm_bf16(const void* A, const void* B, void* C, int M, int N,
   p.num_m_tiles = (M + GEMM_BM - 1) / GEMM_BM;
   p.num_n_tiles = (N + bn - 1) / bn;
   p.k_blocks = (K + GEMM_BK - 1) / GEMM_BK;
-  p.tile_expert = nullptr; p.seg_start = nullptr; p.group_rows = 0; p.num_groups = 1; p.act = 0;
+  p.tile_expert = nullptr; p.seg_start = nullptr; p.group_rows = 0; p.num_groups = 1; p.act = act;
+  p.act_cap = act_cap;
   p.c_bytes = (static_cast<size_t>(M - 1) * ldc + N) * (out_fp32 ? 4 : 2);
 #ifdef TS_DEBUG
   // test hook of the debug build: pretend C ends `TS_DEBUG_SHRINK_C_ROWS` rows early, so that the bounds check (and
@@ -605,6 +618,11 @@ extern "C" int ts_gemm_bf16(const void* A, const void* B, void* C, int M, int N,
   if (bn == 256) return launch_gemm<256>(tmA, tmB, p, st);
   if (bn == 128) return launch_gemm<128>(tmA, tmB, p, st);
   return launch_gemm<64>(tmA, tmB, p, st);
+}
+
+extern "C" int ts_gemm_bf16(const void* A, const void* B, void* C, int M, int N, int K, int lda, int ldb, int ldc,
+                            int a_mn, int b_mn, int out_fp32, int accumulate, float alpha, int bn, void* stream) {
+  return ts_gemm_bf16_act(A, B, C, M, N, K, lda, ldb, ldc, a_mn, b_mn, out_fp32, accumulate, alpha, bn, 0, 0.f, stream);
 }
 
 // Grouped GEMM over an expert-sorted token buffer whose per-expert segments start on 128-row boundaries.
@@ -649,7 +667,7 @@ extern "C" int ts_gemm_grouped_bf16_act(const void* A, const void* B, void* C, i
   p.seg_start = (mode == 2) ? groups : nullptr;
   p.group_rows = b_mn ? K : N;
   p.num_groups = num_groups;
-  p.act = act;
+  p.act = act; p.act_cap = 0.f;
   p.c_bytes = (static_cast<size_t>((mode == 2 ? num_groups : 1)) * M - 1) * ldc * (out_fp32 ? 4 : 2) +
               static_cast<size_t>(N) * (out_fp32 ? 4 : 2);
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);

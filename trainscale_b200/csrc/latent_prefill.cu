@@ -1,4 +1,6 @@
-// Windowed causal attention for portions of prompts whose keys come from a latent cache (tcgen05 / TMEM / TMA).
+// Windowed causal attention for portions of prompts (tcgen05 / TMEM / TMA), two entry points:
+//   ts_latent_prefill  keys come from a latent cache
+//   ts_window_prefill  keys and values per key/value head (grouped queries), query / key and value sizes of their own
 //
 // The latents a portion needs (its own tokens and the window before them) have been expanded to per-head keys and values
 // by one GEMM; the rotated key part is shared by all heads and read from the latent rows.  Scores are therefore a sum of
@@ -55,7 +57,9 @@ struct LatentPrefillParams {
   int vdim, v_cols;                      // value size; rounded up to 16
   int k_stages, v_stages;
   int window;
+  int kv_group;                          // query heads that share a key/value head
   float scale_log2;
+  float o_scale;                         // factor of the result
   __nv_bfloat16* o;                      // [rows][o_stride], head h at column h * vdim
   long long o_stride;
 };
@@ -85,6 +89,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h = blockIdx.x % p.H, b = blockIdx.x / p.H;
+  const int hk = h / p.kv_group;
   const int q_start = p.cu_q[b], Lq = p.cu_q[b + 1] - q_start;
   const int k_start = p.cu_k[b], Lk = p.cu_k[b + 1] - k_start;
   const int n_qblocks = (Lq + 255) / 256;
@@ -136,13 +141,13 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
         if (!mbar_wait(&k_empty[ks], ((ki / p.k_stages) & 1u) ^ 1u, alive, 400)) break;
         mbar_expect_tx(&k_full[ks], k_bytes);
         for (int j = 0; j < p.nb_n; ++j)
-          tma_load_3d(k_base + ks * k_bytes + j * LP_BLOCK, &tmKn, &k_full[ks], j * 64, h, row);
+          tma_load_3d(k_base + ks * k_bytes + j * LP_BLOCK, &tmKn, &k_full[ks], j * 64, hk, row);
         for (int j = 0; j < p.nb_r; ++j)
           tma_load_2d(k_base + ks * k_bytes + (p.nb_n + j) * LP_BLOCK, &tmKr, &k_full[ks], j * 64, row);
         if (!mbar_wait(&v_empty[vs], ((vi / p.v_stages) & 1u) ^ 1u, alive, 401)) break;
         mbar_expect_tx(&v_full[vs], v_bytes);
         for (int j = 0; j < p.nb_v; ++j)
-          tma_load_3d(v_base + vs * v_bytes + j * LP_BLOCK, &tmV, &v_full[vs], j * 64, h, row);
+          tma_load_3d(v_base + vs * v_bytes + j * LP_BLOCK, &tmV, &v_full[vs], j * 64, hk, row);
       }
     }
   } else if (warp == 1) {
@@ -291,7 +296,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
     }
     if (nt > 0 && alive && mbar_wait(&o_full[t], 0, alive, 601)) {
       tc_fence_after_sync();
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      const float inv = l > 0.f ? p.o_scale / l : 0.f;
       const bool valid = row < Lq;
       __nv_bfloat16* dst = p.o + (q_start + row) * p.o_stride + h * p.vdim;
 #pragma unroll 1
@@ -345,6 +350,24 @@ static bool plan_prefill(int dim, int rot, int vdim, LatentPrefillPlan& pl) {
   return false;
 }
 
+// Tensor maps are the caller's; `p` still lacks what follows from the sizes.
+static int launch_prefill(const CUtensorMap& tQn, const CUtensorMap& tQr, const CUtensorMap& tKn, const CUtensorMap& tKr,
+                          const CUtensorMap& tV, const LatentPrefillPlan& pl, LatentPrefillParams p, int dim, int rot,
+                          int vdim, int sequences, int max_q, void* stream) {
+  p.nb_n = pl.nb_n; p.nb_r = pl.nb_r; p.nb_v = pl.nb_v;
+  p.ks_n = (dim + 15) / 16; p.ks_r = (rot + 15) / 16; p.vdim = vdim; p.v_cols = (vdim + 15) / 16 * 16;
+  p.k_stages = pl.k_stages; p.v_stages = pl.v_stages;
+  static bool configured = false;
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(latent_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+    if (e != cudaSuccess) return (int)e;
+    configured = true;
+  }
+  const dim3 grid((unsigned)(p.H * sequences), (unsigned)((max_q + 255) / 256));
+  latent_prefill_kernel<<<grid, LP_THREADS, pl.smem, reinterpret_cast<cudaStream_t>(stream)>>>(tQn, tQr, tKn, tKr, tV, p);
+  return (int)cudaGetLastError();
+}
+
 }  // namespace ts
 
 TS_DEFINE_ERROR_API(ts_latent_prefill)
@@ -385,18 +408,34 @@ extern "C" int ts_latent_prefill(const void* q, long long q_ld, long long q_rows
     rc = make_tmap_2d(&tKr, k_rot, dt, 2, k_rows, rot, kr_ld, 128, 64);
     if (rc) return rc * 100 - 5;
   }
-  LatentPrefillParams p;
-  p.cu_q = cu_q; p.cu_k = cu_k; p.H = H; p.nb_n = pl.nb_n; p.nb_r = pl.nb_r; p.nb_v = pl.nb_v;
-  p.ks_n = (dim + 15) / 16; p.ks_r = (rot + 15) / 16; p.vdim = vdim; p.v_cols = (vdim + 15) / 16 * 16;
-  p.k_stages = pl.k_stages; p.v_stages = pl.v_stages; p.window = window; p.scale_log2 = scale * 1.4426950408889634f;
+  LatentPrefillParams p = {};
+  p.cu_q = cu_q; p.cu_k = cu_k; p.H = H; p.window = window; p.kv_group = 1; p.o_scale = 1.f;
+  p.scale_log2 = scale * 1.4426950408889634f;
   p.o = reinterpret_cast<__nv_bfloat16*>(out); p.o_stride = o_stride;
-  static bool configured = false;
-  if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(latent_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
-    if (e != cudaSuccess) return (int)e;
-    configured = true;
-  }
-  const dim3 grid((unsigned)(H * sequences), (unsigned)((max_q + 255) / 256));
-  latent_prefill_kernel<<<grid, LP_THREADS, pl.smem, reinterpret_cast<cudaStream_t>(stream)>>>(tQn, tQr, tKn, tKr, tV, p);
-  return (int)cudaGetLastError();
+  return launch_prefill(tQn, tQr, tKn, tKr, tV, pl, p, dim, rot, vdim, sequences, max_q, stream);
+}
+
+// q: rows [q_rows][q_ld], head h at column h * dim.  k / v: rows [k_rows][kv_ld], key/value head g at columns g * dim and
+// g * vdim.  cu_q / cu_k: [sequences + 1].  out: [q_rows][o_stride] = o_scale * attention.
+extern "C" int ts_window_prefill(const void* q, long long q_ld, long long q_rows, const void* k, const void* v,
+                                 long long kv_ld, long long k_rows, const int* cu_q, const int* cu_k, int sequences,
+                                 int max_q, int H, int G, int dim, int vdim, int window, float scale, float o_scale,
+                                 void* out, long long o_stride, void* stream) {
+  if (sequences <= 0 || max_q <= 0) return 0;
+  LatentPrefillPlan pl;
+  if (H <= 0 || G <= 0 || H % G || window <= 0 || !(scale > 0.f) || !plan_prefill(dim, 0, vdim, pl)) return -10;
+  if (q_ld % 8 || kv_ld % 8 || o_stride % 8 || (reinterpret_cast<uintptr_t>(out) & 15u)) return -11;
+  CUtensorMap tQ, tK, tV;
+  const CUtensorMapDataType dt = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
+  int rc = make_tmap_3d(&tQ, q, dt, 2, dim, H, q_rows, dim, q_ld, 64, 1, 128);
+  if (rc) return rc * 100 - 1;
+  rc = make_tmap_3d(&tK, k, dt, 2, dim, G, k_rows, dim, kv_ld, 64, 1, 128);
+  if (rc) return rc * 100 - 2;
+  rc = make_tmap_3d(&tV, v, dt, 2, vdim, G, k_rows, vdim, kv_ld, 64, 1, 128);
+  if (rc) return rc * 100 - 3;
+  LatentPrefillParams p = {};
+  p.cu_q = cu_q; p.cu_k = cu_k; p.H = H; p.window = window; p.kv_group = H / G; p.o_scale = o_scale;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.o = reinterpret_cast<__nv_bfloat16*>(out); p.o_stride = o_stride;
+  return launch_prefill(tQ, tQ, tK, tK, tV, pl, p, dim, 0, vdim, sequences, max_q, stream);
 }

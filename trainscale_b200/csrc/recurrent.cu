@@ -1,0 +1,1075 @@
+// Recurrent mixers with a matrix state per head, S [dim keys x vdim values], carried in fp32 from step to step:
+//
+//   gated delta rule   S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q        (g, beta one number per head)
+//   WKV                o = (S + diag(u) k v^T)^T r;  S <- diag(w) S + k v^T                (w per key channel)
+//
+// Rows are tokens of a flattened batch.  A portion of a prompt runs as: inputs (short convolution, unit norms, gates), a
+// scan over its tokens, the gated norm of the result.  A single decoded row is one launch from projection to gated norm.
+// A state row of a sequence holds [convolution inputs (taps - 1) x C | S per head] or [token-shift row | S per head];
+// a step reads one row and writes another, so nothing of a launch is overwritten while it is still read.
+//
+// The scan keeps S in registers, 8 key rows x 4 value columns per thread, and walks BLOCKS of tokens: for four tokens of
+// the delta rule all products S^T k and S^T q with the state before the block are formed at once (eight vectors, one
+// reduction over the lanes that share a column), the four-step triangular recurrence that is left is solved per column
+// with the block's small Gram matrices, and the state is updated with all four writes.  So the latency of a reduction is
+// paid once per block, not per token.  Everything is fp32 arithmetic on the FMA pipe in packed pairs: the warp MMA forms
+// that keep fp32 accuracy (three TF32 products) have no higher rate, and a 128-row tensor-memory tile would need the state
+// split into two operands and written to shared memory again for every chunk.
+#include "common.cuh"
+#include "host_common.h"
+
+namespace ts {
+
+template <typename T> __device__ __forceinline__ T from_f32(float v);
+template <> __device__ __forceinline__ float from_f32<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
+__device__ __forceinline__ float to_f32(float v) { return v; }
+__device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ float silu(float x) { return x / (1.f + expf(-x)); }
+__device__ __forceinline__ float sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
+__device__ __forceinline__ float softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
+
+__device__ __forceinline__ uint64_t pack2(float lo, float hi) {
+  uint64_t d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+  return d;
+}
+__device__ __forceinline__ float2 unpack2(uint64_t v) {
+  float2 d;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(d.x), "=f"(d.y) : "l"(v));
+  return d;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ void cp_async16(void* dst, const void* src, bool valid) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(valid ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_async4(void* dst, const void* src, bool valid) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(valid ? 4 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// ---------------------------------------------------------------------------------------------------------
+// gated delta rule
+// ---------------------------------------------------------------------------------------------------------
+struct DeltaParams {
+  const void* proj;            // rows [q G x D | k G x D | v H x V | gate H x V | b H | a H]
+  long long ld;
+  const float* conv_w;         // [C][taps], C = 2 G D + H V
+  const float* A_log;          // [H]
+  const float* dt_bias;        // [H]
+  const float* norm_w;         // [V]
+  float eps, q_scale;
+  float* state;
+  long long state_ld;
+  int s_off;                   // first value of S in a state row
+  const int* row_prev;         // [rows] state row a sequence continues from (>= 0), else zeros / the row before
+  const int* row_next;         // [rows] state row to leave, -1: not a last row
+  const int* cu;               // portions: [n + 1] first rows
+  const int* row_seq;          // portions: sequence of a row; the first portion is seq0
+  int seq0;
+  float* qkv;                  // portions: [rows][C] convolved inputs
+  float* gates;                // portions: [rows][2 H] log g | beta
+  float* o;                    // portions: [rows][H V]
+  void* out;                   // decoding: [rows][out_ld]
+  long long out_ld;
+  float out_scale;
+  int rows, H, G, D, V, taps;
+};
+
+// input of channel c at row `src` of a sequence whose portion starts at row `start`; rows before it come from the state
+template <typename T>
+__device__ __forceinline__ float conv_input(const DeltaParams& p, int src, int start, int prev, int c, int C) {
+  if (src >= start) return to_f32(reinterpret_cast<const T*>(p.proj)[src * p.ld + c]);
+  const int i = src - start + p.taps - 1;
+  return prev >= 0 && i >= 0 ? p.state[prev * p.state_ld + static_cast<long long>(i) * C + c] : 0.f;
+}
+
+constexpr int DI_TOKENS = 8;
+
+// A warp takes DI_TOKENS rows of one head of q, k or v (or the gates); lanes hold VEC neighbouring channels, NI times.
+// FAST: at most four taps, inputs of the rows before stay in registers.
+template <typename T, int VEC, int NI, bool FAST>
+__global__ void __launch_bounds__(128) delta_inputs_kernel(DeltaParams p) {
+  const int lane = threadIdx.x & 31, units = 2 * p.G + p.H + 1;
+  const int unit = blockIdx.y * 4 + (threadIdx.x >> 5);
+  if (unit >= units) return;
+  const int t0 = blockIdx.x * DI_TOKENS, t1 = min(p.rows, t0 + DI_TOKENS);
+  const int C = 2 * p.G * p.D + p.H * p.V;
+  const T* proj = reinterpret_cast<const T*>(p.proj);
+  if (unit == units - 1) {
+    const int b0 = C + p.H * p.V;
+    for (int i = lane; i < (t1 - t0) * p.H; i += 32) {
+      const int t = t0 + i / p.H, h = i % p.H;
+      const float b = to_f32(proj[t * p.ld + b0 + h]), a = to_f32(proj[t * p.ld + b0 + p.H + h]);
+      p.gates[static_cast<long long>(t) * 2 * p.H + h] = -expf(p.A_log[h]) * softplus(a + p.dt_bias[h]);
+      p.gates[static_cast<long long>(t) * 2 * p.H + p.H + h] = sigmoid(b);
+    }
+    return;
+  }
+  const int n = unit < 2 * p.G ? p.D : p.V;                       // channels of this head
+  const int c0 = unit < 2 * p.G ? unit * p.D : 2 * p.G * p.D + (unit - 2 * p.G) * p.V;
+  const int taps = p.taps;
+  float w[4][NI * VEC], hist[3][NI * VEC];
+  if (FAST) {
+#pragma unroll
+    for (int i = 0; i < NI; ++i)
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        const int c = i * 32 * VEC + lane * VEC + e;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const int k = j - (4 - taps);                           // fewer taps: leading zeros
+          w[j][i * VEC + e] = c < n && k >= 0 ? p.conv_w[static_cast<long long>(c0 + c) * taps + k] : 0.f;
+        }
+      }
+  }
+  int start = -1, prev = -1;
+  for (int t = t0; t < t1; ++t) {
+    const int b = p.row_seq[t] - p.seq0;
+    if (start < 0 || p.cu[b] != start) {
+      start = p.cu[b];
+      prev = p.row_prev[start];
+      if (FAST) {
+#pragma unroll
+        for (int i = 0; i < NI * VEC; ++i) {
+          const int c = (i / VEC) * 32 * VEC + lane * VEC + i % VEC;
+#pragma unroll
+          for (int j = 0; j < 3; ++j) hist[j][i] = c < n ? conv_input<T>(p, t - 3 + j, start, prev, c0 + c, C) : 0.f;
+        }
+      }
+    }
+    float y[NI * VEC], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int cb = i * 32 * VEC + lane * VEC;
+      float x[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) x[e] = 0.f;
+      if (cb < n) {
+        if (VEC == 2 && sizeof(T) == 2) {
+          const float2 f = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(proj + t * p.ld + c0 + cb));
+          x[0] = f.x;
+          x[VEC - 1] = f.y;
+        } else {
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) x[e] = to_f32(proj[t * p.ld + c0 + cb + e]);
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        const int q = i * VEC + e, c = cb + e;
+        float v = 0.f;
+        if (FAST) {
+          v = w[0][q] * hist[0][q] + w[1][q] * hist[1][q] + w[2][q] * hist[2][q] + w[3][q] * x[e];
+          hist[0][q] = hist[1][q];
+          hist[1][q] = hist[2][q];
+          hist[2][q] = x[e];
+        } else if (c < n) {
+          for (int j = 0; j < taps; ++j)
+            v += p.conv_w[static_cast<long long>(c0 + c) * taps + j] *
+                 conv_input<T>(p, t - (taps - 1) + j, start, prev, c0 + c, C);
+        }
+        y[q] = silu(v);
+        ss += y[q] * y[q];
+      }
+    }
+    float f = 1.f;
+    if (unit < 2 * p.G) f = (unit < p.G ? p.q_scale : 1.f) / sqrtf(warp_sum(ss) + 1e-6f);
+    float* dst = p.qkv + static_cast<long long>(t) * C + c0;
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int cb = i * 32 * VEC + lane * VEC;
+      if (cb < n) {
+        if (VEC == 2) *reinterpret_cast<float2*>(dst + cb) = make_float2(y[i * VEC] * f, y[i * VEC + VEC - 1] * f);
+        else dst[cb] = y[i] * f;
+      }
+    }
+    const int next = p.row_next[t];
+    if (next >= 0)
+      for (int c = lane; c < n; c += 32)
+        for (int j = 0; j < taps - 1; ++j)
+          p.state[next * p.state_ld + static_cast<long long>(j) * C + c0 + c] =
+              conv_input<T>(p, t - (taps - 2) + j, start, prev, c0 + c, C);
+  }
+}
+
+constexpr int SC_TILE = 32;                // tokens staged at a time
+constexpr int SC_WARPS = 4;
+
+// sum of v[32] over the LANES lanes of a column group; afterwards lane rl holds sums rl * 32 / LANES, ... in v[0 ..]
+template <int LANES> __device__ __forceinline__ void reduce_scatter(float (&v)[32], int rl) {
+#pragma unroll
+  for (int m = LANES / 2, n = 16; m > 0; m >>= 1, n >>= 1) {
+    const bool up = (rl & m) != 0;
+#pragma unroll
+    for (int j = 0; j < 16; ++j)
+      if (j < n) {
+        const float send = up ? v[j] : v[j + n], keep = up ? v[j + n] : v[j];
+        v[j] = keep + __shfl_xor_sync(0xffffffffu, send, m);
+      }
+  }
+}
+
+template <int LANES> struct DeltaScan {
+  static constexpr int DP = LANES * 8;                 // key rows, padded
+  static constexpr int KS = DP + 4;                    // row stride of a staged vector
+  static constexpr int NCW = 4 * (32 / LANES);         // columns per warp
+  static constexpr int NC = NCW * SC_WARPS;            // columns per CTA
+  static constexpr int STAGE = SC_TILE * (2 * KS + NC + 2);   // floats: q, k | v | log g, beta
+  static constexpr int COEF = 32;                      // per block: 6 L, 10 A, 4 beta g, 4 g, 4 r, 4 beta
+  static constexpr int XS = 16 * NCW;                  // per warp: 8 sums, 4 u, 4 r u per column
+  static constexpr size_t SMEM = (2 * STAGE + SC_TILE / 4 * COEF + SC_WARPS * XS) * sizeof(float);
+};
+
+// grid (column tiles, H, portions)
+template <int LANES>
+__global__ void __launch_bounds__(SC_WARPS * 32, LANES <= 16 ? 2 : 1) delta_scan_kernel(DeltaParams p) {
+  using Z = DeltaScan<LANES>;
+  extern __shared__ __align__(16) float smf[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, cg = lane / LANES, rl = lane % LANES;
+  const int h = blockIdx.y, g = h / (p.H / p.G), col_cta = blockIdx.x * Z::NC;
+  const int row0 = p.cu[blockIdx.z], n = p.cu[blockIdx.z + 1] - row0;
+  if (n <= 0) return;
+  const int C = 2 * p.G * p.D + p.H * p.V;
+  const int wc = warp * Z::NCW, col0 = col_cta + wc + cg * 4;      // this lane's four columns
+  float* coef = smf + 2 * Z::STAGE;
+  float* xs = coef + SC_TILE / 4 * Z::COEF + warp * Z::XS;         // [8][NCW]
+  float* us = xs + 8 * Z::NCW;                                     // [4][NCW]
+  float* ur = us + 4 * Z::NCW;                                     // [4][NCW]
+  const bool vec = p.D % 4 == 0 && p.V % 4 == 0;                   // then every staged piece is 16-byte aligned
+
+  auto stage_tile = [&](int s, int t) {
+    float* base = smf + s * Z::STAGE;
+    const float* src = p.qkv + static_cast<long long>(row0 + t) * C;
+    if (vec) {
+      constexpr int U = Z::DP / 4;
+      for (int i = threadIdx.x; i < SC_TILE * 2 * U; i += SC_WARPS * 32) {
+        const int tk = i / (2 * U), r = i - tk * 2 * U, w = r / U, c = (r - w * U) * 4;
+        const bool ok = t + tk < n && c < p.D;
+        cp_async16(base + (tk * 2 + w) * Z::KS + c, ok ? src + static_cast<long long>(tk) * C + (w * p.G + g) * p.D + c : p.qkv, ok);
+      }
+      for (int i = threadIdx.x; i < SC_TILE * Z::NC / 4; i += SC_WARPS * 32) {
+        const int tk = i / (Z::NC / 4), c = (i - tk * (Z::NC / 4)) * 4;
+        const bool ok = t + tk < n && col_cta + c < p.V;
+        cp_async16(base + SC_TILE * 2 * Z::KS + tk * Z::NC + c,
+                   ok ? src + static_cast<long long>(tk) * C + 2 * p.G * p.D + h * p.V + col_cta + c : p.qkv, ok);
+      }
+    } else {
+      for (int i = threadIdx.x; i < SC_TILE * 2 * Z::DP; i += SC_WARPS * 32) {
+        const int tk = i / (2 * Z::DP), r = i - tk * 2 * Z::DP, w = r / Z::DP, c = r - w * Z::DP;
+        const bool ok = t + tk < n && c < p.D;
+        cp_async4(base + (tk * 2 + w) * Z::KS + c, ok ? src + static_cast<long long>(tk) * C + (w * p.G + g) * p.D + c : p.qkv, ok);
+      }
+      for (int i = threadIdx.x; i < SC_TILE * Z::NC; i += SC_WARPS * 32) {
+        const int tk = i / Z::NC, c = i - tk * Z::NC;
+        const bool ok = t + tk < n && col_cta + c < p.V;
+        cp_async4(base + SC_TILE * 2 * Z::KS + tk * Z::NC + c,
+                  ok ? src + static_cast<long long>(tk) * C + 2 * p.G * p.D + h * p.V + col_cta + c : p.qkv, ok);
+      }
+    }
+    float* gt = base + SC_TILE * (2 * Z::KS + Z::NC);
+    for (int i = threadIdx.x; i < SC_TILE * 2; i += SC_WARPS * 32) {
+      const int tk = i >> 1;
+      const bool ok = t + tk < n;
+      cp_async4(gt + i, ok ? p.gates + static_cast<long long>(row0 + t + tk) * 2 * p.H + (i & 1) * p.H + h : p.gates, ok);
+    }
+    cp_commit();
+  };
+
+  // state: pairs of key rows r, r + 1 of column c; the lane's rows are 4 LANES j + 4 rl + {0, 1, 2, 3}
+  uint64_t S[4][4];
+  const int prev = p.row_prev[row0];
+#pragma unroll
+  for (int c = 0; c < 4; ++c)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int r = (j >> 1) * LANES * 4 + rl * 4 + (j & 1) * 2;
+      float a = 0.f, b = 0.f;
+      if (prev >= 0 && col0 + c < p.V) {
+        const float* src = p.state + prev * p.state_ld + p.s_off + static_cast<long long>(h) * p.D * p.V + col0 + c;
+        if (r < p.D) a = src[static_cast<long long>(r) * p.V];
+        if (r + 1 < p.D) b = src[static_cast<long long>(r + 1) * p.V];
+      }
+      S[c][j] = pack2(a, b);
+    }
+
+  stage_tile(0, 0);
+  int s = 0;
+  for (int t = 0; t < n; t += SC_TILE, s ^= 1) {
+    if (t + SC_TILE < n) {
+      stage_tile(s ^ 1, t + SC_TILE);
+      cp_wait<1>();
+    } else {
+      cp_wait<0>();
+    }
+    __syncthreads();
+    const float* base = smf + s * Z::STAGE;
+    const float* vt = base + SC_TILE * 2 * Z::KS;
+    const float* gt = vt + SC_TILE * Z::NC;
+    {   // Gram matrices and decays of the tile's blocks: 16 threads per block of four tokens
+      const int blk = threadIdx.x >> 4, e = threadIdx.x & 15;
+      int i, j, q = 0;                                   // pair (i, j): k_i . k_j for e < 6, q_i . k_j after that
+      if (e < 6) {
+        i = e < 1 ? 1 : (e < 3 ? 2 : 3);
+        j = e - i * (i - 1) / 2;
+        q = 1;
+      } else {
+        const int f = e - 6;
+        i = f < 1 ? 0 : (f < 3 ? 1 : (f < 6 ? 2 : 3));
+        j = f - i * (i + 1) / 2;
+      }
+      const float* x = base + ((blk * 4 + i) * 2 + q) * Z::KS;
+      const float* y = base + ((blk * 4 + j) * 2 + 1) * Z::KS;
+      float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f;
+#pragma unroll 8
+      for (int c = 0; c < Z::DP; c += 4) {
+        const float4 a = *reinterpret_cast<const float4*>(x + c), b = *reinterpret_cast<const float4*>(y + c);
+        d0 += a.x * b.x; d1 += a.y * b.y; d2 += a.z * b.z; d3 += a.w * b.w;
+      }
+      const float* lg = gt + blk * 8;                    // log g, beta alternate
+      float decay = 0.f;
+      for (int z = j + 1; z <= i; ++z) decay += lg[2 * z];
+      const float v = expf(decay) * ((d0 + d1) + (d2 + d3));
+      float* co = coef + blk * Z::COEF;
+      co[e] = e < 6 ? lg[2 * i + 1] * v : v;
+      if (e < 4) {
+        float head = 0.f, tail = 0.f;
+        for (int z = 0; z <= e; ++z) head += lg[2 * z];
+        for (int z = e + 1; z < 4; ++z) tail += lg[2 * z];
+        const float gh = expf(head), beta = lg[2 * e + 1];
+        co[16 + e] = beta * gh;
+        co[20 + e] = gh;
+        co[24 + e] = expf(tail);
+        co[28 + e] = beta;
+      }
+    }
+    __syncthreads();
+    const int blocks = (min(n - t, SC_TILE) + 3) / 4;
+    for (int blk = 0; blk < blocks; ++blk) {
+      const float* tok = base + blk * 4 * 2 * Z::KS;
+      const float* co = coef + blk * Z::COEF;
+      float v[32];                                       // [vector: k of four tokens, q of four tokens][column]
+      uint64_t kk[4][4];
+#pragma unroll
+      for (int x = 0; x < 8; ++x) {
+        const float* src = tok + ((x & 3) * 2 + (x < 4 ? 1 : 0)) * Z::KS + rl * 4;
+        const ulonglong2 a = *reinterpret_cast<const ulonglong2*>(src);
+        const ulonglong2 b = *reinterpret_cast<const ulonglong2*>(src + LANES * 4);
+        if (x < 4) {
+          kk[x][0] = a.x; kk[x][1] = a.y; kk[x][2] = b.x; kk[x][3] = b.y;
+        }
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          const float2 d = unpack2(fma2(S[c][3], b.y, fma2(S[c][2], b.x, fma2(S[c][1], a.y, mul2(S[c][0], a.x)))));
+          v[x * 4 + c] = d.x + d.y;
+        }
+      }
+      reduce_scatter<LANES>(v, rl);
+#pragma unroll
+      for (int e = 0; e < 32 / LANES; ++e) {
+        const int idx = rl * (32 / LANES) + e;
+        xs[(idx >> 2) * Z::NCW + cg * 4 + (idx & 3)] = v[e];
+      }
+      __syncwarp();
+      if (lane < Z::NCW) {                               // u of the four tokens, one column per lane
+        const float* vv = vt + blk * 4 * Z::NC + wc + lane;
+        const float4 bg = *reinterpret_cast<const float4*>(co + 16), rr = *reinterpret_cast<const float4*>(co + 24);
+        const float4 be = *reinterpret_cast<const float4*>(co + 28);
+        const float u0 = be.x * vv[0] - bg.x * xs[lane];
+        float u1 = be.y * vv[Z::NC] - bg.y * xs[Z::NCW + lane];
+        float u2 = be.z * vv[2 * Z::NC] - bg.z * xs[2 * Z::NCW + lane];
+        float u3 = be.w * vv[3 * Z::NC] - bg.w * xs[3 * Z::NCW + lane];
+        u1 -= co[0] * u0;
+        u2 -= co[1] * u0;
+        u3 -= co[3] * u0;
+        u2 -= co[2] * u1;
+        u3 -= co[4] * u1;
+        u3 -= co[5] * u2;
+        us[lane] = u0; us[Z::NCW + lane] = u1; us[2 * Z::NCW + lane] = u2; us[3 * Z::NCW + lane] = u3;
+        ur[lane] = rr.x * u0; ur[Z::NCW + lane] = rr.y * u1; ur[2 * Z::NCW + lane] = rr.z * u2; ur[3 * Z::NCW + lane] = rr.w * u3;
+      }
+      __syncwarp();
+      const uint64_t g4 = pack2(co[23], co[23]);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float4 f = *reinterpret_cast<const float4*>(ur + i * Z::NCW + cg * 4);
+        const uint64_t w[4] = {pack2(f.x, f.x), pack2(f.y, f.y), pack2(f.z, f.z), pack2(f.w, f.w)};
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) S[c][j] = fma2(kk[i][j], w[c], i == 0 ? mul2(S[c][j], g4) : S[c][j]);
+      }
+#pragma unroll
+      for (int x = 0; x < (4 * Z::NCW + 31) / 32; ++x) {
+        const int idx = x * 32 + lane, i = idx / Z::NCW, c = idx % Z::NCW;
+        if (idx < 4 * Z::NCW && t + blk * 4 + i < n && col_cta + wc + c < p.V) {
+          const float* A = co + 6 + i * (i + 1) / 2;
+          float o = co[20 + i] * xs[(4 + i) * Z::NCW + c];
+          for (int j = 0; j <= i; ++j) o += A[j] * us[j * Z::NCW + c];
+          p.o[static_cast<long long>(row0 + t + blk * 4 + i) * p.H * p.V + h * p.V + col_cta + wc + c] = o;
+        }
+      }
+      __syncwarp();
+    }
+    __syncthreads();
+  }
+  const int next = p.row_next[row0 + n - 1];
+  if (next >= 0) {
+#pragma unroll
+    for (int c = 0; c < 4; ++c)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int r = (j >> 1) * LANES * 4 + rl * 4 + (j & 1) * 2;
+        const float2 d = unpack2(S[c][j]);
+        if (col0 + c < p.V) {
+          float* dst = p.state + next * p.state_ld + p.s_off + static_cast<long long>(h) * p.D * p.V + col0 + c;
+          if (r < p.D) dst[static_cast<long long>(r) * p.V] = d.x;
+          if (r + 1 < p.D) dst[static_cast<long long>(r + 1) * p.V] = d.y;
+        }
+      }
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------
+// WKV
+// ---------------------------------------------------------------------------------------------------------
+struct WkvParams {
+  const void* rkvg;            // rows [r | k | v | gate], each H x D
+  long long ld;
+  const float* w_raw;          // [rows][H D]: exponent of the decay before '+ w0'
+  const float* w0;             // [H D]
+  const float* u;              // [H D]
+  const float* norm_w;         // [H D]
+  float eps;
+  float* state;
+  long long state_ld;
+  int s_off;
+  const int* row_prev;
+  const int* row_next;
+  const int* cu;               // portions
+  float* o;                    // portions: [rows][H D]
+  void* out;                   // decoding: [rows][out_ld]
+  long long out_ld;
+  int rows, H, D;
+};
+
+template <int LANES, typename T> struct WkvScan {
+  static constexpr int TT = LANES == 32 ? 16 : SC_TILE;            // tokens staged at a time
+  static constexpr int DP = LANES * 8;
+  static constexpr int NCW = 4 * (32 / LANES);
+  static constexpr int NC = NCW * SC_WARPS;
+  static constexpr int RAW = TT * ((2 * DP + NC) * static_cast<int>(sizeof(T)) + DP * 4);   // bytes: r | k | v | w
+  static constexpr int TILE = TT * (3 * DP + NC + 1);         // floats: r, k, decay | v | r . (u k)
+  static constexpr int XS = 8 * NCW;
+  static constexpr size_t SMEM = 2 * RAW + (TILE + SC_WARPS * XS + 2 * DP) * sizeof(float);
+};
+
+// grid (column tiles, H, portions)
+template <int LANES, typename T>
+__global__ void __launch_bounds__(SC_WARPS * 32) wkv_scan_kernel(WkvParams p) {
+  using Z = WkvScan<LANES, T>;
+  extern __shared__ __align__(16) uint8_t smb[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, cg = lane / LANES, rl = lane % LANES;
+  const int h = blockIdx.y, col_cta = blockIdx.x * Z::NC;
+  const int row0 = p.cu[blockIdx.z], n = p.cu[blockIdx.z + 1] - row0;
+  if (n <= 0) return;
+  const int HD = p.H * p.D, D = p.D;
+  const int wc = warp * Z::NCW, col0 = col_cta + wc + cg * 4;
+  float* tile = reinterpret_cast<float*>(smb + 2 * Z::RAW);        // [Z::TT][3][DP]
+  float* vt = tile + Z::TT * 3 * Z::DP;                          // [Z::TT][NC]
+  float* rk = vt + Z::TT * Z::NC;                                // [Z::TT]
+  float* xs = rk + Z::TT + warp * Z::XS;                         // [8][NCW]
+  float* w0s = rk + Z::TT + SC_WARPS * Z::XS;                    // [DP]
+  float* uss = w0s + Z::DP;                                        // [DP]
+  for (int c = threadIdx.x; c < Z::DP; c += SC_WARPS * 32) {
+    w0s[c] = c < D ? p.w0[h * D + c] : 0.f;
+    uss[c] = c < D ? p.u[h * D + c] : 0.f;
+  }
+  constexpr int E = 16 / sizeof(T);
+  const bool vec = D % 8 == 0 && p.ld % 8 == 0;
+  auto stage_tile = [&](int s, int t) {
+    T* raw = reinterpret_cast<T*>(smb + s * Z::RAW);
+    float* wr = reinterpret_cast<float*>(raw + Z::TT * (2 * Z::DP + Z::NC));
+    const T* src = reinterpret_cast<const T*>(p.rkvg) + (row0 + t) * p.ld + h * D;
+    const float* wsrc = p.w_raw + static_cast<long long>(row0 + t) * HD + h * D;
+    if (vec) {
+      for (int i = threadIdx.x; i < Z::TT * 2 * (Z::DP / E); i += SC_WARPS * 32) {
+        const int tk = i / (2 * (Z::DP / E)), r = i - tk * 2 * (Z::DP / E), w = r / (Z::DP / E), c = (r - w * (Z::DP / E)) * E;
+        const bool ok = t + tk < n && c < D;
+        cp_async16(raw + (tk * 2 + w) * Z::DP + c, ok ? src + tk * p.ld + w * HD + c : p.rkvg, ok);
+      }
+      for (int i = threadIdx.x; i < Z::TT * (Z::NC / E); i += SC_WARPS * 32) {
+        const int tk = i / (Z::NC / E), c = (i - tk * (Z::NC / E)) * E;
+        const bool ok = t + tk < n && col_cta + c < D;
+        cp_async16(raw + Z::TT * 2 * Z::DP + tk * Z::NC + c, ok ? src + tk * p.ld + 2 * HD + col_cta + c : p.rkvg, ok);
+      }
+      for (int i = threadIdx.x; i < Z::TT * (Z::DP / 4); i += SC_WARPS * 32) {
+        const int tk = i / (Z::DP / 4), c = (i - tk * (Z::DP / 4)) * 4;
+        const bool ok = t + tk < n && c < D;
+        cp_async16(wr + tk * Z::DP + c, ok ? wsrc + static_cast<long long>(tk) * HD + c : p.w_raw, ok);
+      }
+    } else {
+      const T zero = from_f32<T>(0.f);
+      for (int i = threadIdx.x; i < Z::TT * 2 * Z::DP; i += SC_WARPS * 32) {
+        const int tk = i / (2 * Z::DP), r = i - tk * 2 * Z::DP, w = r / Z::DP, c = r - w * Z::DP;
+        raw[i] = t + tk < n && c < D ? src[tk * p.ld + w * HD + c] : zero;
+      }
+      for (int i = threadIdx.x; i < Z::TT * Z::NC; i += SC_WARPS * 32) {
+        const int tk = i / Z::NC, c = i - tk * Z::NC;
+        raw[Z::TT * 2 * Z::DP + i] = t + tk < n && col_cta + c < D ? src[tk * p.ld + 2 * HD + col_cta + c] : zero;
+      }
+      for (int i = threadIdx.x; i < Z::TT * Z::DP; i += SC_WARPS * 32) {
+        const int tk = i / Z::DP, c = i - tk * Z::DP;
+        wr[i] = t + tk < n && c < D ? wsrc[static_cast<long long>(tk) * HD + c] : 0.f;
+      }
+    }
+    cp_commit();
+  };
+
+  uint64_t S[4][4];
+  const int prev = p.row_prev[row0];
+#pragma unroll
+  for (int c = 0; c < 4; ++c)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int r = (j >> 1) * LANES * 4 + rl * 4 + (j & 1) * 2;
+      float a = 0.f, b = 0.f;
+      if (prev >= 0 && col0 + c < D) {
+        const float* src = p.state + prev * p.state_ld + p.s_off + static_cast<long long>(h) * D * D + col0 + c;
+        if (r < D) a = src[static_cast<long long>(r) * D];
+        if (r + 1 < D) b = src[static_cast<long long>(r + 1) * D];
+      }
+      S[c][j] = pack2(a, b);
+    }
+
+  stage_tile(0, 0);
+  int s = 0;
+  for (int t = 0; t < n; t += Z::TT, s ^= 1) {
+    if (t + Z::TT < n) {
+      stage_tile(s ^ 1, t + Z::TT);
+      cp_wait<1>();
+    } else {
+      cp_wait<0>();
+    }
+    __syncthreads();
+    {
+      const T* raw = reinterpret_cast<const T*>(smb + s * Z::RAW);
+      const float* wr = reinterpret_cast<const float*>(raw + Z::TT * (2 * Z::DP + Z::NC));
+      for (int tk = warp; tk < Z::TT; tk += SC_WARPS) {
+        float dot = 0.f;
+        for (int c = lane; c < Z::DP; c += 32) {
+          const float r = to_f32(raw[tk * 2 * Z::DP + c]), k = to_f32(raw[(tk * 2 + 1) * Z::DP + c]);
+          tile[tk * 3 * Z::DP + c] = r;
+          tile[(tk * 3 + 1) * Z::DP + c] = k;
+          tile[(tk * 3 + 2) * Z::DP + c] = expf(-expf(wr[tk * Z::DP + c] + w0s[c]));
+          dot += r * uss[c] * k;
+        }
+        dot = warp_sum(dot);
+        if (lane == 0) rk[tk] = dot;
+        for (int c = lane; c < Z::NC; c += 32) vt[tk * Z::NC + c] = to_f32(raw[Z::TT * 2 * Z::DP + tk * Z::NC + c]);
+      }
+    }
+    __syncthreads();
+    const int m = min(n - t, Z::TT);
+    for (int b0 = 0; b0 < m; b0 += 8) {
+      float v[32];                                       // [token of the block][column]
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        if (b0 + i < m) {
+          const float* src = tile + (b0 + i) * 3 * Z::DP + rl * 4;
+          const ulonglong2 ra = *reinterpret_cast<const ulonglong2*>(src), rb = *reinterpret_cast<const ulonglong2*>(src + LANES * 4);
+          const ulonglong2 ka = *reinterpret_cast<const ulonglong2*>(src + Z::DP), kb = *reinterpret_cast<const ulonglong2*>(src + Z::DP + LANES * 4);
+          const ulonglong2 da = *reinterpret_cast<const ulonglong2*>(src + 2 * Z::DP), db = *reinterpret_cast<const ulonglong2*>(src + 2 * Z::DP + LANES * 4);
+          const float4 f = *reinterpret_cast<const float4*>(vt + (b0 + i) * Z::NC + wc + cg * 4);
+          const uint64_t w[4] = {pack2(f.x, f.x), pack2(f.y, f.y), pack2(f.z, f.z), pack2(f.w, f.w)};
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            const float2 d = unpack2(fma2(S[c][3], rb.y, fma2(S[c][2], rb.x, fma2(S[c][1], ra.y, mul2(S[c][0], ra.x)))));
+            v[i * 4 + c] = d.x + d.y;
+            S[c][0] = fma2(S[c][0], da.x, mul2(ka.x, w[c]));
+            S[c][1] = fma2(S[c][1], da.y, mul2(ka.y, w[c]));
+            S[c][2] = fma2(S[c][2], db.x, mul2(kb.x, w[c]));
+            S[c][3] = fma2(S[c][3], db.y, mul2(kb.y, w[c]));
+          }
+        } else {
+#pragma unroll
+          for (int c = 0; c < 4; ++c) v[i * 4 + c] = 0.f;
+        }
+      }
+      reduce_scatter<LANES>(v, rl);
+#pragma unroll
+      for (int e = 0; e < 32 / LANES; ++e) {
+        const int idx = rl * (32 / LANES) + e;
+        xs[(idx >> 2) * Z::NCW + cg * 4 + (idx & 3)] = v[e];
+      }
+      __syncwarp();
+#pragma unroll
+      for (int x = 0; x < (8 * Z::NCW + 31) / 32; ++x) {
+        const int idx = x * 32 + lane, i = idx / Z::NCW, c = idx % Z::NCW;
+        if (idx < 8 * Z::NCW && b0 + i < m && col_cta + wc + c < D)
+          p.o[static_cast<long long>(row0 + t + b0 + i) * HD + h * D + col_cta + wc + c] =
+              xs[i * Z::NCW + c] + rk[b0 + i] * vt[(b0 + i) * Z::NC + wc + c];
+      }
+      __syncwarp();
+    }
+    __syncthreads();
+  }
+  const int next = p.row_next[row0 + n - 1];
+  if (next >= 0) {
+#pragma unroll
+    for (int c = 0; c < 4; ++c)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int r = (j >> 1) * LANES * 4 + rl * 4 + (j & 1) * 2;
+        const float2 d = unpack2(S[c][j]);
+        if (col0 + c < D) {
+          float* dst = p.state + next * p.state_ld + p.s_off + static_cast<long long>(h) * D * D + col0 + c;
+          if (r < D) dst[static_cast<long long>(r) * D] = d.x;
+          if (r + 1 < D) dst[static_cast<long long>(r + 1) * D] = d.y;
+        }
+      }
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------
+// norm and gate of a scan's result: out = o / rms_head(o) * w * silu(gate) * scale, one warp per (row, head)
+// ---------------------------------------------------------------------------------------------------------
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+gated_norm_kernel(const float* __restrict__ o, const float* __restrict__ w, int w_head, const T* __restrict__ gate,
+                  long long gate_ld, T* __restrict__ out, long long out_ld, int rows, int H, int V, float eps, float scale) {
+  const int lane = threadIdx.x & 31;
+  const long long item = blockIdx.x * 8ll + (threadIdx.x >> 5);
+  if (item >= static_cast<long long>(rows) * H) return;
+  const int t = static_cast<int>(item / H), h = static_cast<int>(item % H);
+  const float* src = o + item * V;
+  float ss = 0.f;
+  for (int c = lane * VEC; c < V; c += 32 * VEC) {
+    if (VEC == 4) {
+      const float4 a = *reinterpret_cast<const float4*>(src + c);
+      ss += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
+    } else {
+      ss += src[c] * src[c];
+    }
+  }
+  const float inv = scale / sqrtf(warp_sum(ss) / static_cast<float>(V) + eps);
+  const T* g = gate + t * gate_ld + h * V;
+  T* dst = out + t * out_ld + h * V;
+  const float* wh = w + h * w_head;
+  for (int c = lane * VEC; c < V; c += 32 * VEC) {
+    float a[VEC], b[VEC];
+    if (VEC == 4) {
+      const float4 f = *reinterpret_cast<const float4*>(src + c);
+      a[0] = f.x; a[VEC > 1 ? 1 : 0] = f.y; a[VEC > 2 ? 2 : 0] = f.z; a[VEC > 3 ? 3 : 0] = f.w;
+    } else {
+      a[0] = src[c];
+    }
+    if (VEC == 4 && sizeof(T) == 2) {
+      const uint2 r = *reinterpret_cast<const uint2*>(g + c);
+      const float2 x = unpack_bf16x2(r.x), y = unpack_bf16x2(r.y);
+      b[0] = x.x; b[VEC > 1 ? 1 : 0] = x.y; b[VEC > 2 ? 2 : 0] = y.x; b[VEC > 3 ? 3 : 0] = y.y;
+    } else {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) b[e] = to_f32(g[c + e]);
+    }
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) a[e] = a[e] * inv * wh[c + e] * silu(b[e]);
+    if (VEC == 4 && sizeof(T) == 2) {
+      *reinterpret_cast<uint2*>(dst + c) = make_uint2(pack_bf16x2(a[0], a[VEC > 1 ? 1 : 0]), pack_bf16x2(a[VEC > 2 ? 2 : 0], a[VEC > 3 ? 3 : 0]));
+    } else {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) dst[c + e] = from_f32<T>(a[e]);
+    }
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------
+// single rows: projection -> gated result in one launch, one CTA per (row, head)
+// ---------------------------------------------------------------------------------------------------------
+constexpr int RS_THREADS = 256;
+
+template <int VEC> __device__ __forceinline__ void load_vec(const float* p, float (&v)[VEC]) {
+  if (VEC == 4) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    v[0] = a.x; v[VEC > 1 ? 1 : 0] = a.y; v[VEC > 2 ? 2 : 0] = a.z; v[VEC > 3 ? 3 : 0] = a.w;
+  } else {
+    v[0] = *p;
+  }
+}
+template <int VEC> __device__ __forceinline__ void store_vec(float* p, const float (&v)[VEC]) {
+  if (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[VEC > 1 ? 1 : 0], v[VEC > 2 ? 2 : 0], v[VEC > 3 ? 3 : 0]);
+  else *p = v[0];
+}
+
+// NR: key rows of the state a thread keeps in registers between the two passes (0: it reads them twice)
+template <typename T, int VEC, int NR>
+__global__ void __launch_bounds__(RS_THREADS) delta_step_kernel(DeltaParams p) {
+  extern __shared__ __align__(16) float smf[];
+  __shared__ float scratch[32];
+  const int row = blockIdx.x, h = blockIdx.y, g = h / (p.H / p.G), D = p.D, V = p.V, taps = p.taps, tid = threadIdx.x;
+  const int C = 2 * p.G * D + p.H * V, nvec = V / VEC, groups = RS_THREADS / nvec;
+  float* qs = smf;                         // [D]
+  float* ks = qs + D;                      // [D]
+  float* vs = ks + D;                      // [V], later u
+  float* part = smf + (2 * D + V + 3) / 4 * 4;   // [groups][V]
+  const int prev = p.row_prev[row], next = p.row_next[row];
+  const T* proj = reinterpret_cast<const T*>(p.proj) + row * p.ld;
+  const float* S = prev >= 0 ? p.state + prev * p.state_ld + p.s_off + static_cast<long long>(h) * D * V : nullptr;
+  float* N = next >= 0 ? p.state + next * p.state_ld + p.s_off + static_cast<long long>(h) * D * V : nullptr;
+  const int grp = tid / nvec, cv = (tid - grp * nvec) * VEC;
+  const bool on = grp < groups;
+  float st[NR > 0 ? NR : 1][VEC];
+  if (NR > 0) {                            // the state is on its way while the inputs are formed
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+      const int r = grp + i * groups;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) st[i][e] = 0.f;
+      if (on && S && r < D) load_vec<VEC>(S + static_cast<long long>(r) * V + cv, st[i]);
+    }
+  }
+  const bool owner = h % (p.H / p.G) == 0; // of the group's query / key convolution inputs
+  float sq = 0.f, sk = 0.f;
+  for (int i = tid; i < 2 * D + V; i += RS_THREADS) {
+    const int c = i < D ? g * D + i : (i < 2 * D ? p.G * D + g * D + i - D : 2 * p.G * D + h * V + i - 2 * D);
+    const float x = to_f32(proj[c]);
+    float y = p.conv_w[static_cast<long long>(c) * taps + taps - 1] * x;
+    const float* tail = prev >= 0 ? p.state + prev * p.state_ld + c : nullptr;
+    float* keep = next >= 0 && (i >= 2 * D || owner) ? p.state + next * p.state_ld + c : nullptr;
+    for (int j = 0; j < taps - 1; ++j) {
+      const float in = tail ? tail[static_cast<long long>(j) * C] : 0.f;
+      y += p.conv_w[static_cast<long long>(c) * taps + j] * in;
+      if (keep && j > 0) keep[static_cast<long long>(j - 1) * C] = in;
+    }
+    if (keep && taps > 1) keep[static_cast<long long>(taps - 2) * C] = x;
+    y = silu(y);
+    smf[i] = y;
+    if (i < D) sq += y * y;
+    else if (i < 2 * D) sk += y * y;
+  }
+  sq = block_sum(sq, scratch);
+  sk = block_sum(sk, scratch);             // also orders the inputs
+  const float fq = p.q_scale / sqrtf(sq + 1e-6f), fk = 1.f / sqrtf(sk + 1e-6f);
+  const int b0 = C + p.H * V;
+  const float beta = sigmoid(to_f32(proj[b0 + h]));
+  const float dec = expf(-expf(p.A_log[h]) * softplus(to_f32(proj[b0 + p.H + h]) + p.dt_bias[h]));
+  float acc[VEC];
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
+  if (on && S) {
+    if (NR > 0) {
+#pragma unroll
+      for (int i = 0; i < NR; ++i) {
+        const int r = grp + i * groups;
+        if (r < D) {
+          const float k = ks[r] * fk;
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) acc[e] += st[i][e] * k;
+        }
+      }
+    } else {
+      for (int r = grp; r < D; r += groups) {
+        float x[VEC];
+        load_vec<VEC>(S + static_cast<long long>(r) * V + cv, x);
+        const float k = ks[r] * fk;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) acc[e] += x[e] * k;
+      }
+    }
+  }
+  if (on) store_vec<VEC>(part + grp * V + cv, acc);
+  __syncthreads();
+  for (int c = tid; c < V; c += RS_THREADS) {
+    float s = 0.f;
+    for (int i = 0; i < groups; ++i) s += part[i * V + c];
+    vs[c] = beta * (vs[c] - dec * s);
+  }
+  __syncthreads();
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
+  if (on) {
+    float u[VEC];
+    load_vec<VEC>(vs + cv, u);
+    auto advance = [&](int r, float (&x)[VEC]) {
+      const float k = ks[r] * fk, q = qs[r] * fq;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        x[e] = dec * x[e] + k * u[e];
+        acc[e] += x[e] * q;
+      }
+      if (N) store_vec<VEC>(N + static_cast<long long>(r) * V + cv, x);
+    };
+    if (NR > 0) {
+#pragma unroll
+      for (int i = 0; i < NR; ++i) {
+        const int r = grp + i * groups;
+        if (r < D) advance(r, st[i]);
+      }
+    } else {
+      for (int r = grp; r < D; r += groups) {
+        float x[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x[e] = 0.f;
+        if (S) load_vec<VEC>(S + static_cast<long long>(r) * V + cv, x);
+        advance(r, x);
+      }
+    }
+    store_vec<VEC>(part + grp * V + cv, acc);
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int c = tid; c < V; c += RS_THREADS) {
+    float s = 0.f;
+    for (int i = 0; i < groups; ++i) s += part[i * V + c];
+    vs[c] = s;
+    ss += s * s;
+  }
+  ss = block_sum(ss, scratch);
+  const float inv = p.out_scale / sqrtf(ss / static_cast<float>(V) + p.eps);
+  T* out = reinterpret_cast<T*>(p.out) + row * p.out_ld + h * V;
+  for (int c = tid; c < V; c += RS_THREADS)
+    out[c] = from_f32<T>(vs[c] * inv * p.norm_w[c] * silu(to_f32(proj[C + h * V + c])));
+}
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(RS_THREADS) wkv_step_kernel(WkvParams p) {
+  extern __shared__ __align__(16) float smf[];
+  __shared__ float scratch[32];
+  const int row = blockIdx.x, h = blockIdx.y, D = p.D, HD = p.H * D, tid = threadIdx.x;
+  const int nvec = D / VEC, groups = RS_THREADS / nvec;
+  float* rs = smf;
+  float* ks = rs + D;
+  float* ws = ks + D;
+  float* vs = ws + D;
+  float* part = smf + (4 * D + 3) / 4 * 4;       // [groups][D]
+  const int prev = p.row_prev[row], next = p.row_next[row];
+  const T* x = reinterpret_cast<const T*>(p.rkvg) + row * p.ld + h * D;
+  float bonus = 0.f;
+  for (int c = tid; c < D; c += RS_THREADS) {
+    const float r = to_f32(x[c]), k = to_f32(x[HD + c]);
+    rs[c] = r;
+    ks[c] = k;
+    vs[c] = to_f32(x[2 * HD + c]);
+    ws[c] = expf(-expf(p.w_raw[static_cast<long long>(row) * HD + h * D + c] + p.w0[h * D + c]));
+    bonus += r * p.u[h * D + c] * k;
+  }
+  bonus = block_sum(bonus, scratch);
+  const int grp = tid / nvec, cv = (tid - grp * nvec) * VEC;
+  const float* S = prev >= 0 ? p.state + prev * p.state_ld + p.s_off + static_cast<long long>(h) * D * D : nullptr;
+  float* N = next >= 0 ? p.state + next * p.state_ld + p.s_off + static_cast<long long>(h) * D * D : nullptr;
+  if (grp < groups) {
+    float acc[VEC], v[VEC];
+    load_vec<VEC>(vs + cv, v);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
+#pragma unroll 4
+    for (int r = grp; r < D; r += groups) {
+      float st[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) st[e] = 0.f;
+      if (S) load_vec<VEC>(S + static_cast<long long>(r) * D + cv, st);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        acc[e] += st[e] * rs[r];
+        st[e] = ws[r] * st[e] + ks[r] * v[e];
+      }
+      if (N) store_vec<VEC>(N + static_cast<long long>(r) * D + cv, st);
+    }
+    store_vec<VEC>(part + grp * D + cv, acc);
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int c = tid; c < D; c += RS_THREADS) {
+    float s = bonus * vs[c];
+    for (int i = 0; i < groups; ++i) s += part[i * D + c];
+    rs[c] = s;                             // the row's r is no longer needed
+    ss += s * s;
+  }
+  ss = block_sum(ss, scratch);
+  const float inv = 1.f / sqrtf(ss / static_cast<float>(D) + p.eps);
+  T* out = reinterpret_cast<T*>(p.out) + row * p.out_ld + h * D;
+  for (int c = tid; c < D; c += RS_THREADS)
+    out[c] = from_f32<T>(rs[c] * inv * p.norm_w[h * D + c] * silu(to_f32(x[3 * HD + c])));
+}
+
+// ---------------------------------------------------------------------------------------------------------
+// launchers
+// ---------------------------------------------------------------------------------------------------------
+template <typename K> static int allow_smem(K kernel, size_t bytes) {
+  return bytes <= 48 * 1024 ? 0 : (int)cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
+}
+
+template <typename T, int VEC, int NI>
+static int launch_inputs(const DeltaParams& p, cudaStream_t st) {
+  const int units = 2 * p.G + p.H + 1;
+  const dim3 grid((p.rows + DI_TOKENS - 1) / DI_TOKENS, (units + 3) / 4);
+  if (p.taps <= 4) delta_inputs_kernel<T, VEC, NI, true><<<grid, 128, 0, st>>>(p);
+  else delta_inputs_kernel<T, VEC, NI, false><<<grid, 128, 0, st>>>(p);
+  return (int)cudaGetLastError();
+}
+
+template <typename T> static int dispatch_inputs(const DeltaParams& p, cudaStream_t st) {
+  const int most = p.D > p.V ? p.D : p.V;
+  if (p.D % 2 == 0 && p.V % 2 == 0 && p.ld % 2 == 0 && (reinterpret_cast<uintptr_t>(p.proj) & 3u) == 0) {
+    if (most <= 64) return launch_inputs<T, 2, 1>(p, st);
+    if (most <= 128) return launch_inputs<T, 2, 2>(p, st);
+    return launch_inputs<T, 2, 4>(p, st);
+  }
+  return most <= 64 ? launch_inputs<T, 1, 2>(p, st) : launch_inputs<T, 1, 8>(p, st);
+}
+
+template <int LANES> static int launch_delta_scan(const DeltaParams& p, int portions, cudaStream_t st) {
+  using Z = DeltaScan<LANES>;
+  if (int e = allow_smem(delta_scan_kernel<LANES>, Z::SMEM)) return e;
+  delta_scan_kernel<LANES><<<dim3((p.V + Z::NC - 1) / Z::NC, p.H, portions), SC_WARPS * 32, Z::SMEM, st>>>(p);
+  return (int)cudaGetLastError();
+}
+
+template <int LANES, typename T> static int launch_wkv_scan(const WkvParams& p, int portions, cudaStream_t st) {
+  using Z = WkvScan<LANES, T>;
+  if (int e = allow_smem(wkv_scan_kernel<LANES, T>, Z::SMEM)) return e;
+  wkv_scan_kernel<LANES, T><<<dim3((p.D + Z::NC - 1) / Z::NC, p.H, portions), SC_WARPS * 32, Z::SMEM, st>>>(p);
+  return (int)cudaGetLastError();
+}
+
+template <typename T> static int dispatch_wkv_scan(const WkvParams& p, int portions, cudaStream_t st) {
+  if (p.D <= 32) return launch_wkv_scan<4, T>(p, portions, st);
+  if (p.D <= 64) return launch_wkv_scan<8, T>(p, portions, st);
+  if (p.D <= 128) return launch_wkv_scan<16, T>(p, portions, st);
+  return launch_wkv_scan<32, T>(p, portions, st);
+}
+
+template <typename T, int VEC> static int launch_delta_step(const DeltaParams& p, cudaStream_t st) {
+  const int nvec = p.V / VEC, groups = RS_THREADS / nvec, per = (p.D + groups - 1) / groups;
+  const size_t smem = ((2 * p.D + p.V + 3) / 4 * 4 + static_cast<size_t>(groups) * p.V) * sizeof(float);
+  const dim3 grid(p.rows, p.H);
+  if (per <= 4) delta_step_kernel<T, VEC, 4><<<grid, RS_THREADS, smem, st>>>(p);
+  else if (per <= 8) delta_step_kernel<T, VEC, 8><<<grid, RS_THREADS, smem, st>>>(p);
+  else if (per <= 16) delta_step_kernel<T, VEC, 16><<<grid, RS_THREADS, smem, st>>>(p);
+  else delta_step_kernel<T, VEC, 0><<<grid, RS_THREADS, smem, st>>>(p);
+  return (int)cudaGetLastError();
+}
+
+template <typename T> static int launch_gated_norm(const float* o, const float* w, int w_head, const void* gate, long long gate_ld,
+                                                   void* out, long long out_ld, int rows, int H, int V, float eps, float scale,
+                                                   cudaStream_t st) {
+  const unsigned grid = (unsigned)((static_cast<long long>(rows) * H + 7) / 8);
+  const uintptr_t bits = reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(out);
+  const bool vec = V % 4 == 0 && gate_ld % 4 == 0 && out_ld % 4 == 0 && bits % (4 * sizeof(T)) == 0;
+  const T* g = reinterpret_cast<const T*>(gate);
+  T* d = reinterpret_cast<T*>(out);
+  if (vec) gated_norm_kernel<T, 4><<<grid, 256, 0, st>>>(o, w, w_head, g, gate_ld, d, out_ld, rows, H, V, eps, scale);
+  else gated_norm_kernel<T, 1><<<grid, 256, 0, st>>>(o, w, w_head, g, gate_ld, d, out_ld, rows, H, V, eps, scale);
+  return (int)cudaGetLastError();
+}
+
+static bool delta_sizes_ok(int H, int G, int D, int V, int taps) {
+  return H > 0 && G > 0 && H % G == 0 && D > 0 && V > 0 && D <= 256 && V <= 256 && taps >= 1 && H <= 65535;
+}
+
+}  // namespace ts
+
+TS_DEFINE_ERROR_API(ts_recurrent)
+using namespace ts;
+#define ST(s) reinterpret_cast<cudaStream_t>(s)
+
+// Portions of prompts, step 1: convolved inputs [rows][C] and gates [rows][2 H]; leaves the convolution state.
+extern "C" int ts_delta_inputs(const void* proj, long long ld, const float* conv_w, const float* A_log, const float* dt_bias,
+                               float q_scale, float* state, long long state_ld, const int* row_prev, const int* row_next,
+                               const int* cu, const int* row_seq, int seq0, float* qkv, float* gates, int rows, int H, int G,
+                               int D, int V, int taps, int fp32, void* stream) {
+  if (rows <= 0) return 0;
+  if (!delta_sizes_ok(H, G, D, V, taps)) return -10;
+  DeltaParams p = {};
+  p.proj = proj; p.ld = ld; p.conv_w = conv_w; p.A_log = A_log; p.dt_bias = dt_bias; p.q_scale = q_scale; p.state = state;
+  p.state_ld = state_ld; p.row_prev = row_prev; p.row_next = row_next; p.cu = cu; p.row_seq = row_seq; p.seq0 = seq0;
+  p.qkv = qkv; p.gates = gates; p.rows = rows; p.H = H; p.G = G; p.D = D; p.V = V; p.taps = taps;
+  return fp32 ? dispatch_inputs<float>(p, ST(stream)) : dispatch_inputs<__nv_bfloat16>(p, ST(stream));
+}
+
+// Portions, step 2: o [rows][H V] of the recurrence, the last state of every portion to its state row.
+extern "C" int ts_delta_scan(const float* qkv, const float* gates, float* state, long long state_ld, int s_off,
+                             const int* row_prev, const int* row_next, const int* cu, int portions, float* o, int H, int G,
+                             int D, int V, void* stream) {
+  if (portions <= 0) return 0;
+  if (!delta_sizes_ok(H, G, D, V, 1) || portions > 65535) return -10;
+  DeltaParams p = {};
+  p.qkv = const_cast<float*>(qkv); p.gates = const_cast<float*>(gates); p.state = state; p.state_ld = state_ld;
+  p.s_off = s_off; p.row_prev = row_prev; p.row_next = row_next; p.cu = cu; p.o = o; p.H = H; p.G = G; p.D = D; p.V = V;
+  if (D <= 32) return launch_delta_scan<4>(p, portions, ST(stream));
+  if (D <= 64) return launch_delta_scan<8>(p, portions, ST(stream));
+  if (D <= 128) return launch_delta_scan<16>(p, portions, ST(stream));
+  return launch_delta_scan<32>(p, portions, ST(stream));
+}
+
+// Portions, last step (either recurrence): o [rows][H V] fp32; w per channel (w_head = V) or shared by heads (w_head = 0).
+extern "C" int ts_gated_norm(const float* o, const float* w, int w_head, const void* gate, long long gate_ld, void* out,
+                             long long out_ld, int rows, int H, int V, float eps, float scale, int fp32, void* stream) {
+  if (rows <= 0) return 0;
+  if (H <= 0 || V <= 0) return -10;
+  return fp32 ? launch_gated_norm<float>(o, w, w_head, gate, gate_ld, out, out_ld, rows, H, V, eps, scale, ST(stream))
+              : launch_gated_norm<__nv_bfloat16>(o, w, w_head, gate, gate_ld, out, out_ld, rows, H, V, eps, scale, ST(stream));
+}
+
+// Single rows: projection -> out [rows][out_ld] = out_scale * gated norm, state and convolution state advanced.
+extern "C" int ts_delta_step(const void* proj, long long ld, const float* conv_w, const float* A_log, const float* dt_bias,
+                             const float* norm_w, float eps, float q_scale, float* state, long long state_ld, int s_off,
+                             const int* row_prev, const int* row_next, void* out, long long out_ld, float out_scale,
+                             int rows, int H, int G, int D, int V, int taps, int fp32, void* stream) {
+  if (rows <= 0) return 0;
+  if (!delta_sizes_ok(H, G, D, V, taps)) return -10;
+  DeltaParams p = {};
+  p.proj = proj; p.ld = ld; p.conv_w = conv_w; p.A_log = A_log; p.dt_bias = dt_bias; p.norm_w = norm_w; p.eps = eps;
+  p.q_scale = q_scale; p.state = state; p.state_ld = state_ld; p.s_off = s_off; p.row_prev = row_prev;
+  p.row_next = row_next; p.out = out; p.out_ld = out_ld; p.out_scale = out_scale; p.rows = rows; p.H = H; p.G = G;
+  p.D = D; p.V = V; p.taps = taps;
+  const bool vec = V % 4 == 0 && D % 2 == 0 && s_off % 4 == 0 && state_ld % 4 == 0;
+  if (fp32) return vec ? launch_delta_step<float, 4>(p, ST(stream)) : launch_delta_step<float, 1>(p, ST(stream));
+  return vec ? launch_delta_step<__nv_bfloat16, 4>(p, ST(stream)) : launch_delta_step<__nv_bfloat16, 1>(p, ST(stream));
+}
+
+// Portions: o [rows][H D] of the WKV recurrence.  rkvg rows: r | k | v | gate.
+extern "C" int ts_wkv_scan(const void* rkvg, long long ld, const float* w_raw, const float* w0, const float* u, float* state,
+                           long long state_ld, int s_off, const int* row_prev, const int* row_next, const int* cu,
+                           int portions, float* o, int H, int D, int fp32, void* stream) {
+  if (portions <= 0) return 0;
+  if (!delta_sizes_ok(H, H, D, D, 1) || portions > 65535) return -10;
+  WkvParams p = {};
+  p.rkvg = rkvg; p.ld = ld; p.w_raw = w_raw; p.w0 = w0; p.u = u; p.state = state; p.state_ld = state_ld; p.s_off = s_off;
+  p.row_prev = row_prev; p.row_next = row_next; p.cu = cu; p.o = o; p.H = H; p.D = D;
+  return fp32 ? dispatch_wkv_scan<float>(p, portions, ST(stream)) : dispatch_wkv_scan<__nv_bfloat16>(p, portions, ST(stream));
+}
+
+// Single rows of the WKV recurrence: projections -> out = gated norm, state advanced.
+extern "C" int ts_wkv_step(const void* rkvg, long long ld, const float* w_raw, const float* w0, const float* u,
+                           const float* norm_w, float eps, float* state, long long state_ld, int s_off, const int* row_prev,
+                           const int* row_next, void* out, long long out_ld, int rows, int H, int D, int fp32, void* stream) {
+  if (rows <= 0) return 0;
+  if (!delta_sizes_ok(H, H, D, D, 1)) return -10;
+  WkvParams p = {};
+  p.rkvg = rkvg; p.ld = ld; p.w_raw = w_raw; p.w0 = w0; p.u = u; p.norm_w = norm_w; p.eps = eps; p.state = state;
+  p.state_ld = state_ld; p.s_off = s_off; p.row_prev = row_prev; p.row_next = row_next; p.out = out; p.out_ld = out_ld;
+  p.rows = rows; p.H = H; p.D = D;
+  const bool vec = D % 4 == 0 && s_off % 4 == 0 && state_ld % 4 == 0;
+  const int groups = RS_THREADS / (vec ? D / 4 : D);
+  const size_t smem = ((4 * D + 3) / 4 * 4 + static_cast<size_t>(groups) * D) * sizeof(float);
+  const dim3 grid(rows, H);
+  if (fp32) {
+    if (vec) wkv_step_kernel<float, 4><<<grid, RS_THREADS, smem, ST(stream)>>>(p);
+    else wkv_step_kernel<float, 1><<<grid, RS_THREADS, smem, ST(stream)>>>(p);
+  } else {
+    if (vec) wkv_step_kernel<__nv_bfloat16, 4><<<grid, RS_THREADS, smem, ST(stream)>>>(p);
+    else wkv_step_kernel<__nv_bfloat16, 1><<<grid, RS_THREADS, smem, ST(stream)>>>(p);
+  }
+  return (int)cudaGetLastError();
+}

@@ -27,17 +27,10 @@ struct SkinnyParams {
   const int* count;            // [groups] rows of the group (nullptr: M)
   int a_div;                   // row of A = slot / a_div
   int M, N, K;
-  int act;                     // 0: none, 1: squared ReLU
+  int act;                     // of common.cuh product_act (0: none)
+  float act_cap;
   int out_fp32;
 };
-
-__device__ __forceinline__ float skinny_act(float v, int act) {
-  if (act == 1) {
-    v = fmaxf(v, 0.f);
-    return v * v;
-  }
-  return v;
-}
 
 __device__ __forceinline__ void mma_bf16_16816(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3,
                                                uint32_t b0, uint32_t b1) {
@@ -135,7 +128,7 @@ skinny_gemm_kernel(SkinnyParams p) {
         float v = 0.f;
 #pragma unroll
         for (int w = 0; w < KW; ++w) v += red[tile * KW + w][n][tk];
-        v = skinny_act(v, p.act);
+        v = product_act(v, p.act, p.act_cap);
         const int slot = p.order ? p.order[first + base + tk] : base + tk;
         const long long at = g * p.o_group + static_cast<long long>(slot) * p.ldo + nn;
         if (p.out_fp32) reinterpret_cast<float*>(p.out)[at] = v;
@@ -177,7 +170,7 @@ __global__ void __launch_bounds__(256) grouped_simt_kernel(SkinnyParams p) {
     }
 #pragma unroll
     for (int t = 0; t < TM; ++t) {
-      const float v = skinny_act(warp_sum(acc[t]), p.act);
+      const float v = product_act(warp_sum(acc[t]), p.act, p.act_cap);
       if (lane == 0 && base + t < m_total) {
         const long long at = g * p.o_group + static_cast<long long>(slot[t]) * p.ldo + n;
         if (p.out_fp32) reinterpret_cast<float*>(p.out)[at] = v;
@@ -207,14 +200,14 @@ using namespace ts;
 extern "C" int ts_skinny_gemm(const void* A, const void* W, void* out, long long lda, long long ldw, long long ldo,
                               long long a_group, long long w_group, long long o_group, const int* order,
                               const int* start, const int* count, int a_div, int groups, int M, int N, int K, int act,
-                              int fp32, int out_fp32, int typical, void* stream) {
+                              float act_cap, int fp32, int out_fp32, int typical, void* stream) {
   if (M <= 0 || groups <= 0) return 0;
-  if (N <= 0 || K <= 0 || a_div <= 0 || act < 0 || act > 1 || groups > 65535) return -10;
+  if (N <= 0 || K <= 0 || a_div <= 0 || act < 0 || act > 3 || (act == 3 && !(act_cap > 0.f)) || groups > 65535) return -10;
   if (fp32 && !out_fp32) return -11;
   SkinnyParams p;
   p.A = A; p.W = W; p.out = out; p.lda = lda; p.ldw = ldw; p.ldo = ldo; p.a_group = a_group; p.w_group = w_group;
   p.o_group = o_group; p.order = order; p.start = start; p.count = count; p.a_div = a_div; p.M = M; p.N = N; p.K = K;
-  p.act = act; p.out_fp32 = out_fp32;
+  p.act = act; p.act_cap = act_cap; p.out_fp32 = out_fp32;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   const bool vec = !fp32 && K % 8 == 0 && lda % 8 == 0 && ldw % 8 == 0 && a_group % 8 == 0 && w_group % 8 == 0 &&
                    aligned16(A) && aligned16(W);

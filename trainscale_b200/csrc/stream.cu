@@ -11,6 +11,11 @@
 // before in registers; for its first row it recomputes the row before (a halo) unless that row starts from a state
 // row or from zeros.  The stream, the history, the state and all arithmetic are fp32; h and hs leave in the activation
 // type.  Bandwidth-bound: every value of the history is read once per row (plus one halo row per run).
+//
+// `postnorm_kernel` is the boundary of decoders that norm a sublayer's OUTPUT and keep no history:
+//   source        x' = x + y / sqrt(mean(y^2) + eps) * (1 + w), or x' = embed[token] * scale
+//   outputs       x' (fp32); x' in the activation type, or n token-shift mixes of it, x' + (x'_prev - x') * mu_s;
+//                 last boundary: x' normed once more with the final weight, only for the rows that are wanted
 #include "common.cuh"
 #include "host_common.h"
 
@@ -290,6 +295,186 @@ static int launch_stream(const StreamParams& p, cudaStream_t st) {
   return -11;
 }
 
+struct PostnormParams {
+  const long long* tok;        // embedding source: [T]
+  const void* embed;           // [vocab][W]
+  float embed_scale;
+  int vocab;
+  const float* x_in;           // sublayer source: [T][W]
+  const void* y;               // [T][y_ld]
+  long long y_ld;
+  const float* w;              // [W], around zero
+  float eps;
+  float* x_out;                // [T][W] (not for FINAL)
+  void* h;                     // [rows][W], or [rows][n_mix][W]
+  const float* mu;             // [n_mix][W] or nullptr
+  int n_mix;
+  const int* row_prev;         // with mixes: as in StreamParams
+  const int* row_next;
+  float* state;                // previous x' of a sequence: first W values of a state row
+  long long state_ld;
+  const float* final_w;        // FINAL: [W]
+  const int* rows;             // FINAL: the rows to produce
+  int n_rows, W, rows_per_cta;
+};
+
+template <typename T, int MODE, int V, int NV>
+__global__ void __launch_bounds__(V == 4 ? 512 : 1024)
+postnorm_kernel(PostnormParams p) {
+  __shared__ float scratch[32];
+  const int W = p.W, nvec = W / V;
+
+  // v / rms(v) * (1 + w), in place
+  auto normed = [&](float (&v)[NV][V], const float* w) {
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+      if (threadIdx.x + i * blockDim.x < nvec) {
+#pragma unroll
+        for (int q = 0; q < V; ++q) ss += v[i][q] * v[i][q];
+      }
+    ss = block_sum(ss, scratch);
+    const float rms = sqrtf(ss / static_cast<float>(W) + p.eps);
+    const float inv = 1.f / rms;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c < nvec) {
+        float g[V];
+        VecIO<float>::load<V>(w + c * V, g);
+#pragma unroll
+        for (int q = 0; q < V; ++q) v[i][q] = v[i][q] * inv * (1.f + g[q]);
+      }
+    }
+  };
+
+  auto row_value = [&](int t, float (&v)[NV][V]) {
+    if (MODE == STREAM_EMBED) {
+      long long tok = p.tok[t];
+      if (tok < 0 || tok >= p.vocab) {
+        if (threadIdx.x == 0) ts_report_error(ERR_BOUNDS, 8001, static_cast<unsigned int>(tok));
+        tok = 0;
+      }
+      const T* e = reinterpret_cast<const T*>(p.embed) + static_cast<size_t>(tok) * W;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int c = threadIdx.x + i * blockDim.x;
+        if (c < nvec) {
+          VecIO<T>::template load<V>(e + c * V, v[i]);
+#pragma unroll
+          for (int q = 0; q < V; ++q) v[i][q] *= p.embed_scale;
+        }
+      }
+      return;
+    }
+    float x[NV][V];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c < nvec) {
+        VecIO<T>::template load<V>(reinterpret_cast<const T*>(p.y) + t * p.y_ld + c * V, v[i]);
+        VecIO<float>::load<V>(p.x_in + static_cast<size_t>(t) * W + c * V, x[i]);
+      }
+    }
+    normed(v, p.w);
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+      if (threadIdx.x + i * blockDim.x < nvec) {
+#pragma unroll
+        for (int q = 0; q < V; ++q) v[i][q] += x[i][q];
+      }
+  };
+
+  if (MODE == STREAM_FINAL) {
+    float v[NV][V];
+    row_value(p.rows[blockIdx.x], v);
+    normed(v, p.final_w);
+    T* h = reinterpret_cast<T*>(p.h) + static_cast<size_t>(blockIdx.x) * W;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c < nvec) VecIO<T>::template store<V>(h + c * V, v[i]);
+    }
+    return;
+  }
+
+  const int r0 = blockIdx.x * p.rows_per_cta, r1 = min(p.n_rows, r0 + p.rows_per_cta);
+  if (r0 >= r1) return;
+  float hp[NV][V];
+  if (p.n_mix && p.row_prev[r0] == -2) row_value(r0 - 1, hp);
+  for (int t = r0; t < r1; ++t) {
+    float v[NV][V];
+    row_value(t, v);
+    const int prev = p.n_mix ? p.row_prev[t] : -1, next = p.n_mix ? p.row_next[t] : -1;
+    const size_t base = static_cast<size_t>(t) * W;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c < nvec) {
+        VecIO<float>::store<V>(p.x_out + base + c * V, v[i]);
+        if (p.n_mix == 0) {
+          VecIO<T>::template store<V>(reinterpret_cast<T*>(p.h) + base + c * V, v[i]);
+        } else {
+          if (prev >= 0) {
+            VecIO<float>::load<V>(p.state + prev * p.state_ld + c * V, hp[i]);
+          } else if (prev == -1) {
+#pragma unroll
+            for (int q = 0; q < V; ++q) hp[i][q] = 0.f;
+          }
+          for (int s = 0; s < p.n_mix; ++s) {
+            float mu[V], m[V];
+            VecIO<float>::load<V>(p.mu + static_cast<size_t>(s) * W + c * V, mu);
+#pragma unroll
+            for (int q = 0; q < V; ++q) m[q] = v[i][q] + (hp[i][q] - v[i][q]) * mu[q];
+            VecIO<T>::template store<V>(reinterpret_cast<T*>(p.h) + base * p.n_mix + static_cast<size_t>(s) * W + c * V, m);
+          }
+          if (next >= 0) VecIO<float>::store<V>(p.state + next * p.state_ld + c * V, v[i]);
+#pragma unroll
+          for (int q = 0; q < V; ++q) hp[i][q] = v[i][q];
+        }
+      }
+    }
+  }
+}
+
+template <typename T, int MODE, int V, int NV>
+static int launch_postnorm_nv(PostnormParams p, int threads, cudaStream_t st) {
+  int grid = p.n_rows;
+  p.rows_per_cta = 1;
+  if (MODE != STREAM_FINAL && p.n_mix) {
+    static int per_sm[33] = {};
+    int& occ = per_sm[threads / 32];
+    if (occ == 0 && (cudaOccupancyMaxActiveBlocksPerMultiprocessor(&occ, postnorm_kernel<T, MODE, V, NV>, threads, 0) !=
+                         cudaSuccess || occ < 1))
+      occ = 1;
+    const int slots = occ * sm_count();
+    p.rows_per_cta = (p.n_rows + slots - 1) / slots;
+    if (p.rows_per_cta > 32) p.rows_per_cta = 32;
+    grid = (p.n_rows + p.rows_per_cta - 1) / p.rows_per_cta;
+  }
+  postnorm_kernel<T, MODE, V, NV><<<grid, threads, 0, st>>>(p);
+  return (int)cudaGetLastError();
+}
+
+template <typename T, int MODE>
+static int launch_postnorm(const PostnormParams& p, cudaStream_t st) {
+  const bool vec = p.W % 4 == 0 && p.y_ld % 4 == 0 && p.state_ld % 4 == 0;
+  const int nvec = vec ? p.W / 4 : p.W, cap = vec ? 512 : 1024;
+  int threads = (nvec + 31) / 32 * 32;
+  if (threads > cap) threads = cap;
+  const int nv = (nvec + threads - 1) / threads;
+  if (vec) {
+    if (nv <= 1) return launch_postnorm_nv<T, MODE, 4, 1>(p, threads, st);
+    if (nv <= 2) return launch_postnorm_nv<T, MODE, 4, 2>(p, threads, st);
+    if (nv <= 4) return launch_postnorm_nv<T, MODE, 4, 4>(p, threads, st);
+    if (nv <= 8) return launch_postnorm_nv<T, MODE, 4, 8>(p, threads, st);
+    return -11;
+  }
+  if (nv <= 1) return launch_postnorm_nv<T, MODE, 1, 1>(p, threads, st);
+  if (nv <= 8) return launch_postnorm_nv<T, MODE, 1, 8>(p, threads, st);
+  return -11;
+}
+
 }  // namespace ts
 
 TS_DEFINE_ERROR_API(ts_stream)
@@ -328,4 +513,35 @@ extern "C" int ts_stream_layer(const float* x_in, const void* mixer, int mixer_l
   if (rows_list)
     return fp32_act ? launch_stream<float, STREAM_FINAL>(p, st) : launch_stream<__nv_bfloat16, STREAM_FINAL>(p, st);
   return fp32_act ? launch_stream<float, STREAM_LAYER>(p, st) : launch_stream<__nv_bfloat16, STREAM_LAYER>(p, st);
+}
+
+// Boundary of output-normed decoders.  `tok`: embedding source (then x_in, y, w are unused).  `mu` with n_mix rows: h
+// receives the token-shift mixes [rows][n_mix][W] and the state row of `row_next` the row itself.
+extern "C" int ts_stream_postnorm(const long long* tok, const void* embed, int vocab, float embed_scale, const float* x_in,
+                                  const void* y, long long y_ld, const float* w, float eps, float* x_out, void* h,
+                                  const float* mu, int n_mix, const int* row_prev, const int* row_next, float* state,
+                                  long long state_ld, int rows, int W, int fp32_act, void* stream) {
+  if (rows <= 0) return 0;
+  if (W <= 0 || n_mix < 0 || (n_mix && (!mu || !state || state_ld < W))) return -10;
+  PostnormParams p = {};
+  p.tok = tok; p.embed = embed; p.vocab = vocab; p.embed_scale = embed_scale; p.x_in = x_in; p.y = y; p.y_ld = y_ld;
+  p.w = w; p.eps = eps; p.x_out = x_out; p.h = h; p.mu = mu; p.n_mix = n_mix; p.row_prev = row_prev;
+  p.row_next = row_next; p.state = state; p.state_ld = state_ld; p.n_rows = rows; p.W = W;
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  if (tok)
+    return fp32_act ? launch_postnorm<float, STREAM_EMBED>(p, st) : launch_postnorm<__nv_bfloat16, STREAM_EMBED>(p, st);
+  return fp32_act ? launch_postnorm<float, STREAM_LAYER>(p, st) : launch_postnorm<__nv_bfloat16, STREAM_LAYER>(p, st);
+}
+
+// Last boundary: the rows `rows_list`, residual sum and final norm -> h [n_out][W].
+extern "C" int ts_stream_postnorm_final(const float* x_in, const void* y, long long y_ld, const float* w,
+                                        const float* final_w, float eps, void* h, const int* rows_list, int n_out, int W,
+                                        int fp32_act, void* stream) {
+  if (n_out <= 0) return 0;
+  if (W <= 0) return -10;
+  PostnormParams p = {};
+  p.x_in = x_in; p.y = y; p.y_ld = y_ld; p.w = w; p.final_w = final_w; p.eps = eps; p.h = h; p.rows = rows_list;
+  p.n_rows = n_out; p.W = W;
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  return fp32_act ? launch_postnorm<float, STREAM_FINAL>(p, st) : launch_postnorm<__nv_bfloat16, STREAM_FINAL>(p, st);
 }

@@ -1,0 +1,548 @@
+// Sliding-window attention with grouped queries over a paged cache whose rows hold a token's keys and values side by side:
+// row = [G key heads x dim | G value heads x vdim | padding].
+//
+//   ts_window_prep    per-head RMS norm of queries and keys, rotary embedding of the first `rot` dimensions of a head
+//                     (in place in the projection), cache write of keys and values - one launch
+//   ts_window_attend  single query rows (decoding, fp32, and head sizes the prefill kernel does not take) against the paged
+//                     cache: keys max(0, len - window) <= j < len of the row's sequence
+// Portions of prompts: ts_window_prefill (latent_prefill.cu).
+//
+// Decoding reads every cached key and value in the window once per key/value head.  `window_attend_mma_kernel` (bf16): the
+// query heads of a group are the 16 rows of warp MMAs; every warp walks its own 16-key tiles through its own ring of
+// shared-memory stages (cp.async), with its own running softmax, so nothing in the loop waits for another warp.  Long
+// windows are split over CTAs and merged by log-sum-exp.  `window_attend_simt_kernel`: fp32 and sizes the tiles do not fit.
+#include "common.cuh"
+#include "host_common.h"
+
+namespace ts {
+
+template <typename T> __device__ __forceinline__ T from_f32(float v);
+template <> __device__ __forceinline__ float from_f32<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
+__device__ __forceinline__ float to_f32(float v) { return v; }
+__device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
+
+// ---------------------------------------------------------------------------------------------------------
+// norm, rotation, cache write
+// ---------------------------------------------------------------------------------------------------------
+struct WindowPrepParams {
+  void* proj;                  // rows [H x dim | G x dim | G x vdim | ...]
+  long long ld;
+  const float* q_norm;         // [dim]
+  const float* k_norm;
+  float eps;
+  const float* inv_freq;       // [rot / 2]
+  const int* pos;
+  const long long* slots;
+  void* cache;
+  int T, H, G, dim, vdim, rot, row_width;
+};
+
+constexpr int WP_WARPS = 4;
+
+// One CTA per token; a warp takes heads in turn.
+template <typename T>
+__global__ void __launch_bounds__(WP_WARPS * 32) window_prep_kernel(WindowPrepParams p) {
+  extern __shared__ float sm[];            // cos | sin of the token's angles
+  const int t = blockIdx.x, half = p.rot / 2, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float* cs = sm;
+  T* row = reinterpret_cast<T*>(p.proj) + t * p.ld;
+  T* crow = reinterpret_cast<T*>(p.cache) + p.slots[t] * p.row_width;
+  const float ps = static_cast<float>(p.pos[t]);
+  for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(ps * p.inv_freq[i], &cs[half + i], &cs[i]);
+  const T* v = row + (p.H + p.G) * p.dim;
+  for (int c = threadIdx.x; c < p.row_width - p.G * p.dim; c += blockDim.x)
+    crow[p.G * p.dim + c] = c < p.G * p.vdim ? v[c] : from_f32<T>(0.f);
+  __syncthreads();
+  for (int h = warp; h < p.H + p.G; h += WP_WARPS) {
+    T* x = row + h * p.dim;
+    float ss = 0.f;
+    for (int c = lane; c < p.dim; c += 32) {
+      const float a = to_f32(x[c]);
+      ss += a * a;
+    }
+    ss = warp_sum(ss);
+    const float inv = 1.f / sqrtf(ss / static_cast<float>(p.dim) + p.eps);
+    const float* w = h < p.H ? p.q_norm : p.k_norm;
+    T* out2 = h < p.H ? nullptr : crow + (h - p.H) * p.dim;
+    for (int i = lane; i < half; i += 32) {
+      const float a = to_f32(x[i]) * inv * w[i], b = to_f32(x[i + half]) * inv * w[i + half];
+      const T lo = from_f32<T>(a * cs[i] - b * cs[half + i]), hi = from_f32<T>(b * cs[i] + a * cs[half + i]);
+      x[i] = lo;
+      x[i + half] = hi;
+      if (out2) {
+        out2[i] = lo;
+        out2[i + half] = hi;
+      }
+    }
+    for (int c = p.rot + lane; c < p.dim; c += 32) {
+      const T y = from_f32<T>(to_f32(x[c]) * inv * w[c]);
+      x[c] = y;
+      if (out2) out2[c] = y;
+    }
+  }
+}
+
+// bf16, all sizes multiples of eight: LPH lanes hold one head as 16-byte vectors, 32 / LPH heads per warp pass; the two
+// halves of a rotated pair meet through shared memory.
+template <int LPH>
+__global__ void __launch_bounds__(WP_WARPS * 32) window_prep_vec_kernel(WindowPrepParams p) {
+  constexpr int HPW = 32 / LPH;
+  extern __shared__ float sm[];            // cos | sin [rot] | q_norm | k_norm | per warp and head slot [dim]
+  const int half = p.rot / 2, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float* cs = sm;
+  float* wq = sm + (p.rot + 3) / 4 * 4;
+  float* buf = wq + 2 * p.dim + (warp * HPW + lane / LPH) * p.dim;
+  const int sub = lane % LPH;
+  const bool in = sub * 8 < p.dim;
+  for (int c = threadIdx.x; c < 2 * p.dim; c += blockDim.x) wq[c] = c < p.dim ? p.q_norm[c] : p.k_norm[c - p.dim];
+  for (int t = blockIdx.x; t < p.T; t += gridDim.x) {
+    __nv_bfloat16* row = reinterpret_cast<__nv_bfloat16*>(p.proj) + t * p.ld;
+    __nv_bfloat16* crow = reinterpret_cast<__nv_bfloat16*>(p.cache) + p.slots[t] * p.row_width;
+    const float ps = static_cast<float>(p.pos[t]);
+    __syncthreads();                       // the angles of the token before are no longer read
+    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(ps * p.inv_freq[i], &cs[half + i], &cs[i]);
+    const uint4* v = reinterpret_cast<const uint4*>(row + (p.H + p.G) * p.dim);
+    uint4* cv = reinterpret_cast<uint4*>(crow + p.G * p.dim);
+    for (int c = threadIdx.x; c < p.G * p.vdim / 8; c += blockDim.x) cv[c] = v[c];
+    __syncthreads();
+    for (int h0 = warp * HPW; h0 < p.H + p.G; h0 += WP_WARPS * HPW) {
+      const int h = h0 + lane / LPH;
+      const bool on = in && h < p.H + p.G;
+      __nv_bfloat16* x = row + h * p.dim + sub * 8;
+      float a[8];
+      float ss = 0.f;
+      if (on) {
+        const uint4 raw = *reinterpret_cast<const uint4*>(x);
+        const uint32_t r[4] = {raw.x, raw.y, raw.z, raw.w};
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const float2 f = unpack_bf16x2(r[j]);
+          a[2 * j] = f.x;
+          a[2 * j + 1] = f.y;
+          ss += f.x * f.x + f.y * f.y;
+        }
+      }
+#pragma unroll
+      for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      const float inv = 1.f / sqrtf(ss / static_cast<float>(p.dim) + p.eps);
+      if (on) {
+        const float* w = (h < p.H ? wq : wq + p.dim) + sub * 8;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          a[j] *= inv * w[j];
+          if (sub * 8 < p.rot) buf[sub * 8 + j] = a[j];
+        }
+      }
+      __syncwarp();
+      if (on) {
+        if (sub * 8 < p.rot) {
+#pragma unroll
+          for (int j = 0; j < 8; ++j) {
+            const int c = sub * 8 + j;
+            if (c < half) a[j] = a[j] * cs[c] - buf[c + half] * cs[half + c];
+            else if (c < p.rot) a[j] = a[j] * cs[c - half] + buf[c - half] * cs[c];
+          }
+        }
+        const uint4 o = make_uint4(pack_bf16x2(a[0], a[1]), pack_bf16x2(a[2], a[3]), pack_bf16x2(a[4], a[5]),
+                                   pack_bf16x2(a[6], a[7]));
+        *reinterpret_cast<uint4*>(x) = o;
+        if (h >= p.H) *reinterpret_cast<uint4*>(crow + (h - p.H) * p.dim + sub * 8) = o;
+      }
+      __syncwarp();
+    }
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------
+// attention of single rows
+// ---------------------------------------------------------------------------------------------------------
+struct WindowAttendParams {
+  const void* q;               // rows [H x dim | ...]
+  long long q_ld;
+  const void* cache;           // [slots][row_width]
+  const int* block_table;      // [sequences][max_blocks]
+  const int* row_seq;          // [rows]
+  const int* row_len;          // [rows] keys visible before the window is applied (position + 1)
+  void* out;                   // [rows][out_ld], head h at column h * vdim
+  long long out_ld;
+  float* part_out;             // [rows][H][splits][vdim]
+  float* part_lse;             // [rows][H][splits]
+  int rows, H, G, dim, vdim, row_width, max_blocks, block_size, window, chunk, splits;
+  float scale, o_scale;
+};
+
+constexpr int WS_CHUNK = 512;
+
+// grid (rows, H).  Scores of WS_CHUNK keys at a time in shared memory, then threads own value columns.
+template <typename T>
+__global__ void __launch_bounds__(128) window_attend_simt_kernel(WindowAttendParams p) {
+  extern __shared__ float sm[];
+  __shared__ float scratch[32];
+  float* qs = sm;                          // [dim]
+  float* acc = sm + p.dim;                 // [vdim]
+  float* sc = acc + p.vdim;                // [WS_CHUNK]
+  const int row = blockIdx.x, h = blockIdx.y, g = h / (p.H / p.G);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  const int len = p.row_len[row];
+  const int* bt = p.block_table + static_cast<long long>(p.row_seq[row]) * p.max_blocks;
+  const T* cache = reinterpret_cast<const T*>(p.cache);
+  const T* q = reinterpret_cast<const T*>(p.q) + row * p.q_ld + h * p.dim;
+  for (int i = threadIdx.x; i < p.dim; i += blockDim.x) qs[i] = to_f32(q[i]);
+  for (int i = threadIdx.x; i < p.vdim; i += blockDim.x) acc[i] = 0.f;
+  float m = -INFINITY, l = 0.f;
+  for (int j0 = max(0, len - p.window); j0 < len; j0 += WS_CHUNK) {
+    const int j1 = min(len, j0 + WS_CHUNK);
+    __syncthreads();
+    float mx = -INFINITY;
+    for (int j = j0 + warp; j < j1; j += nw) {
+      const T* c = cache + (static_cast<long long>(bt[j / p.block_size]) * p.block_size + j % p.block_size) * p.row_width + g * p.dim;
+      float s = 0.f;
+      for (int i = lane; i < p.dim; i += 32) s += qs[i] * to_f32(c[i]);
+      s = warp_sum(s) * p.scale;
+      if (lane == 0) sc[j - j0] = s;
+      mx = fmaxf(mx, s);
+    }
+    const float m_new = fmaxf(m, block_max(mx, scratch));
+    const float alpha = expf(m - m_new);   // m = -inf at first: 0
+    float part = 0.f;
+    for (int j = j0 + threadIdx.x; j < j1; j += blockDim.x) {
+      const float w = expf(sc[j - j0] - m_new);
+      sc[j - j0] = w;
+      part += w;
+    }
+    l = l * alpha + block_sum(part, scratch);    // also orders the weights
+    m = m_new;
+    for (int r = threadIdx.x; r < p.vdim; r += blockDim.x) {
+      float a = acc[r] * alpha;
+      for (int j = j0; j < j1; ++j)
+        a += sc[j - j0] * to_f32(cache[(static_cast<long long>(bt[j / p.block_size]) * p.block_size + j % p.block_size) * p.row_width +
+                                       p.G * p.dim + g * p.vdim + r]);
+      acc[r] = a;
+    }
+  }
+  const float inv = l > 0.f ? p.o_scale / l : 0.f;
+  T* out = reinterpret_cast<T*>(p.out) + row * p.out_ld + h * p.vdim;
+  for (int r = threadIdx.x; r < p.vdim; r += blockDim.x) out[r] = from_f32<T>(acc[r] * inv);
+}
+
+constexpr int WA_WARPS = 4;
+constexpr int WA_STAGES = 3;
+constexpr int WA_KT = 16;
+
+__device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(addr));
+}
+__device__ __forceinline__ void ldsm_x4_t(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(addr));
+}
+__device__ __forceinline__ void mma_16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool valid) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(valid ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// shared-memory row stride in elements for `cols` columns (rounded up to 16): an odd number of 16-byte units
+__host__ __device__ inline int window_stride(int cols) { return (cols + 15) / 16 * 16 + 8; }
+static size_t window_smem(int dim, int vdim) {
+  const size_t ring = static_cast<size_t>(WA_WARPS) * WA_STAGES * WA_KT * (window_stride(dim) + window_stride(vdim)) * 2;
+  const size_t merge = static_cast<size_t>(WA_WARPS) * 16 * (vdim + 2) * 4;
+  return (ring > merge ? ring : merge) + 16 * window_stride(dim) * 2;
+}
+
+// grid (rows, G * ceil(group / 16), splits).  DC: head sizes up to DC columns.
+template <int DC>
+__global__ void __launch_bounds__(WA_WARPS * 32) window_attend_mma_kernel(WindowAttendParams p) {
+  constexpr int KS = DC / 16, NV = DC / 8;
+  extern __shared__ __align__(16) uint8_t raw[];
+  const int kst = window_stride(p.dim), vst = window_stride(p.vdim);
+  __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(raw);                       // [16][kst]
+  __nv_bfloat16* ring = qs + 16 * kst;
+  const int row = blockIdx.x, split = blockIdx.z;
+  const int group = p.H / p.G, tiles_h = (group + 15) / 16;
+  const int g = blockIdx.y / tiles_h, h0 = g * group + (blockIdx.y % tiles_h) * 16;
+  const int nh = min(16, (g + 1) * group - h0);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
+  const int len = p.row_len[row];
+  const int lo = max(0, len - p.window);
+  const int j0 = lo + split * p.chunk, j1 = min(len, j0 + p.chunk);
+  const int* bt = p.block_table + static_cast<long long>(p.row_seq[row]) * p.max_blocks;
+  const __nv_bfloat16* kc = reinterpret_cast<const __nv_bfloat16*>(p.cache) + g * p.dim;
+  const __nv_bfloat16* vc = reinterpret_cast<const __nv_bfloat16*>(p.cache) + p.G * p.dim + g * p.vdim;
+  const int ku = (p.dim + 15) / 16 * 2, vu = (p.vdim + 15) / 16 * 2;               // 16-byte units of a staged row
+  {
+    const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(p.q) + row * p.q_ld + h0 * p.dim;
+    for (int i = threadIdx.x; i < 16 * ku; i += blockDim.x) {
+      const int r = i / ku, c = i - r * ku;
+      *reinterpret_cast<uint4*>(qs + r * kst + c * 8) =
+          r < nh && c * 8 < p.dim ? *reinterpret_cast<const uint4*>(q + r * p.dim + c * 8) : make_uint4(0u, 0u, 0u, 0u);
+    }
+  }
+  __nv_bfloat16* mine = ring + warp * WA_STAGES * WA_KT * (kst + vst);
+  // this warp's tiles: keys t * 16 .. + 15 (absolute positions) for t = t_first + warp, + 4, ...
+  const int t_first = j0 / WA_KT, t_end = j1 > j0 ? (j1 + WA_KT - 1) / WA_KT : t_first;
+  auto slot_of = [&](int tile) {         // cache row of key tile * 16 + lane % 16 (-1: outside the range)
+    const int j = tile * WA_KT + (lane & 15);
+    return tile < t_end && j >= j0 && j < j1 ? bt[j / p.block_size] * p.block_size + j % p.block_size : -1;
+  };
+  auto load = [&](int stage, int slot) {
+    const uint32_t kd = smem_u32(mine + stage * WA_KT * (kst + vst)), vd = kd + WA_KT * kst * 2;
+    for (int i = lane; i < WA_KT * ku + (32 - WA_KT * ku % 32) % 32; i += 32) {
+      const int r = min(i / ku, WA_KT - 1), c = i - r * ku;
+      const int s = __shfl_sync(0xffffffffu, slot, r);
+      if (i < WA_KT * ku) {
+        const bool ok = s >= 0 && c * 8 < p.dim;
+        cp_async16(kd + (r * kst + c * 8) * 2, ok ? kc + static_cast<long long>(s) * p.row_width + c * 8 : kc, ok);
+      }
+    }
+    for (int i = lane; i < WA_KT * vu + (32 - WA_KT * vu % 32) % 32; i += 32) {
+      const int r = min(i / vu, WA_KT - 1), c = i - r * vu;
+      const int s = __shfl_sync(0xffffffffu, slot, r);
+      if (i < WA_KT * vu) {
+        const bool ok = s >= 0 && c * 8 < p.vdim;
+        cp_async16(vd + (r * vst + c * 8) * 2, ok ? vc + static_cast<long long>(s) * p.row_width + c * 8 : vc, ok);
+      }
+    }
+  };
+  int next = t_first + warp;
+  int slot = slot_of(next);
+#pragma unroll
+  for (int s = 0; s < WA_STAGES - 1; ++s) {
+    if (next < t_end) load(s, slot);
+    cp_commit();
+    next += WA_WARPS;
+    slot = slot_of(next);
+  }
+  __syncthreads();                         // queries staged
+  uint32_t qf[KS][4];
+#pragma unroll
+  for (int k = 0; k < KS; ++k)
+    if (k * 16 < p.dim) ldsm_x4(qf[k], smem_u32(qs + (lane & 15) * kst + k * 16 + (lane >> 4) * 8));
+  float o[NV][4];
+#pragma unroll
+  for (int n = 0; n < NV; ++n)
+#pragma unroll
+    for (int q = 0; q < 4; ++q) o[n][q] = 0.f;
+  float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
+  const float sl = p.scale * 1.4426950408889634f;
+  int stage = 0;
+  for (int t = t_first + warp; t < t_end; t += WA_WARPS) {
+    cp_wait<WA_STAGES - 2>();
+    __syncwarp();
+    const __nv_bfloat16* kt = mine + stage * WA_KT * (kst + vst);
+    const __nv_bfloat16* vt = kt + WA_KT * kst;
+    float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
+    const uint32_t ka = smem_u32(kt + ((lane & 7) + (lane >> 4) * 8) * kst + ((lane >> 3) & 1) * 8);
+#pragma unroll
+    for (int k = 0; k < KS; ++k)
+      if (k * 16 < p.dim) {
+        uint32_t b[4];                     // keys 0-7: b[0], b[1]; keys 8-15: b[2], b[3]
+        ldsm_x4(b, ka + k * 32);
+        mma_16816(s0, qf[k], b[0], b[1]);
+        mma_16816(s1, qf[k], b[2], b[3]);
+      }
+    const int j = t * WA_KT + tig * 2;
+    auto keep = [&](float v, int key) { return key >= j0 && key < j1 ? v * sl : -INFINITY; };
+    s0[0] = keep(s0[0], j); s0[1] = keep(s0[1], j + 1); s0[2] = keep(s0[2], j); s0[3] = keep(s0[3], j + 1);
+    s1[0] = keep(s1[0], j + 8); s1[1] = keep(s1[1], j + 9); s1[2] = keep(s1[2], j + 8); s1[3] = keep(s1[3], j + 9);
+    float a = fmaxf(fmaxf(s0[0], s0[1]), fmaxf(s1[0], s1[1])), b = fmaxf(fmaxf(s0[2], s0[3]), fmaxf(s1[2], s1[3]));
+    a = fmaxf(a, __shfl_xor_sync(0xffffffffu, a, 1));
+    b = fmaxf(b, __shfl_xor_sync(0xffffffffu, b, 1));
+    a = fmaxf(m0, fmaxf(a, __shfl_xor_sync(0xffffffffu, a, 2)));   // finite: every tile has a key in the range
+    b = fmaxf(m1, fmaxf(b, __shfl_xor_sync(0xffffffffu, b, 2)));
+    const float f0 = fast_ex2(m0 - a), f1 = fast_ex2(m1 - b);
+    m0 = a;
+    m1 = b;
+    s0[0] = fast_ex2(s0[0] - a); s0[1] = fast_ex2(s0[1] - a); s1[0] = fast_ex2(s1[0] - a); s1[1] = fast_ex2(s1[1] - a);
+    s0[2] = fast_ex2(s0[2] - b); s0[3] = fast_ex2(s0[3] - b); s1[2] = fast_ex2(s1[2] - b); s1[3] = fast_ex2(s1[3] - b);
+    l0 = l0 * f0 + ((s0[0] + s0[1]) + (s1[0] + s1[1]));
+    l1 = l1 * f1 + ((s0[2] + s0[3]) + (s1[2] + s1[3]));
+    const uint32_t pf[4] = {pack_bf16x2(s0[0], s0[1]), pack_bf16x2(s0[2], s0[3]), pack_bf16x2(s1[0], s1[1]),
+                            pack_bf16x2(s1[2], s1[3])};
+    const uint32_t va = smem_u32(vt + (lane & 15) * vst + (lane >> 4) * 8);
+#pragma unroll
+    for (int n = 0; n < NV; n += 2)
+      if (n * 8 < p.vdim) {
+        uint32_t bv[4];                    // columns 8 n: bv[0], bv[1]; the next eight: bv[2], bv[3]
+        ldsm_x4_t(bv, va + n * 16);
+        o[n][0] *= f0; o[n][1] *= f0; o[n][2] *= f1; o[n][3] *= f1;
+        o[n + 1][0] *= f0; o[n + 1][1] *= f0; o[n + 1][2] *= f1; o[n + 1][3] *= f1;
+        mma_16816(o[n], pf, bv[0], bv[1]);
+        mma_16816(o[n + 1], pf, bv[2], bv[3]);
+      }
+    __syncwarp();                          // all lanes are done with the stage that is filled next
+    {
+      const int fill = stage == 0 ? WA_STAGES - 1 : stage - 1;
+      if (next < t_end) load(fill, slot);
+      cp_commit();
+      next += WA_WARPS;
+      slot = slot_of(next);
+    }
+    stage = stage + 1 == WA_STAGES ? 0 : stage + 1;
+  }
+  l0 += __shfl_xor_sync(0xffffffffu, l0, 1);
+  l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
+  l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
+  l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+  cp_wait<0>();
+  __syncthreads();
+  // merge of the four warps: [warp][16][vdim + 2] = sums, maximum, weight
+  float* mg = reinterpret_cast<float*>(ring);
+  const int ms = p.vdim + 2;
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {
+    float* d = mg + (warp * 16 + gid + half * 8) * ms;
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+      const int c = n * 8 + tig * 2;
+      if (c < p.vdim) {
+        d[c] = o[n][2 * half];
+        d[c + 1] = o[n][2 * half + 1];
+      }
+    }
+    if (tig == 0) {
+      d[p.vdim] = half ? m1 : m0;
+      d[p.vdim + 1] = half ? l1 : l0;
+    }
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < nh * p.vdim; i += blockDim.x) {
+    const int r = i / p.vdim, c = i - r * p.vdim;
+    float mm = -INFINITY, l = 0.f, acc = 0.f;
+#pragma unroll
+    for (int w = 0; w < WA_WARPS; ++w) mm = fmaxf(mm, mg[(w * 16 + r) * ms + p.vdim]);
+#pragma unroll
+    for (int w = 0; w < WA_WARPS; ++w) {
+      const float* d = mg + (w * 16 + r) * ms;
+      const float f = d[p.vdim] == -INFINITY ? 0.f : fast_ex2(d[p.vdim] - mm);
+      l += d[p.vdim + 1] * f;
+      acc += d[c] * f;
+    }
+    const int h = h0 + r;
+    if (p.splits == 1) {
+      reinterpret_cast<__nv_bfloat16*>(p.out)[row * p.out_ld + h * p.vdim + c] = __float2bfloat16(l > 0.f ? acc * (p.o_scale / l) : 0.f);
+    } else {
+      const long long at = (static_cast<long long>(row) * p.H + h) * p.splits + split;
+      p.part_out[at * p.vdim + c] = l > 0.f ? acc / l : 0.f;
+      if (c == 0) p.part_lse[at] = l > 0.f ? mm + log2f(l) : -INFINITY;      // in powers of two
+    }
+  }
+}
+
+constexpr int WM_MAX_SPLITS = 64;
+__global__ void __launch_bounds__(128) window_merge_kernel(WindowAttendParams p) {
+  const int row = blockIdx.x, h = blockIdx.y;
+  const long long base = (static_cast<long long>(row) * p.H + h) * p.splits;
+  float mm = -INFINITY, l = 0.f;
+  for (int s = 0; s < p.splits; ++s) mm = fmaxf(mm, p.part_lse[base + s]);
+  for (int s = 0; s < p.splits; ++s) l += fast_ex2(p.part_lse[base + s] - mm);
+  for (int c = threadIdx.x; c < p.vdim; c += blockDim.x) {
+    float acc = 0.f;
+    for (int s = 0; s < p.splits; ++s) acc += fast_ex2(p.part_lse[base + s] - mm) * p.part_out[(base + s) * p.vdim + c];
+    reinterpret_cast<__nv_bfloat16*>(p.out)[row * p.out_ld + h * p.vdim + c] = __float2bfloat16(acc * (p.o_scale / l));
+  }
+}
+
+template <int DC> static int launch_window_mma(const WindowAttendParams& p, cudaStream_t st) {
+  const size_t smem = window_smem(p.dim, p.vdim);
+  static bool configured = false;
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(window_attend_mma_kernel<DC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+    if (e != cudaSuccess) return (int)e;
+    configured = true;
+  }
+  const int tiles_h = (p.H / p.G + 15) / 16;
+  window_attend_mma_kernel<DC><<<dim3(p.rows, p.G * tiles_h, p.splits), WA_WARPS * 32, smem, st>>>(p);
+  return (int)cudaGetLastError();
+}
+
+static bool window_mma_ok(int dim, int vdim, int fp32) {
+  return !fp32 && dim % 8 == 0 && vdim % 8 == 0 && dim <= 256 && vdim <= 256 && window_smem(dim, vdim) <= 227 * 1024;
+}
+
+}  // namespace ts
+
+TS_DEFINE_ERROR_API(ts_window)
+using namespace ts;
+#define ST(s) reinterpret_cast<cudaStream_t>(s)
+
+extern "C" int ts_window_prep(void* proj, long long ld, const float* q_norm, const float* k_norm, float eps,
+                              const float* inv_freq, const int* pos, const long long* slots, void* cache, int T, int H,
+                              int G, int dim, int vdim, int rot, int row_width, int fp32, void* stream) {
+  if (T <= 0) return 0;
+  if (H <= 0 || G <= 0 || dim <= 0 || vdim <= 0 || rot < 0 || rot > dim || rot % 2 || row_width < G * (dim + vdim)) return -10;
+  WindowPrepParams p;
+  p.proj = proj; p.ld = ld; p.q_norm = q_norm; p.k_norm = k_norm; p.eps = eps; p.inv_freq = inv_freq; p.pos = pos;
+  p.slots = slots; p.cache = cache; p.T = T; p.H = H; p.G = G; p.dim = dim; p.vdim = vdim; p.rot = rot;
+  p.row_width = row_width;
+  const bool vec = !fp32 && dim % 8 == 0 && vdim % 8 == 0 && dim <= 256 && ld % 8 == 0 && row_width % 8 == 0 &&
+                   row_width == G * (dim + vdim) && (reinterpret_cast<uintptr_t>(proj) & 15u) == 0;
+  if (vec) {
+    int lph = 4;
+    while (lph * 8 < dim) lph *= 2;
+    const size_t smem = ((rot + 3) / 4 * 4 + 2 * dim + static_cast<size_t>(WP_WARPS) * (32 / lph) * dim) * 4;
+    int grid = sm_count() * 8;
+    if (grid > T) grid = T;
+    if (lph == 4) window_prep_vec_kernel<4><<<grid, WP_WARPS * 32, smem, ST(stream)>>>(p);
+    else if (lph == 8) window_prep_vec_kernel<8><<<grid, WP_WARPS * 32, smem, ST(stream)>>>(p);
+    else if (lph == 16) window_prep_vec_kernel<16><<<grid, WP_WARPS * 32, smem, ST(stream)>>>(p);
+    else window_prep_vec_kernel<32><<<grid, WP_WARPS * 32, smem, ST(stream)>>>(p);
+    return (int)cudaGetLastError();
+  }
+  const size_t smem = (rot + 4) * sizeof(float);
+  if (fp32) window_prep_kernel<float><<<T, WP_WARPS * 32, smem, ST(stream)>>>(p);
+  else window_prep_kernel<__nv_bfloat16><<<T, WP_WARPS * 32, smem, ST(stream)>>>(p);
+  return (int)cudaGetLastError();
+}
+
+// Split count of ts_window_attend for `keys` visible keys: enough CTAs for two per SM, at least 128 keys each.
+extern "C" int ts_window_splits(int rows, int H, int G, int dim, int vdim, int keys, int fp32) {
+  if (!window_mma_ok(dim, vdim, fp32)) return 1;
+  const int ctas = rows * G * ((H / G + 15) / 16);
+  int s = (2 * sm_count() + ctas - 1) / ctas, most = (keys + 127) / 128;
+  if (s > most) s = most;
+  if (s > WM_MAX_SPLITS) s = WM_MAX_SPLITS;
+  return s < 1 ? 1 : s;
+}
+
+// `keys`: upper bound of the keys a row sees; `splits` of ts_window_splits with the workspaces it needs (splits > 1).
+extern "C" int ts_window_attend(const void* q, long long q_ld, const void* cache, const int* block_table, int max_blocks,
+                                const int* row_seq, const int* row_len, void* out, long long out_ld, float* part_out,
+                                float* part_lse, int rows, int H, int G, int dim, int vdim, int row_width, int block_size,
+                                int window, int keys, int splits, float scale, float o_scale, int fp32, void* stream) {
+  if (rows <= 0) return 0;
+  if (H <= 0 || G <= 0 || H % G || dim <= 0 || vdim <= 0 || window <= 0 || keys <= 0 || splits < 1 || splits > WM_MAX_SPLITS)
+    return -10;
+  WindowAttendParams p;
+  p.q = q; p.q_ld = q_ld; p.cache = cache; p.block_table = block_table; p.row_seq = row_seq; p.row_len = row_len; p.out = out;
+  p.out_ld = out_ld; p.part_out = part_out; p.part_lse = part_lse; p.rows = rows; p.H = H; p.G = G; p.dim = dim;
+  p.vdim = vdim; p.row_width = row_width; p.max_blocks = max_blocks; p.block_size = block_size; p.window = window;
+  p.splits = splits; p.chunk = ((keys + splits - 1) / splits + 15) / 16 * 16; p.scale = scale; p.o_scale = o_scale;
+  const bool vec = window_mma_ok(dim, vdim, fp32) && scale > 0.f && q_ld % 8 == 0 && row_width % 8 == 0 &&
+                   (reinterpret_cast<uintptr_t>(q) & 15u) == 0 && (reinterpret_cast<uintptr_t>(cache) & 15u) == 0;
+  if (!vec) {
+    const size_t smem = (dim + vdim + WS_CHUNK) * sizeof(float);
+    if (smem > 48 * 1024) return -11;
+    if (fp32) window_attend_simt_kernel<float><<<dim3(rows, H), 128, smem, ST(stream)>>>(p);
+    else window_attend_simt_kernel<__nv_bfloat16><<<dim3(rows, H), 128, smem, ST(stream)>>>(p);
+    return (int)cudaGetLastError();
+  }
+  const int dc = dim > vdim ? dim : vdim;
+  int rc = dc <= 64 ? launch_window_mma<64>(p, ST(stream))
+                    : (dc <= 128 ? launch_window_mma<128>(p, ST(stream)) : launch_window_mma<256>(p, ST(stream)));
+  if (rc == 0 && splits > 1) {
+    window_merge_kernel<<<dim3(rows, H), 128, 0, ST(stream)>>>(p);
+    rc = (int)cudaGetLastError();
+  }
+  return rc;
+}

@@ -32,6 +32,17 @@ class PromptContext:
     slots: torch.Tensor | None    # cache slot of every key row; None: the keys are exactly the new tokens
 
 
+@dataclass
+class Portions:
+    """The batch's multi-token entries, by row relative to the first multi-token row."""
+    offsets: list[int]            # [count + 1]
+    cu: torch.Tensor              # int32 copy on the device
+
+    @property
+    def count(self) -> int:
+        return len(self.offsets) - 1
+
+
 class HostBatch:
     """Host side of a step: tokens are appended to the cache, index lists are built.  Single-token entries come first
     (`order` maps batch position -> entry), so that decoding rows and portions of prompts are contiguous."""
@@ -132,6 +143,18 @@ class StepBatch:
                 cu.append(cu[-1] + n)
             self._contexts["cu_q"] = torch.tensor(cu, dtype=torch.int32).to(self.token_ids.device)
         return self._contexts["cu_q"]
+
+    @property
+    def portions(self) -> Portions | None:
+        """Row offsets of the multi-token entries (None: no such entries)."""
+        if self.host is None or self.host.all_single:
+            return None
+        if "portions" not in self._contexts:
+            at = [0]
+            for n in self.host.q_lens[self.host.n_single:]:
+                at.append(at[-1] + n)
+            self._contexts["portions"] = Portions(at, torch.tensor(at, dtype=torch.int32).to(self.token_ids.device))
+        return self._contexts["portions"]
 
     def prompt_context(self, window: int) -> PromptContext | None:
         """Key rows of the multi-token entries when a position sees `window` keys (None: no such entries)."""

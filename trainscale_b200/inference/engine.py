@@ -536,7 +536,7 @@ class EngineCore:
         spec = self.model.cache_spec() if hasattr(self.model, "cache_spec") else \
             CacheSpec.kv(c.num_hidden_layers, c.num_key_value_heads // tps, c.head_dim)
         if nb is None:
-            per_block = cc.block_size * spec.bytes_per_token(2 if dtype != torch.float32 else 4)
+            per_block = max(1, cc.block_size * spec.bytes_per_token(2 if dtype != torch.float32 else 4))
             if self.device.type == "cuda":
                 free, _ = torch.cuda.mem_get_info(self.device)
                 nb = max(64, int(free * cc.gpu_memory_utilization * 0.5) // per_block)

@@ -9,27 +9,33 @@ import torch
 from . import _lib
 
 _ll = ctypes.c_longlong
-ACT_NONE, ACT_RELU_SQUARED = 0, 1
+ACT_NONE, ACT_RELU_SQUARED, ACT_TANH, ACT_SOFTCAP = 0, 1, 2, 3
 
 
-def activate(x: torch.Tensor, act: int) -> torch.Tensor:
-    return torch.relu(x).square() if act == ACT_RELU_SQUARED else x
+def activate(x: torch.Tensor, act: int, cap: float = 0.0) -> torch.Tensor:
+    if act == ACT_RELU_SQUARED:
+        return torch.relu(x).square()
+    if act == ACT_TANH:
+        return torch.tanh(x)
+    return cap * torch.tanh(x / cap) if act == ACT_SOFTCAP else x
 
 
 def _launch(A, W, out, lda, ldw, ldo, a_group, w_group, o_group, order, start, count, a_div, groups, M, N, K, act,
-            typical=0):
+            typical=0, cap=0.0):
     rc = _lib.load("skinny").ts_skinny_gemm(
         _lib.ptr(A), _lib.ptr(W), _lib.ptr(out), _ll(lda), _ll(ldw), _ll(ldo), _ll(a_group), _ll(w_group), _ll(o_group),
-        _lib.ptr(order), _lib.ptr(start), _lib.ptr(count), a_div, groups, M, N, K, act, int(A.dtype == torch.float32),
-        int(out.dtype == torch.float32), typical, _lib.stream_ptr())
+        _lib.ptr(order), _lib.ptr(start), _lib.ptr(count), a_div, groups, M, N, K, act, ctypes.c_float(cap),
+        int(A.dtype == torch.float32), int(out.dtype == torch.float32), typical, _lib.stream_ptr())
     _lib.check(rc, "ts_skinny_gemm")
 
 
-def rows_linear(x: torch.Tensor, w: torch.Tensor, out_dtype=None) -> torch.Tensor:
-    """x [M, K] @ w [N, K]^T for a handful of rows: the cost is one pass over w, spread over N / 16 CTAs."""
-    out = torch.empty(x.shape[0], w.shape[0], dtype=out_dtype or x.dtype, device=x.device)
+def rows_linear(x: torch.Tensor, w: torch.Tensor, out_dtype=None, act: int = ACT_NONE, cap: float = 0.0,
+                out: torch.Tensor | None = None) -> torch.Tensor:
+    """act(x [M, K] @ w [N, K]^T) for a handful of rows: the cost is one pass over w, spread over N / 16 CTAs."""
+    if out is None:
+        out = torch.empty(x.shape[0], w.shape[0], dtype=out_dtype or x.dtype, device=x.device)
     _launch(x, w, out, x.stride(0), w.stride(0), out.stride(0), 0, 0, 0, None, None, None, 1, 1, x.shape[0], w.shape[0],
-            w.shape[1], ACT_NONE)
+            w.shape[1], act, cap=cap)
     return out
 
 

@@ -118,3 +118,70 @@ def final(x, mixer, experts, hist, dwa, n: int, gain, eps: float, out_rows, act_
     if out_rows.numel():
         _boundary_raw(x, mixer, experts, hist, dwa, n, None, gain, eps, None, h, None, None, None, out_rows)
     return h
+
+
+# ---------------------------------------------------------------------------------------------- output-normed boundaries
+def offset_rmsnorm(x: torch.Tensor, w: torch.Tensor, eps: float) -> torch.Tensor:
+    """x / rms(x) * (1 + w)."""
+    return x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) * (1 + w)
+
+
+def _mixes(x: torch.Tensor, mu: torch.Tensor, rows: StreamRows, state: torch.Tensor) -> torch.Tensor:
+    W = x.shape[1]
+    prev = torch.cat([torch.zeros_like(x[:1]), x[:-1]])
+    p, n = rows.prev.long(), rows.next.long()
+    prev = torch.where((p >= 0)[:, None], state[p.clamp(min=0), :W], prev)
+    prev = torch.where((p == ROW_ZERO)[:, None], torch.zeros_like(prev), prev)
+    state[n[n >= 0], :W] = x[n >= 0]
+    return x[:, None] + (prev - x)[:, None] * mu
+
+
+def _postnorm_raw(tok, table, scale, x, y, w, eps, x_out, h, mu, rows, state):
+    T, W = x_out.shape
+    n_mix = 0 if mu is None else mu.shape[0]
+    rc = _lib.load("stream").ts_stream_postnorm(
+        _lib.ptr(tok), _lib.ptr(table), 0 if table is None else table.shape[0], _f(scale), _lib.ptr(x), _lib.ptr(y),
+        _ll(0 if y is None else y.stride(0)), _lib.ptr(w), _f(eps), _lib.ptr(x_out), _lib.ptr(h), _lib.ptr(mu), n_mix,
+        _lib.ptr(rows.prev if n_mix else None), _lib.ptr(rows.next if n_mix else None), _lib.ptr(state if n_mix else None),
+        _ll(state.stride(0) if n_mix else 0), T, W, _fp32(h), _lib.stream_ptr())
+    _lib.check(rc, "ts_stream_postnorm")
+
+
+def _postnorm_outputs(T: int, W: int, mu, dtype, device):
+    shape = (T, W) if mu is None else (T, mu.shape[0], W)
+    return torch.empty(T, W, dtype=torch.float32, device=device), torch.empty(shape, dtype=dtype, device=device)
+
+
+def scaled_embed(tok, table, scale: float, mu, rows: StreamRows, state):
+    """x = table[tok] * scale (fp32).  Returns (x, h): h is x in the table's dtype [T, W], or with `mu` [n, W] the token-shift
+    mixes x + (x of the token before - x) * mu_s [T, n, W]; `state` [rows, >= W] keeps a sequence's last x."""
+    T, W = tok.shape[0], table.shape[1]
+    if not tok.is_cuda:
+        x = table[tok.long()].float() * scale
+        return x, (x if mu is None else _mixes(x, mu, rows, state)).to(table.dtype)
+    x, h = _postnorm_outputs(T, W, mu, table.dtype, tok.device)
+    _postnorm_raw(tok, table, scale, None, None, None, 0.0, x, h, mu, rows, state)
+    return x, h
+
+
+def postnorm(x, y, w, eps: float, mu, rows: StreamRows, state, act_dtype):
+    """x' = x + y / rms(y) * (1 + w) with y [T, W] the sublayer's output; returns (x', h) as `scaled_embed` does."""
+    if not x.is_cuda:
+        x = x + offset_rmsnorm(y.float(), w, eps)
+        return x, (x if mu is None else _mixes(x, mu, rows, state)).to(act_dtype)
+    x_out, h = _postnorm_outputs(*x.shape, mu, act_dtype, x.device)
+    _postnorm_raw(None, None, 0.0, x, y, w, eps, x_out, h, mu, rows, state)
+    return x_out, h
+
+
+def postnorm_final(x, y, w, final_w, eps: float, out_rows, act_dtype) -> torch.Tensor:
+    """Final norm (weight around zero) of x + y / rms(y) * (1 + w) for the rows `out_rows` (int32)."""
+    if not x.is_cuda:
+        r = out_rows.long()
+        return offset_rmsnorm(x[r] + offset_rmsnorm(y[r].float(), w, eps), final_w, eps).to(act_dtype)
+    h = torch.empty(out_rows.numel(), x.shape[1], dtype=act_dtype, device=x.device)
+    rc = _lib.load("stream").ts_stream_postnorm_final(
+        _lib.ptr(x), _lib.ptr(y), _ll(y.stride(0)), _lib.ptr(w), _lib.ptr(final_w), _f(eps), _lib.ptr(h), _lib.ptr(out_rows),
+        out_rows.numel(), x.shape[1], _fp32(h), _lib.stream_ptr())
+    _lib.check(rc, "ts_stream_postnorm_final")
+    return h

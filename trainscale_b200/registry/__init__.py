@@ -411,6 +411,9 @@ register_models_from_meta([
               notes="shared expert + per-layer dense/sparse mix not covered"),
     ModelInfo("mezilix", "trainscale", ("4B",), "MezilixForCausalLM", attention="latent", mlp="moe (squared ReLU)",
               norm="scalar rmsnorm", notes="serving only: models/mezilix.py; windowed latent cache, state per sequence"),
+    ModelInfo("vibepel", "trainscale", ("2B",), "VibepelForCausalLM", attention="sliding window + gated delta rule, wkv",
+              mlp="dense (squared ReLU)", norm="output rmsnorm (offset weight)",
+              notes="serving only: models/vibepel.py; windowed cache and matrix state per sequence"),
     ModelInfo("llava", "llava-hf", ("7B", "13B"), "LlavaForConditionalGeneration", supported=False, notes="vision tower not covered"),
 ])
 
