@@ -291,11 +291,12 @@ def run_serving(args) -> None:
     """One JSON line per size; device-timed, L2 flushed between steps, random weights and tokens."""
     from trainscale_b200.inference import bench_serving
     sampler = ClockSampler(0)
-    for size in args.serve or list(bench_serving.SIZES):
+    for size in args.serve or list(bench_serving.DESIGNS[args.serve_model].sizes):
         sampler.samples.clear()
         sampler.start()
-        res = bench_serving.run([size], ROOT / "MEASURED_PEAKS.json", max(args.steps, 5))[size]
-        print(json.dumps({"size": size, "dtype": "bf16", "data": "random weights and tokens", **res,
+        res = bench_serving.run([size], ROOT / "MEASURED_PEAKS.json", max(args.steps, 5),
+                                args.serve_model)[size]
+        print(json.dumps({"design": args.serve_model, "size": size, "dtype": "bf16", "data": "random weights and tokens", **res,
                           "clocks": sampler.stop()}), flush=True)
 
 
@@ -314,8 +315,9 @@ def main():
     ap.add_argument("--no-secondary", action="store_true", help="skip the measurement of the other sharding mode")
     ap.add_argument("--secondary-timeout", type=float, default=300.0)
     ap.add_argument("--serve", nargs="*", default=None, metavar="SIZE",
-                    help="instead: prefill / decode throughput of the Mezilix decoder beside the closest model at these "
+                    help="instead: prefill / decode throughput of a served design beside the closest model at these "
                          "sizes (default all), with per-op roofline fractions; one GPU")
+    ap.add_argument("--serve-model", default="mezilix", choices=["mezilix", "vibepel"], help="design that --serve measures")
     args = ap.parse_args()
     if args.serve is not None:
         return run_serving(args)

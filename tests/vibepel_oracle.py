@@ -188,3 +188,84 @@ def greedy(w, cfg, tokens, n):
     for _ in range(n):
         ids.append(int(logits(w, cfg, ids)[-1].argmax()))
     return ids[len(tokens):]
+
+
+# ---------------------------------------------------------------------------------------------- test models
+def at(v, i):
+    """Value of layer i: lists hold one value per layer (repeated)."""
+    return v[i % len(v)] if isinstance(v, (list, tuple)) else v
+
+
+SCALING = {"factor": 3.0, "low": 1.0, "high": 3.5, "original": 90}
+
+
+def make_config(width=64, vocab=300, types=("parallel", "wkv", "parallel"), heads=4, kv_heads=2, dim=16, vdim=24, window=7, rot=8,
+                base=500.0, scaling=SCALING, scale=None, dheads=4, dkv=2, ddim=16, dvdim=24, taps=3, left_scale=0.8,
+                right_scale=1.3, wheads=3, wdim=16, ff=80, embed_scale=2.5, softcap=20.0, eps=1e-5, decay_rank=12, mlp_every=1):
+    """A configuration dictionary as a checkpoint's config.json holds it.  Sizes may be lists (one value per layer);
+    `mlp_every` > 1 leaves layers without a feed-forward in between."""
+    ls = []
+    for i, kind in enumerate(types):
+        if kind == "wkv":
+            mixer = {"heads": at(wheads, i), "dim": at(wdim, i), "decay_rank": at(decay_rank, i)}
+        else:
+            d, sc = at(dim, i), at(scaling, i)
+            r = {"base": at(base, i), "dims": at(rot, i)}
+            if sc:
+                r["scaling"] = dict(sc)
+            mixer = {"left": {"heads": at(heads, i), "kv_heads": at(kv_heads, i), "dim": d, "vdim": at(vdim, i),
+                              "mask": {"size": at(window, i)}, "rot": r,
+                              "scale": at(scale, i) if scale is not None else d ** -0.5},
+                     "right": {"heads": at(dheads, i), "kv_heads": at(dkv, i), "dim": at(ddim, i), "vdim": at(dvdim, i),
+                               "conv": at(taps, i)},
+                     "left_scale": at(left_scale, i), "right_scale": at(right_scale, i)}
+        ls.append({"type": kind, "mixer": mixer, "mlp": {"kind": "dense", "ff": at(ff, i)} if i % mlp_every == 0 else None})
+    return {"architecture": "Vibepel", "vocab": vocab, "width": width, "norm": {"eps": eps}, "embedding": {"scale": embed_scale},
+            "logit_softcap": softcap, "layers": ls}
+
+
+def make_weights(cfg, seed=0, sharp=1.0, slow=False):
+    """Random weights (bf16-representable float32).  `sharp` scales the norm weights of queries and keys, so that a wrong key
+    changes the outcome instead of drowning in an even average; `slow` lets recurrent states remember for long."""
+    g = torch.Generator().manual_seed(seed)
+    W = cfg["width"]
+
+    def lin(o, i, s=1.0):
+        return torch.randn(o, i, generator=g) * (s / math.sqrt(i))
+
+    def near(n, c, s=0.2):
+        return c + s * torch.randn(n, generator=g)
+
+    w = {"embed": torch.randn(cfg["vocab"], W, generator=g) / math.sqrt(W) * 2}
+    for i, layer in enumerate(cfg["layers"]):
+        m, p = layer["mixer"], f"l{i}.mix."
+        w[f"l{i}.norm1"] = near(W, 0.0)
+        if layer["type"] == "wkv":
+            n = m["heads"] * m["dim"]
+            for s in "rkvgw":
+                w[p + "mu." + s] = torch.rand(W, generator=g)
+            for s in "rkvg":
+                w[p + s] = lin(n, W)
+            w[p + "w1"], w[p + "w2"] = lin(m["decay_rank"], W), lin(n, m["decay_rank"], 2.0)
+            w[p + "w0"] = near(n, -5.0 if slow else -1.5, 1.0)
+            w[p + "u"], w[p + "norm"], w[p + "o"] = near((m["heads"], m["dim"]), 0.5, 0.5), near(n, 1.0), lin(W, n)
+        else:
+            a, b = m["left"], m["right"]
+            H, G, D, V = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+            w[p + "left.q"], w[p + "left.k"], w[p + "left.v"] = lin(H * D, W), lin(G * D, W), lin(G * V, W)
+            w[p + "left.q.norm"], w[p + "left.k.norm"] = near(D, sharp), near(D, sharp)
+            w[p + "left.o"] = lin(W, H * V)
+            H, G, D, V = b["heads"], b["kv_heads"], b["dim"], b["vdim"]
+            for s, n in (("q", G * D), ("k", G * D), ("v", H * V)):
+                w[p + "right." + s] = lin(n, W)
+                w[p + f"right.{s}.conv"] = torch.randn(n, b["conv"], generator=g) * 0.7
+            w[p + "right.b"], w[p + "right.a"], w[p + "right.g"] = lin(H, W), lin(H, W), lin(H * V, W)
+            w[p + "right.A_log"] = near(H, 0.0, 0.5)
+            w[p + "right.dt_bias"] = near(H, -5.0 if slow else -1.0, 0.5)
+            w[p + "right.norm"], w[p + "right.o"] = near(V, 1.0), lin(W, H * V)
+        if layer["mlp"] is not None:
+            ff = layer["mlp"]["ff"]
+            w[f"l{i}.norm2"] = near(W, 0.0)
+            w[f"l{i}.mlp.up"], w[f"l{i}.mlp.down"] = lin(ff, W), lin(W, ff)
+    w["final.norm"] = near(W, 0.5)
+    return {k: v.to(torch.bfloat16).float() for k, v in w.items()}

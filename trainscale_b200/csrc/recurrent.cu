@@ -642,6 +642,396 @@ __global__ void __launch_bounds__(SC_WARPS * 32) wkv_scan_kernel(WkvParams p) {
 }
 
 // ---------------------------------------------------------------------------------------------------------
+// scan of portions in bf16 models: blocks of eight tokens on the tensor cores, operands split into two TF32 parts (three
+// products), which keeps fp32 accuracy
+//
+// Within a block (states S0 -> S8, gamma_i the decay from the block's start to token i, inclusive):
+//   delta rule   U = T (V - gamma S0^T K),  T = (I + L)^-1 diag(beta),  L_ij = beta_i gamma_i / gamma_j (k_i . k_j)  (j < i)
+//                O = gamma S0^T Q + A U,    A_ij = gamma_i / gamma_j (q_i . k_j)                               (j <= i)
+//                S8 = gamma_8 S0 + K^T diag(gamma_8 / gamma_j) U
+//   WKV          O = S0^T R~ + A V,         R~_i = r_i gamma_(i-1),  A_ij = sum_d r_id k_jd gamma_(i-1)d / gamma_jd  (j < i)
+//                S8 = diag(gamma_8) S0 + K~^T V,  K~_j = k_j gamma_8 / gamma_j;  A_ii = sum_d r_id u_d k_id
+// T, A and (WKV) R~, K~ depend on the inputs alone and come from a launch over all blocks at once.  Every decay above is a
+// product of factors <= 1 formed directly, never a quotient.
+//
+// A warp owns 16 value columns x 8 NT key rows of S^T as MMA accumulators.  The accumulator layout (column g, rows 2t and
+// 2t + 1) IS the layout of an A operand if the reduction index is renumbered (t -> 2t, t + 4 -> 2t + 1), the same way for
+// the B operand; so S, the products with it and U go from one MMA to the next in registers, without a shuffle.
+// WR warps share the key rows of 16 columns and add their partial products through shared memory.
+// ---------------------------------------------------------------------------------------------------------
+constexpr int BS_BLOCK = 8;                // tokens of a block
+constexpr int BS_TILE = 32;                // tokens staged at a time
+constexpr int BS_COEF = 144;               // delta rule, per block and head: T [8][8], A [8][8], gamma [8], gamma_8 / gamma_j [8]
+constexpr int BS_COEF_WKV = 64;            // WKV: A [8][8] (the decay of the key rows is kept beside it)
+
+struct BlockScanParams {
+  const float* q;              // first row, head 0; row stride below
+  const float* k;
+  const void* v;
+  long long qk_ld, v_ld;
+  int rep;                     // heads per query / key head
+  const float* coef;           // [blocks][H][BS_COEF or BS_COEF_WKV]
+  const float* row_decay;      // WKV: [blocks][H][D]
+  float* state;
+  long long state_ld;
+  int s_off;
+  const int* row_prev;
+  const int* row_next;
+  const int* cu;
+  float* o;                    // [rows][H V]
+  int H, D, V;
+};
+
+// block 0 of portion z; the portions' ranges do not overlap
+__device__ __forceinline__ long long first_block(const int* cu, int z) { return cu[z] / BS_BLOCK + z; }
+
+__device__ __forceinline__ void split_tf32(float x, uint32_t& hi, uint32_t& lo) {
+  asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(hi) : "f"(x));
+  lo = __float_as_uint(x - __uint_as_float(hi));
+}
+__device__ __forceinline__ void mma_tf32(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// A operand of an accumulator tile
+__device__ __forceinline__ void split_tile(const float (&c)[4], uint32_t (&hi)[4], uint32_t (&lo)[4]) {
+  split_tf32(c[0], hi[0], lo[0]);
+  split_tf32(c[2], hi[1], lo[1]);
+  split_tf32(c[1], hi[2], lo[2]);
+  split_tf32(c[3], hi[3], lo[3]);
+}
+// c += A b, the small products into `d`
+__device__ __forceinline__ void mma_split(float (&c)[4], float (&d)[4], const uint32_t (&hi)[4], const uint32_t (&lo)[4], float b0,
+                                          float b1) {
+  uint32_t h0, l0, h1, l1;
+  split_tf32(b0, h0, l0);
+  split_tf32(b1, h1, l1);
+  mma_tf32(c, hi, h0, h1);
+  mma_tf32(d, hi, l0, l1);
+  mma_tf32(d, lo, h0, h1);
+}
+
+template <bool DELTA, int NT, int WR, typename TV> struct BlockScan {
+  static constexpr int WC = 4 / WR;                    // column groups of a CTA
+  static constexpr int NC = 16 * WC;
+  static constexpr int DP = 8 * NT * WR;               // key rows, padded
+  static constexpr int KS = DP + 4;
+  static constexpr int VS = NC + 8;
+  static constexpr int CO = DELTA ? BS_COEF : BS_COEF_WKV + DP;
+  static constexpr int QK = BS_TILE * 2 * KS * 4, VB = BS_TILE * VS * static_cast<int>(sizeof(TV));     // bytes
+  static constexpr int STAGE = QK + VB + BS_TILE / BS_BLOCK * CO * 4;
+  static constexpr int EX = WR > 1 ? 2 * 4 * 32 * 8 * 4 : 0;      // two blocks' partial products of the four warps
+  static constexpr size_t SMEM = 2 * STAGE + EX;
+};
+
+// grid (column tiles, H, portions)
+template <bool DELTA, int NT, int WR, typename TV>
+__global__ void __launch_bounds__(128, 2) block_scan_kernel(BlockScanParams p) {
+  using Z = BlockScan<DELTA, NT, WR, TV>;
+  extern __shared__ __align__(16) uint8_t smb[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
+  const int wr = warp % WR, wc = warp / WR;
+  const int h = blockIdx.y, g = h / p.rep, col_cta = blockIdx.x * Z::NC;
+  const int row0 = p.cu[blockIdx.z], n = p.cu[blockIdx.z + 1] - row0;
+  if (n <= 0) return;
+  const long long block0 = first_block(p.cu, blockIdx.z);
+  const int r_first = wr * NT * 8;                       // this warp's key rows
+  const int c0 = col_cta + wc * 16 + gid;                // and value columns c0, c0 + 8
+  const TV* vsrc = reinterpret_cast<const TV*>(p.v);
+
+  auto stage_tile = [&](int s, int t) {
+    float* qk = reinterpret_cast<float*>(smb + s * Z::STAGE);
+    TV* vt = reinterpret_cast<TV*>(smb + s * Z::STAGE + Z::QK);
+    float* co = reinterpret_cast<float*>(smb + s * Z::STAGE + Z::QK + Z::VB);
+    constexpr int U = Z::DP / 4;
+    for (int i = threadIdx.x; i < BS_TILE * 2 * U; i += 128) {
+      const int tk = i / (2 * U), r = i - tk * 2 * U, w = r / U, c = (r - w * U) * 4;
+      const bool ok = t + tk < n && c < p.D;
+      const float* src = (w ? p.k : p.q) + (row0 + t + tk) * p.qk_ld + g * p.D + c;
+      cp_async16(qk + (tk * 2 + w) * Z::KS + c, ok ? src : p.q, ok);
+    }
+    constexpr int E = 16 / sizeof(TV);
+    for (int i = threadIdx.x; i < BS_TILE * (Z::NC / E); i += 128) {
+      const int tk = i / (Z::NC / E), c = (i - tk * (Z::NC / E)) * E;
+      const bool ok = t + tk < n && col_cta + c < p.V;
+      cp_async16(vt + tk * Z::VS + c, ok ? vsrc + (row0 + t + tk) * p.v_ld + h * p.V + col_cta + c : vsrc, ok);
+    }
+    constexpr int CU = Z::CO / 4;
+    for (int i = threadIdx.x; i < BS_TILE / BS_BLOCK * CU; i += 128) {
+      const int b = i / CU, c = (i - b * CU) * 4;
+      const bool in = t + b * BS_BLOCK < n;
+      const long long at = (block0 + t / BS_BLOCK + b) * p.H + h;
+      if (DELTA) {
+        cp_async16(co + b * Z::CO + c, in ? p.coef + at * BS_COEF + c : p.coef, in);
+      } else {
+        const bool mat = c < BS_COEF_WKV, ok = in && (mat || c - BS_COEF_WKV < p.D);
+        cp_async16(co + b * Z::CO + c,
+                   !ok ? p.coef : (mat ? p.coef + at * BS_COEF_WKV + c : p.row_decay + at * p.D + c - BS_COEF_WKV), ok);
+      }
+    }
+    cp_commit();
+  };
+
+  float S[NT][4];
+  const int prev = p.row_prev[row0];
+  const float* s_in = p.state + (prev >= 0 ? prev * p.state_ld : 0) + p.s_off + static_cast<long long>(h) * p.D * p.V;
+#pragma unroll
+  for (int x = 0; x < NT; ++x)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int r = r_first + x * 8 + tig * 2 + (e & 1), c = c0 + (e >> 1) * 8;
+      S[x][e] = prev >= 0 && r < p.D && c < p.V ? s_in[static_cast<long long>(r) * p.V + c] : 0.f;
+    }
+
+  stage_tile(0, 0);
+  int s = 0, parity = 0;
+  for (int t = 0; t < n; t += BS_TILE, s ^= 1) {
+    cp_wait<0>();
+    __syncthreads();                                     // the tile is here; nobody reads the other stage any more
+    if (t + BS_TILE < n) stage_tile(s ^ 1, t + BS_TILE);
+    const float* qk = reinterpret_cast<const float*>(smb + s * Z::STAGE);
+    const TV* vt = reinterpret_cast<const TV*>(smb + s * Z::STAGE + Z::QK);
+    const float* cof = reinterpret_cast<const float*>(smb + s * Z::STAGE + Z::QK + Z::VB);
+    const int blocks = (min(n - t, BS_TILE) + BS_BLOCK - 1) / BS_BLOCK;
+    for (int b = 0; b < blocks; ++b) {
+      const float* tok = qk + b * BS_BLOCK * 2 * Z::KS + r_first;            // [token][q, k][row]
+      const float* co = cof + b * Z::CO;
+      // products with the state before the block: column g (g + 8), tokens 2t, 2t + 1
+      float xk[4] = {0.f, 0.f, 0.f, 0.f}, xq[4] = {0.f, 0.f, 0.f, 0.f};
+      {
+        float yk[4] = {0.f, 0.f, 0.f, 0.f}, yq[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int x = 0; x < NT; ++x) {
+          uint32_t hi[4], lo[4];
+          split_tile(S[x], hi, lo);
+          const float* src = tok + gid * 2 * Z::KS + x * 8 + tig * 2;
+          if (DELTA) {
+            const float2 kv = *reinterpret_cast<const float2*>(src + Z::KS);
+            mma_split(xk, yk, hi, lo, kv.x, kv.y);
+          }
+          const float2 qv = *reinterpret_cast<const float2*>(src);
+          mma_split(xq, yq, hi, lo, qv.x, qv.y);
+        }
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          xk[e] += yk[e];
+          xq[e] += yq[e];
+        }
+      }
+      if (WR > 1) {                                      // sum over the warps that share the columns, in a fixed order
+        float4* ex = reinterpret_cast<float4*>(smb + 2 * Z::STAGE) + parity * 4 * 64;
+        if (DELTA) ex[warp * 64 + lane] = make_float4(xk[0], xk[1], xk[2], xk[3]);
+        ex[warp * 64 + 32 + lane] = make_float4(xq[0], xq[1], xq[2], xq[3]);
+        if (wc == 0) asm volatile("bar.sync 1, %0;" ::"n"(WR * 32) : "memory");
+        else asm volatile("bar.sync 2, %0;" ::"n"(WR * 32) : "memory");
+#pragma unroll
+        for (int w = 0; w < WR; ++w) {
+          const float4 a = ex[(wc * WR + w) * 64 + 32 + lane];
+          xq[0] = w ? xq[0] + a.x : a.x; xq[1] = w ? xq[1] + a.y : a.y;
+          xq[2] = w ? xq[2] + a.z : a.z; xq[3] = w ? xq[3] + a.w : a.w;
+          if (DELTA) {
+            const float4 k4 = ex[(wc * WR + w) * 64 + lane];
+            xk[0] = w ? xk[0] + k4.x : k4.x; xk[1] = w ? xk[1] + k4.y : k4.y;
+            xk[2] = w ? xk[2] + k4.z : k4.z; xk[3] = w ? xk[3] + k4.w : k4.w;
+          }
+        }
+        parity ^= 1;
+      }
+      float u[4];                                        // v, then U
+      {
+        const TV* vv = vt + (b * BS_BLOCK + tig * 2) * Z::VS + wc * 16 + gid;
+        u[0] = to_f32(vv[0]);
+        u[1] = to_f32(vv[Z::VS]);
+        u[2] = to_f32(vv[8]);
+        u[3] = to_f32(vv[Z::VS + 8]);
+      }
+      uint32_t uh[4], ul[4];
+      const float* A = co + (DELTA ? 64 : 0);
+      if (DELTA) {
+        const float2 gm = *reinterpret_cast<const float2*>(co + 128 + tig * 2);
+        u[0] -= gm.x * xk[0]; u[1] -= gm.y * xk[1]; u[2] -= gm.x * xk[2]; u[3] -= gm.y * xk[3];
+        xq[0] *= gm.x; xq[1] *= gm.y; xq[2] *= gm.x; xq[3] *= gm.y;
+        split_tile(u, uh, ul);
+        const float2 tv = *reinterpret_cast<const float2*>(co + gid * 8 + tig * 2);
+        float c[4] = {0.f, 0.f, 0.f, 0.f}, d[4] = {0.f, 0.f, 0.f, 0.f};
+        mma_split(c, d, uh, ul, tv.x, tv.y);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) u[e] = c[e] + d[e];
+      }
+      split_tile(u, uh, ul);
+      if (wr == 0) {
+        const float2 av = *reinterpret_cast<const float2*>(A + gid * 8 + tig * 2);
+        float d[4] = {0.f, 0.f, 0.f, 0.f};
+        mma_split(xq, d, uh, ul, av.x, av.y);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int tt = t + b * BS_BLOCK + tig * 2 + (e & 1), c = c0 + (e >> 1) * 8;
+          if (tt < n && c < p.V) p.o[static_cast<long long>(row0 + tt) * p.H * p.V + h * p.V + c] = xq[e] + d[e];
+        }
+      }
+      if (DELTA) {
+        const float2 rt = *reinterpret_cast<const float2*>(co + 136 + tig * 2);
+        u[0] *= rt.x; u[1] *= rt.y; u[2] *= rt.x; u[3] *= rt.y;
+        split_tile(u, uh, ul);
+      }
+      const float* kt = tok + Z::KS;
+#pragma unroll
+      for (int x = 0; x < NT; ++x) {
+        if (DELTA) {
+          const float g8 = co[128 + 7];
+#pragma unroll
+          for (int e = 0; e < 4; ++e) S[x][e] *= g8;
+        } else {
+          const float2 pd = *reinterpret_cast<const float2*>(co + BS_COEF_WKV + r_first + x * 8 + tig * 2);
+          S[x][0] *= pd.x; S[x][1] *= pd.y; S[x][2] *= pd.x; S[x][3] *= pd.y;
+        }
+        const float b0 = kt[tig * 4 * Z::KS + x * 8 + gid], b1 = kt[(tig * 4 + 2) * Z::KS + x * 8 + gid];
+        mma_split(S[x], S[x], uh, ul, b0, b1);
+      }
+    }
+  }
+  const int next = p.row_next[row0 + n - 1];
+  if (next >= 0) {
+    float* s_out = p.state + next * p.state_ld + p.s_off + static_cast<long long>(h) * p.D * p.V;
+#pragma unroll
+    for (int x = 0; x < NT; ++x)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int r = r_first + x * 8 + tig * 2 + (e & 1), c = c0 + (e >> 1) * 8;
+        if (r < p.D && c < p.V) s_out[static_cast<long long>(r) * p.V + c] = S[x][e];
+      }
+  }
+}
+
+// T, A, gamma of every block of the delta rule.  grid (blocks of the longest portion, G, portions), 128 threads.
+__global__ void __launch_bounds__(128) delta_blocks_kernel(const float* __restrict__ qkv, const float* __restrict__ gates,
+                                                           const int* __restrict__ cu, float* __restrict__ coef, int H, int G,
+                                                           int D, int V) {
+  extern __shared__ __align__(16) float sm[];            // q, k of the block [8][2][D + 4]
+  __shared__ float dots[2][8][8], lg[8], bt[8], Lm[8][8];
+  const int z = blockIdx.z, g = blockIdx.y, rep = H / G, C = 2 * G * D + H * V, KS = D + 4, tid = threadIdx.x;
+  const int row0 = cu[z] + blockIdx.x * BS_BLOCK, n = min(BS_BLOCK, cu[z + 1] - row0);
+  if (n <= 0) return;
+  for (int i = tid; i < BS_BLOCK * 2 * (D / 4); i += 128) {
+    const int tk = i / (2 * (D / 4)), r = i - tk * 2 * (D / 4), w = r / (D / 4), c = (r - w * (D / 4)) * 4;
+    *reinterpret_cast<float4*>(sm + (tk * 2 + w) * KS + c) =
+        tk < n ? *reinterpret_cast<const float4*>(qkv + static_cast<long long>(row0 + tk) * C + (w * G + g) * D + c)
+               : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  __syncthreads();
+  {   // thread (i, j, which): k_i . k_j or q_i . k_j, the lower triangle
+    const int which = tid >> 6, i = (tid >> 3) & 7, j = tid & 7;
+    float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f;
+    if (j <= i) {
+      const float *x = sm + (i * 2 + 1 - which) * KS, *y = sm + (j * 2 + 1) * KS;
+#pragma unroll 8
+      for (int c = 0; c < D; c += 4) {
+        const float4 a = *reinterpret_cast<const float4*>(x + c), b = *reinterpret_cast<const float4*>(y + c);
+        d0 += a.x * b.x; d1 += a.y * b.y; d2 += a.z * b.z; d3 += a.w * b.w;
+      }
+    }
+    dots[which][i][j] = (d0 + d1) + (d2 + d3);
+  }
+  for (int hh = 0; hh < rep; ++hh) {
+    const int h = g * rep + hh;
+    __syncthreads();
+    if (tid < 8) {
+      lg[tid] = tid < n ? gates[static_cast<long long>(row0 + tid) * 2 * H + h] : 0.f;
+      bt[tid] = tid < n ? gates[static_cast<long long>(row0 + tid) * 2 * H + H + h] : 0.f;
+    }
+    __syncthreads();
+    float* out = coef + ((first_block(cu, z) + blockIdx.x) * H + h) * BS_COEF;
+    if (tid < 64) {
+      const int i = tid >> 3, j = tid & 7;
+      float e = 0.f;
+      for (int l = j + 1; l <= i; ++l) e += lg[l];
+      e = expf(e);
+      Lm[i][j] = bt[i] * e * dots[0][i][j];
+      out[64 + tid] = j <= i ? e * dots[1][i][j] : 0.f;
+    } else if (tid < 80) {
+      const int i = tid & 7;
+      float e = 0.f;
+      if (tid < 72) {
+        for (int l = 0; l <= i; ++l) e += lg[l];
+      } else {
+        for (int l = i + 1; l < 8; ++l) e += lg[l];
+      }
+      out[64 + tid] = expf(e);
+    }
+    __syncthreads();
+    if (tid < 8) {                                       // column tid of (I + L)^-1, times beta
+      float col[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        float v = i == tid ? 1.f : 0.f;
+#pragma unroll
+        for (int l = 0; l < 8; ++l)
+          if (l < i) v -= Lm[i][l] * col[l];
+        col[i] = i < tid ? 0.f : v;
+        out[i * 8 + tid] = col[i] * bt[tid];
+      }
+    }
+  }
+}
+
+// R~, K~, A and the decay of every block of the WKV recurrence: one warp per (block, head).  grid (blocks of the longest
+// portion, ceil(H / 4), portions).
+template <typename T>
+__global__ void __launch_bounds__(128) wkv_blocks_kernel(WkvParams p, float* __restrict__ rt, float* __restrict__ kt,
+                                                         float* __restrict__ coef, float* __restrict__ row_decay) {
+  const int z = blockIdx.z, h = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31, D = p.D, HD = p.H * D;
+  const int row0 = p.cu[z] + blockIdx.x * BS_BLOCK, n = min(BS_BLOCK, p.cu[z + 1] - row0);
+  if (n <= 0 || h >= p.H) return;
+  const long long at = (first_block(p.cu, z) + blockIdx.x) * p.H + h;
+  float low[32], diag[8];                                // A below the diagonal (28 values) and on it
+#pragma unroll
+  for (int i = 0; i < 32; ++i) low[i] = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) diag[i] = 0.f;
+  for (int c = lane; c < D; c += 32) {
+    const float w0 = p.w0[h * D + c], uu = p.u[h * D + c];
+    float r[8], k[8], w[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const T* x = reinterpret_cast<const T*>(p.rkvg) + (row0 + i) * p.ld + h * D + c;
+      r[i] = i < n ? to_f32(x[0]) : 0.f;
+      k[i] = i < n ? to_f32(x[HD]) : 0.f;
+      w[i] = i < n ? expf(-expf(p.w_raw[static_cast<long long>(row0 + i) * HD + h * D + c] + w0)) : 1.f;
+    }
+    float head = 1.f, tail = 1.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      if (i < n) rt[static_cast<long long>(row0 + i) * HD + h * D + c] = r[i] * head;
+      head *= w[i];
+      diag[i] += r[i] * uu * k[i];
+    }
+    row_decay[at * D + c] = head;
+#pragma unroll
+    for (int j = 7; j >= 0; --j) {
+      if (j < n) kt[static_cast<long long>(row0 + j) * HD + h * D + c] = k[j] * tail;
+      tail *= w[j];
+      float f = k[j];
+#pragma unroll
+      for (int i = j + 1; i < 8; ++i) {
+        low[i * (i - 1) / 2 + j] += r[i] * f;
+        f *= w[i];
+      }
+    }
+  }
+  reduce_scatter<32>(low, lane);                         // lane l holds entry l
+#pragma unroll
+  for (int i = 0; i < 8; ++i) diag[i] = warp_sum(diag[i]);
+  float* A = coef + at * BS_COEF_WKV;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    if (lane >= i * (i - 1) / 2 && lane < i * (i + 1) / 2) A[i * 8 + lane - i * (i - 1) / 2] = low[0];
+    if (lane >= i && lane < 8) A[i * 8 + lane] = lane == i ? diag[i] : 0.f;
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------
 // norm and gate of a scan's result: out = o / rms_head(o) * w * silu(gate) * scale, one warp per (row, head)
 // ---------------------------------------------------------------------------------------------------------
 template <typename T, int VEC>
@@ -973,6 +1363,25 @@ template <typename T> static int launch_gated_norm(const float* o, const float* 
   return (int)cudaGetLastError();
 }
 
+template <bool DELTA, int NT, int WR, typename TV>
+static int launch_block_scan(const BlockScanParams& p, int portions, cudaStream_t st) {
+  using Z = BlockScan<DELTA, NT, WR, TV>;
+  if (int e = allow_smem(block_scan_kernel<DELTA, NT, WR, TV>, Z::SMEM)) return e;
+  block_scan_kernel<DELTA, NT, WR, TV><<<dim3((p.V + Z::NC - 1) / Z::NC, p.H, portions), 128, Z::SMEM, st>>>(p);
+  return (int)cudaGetLastError();
+}
+
+// key rows of a head split over WR warps; more of them when the grid would leave SMs idle
+template <bool DELTA, typename TV> static int dispatch_block_scan(const BlockScanParams& p, int portions, cudaStream_t st) {
+  const bool few = static_cast<long long>((p.V + 63) / 64) * p.H * portions < sm_count();
+  if (p.D <= 32) return launch_block_scan<DELTA, 4, 1, TV>(p, portions, st);
+  if (p.D <= 64) return few ? launch_block_scan<DELTA, 4, 2, TV>(p, portions, st) : launch_block_scan<DELTA, 8, 1, TV>(p, portions, st);
+  if (p.D <= 128) return launch_block_scan<DELTA, 8, 2, TV>(p, portions, st);
+  return launch_block_scan<DELTA, 8, 4, TV>(p, portions, st);
+}
+
+static bool blocked_ok(int D, int V) { return D % 8 == 0 && V % 8 == 0; }
+
 static bool delta_sizes_ok(int H, int G, int D, int V, int taps) {
   return H > 0 && G > 0 && H % G == 0 && D > 0 && V > 0 && D <= 256 && V <= 256 && taps >= 1 && H <= 65535;
 }
@@ -1010,6 +1419,50 @@ extern "C" int ts_delta_scan(const float* qkv, const float* gates, float* state,
   if (D <= 64) return launch_delta_scan<8>(p, portions, ST(stream));
   if (D <= 128) return launch_delta_scan<16>(p, portions, ST(stream));
   return launch_delta_scan<32>(p, portions, ST(stream));
+}
+
+// 1 when the block scans take these head sizes.
+extern "C" int ts_block_scan_supported(int D, int V) { return blocked_ok(D, V) ? 1 : 0; }
+// Blocks of `rows` rows in `portions` portions (upper bound) and the floats a block and head needs.
+extern "C" int ts_block_scan_blocks(int rows, int portions) { return rows / BS_BLOCK + portions + 1; }
+extern "C" int ts_block_scan_coef(int delta) { return delta ? BS_COEF : BS_COEF_WKV; }
+
+// Portions, step 2 of bf16 models: as ts_delta_scan, on the tensor cores.  coef: [blocks][H][BS_COEF] workspace.
+extern "C" int ts_delta_block_scan(const float* qkv, const float* gates, float* coef, float* state, long long state_ld, int s_off,
+                                   const int* row_prev, const int* row_next, const int* cu, int portions, int max_rows, float* o,
+                                   int H, int G, int D, int V, void* stream) {
+  if (portions <= 0) return 0;
+  if (!delta_sizes_ok(H, G, D, V, 1) || !blocked_ok(D, V) || portions > 65535) return -10;
+  const dim3 grid((max_rows + BS_BLOCK - 1) / BS_BLOCK, G, portions);
+  delta_blocks_kernel<<<grid, 128, BS_BLOCK * 2 * (D + 4) * sizeof(float), ST(stream)>>>(qkv, gates, cu, coef, H, G, D, V);
+  if (int e = (int)cudaGetLastError()) return e;
+  BlockScanParams p = {};
+  p.q = qkv; p.k = qkv + G * D; p.v = qkv + 2 * G * D; p.qk_ld = p.v_ld = 2 * G * D + H * V; p.rep = H / G; p.coef = coef;
+  p.state = state; p.state_ld = state_ld; p.s_off = s_off; p.row_prev = row_prev; p.row_next = row_next; p.cu = cu; p.o = o;
+  p.H = H; p.D = D; p.V = V;
+  return dispatch_block_scan<true, float>(p, portions, ST(stream));
+}
+
+// Portions of the WKV recurrence of bf16 models.  Workspaces: rt, kt [rows][H D], coef [blocks][H][BS_COEF_WKV], row_decay
+// [blocks][H][D].
+extern "C" int ts_wkv_block_scan(const void* rkvg, long long ld, const float* w_raw, const float* w0, const float* u, float* rt,
+                                 float* kt, float* coef, float* row_decay, float* state, long long state_ld, int s_off,
+                                 const int* row_prev, const int* row_next, const int* cu, int portions, int max_rows, float* o,
+                                 int H, int D, void* stream) {
+  if (portions <= 0) return 0;
+  if (!delta_sizes_ok(H, H, D, D, 1) || !blocked_ok(D, D) || portions > 65535 || ld % 8 ||
+      (reinterpret_cast<uintptr_t>(rkvg) & 15u))
+    return -10;
+  WkvParams w = {};
+  w.rkvg = rkvg; w.ld = ld; w.w_raw = w_raw; w.w0 = w0; w.u = u; w.cu = cu; w.H = H; w.D = D;
+  const dim3 grid((max_rows + BS_BLOCK - 1) / BS_BLOCK, (H + 3) / 4, portions);
+  wkv_blocks_kernel<__nv_bfloat16><<<grid, 128, 0, ST(stream)>>>(w, rt, kt, coef, row_decay);
+  if (int e = (int)cudaGetLastError()) return e;
+  BlockScanParams p = {};
+  p.q = rt; p.k = kt; p.v = reinterpret_cast<const __nv_bfloat16*>(rkvg) + 2 * H * D; p.qk_ld = H * D; p.v_ld = ld; p.rep = 1;
+  p.coef = coef; p.row_decay = row_decay; p.state = state; p.state_ld = state_ld; p.s_off = s_off; p.row_prev = row_prev;
+  p.row_next = row_next; p.cu = cu; p.o = o; p.H = H; p.D = D; p.V = D;
+  return dispatch_block_scan<false, __nv_bfloat16>(p, portions, ST(stream));
 }
 
 // Portions, last step (either recurrence): o [rows][H V] fp32; w per channel (w_head = V) or shared by heads (w_head = 0).

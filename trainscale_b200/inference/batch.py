@@ -42,6 +42,10 @@ class Portions:
     def count(self) -> int:
         return len(self.offsets) - 1
 
+    @property
+    def longest(self) -> int:
+        return max(b - a for a, b in zip(self.offsets[:-1], self.offsets[1:]))
+
 
 class HostBatch:
     """Host side of a step: tokens are appended to the cache, index lists are built.  Single-token entries come first

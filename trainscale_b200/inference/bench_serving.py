@@ -1,5 +1,5 @@
 """Prefill and decode throughput of a served design beside the framework's closest existing model at equal size, with the
-device time of every op and its distance from the roofline (`bench.py --serve`).
+device time of every op and its distance from the roofline (`bench.py --serve`, `--serve-model`).
 
 Both models run through `ModelRunner` on the engine's cache with random weights and random tokens.  Step times are CUDA
 events around whole steps; for the per-op table the host first queues a spin kernel, so that a whole step is enqueued
@@ -10,7 +10,9 @@ from __future__ import annotations
 import json
 import math
 import statistics
+from dataclasses import dataclass
 from pathlib import Path
+from typing import Callable
 
 import torch
 
@@ -23,7 +25,15 @@ SIZES = {
     "2k": dict(layers=16, width=2048, heads=16, dim=128, rot=64, vdim=128, rank=512, window=1024, experts=32, top=4, ff=1536),
     "4k": dict(layers=8, width=4096, heads=32, dim=128, rot=64, vdim=128, rank=512, window=4096, experts=64, top=6, ff=1536),
 }
+# every fourth layer mixes with WKV, the others with attention and the delta rule in parallel; the closest model has gated
+# feed-forwards of 2/3 ff and the attention of `heads` / `kv` in every layer
+VIBEPEL_SIZES = {
+    "1k": dict(layers=12, width=1024, heads=8, kv=2, dim=128, window=512, ff=4096, dheads=8, dkv=4, ddim=128, wheads=16, wdim=64),
+    "2k": dict(layers=16, width=2048, heads=16, kv=4, dim=128, window=1024, ff=8192, dheads=16, dkv=8, ddim=128, wheads=32, wdim=64),
+    "4k": dict(layers=8, width=4096, heads=32, kv=8, dim=128, window=4096, ff=16384, dheads=32, dkv=16, ddim=128, wheads=64, wdim=64),
+}
 VOCAB = 32000
+FP32_TFLOPS = 74.4            # nominal: 148 SMs x 128 lanes x 2 x 1.965 GHz
 
 
 def build_mezilix(z: dict):
@@ -41,6 +51,24 @@ def build_closest(z: dict):
                       num_hidden_layers=z["layers"], num_attention_heads=z["heads"], num_key_value_heads=max(1, z["heads"] // 4),
                       head_dim=z["vdim"], num_local_experts=z["experts"], num_experts_per_tok=z["top"],
                       model_type="mixtral", max_position_embeddings=16384)
+    return build_model(cfg, torch.bfloat16, "cuda", seed=0, init_on_device=True)
+
+
+def build_vibepel(z: dict):
+    from ..models.vibepel import build_model, pattern_config
+    return build_model(pattern_config(layers=z["layers"], vocab=VOCAB, width=z["width"], heads=z["heads"], kv_heads=z["kv"],
+                                      dim=z["dim"], window=z["window"], ff=z["ff"], delta_heads=z["dheads"],
+                                      delta_kv_heads=z["dkv"], delta_dim=z["ddim"], delta_vdim=z["ddim"],
+                                      wkv_heads=z["wheads"], wkv_dim=z["wdim"], rot_dims=z["dim"] // 2),
+                       torch.bfloat16, "cuda", seed=0)
+
+
+def build_closest_dense(z: dict):
+    """Llama decoder with dense gated feed-forwards: same width, depth, attention heads and feed-forward weights."""
+    from ..models.llama import LlamaConfig, build_model
+    cfg = LlamaConfig(vocab_size=VOCAB, hidden_size=z["width"], intermediate_size=-(-z["ff"] * 2 // 3 // 64) * 64,
+                      num_hidden_layers=z["layers"], num_attention_heads=z["heads"], num_key_value_heads=z["kv"],
+                      head_dim=z["dim"], max_position_embeddings=16384, tie_word_embeddings=True)
     return build_model(cfg, torch.bfloat16, "cuda", seed=0, init_on_device=True)
 
 
@@ -79,7 +107,8 @@ def _bytes(*ts) -> int:
 
 
 class OpTimer:
-    """Events around every call of the wrapped op functions; `cost(args, kwargs, result) -> (bytes, flops)`."""
+    """Events around every call of the wrapped op functions; `cost(args, kwargs, result) -> (bytes, tensor-core flops)` or
+    `(bytes, tensor-core flops, fp32 flops)`."""
 
     def __init__(self, table: list[tuple]):
         self.table, self.records, self.saved, self.depth = table, [], [], 0
@@ -114,9 +143,10 @@ class OpTimer:
     def summary(self, peaks: dict) -> dict:
         torch.cuda.synchronize()
         acc: dict = {}
-        for name, e0, e1, nbytes, flops in self.records:
+        for name, e0, e1, nbytes, flops, *fp32 in self.records:
             r = acc.setdefault(name, [0, 0.0, 0.0])
-            floor = max(nbytes / (peaks["hbm_gbs"] * 1e9), flops / (peaks["bf16_tflops"] * 1e12)) * 1e3
+            floor = max(nbytes / (peaks["hbm_gbs"] * 1e9), flops / (peaks["bf16_tflops"] * 1e12),
+                        sum(fp32) / (FP32_TFLOPS * 1e12)) * 1e3
             r[0] += 1
             r[1] += e0.elapsed_time(e1)
             r[2] += floor
@@ -183,10 +213,52 @@ def mezilix_table(z: dict, rows: int, keys: float, pairs: float) -> list[tuple]:
     ]
 
 
+def vibepel_table(z: dict, rows: int, keys: float, pairs: float) -> list[tuple]:
+    """The scans' arithmetic is fp32: three products of every state element per token."""
+    from ..ops import gemm, grouped, latent_attention as latent, recurrent, stream, window_attention as window
+    W, H, G, D = z["width"], z["heads"], z["kv"], z["dim"]
+
+    def boundary(a, k, out):
+        if isinstance(out, torch.Tensor):                      # last boundary: only the wanted rows
+            return out.shape[0] * W * (4 + 2 + 2), 0.0
+        return _bytes(*out) + out[0].shape[0] * W * (2 + 4), 0.0
+
+    def state(s, n):                                           # n sequences: S read and written
+        return 2 * n * (s.state_width - s.matrix_offset) * 4
+
+    return [
+        (stream, "scaled_embed", "embedding", boundary),
+        (stream, "postnorm", lambda a, o: "output norm, sum, mixes" if o[1].dim() == 3 else "output norm, sum", boundary),
+        (stream, "postnorm_final", "last norms", boundary),
+        (gemm, "serve_linear", _linear_name("gemm"), _linear_cost),
+        (grouped, "head_linear", lambda a, o: f"gemm 4 x {a[1].shape[1]}x{a[1].shape[2]}",
+         lambda a, k, o: (_bytes(a[0], a[1], o), 2.0 * a[0].shape[0] * a[1].numel())),
+        (window, "prepare", "head norms, rotary, cache write",
+         lambda a, k, o: (a[0].shape[0] * 2 * (2 * (a[1].q_width + a[1].kv_heads * a[1].dim) + a[1].kv_heads * a[1].vdim +
+                                               a[1].kv_width), 0.0)),
+        (latent, "gather_rows", "key gather", lambda a, k, o: (2 * _bytes(o), 0.0)),
+        (window, "attend_rows", "attention (rows)",
+         lambda a, k, o: (keys * a[1].kv_width * 2 + a[0].shape[0] * (a[1].q_width + a[1].out_width) * 2, 4.0 * pairs * H * D)),
+        (window, "attend_portions", "attention (portions)",
+         lambda a, k, o: (a[0].shape[0] * (a[1].q_width + a[1].kv_width + a[1].out_width) * 2, 4.0 * pairs * H * D)),
+        (recurrent, "delta_step", "delta rule step",
+         lambda a, k, o: (a[0].shape[0] * (a[1].proj_width + a[1].out_width) * 2 + state(a[1], a[0].shape[0]), 0.0)),
+        (recurrent, "delta_inputs", "delta rule inputs",
+         lambda a, k, o: (a[0].shape[0] * (a[1].channels + 2 * a[1].heads) * 2 + _bytes(*o), 0.0)),
+        (recurrent, "delta_scan", "delta rule scan",
+         lambda a, k, o: (_bytes(a[0], a[1], o), 0.0, 6.0 * o.numel() * a[2].dim)),
+        (recurrent, "gated_norm", "gated norm", lambda a, k, o: (_bytes(a[0]) + 2 * _bytes(a[4]), 0.0)),
+        (recurrent, "wkv_step", "WKV step",
+         lambda a, k, o: (_bytes(a[0], a[1], a[7]) + state(a[2], a[0].shape[0]), 0.0)),
+        (recurrent, "wkv_scan", "WKV scan",
+         lambda a, k, o: (_bytes(a[0]) * 3 // 4 + _bytes(a[1], o), 0.0, 6.0 * o.numel() * a[2].dim)),
+    ]
+
+
 def closest_table(z: dict, rows: int, keys: float, pairs: float, runner) -> list[tuple]:
     from ..ops import activation, gemm, moe, norm, rope
-    W, H, D = z["width"], z["heads"], z["vdim"]
-    hkv = max(1, H // 4)
+    W, H, D = z["width"], z["heads"], z.get("vdim") or z["dim"]
+    hkv = z.get("kv") or max(1, H // 4)
 
     def grouped_cost(a, k, out):
         E, N, K = a[1].shape
@@ -202,7 +274,7 @@ def closest_table(z: dict, rows: int, keys: float, pairs: float, runner) -> list
         (moe, "make_plan", "routing plan", lambda a, k, o: (_bytes(a[0], o.dest, o.src_of_row), 0.0)),
         (moe, "_permute_raw", "permute", lambda a, k, o: (_bytes(a[0]) + a[1].n * W * 2, 0.0)),
         (moe, "grouped_linear", lambda a, o: f"experts {a[1].shape[1]}x{a[1].shape[2]}", grouped_cost),
-        (activation, "glu", "gated activation", lambda a, k, o: (rows * z["top"] * 3 * o.shape[1] * 2, 0.0)),
+        (activation, "glu", "gated activation", lambda a, k, o: (rows * z.get("top", 1) * 3 * o.shape[1] * 2, 0.0)),
         (moe, "_combine_raw", "combine", lambda a, k, o: (rows * z["top"] * W * 2 + _bytes(o), 0.0)),
     ]
 
@@ -213,18 +285,31 @@ def _visible_pairs(lengths: list[tuple[int, int]], window: int) -> float:
     return float(sum(min(p + 1, window) for start, n in lengths for p in range(start, start + n)))
 
 
-def measure(name: str, z: dict, peaks: dict, prompts: int = 2, prompt_len: int = 4096, batches=(8, 64), context: int = 2048,
+@dataclass(frozen=True)
+class Design:
+    sizes: dict
+    build: Callable
+    closest: Callable
+    table: Callable
+
+
+DESIGNS = {"mezilix": Design(SIZES, build_mezilix, build_closest, mezilix_table),
+           "vibepel": Design(VIBEPEL_SIZES, build_vibepel, build_closest_dense, vibepel_table)}
+
+
+def measure(design: str, name: str, peaks: dict, prompts: int = 2, prompt_len: int = 4096, batches=(8, 64), context: int = 2048,
             iters: int = 5) -> dict:
+    spec = DESIGNS[design]
+    z = spec.sizes[name]
     out: dict = {"sizes": z, "models": {}}
-    for kind, build in (("mezilix", build_mezilix), ("closest", build_closest)):
+    for kind, build in ((design, spec.build), ("closest", spec.closest)):
         model = build(z)
         core = make_core(model, max(prompts * prompt_len, max(batches) * (context + 64)), max(max(batches), prompts))
-        window = z["window"] if kind == "mezilix" else 1 << 30
+        window = z["window"] if kind == design else 1 << 30
         res: dict = {"parameters": sum(p.numel() for p in model.parameters())}
 
         def table(rows, keys, pairs):
-            return mezilix_table(z, rows, keys, pairs) if kind == "mezilix" else \
-                closest_table(z, rows, keys, pairs, core.runner)
+            return spec.table(z, rows, keys, pairs) if kind == design else closest_table(z, rows, keys, pairs, core.runner)
 
         def profile(step, rows, keys, pairs):
             with OpTimer(table(rows, keys, pairs)) as t:
@@ -242,7 +327,7 @@ def measure(name: str, z: dict, peaks: dict, prompts: int = 2, prompt_len: int =
         res["prefill"] = {"tokens": T, "ms": ms, "tokens_per_s": T / ms * 1e3,
                           "ops": profile(step, T, T, _visible_pairs([(0, prompt_len)] * prompts, window))}
         # portions that continue cached prompts
-        if kind == "mezilix":
+        if kind == design:
             for i in range(prompts):
                 core.release(i)
             half = prompt_len // 2
@@ -273,21 +358,20 @@ def measure(name: str, z: dict, peaks: dict, prompts: int = 2, prompt_len: int =
         out["models"][kind] = res
         del core, model, batch, host, step
         torch.cuda.empty_cache()
-    m = out["models"]
-    out["mezilix_over_closest"] = {
-        "prefill": m["mezilix"]["prefill"]["tokens_per_s"] / m["closest"]["prefill"]["tokens_per_s"],
-        **{f"decode_{n}": m["mezilix"]["decode"][n]["tokens_per_s"] / m["closest"]["decode"][n]["tokens_per_s"]
-           for n in m["mezilix"]["decode"]}}
+    ours, closest = out["models"][design], out["models"]["closest"]
+    out[f"{design}_over_closest"] = {
+        "prefill": ours["prefill"]["tokens_per_s"] / closest["prefill"]["tokens_per_s"],
+        **{f"decode_{n}": ours["decode"][n]["tokens_per_s"] / closest["decode"][n]["tokens_per_s"] for n in ours["decode"]}}
     return out
 
 
-def run(sizes: list[str], peaks_file: Path, iters: int = 5) -> dict:
+def run(sizes: list[str], peaks_file: Path, iters: int = 5, design: str = "mezilix") -> dict:
     peaks = {"hbm_gbs": 6538.9, "bf16_tflops": 1608.3}
     try:
         peaks.update(json.loads(peaks_file.read_text()))
     except OSError:
         pass
     from ..ops import _lib
-    out = {n: measure(n, SIZES[n], peaks, iters=iters) for n in sizes}
+    out = {n: measure(design, n, peaks, iters=iters) for n in sizes}
     _lib.raise_on_loaded_device_error()
     return out

@@ -9,6 +9,7 @@ take PyTorch math.
 from __future__ import annotations
 
 import ctypes
+import functools
 from dataclasses import dataclass
 
 import torch
@@ -142,7 +143,7 @@ def delta_rule(proj: torch.Tensor, s: DeltaShape, w: DeltaWeights, eps: float, r
     if n_single < T:
         tail = StreamRows(rows.prev[n_single:], rows.next[n_single:])
         qkv, gates = delta_inputs(proj[n_single:], s, w, tail, row_seq[n_single:], state, n_single, portions)
-        o = delta_scan(qkv, gates, s, tail, state, portions)
+        o = delta_scan(qkv, gates, s, tail, state, portions, proj.dtype == torch.bfloat16)
         gate = proj[n_single:, s.channels:s.channels + s.out_width]
         gated_norm(o, w.norm, 0, gate, out[n_single:], s.heads, s.vdim, eps, out_scale)
 
@@ -171,9 +172,31 @@ def delta_inputs(proj, s: DeltaShape, w: DeltaWeights, rows: StreamRows, row_seq
     return qkv, gates
 
 
-def delta_scan(qkv, gates, s: DeltaShape, rows: StreamRows, state, portions) -> torch.Tensor:
-    """The recurrence over portions: results [T, heads * vdim] fp32; leaves every portion's last state."""
-    o = torch.empty(qkv.shape[0], s.out_width, dtype=torch.float32, device=qkv.device)
+@functools.lru_cache(maxsize=None)
+def _blocked(dim: int, vdim: int) -> bool:
+    return bool(_lib.load("recurrent").ts_block_scan_supported(dim, vdim))
+
+
+def _workspace(T: int, portions, delta: int, *shape, device) -> torch.Tensor:
+    """Uninitialised fp32 [blocks, heads, ...] for the per-block quantities of a block scan."""
+    lib = _lib.load("recurrent")
+    last = shape[1:] or (lib.ts_block_scan_coef(delta),)
+    return torch.empty(lib.ts_block_scan_blocks(T, portions.count), shape[0], *last, dtype=torch.float32, device=device)
+
+
+def delta_scan(qkv, gates, s: DeltaShape, rows: StreamRows, state, portions, blocked: bool = False) -> torch.Tensor:
+    """The recurrence over portions: results [T, heads * vdim] fp32; leaves every portion's last state.  `blocked`: blocks of
+    tokens on the tensor cores with split operands (head sizes that are multiples of 8), else plain fp32 arithmetic."""
+    T = qkv.shape[0]
+    o = torch.empty(T, s.out_width, dtype=torch.float32, device=qkv.device)
+    if blocked and _blocked(s.dim, s.vdim):
+        coef = _workspace(T, portions, 1, s.heads, device=qkv.device)
+        rc = _lib.load("recurrent").ts_delta_block_scan(
+            _lib.ptr(qkv), _lib.ptr(gates), _lib.ptr(coef), _lib.ptr(state),
+            _ll(state.stride(0)), s.matrix_offset, _lib.ptr(rows.prev), _lib.ptr(rows.next), _lib.ptr(portions.cu),
+            portions.count, portions.longest, _lib.ptr(o), s.heads, s.kv_heads, s.dim, s.vdim, _lib.stream_ptr())
+        _lib.check(rc, "ts_delta_block_scan")
+        return o
     rc = _lib.load("recurrent").ts_delta_scan(
         _lib.ptr(qkv), _lib.ptr(gates), _lib.ptr(state), _ll(state.stride(0)), s.matrix_offset, _lib.ptr(rows.prev),
         _lib.ptr(rows.next), _lib.ptr(portions.cu), portions.count, _lib.ptr(o), s.heads, s.kv_heads, s.dim, s.vdim,
@@ -219,7 +242,7 @@ def wkv(rkvg: torch.Tensor, w_raw: torch.Tensor, s: WkvShape, w: WkvWeights, eps
         wkv_step(rkvg[:n_single], w_raw[:n_single], s, w, eps, rows, state, out[:n_single])
     if n_single < T:
         tail = StreamRows(rows.prev[n_single:], rows.next[n_single:])
-        o = wkv_scan(rkvg[n_single:], w_raw[n_single:], s, w, tail, state, portions)
+        o = wkv_scan(rkvg[n_single:], w_raw[n_single:], s, w, tail, state, portions, rkvg.dtype == torch.bfloat16)
         gated_norm(o, w.norm, s.dim, rkvg[n_single:, 3], out[n_single:], s.heads, s.dim, eps)
 
 
@@ -231,8 +254,20 @@ def wkv_step(rkvg, w_raw, s: WkvShape, w: WkvWeights, eps: float, rows: StreamRo
     _lib.check(rc, "ts_wkv_step")
 
 
-def wkv_scan(rkvg, w_raw, s: WkvShape, w: WkvWeights, rows: StreamRows, state, portions) -> torch.Tensor:
-    o = torch.empty(rkvg.shape[0], s.inner, dtype=torch.float32, device=rkvg.device)
+def wkv_scan(rkvg, w_raw, s: WkvShape, w: WkvWeights, rows: StreamRows, state, portions, blocked: bool = False) -> torch.Tensor:
+    """As `delta_scan`; `blocked` takes bf16 projections."""
+    T, dev = rkvg.shape[0], rkvg.device
+    o = torch.empty(T, s.inner, dtype=torch.float32, device=dev)
+    if blocked and _blocked(s.dim, s.dim):
+        rt, kt = (torch.empty(T, s.inner, dtype=torch.float32, device=dev) for _ in range(2))
+        coef, decay = _workspace(T, portions, 0, s.heads, device=dev), _workspace(T, portions, 0, s.heads, s.dim, device=dev)
+        rc = _lib.load("recurrent").ts_wkv_block_scan(
+            _lib.ptr(rkvg), _ll(rkvg.stride(0)), _lib.ptr(w_raw), _lib.ptr(w.w0), _lib.ptr(w.u), _lib.ptr(rt), _lib.ptr(kt),
+            _lib.ptr(coef), _lib.ptr(decay), _lib.ptr(state), _ll(state.stride(0)), s.matrix_offset, _lib.ptr(rows.prev),
+            _lib.ptr(rows.next), _lib.ptr(portions.cu), portions.count, portions.longest, _lib.ptr(o), s.heads, s.dim,
+            _lib.stream_ptr())
+        _lib.check(rc, "ts_wkv_block_scan")
+        return o
     rc = _lib.load("recurrent").ts_wkv_scan(
         _lib.ptr(rkvg), _ll(rkvg.stride(0)), _lib.ptr(w_raw), _lib.ptr(w.w0), _lib.ptr(w.u), _lib.ptr(state),
         _ll(state.stride(0)), s.matrix_offset, _lib.ptr(rows.prev), _lib.ptr(rows.next), _lib.ptr(portions.cu),
