@@ -139,7 +139,7 @@ def test_head_norms_rotary_and_cache_write(dtype, H, G, D, V, rot):
     r = {"dims": rot, "base": 1000.0, "scaling": O.SCALING}
     f = O.frequencies(r).float().cuda()
     cache = torch.full((8, 8, s.row_width), 3.0, dtype=dtype, device="cuda")
-    wa.prepare(proj, s, qn, kn, 1e-5, f, pos, slots, cache)
+    wa.prepare(proj, s, qn, kn, 1e-5, wa.angles(f, pos), slots, cache)
 
     def normed(x, w):
         return O.rotate_half(O.rms(x.double().cpu(), 1e-5) * w.double().cpu(), pos.cpu(), r)
@@ -234,10 +234,6 @@ def _portions(lens):
     return Portions(at, i32(*at))
 
 
-def _row_seq(lens, first=0):
-    return i32(*[first + b for b, n in enumerate(lens) for _ in range(n)])
-
-
 PREV = [3, -1, 7, 5, -1]
 
 
@@ -287,8 +283,7 @@ def test_delta_rule_portions(dtype, H, G, D, V, taps, lens, strong):
     rows.next[:ns] = -1
     out = torch.zeros(T + ns, s.out_width + 8, dtype=dtype, device="cuda")
     before = state.clone()
-    row_seq = torch.cat([i32(*range(ns)), _row_seq(lens, ns)])
-    recurrent.delta_rule(proj[:, :s.proj_width], s, w, eps, rows, row_seq, state, ns, _portions(lens), out[:, :s.out_width], 0.6)
+    recurrent.delta_rule(proj[:, :s.proj_width], s, w, eps, rows, state, ns, _portions(lens), out[:, :s.out_width], 0.6)
     at = ns
     for b, n in enumerate(lens):
         x = proj[at:at + n].double().cpu()
@@ -315,7 +310,7 @@ def test_delta_rule_steps_equal_a_portion(dtype, H, G, D, V, taps):
         rows = StreamRows(prev, i32(10 + ((t + 1) & 1), 12 + ((t + 1) & 1)))
         x = proj[[t, n + t]][:, :s.proj_width].contiguous()
         o = torch.empty(2, s.out_width, dtype=dtype, device="cuda")
-        recurrent.delta_rule(x, s, w, eps, rows, i32(0, 1), state, 2, None, o)
+        recurrent.delta_rule(x, s, w, eps, rows, state, 2, None, o)
         outs[t], outs[n + t] = o[0], o[1]
     first = delta_case(H, G, D, V, taps, 1, dtype, seed=40)[3]
     for b, st in ((0, None), (1, first[4].double().cpu())):
@@ -381,7 +376,7 @@ def test_scans_with_many_and_few_heads(D, H):
     lens = [37, 64]
     s, w, proj, state = delta_case(H, H // 2, D, D, 3, sum(lens), torch.float32, seed=60)
     rows, por = _rows(lens, [3, -1]), _portions(lens)
-    qkv, gates = recurrent.delta_inputs(proj[:, :s.proj_width], s, w, rows, _row_seq(lens), state, 0, por)
+    qkv, gates = recurrent.delta_inputs(proj[:, :s.proj_width], s, w, rows, state, por)
     a, st = state.clone(), state.clone()
     plain = recurrent.delta_scan(qkv, gates, s, rows, a, por)
     blocked = recurrent.delta_scan(qkv, gates, s, rows, st, por, True)

@@ -26,6 +26,10 @@ template <> __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(flo
 __device__ __forceinline__ float to_f32(float v) { return v; }
 __device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
 __device__ __forceinline__ float silu(float x) { return x / (1.f + expf(-x)); }
+// activations of 16-bit models: fp32 arithmetic with the approximate exponential and quotient
+template <typename T> __device__ __forceinline__ float act_silu(float x) {
+  return sizeof(T) == 2 ? __fdividef(x, 1.f + __expf(-x)) : silu(x);
+}
 __device__ __forceinline__ float sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 
@@ -75,8 +79,7 @@ struct DeltaParams {
   const int* row_prev;         // [rows] state row a sequence continues from (>= 0), else zeros / the row before
   const int* row_next;         // [rows] state row to leave, -1: not a last row
   const int* cu;               // portions: [n + 1] first rows
-  const int* row_seq;          // portions: sequence of a row; the first portion is seq0
-  int seq0;
+  int portions, max_rows;      // portions: count, rows of the longest
   float* qkv;                  // portions: [rows][C] convolved inputs
   float* gates;                // portions: [rows][2 H] log g | beta
   float* o;                    // portions: [rows][H V]
@@ -96,14 +99,17 @@ __device__ __forceinline__ float conv_input(const DeltaParams& p, int src, int s
 
 constexpr int DI_TOKENS = 8;
 
-// A warp takes DI_TOKENS rows of one head of q, k or v (or the gates); lanes hold VEC neighbouring channels, NI times.
-// FAST: at most four taps, inputs of the rows before stay in registers.
+// A warp takes DI_TOKENS rows of a portion, one head of q, k or v (or the gates); lanes hold VEC neighbouring channels, NI
+// times.  FAST: at most four taps, inputs of the rows before stay in registers.  grid (runs of the longest portion, units / 4,
+// portions).
 template <typename T, int VEC, int NI, bool FAST>
 __global__ void __launch_bounds__(128) delta_inputs_kernel(DeltaParams p) {
   const int lane = threadIdx.x & 31, units = 2 * p.G + p.H + 1;
   const int unit = blockIdx.y * 4 + (threadIdx.x >> 5);
   if (unit >= units) return;
-  const int t0 = blockIdx.x * DI_TOKENS, t1 = min(p.rows, t0 + DI_TOKENS);
+  const int start = p.cu[blockIdx.z], end = p.cu[blockIdx.z + 1];
+  const int t0 = start + blockIdx.x * DI_TOKENS, t1 = min(end, t0 + DI_TOKENS);
+  if (t0 >= t1) return;
   const int C = 2 * p.G * p.D + p.H * p.V;
   const T* proj = reinterpret_cast<const T*>(p.proj);
   if (unit == units - 1) {
@@ -133,53 +139,54 @@ __global__ void __launch_bounds__(128) delta_inputs_kernel(DeltaParams p) {
         }
       }
   }
-  int start = -1, prev = -1;
-  for (int t = t0; t < t1; ++t) {
-    const int b = p.row_seq[t] - p.seq0;
-    if (start < 0 || p.cu[b] != start) {
-      start = p.cu[b];
-      prev = p.row_prev[start];
-      if (FAST) {
+  float in[DI_TOKENS][NI * VEC];           // the run's own inputs, all loads issued at once
 #pragma unroll
-        for (int i = 0; i < NI * VEC; ++i) {
-          const int c = (i / VEC) * 32 * VEC + lane * VEC + i % VEC;
+  for (int k = 0; k < DI_TOKENS; ++k) {
+    const T* x = proj + min(t0 + k, t1 - 1) * p.ld + c0;
 #pragma unroll
-          for (int j = 0; j < 3; ++j) hist[j][i] = c < n ? conv_input<T>(p, t - 3 + j, start, prev, c0 + c, C) : 0.f;
-        }
+    for (int i = 0; i < NI; ++i) {
+      const int c = min(i * 32 * VEC + lane * VEC, n - VEC);
+      if (VEC == 2 && sizeof(T) == 2) {
+        const float2 f = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(x + c));
+        in[k][i * VEC] = f.x;
+        in[k][i * VEC + VEC - 1] = f.y;
+      } else {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) in[k][i * VEC + e] = to_f32(x[c + e]);
       }
     }
+  }
+  const int prev = p.row_prev[start];
+  if (FAST) {
+#pragma unroll
+    for (int i = 0; i < NI * VEC; ++i) {
+      const int c = (i / VEC) * 32 * VEC + lane * VEC + i % VEC;
+#pragma unroll
+      for (int j = 0; j < 3; ++j) hist[j][i] = c < n ? conv_input<T>(p, t0 - 3 + j, start, prev, c0 + c, C) : 0.f;
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < DI_TOKENS; ++k) {
+    const int t = t0 + k;
+    if (t >= t1) break;
     float y[NI * VEC], ss = 0.f;
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
-      const int cb = i * 32 * VEC + lane * VEC;
-      float x[VEC];
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) x[e] = 0.f;
-      if (cb < n) {
-        if (VEC == 2 && sizeof(T) == 2) {
-          const float2 f = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(proj + t * p.ld + c0 + cb));
-          x[0] = f.x;
-          x[VEC - 1] = f.y;
-        } else {
-#pragma unroll
-          for (int e = 0; e < VEC; ++e) x[e] = to_f32(proj[t * p.ld + c0 + cb + e]);
-        }
-      }
 #pragma unroll
       for (int e = 0; e < VEC; ++e) {
-        const int q = i * VEC + e, c = cb + e;
+        const int q = i * VEC + e, c = i * 32 * VEC + lane * VEC + e;
         float v = 0.f;
         if (FAST) {
-          v = w[0][q] * hist[0][q] + w[1][q] * hist[1][q] + w[2][q] * hist[2][q] + w[3][q] * x[e];
+          v = w[0][q] * hist[0][q] + w[1][q] * hist[1][q] + w[2][q] * hist[2][q] + w[3][q] * in[k][q];
           hist[0][q] = hist[1][q];
           hist[1][q] = hist[2][q];
-          hist[2][q] = x[e];
+          hist[2][q] = in[k][q];
         } else if (c < n) {
           for (int j = 0; j < taps; ++j)
             v += p.conv_w[static_cast<long long>(c0 + c) * taps + j] *
                  conv_input<T>(p, t - (taps - 1) + j, start, prev, c0 + c, C);
         }
-        y[q] = silu(v);
+        y[q] = c < n ? act_silu<T>(v) : 0.f;
         ss += y[q] * y[q];
       }
     }
@@ -194,13 +201,13 @@ __global__ void __launch_bounds__(128) delta_inputs_kernel(DeltaParams p) {
         else dst[cb] = y[i] * f;
       }
     }
-    const int next = p.row_next[t];
-    if (next >= 0)
-      for (int c = lane; c < n; c += 32)
-        for (int j = 0; j < taps - 1; ++j)
-          p.state[next * p.state_ld + static_cast<long long>(j) * C + c0 + c] =
-              conv_input<T>(p, t - (taps - 2) + j, start, prev, c0 + c, C);
   }
+  const int next = t1 == end ? p.row_next[end - 1] : -1;
+  if (next >= 0)
+    for (int c = lane; c < n; c += 32)
+      for (int j = 0; j < taps - 1; ++j)
+        p.state[next * p.state_ld + static_cast<long long>(j) * C + c0 + c] =
+            conv_input<T>(p, end - (taps - 1) + j, start, prev, c0 + c, C);
 }
 
 constexpr int SC_TILE = 32;                // tokens staged at a time
@@ -685,8 +692,9 @@ struct BlockScanParams {
 // block 0 of portion z; the portions' ranges do not overlap
 __device__ __forceinline__ long long first_block(const int* cu, int z) { return cu[z] / BS_BLOCK + z; }
 
+// x = hi + lo exactly: hi keeps the 11 leading bits (a TF32 number), lo the other 13, of which the product uses 11
 __device__ __forceinline__ void split_tf32(float x, uint32_t& hi, uint32_t& lo) {
-  asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(hi) : "f"(x));
+  hi = __float_as_uint(x) & 0xffffe000u;
   lo = __float_as_uint(x - __uint_as_float(hi));
 }
 __device__ __forceinline__ void mma_tf32(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
@@ -702,15 +710,27 @@ __device__ __forceinline__ void split_tile(const float (&c)[4], uint32_t (&hi)[4
   split_tf32(c[1], hi[2], lo[2]);
   split_tf32(c[3], hi[3], lo[3]);
 }
-// c += A b, the small products into `d`
-__device__ __forceinline__ void mma_split(float (&c)[4], float (&d)[4], const uint32_t (&hi)[4], const uint32_t (&lo)[4], float b0,
-                                          float b1) {
-  uint32_t h0, l0, h1, l1;
-  split_tf32(b0, h0, l0);
-  split_tf32(b1, h1, l1);
-  mma_tf32(c, hi, h0, h1);
-  mma_tf32(d, hi, l0, l1);
-  mma_tf32(d, lo, h0, h1);
+// B operand of two values, split
+struct SplitB {
+  uint32_t h0, h1, l0, l1;
+  __device__ __forceinline__ SplitB() {}
+  __device__ __forceinline__ SplitB(float b0, float b1) {
+    split_tf32(b0, h0, l0);
+    split_tf32(b1, h1, l1);
+  }
+};
+// the three products of a split A operand with a split B operand, each into an accumulator of its own: no product waits for
+// the one before
+__device__ __forceinline__ void mma_split(float (&c)[3][4], const uint32_t (&hi)[4], const uint32_t (&lo)[4], const SplitB& b) {
+  mma_tf32(c[0], hi, b.h0, b.h1);
+  mma_tf32(c[1], hi, b.l0, b.l1);
+  mma_tf32(c[2], lo, b.h0, b.h1);
+}
+__device__ __forceinline__ void zero_acc(float (&c)[3][4]) {
+#pragma unroll
+  for (int i = 0; i < 3; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) c[i][e] = 0.f;
 }
 
 template <bool DELTA, int NT, int WR, typename TV> struct BlockScan {
@@ -730,6 +750,7 @@ template <bool DELTA, int NT, int WR, typename TV> struct BlockScan {
 template <bool DELTA, int NT, int WR, typename TV>
 __global__ void __launch_bounds__(128, 2) block_scan_kernel(BlockScanParams p) {
   using Z = BlockScan<DELTA, NT, WR, TV>;
+  constexpr int XT = NT < 4 ? NT : 4;
   extern __shared__ __align__(16) uint8_t smb[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
   const int wr = warp % WR, wc = warp / WR;
@@ -798,10 +819,30 @@ __global__ void __launch_bounds__(128, 2) block_scan_kernel(BlockScanParams p) {
     for (int b = 0; b < blocks; ++b) {
       const float* tok = qk + b * BS_BLOCK * 2 * Z::KS + r_first;            // [token][q, k][row]
       const float* co = cof + b * Z::CO;
-      // products with the state before the block: column g (g + 8), tokens 2t, 2t + 1
-      float xk[4] = {0.f, 0.f, 0.f, 0.f}, xq[4] = {0.f, 0.f, 0.f, 0.f};
+      const float* A = co + (DELTA ? 64 : 0);
+      const float2 av = *reinterpret_cast<const float2*>(A + gid * 8 + tig * 2);
+      float2 tv, gm, rt;
+      float g8 = 1.f;
+      if (DELTA) {
+        tv = *reinterpret_cast<const float2*>(co + gid * 8 + tig * 2);
+        gm = *reinterpret_cast<const float2*>(co + 128 + tig * 2);
+        rt = *reinterpret_cast<const float2*>(co + 136 + tig * 2);
+        g8 = co[128 + 7];
+      }
+      float u[4];                                        // v, then U: column g (g + 8), tokens 2t, 2t + 1
       {
-        float yk[4] = {0.f, 0.f, 0.f, 0.f}, yq[4] = {0.f, 0.f, 0.f, 0.f};
+        const TV* vv = vt + (b * BS_BLOCK + tig * 2) * Z::VS + wc * 16 + gid;
+        u[0] = to_f32(vv[0]);
+        u[1] = to_f32(vv[Z::VS]);
+        u[2] = to_f32(vv[8]);
+        u[3] = to_f32(vv[Z::VS + 8]);
+      }
+      // products with the state before the block
+      float xk[4], xq[4];
+      {
+        float ck[3][4], cq[3][4];
+        zero_acc(ck);
+        zero_acc(cq);
 #pragma unroll
         for (int x = 0; x < NT; ++x) {
           uint32_t hi[4], lo[4];
@@ -809,15 +850,15 @@ __global__ void __launch_bounds__(128, 2) block_scan_kernel(BlockScanParams p) {
           const float* src = tok + gid * 2 * Z::KS + x * 8 + tig * 2;
           if (DELTA) {
             const float2 kv = *reinterpret_cast<const float2*>(src + Z::KS);
-            mma_split(xk, yk, hi, lo, kv.x, kv.y);
+            mma_split(ck, hi, lo, SplitB(kv.x, kv.y));
           }
           const float2 qv = *reinterpret_cast<const float2*>(src);
-          mma_split(xq, yq, hi, lo, qv.x, qv.y);
+          mma_split(cq, hi, lo, SplitB(qv.x, qv.y));
         }
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          xk[e] += yk[e];
-          xq[e] += yq[e];
+          xk[e] = ck[0][e] + (ck[1][e] + ck[2][e]);
+          xq[e] = cq[0][e] + (cq[1][e] + cq[2][e]);
         }
       }
       if (WR > 1) {                                      // sum over the warps that share the columns, in a fixed order
@@ -839,56 +880,63 @@ __global__ void __launch_bounds__(128, 2) block_scan_kernel(BlockScanParams p) {
         }
         parity ^= 1;
       }
-      float u[4];                                        // v, then U
-      {
-        const TV* vv = vt + (b * BS_BLOCK + tig * 2) * Z::VS + wc * 16 + gid;
-        u[0] = to_f32(vv[0]);
-        u[1] = to_f32(vv[Z::VS]);
-        u[2] = to_f32(vv[8]);
-        u[3] = to_f32(vv[Z::VS + 8]);
-      }
-      uint32_t uh[4], ul[4];
-      const float* A = co + (DELTA ? 64 : 0);
+      uint32_t uh[4], ul[4], wh[4], wl[4];               // U; U with the decay to the block's end
       if (DELTA) {
-        const float2 gm = *reinterpret_cast<const float2*>(co + 128 + tig * 2);
         u[0] -= gm.x * xk[0]; u[1] -= gm.y * xk[1]; u[2] -= gm.x * xk[2]; u[3] -= gm.y * xk[3];
-        xq[0] *= gm.x; xq[1] *= gm.y; xq[2] *= gm.x; xq[3] *= gm.y;
         split_tile(u, uh, ul);
-        const float2 tv = *reinterpret_cast<const float2*>(co + gid * 8 + tig * 2);
-        float c[4] = {0.f, 0.f, 0.f, 0.f}, d[4] = {0.f, 0.f, 0.f, 0.f};
-        mma_split(c, d, uh, ul, tv.x, tv.y);
+        float c[3][4];
+        zero_acc(c);
+        mma_split(c, uh, ul, SplitB(tv.x, tv.y));
 #pragma unroll
-        for (int e = 0; e < 4; ++e) u[e] = c[e] + d[e];
-      }
-      split_tile(u, uh, ul);
-      if (wr == 0) {
-        const float2 av = *reinterpret_cast<const float2*>(A + gid * 8 + tig * 2);
-        float d[4] = {0.f, 0.f, 0.f, 0.f};
-        mma_split(xq, d, uh, ul, av.x, av.y);
+        for (int e = 0; e < 4; ++e) u[e] = c[0][e] + (c[1][e] + c[2][e]);
+        split_tile(u, uh, ul);
+        u[0] *= rt.x; u[1] *= rt.y; u[2] *= rt.x; u[3] *= rt.y;
+        split_tile(u, wh, wl);
+      } else {
+        split_tile(u, uh, ul);
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const int tt = t + b * BS_BLOCK + tig * 2 + (e & 1), c = c0 + (e >> 1) * 8;
-          if (tt < n && c < p.V) p.o[static_cast<long long>(row0 + tt) * p.H * p.V + h * p.V + c] = xq[e] + d[e];
+          wh[e] = uh[e];
+          wl[e] = ul[e];
         }
-      }
-      if (DELTA) {
-        const float2 rt = *reinterpret_cast<const float2*>(co + 136 + tig * 2);
-        u[0] *= rt.x; u[1] *= rt.y; u[2] *= rt.x; u[3] *= rt.y;
-        split_tile(u, uh, ul);
       }
       const float* kt = tok + Z::KS;
 #pragma unroll
-      for (int x = 0; x < NT; ++x) {
-        if (DELTA) {
-          const float g8 = co[128 + 7];
+      for (int x0 = 0; x0 < NT; x0 += XT) {              // XT row tiles at a time: their products interleave
+        SplitB kb[XT];
 #pragma unroll
-          for (int e = 0; e < 4; ++e) S[x][e] *= g8;
-        } else {
-          const float2 pd = *reinterpret_cast<const float2*>(co + BS_COEF_WKV + r_first + x * 8 + tig * 2);
-          S[x][0] *= pd.x; S[x][1] *= pd.y; S[x][2] *= pd.x; S[x][3] *= pd.y;
+        for (int x = 0; x < XT; ++x) {
+          const float* src = kt + tig * 4 * Z::KS + (x0 + x) * 8 + gid;
+          kb[x] = SplitB(src[0], src[2 * Z::KS]);
+          float (&s4)[4] = S[x0 + x];
+          if (DELTA) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) s4[e] *= g8;
+          } else {
+            const float2 pd = *reinterpret_cast<const float2*>(co + BS_COEF_WKV + r_first + (x0 + x) * 8 + tig * 2);
+            s4[0] *= pd.x; s4[1] *= pd.y; s4[2] *= pd.x; s4[3] *= pd.y;
+          }
         }
-        const float b0 = kt[tig * 4 * Z::KS + x * 8 + gid], b1 = kt[(tig * 4 + 2) * Z::KS + x * 8 + gid];
-        mma_split(S[x], S[x], uh, ul, b0, b1);
+#pragma unroll
+        for (int x = 0; x < XT; ++x) mma_tf32(S[x0 + x], wh, kb[x].l0, kb[x].l1);
+#pragma unroll
+        for (int x = 0; x < XT; ++x) mma_tf32(S[x0 + x], wl, kb[x].h0, kb[x].h1);
+#pragma unroll
+        for (int x = 0; x < XT; ++x) mma_tf32(S[x0 + x], wh, kb[x].h0, kb[x].h1);
+      }
+      if (wr == 0) {
+        float c[3][4];
+        zero_acc(c);
+        mma_split(c, uh, ul, SplitB(av.x, av.y));
+        if (DELTA) {
+          xq[0] *= gm.x; xq[1] *= gm.y; xq[2] *= gm.x; xq[3] *= gm.y;
+        }
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int tt = t + b * BS_BLOCK + tig * 2 + (e & 1), cc = c0 + (e >> 1) * 8;
+          if (tt < n && cc < p.V)
+            p.o[static_cast<long long>(row0 + tt) * p.H * p.V + h * p.V + cc] = (xq[e] + c[0][e]) + (c[1][e] + c[2][e]);
+        }
       }
     }
   }
@@ -979,7 +1027,7 @@ __global__ void __launch_bounds__(128) delta_blocks_kernel(const float* __restri
 // R~, K~, A and the decay of every block of the WKV recurrence: one warp per (block, head).  grid (blocks of the longest
 // portion, ceil(H / 4), portions).
 template <typename T>
-__global__ void __launch_bounds__(128) wkv_blocks_kernel(WkvParams p, float* __restrict__ rt, float* __restrict__ kt,
+__global__ void __launch_bounds__(128, 3) wkv_blocks_kernel(WkvParams p, float* __restrict__ rt, float* __restrict__ kt,
                                                          float* __restrict__ coef, float* __restrict__ row_decay) {
   const int z = blockIdx.z, h = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31, D = p.D, HD = p.H * D;
   const int row0 = p.cu[z] + blockIdx.x * BS_BLOCK, n = min(BS_BLOCK, p.cu[z + 1] - row0);
@@ -990,33 +1038,47 @@ __global__ void __launch_bounds__(128) wkv_blocks_kernel(WkvParams p, float* __r
   for (int i = 0; i < 32; ++i) low[i] = 0.f;
 #pragma unroll
   for (int i = 0; i < 8; ++i) diag[i] = 0.f;
-  for (int c = lane; c < D; c += 32) {
-    const float w0 = p.w0[h * D + c], uu = p.u[h * D + c];
-    float r[8], k[8], w[8];
+  const T* x = reinterpret_cast<const T*>(p.rkvg) + row0 * p.ld + h * D;
+  const float* raw = p.w_raw + static_cast<long long>(row0) * HD + h * D;
+  for (int c = lane * 2; c < D; c += 64) {               // two neighbouring channels per lane
+    float r[8][2], k[8][2], w[8][2];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {                        // all loads of the block at once
+      const int ii = min(i, n - 1);
+      const float2 rr = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(x + ii * p.ld + c));
+      const float2 kk = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(x + ii * p.ld + HD + c));
+      const float2 ww = *reinterpret_cast<const float2*>(raw + static_cast<long long>(ii) * HD + c);
+      r[i][0] = rr.x; r[i][1] = rr.y; k[i][0] = kk.x; k[i][1] = kk.y; w[i][0] = ww.x; w[i][1] = ww.y;
+    }
+    const float2 w0 = *reinterpret_cast<const float2*>(p.w0 + h * D + c), uu = *reinterpret_cast<const float2*>(p.u + h * D + c);
+    float head[2] = {1.f, 1.f}, tail[2] = {1.f, 1.f};
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
-      const T* x = reinterpret_cast<const T*>(p.rkvg) + (row0 + i) * p.ld + h * D + c;
-      r[i] = i < n ? to_f32(x[0]) : 0.f;
-      k[i] = i < n ? to_f32(x[HD]) : 0.f;
-      w[i] = i < n ? expf(-expf(p.w_raw[static_cast<long long>(row0 + i) * HD + h * D + c] + w0)) : 1.f;
-    }
-    float head = 1.f, tail = 1.f;
+      const bool in = i < n;
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      if (i < n) rt[static_cast<long long>(row0 + i) * HD + h * D + c] = r[i] * head;
-      head *= w[i];
-      diag[i] += r[i] * uu * k[i];
+      for (int e = 0; e < 2; ++e) {
+        r[i][e] = in ? r[i][e] : 0.f;
+        k[i][e] = in ? k[i][e] : 0.f;
+        w[i][e] = in ? expf(-expf(w[i][e] + (e ? w0.y : w0.x))) : 1.f;
+        diag[i] += r[i][e] * (e ? uu.y : uu.x) * k[i][e];
+      }
+      if (in) *reinterpret_cast<float2*>(rt + static_cast<long long>(row0 + i) * HD + h * D + c) = make_float2(r[i][0] * head[0], r[i][1] * head[1]);
+      head[0] *= w[i][0];
+      head[1] *= w[i][1];
     }
-    row_decay[at * D + c] = head;
+    *reinterpret_cast<float2*>(row_decay + at * D + c) = make_float2(head[0], head[1]);
 #pragma unroll
     for (int j = 7; j >= 0; --j) {
-      if (j < n) kt[static_cast<long long>(row0 + j) * HD + h * D + c] = k[j] * tail;
-      tail *= w[j];
-      float f = k[j];
+      if (j < n) *reinterpret_cast<float2*>(kt + static_cast<long long>(row0 + j) * HD + h * D + c) = make_float2(k[j][0] * tail[0], k[j][1] * tail[1]);
 #pragma unroll
-      for (int i = j + 1; i < 8; ++i) {
-        low[i * (i - 1) / 2 + j] += r[i] * f;
-        f *= w[i];
+      for (int e = 0; e < 2; ++e) {
+        tail[e] *= w[j][e];
+        float f = k[j][e];
+#pragma unroll
+        for (int i = j + 1; i < 8; ++i) {
+          low[i * (i - 1) / 2 + j] += r[i][e] * f;
+          f *= w[i][e];
+        }
       }
     }
   }
@@ -1034,51 +1096,75 @@ __global__ void __launch_bounds__(128) wkv_blocks_kernel(WkvParams p, float* __r
 // ---------------------------------------------------------------------------------------------------------
 // norm and gate of a scan's result: out = o / rms_head(o) * w * silu(gate) * scale, one warp per (row, head)
 // ---------------------------------------------------------------------------------------------------------
-template <typename T, int VEC>
+template <typename T, int VEC> __device__ __forceinline__ void load_act(const T* p, float (&v)[VEC]) {
+  if (VEC == 4 && sizeof(T) == 2) {
+    const uint2 r = *reinterpret_cast<const uint2*>(p);
+    const float2 x = unpack_bf16x2(r.x), y = unpack_bf16x2(r.y);
+    v[0] = x.x; v[VEC > 1 ? 1 : 0] = x.y; v[VEC > 2 ? 2 : 0] = y.x; v[VEC > 3 ? 3 : 0] = y.y;
+  } else {
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) v[e] = to_f32(p[e]);
+  }
+}
+
+constexpr int GN_ROWS = 4;       // rows of a warp, their loads in flight together
+
+// grid (ceil(rows / GN_ROWS), ceil(H / heads of a CTA)); LPH lanes per head of up to LPH * VEC * NI values
+template <typename T, int VEC, int NI, int LPH>
 __global__ void __launch_bounds__(256)
 gated_norm_kernel(const float* __restrict__ o, const float* __restrict__ w, int w_head, const T* __restrict__ gate,
                   long long gate_ld, T* __restrict__ out, long long out_ld, int rows, int H, int V, float eps, float scale) {
-  const int lane = threadIdx.x & 31;
-  const long long item = blockIdx.x * 8ll + (threadIdx.x >> 5);
-  if (item >= static_cast<long long>(rows) * H) return;
-  const int t = static_cast<int>(item / H), h = static_cast<int>(item % H);
-  const float* src = o + item * V;
-  float ss = 0.f;
-  for (int c = lane * VEC; c < V; c += 32 * VEC) {
-    if (VEC == 4) {
-      const float4 a = *reinterpret_cast<const float4*>(src + c);
-      ss += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
-    } else {
-      ss += src[c] * src[c];
+  constexpr int HPW = 32 / LPH;
+  const int lane = threadIdx.x & 31, sub = lane % LPH, t0 = blockIdx.x * GN_ROWS;
+  const int h = (blockIdx.y * 8 + (threadIdx.x >> 5)) * HPW + lane / LPH;
+  const bool on = h < H;
+  float a[GN_ROWS][NI][VEC], b[GN_ROWS][NI][VEC];
+#pragma unroll
+  for (int k = 0; k < GN_ROWS; ++k) {
+    const long long t = min(t0 + k, rows - 1);
+    const float* src = o + (t * H + h) * V;
+    const T* g = gate + t * gate_ld + h * V;
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int c = (i * LPH + sub) * VEC;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) a[k][i][e] = b[k][i][e] = 0.f;
+      if (on && c < V) {
+        if (VEC == 4) {
+          const float4 f = *reinterpret_cast<const float4*>(src + c);
+          a[k][i][0] = f.x; a[k][i][VEC > 1 ? 1 : 0] = f.y; a[k][i][VEC > 2 ? 2 : 0] = f.z; a[k][i][VEC > 3 ? 3 : 0] = f.w;
+        } else {
+          a[k][i][0] = src[c];
+        }
+        load_act<T, VEC>(g + c, b[k][i]);
+      }
     }
   }
-  const float inv = scale / sqrtf(warp_sum(ss) / static_cast<float>(V) + eps);
-  const T* g = gate + t * gate_ld + h * V;
-  T* dst = out + t * out_ld + h * V;
-  const float* wh = w + h * w_head;
-  for (int c = lane * VEC; c < V; c += 32 * VEC) {
-    float a[VEC], b[VEC];
-    if (VEC == 4) {
-      const float4 f = *reinterpret_cast<const float4*>(src + c);
-      a[0] = f.x; a[VEC > 1 ? 1 : 0] = f.y; a[VEC > 2 ? 2 : 0] = f.z; a[VEC > 3 ? 3 : 0] = f.w;
-    } else {
-      a[0] = src[c];
-    }
-    if (VEC == 4 && sizeof(T) == 2) {
-      const uint2 r = *reinterpret_cast<const uint2*>(g + c);
-      const float2 x = unpack_bf16x2(r.x), y = unpack_bf16x2(r.y);
-      b[0] = x.x; b[VEC > 1 ? 1 : 0] = x.y; b[VEC > 2 ? 2 : 0] = y.x; b[VEC > 3 ? 3 : 0] = y.y;
-    } else {
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) b[e] = to_f32(g[c + e]);
-    }
+  for (int k = 0; k < GN_ROWS; ++k) {
+    float ss = 0.f;
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) a[e] = a[e] * inv * wh[c + e] * silu(b[e]);
-    if (VEC == 4 && sizeof(T) == 2) {
-      *reinterpret_cast<uint2*>(dst + c) = make_uint2(pack_bf16x2(a[0], a[VEC > 1 ? 1 : 0]), pack_bf16x2(a[VEC > 2 ? 2 : 0], a[VEC > 3 ? 3 : 0]));
-    } else {
+    for (int i = 0; i < NI; ++i)
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) dst[c + e] = from_f32<T>(a[e]);
+      for (int e = 0; e < VEC; ++e) ss += a[k][i][e] * a[k][i][e];
+#pragma unroll
+    for (int m = LPH / 2; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+    const float inv = scale / sqrtf(ss / static_cast<float>(V) + eps);
+    T* dst = out + (t0 + k) * out_ld + h * V;
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int c = (i * LPH + sub) * VEC;
+      if (on && c < V && t0 + k < rows) {
+        float r[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) r[e] = a[k][i][e] * inv * w[h * w_head + c + e] * act_silu<T>(b[k][i][e]);
+        if (VEC == 4 && sizeof(T) == 2) {
+          *reinterpret_cast<uint2*>(dst + c) = make_uint2(pack_bf16x2(r[0], r[VEC > 1 ? 1 : 0]), pack_bf16x2(r[VEC > 2 ? 2 : 0], r[VEC > 3 ? 3 : 0]));
+        } else {
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) dst[c + e] = from_f32<T>(r[e]);
+        }
+      }
     }
   }
 }
@@ -1302,7 +1388,7 @@ template <typename K> static int allow_smem(K kernel, size_t bytes) {
 template <typename T, int VEC, int NI>
 static int launch_inputs(const DeltaParams& p, cudaStream_t st) {
   const int units = 2 * p.G + p.H + 1;
-  const dim3 grid((p.rows + DI_TOKENS - 1) / DI_TOKENS, (units + 3) / 4);
+  const dim3 grid((p.max_rows + DI_TOKENS - 1) / DI_TOKENS, (units + 3) / 4, p.portions);
   if (p.taps <= 4) delta_inputs_kernel<T, VEC, NI, true><<<grid, 128, 0, st>>>(p);
   else delta_inputs_kernel<T, VEC, NI, false><<<grid, 128, 0, st>>>(p);
   return (int)cudaGetLastError();
@@ -1353,13 +1439,15 @@ template <typename T, int VEC> static int launch_delta_step(const DeltaParams& p
 template <typename T> static int launch_gated_norm(const float* o, const float* w, int w_head, const void* gate, long long gate_ld,
                                                    void* out, long long out_ld, int rows, int H, int V, float eps, float scale,
                                                    cudaStream_t st) {
-  const unsigned grid = (unsigned)((static_cast<long long>(rows) * H + 7) / 8);
   const uintptr_t bits = reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(out);
   const bool vec = V % 4 == 0 && gate_ld % 4 == 0 && out_ld % 4 == 0 && bits % (4 * sizeof(T)) == 0;
   const T* g = reinterpret_cast<const T*>(gate);
   T* d = reinterpret_cast<T*>(out);
-  if (vec) gated_norm_kernel<T, 4><<<grid, 256, 0, st>>>(o, w, w_head, g, gate_ld, d, out_ld, rows, H, V, eps, scale);
-  else gated_norm_kernel<T, 1><<<grid, 256, 0, st>>>(o, w, w_head, g, gate_ld, d, out_ld, rows, H, V, eps, scale);
+  auto grid = [&](int heads_per_warp) { return dim3((rows + GN_ROWS - 1) / GN_ROWS, (H + 8 * heads_per_warp - 1) / (8 * heads_per_warp)); };
+  if (vec && V <= 64) gated_norm_kernel<T, 4, 1, 16><<<grid(2), 256, 0, st>>>(o, w, w_head, g, gate_ld, d, out_ld, rows, H, V, eps, scale);
+  else if (vec && V <= 128) gated_norm_kernel<T, 4, 1, 32><<<grid(1), 256, 0, st>>>(o, w, w_head, g, gate_ld, d, out_ld, rows, H, V, eps, scale);
+  else if (vec) gated_norm_kernel<T, 4, 2, 32><<<grid(1), 256, 0, st>>>(o, w, w_head, g, gate_ld, d, out_ld, rows, H, V, eps, scale);
+  else gated_norm_kernel<T, 1, 8, 32><<<grid(1), 256, 0, st>>>(o, w, w_head, g, gate_ld, d, out_ld, rows, H, V, eps, scale);
   return (int)cudaGetLastError();
 }
 
@@ -1371,12 +1459,16 @@ static int launch_block_scan(const BlockScanParams& p, int portions, cudaStream_
   return (int)cudaGetLastError();
 }
 
-// key rows of a head split over WR warps; more of them when the grid would leave SMs idle
+// The key rows of a head are split over WR warps: over more when there are few (head, portion) pairs.
 template <bool DELTA, typename TV> static int dispatch_block_scan(const BlockScanParams& p, int portions, cudaStream_t st) {
-  const bool few = static_cast<long long>((p.V + 63) / 64) * p.H * portions < sm_count();
-  if (p.D <= 32) return launch_block_scan<DELTA, 4, 1, TV>(p, portions, st);
-  if (p.D <= 64) return few ? launch_block_scan<DELTA, 4, 2, TV>(p, portions, st) : launch_block_scan<DELTA, 8, 1, TV>(p, portions, st);
-  if (p.D <= 128) return launch_block_scan<DELTA, 8, 2, TV>(p, portions, st);
+  const long long cols = static_cast<long long>((p.V + 15) / 16) * p.H * portions;    // 16-column groups
+  const bool few = cols * (p.D <= 64 ? 1 : 2) < 6 * sm_count();
+  if (p.D <= 32) return few ? launch_block_scan<DELTA, 2, 2, TV>(p, portions, st) : launch_block_scan<DELTA, 4, 1, TV>(p, portions, st);
+  if (p.D <= 64) {
+    if (!few) return launch_block_scan<DELTA, 8, 1, TV>(p, portions, st);
+    return cols < 3 * sm_count() ? launch_block_scan<DELTA, 2, 4, TV>(p, portions, st) : launch_block_scan<DELTA, 4, 2, TV>(p, portions, st);
+  }
+  if (p.D <= 128) return few ? launch_block_scan<DELTA, 4, 4, TV>(p, portions, st) : launch_block_scan<DELTA, 8, 2, TV>(p, portions, st);
   return launch_block_scan<DELTA, 8, 4, TV>(p, portions, st);
 }
 
@@ -1395,14 +1487,14 @@ using namespace ts;
 // Portions of prompts, step 1: convolved inputs [rows][C] and gates [rows][2 H]; leaves the convolution state.
 extern "C" int ts_delta_inputs(const void* proj, long long ld, const float* conv_w, const float* A_log, const float* dt_bias,
                                float q_scale, float* state, long long state_ld, const int* row_prev, const int* row_next,
-                               const int* cu, const int* row_seq, int seq0, float* qkv, float* gates, int rows, int H, int G,
-                               int D, int V, int taps, int fp32, void* stream) {
-  if (rows <= 0) return 0;
-  if (!delta_sizes_ok(H, G, D, V, taps)) return -10;
+                               const int* cu, int portions, int max_rows, float* qkv, float* gates, int H, int G, int D, int V,
+                               int taps, int fp32, void* stream) {
+  if (portions <= 0) return 0;
+  if (!delta_sizes_ok(H, G, D, V, taps) || portions > 65535 || max_rows <= 0) return -10;
   DeltaParams p = {};
   p.proj = proj; p.ld = ld; p.conv_w = conv_w; p.A_log = A_log; p.dt_bias = dt_bias; p.q_scale = q_scale; p.state = state;
-  p.state_ld = state_ld; p.row_prev = row_prev; p.row_next = row_next; p.cu = cu; p.row_seq = row_seq; p.seq0 = seq0;
-  p.qkv = qkv; p.gates = gates; p.rows = rows; p.H = H; p.G = G; p.D = D; p.V = V; p.taps = taps;
+  p.state_ld = state_ld; p.row_prev = row_prev; p.row_next = row_next; p.cu = cu; p.portions = portions;
+  p.max_rows = max_rows; p.qkv = qkv; p.gates = gates; p.H = H; p.G = G; p.D = D; p.V = V; p.taps = taps;
   return fp32 ? dispatch_inputs<float>(p, ST(stream)) : dispatch_inputs<__nv_bfloat16>(p, ST(stream));
 }
 
@@ -1469,7 +1561,7 @@ extern "C" int ts_wkv_block_scan(const void* rkvg, long long ld, const float* w_
 extern "C" int ts_gated_norm(const float* o, const float* w, int w_head, const void* gate, long long gate_ld, void* out,
                              long long out_ld, int rows, int H, int V, float eps, float scale, int fp32, void* stream) {
   if (rows <= 0) return 0;
-  if (H <= 0 || V <= 0) return -10;
+  if (H <= 0 || V <= 0 || V > 256) return -10;
   return fp32 ? launch_gated_norm<float>(o, w, w_head, gate, gate_ld, out, out_ld, rows, H, V, eps, scale, ST(stream))
               : launch_gated_norm<__nv_bfloat16>(o, w, w_head, gate, gate_ld, out, out_ld, rows, H, V, eps, scale, ST(stream));
 }

@@ -1,6 +1,7 @@
 // Sliding-window attention with grouped queries over a paged cache whose rows hold a token's keys and values side by side:
 // row = [G key heads x dim | G value heads x vdim | padding].
 //
+//   ts_window_angles  cosines and sines of a step's positions, shared by all layers with the same frequencies
 //   ts_window_prep    per-head RMS norm of queries and keys, rotary embedding of the first `rot` dimensions of a head
 //                     (in place in the projection), cache write of keys and values - one launch
 //   ts_window_attend  single query rows (decoding, fp32, and head sizes the prefill kernel does not take) against the paged
@@ -31,29 +32,35 @@ struct WindowPrepParams {
   const float* q_norm;         // [dim]
   const float* k_norm;
   float eps;
-  const float* inv_freq;       // [rot / 2]
-  const int* pos;
+  const float* angles;         // [T][cos (rot / 2) | sin (rot / 2)]
   const long long* slots;
   void* cache;
   int T, H, G, dim, vdim, rot, row_width;
 };
 
-constexpr int WP_WARPS = 4;
+__global__ void window_angles_kernel(const float* __restrict__ inv_freq, const int* __restrict__ pos, float* __restrict__ out, int T,
+                                     int half) {
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= T * half) return;
+  const int t = i / half, f = i - t * half;
+  float s, c;
+  sincosf(static_cast<float>(pos[t]) * inv_freq[f], &s, &c);
+  out[static_cast<long long>(t) * 2 * half + f] = c;
+  out[static_cast<long long>(t) * 2 * half + half + f] = s;
+}
 
-// One CTA per token; a warp takes heads in turn.
+constexpr int WP_WARPS = 8;
+
+// Any sizes: one CTA per token, a warp takes heads in turn.
 template <typename T>
 __global__ void __launch_bounds__(WP_WARPS * 32) window_prep_kernel(WindowPrepParams p) {
-  extern __shared__ float sm[];            // cos | sin of the token's angles
   const int t = blockIdx.x, half = p.rot / 2, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  float* cs = sm;
+  const float* cs = p.angles + static_cast<long long>(t) * p.rot;
   T* row = reinterpret_cast<T*>(p.proj) + t * p.ld;
   T* crow = reinterpret_cast<T*>(p.cache) + p.slots[t] * p.row_width;
-  const float ps = static_cast<float>(p.pos[t]);
-  for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(ps * p.inv_freq[i], &cs[half + i], &cs[i]);
   const T* v = row + (p.H + p.G) * p.dim;
   for (int c = threadIdx.x; c < p.row_width - p.G * p.dim; c += blockDim.x)
     crow[p.G * p.dim + c] = c < p.G * p.vdim ? v[c] : from_f32<T>(0.f);
-  __syncthreads();
   for (int h = warp; h < p.H + p.G; h += WP_WARPS) {
     T* x = row + h * p.dim;
     float ss = 0.f;
@@ -83,74 +90,82 @@ __global__ void __launch_bounds__(WP_WARPS * 32) window_prep_kernel(WindowPrepPa
   }
 }
 
-// bf16, all sizes multiples of eight: LPH lanes hold one head as 16-byte vectors, 32 / LPH heads per warp pass; the two
-// halves of a rotated pair meet through shared memory.
+// bf16, head sizes multiples of eight.  A warp takes 32 / LPH heads of a token, LPH lanes hold one head as 16-byte vectors;
+// or it copies 32 vectors of the token's values.  The halves of a rotated pair meet by shuffles when they are whole vectors
+// apart, else through shared memory.
 template <int LPH>
 __global__ void __launch_bounds__(WP_WARPS * 32) window_prep_vec_kernel(WindowPrepParams p) {
   constexpr int HPW = 32 / LPH;
-  extern __shared__ float sm[];            // cos | sin [rot] | q_norm | k_norm | per warp and head slot [dim]
+  __shared__ float swap[WP_WARPS][HPW][LPH * 8];
   const int half = p.rot / 2, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  float* cs = sm;
-  float* wq = sm + (p.rot + 3) / 4 * 4;
-  float* buf = wq + 2 * p.dim + (warp * HPW + lane / LPH) * p.dim;
-  const int sub = lane % LPH;
-  const bool in = sub * 8 < p.dim;
-  for (int c = threadIdx.x; c < 2 * p.dim; c += blockDim.x) wq[c] = c < p.dim ? p.q_norm[c] : p.k_norm[c - p.dim];
-  for (int t = blockIdx.x; t < p.T; t += gridDim.x) {
-    __nv_bfloat16* row = reinterpret_cast<__nv_bfloat16*>(p.proj) + t * p.ld;
-    __nv_bfloat16* crow = reinterpret_cast<__nv_bfloat16*>(p.cache) + p.slots[t] * p.row_width;
-    const float ps = static_cast<float>(p.pos[t]);
-    __syncthreads();                       // the angles of the token before are no longer read
-    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(ps * p.inv_freq[i], &cs[half + i], &cs[i]);
-    const uint4* v = reinterpret_cast<const uint4*>(row + (p.H + p.G) * p.dim);
-    uint4* cv = reinterpret_cast<uint4*>(crow + p.G * p.dim);
-    for (int c = threadIdx.x; c < p.G * p.vdim / 8; c += blockDim.x) cv[c] = v[c];
-    __syncthreads();
-    for (int h0 = warp * HPW; h0 < p.H + p.G; h0 += WP_WARPS * HPW) {
-      const int h = h0 + lane / LPH;
-      const bool on = in && h < p.H + p.G;
-      __nv_bfloat16* x = row + h * p.dim + sub * 8;
-      float a[8];
-      float ss = 0.f;
-      if (on) {
-        const uint4 raw = *reinterpret_cast<const uint4*>(x);
-        const uint32_t r[4] = {raw.x, raw.y, raw.z, raw.w};
+  const int head_items = (p.H + p.G + HPW - 1) / HPW, per_token = head_items + (p.G * p.vdim / 8 + 31) / 32;
+  const unsigned item = blockIdx.x * WP_WARPS + warp;
+  const int t = item / per_token, part = item - t * per_token;
+  if (t >= p.T) return;
+  __nv_bfloat16* row = reinterpret_cast<__nv_bfloat16*>(p.proj) + t * p.ld;
+  __nv_bfloat16* crow = reinterpret_cast<__nv_bfloat16*>(p.cache) + p.slots[t] * p.row_width;
+  if (part >= head_items) {
+    const int c = (part - head_items) * 32 + lane;
+    if (c < p.G * p.vdim / 8)
+      reinterpret_cast<uint4*>(crow + p.G * p.dim)[c] = reinterpret_cast<const uint4*>(row + (p.H + p.G) * p.dim)[c];
+    return;
+  }
+  const int sub = lane % LPH, slot = lane / LPH, h = part * HPW + slot, c0 = sub * 8;
+  const bool on = c0 < p.dim && h < p.H + p.G;
+  __nv_bfloat16* x = row + h * p.dim + c0;
+  float a[8];
+  float ss = 0.f;
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          const float2 f = unpack_bf16x2(r[j]);
-          a[2 * j] = f.x;
-          a[2 * j + 1] = f.y;
-          ss += f.x * f.x + f.y * f.y;
-        }
-      }
+  for (int j = 0; j < 8; ++j) a[j] = 0.f;
+  if (on) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(x);
+    const uint32_t r[4] = {raw.x, raw.y, raw.z, raw.w};
 #pragma unroll
-      for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-      const float inv = 1.f / sqrtf(ss / static_cast<float>(p.dim) + p.eps);
-      if (on) {
-        const float* w = (h < p.H ? wq : wq + p.dim) + sub * 8;
-#pragma unroll
-        for (int j = 0; j < 8; ++j) {
-          a[j] *= inv * w[j];
-          if (sub * 8 < p.rot) buf[sub * 8 + j] = a[j];
-        }
-      }
-      __syncwarp();
-      if (on) {
-        if (sub * 8 < p.rot) {
-#pragma unroll
-          for (int j = 0; j < 8; ++j) {
-            const int c = sub * 8 + j;
-            if (c < half) a[j] = a[j] * cs[c] - buf[c + half] * cs[half + c];
-            else if (c < p.rot) a[j] = a[j] * cs[c - half] + buf[c - half] * cs[c];
-          }
-        }
-        const uint4 o = make_uint4(pack_bf16x2(a[0], a[1]), pack_bf16x2(a[2], a[3]), pack_bf16x2(a[4], a[5]),
-                                   pack_bf16x2(a[6], a[7]));
-        *reinterpret_cast<uint4*>(x) = o;
-        if (h >= p.H) *reinterpret_cast<uint4*>(crow + (h - p.H) * p.dim + sub * 8) = o;
-      }
-      __syncwarp();
+    for (int j = 0; j < 4; ++j) {
+      const float2 f = unpack_bf16x2(r[j]);
+      a[2 * j] = f.x;
+      a[2 * j + 1] = f.y;
+      ss += f.x * f.x + f.y * f.y;
     }
+  }
+  const float* w = (h < p.H ? p.q_norm : p.k_norm) + c0;
+  const float* cs = p.angles + static_cast<long long>(t) * p.rot;
+#pragma unroll
+  for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  const float inv = 1.f / sqrtf(ss / static_cast<float>(p.dim) + p.eps);
+  if (on) {
+#pragma unroll
+    for (int j = 0; j < 8; ++j) a[j] *= inv * w[j];
+  }
+  if (half % 8 == 0 && p.rot > 0) {
+    const bool first = c0 < half, rotated = c0 < p.rot;
+    const int other = slot * LPH + (first ? sub + half / 8 : (rotated ? sub - half / 8 : sub)), f0 = first ? c0 : c0 - half;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const float b = __shfl_sync(0xffffffffu, a[j], other);
+      if (on && rotated) {
+        const float c = cs[f0 + j], s = cs[half + f0 + j];
+        a[j] = first ? a[j] * c - b * s : a[j] * c + b * s;
+      }
+    }
+  } else if (p.rot > 0) {
+    float* buf = swap[warp][slot];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) buf[c0 + j] = a[j];
+    __syncwarp();
+    if (on) {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const int c = c0 + j;
+        if (c < half) a[j] = a[j] * cs[c] - buf[c + half] * cs[half + c];
+        else if (c < p.rot) a[j] = a[j] * cs[c - half] + buf[c - half] * cs[c];
+      }
+    }
+  }
+  if (on) {
+    const uint4 o = make_uint4(pack_bf16x2(a[0], a[1]), pack_bf16x2(a[2], a[3]), pack_bf16x2(a[4], a[5]), pack_bf16x2(a[6], a[7]));
+    *reinterpret_cast<uint4*>(x) = o;
+    if (h >= p.H) *reinterpret_cast<uint4*>(crow + (h - p.H) * p.dim + c0) = o;
   }
 }
 
@@ -476,32 +491,37 @@ TS_DEFINE_ERROR_API(ts_window)
 using namespace ts;
 #define ST(s) reinterpret_cast<cudaStream_t>(s)
 
+// out: [T][cos | sin of pos * inv_freq], half frequencies.
+extern "C" int ts_window_angles(const float* inv_freq, const int* pos, float* out, int T, int half, void* stream) {
+  if (T <= 0 || half <= 0) return 0;
+  window_angles_kernel<<<(T * half + 255) / 256, 256, 0, ST(stream)>>>(inv_freq, pos, out, T, half);
+  return (int)cudaGetLastError();
+}
+
+// angles: of ts_window_angles (unused without rotated dimensions).
 extern "C" int ts_window_prep(void* proj, long long ld, const float* q_norm, const float* k_norm, float eps,
-                              const float* inv_freq, const int* pos, const long long* slots, void* cache, int T, int H,
-                              int G, int dim, int vdim, int rot, int row_width, int fp32, void* stream) {
+                              const float* angles, const long long* slots, void* cache, int T, int H, int G, int dim, int vdim,
+                              int rot, int row_width, int fp32, void* stream) {
   if (T <= 0) return 0;
   if (H <= 0 || G <= 0 || dim <= 0 || vdim <= 0 || rot < 0 || rot > dim || rot % 2 || row_width < G * (dim + vdim)) return -10;
   WindowPrepParams p;
-  p.proj = proj; p.ld = ld; p.q_norm = q_norm; p.k_norm = k_norm; p.eps = eps; p.inv_freq = inv_freq; p.pos = pos;
-  p.slots = slots; p.cache = cache; p.T = T; p.H = H; p.G = G; p.dim = dim; p.vdim = vdim; p.rot = rot;
-  p.row_width = row_width;
-  const bool vec = !fp32 && dim % 8 == 0 && vdim % 8 == 0 && dim <= 256 && ld % 8 == 0 && row_width % 8 == 0 &&
-                   row_width == G * (dim + vdim) && (reinterpret_cast<uintptr_t>(proj) & 15u) == 0;
+  p.proj = proj; p.ld = ld; p.q_norm = q_norm; p.k_norm = k_norm; p.eps = eps; p.angles = angles; p.slots = slots;
+  p.cache = cache; p.T = T; p.H = H; p.G = G; p.dim = dim; p.vdim = vdim; p.rot = rot; p.row_width = row_width;
+  const bool vec = !fp32 && dim % 8 == 0 && vdim % 8 == 0 && dim <= 256 && ld % 8 == 0 && row_width == G * (dim + vdim) &&
+                   ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(cache)) & 15u) == 0;
   if (vec) {
     int lph = 4;
     while (lph * 8 < dim) lph *= 2;
-    const size_t smem = ((rot + 3) / 4 * 4 + 2 * dim + static_cast<size_t>(WP_WARPS) * (32 / lph) * dim) * 4;
-    int grid = sm_count() * 8;
-    if (grid > T) grid = T;
-    if (lph == 4) window_prep_vec_kernel<4><<<grid, WP_WARPS * 32, smem, ST(stream)>>>(p);
-    else if (lph == 8) window_prep_vec_kernel<8><<<grid, WP_WARPS * 32, smem, ST(stream)>>>(p);
-    else if (lph == 16) window_prep_vec_kernel<16><<<grid, WP_WARPS * 32, smem, ST(stream)>>>(p);
-    else window_prep_vec_kernel<32><<<grid, WP_WARPS * 32, smem, ST(stream)>>>(p);
+    const int hpw = 32 / lph, per_token = (H + G + hpw - 1) / hpw + (G * vdim / 8 + 31) / 32;
+    const unsigned grid = (unsigned)((static_cast<long long>(T) * per_token + WP_WARPS - 1) / WP_WARPS);
+    if (lph == 4) window_prep_vec_kernel<4><<<grid, WP_WARPS * 32, 0, ST(stream)>>>(p);
+    else if (lph == 8) window_prep_vec_kernel<8><<<grid, WP_WARPS * 32, 0, ST(stream)>>>(p);
+    else if (lph == 16) window_prep_vec_kernel<16><<<grid, WP_WARPS * 32, 0, ST(stream)>>>(p);
+    else window_prep_vec_kernel<32><<<grid, WP_WARPS * 32, 0, ST(stream)>>>(p);
     return (int)cudaGetLastError();
   }
-  const size_t smem = (rot + 4) * sizeof(float);
-  if (fp32) window_prep_kernel<float><<<T, WP_WARPS * 32, smem, ST(stream)>>>(p);
-  else window_prep_kernel<__nv_bfloat16><<<T, WP_WARPS * 32, smem, ST(stream)>>>(p);
+  if (fp32) window_prep_kernel<float><<<T, WP_WARPS * 32, 0, ST(stream)>>>(p);
+  else window_prep_kernel<__nv_bfloat16><<<T, WP_WARPS * 32, 0, ST(stream)>>>(p);
   return (int)cudaGetLastError();
 }
 

@@ -16,7 +16,7 @@ layer (the inner size of the WKV decay from its tensor).
 from __future__ import annotations
 
 import math
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 from typing import Any
 
 import torch
@@ -174,6 +174,21 @@ def _up8(n: int) -> int:
     return -(-n // 8) * 8
 
 
+@dataclass
+class StepContext:
+    """What the layers of one step share."""
+    rows: stream.StreamRows
+    positions: torch.Tensor
+    row_len: torch.Tensor                       # keys of a row before the window is applied
+    side: "torch.cuda.Stream | None"            # captured decode: stream of the second mixer of a parallel layer
+    _angles: dict[Rotation, torch.Tensor] = field(default_factory=dict)
+
+    def angles(self, rot: Rotation, inv_freq: torch.Tensor) -> torch.Tensor:
+        if rot not in self._angles:
+            self._angles[rot] = window.angles(inv_freq, self.positions)
+        return self._angles[rot]
+
+
 class ParallelMixer(nn.Module):
     """Windowed attention (left) and gated delta rule (right) on the same input; projection row:
     left q | k | v | right q | k | v | gate | beta | decay."""
@@ -218,20 +233,20 @@ class ParallelMixer(nn.Module):
     def state_width(self) -> int:
         return self.cfg.right.state_width
 
-    def _attend(self, proj: torch.Tensor, out: torch.Tensor, batch, cache: torch.Tensor, row_len: torch.Tensor) -> None:
+    def _attend(self, proj: torch.Tensor, out: torch.Tensor, batch, cache: torch.Tensor, ctx: "StepContext") -> None:
         s, T = self.cfg.left, proj.shape[0]
         tensor_cores = proj.is_cuda and proj.dtype == torch.bfloat16 and window.portions_supported(s)
         nd = batch.n_single if tensor_cores else T
-        window.prepare(proj, s, self.q_norm, self.k_norm, self.eps, self.inv_freq, batch.positions, batch.slots, cache)
+        window.prepare(proj, s, self.q_norm, self.k_norm, self.eps, ctx.angles(self.cfg.rot, self.inv_freq), batch.slots, cache)
         if nd > 0:
-            window.attend_rows(proj[:nd], s, cache, batch.block_table, batch.row_seq[:nd], row_len[:nd], batch.max_len, out[:nd],
+            window.attend_rows(proj[:nd], s, cache, batch.block_table, batch.row_seq[:nd], ctx.row_len[:nd], batch.max_len, out[:nd],
                                self.cfg.left_scale)
         if nd < T:
-            ctx = batch.prompt_context(s.window)
-            rows = None if ctx.slots is None else latent.gather_rows(cache, ctx.slots)
-            window.attend_portions(proj[nd:], s, rows, ctx.cu_q, ctx.cu_k, ctx.max_q, out[nd:], self.cfg.left_scale)
+            keys = batch.prompt_context(s.window)
+            rows = None if keys.slots is None else latent.gather_rows(cache, keys.slots)
+            window.attend_portions(proj[nd:], s, rows, keys.cu_q, keys.cu_k, keys.max_q, out[nd:], self.cfg.left_scale)
 
-    def forward(self, h: torch.Tensor, batch, cache, state: torch.Tensor, rows, row_len, side) -> torch.Tensor:
+    def forward(self, h: torch.Tensor, batch, cache, state: torch.Tensor, ctx: "StepContext") -> torch.Tensor:
         a, b = self.cfg.left, self.cfg.right
         T, used = h.shape[0], a.out_width + b.out_width
         proj = gemm.serve_linear(h, self.w_in)
@@ -241,18 +256,18 @@ class ParallelMixer(nn.Module):
 
         def right():
             recurrent.delta_rule(proj[:, self.right_at:], b, DeltaWeights(self.conv, self.A_log, self.dt_bias, self.norm),
-                                 self.eps, rows, batch.row_seq, state, batch.n_single, batch.portions,
+                                 self.eps, ctx.rows, state, batch.n_single, batch.portions,
                                  both[:, a.out_width:used], self.cfg.right_scale)
 
-        if side is not None:        # a captured decode step is a chain of short kernels: both mixers at once
+        if ctx.side is not None:    # a captured decode step is a chain of short kernels: both mixers at once
             main = torch.cuda.current_stream()
-            side.wait_stream(main)
-            with torch.cuda.stream(side):
+            ctx.side.wait_stream(main)
+            with torch.cuda.stream(ctx.side):
                 right()
-            self._attend(proj, both[:, :a.out_width], batch, cache["kv"], row_len)
-            main.wait_stream(side)
+            self._attend(proj, both[:, :a.out_width], batch, cache["kv"], ctx)
+            main.wait_stream(ctx.side)
         else:
-            self._attend(proj, both[:, :a.out_width], batch, cache["kv"], row_len)
+            self._attend(proj, both[:, :a.out_width], batch, cache["kv"], ctx)
             right()
         return gemm.serve_linear(both, self.w_o)
 
@@ -284,7 +299,7 @@ class WkvMixer(nn.Module):
     def state_width(self) -> int:
         return self.cfg.shape.state_width
 
-    def forward(self, mixes: torch.Tensor, batch, cache, state: torch.Tensor, rows, row_len, side) -> torch.Tensor:
+    def forward(self, mixes: torch.Tensor, batch, cache, state: torch.Tensor, ctx: "StepContext") -> torch.Tensor:
         s, T = self.cfg.shape, mixes.shape[0]
         rkvg = torch.empty(T, 4, s.inner, dtype=mixes.dtype, device=mixes.device)
         if mixes.is_cuda and gemm.few_rows(T, 4 * s.inner, mixes.shape[2]):
@@ -295,7 +310,7 @@ class WkvMixer(nn.Module):
         inner = gemm.serve_linear(mixes[:, 4], self.w1, act=grouped.ACT_TANH)
         w_raw = gemm.serve_linear(inner, self.w2, torch.float32)
         out = torch.empty(T, s.inner, dtype=mixes.dtype, device=mixes.device)
-        recurrent.wkv(rkvg, w_raw, s, WkvWeights(self.w0, self.u, self.norm), self.eps, rows, state, batch.n_single,
+        recurrent.wkv(rkvg, w_raw, s, WkvWeights(self.w0, self.u, self.norm), self.eps, ctx.rows, state, batch.n_single,
                       batch.portions, out)
         return gemm.serve_linear(out, self.w_o)
 
@@ -394,11 +409,10 @@ class VibepelForCausalLM(nn.Module):
         the last)."""
         cfg, L, dtype = self.config, len(self.layers), self.embed.dtype
         rows = stream.StreamRows(batch.row_prev, batch.row_next)
-        row_len = batch.positions + 1
-        side = self._side_stream() if batch.captured else None
+        ctx = StepContext(rows, batch.positions, batch.positions + 1, self._side_stream() if batch.captured else None)
         x, h = stream.scaled_embed(batch.token_ids, self.embed, cfg.embed_scale, self.layers[0].mixer.mu, rows, cache.state[0])
         for i, layer in enumerate(self.layers):
-            y = layer.mixer(h, batch, cache.entries[i], cache.state[i], rows, row_len, side)
+            y = layer.mixer(h, batch, cache.entries[i], cache.state[i], ctx)
             norm = layer.norm1
             if layer.ff is not None:
                 x, h = stream.postnorm(x, y, norm, cfg.eps, None, rows, None, dtype)

@@ -131,7 +131,7 @@ def _delta_reference(proj, s: DeltaShape, w: DeltaWeights, eps, rows, state, n_s
             state[nxt, s.matrix_offset:s.matrix_offset + S.numel()] = S.reshape(-1)
 
 
-def delta_rule(proj: torch.Tensor, s: DeltaShape, w: DeltaWeights, eps: float, rows: StreamRows, row_seq, state: torch.Tensor,
+def delta_rule(proj: torch.Tensor, s: DeltaShape, w: DeltaWeights, eps: float, rows: StreamRows, state: torch.Tensor,
                n_single: int, portions, out: torch.Tensor, out_scale: float = 1.0) -> None:
     """proj [T, proj_width] (a column slice of a wider projection) -> out [T, heads * vdim] = out_scale * gated norm of the
     rule's result.  `portions`: offsets of the multi-token sequences after the `n_single` single rows (inference/batch)."""
@@ -142,7 +142,7 @@ def delta_rule(proj: torch.Tensor, s: DeltaShape, w: DeltaWeights, eps: float, r
         delta_step(proj[:n_single], s, w, eps, rows, state, out[:n_single], out_scale)
     if n_single < T:
         tail = StreamRows(rows.prev[n_single:], rows.next[n_single:])
-        qkv, gates = delta_inputs(proj[n_single:], s, w, tail, row_seq[n_single:], state, n_single, portions)
+        qkv, gates = delta_inputs(proj[n_single:], s, w, tail, state, portions)
         o = delta_scan(qkv, gates, s, tail, state, portions, proj.dtype == torch.bfloat16)
         gate = proj[n_single:, s.channels:s.channels + s.out_width]
         gated_norm(o, w.norm, 0, gate, out[n_single:], s.heads, s.vdim, eps, out_scale)
@@ -158,7 +158,7 @@ def delta_step(proj, s: DeltaShape, w: DeltaWeights, eps: float, rows: StreamRow
     _lib.check(rc, "ts_delta_step")
 
 
-def delta_inputs(proj, s: DeltaShape, w: DeltaWeights, rows: StreamRows, row_seq, state, seq0: int, portions):
+def delta_inputs(proj, s: DeltaShape, w: DeltaWeights, rows: StreamRows, state, portions):
     """Convolved and normed q | k | v [T, channels] and log decay | beta [T, 2 heads] of portions, both fp32."""
     T = proj.shape[0]
     qkv = torch.empty(T, s.channels, dtype=torch.float32, device=proj.device)
@@ -166,7 +166,7 @@ def delta_inputs(proj, s: DeltaShape, w: DeltaWeights, rows: StreamRows, row_seq
     rc = _lib.load("recurrent").ts_delta_inputs(
         _lib.ptr(proj), _ll(proj.stride(0)), _lib.ptr(w.conv), _lib.ptr(w.A_log), _lib.ptr(w.dt_bias), _f(s.dim ** -0.5),
         _lib.ptr(state), _ll(state.stride(0)), _lib.ptr(rows.prev), _lib.ptr(rows.next), _lib.ptr(portions.cu),
-        _lib.ptr(row_seq), seq0, _lib.ptr(qkv), _lib.ptr(gates), T, s.heads, s.kv_heads, s.dim, s.vdim, s.taps,
+        portions.count, portions.longest, _lib.ptr(qkv), _lib.ptr(gates), s.heads, s.kv_heads, s.dim, s.vdim, s.taps,
         int(proj.dtype == torch.float32), _lib.stream_ptr())
     _lib.check(rc, "ts_delta_inputs")
     return qkv, gates

@@ -58,13 +58,24 @@ def _norm_rotate(x: torch.Tensor, w: torch.Tensor, eps: float, cos: torch.Tensor
     return torch.cat([u * cos - v * sin, v * cos + u * sin, y[..., rot:]], dim=-1).to(x.dtype)
 
 
-def prepare(proj: torch.Tensor, s: WindowShape, q_norm, k_norm, eps: float, inv_freq, pos, slots, cache) -> None:
-    """proj [T, >= q_width + kv_width] = (queries | keys | values | ...).  Norms and rotates queries and keys in place and
-    writes keys and values to cache rows `slots`."""
+def angles(inv_freq: torch.Tensor, pos: torch.Tensor) -> torch.Tensor:
+    """cos | sin of pos * inv_freq, fp32 [T, 2 * frequencies]: once per step for all layers that rotate alike."""
+    if not pos.is_cuda:
+        a = pos.float()[:, None] * inv_freq
+        return torch.cat([a.cos(), a.sin()], dim=-1)
+    out = torch.empty(pos.shape[0], 2 * inv_freq.shape[0], dtype=torch.float32, device=pos.device)
+    rc = _lib.load("window").ts_window_angles(_lib.ptr(inv_freq), _lib.ptr(pos), _lib.ptr(out), pos.shape[0], inv_freq.shape[0],
+                                              _lib.stream_ptr())
+    _lib.check(rc, "ts_window_angles")
+    return out
+
+
+def prepare(proj: torch.Tensor, s: WindowShape, q_norm, k_norm, eps: float, cs: torch.Tensor, slots, cache) -> None:
+    """proj [T, >= q_width + kv_width] = (queries | keys | values | ...); cs of `angles`.  Norms and rotates queries and keys
+    in place and writes keys and values to cache rows `slots`."""
     T = proj.shape[0]
     if not proj.is_cuda:
-        ang = pos.float()[:, None] * inv_freq
-        cos, sin = ang.cos()[:, None], ang.sin()[:, None]
+        cos, sin = cs[:, None, :s.rot // 2], cs[:, None, s.rot // 2:]
         q = proj[:, :s.q_width].view(T, s.heads, s.dim)
         k = proj[:, s.q_width:s.q_width + s.kv_heads * s.dim].view(T, s.kv_heads, s.dim)
         q.copy_(_norm_rotate(q, q_norm, eps, cos, sin, s.rot))
@@ -72,9 +83,9 @@ def prepare(proj: torch.Tensor, s: WindowShape, q_norm, k_norm, eps: float, inv_
         cache.view(-1, s.row_width)[slots, :s.kv_width] = proj[:, s.q_width:s.q_width + s.kv_width]
         return
     rc = _lib.load("window").ts_window_prep(
-        _lib.ptr(proj), _ll(proj.stride(0)), _lib.ptr(q_norm), _lib.ptr(k_norm), _f(eps), _lib.ptr(inv_freq), _lib.ptr(pos),
-        _lib.ptr(slots), _lib.ptr(cache), T, s.heads, s.kv_heads, s.dim, s.vdim, s.rot, s.row_width,
-        int(proj.dtype == torch.float32), _lib.stream_ptr())
+        _lib.ptr(proj), _ll(proj.stride(0)), _lib.ptr(q_norm), _lib.ptr(k_norm), _f(eps), _lib.ptr(cs), _lib.ptr(slots),
+        _lib.ptr(cache), T, s.heads, s.kv_heads, s.dim, s.vdim, s.rot, s.row_width, int(proj.dtype == torch.float32),
+        _lib.stream_ptr())
     _lib.check(rc, "ts_window_prep")
 
 
