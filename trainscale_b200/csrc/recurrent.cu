@@ -953,74 +953,88 @@ __global__ void __launch_bounds__(128, 2) block_scan_kernel(BlockScanParams p) {
   }
 }
 
-// T, A, gamma of every block of the delta rule.  grid (blocks of the longest portion, G, portions), 128 threads.
+// T, A, gamma of every block of the delta rule, one warp per (block, query / key head): k_i . k_j and q_i . k_j are one MMA
+// with the rows [K; Q] and the columns K, whose operands are read once, straight from global memory.
+// grid (blocks of the longest portion, ceil(G / 4), portions)
 __global__ void __launch_bounds__(128) delta_blocks_kernel(const float* __restrict__ qkv, const float* __restrict__ gates,
                                                            const int* __restrict__ cu, float* __restrict__ coef, int H, int G,
                                                            int D, int V) {
-  extern __shared__ __align__(16) float sm[];            // q, k of the block [8][2][D + 4]
-  __shared__ float dots[2][8][8], lg[8], bt[8], Lm[8][8];
-  const int z = blockIdx.z, g = blockIdx.y, rep = H / G, C = 2 * G * D + H * V, KS = D + 4, tid = threadIdx.x;
+  __shared__ float lower[4][8][9];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
+  const int z = blockIdx.z, g = blockIdx.y * 4 + warp, rep = H / G, C = 2 * G * D + H * V;
   const int row0 = cu[z] + blockIdx.x * BS_BLOCK, n = min(BS_BLOCK, cu[z + 1] - row0);
-  if (n <= 0) return;
-  for (int i = tid; i < BS_BLOCK * 2 * (D / 4); i += 128) {
-    const int tk = i / (2 * (D / 4)), r = i - tk * 2 * (D / 4), w = r / (D / 4), c = (r - w * (D / 4)) * 4;
-    *reinterpret_cast<float4*>(sm + (tk * 2 + w) * KS + c) =
-        tk < n ? *reinterpret_cast<const float4*>(qkv + static_cast<long long>(row0 + tk) * C + (w * G + g) * D + c)
-               : make_float4(0.f, 0.f, 0.f, 0.f);
-  }
-  __syncthreads();
-  {   // thread (i, j, which): k_i . k_j or q_i . k_j, the lower triangle
-    const int which = tid >> 6, i = (tid >> 3) & 7, j = tid & 7;
-    float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f;
-    if (j <= i) {
-      const float *x = sm + (i * 2 + 1 - which) * KS, *y = sm + (j * 2 + 1) * KS;
-#pragma unroll 8
-      for (int c = 0; c < D; c += 4) {
-        const float4 a = *reinterpret_cast<const float4*>(x + c), b = *reinterpret_cast<const float4*>(y + c);
-        d0 += a.x * b.x; d1 += a.y * b.y; d2 += a.z * b.z; d3 += a.w * b.w;
+  if (n <= 0 || g >= G) return;
+  const long long block = first_block(cu, z) + blockIdx.x;
+  float (&Lm)[8][9] = lower[warp];
+  float dots[3][4];                                      // k_i . k_j (0, 1) and q_i . k_j (2, 3): i = gid, j = 2 tig, 2 tig + 1
+  zero_acc(dots);
+  {
+    const bool in = gid < n;
+    const float* q = qkv + static_cast<long long>(row0 + (in ? gid : 0)) * C + g * D + tig * 2;
+    const float* k = q + G * D;
+    for (int c0 = 0; c0 < D; c0 += 64) {
+      float2 qv[8], kv[8];
+#pragma unroll
+      for (int x = 0; x < 8; ++x) {
+        const bool ok = in && c0 + x * 8 < D;
+        qv[x] = ok ? *reinterpret_cast<const float2*>(q + c0 + x * 8) : make_float2(0.f, 0.f);
+        kv[x] = ok ? *reinterpret_cast<const float2*>(k + c0 + x * 8) : make_float2(0.f, 0.f);
+      }
+#pragma unroll
+      for (int x = 0; x < 8; ++x) {
+        const SplitB b(kv[x].x, kv[x].y);
+        uint32_t hi[4] = {b.h0, 0, b.h1, 0}, lo[4] = {b.l0, 0, b.l1, 0};
+        split_tf32(qv[x].x, hi[1], lo[1]);
+        split_tf32(qv[x].y, hi[3], lo[3]);
+        mma_split(dots, hi, lo, b);
       }
     }
-    dots[which][i][j] = (d0 + d1) + (d2 + d3);
   }
+  float d[4];
+#pragma unroll
+  for (int e = 0; e < 4; ++e) d[e] = dots[0][e] + (dots[1][e] + dots[2][e]);
+  const int j0 = tig * 2;
   for (int hh = 0; hh < rep; ++hh) {
     const int h = g * rep + hh;
-    __syncthreads();
-    if (tid < 8) {
-      lg[tid] = tid < n ? gates[static_cast<long long>(row0 + tid) * 2 * H + h] : 0.f;
-      bt[tid] = tid < n ? gates[static_cast<long long>(row0 + tid) * 2 * H + H + h] : 0.f;
+    float lg = 0.f, bt = 0.f;                            // of token `lane`
+    if (lane < n) {
+      lg = gates[static_cast<long long>(row0 + lane) * 2 * H + h];
+      bt = gates[static_cast<long long>(row0 + lane) * 2 * H + H + h];
     }
-    __syncthreads();
-    float* out = coef + ((first_block(cu, z) + blockIdx.x) * H + h) * BS_COEF;
-    if (tid < 64) {
-      const int i = tid >> 3, j = tid & 7;
-      float e = 0.f;
-      for (int l = j + 1; l <= i; ++l) e += lg[l];
-      e = expf(e);
-      Lm[i][j] = bt[i] * e * dots[0][i][j];
-      out[64 + tid] = j <= i ? e * dots[1][i][j] : 0.f;
-    } else if (tid < 80) {
-      const int i = tid & 7;
-      float e = 0.f;
-      if (tid < 72) {
-        for (int l = 0; l <= i; ++l) e += lg[l];
-      } else {
-        for (int l = i + 1; l < 8; ++l) e += lg[l];
-      }
-      out[64 + tid] = expf(e);
+    float e0 = 0.f, e1 = 0.f, head = 0.f, tail = 0.f;    // sums of log decays: j + 1 .. i; start .. lane; lane + 1 .. end
+#pragma unroll
+    for (int l = 0; l < 8; ++l) {
+      const float v = __shfl_sync(0xffffffffu, lg, l);
+      if (l > j0 && l <= gid) e0 += v;
+      if (l > j0 + 1 && l <= gid) e1 += v;
+      if (l <= lane) head += v;
+      else tail += v;
     }
-    __syncthreads();
-    if (tid < 8) {                                       // column tid of (I + L)^-1, times beta
+    e0 = expf(e0);
+    e1 = expf(e1);
+    const float bi = __shfl_sync(0xffffffffu, bt, gid);
+    float* out = coef + (block * H + h) * BS_COEF;
+    Lm[gid][j0] = bi * e0 * d[0];
+    Lm[gid][j0 + 1] = bi * e1 * d[1];
+    *reinterpret_cast<float2*>(out + 64 + gid * 8 + j0) = make_float2(j0 <= gid ? e0 * d[2] : 0.f, j0 + 1 <= gid ? e1 * d[3] : 0.f);
+    if (lane < 8) {
+      out[128 + lane] = expf(head);
+      out[136 + lane] = expf(tail);
+    }
+    __syncwarp();
+    if (lane < 8) {                                      // column `lane` of (I + L)^-1, times beta
       float col[8];
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
-        float v = i == tid ? 1.f : 0.f;
+        float v = i == lane ? 1.f : 0.f;
 #pragma unroll
         for (int l = 0; l < 8; ++l)
           if (l < i) v -= Lm[i][l] * col[l];
-        col[i] = i < tid ? 0.f : v;
-        out[i * 8 + tid] = col[i] * bt[tid];
+        col[i] = i < lane ? 0.f : v;
+        out[i * 8 + lane] = col[i] * bt;
       }
     }
+    __syncwarp();
   }
 }
 
@@ -1059,7 +1073,7 @@ __global__ void __launch_bounds__(128, 3) wkv_blocks_kernel(WkvParams p, float* 
       for (int e = 0; e < 2; ++e) {
         r[i][e] = in ? r[i][e] : 0.f;
         k[i][e] = in ? k[i][e] : 0.f;
-        w[i][e] = in ? expf(-expf(w[i][e] + (e ? w0.y : w0.x))) : 1.f;
+        w[i][e] = in ? __expf(-__expf(w[i][e] + (e ? w0.y : w0.x))) : 1.f;
         diag[i] += r[i][e] * (e ? uu.y : uu.x) * k[i][e];
       }
       if (in) *reinterpret_cast<float2*>(rt + static_cast<long long>(row0 + i) * HD + h * D + c) = make_float2(r[i][0] * head[0], r[i][1] * head[1]);
@@ -1459,16 +1473,18 @@ static int launch_block_scan(const BlockScanParams& p, int portions, cudaStream_
   return (int)cudaGetLastError();
 }
 
-// The key rows of a head are split over WR warps: over more when there are few (head, portion) pairs.
+// The key rows of a head stay with one warp when there are (head, portion) pairs for every SM, else they are split over two or
+// four: half the latency of a block for a third more work.
 template <bool DELTA, typename TV> static int dispatch_block_scan(const BlockScanParams& p, int portions, cudaStream_t st) {
-  const long long cols = static_cast<long long>((p.V + 15) / 16) * p.H * portions;    // 16-column groups
-  const bool few = cols * (p.D <= 64 ? 1 : 2) < 6 * sm_count();
-  if (p.D <= 32) return few ? launch_block_scan<DELTA, 2, 2, TV>(p, portions, st) : launch_block_scan<DELTA, 4, 1, TV>(p, portions, st);
-  if (p.D <= 64) {
-    if (!few) return launch_block_scan<DELTA, 8, 1, TV>(p, portions, st);
-    return cols < 3 * sm_count() ? launch_block_scan<DELTA, 2, 4, TV>(p, portions, st) : launch_block_scan<DELTA, 4, 2, TV>(p, portions, st);
-  }
-  if (p.D <= 128) return few ? launch_block_scan<DELTA, 4, 4, TV>(p, portions, st) : launch_block_scan<DELTA, 8, 2, TV>(p, portions, st);
+  const long long groups = static_cast<long long>((p.V + 15) / 16) * p.H * portions;       // of 16 value columns
+  const int wr = groups >= 4 * sm_count() ? 1 : (groups > sm_count() ? 2 : 4);
+  if (p.D <= 32) return launch_block_scan<DELTA, 4, 1, TV>(p, portions, st);
+  if (p.D <= 64)
+    return wr == 1 ? launch_block_scan<DELTA, 8, 1, TV>(p, portions, st)
+                   : (wr == 2 ? launch_block_scan<DELTA, 4, 2, TV>(p, portions, st) : launch_block_scan<DELTA, 2, 4, TV>(p, portions, st));
+  if (p.D <= 128)
+    return wr == 1 ? launch_block_scan<DELTA, 16, 1, TV>(p, portions, st)
+                   : (wr == 2 ? launch_block_scan<DELTA, 8, 2, TV>(p, portions, st) : launch_block_scan<DELTA, 4, 4, TV>(p, portions, st));
   return launch_block_scan<DELTA, 8, 4, TV>(p, portions, st);
 }
 
@@ -1525,8 +1541,8 @@ extern "C" int ts_delta_block_scan(const float* qkv, const float* gates, float* 
                                    int H, int G, int D, int V, void* stream) {
   if (portions <= 0) return 0;
   if (!delta_sizes_ok(H, G, D, V, 1) || !blocked_ok(D, V) || portions > 65535) return -10;
-  const dim3 grid((max_rows + BS_BLOCK - 1) / BS_BLOCK, G, portions);
-  delta_blocks_kernel<<<grid, 128, BS_BLOCK * 2 * (D + 4) * sizeof(float), ST(stream)>>>(qkv, gates, cu, coef, H, G, D, V);
+  const dim3 grid((max_rows + BS_BLOCK - 1) / BS_BLOCK, (G + 3) / 4, portions);
+  delta_blocks_kernel<<<grid, 128, 0, ST(stream)>>>(qkv, gates, cu, coef, H, G, D, V);
   if (int e = (int)cudaGetLastError()) return e;
   BlockScanParams p = {};
   p.q = qkv; p.k = qkv + G * D; p.v = qkv + 2 * G * D; p.qk_ld = p.v_ld = 2 * G * D + H * V; p.rep = H / G; p.coef = coef;
