@@ -11,6 +11,15 @@ pytestmark = pytest.mark.gpu
 DTYPES = [torch.float32, torch.bfloat16]
 
 
+@pytest.fixture(autouse=True)
+def _true_fp32():
+    """Library products in fp32 proper, whatever a test before this one has chosen."""
+    before = torch.get_float32_matmul_precision()
+    torch.set_float32_matmul_precision("highest")
+    yield
+    torch.set_float32_matmul_precision(before)
+
+
 def rel(got, want):
     got, want = got.double().cpu(), want.double().cpu()
     return ((got - want).pow(2).mean().sqrt() / want.pow(2).mean().sqrt().clamp(min=1e-30)).item()
