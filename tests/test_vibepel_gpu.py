@@ -125,7 +125,7 @@ def attention(q, k, v, scale, window, off):
 
 
 SHAPES = [  # H, G, dim, vdim, rot
-    (6, 1, 96, 96, 24), (8, 2, 128, 128, 64), (4, 4, 64, 64, 64), (5, 5, 40, 72, 12), (24, 1, 80, 48, 16), (3, 1, 20, 12, 6),
+    (5, 1, 96, 96, 40), (8, 2, 128, 128, 64), (4, 4, 64, 64, 64), (5, 5, 40, 72, 12), (24, 1, 80, 48, 16), (3, 1, 20, 12, 6),
     (4, 2, 18, 30, 18), (2, 1, 256, 128, 32), (2, 2, 200, 256, 0)]
 
 
@@ -275,7 +275,7 @@ def delta_oracle(s, w, x, state, eps):
     return o.reshape(-1, s.out_width), inp[x.shape[0]:], S
 
 
-DELTA = [(6, 3, 64, 64, 3), (4, 2, 128, 128, 4), (4, 4, 32, 24, 2), (3, 1, 96, 40, 1), (2, 1, 256, 64, 4), (2, 2, 20, 36, 6),
+DELTA = [(4, 2, 64, 64, 4), (4, 2, 128, 128, 4), (4, 4, 32, 24, 2), (3, 1, 96, 40, 1), (2, 1, 256, 64, 4), (2, 2, 20, 36, 6),
          (3, 3, 17, 9, 4), (2, 1, 128, 256, 2), (8, 1, 8, 8, 3), (2, 2, 256, 256, 4)]
 
 
@@ -329,7 +329,7 @@ def test_delta_rule_steps_equal_a_portion(dtype, H, G, D, V, taps):
         assert rel(left[s.matrix_offset:s.matrix_offset + S.numel()], S.reshape(-1)) < 6e-6
 
 
-WKV = [(4, 32), (2, 64), (3, 128), (1, 256), (2, 48), (3, 20), (2, 7), (5, 8)]
+WKV = [(5, 32), (2, 64), (3, 128), (1, 256), (2, 48), (3, 20), (2, 7), (5, 8)]
 
 
 def wkv_oracle(s, w, x, raw, S, eps):

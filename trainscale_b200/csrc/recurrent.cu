@@ -8,13 +8,13 @@
 // A state row of a sequence holds [convolution inputs (taps - 1) x C | S per head] or [token-shift row | S per head];
 // a step reads one row and writes another, so nothing of a launch is overwritten while it is still read.
 //
-// The scan keeps S in registers, 8 key rows x 4 value columns per thread, and walks BLOCKS of tokens: for four tokens of
-// the delta rule all products S^T k and S^T q with the state before the block are formed at once (eight vectors, one
-// reduction over the lanes that share a column), the four-step triangular recurrence that is left is solved per column
-// with the block's small Gram matrices, and the state is updated with all four writes.  So the latency of a reduction is
-// paid once per block, not per token.  Everything is fp32 arithmetic on the FMA pipe in packed pairs: the warp MMA forms
-// that keep fp32 accuracy (three TF32 products) have no higher rate, and a 128-row tensor-memory tile would need the state
-// split into two operands and written to shared memory again for every chunk.
+// Two scans.  bf16 models (`block_scan_kernel`): blocks of eight tokens as warp MMAs with operands split into two TF32 parts.
+// fp32 models and head sizes that are not multiples of eight (`delta_scan_kernel`, `wkv_scan_kernel`): fp32 arithmetic on the
+// FMA pipe in packed pairs, S in registers, 8 key rows x 4 value columns per thread.  The latter walks blocks too: for four
+// tokens of the delta rule all products S^T k and S^T q with the state before the block are formed at once (eight vectors, one
+// reduction over the lanes that share a column), the four-step triangular recurrence that is left is solved per column with
+// the block's small Gram matrices, and the state is updated with all four writes; the latency of a reduction is paid once
+// per block, not per token.
 #include "common.cuh"
 #include "host_common.h"
 

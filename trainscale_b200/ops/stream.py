@@ -1,8 +1,9 @@
-"""Residual-stream boundary ops of decoders with a depth-averaged fp32 stream (csrc/stream.cu).
+"""Residual-stream boundary ops of decoders with an fp32 stream (csrc/stream.cu).
 
-`embed` starts the stream (token row + bigram row), `boundary` closes one layer and opens the next: residual sum of a
+Depth-averaged stream: `embed` starts it (token row + bigram row), `boundary` closes one layer and opens the next: residual sum of a
 parallel block, expert combine, depth average over every earlier result, scalar-gain RMS norm and token shift in one
-launch; `final` is the last boundary for the rows whose logits are wanted.  The stream, its history and the per-sequence
+launch; `final` is the last boundary for the rows whose logits are wanted.  Output-normed sublayers: `scaled_embed`,
+`postnorm` (sum, cast or token-shift mixes) and `postnorm_final`.  The stream, its history and the per-sequence
 state are fp32; h and hs come out in the activation dtype.  Tensors on the CPU take PyTorch math.
 """
 from __future__ import annotations
