@@ -105,6 +105,21 @@ __device__ __forceinline__ float product_act(float v, int act, float cap) {
   return v;
 }
 
+__device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+
+// Factor sigmoid(gate) of an attention result: one gate per head or one per element.
+constexpr int GATE_HEAD = 1, GATE_ELEMENT = 2;
+
+// Gated products: act 4 is silu(g) * u, act 5 the tanh form of gelu(g) * u, both written as g * sigmoid(y) * u.  `FAST`:
+// for results that are rounded to 16 bits.  Their weights interleave GLU_BLOCK gate rows with the GLU_BLOCK up rows of
+// the same outputs.
+constexpr int GLU_BLOCK = 16;
+constexpr int ACT_FIRST_GLU = 4, ACT_LAST_GLU = 5;
+template <bool FAST> __device__ __forceinline__ float glu_act(float g, float u, int act) {
+  const float y = act == 5 ? 1.5957691216057308f * (g + 0.044715f * g * g * g) : g;     // 2 sqrt(2 / pi)
+  return FAST ? __fdividef(g * u, 1.f + __expf(-y)) : g / (1.f + expf(-y)) * u;
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -41,9 +41,22 @@ struct GemmParams {
   const int* seg_start;     // MODE 2: [E + 1] first row of every expert's (128-aligned) segment along the K axis
   int group_rows;           // MODE 1: rows (K-major B) or K extent (MN-major B) of one expert inside the stacked B
   int num_groups;           // MODE 2: E; C is [E][M][ldc]
-  int act;                  // epilogue activation of common.cuh product_act (modes 0 and 1; 0: none)
+  int act;                  // epilogue activation of common.cuh product_act or glu_act (modes 0 and 1; 0: none)
   float act_cap;
 };
+
+// 32 accumulator columns of a gated product = 16 gates and the 16 factors of the same outputs: 16 results.
+__device__ __forceinline__ void gemm_store_glu(const GemmParams& p, const uint32_t* r, size_t row, int col0) {
+  __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.C) + row * p.ldc + col0 / 2;
+  if (!TS_IN_BOUNDS(reinterpret_cast<const char*>(dst), GLU_BLOCK * 2, p.C, p.c_bytes, 7001)) return;
+  uint32_t o[8];
+#pragma unroll
+  for (int j = 0; j < 8; ++j)
+    o[j] = pack_bf16x2(glu_act<true>(__uint_as_float(r[2 * j]), __uint_as_float(r[GLU_BLOCK + 2 * j]), p.act),
+                       glu_act<true>(__uint_as_float(r[2 * j + 1]), __uint_as_float(r[GLU_BLOCK + 2 * j + 1]), p.act));
+  reinterpret_cast<uint4*>(dst)[0] = make_uint4(o[0], o[1], o[2], o[3]);
+  reinterpret_cast<uint4*>(dst)[1] = make_uint4(o[4], o[5], o[6], o[7]);
+}
 
 // product_act of 32 accumulators; one uniform branch per kind, so that the common kinds stay short
 __device__ __forceinline__ void gemm_activate(uint32_t* r, int act, float cap) {
@@ -334,8 +347,12 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
         uint32_t r[32];
         tmem_ld_32x32b_x32(t_row + c * 32, r);
         tc_wait_ld();
-        if (MODE != 2 && p.act != 0) gemm_activate(r, p.act, p.act_cap);
         const int col0 = n0 + c * 32;
+        if (MODE != 2 && p.act >= ACT_FIRST_GLU) {
+          if (row < p.M && col0 < p.N) gemm_store_glu(p, r, ti.c_row0 + row, col0);
+          continue;
+        }
+        if (MODE != 2 && p.act != 0) gemm_activate(r, p.act, p.act_cap);
         if (row < p.M && col0 < p.N) gemm_store_chunk(p, r, ti.c_row0 + row, col0);
       }
       tc_fence_before_sync();
@@ -497,8 +514,12 @@ gemm_bf16_2cta_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_cons
         uint32_t r[32];
         tmem_ld_32x32b_x32(t_row + c * 32, r);
         tc_wait_ld();
-        if (p.act != 0) gemm_activate(r, p.act, p.act_cap);
         const int col0 = n0 + c * 32;
+        if (p.act >= ACT_FIRST_GLU) {
+          if (row < p.M && col0 < p.N) gemm_store_glu(p, r, static_cast<size_t>(row), col0);
+          continue;
+        }
+        if (p.act != 0) gemm_activate(r, p.act, p.act_cap);
         if (row < p.M && col0 < p.N) gemm_store_chunk(p, r, static_cast<size_t>(row), col0);
       }
       tc_fence_before_sync();
@@ -556,6 +577,13 @@ static int launch_gemm(const CUtensorMap& tmA, const CUtensorMap& tmB, const Gem
   return (int)cudaGetLastError();
 }
 
+// A gated product halves the columns: whole blocks of gates and factors, 16-byte aligned bf16 rows.
+static bool glu_ok(int act, const void* C, int N, int ldc, int out_fp32) {
+  return act < ACT_FIRST_GLU || (N % (2 * GLU_BLOCK) == 0 && !out_fp32 && ldc % 8 == 0 && ldc >= N / 2 &&
+                                 (reinterpret_cast<uintptr_t>(C) & 15u) == 0);
+}
+static int result_cols(int act, int N) { return act >= ACT_FIRST_GLU ? N / 2 : N; }
+
 }  // namespace ts
 
 TS_DEFINE_ERROR_API(ts_gemm)
@@ -566,13 +594,16 @@ TS_DEFINE_ERROR_API(ts_gemm)
 //   out_fp32: C is fp32 (else bf16); accumulate: add into the existing C.
 //   bn: N tile (256, 128 or 64; 0 = choose).
 // Leading dimensions are in elements and must keep rows 16-byte aligned. Returns 0 on success.
-//   act: activation of the result (common.cuh product_act; C must not accumulate then).
+//   act: activation of the result (common.cuh product_act; C must not accumulate then).  The gated ones (glu_act) take B
+//   with gate and up rows in alternating blocks of GLU_BLOCK and write N / 2 columns.
 extern "C" int ts_gemm_bf16_act(const void* A, const void* B, void* C, int M, int N, int K, int lda, int ldb, int ldc,
                                 int a_mn, int b_mn, int out_fp32, int accumulate, float alpha, int bn, int act,
                                 float act_cap, void* stream) {
   using namespace ts;
   if (M <= 0 || N <= 0 || K <= 0) return -10;
-  if (act != 0 && (act < 0 || act > 3 || accumulate || alpha != 1.f || (act == 3 && !(act_cap > 0.f)))) return -13;
+  if (act != 0 && (act < 0 || act > ACT_LAST_GLU || accumulate || alpha != 1.f || (act == 3 && !(act_cap > 0.f)) ||
+                   !glu_ok(act, C, N, ldc, out_fp32)))
+    return -13;
   if (bn == 0) {
     // prefer the widest tile that still gives every SM work
     const int tiles256 = ((M + 127) / 128) * ((N + 255) / 256);
@@ -604,7 +635,7 @@ extern "C" int ts_gemm_bf16_act(const void* A, const void* B, void* C, int M, in
   p.k_blocks = (K + GEMM_BK - 1) / GEMM_BK;
   p.tile_expert = nullptr; p.seg_start = nullptr; p.group_rows = 0; p.num_groups = 1; p.act = act;
   p.act_cap = act_cap;
-  p.c_bytes = (static_cast<size_t>(M - 1) * ldc + N) * (out_fp32 ? 4 : 2);
+  p.c_bytes = (static_cast<size_t>(M - 1) * ldc + result_cols(act, N)) * (out_fp32 ? 4 : 2);
 #ifdef TS_DEBUG
   // test hook of the debug build: pretend C ends `TS_DEBUG_SHRINK_C_ROWS` rows early, so that the bounds check (and
   // nothing else) keeps the kernel from writing them
@@ -631,7 +662,8 @@ extern "C" int ts_gemm_bf16(const void* A, const void* B, void* C, int M, int N,
 //   mode 2 (wgrad): C[e][M][N] = sum over rows r in [seg_start[e], seg_start[e+1]) of A[r][m] * B[r][n]; both operands
 //     MN-major (a_mn = b_mn = 1), K = P.  An empty segment gives a zero slab (or leaves C alone when accumulating).
 // `groups` is the device int32 array tile_expert (mode 1, ceil(P/128) entries) or seg_start (mode 2, E + 1 entries).
-// `act` (mode 1): 1 applies max(v, 0)^2 to the product in the epilogue (C must not accumulate then).
+// `act` (mode 1): 1 applies max(v, 0)^2 to the product in the epilogue, 4 and 5 are the gated products (as above; C must
+// not accumulate then).
 // Serves the grouped expert GEMMs of data_pipeline/trainer/kernels/moe_kernels.py:219-785.
 extern "C" int ts_gemm_grouped_bf16_act(const void* A, const void* B, void* C, int mode, int M, int N, int K, int lda,
                                         int ldb, int ldc, int a_mn, int b_mn, int out_fp32, int accumulate, float alpha,
@@ -640,7 +672,9 @@ extern "C" int ts_gemm_grouped_bf16_act(const void* A, const void* B, void* C, i
   if (M <= 0 || N <= 0 || K <= 0 || num_groups <= 0 || groups == nullptr) return -10;
   // experts stacked along K (b_mn) need whole K blocks; with K-major B the tail of K is zero-filled by the loads
   if (mode == 1 && (a_mn != 0 || (b_mn && K % GEMM_BK != 0))) return -12;
-  if (act != 0 && (mode != 1 || act != 1 || accumulate || alpha != 1.f)) return -13;
+  if (act != 0 && (mode != 1 || (act != 1 && act != 4 && act != 5) || accumulate || alpha != 1.f || out_fp32 ||
+                   !glu_ok(act, C, N, ldc, out_fp32)))
+    return -13;
   if (mode == 2 && (a_mn != 1 || b_mn != 1)) return -12;
   if (mode != 1 && mode != 2) return -11;
   const int bn = (N >= 256) ? 256 : (N >= 128 ? 128 : 64);
@@ -669,7 +703,7 @@ extern "C" int ts_gemm_grouped_bf16_act(const void* A, const void* B, void* C, i
   p.num_groups = num_groups;
   p.act = act; p.act_cap = 0.f;
   p.c_bytes = (static_cast<size_t>((mode == 2 ? num_groups : 1)) * M - 1) * ldc * (out_fp32 ? 4 : 2) +
-              static_cast<size_t>(N) * (out_fp32 ? 4 : 2);
+              static_cast<size_t>(result_cols(act, N)) * (out_fp32 ? 4 : 2);
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   if (mode == 1) {
     if (bn == 256) return launch_gemm<256, 1>(tmA, tmB, p, st);

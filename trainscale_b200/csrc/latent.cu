@@ -28,7 +28,7 @@ __device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162flo
 template <typename T>
 __global__ void __launch_bounds__(128)
 latent_prep_kernel(T* __restrict__ proj, long long ld, int H, int dim, int rot, int rank, const float* __restrict__ norm_w,
-                   float eps, const float* __restrict__ inv_freq, const int* __restrict__ pos,
+                   float eps, const float* __restrict__ inv_freq, float magnitude, int pairs, const int* __restrict__ pos,
                    const long long* __restrict__ slots, T* __restrict__ cache, T* __restrict__ flat, int row_width) {
   extern __shared__ float cs[];     // cos | sin of the token's rot / 2 angles
   __shared__ float scratch[32];
@@ -36,7 +36,12 @@ latent_prep_kernel(T* __restrict__ proj, long long ld, int H, int dim, int rot, 
   T* q = proj + static_cast<long long>(t) * ld;
   const T* down = q + H * (dim + rot);
   const float p = static_cast<float>(pos[t]);
-  for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(p * inv_freq[i], &cs[half + i], &cs[i]);
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float s, c;
+    sincosf(p * inv_freq[i], &s, &c);
+    cs[i] = c * magnitude;
+    cs[half + i] = s * magnitude;
+  }
   float ss = 0.f;
   for (int r = threadIdx.x; r < rank; r += blockDim.x) {
     const float v = to_f32(down[r]);
@@ -51,20 +56,22 @@ latent_prep_kernel(T* __restrict__ proj, long long ld, int H, int dim, int rot, 
     if (r < rank) {
       v = to_f32(down[r]) * inv * norm_w[r];
     } else if (r < rank + rot) {
-      const int i = r - rank;
-      const float a = to_f32(down[r]);
-      v = i < half ? a * cs[i] - to_f32(down[r + half]) * cs[half + i]
-                   : a * cs[i - half] + to_f32(down[r - half]) * cs[i];
+      // the first of a pair turns against the second, the second with the first
+      const int i = r - rank, f = pairs ? i / 2 : (i < half ? i : i - half), step = pairs ? 1 : half;
+      const bool lead = pairs ? i % 2 == 0 : i < half;
+      const float a = to_f32(down[r]), b = to_f32(down[lead ? r + step : r - step]);
+      v = lead ? a * cs[f] - b * cs[half + f] : a * cs[f] + b * cs[half + f];
     }
     crow[r] = from_f32<T>(v);
     if (frow) frow[r] = from_f32<T>(v);
   }
   for (int i = threadIdx.x; i < H * half; i += blockDim.x) {
     const int h = i / half, j = i - h * half;
-    T* a = q + h * (dim + rot) + dim + j;
-    const float u = to_f32(a[0]), v = to_f32(a[half]), c = cs[j], s = cs[half + j];
-    a[0] = from_f32<T>(u * c - v * s);
-    a[half] = from_f32<T>(v * c + u * s);
+    T* a = q + h * (dim + rot) + dim + (pairs ? 2 * j : j);
+    T* b = a + (pairs ? 1 : half);
+    const float u = to_f32(*a), v = to_f32(*b), c = cs[j], s = cs[half + j];
+    *a = from_f32<T>(u * c - v * s);
+    *b = from_f32<T>(v * c + u * s);
   }
 }
 
@@ -418,18 +425,19 @@ using namespace ts;
 // Width of a cache row: rank + rot rounded up to whole 16-column MMA steps.
 extern "C" int ts_latent_row_width(int rank, int rot) { return (rank + rot + 15) / 16 * 16; }
 
+// cos and sin are multiplied by `magnitude`; pairs: rotation partners are coordinates 2 i and 2 i + 1 instead of i and i + rot / 2.
 extern "C" int ts_latent_prep(void* proj, long long ld, int H, int dim, int rot, int rank, const float* norm_w, float eps,
-                              const float* inv_freq, const int* pos, const long long* slots, void* cache, void* flat,
+                              const float* inv_freq, float magnitude, int pairs, const int* pos, const long long* slots, void* cache, void* flat,
                               int row_width, int rows, int fp32, void* stream) {
   if (rows <= 0) return 0;
   if (H <= 0 || rank <= 0 || rot < 0 || rot % 2 || row_width < rank + rot) return -10;
   const size_t sm = sizeof(float) * (rot > 0 ? rot : 2);
   if (fp32)
     latent_prep_kernel<float><<<rows, 128, sm, ST(stream)>>>((float*)proj, ld, H, dim, rot, rank, norm_w, eps, inv_freq,
-                                                             pos, slots, (float*)cache, (float*)flat, row_width);
+                                                             magnitude, pairs, pos, slots, (float*)cache, (float*)flat, row_width);
   else
     latent_prep_kernel<__nv_bfloat16><<<rows, 128, sm, ST(stream)>>>(
-        (__nv_bfloat16*)proj, ld, H, dim, rot, rank, norm_w, eps, inv_freq, pos, slots, (__nv_bfloat16*)cache,
+        (__nv_bfloat16*)proj, ld, H, dim, rot, rank, norm_w, eps, inv_freq, magnitude, pairs, pos, slots, (__nv_bfloat16*)cache,
         (__nv_bfloat16*)flat, row_width);
   return (int)cudaGetLastError();
 }

@@ -12,7 +12,10 @@
 //                size, so heads of any multiple of eight columns use the same code
 //   warp 1       MMA issuer: S_t = Q_t K^T over the unrotated, then the rotated columns; O_t += P_t V, P_t from TMEM
 //   warps 2..9   softmax: one thread per query row; scores, running max and sum in fp32
-// Key tiles outside every row's window are never loaded.  Queries are the LAST Lq of the sequence's Lk keys.
+// Queries are the LAST Lq of the sequence's Lk keys.  A query sees the `window` keys up to its own, or those of its chunk of
+// `window` keys (the first key row then lies on a chunk's border), and besides the first `keep` key rows; these are the
+// sequence's first positions, which a portion's caller may have put right in front of its window.  Key tiles that no row
+// sees are never loaded.  The result may be multiplied by the sigmoid of a gate per head or per element.
 #include "common.cuh"
 #include "host_common.h"
 
@@ -56,13 +59,21 @@ struct LatentPrefillParams {
   int ks_n, ks_r;                        // 16-column MMA steps
   int vdim, v_cols;                      // value size; rounded up to 16
   int k_stages, v_stages;
-  int window;
+  int window, keep, chunked;
   int kv_group;                          // query heads that share a key/value head
+  const __nv_bfloat16* gate;             // [query rows][gate_ld] (nullptr: none)
+  long long gate_ld;
+  int gate_mode;                         // GATE_HEAD: column h, GATE_ELEMENT: column h * vdim + c
   float scale_log2;
   float o_scale;                         // factor of the result
   __nv_bfloat16* o;                      // [rows][o_stride], head h at column h * vdim
   long long o_stride;
 };
+
+// first key row of the window or chunk of the query at key row c
+__device__ __forceinline__ int window_first(const LatentPrefillParams& p, int c) {
+  return p.chunked ? c / p.window * p.window : max(0, c - p.window + 1);
+}
 
 __global__ void __launch_bounds__(LP_THREADS, 1)
 latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_constant__ CUtensorMap tmQr,
@@ -96,16 +107,23 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
   if ((int)blockIdx.y >= n_qblocks) return;
   const int qb = n_qblocks - 1 - blockIdx.y;
   const int off = Lk - Lq;
-  // key tiles entirely left of the first row's window are never loaded; query tile t works on tiles [first[t], nkv[t])
-  int r0[2], first[2], nkv[2];
-  const int kb_lo = max(0, qb * 256 + off - p.window + 1) / 128;
+  // the block's key tiles: those of the kept rows left of its first window, then the windows' (kb_lo on).  Query tile t works
+  // on [0, held[t]), which hold kept rows (also where they are among the windows'), and on [first[t], nkv[t])
+  int r0[2], held[2], first[2], nkv[2];
+  const int keep_tiles = (p.keep + 127) / 128;
+  const int kb_lo = window_first(p, qb * 256 + off) / 128, kept = min(keep_tiles, kb_lo);
 #pragma unroll
   for (int t = 0; t < 2; ++t) {
     r0[t] = qb * 256 + t * 128;
-    first[t] = max(0, r0[t] + off - p.window + 1) / 128 - kb_lo;
-    nkv[t] = r0[t] >= Lq ? 0 : max(0, (min(Lk, r0[t] + 128 + off) + 127) / 128 - kb_lo);
+    first[t] = kept + window_first(p, r0[t] + off) / 128 - kb_lo;
+    held[t] = min(keep_tiles, first[t]);
+    nkv[t] = r0[t] >= Lq ? 0 : max(0, kept + (min(Lk, r0[t] + 128 + off) + 127) / 128 - kb_lo);
   }
   const int n = max(nkv[0], nkv[1]);
+  auto key_tile = [&](int i) { return i < kept ? i : kb_lo + i - kept; };
+  auto works_on = [&](int t, int i) { return i < nkv[t] && (i < held[t] || i >= first[t]); };
+  // how many tiles t has worked on before tile i
+  auto worked = [&](int t, int i) { return i < held[t] ? i : held[t] + i - first[t]; };
 
   if (threadIdx.x == 0) {
     tma_prefetch_desc(&tmQn);
@@ -137,7 +155,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
       }
       uint32_t ki = 0, vi = 0;
       for (int i = 0; i < n && alive; ++i, ++ki, ++vi) {
-        const int ks = ki % p.k_stages, vs = vi % p.v_stages, row = k_start + (kb_lo + i) * 128;
+        const int ks = ki % p.k_stages, vs = vi % p.v_stages, row = k_start + key_tile(i) * 128;
         if (!mbar_wait(&k_empty[ks], ((ki / p.k_stages) & 1u) ^ 1u, alive, 400)) break;
         mbar_expect_tx(&k_full[ks], k_bytes);
         for (int j = 0; j < p.nb_n; ++j)
@@ -173,7 +191,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
       if (n > 0 && mbar_wait(&k_full[0], 0, alive, 501)) {
         tc_fence_after_sync();
         for (int t = 0; t < 2; ++t)
-          if (nkv[t] > 0 && first[t] == 0) issue_s(t, 0);
+          if (works_on(t, 0)) issue_s(t, 0);
         umma_commit(&k_empty[0]);
       }
       for (int i = 0; i < n && alive; ++i) {
@@ -181,17 +199,17 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
         if (!mbar_wait(&v_full[vs], (i / p.v_stages) & 1u, alive, 502)) break;
         bool k_waited = false;
         for (int t = 0; t < 2 && alive; ++t) {
-          if (i >= first[t] && i < nkv[t]) {
-            if (!mbar_wait(&p_full[t], (i - first[t]) & 1u, alive, 503)) break;
+          if (works_on(t, i)) {
+            if (!mbar_wait(&p_full[t], worked(t, i) & 1u, alive, 503)) break;
             tc_fence_after_sync();
             const uint32_t va = smem_u32(v_base + vs * v_bytes);
 #pragma unroll
             for (int kk = 0; kk < 8; ++kk)
               umma_f16_ts(tmem_base + O_COL0 + t * 128, tmem_base + t * 128 + kk * 8,
-                          make_smem_desc_sw128(va + kk * 2048, LP_BLOCK, 1024), idesc_o, (i - first[t]) != 0 || kk != 0);
+                          make_smem_desc_sw128(va + kk * 2048, LP_BLOCK, 1024), idesc_o, worked(t, i) != 0 || kk != 0);
             if (i == nkv[t] - 1) umma_commit(&o_full[t]);
           }
-          if (i + 1 >= first[t] && i + 1 < nkv[t]) {
+          if (works_on(t, i + 1)) {
             if (!k_waited) {
               if (!mbar_wait(&k_full[kn], ((i + 1) / p.k_stages) & 1u, alive, 504)) break;
               tc_fence_after_sync();
@@ -214,28 +232,32 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
     const uint32_t t_s = t_lane + t * 128;
     const uint32_t t_o = t_lane + O_COL0 + t * 128;
     float m_used = -INFINITY, l = 0.f;
-    const int nt = nkv[t], i0 = first[t];
+    const int nt = nkv[t];
     const float sc = p.scale_log2;
-    for (int i = i0; i < nt && alive; ++i) {
-      if (!mbar_wait(&s_full[t], (i - i0) & 1u, alive, 600)) break;
+    const int limit = min(Lk - 1, row + off);          // last visible key
+    const int lo = window_first(p, row + off);         // first key of the window
+    const int lo_last = window_first(p, r0[t] + 127 + off);
+    for (int i = 0; i < nt && alive; ++i) {
+      if (!works_on(t, i)) continue;
+      if (!mbar_wait(&s_full[t], worked(t, i) & 1u, alive, 600)) break;
       tc_fence_after_sync();
-      const int c0 = (kb_lo + i) * 128;
-      const bool need_mask = (c0 + 127 > r0[t] + off) || (c0 + 128 > Lk) || (c0 <= r0[t] + 127 + off - p.window);
-      const int limit = min(Lk - 1, row + off);        // last visible key
-      const int lo = row + off - p.window + 1;         // first visible key
+      const int c0 = key_tile(i) * 128;
+      const bool need_mask = (c0 + 127 > r0[t] + off) || (c0 + 128 > Lk) || (c0 < lo_last && c0 + 128 > p.keep);
       uint32_t v[128];
 #pragma unroll
       for (int c = 0; c < 4; ++c) tmem_ld_32x32b_x32(t_s + c * 32, v + c * 32);
       tc_wait_ld();
       if (need_mask) {
-        // visible columns of the tile are [lo - c0, limit - c0]: one bit per column, a word per 32
-        const int a = max(lo - c0, 0), e = min(limit - c0, 127);
+        // visible columns of the tile are [lo - c0, limit - c0] and the kept ones [0, keep - c0): one bit per column, a word
+        // per 32
+        const int a = max(lo - c0, 0), e = min(limit - c0, 127), kc = p.keep - c0;
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
           const int s0 = a - c * 32, s1 = e - c * 32;      // first and last visible bit of this word
-          uint32_t bits = s1 < 0 || s0 > 31 ? 0u : 0xffffffffu;
+          uint32_t bits = s0 > 31 ? 0u : 0xffffffffu;
           if (s0 > 0) bits &= 0xffffffffu << (s0 & 31);
-          if (s1 < 31) bits &= 0xffffffffu >> (31 - (s1 & 31));
+          if (kc > c * 32) bits |= kc >= c * 32 + 32 ? 0xffffffffu : (1u << (kc - c * 32)) - 1u;
+          if (s1 < 31) bits &= s1 < 0 ? 0u : 0xffffffffu >> (31 - s1);
 #pragma unroll
           for (int j = 0; j < 32; ++j)
             if (!(bits & (1u << j))) v[c * 32 + j] = 0xff800000u;
@@ -258,7 +280,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
         const float alpha = (m_used == -INFINITY) ? 0.f : fast_ex2(m_used - m_new);
         m_used = m_new;
         l *= alpha;
-        if (i > i0) {
+        if (worked(t, i) > 0) {
 #pragma unroll 1
           for (int c = 0; c < p.v_cols / 16; ++c) {
             uint32_t o[16];
@@ -296,8 +318,11 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
     }
     if (nt > 0 && alive && mbar_wait(&o_full[t], 0, alive, 601)) {
       tc_fence_after_sync();
-      const float inv = l > 0.f ? p.o_scale / l : 0.f;
+      float inv = l > 0.f ? p.o_scale / l : 0.f;
       const bool valid = row < Lq;
+      const __nv_bfloat16* gate = p.gate ? p.gate + (q_start + row) * p.gate_ld + (p.gate_mode == GATE_HEAD ? h : h * p.vdim) : nullptr;
+      if (valid && gate && p.gate_mode == GATE_HEAD) inv *= sigmoid(__bfloat162float(*gate));
+      const bool per_element = gate && p.gate_mode == GATE_ELEMENT;
       __nv_bfloat16* dst = p.o + (q_start + row) * p.o_stride + h * p.vdim;
 #pragma unroll 1
       for (int c = 0; c < p.v_cols / 16; ++c) {
@@ -307,6 +332,16 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
           if (valid && c * 16 + j * 8 < p.vdim) {
+            if (per_element) {
+              const uint4 g4 = *reinterpret_cast<const uint4*>(gate + c * 16 + j * 8);
+              const uint32_t g[4] = {g4.x, g4.y, g4.z, g4.w};
+#pragma unroll
+              for (int x = 0; x < 4; ++x) {
+                const float2 f = unpack_bf16x2(g[x]);
+                v[8 * j + 2 * x] = __float_as_uint(__fdividef(__uint_as_float(v[8 * j + 2 * x]), 1.f + __expf(-f.x)));
+                v[8 * j + 2 * x + 1] = __float_as_uint(__fdividef(__uint_as_float(v[8 * j + 2 * x + 1]), 1.f + __expf(-f.y)));
+              }
+            }
             uint4 o4;
             o4.x = pack_bf16x2(__uint_as_float(v[8 * j]) * inv, __uint_as_float(v[8 * j + 1]) * inv);
             o4.y = pack_bf16x2(__uint_as_float(v[8 * j + 2]) * inv, __uint_as_float(v[8 * j + 3]) * inv);
@@ -350,6 +385,13 @@ static bool plan_prefill(int dim, int rot, int vdim, LatentPrefillPlan& pl) {
   return false;
 }
 
+// The gate's rows are read as 16-byte vectors when there is one per element.
+static bool gate_ok(const void* gate, long long ld, int mode, int vdim) {
+  if (!gate) return true;
+  if (mode == GATE_HEAD) return true;
+  return mode == GATE_ELEMENT && ld % 8 == 0 && vdim % 8 == 0 && (reinterpret_cast<uintptr_t>(gate) & 15u) == 0;
+}
+
 // Tensor maps are the caller's; `p` still lacks what follows from the sizes.
 static int launch_prefill(const CUtensorMap& tQn, const CUtensorMap& tQr, const CUtensorMap& tKn, const CUtensorMap& tKr,
                           const CUtensorMap& tV, const LatentPrefillPlan& pl, LatentPrefillParams p, int dim, int rot,
@@ -381,14 +423,16 @@ extern "C" int ts_latent_prefill_supported(int dim, int rot, int vdim) {
 
 // q: projection rows [q_rows][q_ld], head h at column h * (dim + rot).  kv: expanded rows [k_rows][kv_ld], unrotated key
 // of head h at column h * dim, value at column v_col0 + h * vdim.  k_rot: [k_rows][kr_ld] shared rotated key part.
-// cu_q / cu_k: [sequences + 1].  out: [q_rows][o_stride].
+// cu_q / cu_k: [sequences + 1].  out: [q_rows][o_stride], times sigmoid(gate) when there is a gate [q_rows][gate_ld].
 extern "C" int ts_latent_prefill(const void* q, long long q_ld, long long q_rows, const void* kv, long long kv_ld,
                                  int v_col0, const void* k_rot, long long kr_ld, long long k_rows, const int* cu_q,
                                  const int* cu_k, int sequences, int max_q, int H, int dim, int rot, int vdim, int window,
-                                 float scale, void* out, long long o_stride, void* stream) {
+                                 float scale, const void* gate, long long gate_ld, int gate_mode, void* out,
+                                 long long o_stride, void* stream) {
   if (sequences <= 0 || max_q <= 0) return 0;
   LatentPrefillPlan pl;
   if (H <= 0 || window <= 0 || !(scale > 0.f) || !plan_prefill(dim, rot, vdim, pl)) return -10;
+  if (!gate_ok(gate, gate_ld, gate_mode, vdim)) return -12;
   if (q_ld % 8 || kv_ld % 8 || kr_ld % 8 || o_stride % 8 || (reinterpret_cast<uintptr_t>(out) & 15u)) return -11;
   const __nv_bfloat16* qp = reinterpret_cast<const __nv_bfloat16*>(q);
   const __nv_bfloat16* kvp = reinterpret_cast<const __nv_bfloat16*>(kv);
@@ -410,20 +454,24 @@ extern "C" int ts_latent_prefill(const void* q, long long q_ld, long long q_rows
   }
   LatentPrefillParams p = {};
   p.cu_q = cu_q; p.cu_k = cu_k; p.H = H; p.window = window; p.kv_group = 1; p.o_scale = 1.f;
+  p.gate = reinterpret_cast<const __nv_bfloat16*>(gate); p.gate_ld = gate_ld; p.gate_mode = gate_mode;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.o = reinterpret_cast<__nv_bfloat16*>(out); p.o_stride = o_stride;
   return launch_prefill(tQn, tQr, tKn, tKr, tV, pl, p, dim, rot, vdim, sequences, max_q, stream);
 }
 
 // q: rows [q_rows][q_ld], head h at column h * dim.  k / v: rows [k_rows][kv_ld], key/value head g at columns g * dim and
-// g * vdim.  cu_q / cu_k: [sequences + 1].  out: [q_rows][o_stride] = o_scale * attention.
+// g * vdim.  cu_q / cu_k: [sequences + 1].  window, keep, chunked: which keys a query sees (top of the file).
+// out: [q_rows][o_stride] = o_scale * attention (* sigmoid(gate)).
 extern "C" int ts_window_prefill(const void* q, long long q_ld, long long q_rows, const void* k, const void* v,
                                  long long kv_ld, long long k_rows, const int* cu_q, const int* cu_k, int sequences,
-                                 int max_q, int H, int G, int dim, int vdim, int window, float scale, float o_scale,
-                                 void* out, long long o_stride, void* stream) {
+                                 int max_q, int H, int G, int dim, int vdim, int window, int keep, int chunked, float scale,
+                                 float o_scale, const void* gate, long long gate_ld, int gate_mode, void* out,
+                                 long long o_stride, void* stream) {
   if (sequences <= 0 || max_q <= 0) return 0;
   LatentPrefillPlan pl;
-  if (H <= 0 || G <= 0 || H % G || window <= 0 || !(scale > 0.f) || !plan_prefill(dim, 0, vdim, pl)) return -10;
+  if (H <= 0 || G <= 0 || H % G || window <= 0 || keep < 0 || !(scale > 0.f) || !plan_prefill(dim, 0, vdim, pl)) return -10;
+  if (!gate_ok(gate, gate_ld, gate_mode, vdim)) return -12;
   if (q_ld % 8 || kv_ld % 8 || o_stride % 8 || (reinterpret_cast<uintptr_t>(out) & 15u)) return -11;
   CUtensorMap tQ, tK, tV;
   const CUtensorMapDataType dt = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
@@ -435,6 +483,8 @@ extern "C" int ts_window_prefill(const void* q, long long q_ld, long long q_rows
   if (rc) return rc * 100 - 3;
   LatentPrefillParams p = {};
   p.cu_q = cu_q; p.cu_k = cu_k; p.H = H; p.window = window; p.kv_group = H / G; p.o_scale = o_scale;
+  p.keep = keep; p.chunked = chunked;
+  p.gate = reinterpret_cast<const __nv_bfloat16*>(gate); p.gate_ld = gate_ld; p.gate_mode = gate_mode;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.o = reinterpret_cast<__nv_bfloat16*>(out); p.o_stride = o_stride;
   return launch_prefill(tQ, tQ, tK, tK, tV, pl, p, dim, 0, vdim, sequences, max_q, stream);

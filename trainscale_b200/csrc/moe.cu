@@ -4,6 +4,7 @@
 //   ts_moe_permute  token rows -> expert-sorted padded buffer (pad rows zero), optionally scaled per source slot
 //   ts_moe_combine  weighted gather of the k expert outputs of every token (also the backward of the permute)
 //   ts_moe_combine_dw  gradient of the combine weights
+//   ts_moe_topk, ts_moe_route  routers: softmax or group-limited sigmoid scores, top-k (and, for a decode batch, the sort)
 // Replaces the permute / un-permute / top-k-weight kernels of data_pipeline/trainer/kernels/moe_kernels.py:219-785 and
 // the host-side argsort + bincount of data_pipeline/trainer/distributed/expert_parallel.py:219.
 #include "common.cuh"
@@ -160,10 +161,101 @@ __global__ void moe_combine_dw_kernel(const __nv_bfloat16* __restrict__ dout, co
   }
 }
 
-// Router: softmax over E experts and top-k selection, one warp per token (E <= 1024).  probs [E] fp32 (may be null) is
-// written for the auxiliary losses and the backward; weights are the selected probabilities, optionally renormalised to
-// sum to 1.  Ties resolve to the lower expert index, as torch.topk does on equal values in practice for distinct logits.
+// Routers: scores of E experts and top-k selection, one warp per token (E <= 1024).  probs [E] fp32 (may be null) is
+// written for the auxiliary losses and the backward; weights are the selected scores, optionally renormalised to sum to 1.
+// Ties resolve to the lower expert index, as torch.topk does on equal values in practice for distinct logits.
 constexpr int ROUTER_MAX_PER_LANE = 32;
+
+// the lane that holds the largest value of the warp's (value, index) pairs wins; lower index on a tie
+__device__ __forceinline__ void warp_argmax(float& best, int& at) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+    const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+    if (ob > best || (ob == best && oa < at)) {
+      best = ob;
+      at = oa;
+    }
+  }
+}
+
+// the k largest of v (lane l holds expert l + 32 j in v[j], taken and excluded ones are -1); returns their sum
+__device__ __forceinline__ float warp_select(float (&v)[ROUTER_MAX_PER_LANE], int per, int E, int k, float* weights, int* idx) {
+  const int lane = threadIdx.x & 31;
+  float wsum = 0.f;
+  for (int s = 0; s < k; ++s) {
+    float best = -1.f;
+    int best_e = 0x7fffffff;
+#pragma unroll 4
+    for (int j = 0; j < per; ++j) {
+      const int e = lane + j * 32;
+      if (e < E && v[j] > best) {
+        best = v[j];
+        best_e = e;
+      }
+    }
+    warp_argmax(best, best_e);
+    if (best_e >= E) {                         // only without a comparable score (NaN)
+      best = 0.f;
+      best_e = s;
+    }
+    if (lane == 0) {
+      weights[s] = best;
+      idx[s] = best_e;
+    }
+    wsum += best;
+    if ((best_e & 31) == lane) v[best_e >> 5] = -1.f;   // taken
+  }
+  __syncwarp();
+  return wsum;
+}
+
+// Sigmoid scores; only experts of the best `keep` of `groups` equal groups of neighbours can be chosen, a group's value being
+// the sum of its two largest scores.
+__device__ __forceinline__ void warp_topk_groups(const float* __restrict__ logits, float* weights, int* idx, int E, int k,
+                                                 int normalize, int groups, int keep) {
+  const int lane = threadIdx.x & 31, size = E / groups, per = (E + 31) / 32;
+  uint32_t kept = 0xffffffffu;                 // bit j: group lane + 32 j
+  if (keep < groups) {
+    float value[ROUTER_MAX_PER_LANE];
+    const int gper = (groups + 31) / 32;
+    for (int j = 0; j < gper; ++j) {
+      const int g = lane + j * 32;
+      float a = -INFINITY, b = -INFINITY;      // two largest logits: the sigmoid keeps their order
+      if (g < groups)
+        for (int i = 0; i < size; ++i) {
+          const float z = logits[g * size + i];
+          b = fmaxf(b, fminf(a, z));
+          a = fmaxf(a, z);
+        }
+      value[j] = g < groups ? sigmoid(a) + (size > 1 ? sigmoid(b) : 0.f) : -1.f;
+    }
+    kept = 0u;
+    for (int s = 0; s < keep; ++s) {
+      float best = -1.f;
+      int at = 0x7fffffff;
+      for (int j = 0; j < gper; ++j)
+        if (value[j] > best) {
+          best = value[j];
+          at = lane + j * 32;
+        }
+      warp_argmax(best, at);
+      if (at < groups && (at & 31) == lane) {
+        kept |= 1u << (at >> 5);
+        value[at >> 5] = -1.f;
+      }
+    }
+  }
+  float v[ROUTER_MAX_PER_LANE];
+  for (int j = 0; j < per; ++j) {
+    const int e = lane + j * 32, g = min(e, E - 1) / size;
+    const uint32_t mask = __shfl_sync(0xffffffffu, kept, g & 31);
+    v[j] = e < E && ((mask >> (g >> 5)) & 1u) ? sigmoid(logits[e]) : -1.f;
+  }
+  const float sum = warp_select(v, per, E, k, weights, idx);
+  if (normalize && lane < k) weights[lane] /= sum + 1e-20f;
+}
+
 __device__ __forceinline__ void warp_topk_softmax(const float* __restrict__ logits, float* probs, float* weights, int* idx,
                                                   int E, int k, int normalize) {
   const int lane = threadIdx.x & 31;
@@ -191,62 +283,42 @@ __device__ __forceinline__ void warp_topk_softmax(const float* __restrict__ logi
     const int e = lane + j * 32;
     if (probs && e < E) probs[e] = v[j];
   }
-  float wsum = 0.f;
-  for (int s = 0; s < k; ++s) {
-    // arg-max over what is left: (value, lowest index) reduced across the warp
-    float best = -1.f;
-    int best_e = 0x7fffffff;
-#pragma unroll 4
-    for (int j = 0; j < per; ++j) {
-      const int e = lane + j * 32;
-      if (e < E && v[j] > best) {
-        best = v[j];
-        best_e = e;
-      }
-    }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-      const int oe = __shfl_xor_sync(0xffffffffu, best_e, o);
-      if (ob > best || (ob == best && oe < best_e)) {
-        best = ob;
-        best_e = oe;
-      }
-    }
-    if (lane == 0) {
-      weights[s] = best;
-      idx[s] = best_e;
-    }
-    wsum += best;
-    if ((best_e & 31) == lane) v[best_e >> 5] = -1.f;   // taken
-  }
-  __syncwarp();
+  const float wsum = warp_select(v, per, E, k, weights, idx);
   if (normalize && lane < k) weights[lane] /= fmaxf(wsum, 1e-9f);
 }
 
-__global__ void __launch_bounds__(128) moe_topk_softmax_kernel(const float* __restrict__ logits, float* __restrict__ probs,
-                                                              float* __restrict__ weights, int* __restrict__ idx, int T,
-                                                              int E, int k, int normalize) {
-  for (int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5); t < T; t += gridDim.x * (blockDim.x >> 5))
-    warp_topk_softmax(logits + static_cast<size_t>(t) * E, probs ? probs + static_cast<size_t>(t) * E : nullptr,
-                      weights + static_cast<size_t>(t) * k, idx + static_cast<size_t>(t) * k, E, k, normalize);
+// How a router turns logits into scores: groups == 0 is a softmax over all experts, else sigmoids within groups.
+struct RouterRule {
+  int normalize, groups, keep;
+};
+__device__ __forceinline__ void warp_topk(const float* logits, float* probs, float* weights, int* idx, int E, int k,
+                                          const RouterRule& r) {
+  if (r.groups == 0) warp_topk_softmax(logits, probs, weights, idx, E, k, r.normalize);
+  else warp_topk_groups(logits, weights, idx, E, k, r.normalize, r.groups, r.keep);
 }
 
-// Router of a decode batch in one launch (one CTA): softmax, top-k and the expert-sorted slot list.
+__global__ void __launch_bounds__(128) moe_topk_kernel(const float* __restrict__ logits, long long ld, float* __restrict__ probs,
+                                                       float* __restrict__ weights, int* __restrict__ idx, int T, int E, int k,
+                                                       RouterRule rule) {
+  for (int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5); t < T; t += gridDim.x * (blockDim.x >> 5))
+    warp_topk(logits + t * ld, probs ? probs + static_cast<size_t>(t) * E : nullptr, weights + static_cast<size_t>(t) * k,
+              idx + static_cast<size_t>(t) * k, E, k, rule);
+}
+
+// Router of a decode batch in one launch (one CTA): scores, top-k and the expert-sorted slot list.
 //   order [T * k]: slots sorted by expert, stable;  start / count [E]: every expert's run inside `order`
 constexpr int ROUTE_THREADS = 1024;
 constexpr int ROUTE_MAX_SLOTS = 2048;
-__global__ void __launch_bounds__(ROUTE_THREADS) moe_route_kernel(const float* __restrict__ logits,
+__global__ void __launch_bounds__(ROUTE_THREADS) moe_route_kernel(const float* __restrict__ logits, long long ld,
                                                                   float* __restrict__ weights, int* __restrict__ order,
                                                                   int* __restrict__ start, int* __restrict__ count, int T,
-                                                                  int E, int k, int normalize) {
+                                                                  int E, int k, RouterRule rule) {
   __shared__ int ids[ROUTE_MAX_SLOTS];
   __shared__ int first[1024 + 1];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = ROUTE_THREADS / 32;
   const int n = T * k;
   for (int t = warp; t < T; t += nw)
-    warp_topk_softmax(logits + static_cast<size_t>(t) * E, nullptr, weights + static_cast<size_t>(t) * k, ids + t * k, E, k,
-                      normalize);
+    warp_topk(logits + t * ld, nullptr, weights + static_cast<size_t>(t) * k, ids + t * k, E, k, rule);
   __syncthreads();
   for (int e = warp; e < E; e += nw) {
     int c = 0;
@@ -336,22 +408,34 @@ extern "C" int ts_moe_combine_dw(const void* dout, const void* y, const int* des
   return (int)cudaGetLastError();
 }
 
-// logits fp32 [T][E] -> probs fp32 [T][E], weights fp32 [T][k], idx int32 [T][k]
-extern "C" int ts_moe_topk_softmax(const float* logits, float* probs, float* weights, int* idx, int T, int E, int k,
-                                   int normalize, void* stream) {
-  if (T <= 0 || E <= 0 || E > 32 * ROUTER_MAX_PER_LANE || k <= 0 || k > 32 || k > E) return -10;
+static bool router_ok(int T, int E, int k, long long ld, int groups, int keep) {
+  if (T <= 0 || E <= 0 || E > 32 * ROUTER_MAX_PER_LANE || k <= 0 || k > 32 || k > E || ld < E) return false;
+  return groups == 0 || (groups > 0 && E % groups == 0 && keep > 0 && keep <= groups && k <= keep * (E / groups));
+}
+
+// logits fp32 [T][ld] -> probs fp32 [T][E] (softmax only, may be null), weights fp32 [T][k], idx int32 [T][k].
+// groups 0: softmax over the E experts; else sigmoid scores, the best `keep` of `groups` groups can be chosen.
+extern "C" int ts_moe_topk(const float* logits, long long ld, float* probs, float* weights, int* idx, int T, int E, int k,
+                           int normalize, int groups, int keep, void* stream) {
+  if (!router_ok(T, E, k, ld, groups, keep) || (probs && groups)) return -10;
   long long blocks = (T + 3) / 4;
   const long long cap = static_cast<long long>(sm_count()) * 16;
   if (blocks > cap) blocks = cap;
-  moe_topk_softmax_kernel<<<(unsigned)blocks, 128, 0, ST(stream)>>>(logits, probs, weights, idx, T, E, k, normalize);
+  moe_topk_kernel<<<(unsigned)blocks, 128, 0, ST(stream)>>>(logits, ld, probs, weights, idx, T, E, k,
+                                                            RouterRule{normalize, groups, keep});
   return (int)cudaGetLastError();
 }
+extern "C" int ts_moe_topk_softmax(const float* logits, float* probs, float* weights, int* idx, int T, int E, int k,
+                                   int normalize, void* stream) {
+  return ts_moe_topk(logits, E, probs, weights, idx, T, E, k, normalize, 0, 0, stream);
+}
 
-// Decode-sized router: logits fp32 [T][E] -> weights [T][k], order [T * k], start [E], count [E].
+// Decode-sized router: logits fp32 [T][ld] -> weights [T][k], order [T * k], start [E], count [E].
 extern "C" int ts_moe_route_max_slots() { return ROUTE_MAX_SLOTS; }
-extern "C" int ts_moe_route(const float* logits, float* weights, int* order, int* start, int* count, int T, int E, int k,
-                            int normalize, void* stream) {
-  if (T <= 0 || E <= 0 || E > 32 * ROUTER_MAX_PER_LANE || k <= 0 || k > 32 || k > E || T * k > ROUTE_MAX_SLOTS) return -10;
-  moe_route_kernel<<<1, ROUTE_THREADS, 0, ST(stream)>>>(logits, weights, order, start, count, T, E, k, normalize);
+extern "C" int ts_moe_route(const float* logits, long long ld, float* weights, int* order, int* start, int* count, int T, int E,
+                            int k, int normalize, int groups, int keep, void* stream) {
+  if (!router_ok(T, E, k, ld, groups, keep) || T * k > ROUTE_MAX_SLOTS) return -10;
+  moe_route_kernel<<<1, ROUTE_THREADS, 0, ST(stream)>>>(logits, ld, weights, order, start, count, T, E, k,
+                                                        RouterRule{normalize, groups, keep});
   return (int)cudaGetLastError();
 }

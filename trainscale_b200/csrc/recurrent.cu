@@ -30,7 +30,6 @@ __device__ __forceinline__ float silu(float x) { return x / (1.f + expf(-x)); }
 template <typename T> __device__ __forceinline__ float act_silu(float x) {
   return sizeof(T) == 2 ? __fdividef(x, 1.f + __expf(-x)) : silu(x);
 }
-__device__ __forceinline__ float sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 
 __device__ __forceinline__ uint64_t pack2(float lo, float hi) {

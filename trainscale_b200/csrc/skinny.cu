@@ -10,6 +10,9 @@
 //
 // Groups (grid.y) are the experts of a mixture (slots sorted by expert: order / start / count), the heads of a per-head
 // projection (every group takes all rows; A, W and out advance by a stride per group) or one dense matrix.
+//
+// Gated products (glu_act): the 16 weight rows of a tile are eight gate rows and the up rows of the same eight outputs, so
+// both halves of an output meet in the CTA that reduced them.  A result may be multiplied by the sigmoid of a gate operand.
 // `grouped_simt_kernel` computes the same for fp32 operands and for sizes the vector loads cannot take.
 #include "common.cuh"
 #include "host_common.h"
@@ -27,9 +30,11 @@ struct SkinnyParams {
   const int* count;            // [groups] rows of the group (nullptr: M)
   int a_div;                   // row of A = slot / a_div
   int M, N, K;
-  int act;                     // of common.cuh product_act (0: none)
+  int act;                     // of common.cuh product_act or glu_act (0: none)
   float act_cap;
   int out_fp32;
+  const void* gate;            // result *= sigmoid(gate[slot * gate_ld + g * gate_group + n]) (nullptr: none)
+  long long gate_ld, gate_group;
 };
 
 __device__ __forceinline__ void mma_bf16_16816(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3,
@@ -41,6 +46,19 @@ __device__ __forceinline__ void mma_bf16_16816(float (&c)[4], uint32_t a0, uint3
 }
 
 constexpr int SK_WARPS = 8;
+
+__device__ __forceinline__ float to_f32(float v) { return v; }
+__device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
+
+template <typename T>
+__device__ __forceinline__ void skinny_store(const SkinnyParams& p, int g, int slot, int n, float v) {
+  if (p.gate) v *= sigmoid(to_f32(reinterpret_cast<const T*>(p.gate)[slot * p.gate_ld + g * p.gate_group + n]));
+  const long long at = g * p.o_group + static_cast<long long>(slot) * p.ldo + n;
+  if (p.out_fp32) reinterpret_cast<float*>(p.out)[at] = v;
+  else reinterpret_cast<__nv_bfloat16*>(p.out)[at] = __float2bfloat16(v);
+}
+// weight row of the gate of output n (its up row is GLU_BLOCK below)
+__device__ __forceinline__ int glu_row(int n) { return n / GLU_BLOCK * (2 * GLU_BLOCK) + n % GLU_BLOCK; }
 
 __device__ __forceinline__ uint4 ld_stream(const void* p) {   // weights: read once, keep them out of L1
   uint4 v;
@@ -67,12 +85,14 @@ skinny_gemm_kernel(SkinnyParams p) {
   if (m_total == 0) return;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int gid = lane >> 2, tig = lane & 3;
-  const int n0 = (blockIdx.x * TILES + warp / KW) * 16, wk = warp % KW;
+  const bool glu = p.act >= ACT_FIRST_GLU;
+  const int tile0 = blockIdx.x * TILES + warp / KW, wk = warp % KW;
+  const int n0 = glu ? glu_row(tile0 * 8) : tile0 * 16, up = glu ? GLU_BLOCK : 8;      // first weight row, distance of the other half
   const __nv_bfloat16* A = reinterpret_cast<const __nv_bfloat16*>(p.A) + g * p.a_group;
   const __nv_bfloat16* W = reinterpret_cast<const __nv_bfloat16*>(p.W) + g * p.w_group;
-  const bool row0 = n0 + gid < p.N, row1 = n0 + gid + 8 < p.N;
+  const bool row0 = n0 + gid < p.N, row1 = n0 + gid + up < p.N;
   const __nv_bfloat16* w0 = W + (row0 ? n0 + gid : 0) * p.ldw + tig * 8;
-  const __nv_bfloat16* w1 = W + (row1 ? n0 + gid + 8 : 0) * p.ldw + tig * 8;
+  const __nv_bfloat16* w1 = W + (row1 ? n0 + gid + up : 0) * p.ldw + tig * 8;
   const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
 
   for (int base = 0; base < m_total; base += NT * 8) {
@@ -121,28 +141,30 @@ skinny_gemm_kernel(SkinnyParams p) {
       red[warp][gid + 8][t * 8 + tig * 2 + 1] = acc[t][3];
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < TILES * m * 16; i += SK_WARPS * 32) {
-      const int tile = TILES == 1 ? 0 : i / (m * 16), r = i - tile * m * 16;
-      const int tk = r >> 4, n = r & 15, nn = (blockIdx.x * TILES + tile) * 16 + n;
-      if (nn < p.N) {
+    const int lg = glu ? 3 : 4, n_out = glu ? p.N / 2 : p.N;       // outputs of a tile: 8 or 16
+    for (int i = threadIdx.x; i < TILES * m << lg; i += SK_WARPS * 32) {
+      const int tile = TILES == 1 ? 0 : i / (m << lg), r = i - tile * (m << lg);
+      const int tk = r >> lg, n = r & ((1 << lg) - 1), nn = ((blockIdx.x * TILES + tile) << lg) + n;
+      if (nn < n_out) {
         float v = 0.f;
 #pragma unroll
         for (int w = 0; w < KW; ++w) v += red[tile * KW + w][n][tk];
-        v = product_act(v, p.act, p.act_cap);
-        const int slot = p.order ? p.order[first + base + tk] : base + tk;
-        const long long at = g * p.o_group + static_cast<long long>(slot) * p.ldo + nn;
-        if (p.out_fp32) reinterpret_cast<float*>(p.out)[at] = v;
-        else reinterpret_cast<__nv_bfloat16*>(p.out)[at] = __float2bfloat16(v);
+        if (glu) {
+          float f = 0.f;
+#pragma unroll
+          for (int w = 0; w < KW; ++w) f += red[tile * KW + w][n + 8][tk];
+          v = glu_act<true>(v, f, p.act);
+        } else {
+          v = product_act(v, p.act, p.act_cap);
+        }
+        skinny_store<__nv_bfloat16>(p, g, p.order ? p.order[first + base + tk] : base + tk, nn, v);
       }
     }
     __syncthreads();
   }
 }
 
-__device__ __forceinline__ float to_f32(float v) { return v; }
-__device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
-
-// One warp per weight row, four token rows at a time, lanes split the reduction.  Any size, fp32 or bf16 operands.
+// One warp per weight row (gated: per pair of rows), four token rows at a time, lanes split the reduction.  Any size, fp32 or bf16 operands.
 template <typename T>
 __global__ void __launch_bounds__(256) grouped_simt_kernel(SkinnyParams p) {
   constexpr int TM = 4;
@@ -150,9 +172,11 @@ __global__ void __launch_bounds__(256) grouped_simt_kernel(SkinnyParams p) {
   const int n = blockIdx.x * 8 + warp;
   const int m_total = p.count ? p.count[g] : p.M;
   const int first = p.start ? p.start[g] : 0;
-  if (n >= p.N) return;
+  const bool glu = p.act >= ACT_FIRST_GLU;
+  if (n >= (glu ? p.N / 2 : p.N)) return;
   const T* A = reinterpret_cast<const T*>(p.A) + g * p.a_group;
-  const T* w = reinterpret_cast<const T*>(p.W) + g * p.w_group + n * p.ldw;
+  const T* w = reinterpret_cast<const T*>(p.W) + g * p.w_group + (glu ? glu_row(n) : n) * p.ldw;
+  const T* w_up = w + GLU_BLOCK * p.ldw;
   for (int base = blockIdx.z * TM; base < m_total; base += gridDim.z * TM) {
     const T* x[TM];
     int slot[TM];
@@ -162,20 +186,22 @@ __global__ void __launch_bounds__(256) grouped_simt_kernel(SkinnyParams p) {
       slot[t] = p.order ? p.order[first + i] : i;
       x[t] = A + static_cast<long long>(slot[t] / p.a_div) * p.lda;
     }
-    float acc[TM] = {0.f, 0.f, 0.f, 0.f};
+    float acc[TM] = {0.f, 0.f, 0.f, 0.f}, fac[TM] = {0.f, 0.f, 0.f, 0.f};
     for (int k = lane; k < p.K; k += 32) {
       const float wk = to_f32(w[k]);
 #pragma unroll
       for (int t = 0; t < TM; ++t) acc[t] += wk * to_f32(x[t][k]);
+      if (glu) {
+        const float uk = to_f32(w_up[k]);
+#pragma unroll
+        for (int t = 0; t < TM; ++t) fac[t] += uk * to_f32(x[t][k]);
+      }
     }
 #pragma unroll
     for (int t = 0; t < TM; ++t) {
-      const float v = product_act(warp_sum(acc[t]), p.act, p.act_cap);
-      if (lane == 0 && base + t < m_total) {
-        const long long at = g * p.o_group + static_cast<long long>(slot[t]) * p.ldo + n;
-        if (p.out_fp32) reinterpret_cast<float*>(p.out)[at] = v;
-        else reinterpret_cast<__nv_bfloat16*>(p.out)[at] = __float2bfloat16(v);
-      }
+      float v = warp_sum(acc[t]);
+      v = glu ? glu_act<false>(v, warp_sum(fac[t]), p.act) : product_act(v, p.act, p.act_cap);
+      if (lane == 0 && base + t < m_total) skinny_store<T>(p, g, slot[t], n, v);
     }
   }
 }
@@ -196,25 +222,31 @@ TS_DEFINE_ERROR_API(ts_skinny)
 using namespace ts;
 
 // M: rows of every group, or an upper bound of them when `count` is given (`typical`: how many a group usually has; more
-// take further passes over the weights, which then come from L2).  fp32: A and W are fp32 (else bf16).
+// take further passes over the weights, which then come from L2).  fp32: A and W are fp32 (else bf16).  Gated activations:
+// W has N rows in alternating blocks of GLU_BLOCK gate and up rows, the result N / 2 columns.  gate (of the type of A):
+// nullptr or a factor sigmoid(gate) of every result.
 extern "C" int ts_skinny_gemm(const void* A, const void* W, void* out, long long lda, long long ldw, long long ldo,
                               long long a_group, long long w_group, long long o_group, const int* order,
                               const int* start, const int* count, int a_div, int groups, int M, int N, int K, int act,
-                              float act_cap, int fp32, int out_fp32, int typical, void* stream) {
+                              float act_cap, int fp32, int out_fp32, int typical, const void* gate, long long gate_ld,
+                              long long gate_group, void* stream) {
   if (M <= 0 || groups <= 0) return 0;
-  if (N <= 0 || K <= 0 || a_div <= 0 || act < 0 || act > 3 || (act == 3 && !(act_cap > 0.f)) || groups > 65535) return -10;
+  if (N <= 0 || K <= 0 || a_div <= 0 || act < 0 || act > ACT_LAST_GLU || (act == 3 && !(act_cap > 0.f)) || groups > 65535)
+    return -10;
+  if (act >= ACT_FIRST_GLU && N % (2 * GLU_BLOCK)) return -12;
   if (fp32 && !out_fp32) return -11;
   SkinnyParams p;
   p.A = A; p.W = W; p.out = out; p.lda = lda; p.ldw = ldw; p.ldo = ldo; p.a_group = a_group; p.w_group = w_group;
   p.o_group = o_group; p.order = order; p.start = start; p.count = count; p.a_div = a_div; p.M = M; p.N = N; p.K = K;
-  p.act = act; p.act_cap = act_cap; p.out_fp32 = out_fp32;
+  p.act = act; p.act_cap = act_cap; p.out_fp32 = out_fp32; p.gate = gate; p.gate_ld = gate_ld; p.gate_group = gate_group;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   const bool vec = !fp32 && K % 8 == 0 && lda % 8 == 0 && ldw % 8 == 0 && a_group % 8 == 0 && w_group % 8 == 0 &&
                    aligned16(A) && aligned16(W);
   if (!vec) {
     int z = (M + 3) / 4;
     if (z > 64) z = 64;
-    const dim3 grid((N + 7) / 8, groups, z);
+    const int n_out = act >= ACT_FIRST_GLU ? N / 2 : N;
+    const dim3 grid((n_out + 7) / 8, groups, z);
     if (fp32) grouped_simt_kernel<float><<<grid, 256, 0, st>>>(p);
     else grouped_simt_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>(p);
     return (int)cudaGetLastError();

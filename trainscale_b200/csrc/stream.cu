@@ -16,6 +16,10 @@
 //   source        x' = x + y / sqrt(mean(y^2) + eps) * (1 + w), or x' = embed[token] * scale
 //   outputs       x' (fp32); x' in the activation type, or n token-shift mixes of it, x' + (x'_prev - x') * mu_s;
 //                 last boundary: x' normed once more with the final weight, only for the rows that are wanted
+//
+// `prenorm_kernel` is the boundary of decoders that norm a sublayer's INPUT:
+//   source        x' = x + y (* sigmoid(g), one number per row) + sum_j w_j * expert_j, or x' = embed[token]
+//   outputs       x' (fp32); h = x' / sqrt(mean(x'^2) + eps) * (1 + w); last boundary: h only, for the wanted rows
 #include "common.cuh"
 #include "host_common.h"
 
@@ -475,6 +479,129 @@ static int launch_postnorm(const PostnormParams& p, cudaStream_t st) {
   return -11;
 }
 
+struct PrenormParams {
+  const long long* tok;        // embedding source: [T]
+  const void* embed;           // [vocab][W]
+  int vocab;
+  const float* x_in;           // sublayer source: [T][W]
+  const void* y;               // [T][y_ld] or nullptr
+  long long y_ld;
+  const float* y_gate;         // logit of y's factor, stride y_gate_ld per row (nullptr: 1)
+  long long y_gate_ld;
+  const void* experts;         // expert outputs, W wide, or nullptr
+  const int* dest;             // [T * k] row of every routed slot (nullptr: the slot itself)
+  const float* route_w;        // [T * k]
+  int k;
+  const float* w;              // [W], around zero
+  float eps;
+  float* x_out;                // [T][W] (not for FINAL)
+  void* h;                     // [rows][W]
+  const int* rows;             // FINAL: the rows to produce
+  int W;
+};
+
+// grid: rows
+template <typename T, int MODE, int V, int NV>
+__global__ void __launch_bounds__(V == 4 ? 512 : 1024)
+prenorm_kernel(PrenormParams p) {
+  constexpr int AHEAD = NV == 1 ? 8 : (NV == 2 ? 4 : 2);      // expert rows in flight
+  __shared__ float scratch[32];
+  const int nvec = p.W / V, t = MODE == STREAM_FINAL ? p.rows[blockIdx.x] : blockIdx.x;
+  const size_t base = static_cast<size_t>(t) * p.W;
+  float v[NV][V];
+  if (MODE == STREAM_EMBED) {
+    long long tok = p.tok[t];
+    if (tok < 0 || tok >= p.vocab) {
+      if (threadIdx.x == 0) ts_report_error(ERR_BOUNDS, 8002, static_cast<unsigned int>(tok));
+      tok = 0;
+    }
+    const T* e = reinterpret_cast<const T*>(p.embed) + static_cast<size_t>(tok) * p.W;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c < nvec) VecIO<T>::template load<V>(e + c * V, v[i]);
+    }
+  } else {
+    const float f = p.y_gate ? sigmoid(p.y_gate[t * p.y_gate_ld]) : 1.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c < nvec) {
+        VecIO<float>::load<V>(p.x_in + base + c * V, v[i]);
+        if (p.y) {
+          float a[V];
+          VecIO<T>::template load<V>(reinterpret_cast<const T*>(p.y) + t * p.y_ld + c * V, a);
+#pragma unroll
+          for (int q = 0; q < V; ++q) v[i][q] += f * a[q];
+        }
+      }
+    }
+    if (p.experts) {
+#pragma unroll AHEAD
+      for (int j = 0; j < p.k; ++j) {
+        const int slot = t * p.k + j;
+        const float w = p.route_w[slot];
+        const T* src = reinterpret_cast<const T*>(p.experts) + static_cast<size_t>(p.dest ? p.dest[slot] : slot) * p.W;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+          const int c = threadIdx.x + i * blockDim.x;
+          if (c < nvec) {
+            float a[V];
+            VecIO<T>::template load<V>(src + c * V, a);
+#pragma unroll
+            for (int q = 0; q < V; ++q) v[i][q] += w * a[q];
+          }
+        }
+      }
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = threadIdx.x + i * blockDim.x;
+    if (c < nvec) {
+      if (MODE != STREAM_FINAL) VecIO<float>::store<V>(p.x_out + base + c * V, v[i]);
+#pragma unroll
+      for (int q = 0; q < V; ++q) ss += v[i][q] * v[i][q];
+    }
+  }
+  ss = block_sum(ss, scratch);
+  const float inv = 1.f / sqrtf(ss / static_cast<float>(p.W) + p.eps);
+  T* h = reinterpret_cast<T*>(p.h) + static_cast<size_t>(blockIdx.x) * p.W;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = threadIdx.x + i * blockDim.x;
+    if (c < nvec) {
+      float g[V];
+      VecIO<float>::load<V>(p.w + c * V, g);
+#pragma unroll
+      for (int q = 0; q < V; ++q) v[i][q] = v[i][q] * inv * (1.f + g[q]);
+      VecIO<T>::template store<V>(h + c * V, v[i]);
+    }
+  }
+}
+
+template <typename T, int MODE>
+static int launch_prenorm(const PrenormParams& p, int rows, cudaStream_t st) {
+  const bool vec = p.W % 4 == 0 && p.y_ld % 4 == 0;
+  const int nvec = vec ? p.W / 4 : p.W, cap = vec ? 512 : 1024;
+  int threads = (nvec + 31) / 32 * 32;
+  if (threads > cap) threads = cap;
+  const int nv = (nvec + threads - 1) / threads;
+  if (vec) {
+    if (nv <= 1) prenorm_kernel<T, MODE, 4, 1><<<rows, threads, 0, st>>>(p);
+    else if (nv <= 2) prenorm_kernel<T, MODE, 4, 2><<<rows, threads, 0, st>>>(p);
+    else if (nv <= 4) prenorm_kernel<T, MODE, 4, 4><<<rows, threads, 0, st>>>(p);
+    else if (nv <= 8) prenorm_kernel<T, MODE, 4, 8><<<rows, threads, 0, st>>>(p);
+    else return -11;
+  } else {
+    if (nv <= 1) prenorm_kernel<T, MODE, 1, 1><<<rows, threads, 0, st>>>(p);
+    else if (nv <= 8) prenorm_kernel<T, MODE, 1, 8><<<rows, threads, 0, st>>>(p);
+    else return -11;
+  }
+  return (int)cudaGetLastError();
+}
+
 }  // namespace ts
 
 TS_DEFINE_ERROR_API(ts_stream)
@@ -544,4 +671,24 @@ extern "C" int ts_stream_postnorm_final(const float* x_in, const void* y, long l
   p.n_rows = n_out; p.W = W;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   return fp32_act ? launch_postnorm<float, STREAM_FINAL>(p, st) : launch_postnorm<__nv_bfloat16, STREAM_FINAL>(p, st);
+}
+
+// Boundary of input-normed decoders.  `tok`: embedding source (then x_in, y and the experts are unused).  y_gate: logits of a
+// factor of y, one per row.  experts with dest (nullptr: slot order) and route_w [rows * k]: weighted sum of a row's slots.
+// `rows_list` (with n_out entries): last boundary - h of those rows only, nothing else is written.
+extern "C" int ts_stream_prenorm(const long long* tok, const void* embed, int vocab, const float* x_in, const void* y,
+                                 long long y_ld, const float* y_gate, long long y_gate_ld, const void* experts, const int* dest,
+                                 const float* route_w, int k, const float* w, float eps, float* x_out, void* h, int rows,
+                                 const int* rows_list, int n_out, int W, int fp32_act, void* stream) {
+  if (rows_list ? n_out <= 0 : rows <= 0) return 0;
+  if (W <= 0 || (experts && (k <= 0 || !route_w)) || (tok && rows_list)) return -10;
+  PrenormParams p = {};
+  p.tok = tok; p.embed = embed; p.vocab = vocab; p.x_in = x_in; p.y = y; p.y_ld = y_ld; p.y_gate = y_gate;
+  p.y_gate_ld = y_gate_ld; p.experts = experts; p.dest = dest; p.route_w = route_w; p.k = k; p.w = w; p.eps = eps;
+  p.x_out = x_out; p.h = h; p.rows = rows_list; p.W = W;
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  if (tok) return fp32_act ? launch_prenorm<float, STREAM_EMBED>(p, rows, st) : launch_prenorm<__nv_bfloat16, STREAM_EMBED>(p, rows, st);
+  if (rows_list)
+    return fp32_act ? launch_prenorm<float, STREAM_FINAL>(p, n_out, st) : launch_prenorm<__nv_bfloat16, STREAM_FINAL>(p, n_out, st);
+  return fp32_act ? launch_prenorm<float, STREAM_LAYER>(p, rows, st) : launch_prenorm<__nv_bfloat16, STREAM_LAYER>(p, rows, st);
 }

@@ -1,11 +1,15 @@
 // Sliding-window attention with grouped queries over a paged cache whose rows hold a token's keys and values side by side:
 // row = [G key heads x dim | G value heads x vdim | padding].
 //
+// Keys a position sees: itself and the `window` - 1 before it, or the part of its chunk of `window` positions up to itself
+// (chunks count from position 0); besides, the first `keep` positions of the sequence.
+//
 //   ts_window_angles  cosines and sines of a step's positions, shared by all layers with the same frequencies
-//   ts_window_prep    per-head RMS norm of queries and keys, rotary embedding of the first `rot` dimensions of a head
-//                     (in place in the projection), cache write of keys and values - one launch
+//   ts_window_prep    bias, per-head RMS norm of queries and keys, rotary embedding of the first `rot` dimensions of a head
+//                     (in place in the projection), cache write of keys and values - one launch.  Each step but the last
+//                     is optional; values can be the projected keys themselves
 //   ts_window_attend  single query rows (decoding, fp32, and head sizes the prefill kernel does not take) against the paged
-//                     cache: keys max(0, len - window) <= j < len of the row's sequence
+//                     cache; the result may be multiplied by the sigmoid of a gate per head or per element
 // Portions of prompts: ts_window_prefill (latent_prefill.cu).
 //
 // Decoding reads every cached key and value in the window once per key/value head.  `window_attend_mma_kernel` (bf16): the
@@ -29,24 +33,28 @@ __device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162flo
 struct WindowPrepParams {
   void* proj;                  // rows [H x dim | G x dim | G x vdim | ...]
   long long ld;
-  const float* q_norm;         // [dim]
+  const float* bias;           // [(H + G) x dim] or nullptr
+  const float* q_norm;         // [dim] or nullptr (no norms)
   const float* k_norm;
   float eps;
   const float* angles;         // [T][cos (rot / 2) | sin (rot / 2)]
   const long long* slots;
   void* cache;
   int T, H, G, dim, vdim, rot, row_width;
+  int h0;                      // first head that changes (H: queries stay as projected)
+  int pairs;                   // rotation partners: 0 coordinates i and i + rot / 2, 1 coordinates 2 i and 2 i + 1
+  int values_are_keys;         // values: the keys before norm and rotation, also written behind them in the projection
 };
 
 __global__ void window_angles_kernel(const float* __restrict__ inv_freq, const int* __restrict__ pos, float* __restrict__ out, int T,
-                                     int half) {
+                                     int half, float magnitude) {
   const int i = blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= T * half) return;
   const int t = i / half, f = i - t * half;
   float s, c;
   sincosf(static_cast<float>(pos[t]) * inv_freq[f], &s, &c);
-  out[static_cast<long long>(t) * 2 * half + f] = c;
-  out[static_cast<long long>(t) * 2 * half + half + f] = s;
+  out[static_cast<long long>(t) * 2 * half + f] = c * magnitude;
+  out[static_cast<long long>(t) * 2 * half + half + f] = s * magnitude;
 }
 
 constexpr int WP_WARPS = 8;
@@ -58,32 +66,47 @@ __global__ void __launch_bounds__(WP_WARPS * 32) window_prep_kernel(WindowPrepPa
   const float* cs = p.angles + static_cast<long long>(t) * p.rot;
   T* row = reinterpret_cast<T*>(p.proj) + t * p.ld;
   T* crow = reinterpret_cast<T*>(p.cache) + p.slots[t] * p.row_width;
-  const T* v = row + (p.H + p.G) * p.dim;
-  for (int c = threadIdx.x; c < p.row_width - p.G * p.dim; c += blockDim.x)
-    crow[p.G * p.dim + c] = c < p.G * p.vdim ? v[c] : from_f32<T>(0.f);
-  for (int h = warp; h < p.H + p.G; h += WP_WARPS) {
+  T* v = row + (p.H + p.G) * p.dim;
+  for (int c = threadIdx.x; c < p.row_width - p.G * p.dim; c += blockDim.x) {
+    if (c >= p.G * p.vdim) crow[p.G * p.dim + c] = from_f32<T>(0.f);
+    else if (!p.values_are_keys) crow[p.G * p.dim + c] = v[c];
+  }
+  for (int h = p.h0 + warp; h < p.H + p.G; h += WP_WARPS) {
     T* x = row + h * p.dim;
-    float ss = 0.f;
-    for (int c = lane; c < p.dim; c += 32) {
-      const float a = to_f32(x[c]);
-      ss += a * a;
-    }
-    ss = warp_sum(ss);
-    const float inv = 1.f / sqrtf(ss / static_cast<float>(p.dim) + p.eps);
+    const float* bias = p.bias ? p.bias + h * p.dim : nullptr;
+    auto value = [&](int c) { return to_f32(x[c]) + (bias ? bias[c] : 0.f); };
     const float* w = h < p.H ? p.q_norm : p.k_norm;
+    float inv = 1.f;
+    if (w) {
+      float ss = 0.f;
+      for (int c = lane; c < p.dim; c += 32) {
+        const float a = value(c);
+        ss += a * a;
+      }
+      ss = warp_sum(ss);
+      inv = 1.f / sqrtf(ss / static_cast<float>(p.dim) + p.eps);
+    }
+    auto normed = [&](int c) { return w ? value(c) * inv * w[c] : value(c); };
     T* out2 = h < p.H ? nullptr : crow + (h - p.H) * p.dim;
+    if (p.values_are_keys && h >= p.H)
+      for (int c = lane; c < p.dim; c += 32) {
+        const T y = from_f32<T>(value(c));
+        v[(h - p.H) * p.dim + c] = y;
+        crow[p.G * p.dim + (h - p.H) * p.dim + c] = y;
+      }
     for (int i = lane; i < half; i += 32) {
-      const float a = to_f32(x[i]) * inv * w[i], b = to_f32(x[i + half]) * inv * w[i + half];
+      const int c0 = p.pairs ? 2 * i : i, c1 = p.pairs ? 2 * i + 1 : i + half;
+      const float a = normed(c0), b = normed(c1);
       const T lo = from_f32<T>(a * cs[i] - b * cs[half + i]), hi = from_f32<T>(b * cs[i] + a * cs[half + i]);
-      x[i] = lo;
-      x[i + half] = hi;
+      x[c0] = lo;
+      x[c1] = hi;
       if (out2) {
-        out2[i] = lo;
-        out2[i + half] = hi;
+        out2[c0] = lo;
+        out2[c1] = hi;
       }
     }
     for (int c = p.rot + lane; c < p.dim; c += 32) {
-      const T y = from_f32<T>(to_f32(x[c]) * inv * w[c]);
+      const T y = from_f32<T>(normed(c));
       x[c] = y;
       if (out2) out2[c] = y;
     }
@@ -98,7 +121,8 @@ __global__ void __launch_bounds__(WP_WARPS * 32) window_prep_vec_kernel(WindowPr
   constexpr int HPW = 32 / LPH;
   __shared__ float swap[WP_WARPS][HPW][LPH * 8];
   const int half = p.rot / 2, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int head_items = (p.H + p.G + HPW - 1) / HPW, per_token = head_items + (p.G * p.vdim / 8 + 31) / 32;
+  const int head_items = (p.H + p.G - p.h0 + HPW - 1) / HPW;
+  const int per_token = head_items + (p.values_are_keys ? 0 : (p.G * p.vdim / 8 + 31) / 32);
   const unsigned item = blockIdx.x * WP_WARPS + warp;
   const int t = item / per_token, part = item - t * per_token;
   if (t >= p.T) return;
@@ -110,7 +134,7 @@ __global__ void __launch_bounds__(WP_WARPS * 32) window_prep_vec_kernel(WindowPr
       reinterpret_cast<uint4*>(crow + p.G * p.dim)[c] = reinterpret_cast<const uint4*>(row + (p.H + p.G) * p.dim)[c];
     return;
   }
-  const int sub = lane % LPH, slot = lane / LPH, h = part * HPW + slot, c0 = sub * 8;
+  const int sub = lane % LPH, slot = lane / LPH, h = p.h0 + part * HPW + slot, c0 = sub * 8;
   const bool on = c0 < p.dim && h < p.H + p.G;
   __nv_bfloat16* x = row + h * p.dim + c0;
   float a[8];
@@ -125,19 +149,45 @@ __global__ void __launch_bounds__(WP_WARPS * 32) window_prep_vec_kernel(WindowPr
       const float2 f = unpack_bf16x2(r[j]);
       a[2 * j] = f.x;
       a[2 * j + 1] = f.y;
-      ss += f.x * f.x + f.y * f.y;
+    }
+    if (p.bias) {
+      const float* b = p.bias + h * p.dim + c0;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) a[j] += b[j];
+    }
+#pragma unroll
+    for (int j = 0; j < 8; ++j) ss += a[j] * a[j];
+    if (p.values_are_keys && h >= p.H) {
+      const uint4 o = make_uint4(pack_bf16x2(a[0], a[1]), pack_bf16x2(a[2], a[3]), pack_bf16x2(a[4], a[5]), pack_bf16x2(a[6], a[7]));
+      const int at = (h - p.H) * p.dim + c0;
+      *reinterpret_cast<uint4*>(row + (p.H + p.G) * p.dim + at) = o;
+      *reinterpret_cast<uint4*>(crow + p.G * p.dim + at) = o;
     }
   }
-  const float* w = (h < p.H ? p.q_norm : p.k_norm) + c0;
   const float* cs = p.angles + static_cast<long long>(t) * p.rot;
+  if (p.q_norm) {
+    const float* w = (h < p.H ? p.q_norm : p.k_norm) + c0;
 #pragma unroll
-  for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-  const float inv = 1.f / sqrtf(ss / static_cast<float>(p.dim) + p.eps);
-  if (on) {
+    for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const float inv = 1.f / sqrtf(ss / static_cast<float>(p.dim) + p.eps);
+    if (on) {
 #pragma unroll
-    for (int j = 0; j < 8; ++j) a[j] *= inv * w[j];
+      for (int j = 0; j < 8; ++j) a[j] *= inv * w[j];
+    }
   }
-  if (half % 8 == 0 && p.rot > 0) {
+  if (p.pairs) {
+    if (on) {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int f = c0 / 2 + j;
+        if (f < half) {
+          const float c = cs[f], s = cs[half + f], u = a[2 * j], v = a[2 * j + 1];
+          a[2 * j] = u * c - v * s;
+          a[2 * j + 1] = v * c + u * s;
+        }
+      }
+    }
+  } else if (half % 8 == 0 && p.rot > 0) {
     const bool first = c0 < half, rotated = c0 < p.rot;
     const int other = slot * LPH + (first ? sub + half / 8 : (rotated ? sub - half / 8 : sub)), f0 = first ? c0 : c0 - half;
 #pragma unroll
@@ -183,9 +233,29 @@ struct WindowAttendParams {
   long long out_ld;
   float* part_out;             // [rows][H][splits][vdim]
   float* part_lse;             // [rows][H][splits]
-  int rows, H, G, dim, vdim, row_width, max_blocks, block_size, window, chunk, splits;
+  const void* gate;            // result *= sigmoid(gate), type of q: rows [gate_ld], see gate_mode (nullptr: none)
+  long long gate_ld;
+  int gate_mode;               // GATE_HEAD: column h, GATE_ELEMENT: column h * vdim + c
+  int rows, H, G, dim, vdim, row_width, max_blocks, block_size, window, keep, chunked, chunk, splits;
   float scale, o_scale;
 };
+
+// A row's visible keys, numbered 0 .. count - 1 in key order: the kept first positions, then those from `lo` on.
+struct VisibleKeys {
+  int lo, kept, count;
+  __device__ VisibleKeys(const WindowAttendParams& p, int len) {
+    lo = p.chunked ? (len - 1) / p.window * p.window : max(0, len - p.window);
+    kept = min(p.keep, lo);
+    count = len - lo + kept;
+  }
+  __device__ int position(int i) const { return i < kept ? i : i - kept + lo; }
+};
+
+template <typename T> __device__ __forceinline__ float gate_factor(const WindowAttendParams& p, int row, int h, int c) {
+  if (!p.gate) return 1.f;
+  const int col = p.gate_mode == GATE_HEAD ? h : h * p.vdim + c;
+  return sigmoid(to_f32(reinterpret_cast<const T*>(p.gate)[row * p.gate_ld + col]));
+}
 
 constexpr int WS_CHUNK = 512;
 
@@ -206,12 +276,17 @@ __global__ void __launch_bounds__(128) window_attend_simt_kernel(WindowAttendPar
   for (int i = threadIdx.x; i < p.dim; i += blockDim.x) qs[i] = to_f32(q[i]);
   for (int i = threadIdx.x; i < p.vdim; i += blockDim.x) acc[i] = 0.f;
   float m = -INFINITY, l = 0.f;
-  for (int j0 = max(0, len - p.window); j0 < len; j0 += WS_CHUNK) {
-    const int j1 = min(len, j0 + WS_CHUNK);
+  const VisibleKeys vis(p, len);
+  auto key_row = [&](int i) {
+    const int j = vis.position(i);
+    return cache + (static_cast<long long>(bt[j / p.block_size]) * p.block_size + j % p.block_size) * p.row_width;
+  };
+  for (int j0 = 0; j0 < vis.count; j0 += WS_CHUNK) {
+    const int j1 = min(vis.count, j0 + WS_CHUNK);
     __syncthreads();
     float mx = -INFINITY;
     for (int j = j0 + warp; j < j1; j += nw) {
-      const T* c = cache + (static_cast<long long>(bt[j / p.block_size]) * p.block_size + j % p.block_size) * p.row_width + g * p.dim;
+      const T* c = key_row(j) + g * p.dim;
       float s = 0.f;
       for (int i = lane; i < p.dim; i += 32) s += qs[i] * to_f32(c[i]);
       s = warp_sum(s) * p.scale;
@@ -230,15 +305,13 @@ __global__ void __launch_bounds__(128) window_attend_simt_kernel(WindowAttendPar
     m = m_new;
     for (int r = threadIdx.x; r < p.vdim; r += blockDim.x) {
       float a = acc[r] * alpha;
-      for (int j = j0; j < j1; ++j)
-        a += sc[j - j0] * to_f32(cache[(static_cast<long long>(bt[j / p.block_size]) * p.block_size + j % p.block_size) * p.row_width +
-                                       p.G * p.dim + g * p.vdim + r]);
+      for (int j = j0; j < j1; ++j) a += sc[j - j0] * to_f32(key_row(j)[p.G * p.dim + g * p.vdim + r]);
       acc[r] = a;
     }
   }
   const float inv = l > 0.f ? p.o_scale / l : 0.f;
   T* out = reinterpret_cast<T*>(p.out) + row * p.out_ld + h * p.vdim;
-  for (int r = threadIdx.x; r < p.vdim; r += blockDim.x) out[r] = from_f32<T>(acc[r] * inv);
+  for (int r = threadIdx.x; r < p.vdim; r += blockDim.x) out[r] = from_f32<T>(acc[r] * inv * gate_factor<T>(p, row, h, r));
 }
 
 constexpr int WA_WARPS = 4;
@@ -289,8 +362,8 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attend_mma_kernel(Window
   const int nh = min(16, (g + 1) * group - h0);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
   const int len = p.row_len[row];
-  const int lo = max(0, len - p.window);
-  const int j0 = lo + split * p.chunk, j1 = min(len, j0 + p.chunk);
+  const VisibleKeys vis(p, len);
+  const int j0 = split * p.chunk, j1 = min(vis.count, j0 + p.chunk);       // this CTA's share of them
   const int* bt = p.block_table + static_cast<long long>(p.row_seq[row]) * p.max_blocks;
   const __nv_bfloat16* kc = reinterpret_cast<const __nv_bfloat16*>(p.cache) + g * p.dim;
   const __nv_bfloat16* vc = reinterpret_cast<const __nv_bfloat16*>(p.cache) + p.G * p.dim + g * p.vdim;
@@ -304,11 +377,11 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attend_mma_kernel(Window
     }
   }
   __nv_bfloat16* mine = ring + warp * WA_STAGES * WA_KT * (kst + vst);
-  // this warp's tiles: keys t * 16 .. + 15 (absolute positions) for t = t_first + warp, + 4, ...
+  // this warp's tiles: visible keys t * 16 .. + 15 for t = t_first + warp, + 4, ... (a chunk is whole tiles)
   const int t_first = j0 / WA_KT, t_end = j1 > j0 ? (j1 + WA_KT - 1) / WA_KT : t_first;
   auto slot_of = [&](int tile) {         // cache row of key tile * 16 + lane % 16 (-1: outside the range)
-    const int j = tile * WA_KT + (lane & 15);
-    return tile < t_end && j >= j0 && j < j1 ? bt[j / p.block_size] * p.block_size + j % p.block_size : -1;
+    const int i = tile * WA_KT + (lane & 15), j = vis.position(i);
+    return tile < t_end && i < j1 ? bt[j / p.block_size] * p.block_size + j % p.block_size : -1;
   };
   auto load = [&](int stage, int slot) {
     const uint32_t kd = smem_u32(mine + stage * WA_KT * (kst + vst)), vd = kd + WA_KT * kst * 2;
@@ -367,7 +440,7 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attend_mma_kernel(Window
         mma_16816(s1, qf[k], b[2], b[3]);
       }
     const int j = t * WA_KT + tig * 2;
-    auto keep = [&](float v, int key) { return key >= j0 && key < j1 ? v * sl : -INFINITY; };
+    auto keep = [&](float v, int key) { return key < j1 ? v * sl : -INFINITY; };
     s0[0] = keep(s0[0], j); s0[1] = keep(s0[1], j + 1); s0[2] = keep(s0[2], j); s0[3] = keep(s0[3], j + 1);
     s1[0] = keep(s1[0], j + 8); s1[1] = keep(s1[1], j + 9); s1[2] = keep(s1[2], j + 8); s1[3] = keep(s1[3], j + 9);
     float a = fmaxf(fmaxf(s0[0], s0[1]), fmaxf(s1[0], s1[1])), b = fmaxf(fmaxf(s0[2], s0[3]), fmaxf(s1[2], s1[3]));
@@ -445,7 +518,8 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attend_mma_kernel(Window
     }
     const int h = h0 + r;
     if (p.splits == 1) {
-      reinterpret_cast<__nv_bfloat16*>(p.out)[row * p.out_ld + h * p.vdim + c] = __float2bfloat16(l > 0.f ? acc * (p.o_scale / l) : 0.f);
+      reinterpret_cast<__nv_bfloat16*>(p.out)[row * p.out_ld + h * p.vdim + c] =
+          __float2bfloat16(l > 0.f ? acc * (p.o_scale / l) * gate_factor<__nv_bfloat16>(p, row, h, c) : 0.f);
     } else {
       const long long at = (static_cast<long long>(row) * p.H + h) * p.splits + split;
       p.part_out[at * p.vdim + c] = l > 0.f ? acc / l : 0.f;
@@ -464,7 +538,8 @@ __global__ void __launch_bounds__(128) window_merge_kernel(WindowAttendParams p)
   for (int c = threadIdx.x; c < p.vdim; c += blockDim.x) {
     float acc = 0.f;
     for (int s = 0; s < p.splits; ++s) acc += fast_ex2(p.part_lse[base + s] - mm) * p.part_out[(base + s) * p.vdim + c];
-    reinterpret_cast<__nv_bfloat16*>(p.out)[row * p.out_ld + h * p.vdim + c] = __float2bfloat16(acc * (p.o_scale / l));
+    reinterpret_cast<__nv_bfloat16*>(p.out)[row * p.out_ld + h * p.vdim + c] =
+        __float2bfloat16(acc * (p.o_scale / l) * gate_factor<__nv_bfloat16>(p, row, h, c));
   }
 }
 
@@ -491,20 +566,25 @@ TS_DEFINE_ERROR_API(ts_window)
 using namespace ts;
 #define ST(s) reinterpret_cast<cudaStream_t>(s)
 
-// out: [T][cos | sin of pos * inv_freq], half frequencies.
-extern "C" int ts_window_angles(const float* inv_freq, const int* pos, float* out, int T, int half, void* stream) {
+// out: [T][cos | sin of pos * inv_freq], both times `magnitude`, half frequencies.
+extern "C" int ts_window_angles(const float* inv_freq, const int* pos, float* out, int T, int half, float magnitude,
+                                void* stream) {
   if (T <= 0 || half <= 0) return 0;
-  window_angles_kernel<<<(T * half + 255) / 256, 256, 0, ST(stream)>>>(inv_freq, pos, out, T, half);
+  window_angles_kernel<<<(T * half + 255) / 256, 256, 0, ST(stream)>>>(inv_freq, pos, out, T, half, magnitude);
   return (int)cudaGetLastError();
 }
 
-// angles: of ts_window_angles (unused without rotated dimensions).
-extern "C" int ts_window_prep(void* proj, long long ld, const float* q_norm, const float* k_norm, float eps,
+// angles: of ts_window_angles (unused without rotated dimensions).  bias, norms: nullptr for none (both norms or neither).
+// pairs: rotation partners are neighbours.  values_are_keys: the projection has no values, its columns behind the keys
+// receive the keys before norm and rotation.
+extern "C" int ts_window_prep(void* proj, long long ld, const float* bias, const float* q_norm, const float* k_norm, float eps,
                               const float* angles, const long long* slots, void* cache, int T, int H, int G, int dim, int vdim,
-                              int rot, int row_width, int fp32, void* stream) {
+                              int rot, int pairs, int values_are_keys, int row_width, int fp32, void* stream) {
   if (T <= 0) return 0;
   if (H <= 0 || G <= 0 || dim <= 0 || vdim <= 0 || rot < 0 || rot > dim || rot % 2 || row_width < G * (dim + vdim)) return -10;
+  if ((q_norm == nullptr) != (k_norm == nullptr) || (values_are_keys && dim != vdim)) return -10;
   WindowPrepParams p;
+  p.bias = bias; p.pairs = pairs; p.values_are_keys = values_are_keys; p.h0 = bias || q_norm || rot ? 0 : H;
   p.proj = proj; p.ld = ld; p.q_norm = q_norm; p.k_norm = k_norm; p.eps = eps; p.angles = angles; p.slots = slots;
   p.cache = cache; p.T = T; p.H = H; p.G = G; p.dim = dim; p.vdim = vdim; p.rot = rot; p.row_width = row_width;
   const bool vec = !fp32 && dim % 8 == 0 && vdim % 8 == 0 && dim <= 256 && ld % 8 == 0 && row_width == G * (dim + vdim) &&
@@ -512,7 +592,8 @@ extern "C" int ts_window_prep(void* proj, long long ld, const float* q_norm, con
   if (vec) {
     int lph = 4;
     while (lph * 8 < dim) lph *= 2;
-    const int hpw = 32 / lph, per_token = (H + G + hpw - 1) / hpw + (G * vdim / 8 + 31) / 32;
+    const int hpw = 32 / lph;
+    const int per_token = (H + G - p.h0 + hpw - 1) / hpw + (values_are_keys ? 0 : (G * vdim / 8 + 31) / 32);
     const unsigned grid = (unsigned)((static_cast<long long>(T) * per_token + WP_WARPS - 1) / WP_WARPS);
     if (lph == 4) window_prep_vec_kernel<4><<<grid, WP_WARPS * 32, 0, ST(stream)>>>(p);
     else if (lph == 8) window_prep_vec_kernel<8><<<grid, WP_WARPS * 32, 0, ST(stream)>>>(p);
@@ -535,18 +616,21 @@ extern "C" int ts_window_splits(int rows, int H, int G, int dim, int vdim, int k
   return s < 1 ? 1 : s;
 }
 
-// `keys`: upper bound of the keys a row sees; `splits` of ts_window_splits with the workspaces it needs (splits > 1).
+// window, keep, chunked: which keys a row sees (above).  `keys`: upper bound of their number; `splits` of ts_window_splits with the workspaces it needs (splits > 1).
 extern "C" int ts_window_attend(const void* q, long long q_ld, const void* cache, const int* block_table, int max_blocks,
                                 const int* row_seq, const int* row_len, void* out, long long out_ld, float* part_out,
                                 float* part_lse, int rows, int H, int G, int dim, int vdim, int row_width, int block_size,
-                                int window, int keys, int splits, float scale, float o_scale, int fp32, void* stream) {
+                                int window, int keep, int chunked, int keys, int splits, float scale, float o_scale,
+                                const void* gate, long long gate_ld, int gate_mode, int fp32, void* stream) {
   if (rows <= 0) return 0;
-  if (H <= 0 || G <= 0 || H % G || dim <= 0 || vdim <= 0 || window <= 0 || keys <= 0 || splits < 1 || splits > WM_MAX_SPLITS)
+  if (H <= 0 || G <= 0 || H % G || dim <= 0 || vdim <= 0 || window <= 0 || keep < 0 || keys <= 0 || splits < 1 ||
+      splits > WM_MAX_SPLITS)
     return -10;
   WindowAttendParams p;
   p.q = q; p.q_ld = q_ld; p.cache = cache; p.block_table = block_table; p.row_seq = row_seq; p.row_len = row_len; p.out = out;
   p.out_ld = out_ld; p.part_out = part_out; p.part_lse = part_lse; p.rows = rows; p.H = H; p.G = G; p.dim = dim;
   p.vdim = vdim; p.row_width = row_width; p.max_blocks = max_blocks; p.block_size = block_size; p.window = window;
+  p.keep = keep; p.chunked = chunked; p.gate = gate; p.gate_ld = gate_ld; p.gate_mode = gate_mode;
   p.splits = splits; p.chunk = ((keys + splits - 1) / splits + 15) / 16 * 16; p.scale = scale; p.o_scale = o_scale;
   const bool vec = window_mma_ok(dim, vdim, fp32) && scale > 0.f && q_ld % 8 == 0 && row_width % 8 == 0 &&
                    (reinterpret_cast<uintptr_t>(q) & 15u) == 0 && (reinterpret_cast<uintptr_t>(cache) & 15u) == 0;

@@ -6,6 +6,7 @@ from dataclasses import dataclass, field
 
 import torch
 
+from ..ops.masks import KeyMask
 from ..ops.stream import ROW_BEFORE
 from .kv_cache import PagedKVCache
 
@@ -25,7 +26,7 @@ class StepEntry:
 
 @dataclass
 class PromptContext:
-    """Keys of the batch's multi-token entries for one window size: the sequences' rows in key order."""
+    """Keys of the batch's multi-token entries for one mask: the sequences' rows in key order."""
     cu_q: torch.Tensor            # int32 [n + 1], query rows (relative to the first multi-token row)
     cu_k: torch.Tensor            # int32 [n + 1], key rows
     max_q: int
@@ -160,25 +161,26 @@ class StepBatch:
             self._contexts["portions"] = Portions(at, torch.tensor(at, dtype=torch.int32).to(self.token_ids.device))
         return self._contexts["portions"]
 
-    def prompt_context(self, window: int) -> PromptContext | None:
-        """Key rows of the multi-token entries when a position sees `window` keys (None: no such entries)."""
+    def prompt_context(self, mask: KeyMask) -> PromptContext | None:
+        """Key rows that the multi-token entries see through `mask` (None: no such entries)."""
         if self.host is None or self.host.all_single:
             return None
-        if window not in self._contexts:
+        if mask not in self._contexts:
             h = self.host
             first = h.n_single          # entries and rows before it are single tokens
             cu_q, cu_k, slots = [0], [0], []
             fresh = all(s == 0 for s in h.starts[first:])
             bs = h.cache.block_size
             for sid, start, n in zip(h.seq_ids[first:], h.starts[first:], h.q_lens[first:]):
-                lo = max(0, start - (window - 1))
+                lo = mask.first(start)
+                kept = min(mask.keep, lo)
                 cu_q.append(cu_q[-1] + n)
-                cu_k.append(cu_k[-1] + start + n - lo)
+                cu_k.append(cu_k[-1] + kept + start + n - lo)
                 if not fresh:
-                    j = torch.arange(lo, start + n)
+                    j = torch.cat([torch.arange(kept), torch.arange(lo, start + n)])
                     slots.append(torch.tensor(h.cache.seqs[sid].blocks)[j // bs] * bs + j % bs)
             dev = self.token_ids.device
             cu = torch.tensor(cu_q + cu_k, dtype=torch.int32).to(dev)
-            self._contexts[window] = PromptContext(cu[:len(cu_q)], cu[len(cu_q):], max(h.q_lens[first:]),
-                                                   None if fresh else torch.cat(slots).to(dev))
-        return self._contexts[window]
+            self._contexts[mask] = PromptContext(cu[:len(cu_q)], cu[len(cu_q):], max(h.q_lens[first:]),
+                                                 None if fresh else torch.cat(slots).to(dev))
+        return self._contexts[mask]

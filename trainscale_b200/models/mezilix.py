@@ -153,7 +153,7 @@ class MezilixLayer(nn.Module):
             w_uv = self.w_kv[m.heads * m.dim:].view(m.heads, m.vdim, m.rank)
             grouped.head_linear(o, w_uv, out[:nd].view(nd, m.heads, m.vdim))
         if nd < T:
-            ctx = batch.prompt_context(m.window)
+            ctx = batch.prompt_context(m.mask)
             rows = flat[nd:] if ctx.slots is None else latent.gather_rows(cache, ctx.slots)
             kv = gemm.matmul_nt(rows[:, :m.rank], self.w_kv)
             latent.attend_expanded(proj[nd:], kv, rows, m, ctx.cu_q, ctx.cu_k, ctx.max_q, out[nd:])

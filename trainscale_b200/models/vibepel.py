@@ -242,7 +242,7 @@ class ParallelMixer(nn.Module):
             window.attend_rows(proj[:nd], s, cache, batch.block_table, batch.row_seq[:nd], ctx.row_len[:nd], batch.max_len, out[:nd],
                                self.cfg.left_scale)
         if nd < T:
-            keys = batch.prompt_context(s.window)
+            keys = batch.prompt_context(s.mask)
             rows = None if keys.slots is None else latent.gather_rows(cache, keys.slots)
             window.attend_portions(proj[nd:], s, rows, keys.cu_q, keys.cu_k, keys.max_q, out[nd:], self.cfg.left_scale)
 

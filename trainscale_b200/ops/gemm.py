@@ -217,7 +217,7 @@ def few_rows(M: int, N: int, K: int) -> bool:
 def serve_linear(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None = None, act: int = 0, cap: float = 0.0,
                  out: torch.Tensor | None = None) -> torch.Tensor:
     """act(x [M, K] @ w [N, K]^T) for serving (no autograd), optionally with an fp32 result; `act` of ops/grouped (`cap`:
-    constant of the soft cap).  bf16 on the GPU: few rows go to the few-row kernel, more to the tcgen05 GEMM, the
+    constant of the soft cap; a gated act takes a packed weight and halves the columns).  bf16 on the GPU: few rows go to the few-row kernel, more to the tcgen05 GEMM, the
     activation in the epilogue of either; rows that are not whole 16-byte vectors, and fp32, to the library."""
     from . import grouped
     out_dtype = out.dtype if out is not None else out_dtype or x.dtype
@@ -227,7 +227,7 @@ def serve_linear(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None
         return grouped.rows_linear(x, w, out_dtype, act, cap, out)
     if vec:
         if out is None:
-            out = torch.empty(x.shape[0], w.shape[0], dtype=out_dtype, device=x.device)
+            out = torch.empty(x.shape[0], w.shape[0] // (2 if grouped.is_gated(act) else 1), dtype=out_dtype, device=x.device)
         gemm_raw(x, w, out, x.shape[0], w.shape[0], x.shape[1], x.stride(0), w.stride(0), out.stride(0), False, False,
                  act=act, cap=cap)
         return out

@@ -17,6 +17,7 @@ from dataclasses import dataclass
 import torch
 
 from . import _lib
+from .masks import KeyMask
 
 _ll, _f = ctypes.c_longlong, ctypes.c_float
 
@@ -32,10 +33,16 @@ class LatentShape:
     window: int           # keys a position sees: itself and window - 1 before it
     scale: float
     rope_base: float
+    pairs: bool = False   # rotation partners: coordinates 2 i and 2 i + 1 instead of i and i + rot / 2
+    magnitude: float = 1.0  # factor of cos and sin
 
     @property
     def q_width(self) -> int:
         return self.heads * (self.dim + self.rot)
+
+    @property
+    def mask(self) -> KeyMask:
+        return KeyMask(self.window)
 
     @property
     def row_width(self) -> int:
@@ -48,34 +55,46 @@ def expanded_supported(s: LatentShape) -> bool:
     return s.scale > 0 and s.rank % 8 == 0 and bool(_lib.load("latent_prefill").ts_latent_prefill_supported(s.dim, s.rot, s.vdim))
 
 
-def _rotate(x: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor) -> torch.Tensor:
+def _rotate(x: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor, pairs: bool) -> torch.Tensor:
+    if pairs:
+        u, v = x[..., 0::2].float(), x[..., 1::2].float()
+        return torch.stack([u * cos - v * sin, v * cos + u * sin], dim=-1).flatten(-2).to(x.dtype)
     half = x.shape[-1] // 2
     u, v = x[..., :half].float(), x[..., half:].float()
     return torch.cat([u * cos - v * sin, v * cos + u * sin], dim=-1).to(x.dtype)
 
 
 def prepare(proj: torch.Tensor, s: LatentShape, norm_w, eps: float, inv_freq, pos, slots, cache, keep_rows: bool):
-    """proj [T, q_width + rank + rot] = (queries | latent | shared key part).  Rotates the queries in place, writes the
+    """proj [T, >= q_width + rank + rot] = (queries | latent | shared key part | ...).  Rotates the queries in place, writes the
     normed latent and the rotated key part to cache rows `slots`; returns those rows [T, row_width] if `keep_rows`."""
     T = proj.shape[0]
     if not proj.is_cuda:
         ang = pos.float()[:, None] * inv_freq
-        cos, sin = ang.cos(), ang.sin()
+        cos, sin = ang.cos() * s.magnitude, ang.sin() * s.magnitude
         q = proj[:, :s.q_width].view(T, s.heads, s.dim + s.rot)
-        q[..., s.dim:] = _rotate(q[..., s.dim:], cos[:, None], sin[:, None])
+        q[..., s.dim:] = _rotate(q[..., s.dim:], cos[:, None], sin[:, None], s.pairs)
         c = proj[:, s.q_width:s.q_width + s.rank].float()
         rows = torch.zeros(T, s.row_width, dtype=proj.dtype)
         rows[:, :s.rank] = (c / torch.sqrt(c.pow(2).mean(-1, keepdim=True) + eps) * norm_w).to(proj.dtype)
-        rows[:, s.rank:s.rank + s.rot] = _rotate(proj[:, s.q_width + s.rank:], cos, sin)
+        rows[:, s.rank:s.rank + s.rot] = _rotate(proj[:, s.q_width + s.rank:s.q_width + s.rank + s.rot], cos, sin, s.pairs)
         cache.view(-1, s.row_width)[slots] = rows
         return rows if keep_rows else None
     flat = torch.empty(T, s.row_width, dtype=proj.dtype, device=proj.device) if keep_rows else None
     rc = _lib.load("latent").ts_latent_prep(
         _lib.ptr(proj), _ll(proj.stride(0)), s.heads, s.dim, s.rot, s.rank, _lib.ptr(norm_w), _f(eps), _lib.ptr(inv_freq),
-        _lib.ptr(pos), _lib.ptr(slots), _lib.ptr(cache), _lib.ptr(flat), s.row_width, T, int(proj.dtype == torch.float32),
+        _f(s.magnitude), int(s.pairs), _lib.ptr(pos), _lib.ptr(slots), _lib.ptr(cache), _lib.ptr(flat), s.row_width, T, int(proj.dtype == torch.float32),
         _lib.stream_ptr())
     _lib.check(rc, "ts_latent_prep")
     return flat
+
+
+def gate_args(gate: torch.Tensor | None, heads: int, vdim: int, like: torch.Tensor):
+    """Kernel arguments (pointer, row stride, mode) of an attention gate with one column per head or per element."""
+    if gate is None:
+        return _lib.ptr(None), _ll(0), 0
+    if gate.dtype != like.dtype or gate.stride(1) != 1 or gate.shape[1] not in (heads, heads * vdim):
+        raise ValueError("a gate has one contiguous column per head or per element, in the type of the queries")
+    return _lib.ptr(gate), _ll(gate.stride(0)), 2 if gate.shape[1] == heads * vdim and vdim > 1 else 1
 
 
 def gather_rows(cache: torch.Tensor, slots: torch.Tensor) -> torch.Tensor:
@@ -123,13 +142,14 @@ def attend_latent(q_lat: torch.Tensor, proj: torch.Tensor, s: LatentShape, cache
 
 
 def attend_expanded(proj: torch.Tensor, kv: torch.Tensor, rows: torch.Tensor, s: LatentShape, cu_q, cu_k, max_q: int,
-                    out: torch.Tensor) -> None:
+                    out: torch.Tensor, gate: torch.Tensor | None = None) -> None:
     """proj [Tq, ...] with the queries; kv [Tk, H * dim + H * vdim] expanded keys | values of the latent rows `rows`
     [Tk, row_width]; cu_q / cu_k int32 offsets of every sequence (its queries are the last of its keys).  Writes
-    out [Tq, H * vdim]."""
+    out [Tq, H * vdim], times sigmoid(gate) when there is a gate [Tq, H * vdim] or (one per head) [Tq, H]."""
+    gp, gld, mode = gate_args(gate, s.heads, s.vdim, proj)
     rc = _lib.load("latent_prefill").ts_latent_prefill(
         _lib.ptr(proj), _ll(proj.stride(0)), _ll(proj.shape[0]), _lib.ptr(kv), _ll(kv.stride(0)), s.heads * s.dim,
         ctypes.c_void_p(rows.data_ptr() + s.rank * rows.element_size()), _ll(rows.stride(0)), _ll(rows.shape[0]),
         _lib.ptr(cu_q), _lib.ptr(cu_k), cu_q.numel() - 1, max_q, s.heads, s.dim, s.rot, s.vdim, s.window, _f(s.scale),
-        _lib.ptr(out), _ll(out.stride(0)), _lib.stream_ptr())
+        gp, gld, mode, _lib.ptr(out), _ll(out.stride(0)), _lib.stream_ptr())
     _lib.check(rc, "ts_latent_prefill")

@@ -232,59 +232,88 @@ def topk_softmax(logits: torch.Tensor, k: int, normalize: bool = True):
 DECODE_ROWS = 32     # up to this many tokens the experts are read by the few-row kernels instead of 128-row tiles
 
 
-def _topk_raw(logits: torch.Tensor, k: int, normalize: bool):
-    T, E = logits.shape
+@dataclass(frozen=True)
+class Router:
+    """How logits become the chosen experts and their weights.  `groups` 0: softmax over all experts, the `top` largest.
+    Else sigmoid scores; experts form `groups` equal groups of neighbours, and only those of the `keep` groups with the
+    largest sums of their two largest scores can be chosen."""
+    experts: int
+    top: int
+    normalize: bool = False
+    groups: int = 0
+    keep: int = 0
+
+    def choose(self, logits: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor]:
+        """(weights [T, top] fp32, experts [T, top]) in PyTorch math."""
+        z = logits[:, :self.experts].float()
+        if self.groups == 0:
+            return topk_softmax(z, self.top, self.normalize)[:2]
+        s = torch.sigmoid(z)
+        size = self.experts // self.groups
+        value = s.unflatten(1, (self.groups, size)).topk(min(2, size), dim=-1).values.sum(-1)
+        best = torch.zeros_like(value, dtype=torch.bool).scatter_(1, value.topk(self.keep, dim=-1).indices, True)
+        w, idx = s.masked_fill(~best.repeat_interleave(size, dim=1), -1.0).topk(self.top, dim=-1)
+        return (w / (w.sum(-1, keepdim=True) + 1e-20) if self.normalize else w), idx
+
+
+def _topk_raw(logits: torch.Tensor, r: Router):
+    T, k = logits.shape[0], r.top
     w = torch.empty(T, k, dtype=torch.float32, device=logits.device)
     idx = torch.empty(T, k, dtype=torch.int32, device=logits.device)
-    rc = _lib.load("moe").ts_moe_topk_softmax(_lib.ptr(logits), _lib.ptr(None), _lib.ptr(w), _lib.ptr(idx), T, E, int(k),
-                                              int(normalize), _lib.stream_ptr())
-    _lib.check(rc, "ts_moe_topk_softmax")
+    rc = _lib.load("moe").ts_moe_topk(_lib.ptr(logits), _c.c_longlong(logits.stride(0)), _lib.ptr(None), _lib.ptr(w),
+                                      _lib.ptr(idx), T, r.experts, k, int(r.normalize), r.groups, r.keep, _lib.stream_ptr())
+    _lib.check(rc, "ts_moe_topk")
     return w, idx
 
 
-def _route_decode(logits: torch.Tensor, k: int, normalize: bool):
-    T, E = logits.shape
+def _route_decode(logits: torch.Tensor, r: Router):
+    T, E, k = logits.shape[0], r.experts, r.top
     i32 = dict(dtype=torch.int32, device=logits.device)
     w = torch.empty(T, k, dtype=torch.float32, device=logits.device)
     order, start, count = torch.empty(T * k, **i32), torch.empty(E, **i32), torch.empty(E, **i32)
-    rc = _lib.load("moe").ts_moe_route(_lib.ptr(logits), _lib.ptr(w), _lib.ptr(order), _lib.ptr(start), _lib.ptr(count), T, E,
-                                       int(k), int(normalize), _lib.stream_ptr())
+    rc = _lib.load("moe").ts_moe_route(_lib.ptr(logits), _c.c_longlong(logits.stride(0)), _lib.ptr(w), _lib.ptr(order),
+                                       _lib.ptr(start), _lib.ptr(count), T, E, k, int(r.normalize), r.groups, r.keep,
+                                       _lib.stream_ptr())
     _lib.check(rc, "ts_moe_route")
     return w, order, start, count
 
 
 def _grouped_act(x, W, plan: MoEPlan, act: int):
+    from .grouped import is_gated
     E, N, K = W.shape
-    y = torch.empty(plan.P, N, dtype=x.dtype, device=x.device)
+    cols = N // 2 if is_gated(act) else N
+    y = torch.empty(plan.P, cols, dtype=x.dtype, device=x.device)
     rc = _lib.load("gemm").ts_gemm_grouped_bf16_act(
-        _lib.ptr(x), _lib.ptr(W), _lib.ptr(y), 1, plan.P, N, K, K, K, N, 0, 0, 0, 0, _c.c_float(1.0),
+        _lib.ptr(x), _lib.ptr(W), _lib.ptr(y), 1, plan.P, N, K, K, K, cols, 0, 0, 0, 0, _c.c_float(1.0),
         _lib.ptr(plan.tile_expert), E, act, _lib.stream_ptr())
     _lib.check(rc, "ts_gemm_grouped_bf16_act")
     return y
 
 
-def routed_experts(x: torch.Tensor, logits: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, k: int, act: int,
-                   normalize: bool = False):
-    """Ungated experts down(act(up x)) of every token's top-k of softmax(logits), NOT combined: the layer boundary sums
-    them into the fp32 stream.  x [T, H], logits [T, E] fp32, w_up [E, F, H], w_down [E, H, F], act of ops/grouped.
+def routed_experts(x: torch.Tensor, logits: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, router: Router | int, act: int):
+    """Experts down(act(up x)) that the router chooses for every token, NOT combined: the layer boundary sums them into the
+    fp32 stream.  x [T, H], logits [T, >= E] fp32, w_up [E, F, H], w_down [E, H, F], act of ops/grouped (gated: w_up is
+    packed, [E, 2 F, H]); a number k as router is the k largest of a softmax.
     Returns (outputs, dest, weights [T, k]): slot t * k + j is row dest[slot] of the outputs (dest None: row slot).
 
     Few tokens: router, top-k and sort in one kernel, then one pass over the visited experts' weights.  Many (bf16):
     128-row expert segments on the grouped tcgen05 GEMM, the activation in its epilogue."""
     from . import grouped
-    T, E = logits.shape
+    if isinstance(router, int):
+        router = Router(w_up.shape[0], router)
+    T, E, k = x.shape[0], router.experts, router.top
     if not x.is_cuda:
-        w, idx, _ = topk_softmax(logits, k, normalize)
+        w, idx = router.choose(logits)
         y = torch.zeros(T * k, x.shape[1], dtype=x.dtype)
         for e in range(E):
             slots = (idx.reshape(-1) == e).nonzero().squeeze(1)
             y[slots] = grouped.activate(x[slots // k] @ w_up[e].t(), act) @ w_down[e].t()
         return y, None, w
-    H, F = x.shape[1], w_up.shape[1]
+    H, F = x.shape[1], w_down.shape[2]
     if T <= DECODE_ROWS and T * k <= _lib.load("moe").ts_moe_route_max_slots():
-        w, order, start, count = _route_decode(logits, k, normalize)
+        w, order, start, count = _route_decode(logits, router)
     else:
-        w, idx = _topk_raw(logits, k, normalize)
+        w, idx = _topk_raw(logits, router)
         plan = make_plan(idx, E)
         if x.dtype == torch.bfloat16 and H % 8 == 0 and F % 8 == 0:
             h = _grouped_act(_permute_raw(x, plan), w_up, plan, act)

@@ -16,12 +16,13 @@ from . import _lib
 def rope_inv_freq(dim: int, theta: float = 10000.0, scaling: str = "none", factor: float = 1.0,
                   original_max_pos: int = 8192, max_pos: int | None = None, beta_fast: float = 32.0,
                   beta_slow: float = 1.0, low_freq_factor: float = 1.0, high_freq_factor: float = 4.0,
-                  long_factor=None, short_factor=None) -> torch.Tensor:
+                  long_factor=None, short_factor=None, ramp_end: int | None = None) -> torch.Tensor:
     """Inverse frequencies [dim/2] for none | linear | ntk | dynamic_ntk | yarn | llama3 | longrope scaling.
 
     longrope (data_pipeline/trainer/kernels/rope_kernels.py:298-313): every rotary dimension has its own searched
     rescale factor; `long_factor` applies when the table covers more than `original_max_pos` positions, `short_factor`
-    otherwise (both [dim/2]).  Asking for it without the factor list it needs is an error, not a silent fallback."""
+    otherwise (both [dim/2]).  yarn: the ramp between kept and stretched pairs ends at pair `ramp_end` at the latest
+    (default: the last one; a larger number leaves it where the formula puts it).  Asking for it without the factor list it needs is an error, not a silent fallback."""
     half = dim // 2
     idx = torch.arange(0, half, dtype=torch.float64)
     scaling = (scaling or "none").lower()
@@ -49,7 +50,7 @@ def rope_inv_freq(dim: int, theta: float = 10000.0, scaling: str = "none", facto
         def corr_dim(rot):
             return dim * math.log(original_max_pos / (rot * 2 * math.pi)) / (2 * math.log(theta))
         low = max(math.floor(corr_dim(beta_fast)), 0)
-        high = min(math.ceil(corr_dim(beta_slow)), half - 1)
+        high = min(math.ceil(corr_dim(beta_slow)), half - 1 if ramp_end is None else ramp_end)
         ramp = ((idx - low) / max(high - low, 1e-3)).clamp(0, 1)
         inv = inv / factor * ramp + inv * (1 - ramp)
     elif scaling == "llama3":
@@ -61,6 +62,11 @@ def rope_inv_freq(dim: int, theta: float = 10000.0, scaling: str = "none", facto
         mid = (wavelen <= low_w) & (wavelen >= high_w)
         inv = torch.where(mid, (1 - smooth) * inv / factor + smooth * inv, scaled)
     return inv.float()
+
+
+def yarn_magnitude(factor: float) -> float:
+    """Factor of cos and sin that goes with a YaRN stretch."""
+    return 0.1 * math.log(factor) + 1.0
 
 
 def longrope_attention_factor(max_pos: int, original_max_pos: int) -> float:

@@ -414,6 +414,9 @@ register_models_from_meta([
     ModelInfo("vibepel", "trainscale", ("2B",), "VibepelForCausalLM", attention="sliding window + gated delta rule, wkv",
               mlp="dense (squared ReLU)", norm="output rmsnorm (offset weight)",
               notes="serving only: models/vibepel.py; windowed cache and matrix state per sequence"),
+    ModelInfo("kabulix", "trainscale", ("3B",), "KabulixForCausalLM", attention="sliding window with sinks, latent, chunked",
+              mlp="dense (gelu glu), moe (silu glu, grouped sigmoid router, shared expert)", norm="rmsnorm (offset weight)",
+              notes="serving only: models/kabulix.py; window, chunk and latent caches"),
     ModelInfo("llava", "llava-hf", ("7B", "13B"), "LlavaForConditionalGeneration", supported=False, notes="vision tower not covered"),
 ])
 
