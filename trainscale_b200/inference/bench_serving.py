@@ -16,6 +16,7 @@ from typing import Callable
 
 import torch
 
+from ..ops.masks import KeyMask
 from .batch import HostBatch, StepEntry
 from .engine import EngineConfig, EngineCore
 
@@ -31,6 +32,16 @@ VIBEPEL_SIZES = {
     "1k": dict(layers=12, width=1024, heads=8, kv=2, dim=128, window=512, ff=4096, dheads=8, dkv=4, ddim=128, wheads=16, wdim=64),
     "2k": dict(layers=16, width=2048, heads=16, kv=4, dim=128, window=1024, ff=8192, dheads=16, dkv=8, ddim=128, wheads=32, wdim=64),
     "4k": dict(layers=8, width=4096, heads=32, kv=8, dim=128, window=4096, ff=16384, dheads=32, dkv=16, ddim=128, wheads=64, wdim=64),
+}
+# layers take turns: window with sinks, chunks, latent, window with sinks; the first feeds forward densely, the others through
+# experts and a shared one; the closest model has the same routed experts and the attention of `heads` / `kv` in every layer
+KABULIX_SIZES = {
+    "1k": dict(layers=12, width=1024, heads=8, kv=2, dim=128, window=512, keep=4, chunk=1024, ldim=64, lrot=32, lvdim=64, rank=256,
+               experts=16, top=2, groups=4, kept=2, ff=1536),
+    "2k": dict(layers=16, width=2048, heads=16, kv=4, dim=128, window=1024, keep=4, chunk=2048, ldim=128, lrot=64, lvdim=128, rank=512,
+               experts=32, top=4, groups=8, kept=4, ff=1536),
+    "4k": dict(layers=8, width=4096, heads=32, kv=8, dim=128, window=4096, keep=4, chunk=4096, ldim=128, lrot=64, lvdim=128, rank=512,
+               experts=64, top=6, groups=8, kept=4, ff=1536),
 }
 VOCAB = 32000
 FP32_TFLOPS = 74.4            # nominal: 148 SMs x 128 lanes x 2 x 1.965 GHz
@@ -48,8 +59,9 @@ def build_closest(z: dict):
     """Llama decoder with a mixture of gated experts: same width, depth, heads, experts and expert weights."""
     from ..models.llama import LlamaConfig, build_model
     cfg = LlamaConfig(vocab_size=VOCAB, hidden_size=z["width"], intermediate_size=z["ff"] * 2 // 3,
-                      num_hidden_layers=z["layers"], num_attention_heads=z["heads"], num_key_value_heads=max(1, z["heads"] // 4),
-                      head_dim=z["vdim"], num_local_experts=z["experts"], num_experts_per_tok=z["top"],
+                      num_hidden_layers=z["layers"], num_attention_heads=z["heads"],
+                      num_key_value_heads=z.get("kv") or max(1, z["heads"] // 4),
+                      head_dim=z.get("vdim") or z["dim"], num_local_experts=z["experts"], num_experts_per_tok=z["top"],
                       model_type="mixtral", max_position_embeddings=16384)
     return build_model(cfg, torch.bfloat16, "cuda", seed=0, init_on_device=True)
 
@@ -70,6 +82,18 @@ def build_closest_dense(z: dict):
                       num_hidden_layers=z["layers"], num_attention_heads=z["heads"], num_key_value_heads=z["kv"],
                       head_dim=z["dim"], max_position_embeddings=16384, tie_word_embeddings=True)
     return build_model(cfg, torch.bfloat16, "cuda", seed=0, init_on_device=True)
+
+
+def build_kabulix(z: dict):
+    from ..models.kabulix import build_model, pattern_config
+    ff = z["ff"] * 2 // 3                    # three matrices per expert
+    kinds = ("wclw" * z["layers"])[:z["layers"]]
+    return build_model(pattern_config(kinds, vocab=VOCAB, width=z["width"], heads=z["heads"], kv_heads=z["kv"], dim=z["dim"],
+                                      window=z["window"], keep=z["keep"], chunk=z["chunk"], latent_dim=z["ldim"],
+                                      latent_rot=z["lrot"], latent_vdim=z["lvdim"], rank=z["rank"], latent_window=z["window"],
+                                      ff=ff * (z["top"] + 1), experts=z["experts"], top=z["top"], expert_ff=ff, shared_ff=ff,
+                                      groups=z["groups"], keep_groups=z["kept"], rot_dims=z["dim"] // 2),
+                       torch.bfloat16, "cuda", seed=0)
 
 
 def make_core(model, tokens: int, seqs: int) -> EngineCore:
@@ -168,10 +192,22 @@ def _visited(top: int, experts: int, rows: int) -> float:
     return experts * (1.0 - (1.0 - top / experts) ** rows)
 
 
-def mezilix_table(z: dict, rows: int, keys: float, pairs: float) -> list[tuple]:
-    """`keys`: cached rows a step must read per layer; `pairs`: visible (query, key) pairs per layer and head."""
+def _seen(lengths: list[tuple[int, int]], mask: KeyMask) -> tuple[float, float]:
+    """Over (first position, tokens) of a step: key rows its sequences need, and visible (query, key) pairs."""
+    keys = pairs = 0
+    for start, n in lengths:
+        keys += start + n - mask.first(start) + min(mask.keep, mask.first(start))
+        for p in range(start, start + n):
+            lo = mask.first(p)
+            pairs += p + 1 - lo + min(mask.keep, lo)
+    return float(keys), float(pairs)
+
+
+def mezilix_table(z: dict, rows: int, lengths: list[tuple[int, int]]) -> list[tuple]:
+    """`lengths`: (first position, tokens) of the step's sequences, `rows` tokens in all."""
     from ..ops import gemm, grouped, latent_attention as latent, moe, stream
     W, H = z["width"], z["heads"]
+    keys, pairs = _seen(lengths, KeyMask(z["window"]))
     ew = _visited(z["top"], z["experts"], rows) * z["ff"] * W * 2
 
     def boundary(a, k, out):
@@ -213,10 +249,11 @@ def mezilix_table(z: dict, rows: int, keys: float, pairs: float) -> list[tuple]:
     ]
 
 
-def vibepel_table(z: dict, rows: int, keys: float, pairs: float) -> list[tuple]:
+def vibepel_table(z: dict, rows: int, lengths: list[tuple[int, int]]) -> list[tuple]:
     """The scans' arithmetic is fp32: three products of every state element per token."""
     from ..ops import gemm, grouped, latent_attention as latent, recurrent, stream, window_attention as window
     W, H, G, D = z["width"], z["heads"], z["kv"], z["dim"]
+    keys, pairs = _seen(lengths, KeyMask(z["window"]))
 
     def boundary(a, k, out):
         if isinstance(out, torch.Tensor):                      # last boundary: only the wanted rows
@@ -255,9 +292,68 @@ def vibepel_table(z: dict, rows: int, keys: float, pairs: float) -> list[tuple]:
     ]
 
 
-def closest_table(z: dict, rows: int, keys: float, pairs: float, runner) -> list[tuple]:
+def kabulix_table(z: dict, rows: int, lengths: list[tuple[int, int]]) -> list[tuple]:
+    from ..ops import gemm, grouped, latent_attention as latent, moe, stream, window_attention as window
+    W = z["width"]
+    visited = _visited(z["top"], z["experts"], rows)
+
+    def boundary(a, k, out):
+        final = isinstance(out, torch.Tensor)                  # last boundary: only the wanted rows
+        T = (out if final else out[0]).shape[0]
+        per = 4 + 2 + (0 if a[3] is None else 2 * a[3][2].shape[1]) + (0 if final else 4) + 2
+        return per * T * W, 0.0
+
+    def kind(s):
+        return "chunks" if s.chunked else "window"
+
+    def experts(a, k, out):
+        x, w = a[0], a[1]
+        cols = out.shape[-1]
+        return visited * w.shape[1] * w.shape[2] * 2 + rows * z["top"] * (w.shape[2] + cols) * 2, 2.0 * rows * z["top"] * w.shape[1] * w.shape[2]
+
+    def prepared(a, k, out):
+        s = a[1]
+        moved = s.q_width + s.kv_heads * s.dim if a[2] is not None else 0       # read and written in place
+        return a[0].shape[0] * 2 * (2 * moved + (s.kv_heads * s.vdim if s.values_are_keys else s.kv_width - (moved and s.kv_heads * s.dim)) +
+                                    s.kv_width), 0.0
+
+    return [
+        (stream, "prenorm_embed", "embedding, norm", lambda a, k, o: (a[0].shape[0] * W * (2 + 4 + 2), 0.0)),
+        (stream, "prenorm", lambda a, o: "sum, norm" if a[3] is None else "expert combine, sum, norm", boundary),
+        (stream, "prenorm_final", "last norm", boundary),
+        (gemm, "serve_linear", _linear_name("gemm"), _linear_cost),
+        (gemm, "matmul_nt", _linear_name("gemm"), _linear_cost),
+        (window, "prepare", lambda a, o: "bias, head norms, rotary, cache write" if a[2] is not None else "cache write", prepared),
+        (latent, "prepare", "latent norm, rotary, cache write",
+         lambda a, k, o: (a[0].shape[0] * 2 * (2 * a[1].heads * a[1].rot + a[1].rank + a[1].rot + a[1].row_width * (2 if o is not None else 1)), 0.0)),
+        (latent, "gather_rows", "key gather", lambda a, k, o: (2 * _bytes(o), 0.0)),
+        (window, "attend_rows", lambda a, o: f"attention ({kind(a[1])}, rows)",
+         lambda a, k, o: (_seen(lengths, a[1].mask)[0] * a[1].kv_width * 2 + a[0].shape[0] * (a[1].q_width + a[1].out_width) * 2,
+                          2.0 * _seen(lengths, a[1].mask)[1] * a[1].heads * (a[1].dim + a[1].vdim))),
+        (window, "attend_portions", lambda a, o: f"attention ({kind(a[1])}, portions)",
+         lambda a, k, o: (a[0].shape[0] * (a[1].q_width + a[1].kv_width + a[1].out_width) * 2,
+                          2.0 * _seen(lengths, a[1].mask)[1] * a[1].heads * (a[1].dim + a[1].vdim))),
+        (latent, "attend_latent", "attention (latent space)",
+         lambda a, k, o: (_seen(lengths, a[2].mask)[0] * a[2].row_width * 2 + 2 * _bytes(a[0]),
+                          2.0 * _seen(lengths, a[2].mask)[1] * a[2].heads * (2 * a[2].rank + a[2].rot))),
+        (latent, "attend_expanded", "attention (latent, portions)",
+         lambda a, k, o: (_bytes(a[1], a[2]) + a[0].shape[0] * a[3].q_width * 2 + 2 * _bytes(a[7]),
+                          2.0 * _seen(lengths, a[3].mask)[1] * a[3].heads * (a[3].dim + a[3].rot + a[3].vdim))),
+        (grouped, "head_linear", lambda a, o: f"per-head projection {a[1].shape[1]}x{a[1].shape[2]}",
+         lambda a, k, o: (_bytes(a[0], a[1], o), 2.0 * a[0].shape[0] * a[1].numel())),
+        (grouped, "expert_linear", lambda a, o: f"experts {a[1].shape[1]}x{a[1].shape[2]}", experts),
+        (moe, "_route_decode", "router top-k, sort", lambda a, k, o: (_bytes(a[0], *o), 0.0)),
+        (moe, "_topk_raw", "router top-k", lambda a, k, o: (_bytes(a[0], *o), 0.0)),
+        (moe, "make_plan", "routing plan", lambda a, k, o: (_bytes(a[0], o.dest, o.src_of_row), 0.0)),
+        (moe, "_permute_raw", "permute", lambda a, k, o: (_bytes(a[0]) + a[1].n * W * 2, 0.0)),
+        (moe, "_grouped_act", lambda a, o: f"experts {a[1].shape[1]}x{a[1].shape[2]}", experts),
+    ]
+
+
+def closest_table(z: dict, rows: int, lengths: list[tuple[int, int]], runner) -> list[tuple]:
     from ..ops import activation, gemm, moe, norm, rope
     W, H, D = z["width"], z["heads"], z.get("vdim") or z["dim"]
+    keys, pairs = _seen(lengths, KeyMask(1 << 30))
     hkv = z.get("kv") or max(1, H // 4)
 
     def grouped_cost(a, k, out):
@@ -280,11 +376,6 @@ def closest_table(z: dict, rows: int, keys: float, pairs: float, runner) -> list
 
 
 # ---------------------------------------------------------------------------------------------- measurement
-def _visible_pairs(lengths: list[tuple[int, int]], window: int) -> float:
-    """Sum over (first position, tokens) of the keys each position sees."""
-    return float(sum(min(p + 1, window) for start, n in lengths for p in range(start, start + n)))
-
-
 @dataclass(frozen=True)
 class Design:
     sizes: dict
@@ -294,7 +385,8 @@ class Design:
 
 
 DESIGNS = {"mezilix": Design(SIZES, build_mezilix, build_closest, mezilix_table),
-           "vibepel": Design(VIBEPEL_SIZES, build_vibepel, build_closest_dense, vibepel_table)}
+           "vibepel": Design(VIBEPEL_SIZES, build_vibepel, build_closest_dense, vibepel_table),
+           "kabulix": Design(KABULIX_SIZES, build_kabulix, build_closest, kabulix_table)}
 
 
 def measure(design: str, name: str, peaks: dict, prompts: int = 2, prompt_len: int = 4096, batches=(8, 64), context: int = 2048,
@@ -305,14 +397,13 @@ def measure(design: str, name: str, peaks: dict, prompts: int = 2, prompt_len: i
     for kind, build in ((design, spec.build), ("closest", spec.closest)):
         model = build(z)
         core = make_core(model, max(prompts * prompt_len, max(batches) * (context + 64)), max(max(batches), prompts))
-        window = z["window"] if kind == design else 1 << 30
         res: dict = {"parameters": sum(p.numel() for p in model.parameters())}
 
-        def table(rows, keys, pairs):
-            return spec.table(z, rows, keys, pairs) if kind == design else closest_table(z, rows, keys, pairs, core.runner)
+        def table(rows, lengths):
+            return spec.table(z, rows, lengths) if kind == design else closest_table(z, rows, lengths, core.runner)
 
-        def profile(step, rows, keys, pairs):
-            with OpTimer(table(rows, keys, pairs)) as t:
+        def profile(step, rows, lengths):
+            with OpTimer(table(rows, lengths)) as t:
                 torch.cuda._sleep(200_000_000)
                 step()
             return t.summary(peaks)
@@ -325,7 +416,7 @@ def measure(design: str, name: str, peaks: dict, prompts: int = 2, prompt_len: i
         ms = _timed(step, iters)
         T = prompts * prompt_len
         res["prefill"] = {"tokens": T, "ms": ms, "tokens_per_s": T / ms * 1e3,
-                          "ops": profile(step, T, T, _visible_pairs([(0, prompt_len)] * prompts, window))}
+                          "ops": profile(step, T, [(0, prompt_len)] * prompts)}
         # portions that continue cached prompts
         if kind == design:
             for i in range(prompts):
@@ -346,8 +437,7 @@ def measure(design: str, name: str, peaks: dict, prompts: int = 2, prompt_len: i
             host = HostBatch(core.cache, [StepEntry(j, [j + 1]) for j in range(n)])
             batch = host.to_device("cuda")
             step = lambda: core.runner.logits(core.runner.forward(batch))   # noqa: E731
-            keys = float(n * min(window, context + 1))
-            d = {"ms": _timed(step, iters), "ops": profile(step, n, keys, keys)}
+            d = {"ms": _timed(step, iters), "ops": profile(step, n, [(context, 1)] * n)}
             if core.runner.can_graph(host):
                 core.runner.decode_graphed(host)
                 d["graph_ms"] = _timed(lambda: core.runner.decode_graphed(host), iters)
