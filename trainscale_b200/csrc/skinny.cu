@@ -71,8 +71,8 @@ __device__ __forceinline__ uint4 ld_stream(const void* p) {   // weights: read o
 // 32-wide reduction steps a warp has in flight
 __host__ __device__ constexpr int skinny_unroll(int nt) { return nt == 1 ? 8 : (nt <= 4 ? 4 : 2); }
 
-// NT: token tiles of 8 per pass.  KW: warps that share a row tile and split its reduction; the CTA's 8 / KW row tiles are
-// neighbours.  grid (ceil(N / (16 * 8 / KW)), groups).
+// NT: token tiles of 8 per pass; grid.z shares the passes.  KW: warps that share a row tile and split its reduction; the CTA's 8 / KW row tiles are
+// neighbours.  grid (ceil(N / (16 * 8 / KW)), groups, passes side by side).
 template <int NT, int KW>
 __global__ void __launch_bounds__(SK_WARPS * 32)
 skinny_gemm_kernel(SkinnyParams p) {
@@ -95,7 +95,7 @@ skinny_gemm_kernel(SkinnyParams p) {
   const __nv_bfloat16* w1 = W + (row1 ? n0 + gid + up : 0) * p.ldw + tig * 8;
   const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
 
-  for (int base = 0; base < m_total; base += NT * 8) {
+  for (int base = blockIdx.z * NT * 8; base < m_total; base += gridDim.z * NT * 8) {
     const int m = min(NT * 8, m_total - base);
     const __nv_bfloat16* x[NT];
 #pragma unroll
@@ -229,7 +229,7 @@ extern "C" int ts_skinny_gemm(const void* A, const void* W, void* out, long long
                               long long a_group, long long w_group, long long o_group, const int* order,
                               const int* start, const int* count, int a_div, int groups, int M, int N, int K, int act,
                               float act_cap, int fp32, int out_fp32, int typical, const void* gate, long long gate_ld,
-                              long long gate_group, void* stream) {
+                              long long gate_group, int row_tiles, void* stream) {
   if (M <= 0 || groups <= 0) return 0;
   if (N <= 0 || K <= 0 || a_div <= 0 || act < 0 || act > ACT_LAST_GLU || (act == 3 && !(act_cap > 0.f)) || groups > 65535)
     return -10;
@@ -252,11 +252,15 @@ extern "C" int ts_skinny_gemm(const void* A, const void* W, void* out, long long
     return (int)cudaGetLastError();
   }
   const int per_pass = count && typical > 0 && typical < M ? typical : M;
-  const int nt = per_pass <= 8 ? 1 : (per_pass <= 16 ? 2 : (per_pass <= 32 ? 4 : 8));
+  int nt = per_pass <= 8 ? 1 : (per_pass <= 16 ? 2 : (per_pass <= 32 ? 4 : 8)), z = 1;
+  if (row_tiles > 0) {
+    while (nt > row_tiles) nt /= 2;
+    z = (M + nt * 8 - 1) / (nt * 8);
+  }
   int kw = 1;
   while (kw < SK_WARPS && kw * skinny_unroll(nt) * 32 < K) kw *= 2;
   const int rows = 16 * SK_WARPS / kw;
-  const dim3 grid((N + rows - 1) / rows, groups);
+  const dim3 grid((N + rows - 1) / rows, groups, z);
   if (nt == 1) launch_skinny<1>(kw, grid, st, p);
   else if (nt == 2) launch_skinny<2>(kw, grid, st, p);
   else if (nt == 4) launch_skinny<4>(kw, grid, st, p);

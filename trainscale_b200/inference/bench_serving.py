@@ -36,9 +36,9 @@ VIBEPEL_SIZES = {
 # layers take turns: window with sinks, chunks, latent, window with sinks; the first feeds forward densely, the others through
 # experts and a shared one; the closest model has the same routed experts and the attention of `heads` / `kv` in every layer
 KABULIX_SIZES = {
-    "1k": dict(layers=12, width=1024, heads=8, kv=2, dim=128, window=512, keep=4, chunk=1024, ldim=64, lrot=32, lvdim=64, rank=256,
+    "1k": dict(layers=12, width=1024, heads=8, kv=2, dim=128, window=512, keep=4, chunk=1536, ldim=64, lrot=32, lvdim=64, rank=256,
                experts=16, top=2, groups=4, kept=2, ff=1536),
-    "2k": dict(layers=16, width=2048, heads=16, kv=4, dim=128, window=1024, keep=4, chunk=2048, ldim=128, lrot=64, lvdim=128, rank=512,
+    "2k": dict(layers=16, width=2048, heads=16, kv=4, dim=128, window=1024, keep=4, chunk=3072, ldim=128, lrot=64, lvdim=128, rank=512,
                experts=32, top=4, groups=8, kept=4, ff=1536),
     "4k": dict(layers=8, width=4096, heads=32, kv=8, dim=128, window=4096, keep=4, chunk=4096, ldim=128, lrot=64, lvdim=128, rank=512,
                experts=64, top=6, groups=8, kept=4, ff=1536),

@@ -136,7 +136,8 @@ def _read_mlp(i: int, f: dict[str, Any] | None):
         return DenseConfig(f["ff"])
     if f["kind"] != "moe":
         raise ValueError(f"layer {i}: unknown feed-forward {f['kind']!r}")
-    r, g = f["router"], f["router"]["groups"]
+    r = f["router"]
+    g = r.get("groups") or {"count": 1, "keep": 1}
     _require(r["experts"] % g["count"] == 0 and 0 < g["keep"] <= g["count"], i, "equal groups of experts, some of them kept")
     _require(0 < r["top"] <= g["keep"] * (r["experts"] // g["count"]), i, "no more experts per token than the kept groups hold")
     _require(r["top"] <= MAX_TOP and r["experts"] <= MAX_EXPERTS, i, f"at most {MAX_TOP} of {MAX_EXPERTS} experts")

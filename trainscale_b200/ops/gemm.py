@@ -208,9 +208,9 @@ class _SplitLinearCPU(torch.autograd.Function):
 
 
 def few_rows(M: int, N: int, K: int) -> bool:
-    """Whether one pass over the weight by warps (ops/grouped.rows_linear) beats 128-row tcgen05 tiles: measured crossover,
-    later for small weights, whose few tiles leave most of the GPU idle."""
-    return M <= 16 or (M <= 32 and N * K <= 1 << 23)
+    """Whether passes over the weight by warps (ops/grouped.rows_linear) beat 128-row tcgen05 tiles: measured crossover, later
+    for few columns, whose few tiles leave most of the GPU idle."""
+    return M <= 16 or (M <= 64 and M * N <= 3 << 15)
 
 
 @torch.no_grad()

@@ -56,15 +56,20 @@ def activate(x: torch.Tensor, act: int, cap: float = 0.0) -> torch.Tensor:
 
 
 def _launch(A, W, out, lda, ldw, ldo, a_group, w_group, o_group, order, start, count, a_div, groups, M, N, K, act,
-            typical=0, cap=0.0, gate=None):
+            typical=0, cap=0.0, gate=None, row_tiles=0):
     if gate is not None and gate.dtype != A.dtype:
         raise TypeError("the gate has the type of the rows")
     rc = _lib.load("skinny").ts_skinny_gemm(
         _lib.ptr(A), _lib.ptr(W), _lib.ptr(out), _ll(lda), _ll(ldw), _ll(ldo), _ll(a_group), _ll(w_group), _ll(o_group),
         _lib.ptr(order), _lib.ptr(start), _lib.ptr(count), a_div, groups, M, N, K, act, ctypes.c_float(cap),
         int(A.dtype == torch.float32), int(out.dtype == torch.float32), typical, _lib.ptr(gate),
-        _ll(0 if gate is None else gate.stride(0)), _ll(0 if gate is None else gate.stride(1)), _lib.stream_ptr())
+        _ll(0 if gate is None else gate.stride(0)), _ll(0 if gate is None else gate.stride(1)), row_tiles, _lib.stream_ptr())
     _lib.check(rc, "ts_skinny_gemm")
+
+
+def _row_tiles(rows: int, cols: int) -> int:
+    """Tiles of eight rows per pass when the passes run side by side: short passes while there are few of them (measured)."""
+    return 1 if rows * cols <= 1 << 15 else 2
 
 
 def rows_linear(x: torch.Tensor, w: torch.Tensor, out_dtype=None, act: int = ACT_NONE, cap: float = 0.0,
@@ -73,7 +78,7 @@ def rows_linear(x: torch.Tensor, w: torch.Tensor, out_dtype=None, act: int = ACT
     if out is None:
         out = torch.empty(x.shape[0], w.shape[0] // (2 if is_gated(act) else 1), dtype=out_dtype or x.dtype, device=x.device)
     _launch(x, w, out, x.stride(0), w.stride(0), out.stride(0), 0, 0, 0, None, None, None, 1, 1, x.shape[0], w.shape[0],
-            w.shape[1], act, cap=cap)
+            w.shape[1], act, cap=cap, row_tiles=_row_tiles(x.shape[0], w.shape[0]))
     return out
 
 
@@ -88,7 +93,7 @@ def head_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = Non
         y = torch.einsum("thk,hnk->thn", x, w)
         return out.copy_(y if gate is None else y * torch.sigmoid(gate))
     _launch(x, w, out, x.stride(0), w.stride(1), out.stride(0), x.stride(1), w.stride(0), out.stride(1), None, None, None, 1,
-            H, T, N, K, ACT_NONE, gate=gate)
+            H, T, N, K, ACT_NONE, gate=gate, row_tiles=_row_tiles(T, H * N))
     return out
 
 
@@ -99,5 +104,5 @@ def expert_linear(x: torch.Tensor, w: torch.Tensor, order, start, count, slots: 
     E, N, K = w.shape
     out = torch.empty(slots, N // (2 if is_gated(act) else 1), dtype=x.dtype, device=x.device)
     _launch(x, w, out, x.stride(0), w.stride(1), out.stride(0), 0, w.stride(0), 0, order, start, count, per_row, E, max_rows,
-            N, K, act, -(-2 * slots // E))
+            N, K, act, -(-2 * slots // E), row_tiles=4)
     return out

@@ -229,7 +229,8 @@ def topk_softmax(logits: torch.Tensor, k: int, normalize: bool = True):
 
 
 # ---------------------------------------------------------------------------------------------- serving (no autograd)
-DECODE_ROWS = 32     # up to this many tokens the experts are read by the few-row kernels instead of 128-row tiles
+# up to this many tokens and routed slots the experts are read by the few-row kernels instead of 128-row tiles (measured)
+DECODE_ROWS, DECODE_SLOTS = 64, 128
 
 
 @dataclass(frozen=True)
@@ -310,7 +311,7 @@ def routed_experts(x: torch.Tensor, logits: torch.Tensor, w_up: torch.Tensor, w_
             y[slots] = grouped.activate(x[slots // k] @ w_up[e].t(), act) @ w_down[e].t()
         return y, None, w
     H, F = x.shape[1], w_down.shape[2]
-    if T <= DECODE_ROWS and T * k <= _lib.load("moe").ts_moe_route_max_slots():
+    if T <= DECODE_ROWS and T * k <= DECODE_SLOTS:
         w, order, start, count = _route_decode(logits, router)
     else:
         w, idx = _topk_raw(logits, router)
