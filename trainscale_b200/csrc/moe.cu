@@ -431,7 +431,6 @@ extern "C" int ts_moe_topk_softmax(const float* logits, float* probs, float* wei
 }
 
 // Decode-sized router: logits fp32 [T][ld] -> weights [T][k], order [T * k], start [E], count [E].
-extern "C" int ts_moe_route_max_slots() { return ROUTE_MAX_SLOTS; }
 extern "C" int ts_moe_route(const float* logits, long long ld, float* weights, int* order, int* start, int* count, int T, int E,
                             int k, int normalize, int groups, int keep, void* stream) {
   if (!router_ok(T, E, k, ld, groups, keep) || T * k > ROUTE_MAX_SLOTS) return -10;
