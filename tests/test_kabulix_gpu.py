@@ -249,9 +249,9 @@ def test_attend_rows_masks_and_gates(dtype, H, G, D, V, rot, size, keep, chunked
     assert out[:, s.out_width:].abs().sum() == 0
 
 
-PORTION_MASKS = [(50, 4, False), (136, 3, False), (136, 128, False), (100, 130, False), (129, 1, False), (300, 500, False), (1, 1, False), (64, 300, False),
+PORTION_MASKS = [(50, 4, False), (140, 3, False), (140, 128, False), (100, 130, False), (129, 1, False), (300, 500, False), (1, 1, False), (64, 300, False),
                  (4000, 7, False), (128, 0, False), (40, 0, True), (128, 0, True), (200, 0, True), (1, 0, True), (1000, 0, True)]
-PORTIONS = [[(0, 300), (0, 1), (0, 51), (0, 700)], [(0, 1100)], [(128, 2), (700, 260), (3, 40), (600, 600)], [(255, 257), (256, 2), (511, 300), (136, 385)],
+PORTIONS = [[(0, 300), (0, 1), (0, 51), (0, 700)], [(0, 1100)], [(128, 2), (700, 260), (3, 40), (600, 600)], [(255, 257), (256, 2), (511, 300), (140, 385)],
             [(199, 2), (200, 1), (201, 199), (399, 402)]]
 
 
@@ -340,7 +340,7 @@ def test_head_products_with_a_gate(dtype, T, H, K, N):
 
 @pytest.mark.parametrize("shape", [dict(heads=2, dim=24, rot=8, vdim=16, rank=48), dict(heads=3, dim=72, rot=40, vdim=80, rank=40),
                                    dict(heads=2, dim=128, rot=64, vdim=128, rank=96)])
-@pytest.mark.parametrize("window", [1, 72, 128, 300])
+@pytest.mark.parametrize("window", [1, 70, 128, 300])
 def test_attend_expanded_with_a_gate(shape, window):
     from trainscale_b200.ops import latent_attention as L
     s = L.LatentShape(window=window, scale=0.3, rope_base=1e4, **shape)
@@ -432,8 +432,8 @@ def test_whole_prompts_portions_and_decoding(dtype, name):
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_long_prompt_and_long_decoding(dtype):
     """A prompt of several query blocks, and hundreds of tokens decoded one by one past every window and chunk."""
-    cfg = O.make_config(width=64, heads=4, kv_heads=2, dim=32, vdim=32, rot=16, window=136, keep=4, chunk=200, ldim=32, lvdim=32, lrot=16,
-                        rank=48, lwindow=72, mlps=("dense",))
+    cfg = O.make_config(width=64, heads=4, kv_heads=2, dim=32, vdim=32, rot=16, window=150, keep=5, chunk=210, ldim=32, lvdim=32, lrot=16,
+                        rank=48, lwindow=66, mlps=("dense",))
     w = O.make_weights(cfg, 5)
     ref, ids = Reference(w, cfg), tokens(1100, 2)
     want = ref(ids)
