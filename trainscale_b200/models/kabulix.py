@@ -32,6 +32,7 @@ from ..ops.grouped import GluRows, glu_width
 from ..ops.latent_attention import LatentShape
 from ..ops.moe import Router
 from ..ops.window_attention import WindowShape
+from .served import ServedDecoder, fp32_param, require, up8, weight_param
 
 MAX_EXPERTS, MAX_TOP = 1024, 32
 
@@ -104,27 +105,22 @@ class LayerConfig:
     mlp: DenseConfig | MoeConfig | None
 
 
-def _require(ok: bool, layer: int, what: str) -> None:
-    if not ok:
-        raise ValueError(f"layer {layer}: needs {what}")
-
-
 def _read_mixer(i: int, kind: str, m: dict[str, Any]):
     if kind not in ("attention", "latent_attention", "attention_2"):
         raise ValueError(f"layer {i}: unknown mixer {kind!r}")
     mask, scale = m["mask"], float(m["scale"])
-    _require(mask["size"] > 0 and mask.get("keep_first", 0) >= 0, i, "a window or chunk of at least one token")
+    require(mask["size"] > 0 and mask.get("keep_first", 0) >= 0, i, "a window or chunk of at least one token")
     if kind == "latent_attention":
         rot = Rotation.from_dict(m["rot"])
-        _require(rot.dims == m["rot_dim"] and rot.dims % 2 == 0, i, "a rotation of the whole (even) rotated part of a head")
+        require(rot.dims == m["rot_dim"] and rot.dims % 2 == 0, i, "a rotation of the whole (even) rotated part of a head")
         return LatentConfig(LatentShape(m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], mask["size"], scale,
                                         rot.base, True, rot.magnitude), rot)
-    _require(m["heads"] % m["kv_heads"] == 0, i, "whole head groups")
+    require(m["heads"] % m["kv_heads"] == 0, i, "whole head groups")
     if kind == "attention_2":
         return ChunkConfig(WindowShape(m["heads"], m["kv_heads"], m["dim"], m["vdim"], 0, mask["size"], scale, chunked=True))
     rot = Rotation.from_dict(m["rot"])
-    _require(rot.dims % 2 == 0 and rot.dims <= m["dim"], i, "an even number of rotated dimensions inside a head")
-    _require(m["vdim"] == m["dim"], i, "values of the size of the keys, which they are")
+    require(rot.dims % 2 == 0 and rot.dims <= m["dim"], i, "an even number of rotated dimensions inside a head")
+    require(m["vdim"] == m["dim"], i, "values of the size of the keys, which they are")
     return SinkConfig(WindowShape(m["heads"], m["kv_heads"], m["dim"], m["vdim"], rot.dims, mask["size"], scale,
                                   mask.get("keep_first", 0), pairs=True, values_are_keys=True), rot)
 
@@ -138,9 +134,9 @@ def _read_mlp(i: int, f: dict[str, Any] | None):
         raise ValueError(f"layer {i}: unknown feed-forward {f['kind']!r}")
     r = f["router"]
     g = r.get("groups") or {"count": 1, "keep": 1}
-    _require(r["experts"] % g["count"] == 0 and 0 < g["keep"] <= g["count"], i, "equal groups of experts, some of them kept")
-    _require(0 < r["top"] <= g["keep"] * (r["experts"] // g["count"]), i, "no more experts per token than the kept groups hold")
-    _require(r["top"] <= MAX_TOP and r["experts"] <= MAX_EXPERTS, i, f"at most {MAX_TOP} of {MAX_EXPERTS} experts")
+    require(r["experts"] % g["count"] == 0 and 0 < g["keep"] <= g["count"], i, "equal groups of experts, some of them kept")
+    require(0 < r["top"] <= g["keep"] * (r["experts"] // g["count"]), i, "no more experts per token than the kept groups hold")
+    require(r["top"] <= MAX_TOP and r["experts"] <= MAX_EXPERTS, i, f"at most {MAX_TOP} of {MAX_EXPERTS} experts")
     return MoeConfig(Router(r["experts"], r["top"], True, g["count"], g["keep"]), f["expert"]["ff"], f["shared"]["ff"])
 
 
@@ -218,18 +214,6 @@ PRESETS: dict[str, KabulixConfig] = {
 }
 
 
-def _fp32(*shape) -> nn.Parameter:
-    return nn.Parameter(torch.empty(*shape, dtype=torch.float32), requires_grad=False)
-
-
-def _weight(*shape) -> nn.Parameter:
-    return nn.Parameter(torch.zeros(*shape), requires_grad=False)     # padding rows and columns stay zero
-
-
-def _up8(n: int) -> int:
-    return -(-n // 8) * 8
-
-
 @dataclass
 class StepContext:
     """What the layers of one step share."""
@@ -253,15 +237,15 @@ class GroupedMixer(nn.Module):
         self.cfg, self.eps = cfg, eps
         s = cfg.shape
         self.sinks = isinstance(cfg, SinkConfig)
-        self.w_in = _weight(_up8(s.in_width + (0 if self.sinks else s.heads)), width)
-        self.w_o = _weight(width, _up8(s.out_width))
+        self.w_in = weight_param(up8(s.in_width + (0 if self.sinks else s.heads)), width)
+        self.w_o = weight_param(width, up8(s.out_width))
         self.bias = self.q_norm = self.k_norm = None
         if self.sinks:
-            self.bias = _fp32(s.q_width + s.kv_heads * s.dim)
-            self.q_norm, self.k_norm = _fp32(s.dim), _fp32(s.dim)
+            self.bias = fp32_param(s.q_width + s.kv_heads * s.dim)
+            self.q_norm, self.k_norm = fp32_param(s.dim), fp32_param(s.dim)
             self.register_buffer("inv_freq", cfg.rot.inv_freq().to(self.q_norm.device), persistent=False)
         # columns of a projected row: what the GEMM writes, and room for the values where they come from the keys
-        self.columns = max(self.w_in.shape[0], _up8(s.q_width + s.kv_width))
+        self.columns = max(self.w_in.shape[0], up8(s.q_width + s.kv_width))
 
     def tensors(self):
         """(checkpoint name under '.mix.', parameter or view of one)."""
@@ -315,11 +299,11 @@ class LatentMixer(nn.Module):
         super().__init__()
         self.cfg, self.eps = cfg, eps
         m = cfg.shape
-        self.gate_at = _up8(m.q_width + m.rank + m.rot)
-        self.w_in = _weight(_up8(self.gate_at + m.heads * m.vdim), width)
-        self.kv_norm = _fp32(m.rank)
-        self.w_kv = _weight(m.heads * (m.dim + m.vdim), m.rank)          # unrotated keys | values, head by head
-        self.w_o = _weight(width, _up8(m.heads * m.vdim))
+        self.gate_at = up8(m.q_width + m.rank + m.rot)
+        self.w_in = weight_param(up8(self.gate_at + m.heads * m.vdim), width)
+        self.kv_norm = fp32_param(m.rank)
+        self.w_kv = weight_param(m.heads * (m.dim + m.vdim), m.rank)          # unrotated keys | values, head by head
+        self.w_o = weight_param(width, up8(m.heads * m.vdim))
         self.register_buffer("w_uk_t", torch.empty(m.heads, m.rank, m.dim), persistent=False)
         self.register_buffer("inv_freq", cfg.rot.inv_freq().to(self.kv_norm.device), persistent=False)
 
@@ -375,7 +359,7 @@ class GatedProduct(nn.Module):
     def __init__(self, width: int, ff: int, act: int):
         super().__init__()
         self.ff, self.act = ff, act
-        self.w_in, self.w_down = _weight(2 * glu_width(ff), width), _weight(width, glu_width(ff))
+        self.w_in, self.w_down = weight_param(2 * glu_width(ff), width), weight_param(width, glu_width(ff))
 
     def tensors(self):
         yield "gate", GluRows(self.w_in, self.ff, 0)
@@ -406,8 +390,8 @@ class ExpertFeedForward(nn.Module):
         super().__init__()
         self.cfg = cfg
         E, F = cfg.router.experts, glu_width(cfg.ff)
-        self.w_router = _weight(_up8(E + 1), width)
-        self.w_in, self.w_down = _weight(E, 2 * F, width), _weight(E, width, F)
+        self.w_router = weight_param(up8(E + 1), width)
+        self.w_in, self.w_down = weight_param(E, 2 * F, width), weight_param(E, width, F)
         self.shared = GatedProduct(width, cfg.shared_ff, grouped.ACT_SILU_GLU)
 
     def tensors(self):
@@ -444,16 +428,15 @@ class KabulixLayer(nn.Module):
     def __init__(self, cfg: KabulixConfig, index: int):
         super().__init__()
         W, l = cfg.hidden_size, cfg.layers[index]
-        self.norm1 = _fp32(W)
+        self.norm1 = fp32_param(W)
         self.mixer = (LatentMixer if isinstance(l.mixer, LatentConfig) else GroupedMixer)(l.mixer, W, cfg.eps)
         self.ff = None
         if l.mlp is not None:
-            self.norm2 = _fp32(W)
+            self.norm2 = fp32_param(W)
             self.ff = (DenseFeedForward if isinstance(l.mlp, DenseConfig) else ExpertFeedForward)(l.mlp, W)
 
 
-class KabulixForCausalLM(nn.Module):
-    # libraries `serve` needs (compiled together at the first use)
+class KabulixForCausalLM(ServedDecoder):
     LIBRARIES = ("stream", "window", "latent", "latent_prefill", "skinny", "moe", "gemm")
 
     def __init__(self, cfg: KabulixConfig):
@@ -461,8 +444,7 @@ class KabulixForCausalLM(nn.Module):
         self.config = cfg
         self.embed = nn.Parameter(torch.empty(cfg.vocab_size, cfg.hidden_size), requires_grad=False)
         self.layers = nn.ModuleList(KabulixLayer(cfg, i) for i in range(cfg.num_hidden_layers))
-        self.final_norm = _fp32(cfg.hidden_size)
-        self._side = None                 # stream of the shared expert in captured decode steps
+        self.final_norm = fp32_param(cfg.hidden_size)
 
     # ---------------------------------------------------------------- weights
     def _checkpoint_tensors(self):
@@ -492,35 +474,16 @@ class KabulixForCausalLM(nn.Module):
                 t.copy_(torch.empty(t.shape, dtype=torch.float32, device=gen.device).normal_(0.0, 1.0 / math.sqrt(t.shape[-1]), generator=gen))
             else:
                 t.normal_(0.0, 1.0 / math.sqrt(t.shape[-1]), generator=gen)
+        self.finalize()
+
+    def finalize(self) -> None:
         for l in self.layers:
             l.mixer.finalize()
-
-    @torch.no_grad()
-    def load_checkpoint(self, sd: dict[str, torch.Tensor]) -> None:
-        want = dict(self._checkpoint_tensors())
-        missing, extra = sorted(want.keys() - sd.keys()), sorted(sd.keys() - want.keys())
-        if missing or extra:
-            raise KeyError(f"checkpoint does not fit the configuration: missing {missing[:6]}, unknown {extra[:6]}")
-        for name, dst in want.items():
-            if tuple(sd[name].shape) != tuple(dst.shape):
-                raise ValueError(f"{name}: shape {tuple(sd[name].shape)}, the configuration says {tuple(dst.shape)}")
-            dst.copy_(sd[name])
-        for l in self.layers:
-            l.mixer.finalize()
-
-    @torch.no_grad()
-    def to_checkpoint(self) -> dict[str, torch.Tensor]:
-        return {name: t.detach().to(torch.bfloat16).contiguous() for name, t in self._checkpoint_tensors()}
 
     # ---------------------------------------------------------------- serving interface of the engine
     def cache_spec(self):
         from ..inference.kv_cache import CacheSpec
         return CacheSpec([l.mixer.cache_entry() for l in self.layers])
-
-    def _side_stream(self) -> "torch.cuda.Stream":
-        if self._side is None:
-            self._side = torch.cuda.Stream(device=self.embed.device)
-        return self._side
 
     @torch.no_grad()
     def serve(self, batch, cache, observe=None) -> torch.Tensor:
@@ -544,18 +507,6 @@ class KabulixForCausalLM(nn.Module):
     def logits(self, hidden: torch.Tensor) -> torch.Tensor:
         return gemm.serve_linear(hidden, self.embed, torch.float32)
 
-    @torch.no_grad()
-    def forward(self, input_ids: torch.Tensor) -> torch.Tensor:
-        """fp32 logits [B, S, vocab] of whole sequences (a throw-away cache; inference only)."""
-        from ..inference.batch import HostBatch, StepEntry
-        from ..inference.kv_cache import PagedKVCache
-        B, S = input_ids.shape
-        bs = 64
-        cache = PagedKVCache(len(self.layers), B * -(-S // bs), bs, dtype=self.embed.dtype, device=self.embed.device,
-                             spec=self.cache_spec())
-        host = HostBatch(cache, [StepEntry(b, row, list(range(S))) for b, row in enumerate(input_ids.tolist())])
-        return self.logits(self.serve(host.to_device(self.embed.device), cache)).view(B, S, -1)
-
 
 def build_model(config, dtype=torch.bfloat16, device=None, seed: int | None = None) -> KabulixForCausalLM:
     """Randomly initialised model of a preset name, a config.json dictionary or a KabulixConfig."""
@@ -563,26 +514,8 @@ def build_model(config, dtype=torch.bfloat16, device=None, seed: int | None = No
         config = PRESETS[config]
     elif isinstance(config, dict):
         config = KabulixConfig.from_dict(config)
-    model = _empty(config, dtype, device)
-    model.reset_parameters(0 if seed is None else seed)
-    return model
-
-
-def _empty(config: KabulixConfig, dtype, device) -> KabulixForCausalLM:
-    device = torch.device(device or "cpu")
-    if device.type == "cuda":
-        from ..ops import _lib
-        _lib.prepare(list(KabulixForCausalLM.LIBRARIES))
-    prev = torch.get_default_dtype()
-    torch.set_default_dtype(dtype)
-    try:
-        with torch.device(device):
-            return KabulixForCausalLM(config).eval()
-    finally:
-        torch.set_default_dtype(prev)
+    return KabulixForCausalLM.random(config, dtype, device, seed)
 
 
 def load_model(config: dict, state_dict: dict[str, torch.Tensor], dtype=torch.bfloat16, device=None) -> KabulixForCausalLM:
-    model = _empty(KabulixConfig.from_dict(config), dtype, device)
-    model.load_checkpoint(state_dict)
-    return model
+    return KabulixForCausalLM.from_checkpoint(KabulixConfig.from_dict(config), state_dict, dtype, device)

@@ -25,6 +25,7 @@ import torch.nn as nn
 from ..ops import gemm, grouped, latent_attention as latent, recurrent, rope, stream, window_attention as window
 from ..ops.recurrent import DeltaShape, DeltaWeights, WkvShape, WkvWeights
 from ..ops.window_attention import WindowShape
+from .served import ServedDecoder, fp32_param, require, up8, weight_param
 
 SHIFTS = "rkvgw"            # inputs of a WKV mixer, in the order of its mixes
 
@@ -89,7 +90,7 @@ class VibepelConfig:
             if l["type"] == "wkv":
                 w1 = (shapes or {}).get(f"l{i}.mix.w1")
                 mixer = WkvConfig(WkvShape(m["heads"], m["dim"], W), w1[0] if w1 else m.get("decay_rank", 32))
-                _require(m["dim"] <= recurrent.MAX_HEAD, i, f"WKV heads of up to {recurrent.MAX_HEAD} dimensions")
+                require(m["dim"] <= recurrent.MAX_HEAD, i, f"WKV heads of up to {recurrent.MAX_HEAD} dimensions")
             elif l["type"] == "parallel":
                 a, b, r = m["left"], m["right"], m["left"]["rot"]
                 s = r.get("scaling")
@@ -99,11 +100,11 @@ class VibepelConfig:
                     WindowShape(a["heads"], a["kv_heads"], a["dim"], a["vdim"], rot.dims, a["mask"]["size"], float(a["scale"])),
                     rot, DeltaShape(b["heads"], b["kv_heads"], b["dim"], b["vdim"], b["conv"]),
                     float(m["left_scale"]), float(m["right_scale"]))
-                _require(rot.dims % 2 == 0 and rot.dims <= a["dim"], i, "an even number of rotated dimensions inside a head")
-                _require(a["heads"] % a["kv_heads"] == 0 and b["heads"] % b["kv_heads"] == 0, i, "whole head groups")
-                _require(a["mask"]["size"] > 0 and b["conv"] > 0, i, "a window and a convolution of at least one token")
-                _require(max(b["dim"], b["vdim"]) <= recurrent.MAX_HEAD, i,
-                         f"delta rule heads of up to {recurrent.MAX_HEAD} dimensions")
+                require(rot.dims % 2 == 0 and rot.dims <= a["dim"], i, "an even number of rotated dimensions inside a head")
+                require(a["heads"] % a["kv_heads"] == 0 and b["heads"] % b["kv_heads"] == 0, i, "whole head groups")
+                require(a["mask"]["size"] > 0 and b["conv"] > 0, i, "a window and a convolution of at least one token")
+                require(max(b["dim"], b["vdim"]) <= recurrent.MAX_HEAD, i,
+                        f"delta rule heads of up to {recurrent.MAX_HEAD} dimensions")
             else:
                 raise ValueError(f"layer {i}: unknown mixer {l['type']!r}")
             f = l.get("mlp")
@@ -134,11 +135,6 @@ class VibepelConfig:
                 "embedding": {"scale": self.embed_scale}, "logit_softcap": self.logit_softcap, "layers": layers}
 
 
-def _require(ok: bool, layer: int, what: str) -> None:
-    if not ok:
-        raise ValueError(f"layer {layer}: needs {what}")
-
-
 def pattern_config(layers: int, vocab: int, width: int, heads: int, kv_heads: int, dim: int, window: int, ff: int,
                    delta_heads: int, delta_kv_heads: int, delta_dim: int, delta_vdim: int, wkv_heads: int, wkv_dim: int,
                    wkv_every: int = 4, taps: int = 4, rot_dims: int | None = None, rope_base: float = 10000.0,
@@ -160,18 +156,6 @@ PRESETS: dict[str, VibepelConfig] = {
                                  delta_heads=16, delta_kv_heads=8, delta_dim=128, delta_vdim=128, wkv_heads=32, wkv_dim=64,
                                  rot_dims=64, rope_base=500000.0),
 }
-
-
-def _fp32(*shape) -> nn.Parameter:
-    return nn.Parameter(torch.empty(*shape, dtype=torch.float32), requires_grad=False)
-
-
-def _weight(*shape) -> nn.Parameter:
-    return nn.Parameter(torch.zeros(*shape), requires_grad=False)     # padding rows and columns stay zero
-
-
-def _up8(n: int) -> int:
-    return -(-n // 8) * 8
 
 
 @dataclass
@@ -199,10 +183,10 @@ class ParallelMixer(nn.Module):
         self.cfg, self.eps = cfg, eps
         a, b = cfg.left, cfg.right
         self.right_at = a.q_width + a.kv_width
-        self.w_in = _weight(_up8(self.right_at + b.proj_width), width)
-        self.w_o = _weight(width, _up8(a.out_width + b.out_width))
-        self.q_norm, self.k_norm = _fp32(a.dim), _fp32(a.dim)
-        self.conv, self.A_log, self.dt_bias, self.norm = _fp32(b.channels, b.taps), _fp32(b.heads), _fp32(b.heads), _fp32(b.vdim)
+        self.w_in = weight_param(up8(self.right_at + b.proj_width), width)
+        self.w_o = weight_param(width, up8(a.out_width + b.out_width))
+        self.q_norm, self.k_norm = fp32_param(a.dim), fp32_param(a.dim)
+        self.conv, self.A_log, self.dt_bias, self.norm = fp32_param(b.channels, b.taps), fp32_param(b.heads), fp32_param(b.heads), fp32_param(b.vdim)
         self.register_buffer("inv_freq", cfg.rot.inv_freq().to(self.q_norm.device), persistent=False)
 
     def tensors(self):
@@ -277,11 +261,11 @@ class WkvMixer(nn.Module):
         super().__init__()
         self.cfg, self.eps = cfg, eps
         s = cfg.shape
-        self.mu = _fp32(len(SHIFTS), width)
-        self.w_rkvg = _weight(4, s.inner, width)
-        self.w1, self.w2 = _weight(cfg.decay_rank, width), _weight(s.inner, cfg.decay_rank)
-        self.w_o = _weight(width, s.inner)
-        self.w0, self.u, self.norm = _fp32(s.inner), _fp32(s.heads, s.dim), _fp32(s.inner)
+        self.mu = fp32_param(len(SHIFTS), width)
+        self.w_rkvg = weight_param(4, s.inner, width)
+        self.w1, self.w2 = weight_param(cfg.decay_rank, width), weight_param(s.inner, cfg.decay_rank)
+        self.w_o = weight_param(width, s.inner)
+        self.w0, self.u, self.norm = fp32_param(s.inner), fp32_param(s.heads, s.dim), fp32_param(s.inner)
 
     def tensors(self):
         for i, name in enumerate(SHIFTS):
@@ -320,17 +304,16 @@ class VibepelLayer(nn.Module):
         super().__init__()
         W, l = cfg.hidden_size, cfg.layers[index]
         self.mixer = (WkvMixer if isinstance(l.mixer, WkvConfig) else ParallelMixer)(l.mixer, W, cfg.eps)
-        self.norm1 = _fp32(W)
+        self.norm1 = fp32_param(W)
         self.ff = l.ff
         if l.ff is not None:
-            self.norm2, self.w_up, self.w_down = _fp32(W), _weight(l.ff, W), _weight(W, l.ff)
+            self.norm2, self.w_up, self.w_down = fp32_param(W), weight_param(l.ff, W), weight_param(W, l.ff)
 
     def feed_forward(self, h: torch.Tensor) -> torch.Tensor:
         return gemm.serve_linear(gemm.serve_linear(h, self.w_up, act=grouped.ACT_RELU_SQUARED), self.w_down)
 
 
-class VibepelForCausalLM(nn.Module):
-    # libraries `serve` needs (compiled together at the first use)
+class VibepelForCausalLM(ServedDecoder):
     LIBRARIES = ("stream", "window", "recurrent", "latent", "latent_prefill", "skinny", "gemm")
 
     def __init__(self, cfg: VibepelConfig):
@@ -338,8 +321,7 @@ class VibepelForCausalLM(nn.Module):
         self.config = cfg
         self.embed = nn.Parameter(torch.empty(cfg.vocab_size, cfg.hidden_size), requires_grad=False)
         self.layers = nn.ModuleList(VibepelLayer(cfg, i) for i in range(cfg.num_hidden_layers))
-        self.final_norm = _fp32(cfg.hidden_size)
-        self._side = None                 # stream of the delta rule in captured decode steps
+        self.final_norm = fp32_param(cfg.hidden_size)
 
     # ---------------------------------------------------------------- weights
     def _checkpoint_tensors(self):
@@ -378,30 +360,10 @@ class VibepelForCausalLM(nn.Module):
             else:
                 p.normal_(0.0, 0.5 if leaf in ("u", "conv") else 1.0 / math.sqrt(p.shape[-1]), generator=gen)
 
-    @torch.no_grad()
-    def load_checkpoint(self, sd: dict[str, torch.Tensor]) -> None:
-        want = dict(self._checkpoint_tensors())
-        missing, extra = sorted(want.keys() - sd.keys()), sorted(sd.keys() - want.keys())
-        if missing or extra:
-            raise KeyError(f"checkpoint does not fit the configuration: missing {missing[:6]}, unknown {extra[:6]}")
-        for name, dst in want.items():
-            if tuple(sd[name].shape) != tuple(dst.shape):
-                raise ValueError(f"{name}: shape {tuple(sd[name].shape)}, the configuration says {tuple(dst.shape)}")
-            dst.copy_(sd[name])
-
-    @torch.no_grad()
-    def to_checkpoint(self) -> dict[str, torch.Tensor]:
-        return {name: t.detach().to(torch.bfloat16).contiguous() for name, t in self._checkpoint_tensors()}
-
     # ---------------------------------------------------------------- serving interface of the engine
     def cache_spec(self):
         from ..inference.kv_cache import CacheSpec
         return CacheSpec([l.mixer.cache_entry() for l in self.layers], [l.mixer.state_width for l in self.layers])
-
-    def _side_stream(self) -> "torch.cuda.Stream":
-        if self._side is None:
-            self._side = torch.cuda.Stream(device=self.embed.device)
-        return self._side
 
     @torch.no_grad()
     def serve(self, batch, cache, observe=None) -> torch.Tensor:
@@ -427,18 +389,6 @@ class VibepelForCausalLM(nn.Module):
     def logits(self, hidden: torch.Tensor) -> torch.Tensor:
         return gemm.serve_linear(hidden, self.embed, torch.float32, grouped.ACT_SOFTCAP, self.config.logit_softcap)
 
-    @torch.no_grad()
-    def forward(self, input_ids: torch.Tensor) -> torch.Tensor:
-        """fp32 logits [B, S, vocab] of whole sequences (a throw-away cache; inference only)."""
-        from ..inference.batch import HostBatch, StepEntry
-        from ..inference.kv_cache import PagedKVCache
-        B, S = input_ids.shape
-        bs = 64
-        cache = PagedKVCache(len(self.layers), B * -(-S // bs), bs, dtype=self.embed.dtype, device=self.embed.device,
-                             spec=self.cache_spec(), state_slots=B)
-        host = HostBatch(cache, [StepEntry(b, row, list(range(S))) for b, row in enumerate(input_ids.tolist())])
-        return self.logits(self.serve(host.to_device(self.embed.device), cache)).view(B, S, -1)
-
 
 def build_model(config, dtype=torch.bfloat16, device=None, seed: int | None = None) -> VibepelForCausalLM:
     """Randomly initialised model of a preset name, a config.json dictionary or a VibepelConfig."""
@@ -446,26 +396,8 @@ def build_model(config, dtype=torch.bfloat16, device=None, seed: int | None = No
         config = PRESETS[config]
     elif isinstance(config, dict):
         config = VibepelConfig.from_dict(config)
-    model = _empty(config, dtype, device)
-    model.reset_parameters(0 if seed is None else seed)
-    return model
-
-
-def _empty(config: VibepelConfig, dtype, device) -> VibepelForCausalLM:
-    device = torch.device(device or "cpu")
-    if device.type == "cuda":
-        from ..ops import _lib
-        _lib.prepare(list(VibepelForCausalLM.LIBRARIES))
-    prev = torch.get_default_dtype()
-    torch.set_default_dtype(dtype)
-    try:
-        with torch.device(device):
-            return VibepelForCausalLM(config).eval()
-    finally:
-        torch.set_default_dtype(prev)
+    return VibepelForCausalLM.random(config, dtype, device, seed)
 
 
 def load_model(config: dict, state_dict: dict[str, torch.Tensor], dtype=torch.bfloat16, device=None) -> VibepelForCausalLM:
-    model = _empty(VibepelConfig.from_dict(config, {k: tuple(v.shape) for k, v in state_dict.items()}), dtype, device)
-    model.load_checkpoint(state_dict)
-    return model
+    return VibepelForCausalLM.from_checkpoint(VibepelConfig.from_dict(config, {k: tuple(v.shape) for k, v in state_dict.items()}), state_dict, dtype, device)
