@@ -94,14 +94,27 @@ __device__ __forceinline__ float2 unpack_bf16x2(uint32_t v) {
   return __bfloat1622float2(b);
 }
 
-// Activations that a product may apply to its result: 1 squared ReLU, 2 tanh, 3 soft cap c * tanh(v / c)
-__device__ __forceinline__ float product_act(float v, int act, float cap) {
+// a v^2 + v / 2 for v > 0, b (e^v - 1 - v) + v / 2 for v <= 0.  Near zero the bracket is a power series: the difference
+// would cancel.
+template <bool FAST> __device__ __forceinline__ float xielu(float v, float a, float b) {
+  const float n = fminf(v, 0.f);
+  const float series = n * n * (0.5f + n * (1.f / 6.f + n * (1.f / 24.f + n * (1.f / 120.f + n * (1.f / 720.f)))));
+  const float left = n > -0.25f ? series : (FAST ? __expf(n) : expf(n)) - 1.f - n;
+  const float p = fmaxf(v, 0.f);
+  return a * p * p + b * left + 0.5f * v;
+}
+
+// Activations that a product may apply to its result: 1 squared ReLU, 2 tanh, 3 soft cap a * tanh(v / a), 4 a * v,
+// 5 xielu(v; a, b).  `FAST`: for results that are rounded to 16 bits.
+template <bool FAST> __device__ __forceinline__ float product_act(float v, int act, float a, float b) {
   if (act == 1) {
     v = fmaxf(v, 0.f);
     return v * v;
   }
   if (act == 2) return tanhf(v);
-  if (act == 3) return cap * tanhf(v / cap);
+  if (act == 3) return a * tanhf(v / a);
+  if (act == 4) return a * v;
+  if (act == 5) return xielu<FAST>(v, a, b);
   return v;
 }
 
@@ -110,13 +123,13 @@ __device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)
 // Factor sigmoid(gate) of an attention result: one gate per head or one per element.
 constexpr int GATE_HEAD = 1, GATE_ELEMENT = 2;
 
-// Gated products: act 4 is silu(g) * u, act 5 the tanh form of gelu(g) * u, both written as g * sigmoid(y) * u.  `FAST`:
+// Gated products: act 6 is silu(g) * u, act 7 the tanh form of gelu(g) * u, both written as g * sigmoid(y) * u.  `FAST`:
 // for results that are rounded to 16 bits.  Their weights interleave GLU_BLOCK gate rows with the GLU_BLOCK up rows of
 // the same outputs.
 constexpr int GLU_BLOCK = 16;
-constexpr int ACT_FIRST_GLU = 4, ACT_LAST_GLU = 5;
+constexpr int ACT_FIRST_GLU = 6, ACT_LAST_GLU = 7;
 template <bool FAST> __device__ __forceinline__ float glu_act(float g, float u, int act) {
-  const float y = act == 5 ? 1.5957691216057308f * (g + 0.044715f * g * g * g) : g;     // 2 sqrt(2 / pi)
+  const float y = act == 7 ? 1.5957691216057308f * (g + 0.044715f * g * g * g) : g;     // 2 sqrt(2 / pi)
   return FAST ? __fdividef(g * u, 1.f + __expf(-y)) : g / (1.f + expf(-y)) * u;
 }
 

@@ -42,7 +42,8 @@ struct GemmParams {
   int group_rows;           // MODE 1: rows (K-major B) or K extent (MN-major B) of one expert inside the stacked B
   int num_groups;           // MODE 2: E; C is [E][M][ldc]
   int act;                  // epilogue activation of common.cuh product_act or glu_act (modes 0 and 1; 0: none)
-  float act_cap;
+  float act_a, act_b;       // its constants
+  int act_cols;             // columns it applies to, from the first; a multiple of 32 unless all
 };
 
 // 32 accumulator columns of a gated product = 16 gates and the 16 factors of the same outputs: 16 results.
@@ -59,16 +60,24 @@ __device__ __forceinline__ void gemm_store_glu(const GemmParams& p, const uint32
 }
 
 // product_act of 32 accumulators; one uniform branch per kind, so that the common kinds stay short
-__device__ __forceinline__ void gemm_activate(uint32_t* r, int act, float cap) {
-  if (act == 1) {
+__device__ __forceinline__ void gemm_activate(const GemmParams& p, uint32_t* r, int col0) {
+  if (col0 >= p.act_cols) return;
+  const float a = p.act_a;
+  if (p.act == 1) {
 #pragma unroll
-    for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(product_act(__uint_as_float(r[j]), 1, cap));
+    for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(product_act<true>(__uint_as_float(r[j]), 1, a, 0.f));
+  } else if (p.act == 4) {
+#pragma unroll
+    for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(a * __uint_as_float(r[j]));
+  } else if (p.act == 5) {
+#pragma unroll
+    for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(xielu<true>(__uint_as_float(r[j]), a, p.act_b));
   } else {
 #pragma unroll
     for (int j = 0; j < 32; ++j) {
       const float v = __uint_as_float(r[j]);
-      const float t = tanhf(act == 3 ? v / cap : v);
-      r[j] = __float_as_uint(act == 3 ? cap * t : t);
+      const float t = tanhf(p.act == 3 ? v / a : v);
+      r[j] = __float_as_uint(p.act == 3 ? a * t : t);
     }
   }
 }
@@ -352,7 +361,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
           if (row < p.M && col0 < p.N) gemm_store_glu(p, r, ti.c_row0 + row, col0);
           continue;
         }
-        if (MODE != 2 && p.act != 0) gemm_activate(r, p.act, p.act_cap);
+        if (MODE != 2 && p.act != 0) gemm_activate(p, r, col0);
         if (row < p.M && col0 < p.N) gemm_store_chunk(p, r, ti.c_row0 + row, col0);
       }
       tc_fence_before_sync();
@@ -519,7 +528,7 @@ gemm_bf16_2cta_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_cons
           if (row < p.M && col0 < p.N) gemm_store_glu(p, r, static_cast<size_t>(row), col0);
           continue;
         }
-        if (p.act != 0) gemm_activate(r, p.act, p.act_cap);
+        if (p.act != 0) gemm_activate(p, r, col0);
         if (row < p.M && col0 < p.N) gemm_store_chunk(p, r, static_cast<size_t>(row), col0);
       }
       tc_fence_before_sync();
@@ -594,15 +603,16 @@ TS_DEFINE_ERROR_API(ts_gemm)
 //   out_fp32: C is fp32 (else bf16); accumulate: add into the existing C.
 //   bn: N tile (256, 128 or 64; 0 = choose).
 // Leading dimensions are in elements and must keep rows 16-byte aligned. Returns 0 on success.
-//   act: activation of the result (common.cuh product_act; C must not accumulate then).  The gated ones (glu_act) take B
+//   act: activation of the first act_cols columns of the result (common.cuh product_act with the constants act_a, act_b; C must
+//   not accumulate then); act_cols is N or a multiple of 32.  The gated ones (glu_act) take B
 //   with gate and up rows in alternating blocks of GLU_BLOCK and write N / 2 columns.
 extern "C" int ts_gemm_bf16_act(const void* A, const void* B, void* C, int M, int N, int K, int lda, int ldb, int ldc,
                                 int a_mn, int b_mn, int out_fp32, int accumulate, float alpha, int bn, int act,
-                                float act_cap, void* stream) {
+                                float act_a, float act_b, int act_cols, void* stream) {
   using namespace ts;
   if (M <= 0 || N <= 0 || K <= 0) return -10;
-  if (act != 0 && (act < 0 || act > ACT_LAST_GLU || accumulate || alpha != 1.f || (act == 3 && !(act_cap > 0.f)) ||
-                   !glu_ok(act, C, N, ldc, out_fp32)))
+  if (act != 0 && (act < 0 || act > ACT_LAST_GLU || accumulate || alpha != 1.f || (act == 3 && !(act_a > 0.f)) || act_cols < 0 ||
+                   (act_cols < N && (act_cols % 32 || act >= ACT_FIRST_GLU)) || !glu_ok(act, C, N, ldc, out_fp32)))
     return -13;
   if (bn == 0) {
     // prefer the widest tile that still gives every SM work
@@ -634,7 +644,7 @@ extern "C" int ts_gemm_bf16_act(const void* A, const void* B, void* C, int M, in
   p.num_n_tiles = (N + bn - 1) / bn;
   p.k_blocks = (K + GEMM_BK - 1) / GEMM_BK;
   p.tile_expert = nullptr; p.seg_start = nullptr; p.group_rows = 0; p.num_groups = 1; p.act = act;
-  p.act_cap = act_cap;
+  p.act_a = act_a; p.act_b = act_b; p.act_cols = act_cols;
   p.c_bytes = (static_cast<size_t>(M - 1) * ldc + result_cols(act, N)) * (out_fp32 ? 4 : 2);
 #ifdef TS_DEBUG
   // test hook of the debug build: pretend C ends `TS_DEBUG_SHRINK_C_ROWS` rows early, so that the bounds check (and
@@ -653,7 +663,7 @@ extern "C" int ts_gemm_bf16_act(const void* A, const void* B, void* C, int M, in
 
 extern "C" int ts_gemm_bf16(const void* A, const void* B, void* C, int M, int N, int K, int lda, int ldb, int ldc,
                             int a_mn, int b_mn, int out_fp32, int accumulate, float alpha, int bn, void* stream) {
-  return ts_gemm_bf16_act(A, B, C, M, N, K, lda, ldb, ldc, a_mn, b_mn, out_fp32, accumulate, alpha, bn, 0, 0.f, stream);
+  return ts_gemm_bf16_act(A, B, C, M, N, K, lda, ldb, ldc, a_mn, b_mn, out_fp32, accumulate, alpha, bn, 0, 0.f, 0.f, N, stream);
 }
 
 // Grouped GEMM over an expert-sorted token buffer whose per-expert segments start on 128-row boundaries.
@@ -662,7 +672,7 @@ extern "C" int ts_gemm_bf16(const void* A, const void* B, void* C, int M, int N,
 //   mode 2 (wgrad): C[e][M][N] = sum over rows r in [seg_start[e], seg_start[e+1]) of A[r][m] * B[r][n]; both operands
 //     MN-major (a_mn = b_mn = 1), K = P.  An empty segment gives a zero slab (or leaves C alone when accumulating).
 // `groups` is the device int32 array tile_expert (mode 1, ceil(P/128) entries) or seg_start (mode 2, E + 1 entries).
-// `act` (mode 1): 1 applies max(v, 0)^2 to the product in the epilogue, 4 and 5 are the gated products (as above; C must
+// `act` (mode 1): 1 applies max(v, 0)^2 to the product in the epilogue, 6 and 7 are the gated products (as above; C must
 // not accumulate then).
 // Serves the grouped expert GEMMs of data_pipeline/trainer/kernels/moe_kernels.py:219-785.
 extern "C" int ts_gemm_grouped_bf16_act(const void* A, const void* B, void* C, int mode, int M, int N, int K, int lda,
@@ -672,7 +682,7 @@ extern "C" int ts_gemm_grouped_bf16_act(const void* A, const void* B, void* C, i
   if (M <= 0 || N <= 0 || K <= 0 || num_groups <= 0 || groups == nullptr) return -10;
   // experts stacked along K (b_mn) need whole K blocks; with K-major B the tail of K is zero-filled by the loads
   if (mode == 1 && (a_mn != 0 || (b_mn && K % GEMM_BK != 0))) return -12;
-  if (act != 0 && (mode != 1 || (act != 1 && act != 4 && act != 5) || accumulate || alpha != 1.f || out_fp32 ||
+  if (act != 0 && (mode != 1 || (act != 1 && act < ACT_FIRST_GLU) || act > ACT_LAST_GLU || accumulate || alpha != 1.f || out_fp32 ||
                    !glu_ok(act, C, N, ldc, out_fp32)))
     return -13;
   if (mode == 2 && (a_mn != 1 || b_mn != 1)) return -12;
@@ -701,7 +711,7 @@ extern "C" int ts_gemm_grouped_bf16_act(const void* A, const void* B, void* C, i
   p.seg_start = (mode == 2) ? groups : nullptr;
   p.group_rows = b_mn ? K : N;
   p.num_groups = num_groups;
-  p.act = act; p.act_cap = 0.f;
+  p.act = act; p.act_a = p.act_b = 0.f; p.act_cols = N;
   p.c_bytes = (static_cast<size_t>((mode == 2 ? num_groups : 1)) * M - 1) * ldc * (out_fp32 ? 4 : 2) +
               static_cast<size_t>(result_cols(act, N)) * (out_fp32 ? 4 : 2);
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);

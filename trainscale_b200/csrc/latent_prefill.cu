@@ -11,7 +11,9 @@
 //                64-column blocks (128-byte swizzle); 3-D maps (column, head, token) zero-fill columns past the head's
 //                size, so heads of any multiple of eight columns use the same code
 //   warp 1       MMA issuer: S_t = Q_t K^T over the unrotated, then the rotated columns; O_t += P_t V, P_t from TMEM
-//   warps 2..9   softmax: one thread per query row; scores, running max and sum in fp32
+//   warps 2..9   softmax: one thread per query row; scores, running max and sum in fp32.  Or (`SIG`) weights that are not
+//                normalized: sigmoid(score + a number per head - a slope per head times the distance), so there is no running
+//                maximum, no rescaling and no sum
 // Queries are the LAST Lq of the sequence's Lk keys.  A query sees the `window` keys up to its own, or those of its chunk of
 // `window` keys (the first key row then lies on a chunk's border), and besides the first `keep` key rows; these are the
 // sequence's first positions, which a portion's caller may have put right in front of its window.  Key tiles that no row
@@ -51,6 +53,12 @@ __device__ __forceinline__ uint64_t add_f32x2(uint64_t a, uint64_t b) {
   return d;
 }
 
+__device__ __forceinline__ float fast_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 struct LatentPrefillParams {
   const int* cu_q;                       // [sequences + 1] query rows
   const int* cu_k;                       // [sequences + 1] key rows
@@ -64,6 +72,8 @@ struct LatentPrefillParams {
   const __nv_bfloat16* gate;             // [query rows][gate_ld] (nullptr: none)
   long long gate_ld;
   int gate_mode;                         // GATE_HEAD: column h, GATE_ELEMENT: column h * vdim + c
+  const float* slopes;                   // SIG: [H] (nullptr: zeros)
+  const float* add;                      // SIG: [H] (nullptr: zeros)
   float scale_log2;
   float o_scale;                         // factor of the result
   __nv_bfloat16* o;                      // [rows][o_stride], head h at column h * vdim
@@ -75,6 +85,7 @@ __device__ __forceinline__ int window_first(const LatentPrefillParams& p, int c)
   return p.chunked ? c / p.window * p.window : max(0, c - p.window + 1);
 }
 
+template <bool SIG>
 __global__ void __launch_bounds__(LP_THREADS, 1)
 latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_constant__ CUtensorMap tmQr,
                       const __grid_constant__ CUtensorMap tmKn, const __grid_constant__ CUtensorMap tmKr,
@@ -237,6 +248,8 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
     const int limit = min(Lk - 1, row + off);          // last visible key
     const int lo = window_first(p, row + off);         // first key of the window
     const int lo_last = window_first(p, r0[t] + 127 + off);
+    constexpr float LOG2E = 1.4426950408889634f;
+    const float slope = SIG && p.slopes ? p.slopes[h] * LOG2E : 0.f, add = SIG && p.add ? p.add[h] * LOG2E : 0.f;
     for (int i = 0; i < nt && alive; ++i) {
       if (!works_on(t, i)) continue;
       if (!mbar_wait(&s_full[t], worked(t, i) & 1u, alive, 600)) break;
@@ -247,6 +260,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
 #pragma unroll
       for (int c = 0; c < 4; ++c) tmem_ld_32x32b_x32(t_s + c * 32, v + c * 32);
       tc_wait_ld();
+      uint32_t seen[4] = {0xffffffffu, 0xffffffffu, 0xffffffffu, 0xffffffffu};
       if (need_mask) {
         // visible columns of the tile are [lo - c0, limit - c0] and the kept ones [0, keep - c0): one bit per column, a word
         // per 32
@@ -258,10 +272,45 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
           if (s0 > 0) bits &= 0xffffffffu << (s0 & 31);
           if (kc > c * 32) bits |= kc >= c * 32 + 32 ? 0xffffffffu : (1u << (kc - c * 32)) - 1u;
           if (s1 < 31) bits &= s1 < 0 ? 0u : 0xffffffffu >> (31 - s1);
+          if (SIG) {
+            seen[c] = bits;
+          } else {
 #pragma unroll
-          for (int j = 0; j < 32; ++j)
-            if (!(bits & (1u << j))) v[c * 32 + j] = 0xff800000u;
+            for (int j = 0; j < 32; ++j)
+              if (!(bits & (1u << j))) v[c * 32 + j] = 0xff800000u;
+          }
         }
+      }
+      if (SIG) {
+        // weight 1 / (1 + 2^e), e = -(score in powers of two); two columns share a reciprocal: 1 / d0 = d1 / (d0 d1), with e
+        // held below 63 so that the product stays finite
+        const float base = slope * static_cast<float>(row + off - c0) - add;
+        const uint64_t nsc = pack_f32x2(-sc, -sc), nsl = pack_f32x2(-slope, -slope), bs = pack_f32x2(base, base);
+        const uint64_t one = pack_f32x2(1.f, 1.f);
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          uint32_t pk[16];
+#pragma unroll
+          for (int j = 0; j < 32; j += 2) {
+            const int col = c * 32 + j;
+            const uint64_t b2 = fma_f32x2(pack_f32x2(static_cast<float>(col), static_cast<float>(col + 1)), nsl, bs);
+            const float2 e = unpack_f32x2(fma_f32x2(pack_f32x2(__uint_as_float(v[col]), __uint_as_float(v[col + 1])), nsc, b2));
+            const float2 d = unpack_f32x2(add_f32x2(pack_f32x2(fast_ex2(fminf(e.x, 63.f)), fast_ex2(fminf(e.y, 63.f))), one));
+            const float r = fast_rcp(d.x * d.y);
+            pk[j >> 1] = pack_bf16x2(d.y * r, d.x * r);
+          }
+          if (need_mask) {
+#pragma unroll
+            for (int j = 0; j < 32; j += 2)
+              pk[j >> 1] &= ((seen[c] >> j & 1u) ? 0xffffu : 0u) | ((seen[c] >> (j + 1) & 1u) ? 0xffff0000u : 0u);
+          }
+          tmem_st_32x32b_x16(t_s + c * 16, pk);
+        }
+        tc_wait_st();
+        tc_fence_before_sync();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&p_full[t]);
+        continue;
       }
       float mx0 = __uint_as_float(v[0]), mx1 = __uint_as_float(v[1]), mx2 = __uint_as_float(v[2]), mx3 = __uint_as_float(v[3]);
 #pragma unroll
@@ -318,7 +367,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
     }
     if (nt > 0 && alive && mbar_wait(&o_full[t], 0, alive, 601)) {
       tc_fence_after_sync();
-      float inv = l > 0.f ? p.o_scale / l : 0.f;
+      float inv = SIG ? p.o_scale : (l > 0.f ? p.o_scale / l : 0.f);
       const bool valid = row < Lq;
       const __nv_bfloat16* gate = p.gate ? p.gate + (q_start + row) * p.gate_ld + (p.gate_mode == GATE_HEAD ? h : h * p.vdim) : nullptr;
       if (valid && gate && p.gate_mode == GATE_HEAD) inv *= sigmoid(__bfloat162float(*gate));
@@ -393,6 +442,7 @@ static bool gate_ok(const void* gate, long long ld, int mode, int vdim) {
 }
 
 // Tensor maps are the caller's; `p` still lacks what follows from the sizes.
+template <bool SIG>
 static int launch_prefill(const CUtensorMap& tQn, const CUtensorMap& tQr, const CUtensorMap& tKn, const CUtensorMap& tKr,
                           const CUtensorMap& tV, const LatentPrefillPlan& pl, LatentPrefillParams p, int dim, int rot,
                           int vdim, int sequences, int max_q, void* stream) {
@@ -401,12 +451,12 @@ static int launch_prefill(const CUtensorMap& tQn, const CUtensorMap& tQr, const 
   p.k_stages = pl.k_stages; p.v_stages = pl.v_stages;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(latent_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+    cudaError_t e = cudaFuncSetAttribute(latent_prefill_kernel<SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
   const dim3 grid((unsigned)(p.H * sequences), (unsigned)((max_q + 255) / 256));
-  latent_prefill_kernel<<<grid, LP_THREADS, pl.smem, reinterpret_cast<cudaStream_t>(stream)>>>(tQn, tQr, tKn, tKr, tV, p);
+  latent_prefill_kernel<SIG><<<grid, LP_THREADS, pl.smem, reinterpret_cast<cudaStream_t>(stream)>>>(tQn, tQr, tKn, tKr, tV, p);
   return (int)cudaGetLastError();
 }
 
@@ -457,20 +507,22 @@ extern "C" int ts_latent_prefill(const void* q, long long q_ld, long long q_rows
   p.gate = reinterpret_cast<const __nv_bfloat16*>(gate); p.gate_ld = gate_ld; p.gate_mode = gate_mode;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.o = reinterpret_cast<__nv_bfloat16*>(out); p.o_stride = o_stride;
-  return launch_prefill(tQn, tQr, tKn, tKr, tV, pl, p, dim, rot, vdim, sequences, max_q, stream);
+  return launch_prefill<false>(tQn, tQr, tKn, tKr, tV, pl, p, dim, rot, vdim, sequences, max_q, stream);
 }
 
 // q: rows [q_rows][q_ld], head h at column h * dim.  k / v: rows [k_rows][kv_ld], key/value head g at columns g * dim and
 // g * vdim.  cu_q / cu_k: [sequences + 1].  window, keep, chunked: which keys a query sees (top of the file).
-// out: [q_rows][o_stride] = o_scale * attention (* sigmoid(gate)).
+// sigmoid: weights sigmoid(score + add[h] - slopes[h] * distance), not normalized (add and slopes: nullptr for zeros; without
+// sigmoid there are none).  out: [q_rows][o_stride] = o_scale * attention (* sigmoid(gate)).
 extern "C" int ts_window_prefill(const void* q, long long q_ld, long long q_rows, const void* k, const void* v,
                                  long long kv_ld, long long k_rows, const int* cu_q, const int* cu_k, int sequences,
                                  int max_q, int H, int G, int dim, int vdim, int window, int keep, int chunked, float scale,
-                                 float o_scale, const void* gate, long long gate_ld, int gate_mode, void* out,
-                                 long long o_stride, void* stream) {
+                                 float o_scale, const float* slopes, const float* add, int sigmoid, const void* gate,
+                                 long long gate_ld, int gate_mode, void* out, long long o_stride, void* stream) {
   if (sequences <= 0 || max_q <= 0) return 0;
   LatentPrefillPlan pl;
   if (H <= 0 || G <= 0 || H % G || window <= 0 || keep < 0 || !(scale > 0.f) || !plan_prefill(dim, 0, vdim, pl)) return -10;
+  if (!sigmoid && (slopes || add)) return -13;
   if (!gate_ok(gate, gate_ld, gate_mode, vdim)) return -12;
   if (q_ld % 8 || kv_ld % 8 || o_stride % 8 || (reinterpret_cast<uintptr_t>(out) & 15u)) return -11;
   CUtensorMap tQ, tK, tV;
@@ -487,5 +539,7 @@ extern "C" int ts_window_prefill(const void* q, long long q_ld, long long q_rows
   p.gate = reinterpret_cast<const __nv_bfloat16*>(gate); p.gate_ld = gate_ld; p.gate_mode = gate_mode;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.o = reinterpret_cast<__nv_bfloat16*>(out); p.o_stride = o_stride;
-  return launch_prefill(tQ, tQ, tK, tK, tV, pl, p, dim, 0, vdim, sequences, max_q, stream);
+  p.slopes = slopes; p.add = add;
+  return sigmoid ? launch_prefill<true>(tQ, tQ, tK, tK, tV, pl, p, dim, 0, vdim, sequences, max_q, stream)
+                 : launch_prefill<false>(tQ, tQ, tK, tK, tV, pl, p, dim, 0, vdim, sequences, max_q, stream);
 }

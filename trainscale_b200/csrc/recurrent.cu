@@ -2,6 +2,7 @@
 //
 //   gated delta rule   S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q        (g, beta one number per head)
 //   WKV                o = (S + diag(u) k v^T)^T r;  S <- diag(w) S + k v^T                (w per key channel)
+//   retention          S <- g S + k v^T;  o = S^T q, q and k rotated by their position     (g one constant per head)
 //
 // Rows are tokens of a flattened batch.  A portion of a prompt runs as: inputs (short convolution, unit norms, gates), a
 // scan over its tokens, the gated norm of the result.  A single decoded row is one launch from projection to gated norm.
@@ -51,6 +52,18 @@ __device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
   uint64_t d;
   asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
   return d;
+}
+template <int VEC> __device__ __forceinline__ void load_vec(const float* p, float (&v)[VEC]) {
+  if (VEC == 4) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    v[0] = a.x; v[VEC > 1 ? 1 : 0] = a.y; v[VEC > 2 ? 2 : 0] = a.z; v[VEC > 3 ? 3 : 0] = a.w;
+  } else {
+    v[0] = *p;
+  }
+}
+template <int VEC> __device__ __forceinline__ void store_vec(float* p, const float (&v)[VEC]) {
+  if (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[VEC > 1 ? 1 : 0], v[VEC > 2 ? 2 : 0], v[VEC > 3 ? 3 : 0]);
+  else *p = v[0];
 }
 __device__ __forceinline__ void cp_async16(void* dst, const void* src, bool valid) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(valid ? 16 : 0) : "memory");
@@ -657,7 +670,8 @@ __global__ void __launch_bounds__(SC_WARPS * 32) wkv_scan_kernel(WkvParams p) {
 //                S8 = gamma_8 S0 + K^T diag(gamma_8 / gamma_j) U
 //   WKV          O = S0^T R~ + A V,         R~_i = r_i gamma_(i-1),  A_ij = sum_d r_id k_jd gamma_(i-1)d / gamma_jd  (j < i)
 //                S8 = diag(gamma_8) S0 + K~^T V,  K~_j = k_j gamma_8 / gamma_j;  A_ii = sum_d r_id u_d k_id
-// T, A and (WKV) R~, K~ depend on the inputs alone and come from a launch over all blocks at once.  Every decay above is a
+//   retention    as WKV with R~_i = q_i g^(i+1), A_ij = g^(i-j) (q_i . k_j)  (j <= i), one decay g^8 for all key rows
+// T, A and (WKV, retention) R~, K~ depend on the inputs alone and come from a launch over all blocks at once.  Every decay above is a
 // product of factors <= 1 formed directly, never a quotient.
 //
 // A warp owns 16 value columns x 8 NT key rows of S^T as MMA accumulators.  The accumulator layout (column g, rows 2t and
@@ -669,6 +683,8 @@ constexpr int BS_BLOCK = 8;                // tokens of a block
 constexpr int BS_TILE = 32;                // tokens staged at a time
 constexpr int BS_COEF = 144;               // delta rule, per block and head: T [8][8], A [8][8], gamma [8], gamma_8 / gamma_j [8]
 constexpr int BS_COEF_WKV = 64;            // WKV: A [8][8] (the decay of the key rows is kept beside it)
+constexpr int BS_COEF_RET = 68;            // retention: A [8][8], decay of the block, padding
+enum { SCAN_WKV = 0, SCAN_DELTA = 1, SCAN_RETENTION = 2 };
 
 struct BlockScanParams {
   const float* q;              // first row, head 0; row stride below
@@ -676,7 +692,7 @@ struct BlockScanParams {
   const void* v;
   long long qk_ld, v_ld;
   int rep;                     // heads per query / key head
-  const float* coef;           // [blocks][H][BS_COEF or BS_COEF_WKV]
+  const float* coef;           // [blocks][H][BS_COEF, BS_COEF_WKV or BS_COEF_RET]
   const float* row_decay;      // WKV: [blocks][H][D]
   float* state;
   long long state_ld;
@@ -732,13 +748,13 @@ __device__ __forceinline__ void zero_acc(float (&c)[3][4]) {
     for (int e = 0; e < 4; ++e) c[i][e] = 0.f;
 }
 
-template <bool DELTA, int NT, int WR, typename TV> struct BlockScan {
+template <int KIND, int NT, int WR, typename TV> struct BlockScan {
   static constexpr int WC = 4 / WR;                    // column groups of a CTA
   static constexpr int NC = 16 * WC;
   static constexpr int DP = 8 * NT * WR;               // key rows, padded
   static constexpr int KS = DP + 4;
   static constexpr int VS = NC + 8;
-  static constexpr int CO = DELTA ? BS_COEF : BS_COEF_WKV + DP;
+  static constexpr int CO = KIND == SCAN_DELTA ? BS_COEF : (KIND == SCAN_WKV ? BS_COEF_WKV + DP : BS_COEF_RET);
   static constexpr int QK = BS_TILE * 2 * KS * 4, VB = BS_TILE * VS * static_cast<int>(sizeof(TV));     // bytes
   static constexpr int STAGE = QK + VB + BS_TILE / BS_BLOCK * CO * 4;
   static constexpr int EX = WR > 1 ? 2 * 4 * 32 * 8 * 4 : 0;      // two blocks' partial products of the four warps
@@ -746,9 +762,10 @@ template <bool DELTA, int NT, int WR, typename TV> struct BlockScan {
 };
 
 // grid (column tiles, H, portions)
-template <bool DELTA, int NT, int WR, typename TV>
+template <int KIND, int NT, int WR, typename TV>
 __global__ void __launch_bounds__(128, 2) block_scan_kernel(BlockScanParams p) {
-  using Z = BlockScan<DELTA, NT, WR, TV>;
+  using Z = BlockScan<KIND, NT, WR, TV>;
+  constexpr bool DELTA = KIND == SCAN_DELTA;
   constexpr int XT = NT < 4 ? NT : 4;
   extern __shared__ __align__(16) uint8_t smb[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
@@ -785,6 +802,8 @@ __global__ void __launch_bounds__(128, 2) block_scan_kernel(BlockScanParams p) {
       const long long at = (block0 + t / BS_BLOCK + b) * p.H + h;
       if (DELTA) {
         cp_async16(co + b * Z::CO + c, in ? p.coef + at * BS_COEF + c : p.coef, in);
+      } else if (KIND == SCAN_RETENTION) {
+        cp_async16(co + b * Z::CO + c, in ? p.coef + at * BS_COEF_RET + c : p.coef, in);
       } else {
         const bool mat = c < BS_COEF_WKV, ok = in && (mat || c - BS_COEF_WKV < p.D);
         cp_async16(co + b * Z::CO + c,
@@ -828,6 +847,7 @@ __global__ void __launch_bounds__(128, 2) block_scan_kernel(BlockScanParams p) {
         rt = *reinterpret_cast<const float2*>(co + 136 + tig * 2);
         g8 = co[128 + 7];
       }
+      if (KIND == SCAN_RETENTION) g8 = co[64];
       float u[4];                                        // v, then U: column g (g + 8), tokens 2t, 2t + 1
       {
         const TV* vv = vt + (b * BS_BLOCK + tig * 2) * Z::VS + wc * 16 + gid;
@@ -908,7 +928,7 @@ __global__ void __launch_bounds__(128, 2) block_scan_kernel(BlockScanParams p) {
           const float* src = kt + tig * 4 * Z::KS + (x0 + x) * 8 + gid;
           kb[x] = SplitB(src[0], src[2 * Z::KS]);
           float (&s4)[4] = S[x0 + x];
-          if (DELTA) {
+          if (KIND != SCAN_WKV) {
 #pragma unroll
             for (int e = 0; e < 4; ++e) s4[e] *= g8;
           } else {
@@ -1107,6 +1127,211 @@ __global__ void __launch_bounds__(128, 3) wkv_blocks_kernel(WkvParams p, float* 
 }
 
 // ---------------------------------------------------------------------------------------------------------
+// retention
+// ---------------------------------------------------------------------------------------------------------
+struct RetentionParams {
+  const void* proj;            // rows [q H x D | k H x D | v H x V | gate H x V]
+  long long ld;
+  const float* angles;         // [rows][cos (rot / 2) | sin (rot / 2)]
+  const float* powers;         // [H][RT_POWERS] g^0, g^1, ...
+  float k_scale, eps;
+  float* state;
+  long long state_ld;
+  const int* row_prev;
+  const int* row_next;
+  const int* cu;               // portions
+  float* o;                    // portions: [rows][H V]
+  void* out;                   // decoding: [rows][out_ld]
+  long long out_ld;
+  int rows, H, D, V, rot;
+};
+constexpr int RT_POWERS = BS_BLOCK + 1;
+
+// coordinate c of a head whose projected row is x, rotated (halves) and scaled
+template <typename T>
+__device__ __forceinline__ float rotated(const T* x, int c, int rot, const float* cs, float scale) {
+  const int half = rot / 2;
+  float v = to_f32(x[c]);
+  if (c < half) v = v * cs[c] - to_f32(x[c + half]) * cs[half + c];
+  else if (c < rot) v = v * cs[c - half] + to_f32(x[c - half]) * cs[c];
+  return v * scale;
+}
+
+// Plain fp32 scan.  grid (ceil(V / 32), H, portions); a warp owns NR key rows of 32 value columns, a lane one column.
+constexpr int RT_TILE = 8;                 // tokens staged at a time
+template <typename T, int NR>
+__global__ void __launch_bounds__(256) retention_scan_kernel(RetentionParams p) {
+  constexpr int DP = NR * 8;
+  __shared__ __align__(16) float qs[RT_TILE][DP], ks[RT_TILE][DP];
+  __shared__ float vs[RT_TILE][32], part[RT_TILE][8][32];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, h = blockIdx.y, col = blockIdx.x * 32 + lane;
+  const int row0 = p.cu[blockIdx.z], n = p.cu[blockIdx.z + 1] - row0, D = p.D, V = p.V;
+  if (n <= 0) return;
+  const int prev = p.row_prev[row0], next = p.row_next[row0 + n - 1];
+  const float g = p.powers[h * RT_POWERS + 1];
+  const long long head = static_cast<long long>(h) * D * V;
+  float S[NR];
+#pragma unroll
+  for (int i = 0; i < NR; ++i) {
+    const int r = warp * NR + i;
+    S[i] = prev >= 0 && r < D && col < V ? p.state[prev * p.state_ld + head + static_cast<long long>(r) * V + col] : 0.f;
+  }
+  for (int t = 0; t < n; t += RT_TILE) {
+    const int m = min(RT_TILE, n - t);
+    for (int i = threadIdx.x; i < RT_TILE * DP; i += 256) {
+      const int tk = i / DP, c = i - tk * DP;
+      const long long row = row0 + t + min(tk, m - 1);
+      const T* x = reinterpret_cast<const T*>(p.proj) + row * p.ld + h * D;
+      const float* cs = p.angles + row * p.rot;
+      qs[tk][c] = c < D ? rotated(x, c, p.rot, cs, 1.f) : 0.f;
+      ks[tk][c] = c < D ? rotated(x + p.H * D, c, p.rot, cs, p.k_scale) : 0.f;
+    }
+    {
+      const T* x = reinterpret_cast<const T*>(p.proj) + (row0 + t + min(warp, m - 1)) * p.ld + 2 * p.H * D + h * V;
+      vs[warp][lane] = col < V ? to_f32(x[col]) : 0.f;
+    }
+    __syncthreads();
+    for (int tk = 0; tk < m; ++tk) {
+      const float v = vs[tk][lane];
+      float acc = 0.f;
+#pragma unroll
+      for (int i = 0; i < NR; i += 4) {
+        const float4 q = *reinterpret_cast<const float4*>(&qs[tk][warp * NR + i]);
+        const float4 k = *reinterpret_cast<const float4*>(&ks[tk][warp * NR + i]);
+        S[i] = g * S[i] + k.x * v;
+        S[i + 1] = g * S[i + 1] + k.y * v;
+        S[i + 2] = g * S[i + 2] + k.z * v;
+        S[i + 3] = g * S[i + 3] + k.w * v;
+        acc += (S[i] * q.x + S[i + 1] * q.y) + (S[i + 2] * q.z + S[i + 3] * q.w);
+      }
+      part[tk][warp][lane] = acc;
+    }
+    __syncthreads();
+    if (warp < m && col < V) {             // warp: token
+      float s = 0.f;
+#pragma unroll
+      for (int w = 0; w < 8; ++w) s += part[warp][w][lane];
+      p.o[static_cast<long long>(row0 + t + warp) * p.H * V + h * V + col] = s;
+    }
+  }
+  if (next >= 0) {
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+      const int r = warp * NR + i;
+      if (r < D && col < V) p.state[next * p.state_ld + head + static_cast<long long>(r) * V + col] = S[i];
+    }
+  }
+}
+
+// R~, K~, A and decay of every block, one warp per (block, head); a lane holds key channels lane, lane + 32, ...
+// grid (blocks of the longest portion, ceil(H / 4), portions); dynamic shared memory [4 warps][q, k][8][D + 1].
+__global__ void __launch_bounds__(128) retention_blocks_kernel(RetentionParams p, float* __restrict__ rt, float* __restrict__ kt,
+                                                               float* __restrict__ coef) {
+  extern __shared__ __align__(16) float smf[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, z = blockIdx.z, h = blockIdx.y * 4 + warp;
+  const int row0 = p.cu[z] + blockIdx.x * BS_BLOCK, n = min(BS_BLOCK, p.cu[z + 1] - row0);
+  if (n <= 0 || h >= p.H) return;
+  const int D = p.D, ds = D + 1;
+  float* qs = smf + warp * 2 * BS_BLOCK * ds;
+  float* ks = qs + BS_BLOCK * ds;
+  const float* pw = p.powers + h * RT_POWERS;
+  const long long at = (first_block(p.cu, z) + blockIdx.x) * p.H + h;
+  for (int c = lane; c < D; c += 32) {
+#pragma unroll
+    for (int i = 0; i < BS_BLOCK; ++i) {
+      float q = 0.f, k = 0.f;
+      if (i < n) {
+        const __nv_bfloat16* x = reinterpret_cast<const __nv_bfloat16*>(p.proj) + (row0 + i) * p.ld + h * D;
+        const float* cs = p.angles + static_cast<long long>(row0 + i) * p.rot;
+        q = rotated(x, c, p.rot, cs, 1.f);
+        k = rotated(x + p.H * D, c, p.rot, cs, p.k_scale);
+        const long long to = static_cast<long long>(row0 + i) * p.H * D + h * D + c;
+        rt[to] = q * pw[i + 1];
+        kt[to] = k * pw[n - 1 - i];
+      }
+      qs[i * ds + c] = q;
+      ks[i * ds + c] = k;
+    }
+  }
+  __syncwarp();
+  const int i = lane >> 2, j = (lane & 3) * 2;           // A[i][j], A[i][j + 1]
+  float d0 = 0.f, d1 = 0.f;
+#pragma unroll 8
+  for (int c = 0; c < D; ++c) {
+    const float q = qs[i * ds + c];
+    d0 += q * ks[j * ds + c];
+    d1 += q * ks[(j + 1) * ds + c];
+  }
+  float* out = coef + at * BS_COEF_RET;
+  *reinterpret_cast<float2*>(out + i * 8 + j) = make_float2(j <= i ? d0 * pw[max(i - j, 0)] : 0.f, j + 1 <= i ? d1 * pw[max(i - j - 1, 0)] : 0.f);
+  if (lane == 0) out[64] = pw[n];
+}
+
+// Single rows: projection -> gated norm, state advanced.  One CTA per (row, head).
+constexpr int RTS_THREADS = 256;
+template <typename T, int VEC>
+__global__ void __launch_bounds__(RTS_THREADS) retention_step_kernel(RetentionParams p) {
+  extern __shared__ __align__(16) float smf[];
+  __shared__ float scratch[32];
+  const int row = blockIdx.x, h = blockIdx.y, D = p.D, V = p.V, tid = threadIdx.x;
+  const int nvec = V / VEC, span = min(nvec, RTS_THREADS), groups = RTS_THREADS / span;
+  float* vs = smf;                               // [V]
+  float* part = vs + (V + 3) / 4 * 4;            // [groups][V]
+  float* qs = part + (groups * V + 3) / 4 * 4;   // [D]
+  float* ks = qs + D;                            // [D]
+  const int prev = p.row_prev[row], next = p.row_next[row];
+  const T* x = reinterpret_cast<const T*>(p.proj) + row * p.ld;
+  const float* cs = p.angles + static_cast<long long>(row) * p.rot;
+  const long long head = static_cast<long long>(h) * D * V;
+  const float* S = prev >= 0 ? p.state + prev * p.state_ld + head : nullptr;
+  float* N = next >= 0 ? p.state + next * p.state_ld + head : nullptr;
+  const float g = p.powers[h * RT_POWERS + 1];
+  for (int c = tid; c < D; c += RTS_THREADS) {
+    qs[c] = rotated(x + h * D, c, p.rot, cs, 1.f);
+    ks[c] = rotated(x + (p.H + h) * D, c, p.rot, cs, p.k_scale);
+  }
+  for (int c = tid; c < V; c += RTS_THREADS) vs[c] = to_f32(x[2 * p.H * D + h * V + c]);
+  __syncthreads();
+  const int grp = tid / span;
+  for (int base = 0; base < nvec; base += span) {
+    const int cv = (base + tid - grp * span) * VEC;
+    if (grp >= groups || cv >= V) continue;
+    float acc[VEC], v[VEC];
+    load_vec<VEC>(vs + cv, v);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
+#pragma unroll 8
+    for (int r = grp; r < D; r += groups) {
+      float st[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) st[e] = 0.f;
+      if (S) load_vec<VEC>(S + static_cast<long long>(r) * V + cv, st);
+      const float k = ks[r], q = qs[r];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        st[e] = g * st[e] + k * v[e];
+        acc[e] += st[e] * q;
+      }
+      if (N) store_vec<VEC>(N + static_cast<long long>(r) * V + cv, st);
+    }
+    store_vec<VEC>(part + grp * V + cv, acc);
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int c = tid; c < V; c += RTS_THREADS) {
+    float s = 0.f;
+    for (int i = 0; i < groups; ++i) s += part[i * V + c];
+    vs[c] = s;
+    ss += s * s;
+  }
+  ss = block_sum(ss, scratch);
+  const float inv = 1.f / sqrtf(ss / static_cast<float>(V) + p.eps);
+  const T* gate = x + 2 * p.H * D + (p.H + h) * V;
+  T* out = reinterpret_cast<T*>(p.out) + row * p.out_ld + h * V;
+  for (int c = tid; c < V; c += RTS_THREADS) out[c] = from_f32<T>(vs[c] * inv * silu(to_f32(gate[c])));
+}
+
+// ---------------------------------------------------------------------------------------------------------
 // norm and gate of a scan's result: out = o / rms_head(o) * w * silu(gate) * scale, one warp per (row, head)
 // ---------------------------------------------------------------------------------------------------------
 template <typename T, int VEC> __device__ __forceinline__ void load_act(const T* p, float (&v)[VEC]) {
@@ -1170,7 +1395,7 @@ gated_norm_kernel(const float* __restrict__ o, const float* __restrict__ w, int 
       if (on && c < V && t0 + k < rows) {
         float r[VEC];
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) r[e] = a[k][i][e] * inv * w[h * w_head + c + e] * act_silu<T>(b[k][i][e]);
+        for (int e = 0; e < VEC; ++e) r[e] = a[k][i][e] * inv * (w ? w[h * w_head + c + e] : 1.f) * act_silu<T>(b[k][i][e]);
         if (VEC == 4 && sizeof(T) == 2) {
           *reinterpret_cast<uint2*>(dst + c) = make_uint2(pack_bf16x2(r[0], r[VEC > 1 ? 1 : 0]), pack_bf16x2(r[VEC > 2 ? 2 : 0], r[VEC > 3 ? 3 : 0]));
         } else {
@@ -1186,19 +1411,6 @@ gated_norm_kernel(const float* __restrict__ o, const float* __restrict__ w, int 
 // single rows: projection -> gated result in one launch, one CTA per (row, head)
 // ---------------------------------------------------------------------------------------------------------
 constexpr int RS_THREADS = 256;
-
-template <int VEC> __device__ __forceinline__ void load_vec(const float* p, float (&v)[VEC]) {
-  if (VEC == 4) {
-    const float4 a = *reinterpret_cast<const float4*>(p);
-    v[0] = a.x; v[VEC > 1 ? 1 : 0] = a.y; v[VEC > 2 ? 2 : 0] = a.z; v[VEC > 3 ? 3 : 0] = a.w;
-  } else {
-    v[0] = *p;
-  }
-}
-template <int VEC> __device__ __forceinline__ void store_vec(float* p, const float (&v)[VEC]) {
-  if (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[VEC > 1 ? 1 : 0], v[VEC > 2 ? 2 : 0], v[VEC > 3 ? 3 : 0]);
-  else *p = v[0];
-}
 
 // NR: key rows of the state a thread keeps in registers between the two passes (0: it reads them twice)
 template <typename T, int VEC, int NR>
@@ -1459,32 +1671,34 @@ template <typename T> static int launch_gated_norm(const float* o, const float* 
   auto grid = [&](int heads_per_warp) { return dim3((rows + GN_ROWS - 1) / GN_ROWS, (H + 8 * heads_per_warp - 1) / (8 * heads_per_warp)); };
   if (vec && V <= 64) gated_norm_kernel<T, 4, 1, 16><<<grid(2), 256, 0, st>>>(o, w, w_head, g, gate_ld, d, out_ld, rows, H, V, eps, scale);
   else if (vec && V <= 128) gated_norm_kernel<T, 4, 1, 32><<<grid(1), 256, 0, st>>>(o, w, w_head, g, gate_ld, d, out_ld, rows, H, V, eps, scale);
-  else if (vec) gated_norm_kernel<T, 4, 2, 32><<<grid(1), 256, 0, st>>>(o, w, w_head, g, gate_ld, d, out_ld, rows, H, V, eps, scale);
+  else if (vec && V <= 256) gated_norm_kernel<T, 4, 2, 32><<<grid(1), 256, 0, st>>>(o, w, w_head, g, gate_ld, d, out_ld, rows, H, V, eps, scale);
+  else if (vec) gated_norm_kernel<T, 4, 4, 32><<<grid(1), 256, 0, st>>>(o, w, w_head, g, gate_ld, d, out_ld, rows, H, V, eps, scale);
+  else if (V > 256) gated_norm_kernel<T, 1, 16, 32><<<grid(1), 256, 0, st>>>(o, w, w_head, g, gate_ld, d, out_ld, rows, H, V, eps, scale);
   else gated_norm_kernel<T, 1, 8, 32><<<grid(1), 256, 0, st>>>(o, w, w_head, g, gate_ld, d, out_ld, rows, H, V, eps, scale);
   return (int)cudaGetLastError();
 }
 
-template <bool DELTA, int NT, int WR, typename TV>
+template <int KIND, int NT, int WR, typename TV>
 static int launch_block_scan(const BlockScanParams& p, int portions, cudaStream_t st) {
-  using Z = BlockScan<DELTA, NT, WR, TV>;
-  if (int e = allow_smem(block_scan_kernel<DELTA, NT, WR, TV>, Z::SMEM)) return e;
-  block_scan_kernel<DELTA, NT, WR, TV><<<dim3((p.V + Z::NC - 1) / Z::NC, p.H, portions), 128, Z::SMEM, st>>>(p);
+  using Z = BlockScan<KIND, NT, WR, TV>;
+  if (int e = allow_smem(block_scan_kernel<KIND, NT, WR, TV>, Z::SMEM)) return e;
+  block_scan_kernel<KIND, NT, WR, TV><<<dim3((p.V + Z::NC - 1) / Z::NC, p.H, portions), 128, Z::SMEM, st>>>(p);
   return (int)cudaGetLastError();
 }
 
 // The key rows of a head stay with one warp when there are (head, portion) pairs for every SM, else they are split over two or
 // four: half the latency of a block for a third more work.
-template <bool DELTA, typename TV> static int dispatch_block_scan(const BlockScanParams& p, int portions, cudaStream_t st) {
+template <int KIND, typename TV> static int dispatch_block_scan(const BlockScanParams& p, int portions, cudaStream_t st) {
   const long long groups = static_cast<long long>((p.V + 15) / 16) * p.H * portions;       // of 16 value columns
   const int wr = groups >= 4 * sm_count() ? 1 : (groups > sm_count() ? 2 : 4);
-  if (p.D <= 32) return launch_block_scan<DELTA, 4, 1, TV>(p, portions, st);
+  if (p.D <= 32) return launch_block_scan<KIND, 4, 1, TV>(p, portions, st);
   if (p.D <= 64)
-    return wr == 1 ? launch_block_scan<DELTA, 8, 1, TV>(p, portions, st)
-                   : (wr == 2 ? launch_block_scan<DELTA, 4, 2, TV>(p, portions, st) : launch_block_scan<DELTA, 2, 4, TV>(p, portions, st));
+    return wr == 1 ? launch_block_scan<KIND, 8, 1, TV>(p, portions, st)
+                   : (wr == 2 ? launch_block_scan<KIND, 4, 2, TV>(p, portions, st) : launch_block_scan<KIND, 2, 4, TV>(p, portions, st));
   if (p.D <= 128)
-    return wr == 1 ? launch_block_scan<DELTA, 16, 1, TV>(p, portions, st)
-                   : (wr == 2 ? launch_block_scan<DELTA, 8, 2, TV>(p, portions, st) : launch_block_scan<DELTA, 4, 4, TV>(p, portions, st));
-  return launch_block_scan<DELTA, 8, 4, TV>(p, portions, st);
+    return wr == 1 ? launch_block_scan<KIND, 16, 1, TV>(p, portions, st)
+                   : (wr == 2 ? launch_block_scan<KIND, 8, 2, TV>(p, portions, st) : launch_block_scan<KIND, 4, 4, TV>(p, portions, st));
+  return launch_block_scan<KIND, 8, 4, TV>(p, portions, st);
 }
 
 static bool blocked_ok(int D, int V) { return D % 8 == 0 && V % 8 == 0; }
@@ -1532,7 +1746,9 @@ extern "C" int ts_delta_scan(const float* qkv, const float* gates, float* state,
 extern "C" int ts_block_scan_supported(int D, int V) { return blocked_ok(D, V) ? 1 : 0; }
 // Blocks of `rows` rows in `portions` portions (upper bound) and the floats a block and head needs.
 extern "C" int ts_block_scan_blocks(int rows, int portions) { return rows / BS_BLOCK + portions + 1; }
-extern "C" int ts_block_scan_coef(int delta) { return delta ? BS_COEF : BS_COEF_WKV; }
+extern "C" int ts_block_scan_coef(int kind) {
+  return kind == SCAN_DELTA ? BS_COEF : (kind == SCAN_WKV ? BS_COEF_WKV : BS_COEF_RET);
+}
 
 // Portions, step 2 of bf16 models: as ts_delta_scan, on the tensor cores.  coef: [blocks][H][BS_COEF] workspace.
 extern "C" int ts_delta_block_scan(const float* qkv, const float* gates, float* coef, float* state, long long state_ld, int s_off,
@@ -1547,7 +1763,7 @@ extern "C" int ts_delta_block_scan(const float* qkv, const float* gates, float* 
   p.q = qkv; p.k = qkv + G * D; p.v = qkv + 2 * G * D; p.qk_ld = p.v_ld = 2 * G * D + H * V; p.rep = H / G; p.coef = coef;
   p.state = state; p.state_ld = state_ld; p.s_off = s_off; p.row_prev = row_prev; p.row_next = row_next; p.cu = cu; p.o = o;
   p.H = H; p.D = D; p.V = V;
-  return dispatch_block_scan<true, float>(p, portions, ST(stream));
+  return dispatch_block_scan<SCAN_DELTA, float>(p, portions, ST(stream));
 }
 
 // Portions of the WKV recurrence of bf16 models.  Workspaces: rt, kt [rows][H D], coef [blocks][H][BS_COEF_WKV], row_decay
@@ -1569,14 +1785,15 @@ extern "C" int ts_wkv_block_scan(const void* rkvg, long long ld, const float* w_
   p.q = rt; p.k = kt; p.v = reinterpret_cast<const __nv_bfloat16*>(rkvg) + 2 * H * D; p.qk_ld = H * D; p.v_ld = ld; p.rep = 1;
   p.coef = coef; p.row_decay = row_decay; p.state = state; p.state_ld = state_ld; p.s_off = s_off; p.row_prev = row_prev;
   p.row_next = row_next; p.cu = cu; p.o = o; p.H = H; p.D = D; p.V = D;
-  return dispatch_block_scan<false, __nv_bfloat16>(p, portions, ST(stream));
+  return dispatch_block_scan<SCAN_WKV, __nv_bfloat16>(p, portions, ST(stream));
 }
 
-// Portions, last step (either recurrence): o [rows][H V] fp32; w per channel (w_head = V) or shared by heads (w_head = 0).
+// Portions, last step (either recurrence): o [rows][H V] fp32; w per channel (w_head = V), shared by heads (w_head = 0) or
+// absent (nullptr).
 extern "C" int ts_gated_norm(const float* o, const float* w, int w_head, const void* gate, long long gate_ld, void* out,
                              long long out_ld, int rows, int H, int V, float eps, float scale, int fp32, void* stream) {
   if (rows <= 0) return 0;
-  if (H <= 0 || V <= 0 || V > 256) return -10;
+  if (H <= 0 || V <= 0 || V > 512) return -10;
   return fp32 ? launch_gated_norm<float>(o, w, w_head, gate, gate_ld, out, out_ld, rows, H, V, eps, scale, ST(stream))
               : launch_gated_norm<__nv_bfloat16>(o, w, w_head, gate, gate_ld, out, out_ld, rows, H, V, eps, scale, ST(stream));
 }
@@ -1632,4 +1849,84 @@ extern "C" int ts_wkv_step(const void* rkvg, long long ld, const float* w_raw, c
     else wkv_step_kernel<__nv_bfloat16, 1><<<grid, RS_THREADS, smem, ST(stream)>>>(p);
   }
   return (int)cudaGetLastError();
+}
+
+static int retention_params(RetentionParams& p, const void* proj, long long ld, const float* angles, const float* powers,
+                            float k_scale, float* state, long long state_ld, const int* row_prev, const int* row_next, int H, int D,
+                            int V, int rot) {
+  if (H <= 0 || H > 65535 || D <= 0 || D > 256 || V <= 0 || V > 512 || rot < 0 || rot > D || rot % 2 ||
+      state_ld < static_cast<long long>(H) * D * V)
+    return -10;
+  p = {};
+  p.proj = proj; p.ld = ld; p.angles = angles; p.powers = powers; p.k_scale = k_scale; p.state = state; p.state_ld = state_ld;
+  p.row_prev = row_prev; p.row_next = row_next; p.H = H; p.D = D; p.V = V; p.rot = rot;
+  return 0;
+}
+
+// Length of a head's row of powers of its decay, from g^0 on.
+extern "C" int ts_retention_powers() { return RT_POWERS; }
+
+// Single rows of retention: projection -> out [rows][out_ld] = norm * silu(gate), state advanced.
+extern "C" int ts_retention_step(const void* proj, long long ld, const float* angles, const float* powers, float k_scale, float eps,
+                                 float* state, long long state_ld, const int* row_prev, const int* row_next, void* out,
+                                 long long out_ld, int rows, int H, int D, int V, int rot, int fp32, void* stream) {
+  if (rows <= 0) return 0;
+  RetentionParams p;
+  if (int e = retention_params(p, proj, ld, angles, powers, k_scale, state, state_ld, row_prev, row_next, H, D, V, rot)) return e;
+  p.eps = eps; p.out = out; p.out_ld = out_ld; p.rows = rows;
+  const bool vec = V % 4 == 0 && state_ld % 4 == 0;
+  const int nvec = vec ? V / 4 : V, groups = RTS_THREADS / (nvec < RTS_THREADS ? nvec : RTS_THREADS);
+  const size_t smem = ((V + 3) / 4 * 4 + (groups * V + 3) / 4 * 4 + 2 * D) * sizeof(float);
+  const dim3 grid(rows, H);
+  if (fp32) {
+    if (vec) retention_step_kernel<float, 4><<<grid, RTS_THREADS, smem, ST(stream)>>>(p);
+    else retention_step_kernel<float, 1><<<grid, RTS_THREADS, smem, ST(stream)>>>(p);
+  } else {
+    if (vec) retention_step_kernel<__nv_bfloat16, 4><<<grid, RTS_THREADS, smem, ST(stream)>>>(p);
+    else retention_step_kernel<__nv_bfloat16, 1><<<grid, RTS_THREADS, smem, ST(stream)>>>(p);
+  }
+  return (int)cudaGetLastError();
+}
+
+template <typename T> static int dispatch_retention_scan(const RetentionParams& p, int portions, cudaStream_t st) {
+  const dim3 grid((p.V + 31) / 32, p.H, portions);
+  if (p.D <= 32) retention_scan_kernel<T, 4><<<grid, 256, 0, st>>>(p);
+  else if (p.D <= 64) retention_scan_kernel<T, 8><<<grid, 256, 0, st>>>(p);
+  else if (p.D <= 128) retention_scan_kernel<T, 16><<<grid, 256, 0, st>>>(p);
+  else retention_scan_kernel<T, 32><<<grid, 256, 0, st>>>(p);
+  return (int)cudaGetLastError();
+}
+
+// Portions of retention: o [rows][H V] of the recurrence, the last state of every portion to its state row.  fp32 arithmetic.
+extern "C" int ts_retention_scan(const void* proj, long long ld, const float* angles, const float* powers, float k_scale,
+                                 float* state, long long state_ld, const int* row_prev, const int* row_next, const int* cu,
+                                 int portions, float* o, int H, int D, int V, int rot, int fp32, void* stream) {
+  if (portions <= 0) return 0;
+  RetentionParams p;
+  if (int e = retention_params(p, proj, ld, angles, powers, k_scale, state, state_ld, row_prev, row_next, H, D, V, rot)) return e;
+  if (portions > 65535) return -10;
+  p.cu = cu; p.o = o;
+  return fp32 ? dispatch_retention_scan<float>(p, portions, ST(stream)) : dispatch_retention_scan<__nv_bfloat16>(p, portions, ST(stream));
+}
+
+// Portions of retention in bf16 models: as ts_retention_scan, on the tensor cores.  Workspaces: rt, kt [rows][H D], coef
+// [blocks][H][BS_COEF_RET].
+extern "C" int ts_retention_block_scan(const void* proj, long long ld, const float* angles, const float* powers, float k_scale,
+                                       float* rt, float* kt, float* coef, float* state, long long state_ld, const int* row_prev,
+                                       const int* row_next, const int* cu, int portions, int max_rows, float* o, int H, int D,
+                                       int V, int rot, void* stream) {
+  if (portions <= 0) return 0;
+  RetentionParams r;
+  if (int e = retention_params(r, proj, ld, angles, powers, k_scale, state, state_ld, row_prev, row_next, H, D, V, rot)) return e;
+  if (!blocked_ok(D, V) || portions > 65535 || max_rows <= 0 || ld % 8 || (reinterpret_cast<uintptr_t>(proj) & 15u)) return -10;
+  r.cu = cu;
+  const size_t smem = 4 * 2 * BS_BLOCK * (D + 1) * sizeof(float);
+  if (int e = allow_smem(retention_blocks_kernel, smem)) return e;
+  retention_blocks_kernel<<<dim3((max_rows + BS_BLOCK - 1) / BS_BLOCK, (H + 3) / 4, portions), 128, smem, ST(stream)>>>(r, rt, kt, coef);
+  if (int e = (int)cudaGetLastError()) return e;
+  BlockScanParams p = {};
+  p.q = rt; p.k = kt; p.v = reinterpret_cast<const __nv_bfloat16*>(proj) + 2 * H * D; p.qk_ld = H * D; p.v_ld = ld; p.rep = 1;
+  p.coef = coef; p.state = state; p.state_ld = state_ld; p.row_prev = row_prev; p.row_next = row_next; p.cu = cu; p.o = o;
+  p.H = H; p.D = D; p.V = V;
+  return dispatch_block_scan<SCAN_RETENTION, __nv_bfloat16>(p, portions, ST(stream));
 }

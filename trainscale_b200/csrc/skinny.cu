@@ -31,10 +31,12 @@ struct SkinnyParams {
   int a_div;                   // row of A = slot / a_div
   int M, N, K;
   int act;                     // of common.cuh product_act or glu_act (0: none)
-  float act_cap;
+  float act_a, act_b;          // its constants
+  int act_cols;                // outputs it applies to, from the first
   int out_fp32;
-  const void* gate;            // result *= sigmoid(gate[slot * gate_ld + g * gate_group + n]) (nullptr: none)
+  const void* gate;            // result *= sigmoid(gate[slot * gate_ld + g * gate_group + n * gate_col]) (nullptr: none)
   long long gate_ld, gate_group;
+  int gate_col;
 };
 
 __device__ __forceinline__ void mma_bf16_16816(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3,
@@ -52,7 +54,7 @@ __device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162flo
 
 template <typename T>
 __device__ __forceinline__ void skinny_store(const SkinnyParams& p, int g, int slot, int n, float v) {
-  if (p.gate) v *= sigmoid(to_f32(reinterpret_cast<const T*>(p.gate)[slot * p.gate_ld + g * p.gate_group + n]));
+  if (p.gate) v *= sigmoid(to_f32(reinterpret_cast<const T*>(p.gate)[slot * p.gate_ld + g * p.gate_group + n * p.gate_col]));
   const long long at = g * p.o_group + static_cast<long long>(slot) * p.ldo + n;
   if (p.out_fp32) reinterpret_cast<float*>(p.out)[at] = v;
   else reinterpret_cast<__nv_bfloat16*>(p.out)[at] = __float2bfloat16(v);
@@ -155,7 +157,7 @@ skinny_gemm_kernel(SkinnyParams p) {
           for (int w = 0; w < KW; ++w) f += red[tile * KW + w][n + 8][tk];
           v = glu_act<true>(v, f, p.act);
         } else {
-          v = product_act(v, p.act, p.act_cap);
+          if (nn < p.act_cols) v = product_act<false>(v, p.act, p.act_a, p.act_b);
         }
         skinny_store<__nv_bfloat16>(p, g, p.order ? p.order[first + base + tk] : base + tk, nn, v);
       }
@@ -200,7 +202,8 @@ __global__ void __launch_bounds__(256) grouped_simt_kernel(SkinnyParams p) {
 #pragma unroll
     for (int t = 0; t < TM; ++t) {
       float v = warp_sum(acc[t]);
-      v = glu ? glu_act<false>(v, warp_sum(fac[t]), p.act) : product_act(v, p.act, p.act_cap);
+      if (glu) v = glu_act<false>(v, warp_sum(fac[t]), p.act);
+      else if (n < p.act_cols) v = product_act<false>(v, p.act, p.act_a, p.act_b);
       if (lane == 0 && base + t < m_total) skinny_store<T>(p, g, slot[t], n, v);
     }
   }
@@ -223,22 +226,24 @@ using namespace ts;
 
 // M: rows of every group, or an upper bound of them when `count` is given (`typical`: how many a group usually has; more
 // take further passes over the weights, which then come from L2).  fp32: A and W are fp32 (else bf16).  Gated activations:
-// W has N rows in alternating blocks of GLU_BLOCK gate and up rows, the result N / 2 columns.  gate (of the type of A):
-// nullptr or a factor sigmoid(gate) of every result.
+// W has N rows in alternating blocks of GLU_BLOCK gate and up rows, the result N / 2 columns.  `act` (with act_a, act_b)
+// applies to the first act_cols outputs.  gate (of the type of A): nullptr or a factor sigmoid(gate) of every result; gate_col 0:
+// one for all outputs of a row and group.
 extern "C" int ts_skinny_gemm(const void* A, const void* W, void* out, long long lda, long long ldw, long long ldo,
                               long long a_group, long long w_group, long long o_group, const int* order,
                               const int* start, const int* count, int a_div, int groups, int M, int N, int K, int act,
-                              float act_cap, int fp32, int out_fp32, int typical, const void* gate, long long gate_ld,
-                              long long gate_group, int row_tiles, void* stream) {
+                              float act_a, float act_b, int act_cols, int fp32, int out_fp32, int typical, const void* gate,
+                              long long gate_ld, long long gate_group, int gate_col, int row_tiles, void* stream) {
   if (M <= 0 || groups <= 0) return 0;
-  if (N <= 0 || K <= 0 || a_div <= 0 || act < 0 || act > ACT_LAST_GLU || (act == 3 && !(act_cap > 0.f)) || groups > 65535)
+  if (N <= 0 || K <= 0 || a_div <= 0 || act < 0 || act > ACT_LAST_GLU || (act == 3 && !(act_a > 0.f)) || act_cols < 0 || groups > 65535)
     return -10;
   if (act >= ACT_FIRST_GLU && N % (2 * GLU_BLOCK)) return -12;
   if (fp32 && !out_fp32) return -11;
   SkinnyParams p;
   p.A = A; p.W = W; p.out = out; p.lda = lda; p.ldw = ldw; p.ldo = ldo; p.a_group = a_group; p.w_group = w_group;
   p.o_group = o_group; p.order = order; p.start = start; p.count = count; p.a_div = a_div; p.M = M; p.N = N; p.K = K;
-  p.act = act; p.act_cap = act_cap; p.out_fp32 = out_fp32; p.gate = gate; p.gate_ld = gate_ld; p.gate_group = gate_group;
+  p.act = act; p.act_a = act_a; p.act_b = act_b; p.act_cols = act_cols; p.out_fp32 = out_fp32; p.gate = gate; p.gate_ld = gate_ld;
+  p.gate_group = gate_group; p.gate_col = gate_col;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   const bool vec = !fp32 && K % 8 == 0 && lda % 8 == 0 && ldw % 8 == 0 && a_group % 8 == 0 && w_group % 8 == 0 &&
                    aligned16(A) && aligned16(W);

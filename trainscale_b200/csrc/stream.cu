@@ -18,8 +18,9 @@
 //                 last boundary: x' normed once more with the final weight, only for the rows that are wanted
 //
 // `prenorm_kernel` is the boundary of decoders that norm a sublayer's INPUT:
-//   source        x' = x + y (* sigmoid(g), one number per row) + sum_j w_j * expert_j, or x' = embed[token]
-//   outputs       x' (fp32); h = x' / sqrt(mean(x'^2) + eps) * (1 + w); last boundary: h only, for the wanted rows
+//   source        x' = x + y (* sigmoid(g), one number per row, or * sigmoid(g + b), one per element) + sum_j w_j * expert_j, or
+//                 x' = embed[token]
+//   outputs       x' (fp32); h = x' / sqrt(mean(x'^2) + eps) * (base + w); last boundary: h only, for the wanted rows
 #include "common.cuh"
 #include "host_common.h"
 
@@ -488,11 +489,15 @@ struct PrenormParams {
   long long y_ld;
   const float* y_gate;         // logit of y's factor, stride y_gate_ld per row (nullptr: 1)
   long long y_gate_ld;
+  const void* e_gate;          // [T][e_gate_ld] logits of a factor of every element of y, activation type (nullptr: 1)
+  long long e_gate_ld;
+  const float* e_bias;         // [W], added to them
   const void* experts;         // expert outputs, W wide, or nullptr
   const int* dest;             // [T * k] row of every routed slot (nullptr: the slot itself)
   const float* route_w;        // [T * k]
   int k;
-  const float* w;              // [W], around zero
+  const float* w;              // [W]
+  float w_base;                // the norm multiplies by w_base + w
   float eps;
   float* x_out;                // [T][W] (not for FINAL)
   void* h;                     // [rows][W]
@@ -531,6 +536,13 @@ prenorm_kernel(PrenormParams p) {
         if (p.y) {
           float a[V];
           VecIO<T>::template load<V>(reinterpret_cast<const T*>(p.y) + t * p.y_ld + c * V, a);
+          if (p.e_gate) {
+            float g[V], b[V];
+            VecIO<T>::template load<V>(reinterpret_cast<const T*>(p.e_gate) + t * p.e_gate_ld + c * V, g);
+            VecIO<float>::load<V>(p.e_bias + c * V, b);
+#pragma unroll
+            for (int q = 0; q < V; ++q) a[q] *= sigmoid(g[q] + b[q]);
+          }
 #pragma unroll
           for (int q = 0; q < V; ++q) v[i][q] += f * a[q];
         }
@@ -575,7 +587,7 @@ prenorm_kernel(PrenormParams p) {
       float g[V];
       VecIO<float>::load<V>(p.w + c * V, g);
 #pragma unroll
-      for (int q = 0; q < V; ++q) v[i][q] = v[i][q] * inv * (1.f + g[q]);
+      for (int q = 0; q < V; ++q) v[i][q] = v[i][q] * inv * (p.w_base + g[q]);
       VecIO<T>::template store<V>(h + c * V, v[i]);
     }
   }
@@ -583,7 +595,8 @@ prenorm_kernel(PrenormParams p) {
 
 template <typename T, int MODE>
 static int launch_prenorm(const PrenormParams& p, int rows, cudaStream_t st) {
-  const bool vec = p.W % 4 == 0 && p.y_ld % 4 == 0;
+  const bool vec = p.W % 4 == 0 && p.y_ld % 4 == 0 && p.e_gate_ld % 4 == 0 &&
+                   (reinterpret_cast<uintptr_t>(p.y) | reinterpret_cast<uintptr_t>(p.e_gate)) % (4 * sizeof(T)) == 0;
   const int nvec = vec ? p.W / 4 : p.W, cap = vec ? 512 : 1024;
   int threads = (nvec + 31) / 32 * 32;
   if (threads > cap) threads = cap;
@@ -674,17 +687,17 @@ extern "C" int ts_stream_postnorm_final(const float* x_in, const void* y, long l
 }
 
 // Boundary of input-normed decoders.  `tok`: embedding source (then x_in, y and the experts are unused).  y_gate: logits of a
-// factor of y, one per row.  experts with dest (nullptr: slot order) and route_w [rows * k]: weighted sum of a row's slots.
+// factor of y, one per row; e_gate (with e_bias [W]): logits of one per element.  The norm multiplies by w_base + w.  experts with dest (nullptr: slot order) and route_w [rows * k]: weighted sum of a row's slots.
 // `rows_list` (with n_out entries): last boundary - h of those rows only, nothing else is written.
 extern "C" int ts_stream_prenorm(const long long* tok, const void* embed, int vocab, const float* x_in, const void* y,
-                                 long long y_ld, const float* y_gate, long long y_gate_ld, const void* experts, const int* dest,
-                                 const float* route_w, int k, const float* w, float eps, float* x_out, void* h, int rows,
-                                 const int* rows_list, int n_out, int W, int fp32_act, void* stream) {
+                                 long long y_ld, const float* y_gate, long long y_gate_ld, const void* e_gate, long long e_gate_ld,
+                                 const float* e_bias, const void* experts, const int* dest, const float* route_w, int k,
+                                 const float* w, float w_base, float eps, float* x_out, void* h, int rows, const int* rows_list, int n_out, int W, int fp32_act, void* stream) {
   if (rows_list ? n_out <= 0 : rows <= 0) return 0;
-  if (W <= 0 || (experts && (k <= 0 || !route_w)) || (tok && rows_list)) return -10;
+  if (W <= 0 || (experts && (k <= 0 || !route_w)) || (tok && rows_list) || (e_gate && (!y || !e_bias))) return -10;
   PrenormParams p = {};
   p.tok = tok; p.embed = embed; p.vocab = vocab; p.x_in = x_in; p.y = y; p.y_ld = y_ld; p.y_gate = y_gate;
-  p.y_gate_ld = y_gate_ld; p.experts = experts; p.dest = dest; p.route_w = route_w; p.k = k; p.w = w; p.eps = eps;
+  p.y_gate_ld = y_gate_ld; p.e_gate = e_gate; p.e_gate_ld = e_gate_ld; p.e_bias = e_bias; p.w_base = w_base; p.experts = experts; p.dest = dest; p.route_w = route_w; p.k = k; p.w = w; p.eps = eps;
   p.x_out = x_out; p.h = h; p.rows = rows_list; p.W = W;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   if (tok) return fp32_act ? launch_prenorm<float, STREAM_EMBED>(p, rows, st) : launch_prenorm<__nv_bfloat16, STREAM_EMBED>(p, rows, st);

@@ -5,11 +5,15 @@
 // (chunks count from position 0); besides, the first `keep` positions of the sequence.
 //
 //   ts_window_angles  cosines and sines of a step's positions, shared by all layers with the same frequencies
-//   ts_window_prep    bias, per-head RMS norm of queries and keys, rotary embedding of the first `rot` dimensions of a head
-//                     (in place in the projection), cache write of keys and values - one launch.  Each step but the last
+//   ts_window_prep    bias, per-head RMS norm of queries and keys, a factor of the queries that grows with the position, rotary
+//                     embedding of the first `rot` dimensions of a head (in place in the projection), cache write of keys and
+//                     values - one launch.  Each step but the last
 //                     is optional; values can be the projected keys themselves
 //   ts_window_attend  single query rows (decoding, fp32, and head sizes the prefill kernel does not take) against the paged
 //                     cache; the result may be multiplied by the sigmoid of a gate per head or per element
+//
+// Scores are (q . k) * scale, plus a number per head, minus a slope per head times the distance of query and key (either may be
+// absent).  Weights are their softmax over the visible keys or, without any normalization, their sigmoids.
 // Portions of prompts: ts_window_prefill (latent_prefill.cu).
 //
 // Decoding reads every cached key and value in the window once per key/value head.  `window_attend_mma_kernel` (bf16): the
@@ -44,7 +48,14 @@ struct WindowPrepParams {
   int h0;                      // first head that changes (H: queries stay as projected)
   int pairs;                   // rotation partners: 0 coordinates i and i + rot / 2, 1 coordinates 2 i and 2 i + 1
   int values_are_keys;         // values: the keys before norm and rotation, also written behind them in the projection
+  const int* pos;              // [T] (for the queries' factor)
+  float temp_coef;             // queries *= 1 + temp_coef * log(floor((pos + 1) / temp_every) + 1); temp_every 0: no factor
+  int temp_every;
 };
+
+__device__ __forceinline__ float query_factor(const WindowPrepParams& p, int t) {
+  return p.temp_every > 0 ? 1.f + p.temp_coef * logf(static_cast<float>((p.pos[t] + 1) / p.temp_every) + 1.f) : 1.f;
+}
 
 __global__ void window_angles_kernel(const float* __restrict__ inv_freq, const int* __restrict__ pos, float* __restrict__ out, int T,
                                      int half, float magnitude) {
@@ -67,6 +78,7 @@ __global__ void __launch_bounds__(WP_WARPS * 32) window_prep_kernel(WindowPrepPa
   T* row = reinterpret_cast<T*>(p.proj) + t * p.ld;
   T* crow = reinterpret_cast<T*>(p.cache) + p.slots[t] * p.row_width;
   T* v = row + (p.H + p.G) * p.dim;
+  const float qf = query_factor(p, t);
   for (int c = threadIdx.x; c < p.row_width - p.G * p.dim; c += blockDim.x) {
     if (c >= p.G * p.vdim) crow[p.G * p.dim + c] = from_f32<T>(0.f);
     else if (!p.values_are_keys) crow[p.G * p.dim + c] = v[c];
@@ -86,7 +98,8 @@ __global__ void __launch_bounds__(WP_WARPS * 32) window_prep_kernel(WindowPrepPa
       ss = warp_sum(ss);
       inv = 1.f / sqrtf(ss / static_cast<float>(p.dim) + p.eps);
     }
-    auto normed = [&](int c) { return w ? value(c) * inv * w[c] : value(c); };
+    const float factor = h < p.H ? qf : 1.f;
+    auto normed = [&](int c) { return (w ? value(c) * inv * w[c] : value(c)) * factor; };
     T* out2 = h < p.H ? nullptr : crow + (h - p.H) * p.dim;
     if (p.values_are_keys && h >= p.H)
       for (int c = lane; c < p.dim; c += 32) {
@@ -175,6 +188,11 @@ __global__ void __launch_bounds__(WP_WARPS * 32) window_prep_vec_kernel(WindowPr
       for (int j = 0; j < 8; ++j) a[j] *= inv * w[j];
     }
   }
+  if (p.temp_every > 0 && h < p.H) {
+    const float f = query_factor(p, t);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) a[j] *= f;
+  }
   if (p.pairs) {
     if (on) {
 #pragma unroll
@@ -236,6 +254,9 @@ struct WindowAttendParams {
   const void* gate;            // result *= sigmoid(gate), type of q: rows [gate_ld], see gate_mode (nullptr: none)
   long long gate_ld;
   int gate_mode;               // GATE_HEAD: column h, GATE_ELEMENT: column h * vdim + c
+  const float* slopes;         // [H] subtracted from a score per position of distance (nullptr: none)
+  const float* add;            // [H] added to every score (nullptr: none)
+  int sigmoid;                 // weights: sigmoid(score), not normalized
   int rows, H, G, dim, vdim, row_width, max_blocks, block_size, window, keep, chunked, chunk, splits;
   float scale, o_scale;
 };
@@ -257,6 +278,12 @@ template <typename T> __device__ __forceinline__ float gate_factor(const WindowA
   return sigmoid(to_f32(reinterpret_cast<const T*>(p.gate)[row * p.gate_ld + col]));
 }
 
+__device__ __forceinline__ float sigmoid_ex2(float x) {      // 1 / (1 + 2^-x)
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(1.f + fast_ex2(-x)));
+  return y;
+}
+
 constexpr int WS_CHUNK = 512;
 
 // grid (rows, H).  Scores of WS_CHUNK keys at a time in shared memory, then threads own value columns.
@@ -275,7 +302,8 @@ __global__ void __launch_bounds__(128) window_attend_simt_kernel(WindowAttendPar
   const T* q = reinterpret_cast<const T*>(p.q) + row * p.q_ld + h * p.dim;
   for (int i = threadIdx.x; i < p.dim; i += blockDim.x) qs[i] = to_f32(q[i]);
   for (int i = threadIdx.x; i < p.vdim; i += blockDim.x) acc[i] = 0.f;
-  float m = -INFINITY, l = 0.f;
+  float m = p.sigmoid ? 0.f : -INFINITY, l = 0.f;
+  const float slope = p.slopes ? p.slopes[h] : 0.f, add = p.add ? p.add[h] : 0.f;
   const VisibleKeys vis(p, len);
   auto key_row = [&](int i) {
     const int j = vis.position(i);
@@ -289,15 +317,15 @@ __global__ void __launch_bounds__(128) window_attend_simt_kernel(WindowAttendPar
       const T* c = key_row(j) + g * p.dim;
       float s = 0.f;
       for (int i = lane; i < p.dim; i += 32) s += qs[i] * to_f32(c[i]);
-      s = warp_sum(s) * p.scale;
+      s = warp_sum(s) * p.scale - slope * static_cast<float>(len - 1 - vis.position(j)) + add;
       if (lane == 0) sc[j - j0] = s;
       mx = fmaxf(mx, s);
     }
-    const float m_new = fmaxf(m, block_max(mx, scratch));
+    const float top = block_max(mx, scratch), m_new = p.sigmoid ? 0.f : fmaxf(m, top);
     const float alpha = expf(m - m_new);   // m = -inf at first: 0
     float part = 0.f;
     for (int j = j0 + threadIdx.x; j < j1; j += blockDim.x) {
-      const float w = expf(sc[j - j0] - m_new);
+      const float w = p.sigmoid ? sigmoid(sc[j - j0]) : expf(sc[j - j0] - m_new);
       sc[j - j0] = w;
       part += w;
     }
@@ -309,7 +337,7 @@ __global__ void __launch_bounds__(128) window_attend_simt_kernel(WindowAttendPar
       acc[r] = a;
     }
   }
-  const float inv = l > 0.f ? p.o_scale / l : 0.f;
+  const float inv = p.sigmoid ? p.o_scale : (l > 0.f ? p.o_scale / l : 0.f);
   T* out = reinterpret_cast<T*>(p.out) + row * p.out_ld + h * p.vdim;
   for (int r = threadIdx.x; r < p.vdim; r += blockDim.x) out[r] = from_f32<T>(acc[r] * inv * gate_factor<T>(p, row, h, r));
 }
@@ -348,8 +376,8 @@ static size_t window_smem(int dim, int vdim) {
   return (ring > merge ? ring : merge) + 16 * window_stride(dim) * 2;
 }
 
-// grid (rows, G * ceil(group / 16), splits).  DC: head sizes up to DC columns.
-template <int DC>
+// grid (rows, G * ceil(group / 16), splits).  DC: head sizes up to DC columns.  SIG: sigmoid weights.
+template <int DC, bool SIG>
 __global__ void __launch_bounds__(WA_WARPS * 32) window_attend_mma_kernel(WindowAttendParams p) {
   constexpr int KS = DC / 16, NV = DC / 8;
   extern __shared__ __align__(16) uint8_t raw[];
@@ -421,8 +449,14 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attend_mma_kernel(Window
   for (int n = 0; n < NV; ++n)
 #pragma unroll
     for (int q = 0; q < 4; ++q) o[n][q] = 0.f;
-  float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
-  const float sl = p.scale * 1.4426950408889634f;
+  constexpr float LOG2E = 1.4426950408889634f;
+  float m0 = SIG ? 0.f : -INFINITY, m1 = m0, l0 = 0.f, l1 = 0.f;
+  const float sl = p.scale * LOG2E;
+  // slope and addend of this thread's two heads, in powers of two
+  const bool biased = p.slopes || p.add;
+  const int ha = h0 + min(gid, nh - 1), hb = h0 + min(gid + 8, nh - 1);
+  const float slope0 = p.slopes ? p.slopes[ha] * LOG2E : 0.f, slope1 = p.slopes ? p.slopes[hb] * LOG2E : 0.f;
+  const float add0 = p.add ? p.add[ha] * LOG2E : 0.f, add1 = p.add ? p.add[hb] * LOG2E : 0.f;
   int stage = 0;
   for (int t = t_first + warp; t < t_end; t += WA_WARPS) {
     cp_wait<WA_STAGES - 2>();
@@ -443,18 +477,38 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attend_mma_kernel(Window
     auto keep = [&](float v, int key) { return key < j1 ? v * sl : -INFINITY; };
     s0[0] = keep(s0[0], j); s0[1] = keep(s0[1], j + 1); s0[2] = keep(s0[2], j); s0[3] = keep(s0[3], j + 1);
     s1[0] = keep(s1[0], j + 8); s1[1] = keep(s1[1], j + 9); s1[2] = keep(s1[2], j + 8); s1[3] = keep(s1[3], j + 9);
-    float a = fmaxf(fmaxf(s0[0], s0[1]), fmaxf(s1[0], s1[1])), b = fmaxf(fmaxf(s0[2], s0[3]), fmaxf(s1[2], s1[3]));
-    a = fmaxf(a, __shfl_xor_sync(0xffffffffu, a, 1));
-    b = fmaxf(b, __shfl_xor_sync(0xffffffffu, b, 1));
-    a = fmaxf(m0, fmaxf(a, __shfl_xor_sync(0xffffffffu, a, 2)));   // finite: every tile has a key in the range
-    b = fmaxf(m1, fmaxf(b, __shfl_xor_sync(0xffffffffu, b, 2)));
-    const float f0 = fast_ex2(m0 - a), f1 = fast_ex2(m1 - b);
-    m0 = a;
-    m1 = b;
-    s0[0] = fast_ex2(s0[0] - a); s0[1] = fast_ex2(s0[1] - a); s1[0] = fast_ex2(s1[0] - a); s1[1] = fast_ex2(s1[1] - a);
-    s0[2] = fast_ex2(s0[2] - b); s0[3] = fast_ex2(s0[3] - b); s1[2] = fast_ex2(s1[2] - b); s1[3] = fast_ex2(s1[3] - b);
-    l0 = l0 * f0 + ((s0[0] + s0[1]) + (s1[0] + s1[1]));
-    l1 = l1 * f1 + ((s0[2] + s0[3]) + (s1[2] + s1[3]));
+    if (biased) {
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const float da = static_cast<float>(len - 1 - vis.position(j + e)), db = static_cast<float>(len - 1 - vis.position(j + 8 + e));
+        s0[e] += add0 - slope0 * da;
+        s1[e] += add0 - slope0 * db;
+        s0[2 + e] += add1 - slope1 * da;
+        s1[2 + e] += add1 - slope1 * db;
+      }
+    }
+    float f0 = 1.f, f1 = 1.f;
+    if (SIG) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        s0[e] = sigmoid_ex2(s0[e]);
+        s1[e] = sigmoid_ex2(s1[e]);
+      }
+    } else {
+      float a = fmaxf(fmaxf(s0[0], s0[1]), fmaxf(s1[0], s1[1])), b = fmaxf(fmaxf(s0[2], s0[3]), fmaxf(s1[2], s1[3]));
+      a = fmaxf(a, __shfl_xor_sync(0xffffffffu, a, 1));
+      b = fmaxf(b, __shfl_xor_sync(0xffffffffu, b, 1));
+      a = fmaxf(m0, fmaxf(a, __shfl_xor_sync(0xffffffffu, a, 2)));   // finite: every tile has a key in the range
+      b = fmaxf(m1, fmaxf(b, __shfl_xor_sync(0xffffffffu, b, 2)));
+      f0 = fast_ex2(m0 - a);
+      f1 = fast_ex2(m1 - b);
+      m0 = a;
+      m1 = b;
+      s0[0] = fast_ex2(s0[0] - a); s0[1] = fast_ex2(s0[1] - a); s1[0] = fast_ex2(s1[0] - a); s1[1] = fast_ex2(s1[1] - a);
+      s0[2] = fast_ex2(s0[2] - b); s0[3] = fast_ex2(s0[3] - b); s1[2] = fast_ex2(s1[2] - b); s1[3] = fast_ex2(s1[3] - b);
+      l0 = l0 * f0 + ((s0[0] + s0[1]) + (s1[0] + s1[1]));
+      l1 = l1 * f1 + ((s0[2] + s0[3]) + (s1[2] + s1[3]));
+    }
     const uint32_t pf[4] = {pack_bf16x2(s0[0], s0[1]), pack_bf16x2(s0[2], s0[3]), pack_bf16x2(s1[0], s1[1]),
                             pack_bf16x2(s1[2], s1[3])};
     const uint32_t va = smem_u32(vt + (lane & 15) * vst + (lane >> 4) * 8);
@@ -463,8 +517,10 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attend_mma_kernel(Window
       if (n * 8 < p.vdim) {
         uint32_t bv[4];                    // columns 8 n: bv[0], bv[1]; the next eight: bv[2], bv[3]
         ldsm_x4_t(bv, va + n * 16);
-        o[n][0] *= f0; o[n][1] *= f0; o[n][2] *= f1; o[n][3] *= f1;
-        o[n + 1][0] *= f0; o[n + 1][1] *= f0; o[n + 1][2] *= f1; o[n + 1][3] *= f1;
+        if (!SIG) {
+          o[n][0] *= f0; o[n][1] *= f0; o[n][2] *= f1; o[n][3] *= f1;
+          o[n + 1][0] *= f0; o[n + 1][1] *= f0; o[n + 1][2] *= f1; o[n + 1][3] *= f1;
+        }
         mma_16816(o[n], pf, bv[0], bv[1]);
         mma_16816(o[n + 1], pf, bv[2], bv[3]);
       }
@@ -516,6 +572,7 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attend_mma_kernel(Window
       l += d[p.vdim + 1] * f;
       acc += d[c] * f;
     }
+    if (SIG) l = 1.f;                      // the sums are the result
     const int h = h0 + r;
     if (p.splits == 1) {
       reinterpret_cast<__nv_bfloat16*>(p.out)[row * p.out_ld + h * p.vdim + c] =
@@ -523,7 +580,7 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attend_mma_kernel(Window
     } else {
       const long long at = (static_cast<long long>(row) * p.H + h) * p.splits + split;
       p.part_out[at * p.vdim + c] = l > 0.f ? acc / l : 0.f;
-      if (c == 0) p.part_lse[at] = l > 0.f ? mm + log2f(l) : -INFINITY;      // in powers of two
+      if (c == 0 && !SIG) p.part_lse[at] = l > 0.f ? mm + log2f(l) : -INFINITY;      // in powers of two
     }
   }
 }
@@ -532,28 +589,37 @@ constexpr int WM_MAX_SPLITS = 64;
 __global__ void __launch_bounds__(128) window_merge_kernel(WindowAttendParams p) {
   const int row = blockIdx.x, h = blockIdx.y;
   const long long base = (static_cast<long long>(row) * p.H + h) * p.splits;
-  float mm = -INFINITY, l = 0.f;
-  for (int s = 0; s < p.splits; ++s) mm = fmaxf(mm, p.part_lse[base + s]);
-  for (int s = 0; s < p.splits; ++s) l += fast_ex2(p.part_lse[base + s] - mm);
+  float mm = -INFINITY, l = p.sigmoid ? 1.f : 0.f;
+  if (!p.sigmoid) {
+    for (int s = 0; s < p.splits; ++s) mm = fmaxf(mm, p.part_lse[base + s]);
+    for (int s = 0; s < p.splits; ++s) l += fast_ex2(p.part_lse[base + s] - mm);
+  }
   for (int c = threadIdx.x; c < p.vdim; c += blockDim.x) {
     float acc = 0.f;
-    for (int s = 0; s < p.splits; ++s) acc += fast_ex2(p.part_lse[base + s] - mm) * p.part_out[(base + s) * p.vdim + c];
+    for (int s = 0; s < p.splits; ++s)
+      acc += (p.sigmoid ? 1.f : fast_ex2(p.part_lse[base + s] - mm)) * p.part_out[(base + s) * p.vdim + c];
     reinterpret_cast<__nv_bfloat16*>(p.out)[row * p.out_ld + h * p.vdim + c] =
         __float2bfloat16(acc * (p.o_scale / l) * gate_factor<__nv_bfloat16>(p, row, h, c));
   }
 }
 
-template <int DC> static int launch_window_mma(const WindowAttendParams& p, cudaStream_t st) {
+template <int DC, bool SIG> static int launch_window_mma(const WindowAttendParams& p, cudaStream_t st) {
   const size_t smem = window_smem(p.dim, p.vdim);
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(window_attend_mma_kernel<DC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+    cudaError_t e = cudaFuncSetAttribute(window_attend_mma_kernel<DC, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                         227 * 1024);
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
   const int tiles_h = (p.H / p.G + 15) / 16;
-  window_attend_mma_kernel<DC><<<dim3(p.rows, p.G * tiles_h, p.splits), WA_WARPS * 32, smem, st>>>(p);
+  window_attend_mma_kernel<DC, SIG><<<dim3(p.rows, p.G * tiles_h, p.splits), WA_WARPS * 32, smem, st>>>(p);
   return (int)cudaGetLastError();
+}
+
+template <bool SIG> static int dispatch_window_mma(const WindowAttendParams& p, cudaStream_t st) {
+  const int dc = p.dim > p.vdim ? p.dim : p.vdim;
+  return dc <= 64 ? launch_window_mma<64, SIG>(p, st) : (dc <= 128 ? launch_window_mma<128, SIG>(p, st) : launch_window_mma<256, SIG>(p, st));
 }
 
 static bool window_mma_ok(int dim, int vdim, int fp32) {
@@ -576,15 +642,18 @@ extern "C" int ts_window_angles(const float* inv_freq, const int* pos, float* ou
 
 // angles: of ts_window_angles (unused without rotated dimensions).  bias, norms: nullptr for none (both norms or neither).
 // pairs: rotation partners are neighbours.  values_are_keys: the projection has no values, its columns behind the keys
-// receive the keys before norm and rotation.
+// receive the keys before norm and rotation.  pos, temp_coef, temp_every: the queries' factor (temp_every 0: none).
 extern "C" int ts_window_prep(void* proj, long long ld, const float* bias, const float* q_norm, const float* k_norm, float eps,
                               const float* angles, const long long* slots, void* cache, int T, int H, int G, int dim, int vdim,
-                              int rot, int pairs, int values_are_keys, int row_width, int fp32, void* stream) {
+                              int rot, int pairs, int values_are_keys, const int* pos, float temp_coef, int temp_every, int row_width,
+                              int fp32, void* stream) {
   if (T <= 0) return 0;
   if (H <= 0 || G <= 0 || dim <= 0 || vdim <= 0 || rot < 0 || rot > dim || rot % 2 || row_width < G * (dim + vdim)) return -10;
-  if ((q_norm == nullptr) != (k_norm == nullptr) || (values_are_keys && dim != vdim)) return -10;
+  if ((q_norm == nullptr) != (k_norm == nullptr) || (values_are_keys && dim != vdim) || temp_every < 0 || (temp_every > 0 && !pos))
+    return -10;
   WindowPrepParams p;
-  p.bias = bias; p.pairs = pairs; p.values_are_keys = values_are_keys; p.h0 = bias || q_norm || rot ? 0 : H;
+  p.bias = bias; p.pairs = pairs; p.values_are_keys = values_are_keys; p.h0 = bias || q_norm || rot || temp_every ? 0 : H;
+  p.pos = pos; p.temp_coef = temp_coef; p.temp_every = temp_every;
   p.proj = proj; p.ld = ld; p.q_norm = q_norm; p.k_norm = k_norm; p.eps = eps; p.angles = angles; p.slots = slots;
   p.cache = cache; p.T = T; p.H = H; p.G = G; p.dim = dim; p.vdim = vdim; p.rot = rot; p.row_width = row_width;
   const bool vec = !fp32 && dim % 8 == 0 && vdim % 8 == 0 && dim <= 256 && ld % 8 == 0 && row_width == G * (dim + vdim) &&
@@ -616,12 +685,13 @@ extern "C" int ts_window_splits(int rows, int H, int G, int dim, int vdim, int k
   return s < 1 ? 1 : s;
 }
 
-// window, keep, chunked: which keys a row sees (above).  `keys`: upper bound of their number; `splits` of ts_window_splits with the workspaces it needs (splits > 1).
+// window, keep, chunked: which keys a row sees; slopes, add, sigmoid: their weights (top of the file).  `keys`: upper bound of their number; `splits` of ts_window_splits with the workspaces it needs (splits > 1).
 extern "C" int ts_window_attend(const void* q, long long q_ld, const void* cache, const int* block_table, int max_blocks,
                                 const int* row_seq, const int* row_len, void* out, long long out_ld, float* part_out,
                                 float* part_lse, int rows, int H, int G, int dim, int vdim, int row_width, int block_size,
                                 int window, int keep, int chunked, int keys, int splits, float scale, float o_scale,
-                                const void* gate, long long gate_ld, int gate_mode, int fp32, void* stream) {
+                                const float* slopes, const float* add, int sigmoid, const void* gate, long long gate_ld,
+                                int gate_mode, int fp32, void* stream) {
   if (rows <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G || dim <= 0 || vdim <= 0 || window <= 0 || keep < 0 || keys <= 0 || splits < 1 ||
       splits > WM_MAX_SPLITS)
@@ -630,7 +700,7 @@ extern "C" int ts_window_attend(const void* q, long long q_ld, const void* cache
   p.q = q; p.q_ld = q_ld; p.cache = cache; p.block_table = block_table; p.row_seq = row_seq; p.row_len = row_len; p.out = out;
   p.out_ld = out_ld; p.part_out = part_out; p.part_lse = part_lse; p.rows = rows; p.H = H; p.G = G; p.dim = dim;
   p.vdim = vdim; p.row_width = row_width; p.max_blocks = max_blocks; p.block_size = block_size; p.window = window;
-  p.keep = keep; p.chunked = chunked; p.gate = gate; p.gate_ld = gate_ld; p.gate_mode = gate_mode;
+  p.keep = keep; p.chunked = chunked; p.slopes = slopes; p.add = add; p.sigmoid = sigmoid; p.gate = gate; p.gate_ld = gate_ld; p.gate_mode = gate_mode;
   p.splits = splits; p.chunk = ((keys + splits - 1) / splits + 15) / 16 * 16; p.scale = scale; p.o_scale = o_scale;
   const bool vec = window_mma_ok(dim, vdim, fp32) && scale > 0.f && q_ld % 8 == 0 && row_width % 8 == 0 &&
                    (reinterpret_cast<uintptr_t>(q) & 15u) == 0 && (reinterpret_cast<uintptr_t>(cache) & 15u) == 0;
@@ -641,9 +711,7 @@ extern "C" int ts_window_attend(const void* q, long long q_ld, const void* cache
     else window_attend_simt_kernel<__nv_bfloat16><<<dim3(rows, H), 128, smem, ST(stream)>>>(p);
     return (int)cudaGetLastError();
   }
-  const int dc = dim > vdim ? dim : vdim;
-  int rc = dc <= 64 ? launch_window_mma<64>(p, ST(stream))
-                    : (dc <= 128 ? launch_window_mma<128>(p, ST(stream)) : launch_window_mma<256>(p, ST(stream)));
+  int rc = sigmoid ? dispatch_window_mma<true>(p, ST(stream)) : dispatch_window_mma<false>(p, ST(stream));
   if (rc == 0 && splits > 1) {
     window_merge_kernel<<<dim3(rows, H), 128, 0, ST(stream)>>>(p);
     rc = (int)cudaGetLastError();

@@ -63,4 +63,5 @@ def build_preset(name: str, dtype, device=None, seed: int | None = None):
 register_architecture(Architecture("Mezilix", f"{__name__}.mezilix", lambda c: c.get("architecture") == "Mezilix"))
 register_architecture(Architecture("Vibepel", f"{__name__}.vibepel", lambda c: c.get("architecture") == "Vibepel"))
 register_architecture(Architecture("Kabulix", f"{__name__}.kabulix", lambda c: c.get("architecture") == "Kabulix"))
+register_architecture(Architecture("Lovurax", f"{__name__}.lovurax", lambda c: c.get("architecture") == "Lovurax"))
 register_architecture(Architecture("Llama", f"{__name__}.llama", lambda c: "architecture" not in c))

@@ -22,11 +22,11 @@ def _use_cuda(*ts: torch.Tensor) -> bool:
 
 def gemm_raw(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor, M: int, N: int, K: int, lda: int, ldb: int,
              ldc: int, a_mn: bool, b_mn: bool, accumulate: bool = False, alpha: float = 1.0, bn: int = 0, act: int = 0,
-            cap: float = 0.0) -> None:
+            cap: float = 0.0, second: float = 0.0, act_cols: int | None = None) -> None:
     lib = _lib.load("gemm")
     rc = lib.ts_gemm_bf16_act(_lib.ptr(a), _lib.ptr(b), _lib.ptr(out), M, N, K, lda, ldb, ldc, int(a_mn), int(b_mn),
                               int(out.dtype == torch.float32), int(accumulate), _c.c_float(alpha), bn, act,
-                              _c.c_float(cap), _lib.stream_ptr())
+                              _c.c_float(cap), _c.c_float(second), N if act_cols is None else act_cols, _lib.stream_ptr())
     _lib.check(rc, "ts_gemm_bf16_act")
 
 
@@ -215,25 +215,26 @@ def few_rows(M: int, N: int, K: int) -> bool:
 
 @torch.no_grad()
 def serve_linear(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None = None, act: int = 0, cap: float = 0.0,
-                 out: torch.Tensor | None = None) -> torch.Tensor:
-    """act(x [M, K] @ w [N, K]^T) for serving (no autograd), optionally with an fp32 result; `act` of ops/grouped (`cap`:
-    constant of the soft cap; a gated act takes a packed weight and halves the columns).  bf16 on the GPU: few rows go to the few-row kernel, more to the tcgen05 GEMM, the
+                 out: torch.Tensor | None = None, second: float = 0.0, act_cols: int | None = None) -> torch.Tensor:
+    """act(x [M, K] @ w [N, K]^T) for serving (no autograd), optionally with an fp32 result; `act` of ops/grouped (`cap`,
+    `second`: its constants; a gated act takes a packed weight and halves the columns), of all columns or of the first `act_cols`, a
+    multiple of ACT_BLOCK.  bf16 on the GPU: few rows go to the few-row kernel, more to the tcgen05 GEMM, the
     activation in the epilogue of either; rows that are not whole 16-byte vectors, and fp32, to the library."""
     from . import grouped
     out_dtype = out.dtype if out is not None else out_dtype or x.dtype
     vec = (x.is_cuda and x.dtype == torch.bfloat16 and w.shape[1] % 8 == 0 and x.stride(0) % 8 == 0 and x.stride(1) == 1
            and x.data_ptr() % 16 == 0)
     if vec and few_rows(x.shape[0], *w.shape):
-        return grouped.rows_linear(x, w, out_dtype, act, cap, out)
+        return grouped.rows_linear(x, w, out_dtype, act, cap, out, second, act_cols)
     if vec:
         if out is None:
             out = torch.empty(x.shape[0], w.shape[0] // (2 if grouped.is_gated(act) else 1), dtype=out_dtype, device=x.device)
         gemm_raw(x, w, out, x.shape[0], w.shape[0], x.shape[1], x.stride(0), w.stride(0), out.stride(0), False, False,
-                 act=act, cap=cap)
+                 act=act, cap=cap, second=second, act_cols=act_cols)
         return out
     if out_dtype != x.dtype:
         x, w = x.to(out_dtype), w.to(out_dtype)
     y = torch.nn.functional.linear(x, w)
     if act:
-        y = grouped.activate(y, act, cap)
+        y = grouped.activate(y, act, cap, second, act_cols)
     return y if out is None else out.copy_(y)

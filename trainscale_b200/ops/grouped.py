@@ -12,8 +12,11 @@ import torch
 from . import _lib
 
 _ll = ctypes.c_longlong
-ACT_NONE, ACT_RELU_SQUARED, ACT_TANH, ACT_SOFTCAP = 0, 1, 2, 3
-ACT_SILU_GLU, ACT_GELU_GLU = 4, 5            # silu(gate) * up, tanh form of gelu(gate) * up
+ACT_NONE, ACT_RELU_SQUARED, ACT_TANH = 0, 1, 2
+ACT_SOFTCAP, ACT_SCALE = 3, 4                # c tanh(x / c), c x; c is the constant `cap`
+ACT_XIELU = 5                                # x > 0: cap x^2 + x / 2, else second (e^x - 1 - x) + x / 2
+ACT_SILU_GLU, ACT_GELU_GLU = 6, 7            # silu(gate) * up, tanh form of gelu(gate) * up
+ACT_BLOCK = 32                               # an activation of leading columns only takes a multiple of these
 GLU_BLOCK = 16
 
 
@@ -43,7 +46,15 @@ class GluRows:
         self.blocks.copy_(rows.view(self.blocks.shape))
 
 
-def activate(x: torch.Tensor, act: int, cap: float = 0.0) -> torch.Tensor:
+def xielu(x: torch.Tensor, a: float, b: float) -> torch.Tensor:
+    n = x.clamp(max=0.0)
+    return a * x.clamp(min=0.0).square() + b * (torch.expm1(n) - n) + 0.5 * x
+
+
+def activate(x: torch.Tensor, act: int, cap: float = 0.0, second: float = 0.0, act_cols: int | None = None) -> torch.Tensor:
+    """`act` with its constants; `act_cols`: of the first columns, the others stay."""
+    if act_cols is not None and act_cols < x.shape[-1]:
+        return torch.cat([activate(x[..., :act_cols], act, cap, second), x[..., act_cols:]], dim=-1)
     if is_gated(act):
         g, u = x.unflatten(-1, (-1, 2, GLU_BLOCK)).unbind(-2)
         a = torch.nn.functional.silu(g) if act == ACT_SILU_GLU else torch.nn.functional.gelu(g, approximate="tanh")
@@ -52,18 +63,24 @@ def activate(x: torch.Tensor, act: int, cap: float = 0.0) -> torch.Tensor:
         return torch.relu(x).square()
     if act == ACT_TANH:
         return torch.tanh(x)
-    return cap * torch.tanh(x / cap) if act == ACT_SOFTCAP else x
+    if act == ACT_SOFTCAP:
+        return cap * torch.tanh(x / cap)
+    if act == ACT_XIELU:
+        return xielu(x, cap, second)
+    return cap * x if act == ACT_SCALE else x
 
 
 def _launch(A, W, out, lda, ldw, ldo, a_group, w_group, o_group, order, start, count, a_div, groups, M, N, K, act,
-            typical=0, cap=0.0, gate=None, row_tiles=0):
+            typical=0, cap=0.0, gate=None, row_tiles=0, second=0.0, act_cols=None):
     if gate is not None and gate.dtype != A.dtype:
         raise TypeError("the gate has the type of the rows")
     rc = _lib.load("skinny").ts_skinny_gemm(
         _lib.ptr(A), _lib.ptr(W), _lib.ptr(out), _ll(lda), _ll(ldw), _ll(ldo), _ll(a_group), _ll(w_group), _ll(o_group),
         _lib.ptr(order), _lib.ptr(start), _lib.ptr(count), a_div, groups, M, N, K, act, ctypes.c_float(cap),
+        ctypes.c_float(second), N if act_cols is None else act_cols,
         int(A.dtype == torch.float32), int(out.dtype == torch.float32), typical, _lib.ptr(gate),
-        _ll(0 if gate is None else gate.stride(0)), _ll(0 if gate is None else gate.stride(1)), row_tiles, _lib.stream_ptr())
+        _ll(0 if gate is None else gate.stride(0)), _ll(0 if gate is None else gate.stride(1)),
+        0 if gate is None else gate.stride(2), row_tiles, _lib.stream_ptr())
     _lib.check(rc, "ts_skinny_gemm")
 
 
@@ -73,18 +90,18 @@ def _row_tiles(rows: int, cols: int) -> int:
 
 
 def rows_linear(x: torch.Tensor, w: torch.Tensor, out_dtype=None, act: int = ACT_NONE, cap: float = 0.0,
-                out: torch.Tensor | None = None) -> torch.Tensor:
+                out: torch.Tensor | None = None, second: float = 0.0, act_cols: int | None = None) -> torch.Tensor:
     """act(x [M, K] @ w [N, K]^T) for a handful of rows: the cost is one pass over w, spread over N / 16 CTAs."""
     if out is None:
         out = torch.empty(x.shape[0], w.shape[0] // (2 if is_gated(act) else 1), dtype=out_dtype or x.dtype, device=x.device)
     _launch(x, w, out, x.stride(0), w.stride(0), out.stride(0), 0, 0, 0, None, None, None, 1, 1, x.shape[0], w.shape[0],
-            w.shape[1], act, cap=cap, row_tiles=_row_tiles(x.shape[0], w.shape[0]))
+            w.shape[1], act, cap=cap, row_tiles=_row_tiles(x.shape[0], w.shape[0]), second=second, act_cols=act_cols)
     return out
 
 
 def head_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None, gate: torch.Tensor | None = None) -> torch.Tensor:
     """x [T, H, K] (last dimension contiguous), w [H, N, K] -> [T, H, N]: every head has its own matrix.  `gate` [T, H, N]
-    (last dimension contiguous): the result is multiplied by sigmoid(gate)."""
+    (any strides, so it may be one number per head, expanded): the result is multiplied by sigmoid(gate)."""
     T, H, K = x.shape
     N = w.shape[1]
     if out is None:

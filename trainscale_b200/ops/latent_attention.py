@@ -32,7 +32,7 @@ class LatentShape:
     rank: int             # latent size
     window: int           # keys a position sees: itself and window - 1 before it
     scale: float
-    rope_base: float
+    rope_base: float = 10000.0
     pairs: bool = False   # rotation partners: coordinates 2 i and 2 i + 1 instead of i and i + rot / 2
     magnitude: float = 1.0  # factor of cos and sin
 

@@ -4,6 +4,9 @@ from __future__ import annotations
 from dataclasses import dataclass
 
 
+UNBOUNDED = 1 << 30       # size of a window that no sequence outgrows
+
+
 @dataclass(frozen=True)
 class KeyMask:
     """Itself and the `size` - 1 positions before it, or (`chunked`) the positions before it in its chunk of `size`, chunks

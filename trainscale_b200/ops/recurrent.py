@@ -1,8 +1,8 @@
-"""Recurrent mixers with an fp32 matrix state per head: the gated delta rule (with short convolutions in front) and WKV time
-mixing (csrc/recurrent.cu).
+"""Recurrent mixers with an fp32 matrix state per head: the gated delta rule (with short convolutions in front), WKV time
+mixing and retention (csrc/recurrent.cu).
 
-Both run over a flattened batch whose first rows are single tokens (decoding: one launch from projection to gated norm) and
-whose other rows are portions of prompts (a scan).  A sequence's state row holds [convolution inputs or token-shift row |
+All run over a flattened batch whose first rows are single tokens (decoding: one launch from projection to gated norm) and
+whose other rows are portions of prompts (a scan).  A sequence's state row holds [convolution inputs or token-shift row, if any |
 S of every head]; `rows.prev` / `rows.next` name the state rows a sequence continues from and leaves.  Tensors on the CPU
 take PyTorch math.
 """
@@ -20,6 +20,8 @@ from .stream import StreamRows
 
 _ll, _f = ctypes.c_longlong, ctypes.c_float
 MAX_HEAD = 256           # largest key or value size of a head
+MAX_RETENTION_VALUE = 512  # retention: largest value size
+SCAN_WKV, SCAN_DELTA, SCAN_RETENTION = 0, 1, 2
 
 
 def _up4(n: int) -> int:
@@ -74,6 +76,37 @@ class WkvShape:
     @property
     def state_width(self) -> int:
         return _up4(self.matrix_offset + self.heads * self.dim * self.dim)
+
+
+@dataclass(frozen=True)
+class RetentionShape:
+    """Sizes and constants of one retention mixer; its projection row is q | k | v | gate."""
+    heads: int
+    dim: int
+    vdim: int
+    rot: int                       # rotated dimensions of a head
+    decay: tuple[float, ...]       # per head
+
+    @property
+    def qk_width(self) -> int:
+        return self.heads * self.dim
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def proj_width(self) -> int:
+        return 2 * (self.qk_width + self.out_width)
+
+    @property
+    def state_width(self) -> int:
+        return _up4(self.heads * self.dim * self.vdim)
+
+    def powers(self, n: int = 9) -> torch.Tensor:
+        """fp32 [heads, n] g^0 .. g^(n - 1) of the decays as fp32 numbers."""
+        g = torch.tensor(self.decay, dtype=torch.float32).double()
+        return (g[:, None] ** torch.arange(n, dtype=torch.float64)).float()
 
 
 @dataclass
@@ -177,10 +210,10 @@ def _blocked(dim: int, vdim: int) -> bool:
     return bool(_lib.load("recurrent").ts_block_scan_supported(dim, vdim))
 
 
-def _workspace(T: int, portions, delta: int, *shape, device) -> torch.Tensor:
+def _workspace(T: int, portions, kind: int, *shape, device) -> torch.Tensor:
     """Uninitialised fp32 [blocks, heads, ...] for the per-block quantities of a block scan."""
     lib = _lib.load("recurrent")
-    last = shape[1:] or (lib.ts_block_scan_coef(delta),)
+    last = shape[1:] or (lib.ts_block_scan_coef(kind),)
     return torch.empty(lib.ts_block_scan_blocks(T, portions.count), shape[0], *last, dtype=torch.float32, device=device)
 
 
@@ -190,7 +223,7 @@ def delta_scan(qkv, gates, s: DeltaShape, rows: StreamRows, state, portions, blo
     T = qkv.shape[0]
     o = torch.empty(T, s.out_width, dtype=torch.float32, device=qkv.device)
     if blocked and _blocked(s.dim, s.vdim):
-        coef = _workspace(T, portions, 1, s.heads, device=qkv.device)
+        coef = _workspace(T, portions, SCAN_DELTA, s.heads, device=qkv.device)
         rc = _lib.load("recurrent").ts_delta_block_scan(
             _lib.ptr(qkv), _lib.ptr(gates), _lib.ptr(coef), _lib.ptr(state),
             _ll(state.stride(0)), s.matrix_offset, _lib.ptr(rows.prev), _lib.ptr(rows.next), _lib.ptr(portions.cu),
@@ -206,7 +239,7 @@ def delta_scan(qkv, gates, s: DeltaShape, rows: StreamRows, state, portions, blo
 
 
 def gated_norm(o, w, w_head: int, gate, out, heads: int, vdim: int, eps: float, scale: float = 1.0) -> None:
-    """out = o / rms per head * w * silu(gate) * scale; `w_head`: stride of w from head to head (0: shared)."""
+    """out = o / rms per head * w * silu(gate) * scale; `w_head`: stride of w from head to head (0: shared); w None: one."""
     rc = _lib.load("recurrent").ts_gated_norm(
         _lib.ptr(o), _lib.ptr(w), w_head, _lib.ptr(gate), _ll(gate.stride(0)), _lib.ptr(out), _ll(out.stride(0)), o.shape[0],
         heads, vdim, _f(eps), _f(scale), int(out.dtype == torch.float32), _lib.stream_ptr())
@@ -260,7 +293,8 @@ def wkv_scan(rkvg, w_raw, s: WkvShape, w: WkvWeights, rows: StreamRows, state, p
     o = torch.empty(T, s.inner, dtype=torch.float32, device=dev)
     if blocked and _blocked(s.dim, s.dim):
         rt, kt = (torch.empty(T, s.inner, dtype=torch.float32, device=dev) for _ in range(2))
-        coef, decay = _workspace(T, portions, 0, s.heads, device=dev), _workspace(T, portions, 0, s.heads, s.dim, device=dev)
+        coef = _workspace(T, portions, SCAN_WKV, s.heads, device=dev)
+        decay = _workspace(T, portions, SCAN_WKV, s.heads, s.dim, device=dev)
         rc = _lib.load("recurrent").ts_wkv_block_scan(
             _lib.ptr(rkvg), _ll(rkvg.stride(0)), _lib.ptr(w_raw), _lib.ptr(w.w0), _lib.ptr(w.u), _lib.ptr(rt), _lib.ptr(kt),
             _lib.ptr(coef), _lib.ptr(decay), _lib.ptr(state), _ll(state.stride(0)), s.matrix_offset, _lib.ptr(rows.prev),
@@ -273,4 +307,78 @@ def wkv_scan(rkvg, w_raw, s: WkvShape, w: WkvWeights, rows: StreamRows, state, p
         _ll(state.stride(0)), s.matrix_offset, _lib.ptr(rows.prev), _lib.ptr(rows.next), _lib.ptr(portions.cu),
         portions.count, _lib.ptr(o), s.heads, s.dim, int(rkvg.dtype == torch.float32), _lib.stream_ptr())
     _lib.check(rc, "ts_wkv_scan")
+    return o
+
+
+# ---------------------------------------------------------------------------------------------- retention
+def _turn(x: torch.Tensor, cs: torch.Tensor, rot: int) -> torch.Tensor:
+    """x [T, H, D]: coordinate i turns with i + rot / 2; cs [T, rot] = cos | sin."""
+    half = rot // 2
+    c, s = cs[:, None, :half], cs[:, None, half:]
+    u, v = x[..., :half], x[..., half:rot]
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., rot:]], dim=-1)
+
+
+def _retention_reference(proj, s: RetentionShape, powers, eps, cs, rows, state, n_single, cu, out):
+    H, D, V, kw = s.heads, s.dim, s.vdim, s.qk_width
+    g = powers[:, 1, None, None]
+    for a, b, prev, nxt in _sequences(rows, n_single, cu, proj.shape[0]):
+        x = proj[a:b].float()
+        q, k = (_turn(z.reshape(b - a, H, D), cs[a:b], s.rot) for z in (x[:, :kw], x[:, kw:2 * kw]))
+        k = k * D ** -0.5
+        v, gate = x[:, 2 * kw:2 * kw + s.out_width].reshape(b - a, H, V), x[:, 2 * kw + s.out_width:s.proj_width]
+        S = torch.zeros(H, D, V) if prev < 0 else state[prev, :H * D * V].view(H, D, V)
+        for t in range(b - a):
+            S = g * S + k[t, :, :, None] * v[t, :, None]
+            o = _rms(torch.einsum("hdv,hd->hv", S, q[t]), eps)
+            out[a + t] = (o.reshape(-1) * F.silu(gate[t])).to(out.dtype)
+        if nxt >= 0:
+            state[nxt, :S.numel()] = S.reshape(-1)
+
+
+def retention(proj: torch.Tensor, s: RetentionShape, powers: torch.Tensor, eps: float, cs: torch.Tensor, rows: StreamRows,
+              state: torch.Tensor, n_single: int, portions, out: torch.Tensor) -> None:
+    """proj [T, >= proj_width] -> out [T, heads * vdim]: S <- g S + k v^T, o = S^T q with q and k rotated and k times dim^-1/2;
+    o / rms per head * silu(gate).  cs fp32 [T, rot] of ops/window_attention.angles, powers of `RetentionShape.powers`."""
+    if not proj.is_cuda:
+        return _retention_reference(proj, s, powers, eps, cs, rows, state, n_single, portions.offsets if portions else [0], out)
+    T = proj.shape[0]
+    if n_single > 0:
+        retention_step(proj[:n_single], s, powers, eps, cs, rows, state, out[:n_single])
+    if n_single < T:
+        tail = StreamRows(rows.prev[n_single:], rows.next[n_single:])
+        part = proj[n_single:]
+        o = retention_scan(part, s, powers, cs[n_single:], tail, state, portions, proj.dtype == torch.bfloat16)
+        gate = part[:, 2 * s.qk_width + s.out_width:s.proj_width]
+        gated_norm(o, None, 0, gate, out[n_single:], s.heads, s.vdim, eps)
+
+
+def retention_step(proj, s: RetentionShape, powers, eps: float, cs, rows: StreamRows, state, out) -> None:
+    """Single rows: rotation, state update, norm and gate."""
+    rc = _lib.load("recurrent").ts_retention_step(
+        _lib.ptr(proj), _ll(proj.stride(0)), _lib.ptr(cs), _lib.ptr(powers), _f(s.dim ** -0.5), _f(eps), _lib.ptr(state),
+        _ll(state.stride(0)), _lib.ptr(rows.prev), _lib.ptr(rows.next), _lib.ptr(out), _ll(out.stride(0)), proj.shape[0], s.heads,
+        s.dim, s.vdim, s.rot, int(proj.dtype == torch.float32), _lib.stream_ptr())
+    _lib.check(rc, "ts_retention_step")
+
+
+def retention_scan(proj, s: RetentionShape, powers, cs, rows: StreamRows, state, portions, blocked: bool = False) -> torch.Tensor:
+    """As `delta_scan`; `blocked` takes bf16 projections."""
+    T, dev = proj.shape[0], proj.device
+    o = torch.empty(T, s.out_width, dtype=torch.float32, device=dev)
+    lib = _lib.load("recurrent")
+    if blocked and _blocked(s.dim, s.vdim) and proj.stride(0) % 8 == 0:
+        rt, kt = (torch.empty(T, s.qk_width, dtype=torch.float32, device=dev) for _ in range(2))
+        coef = _workspace(T, portions, SCAN_RETENTION, s.heads, device=dev)
+        rc = lib.ts_retention_block_scan(
+            _lib.ptr(proj), _ll(proj.stride(0)), _lib.ptr(cs), _lib.ptr(powers), _f(s.dim ** -0.5), _lib.ptr(rt), _lib.ptr(kt),
+            _lib.ptr(coef), _lib.ptr(state), _ll(state.stride(0)), _lib.ptr(rows.prev), _lib.ptr(rows.next), _lib.ptr(portions.cu),
+            portions.count, portions.longest, _lib.ptr(o), s.heads, s.dim, s.vdim, s.rot, _lib.stream_ptr())
+        _lib.check(rc, "ts_retention_block_scan")
+        return o
+    rc = lib.ts_retention_scan(
+        _lib.ptr(proj), _ll(proj.stride(0)), _lib.ptr(cs), _lib.ptr(powers), _f(s.dim ** -0.5), _lib.ptr(state),
+        _ll(state.stride(0)), _lib.ptr(rows.prev), _lib.ptr(rows.next), _lib.ptr(portions.cu), portions.count, _lib.ptr(o), s.heads,
+        s.dim, s.vdim, s.rot, int(proj.dtype == torch.float32), _lib.stream_ptr())
+    _lib.check(rc, "ts_retention_scan")
     return o

@@ -190,9 +190,25 @@ def postnorm_final(x, y, w, final_w, eps: float, out_rows, act_dtype) -> torch.T
 
 
 # ---------------------------------------------------------------------------------------------- input-normed boundaries
+@dataclass
+class ElementGate:
+    """Factor sigmoid(logits + bias) of every element of an addend."""
+    logits: torch.Tensor      # [T, W], activation dtype
+    bias: torch.Tensor        # [W] fp32
+
+
+def _prenorm_norm(x, w, eps, base):
+    return x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) * (base + w)
+
+
 def _prenorm_sum(x, y, y_gate, experts):
     if y is not None:
-        x = x + (y.float() if y_gate is None else y.float() * torch.sigmoid(y_gate)[:, None])
+        y = y.float()
+        if isinstance(y_gate, ElementGate):
+            y = y * torch.sigmoid(y_gate.logits.float() + y_gate.bias)
+        elif y_gate is not None:
+            y = y * torch.sigmoid(y_gate)[:, None]
+        x = x + y
     if experts is not None:
         e, dest, w = experts
         idx = torch.arange(w.numel()) if dest is None else dest.long()
@@ -200,44 +216,47 @@ def _prenorm_sum(x, y, y_gate, experts):
     return x
 
 
-def _prenorm_raw(tok, table, x, y, y_gate, experts, w, eps, x_out, h, rows, out_rows):
+def _prenorm_raw(tok, table, x, y, y_gate, experts, w, base, eps, x_out, h, rows, out_rows):
+    e_gate, e_bias = (y_gate.logits, y_gate.bias) if isinstance(y_gate, ElementGate) else (None, None)
+    y_gate = None if e_gate is not None else y_gate
     e, dest, route_w = experts if experts is not None else (None, None, None)
     rc = _lib.load("stream").ts_stream_prenorm(
         _lib.ptr(tok), _lib.ptr(table), 0 if table is None else table.shape[0], _lib.ptr(x), _lib.ptr(y),
-        _ll(0 if y is None else y.stride(0)), _lib.ptr(y_gate), _ll(0 if y_gate is None else y_gate.stride(0)), _lib.ptr(e),
-        _lib.ptr(dest), _lib.ptr(route_w), 0 if route_w is None else route_w.shape[1], _lib.ptr(w), _f(eps), _lib.ptr(x_out),
+        _ll(0 if y is None else y.stride(0)), _lib.ptr(y_gate), _ll(0 if y_gate is None else y_gate.stride(0)),
+        _lib.ptr(e_gate), _ll(0 if e_gate is None else e_gate.stride(0)), _lib.ptr(e_bias), _lib.ptr(e), _lib.ptr(dest),
+        _lib.ptr(route_w), 0 if route_w is None else route_w.shape[1], _lib.ptr(w), _f(base), _f(eps), _lib.ptr(x_out),
         _lib.ptr(h), rows, _lib.ptr(out_rows), 0 if out_rows is None else out_rows.numel(), h.shape[1], _fp32(h),
         _lib.stream_ptr())
     _lib.check(rc, "ts_stream_prenorm")
 
 
-def prenorm_embed(tok, table, w, eps: float):
-    """x = table[tok] (fp32); returns (x, h) with h = x / rms(x) * (1 + w) in the table's dtype."""
+def prenorm_embed(tok, table, w, eps: float, base: float = 1.0):
+    """x = table[tok] (fp32); returns (x, h) with h = x / rms(x) * (base + w) in the table's dtype."""
     if not tok.is_cuda:
         x = table[tok.long()].float()
-        return x, offset_rmsnorm(x, w, eps).to(table.dtype)
+        return x, _prenorm_norm(x, w, eps, base).to(table.dtype)
     x = torch.empty(tok.shape[0], table.shape[1], dtype=torch.float32, device=tok.device)
     h = torch.empty(x.shape, dtype=table.dtype, device=tok.device)
-    _prenorm_raw(tok, table, None, None, None, None, w, eps, x, h, tok.shape[0], None)
+    _prenorm_raw(tok, table, None, None, None, None, w, base, eps, x, h, tok.shape[0], None)
     return x, h
 
 
-def prenorm(x, y, y_gate, experts, w, eps: float, act_dtype):
-    """x' = x + y * sigmoid(y_gate) + the weighted sum of a token's experts; returns (x', x' / rms(x') * (1 + w)).
-    y [T, W] or None, y_gate fp32 [T] logits or None (factor one), experts of ops/moe.routed_experts or None."""
+def prenorm(x, y, y_gate, experts, w, eps: float, act_dtype, base: float = 1.0):
+    """x' = x + y * sigmoid(y_gate) + the weighted sum of a token's experts; returns (x', x' / rms(x') * (base + w)).
+    y [T, W] or None, y_gate fp32 [T] logits, an ElementGate or None (factor one), experts of ops/moe.routed_experts or None."""
     if not x.is_cuda:
         x = _prenorm_sum(x, y, y_gate, experts)
-        return x, offset_rmsnorm(x, w, eps).to(act_dtype)
+        return x, _prenorm_norm(x, w, eps, base).to(act_dtype)
     x_out, h = torch.empty_like(x), torch.empty(x.shape, dtype=act_dtype, device=x.device)
-    _prenorm_raw(None, None, x, y, y_gate, experts, w, eps, x_out, h, x.shape[0], None)
+    _prenorm_raw(None, None, x, y, y_gate, experts, w, base, eps, x_out, h, x.shape[0], None)
     return x_out, h
 
 
-def prenorm_final(x, y, y_gate, experts, w, eps: float, out_rows, act_dtype) -> torch.Tensor:
+def prenorm_final(x, y, y_gate, experts, w, eps: float, out_rows, act_dtype, base: float = 1.0) -> torch.Tensor:
     """The norm of `prenorm` for the rows `out_rows` (int32)."""
     if not x.is_cuda:
-        return offset_rmsnorm(_prenorm_sum(x, y, y_gate, experts)[out_rows.long()], w, eps).to(act_dtype)
+        return _prenorm_norm(_prenorm_sum(x, y, y_gate, experts)[out_rows.long()], w, eps, base).to(act_dtype)
     h = torch.empty(out_rows.numel(), x.shape[1], dtype=act_dtype, device=x.device)
     if out_rows.numel():
-        _prenorm_raw(None, None, x, y, y_gate, experts, w, eps, None, h, x.shape[0], out_rows)
+        _prenorm_raw(None, None, x, y, y_gate, experts, w, base, eps, None, h, x.shape[0], out_rows)
     return h

@@ -1,6 +1,8 @@
 """Attention with grouped queries over a part of the keys (csrc/window.cu, csrc/latent_prefill.cu): a sliding window, with or
-without the sequence's first positions, or chunks.  Optional bias, per-head RMS norm of queries and keys, rotary embedding of
-part of a head, a gate on the result; keys and values of unlike sizes side by side in one paged cache row per token.
+without the sequence's first positions, chunks, or all of them (`masks.UNBOUNDED`).  Optional bias, per-head RMS norm of queries and
+keys, a factor of the queries that grows with the position, rotary embedding of part of a head, a gate on the result; keys and
+values of unlike sizes side by side in one paged cache row per token.  Weights are a softmax of the scores or their sigmoids;
+scores may carry a number per head and a slope per head over the distance (`ScoreBias`).
 
 `attend_rows` serves single query rows (decoding, fp32, sizes the tensor-core prefill kernel does not take),
 `attend_portions` portions of prompts in bf16.  Tensors on the CPU take PyTorch math.
@@ -34,6 +36,8 @@ class WindowShape:
     chunked: bool = False
     pairs: bool = False   # rotation partners: coordinates 2 i and 2 i + 1 instead of i and i + rot / 2
     values_are_keys: bool = False   # values are the keys as projected, before norm and rotation
+    sigmoid: bool = False           # weights are sigmoids of the scores, not normalized over keys
+    temperature: tuple[float, int] | None = None   # (coef, every): queries times 1 + coef ln(floor((p + 1) / every) + 1)
 
     @property
     def mask(self) -> KeyMask:
@@ -62,8 +66,24 @@ class WindowShape:
         return -(-self.kv_width // 8) * 8
 
 
+@dataclass
+class ScoreBias:
+    """Terms of a head's scores besides q . k * scale, fp32 [heads]; either may be None."""
+    slopes: torch.Tensor | None = None    # times the distance of query and key, taken off
+    add: torch.Tensor | None = None
+
+
+NO_BIAS = ScoreBias()
+
+
+def distance_slopes(heads: int) -> torch.Tensor:
+    """Slopes 2^(-8 (h + 1) / heads), a geometric series over the heads that ends at 2^-8."""
+    return torch.tensor([2.0 ** (-8.0 * (h + 1) / heads) for h in range(heads)], dtype=torch.float32)
+
+
 @functools.lru_cache(maxsize=None)
 def portions_supported(s: WindowShape) -> bool:
+    """Whether `attend_portions` takes these sizes (a bias of the scores: only with sigmoid weights)."""
     return s.scale > 0 and bool(_lib.load("latent_prefill").ts_latent_prefill_supported(s.dim, 0, s.vdim))
 
 
@@ -96,9 +116,9 @@ def angles(inv_freq: torch.Tensor, pos: torch.Tensor, magnitude: float = 1.0) ->
 
 
 def prepare(proj: torch.Tensor, s: WindowShape, q_norm, k_norm, eps: float, cs: torch.Tensor | None, slots, cache,
-            bias: torch.Tensor | None = None) -> None:
+            bias: torch.Tensor | None = None, pos: torch.Tensor | None = None) -> None:
     """proj [T, >= q_width + kv_width] = (queries | keys | values | ...); cs of `angles`; norms and bias (fp32, of queries and
-    keys) may be None.  Norms and rotates queries and keys in place and writes keys and values to cache rows `slots`; the
+    keys) may be None; pos int32 [T] for shapes with a temperature.  Norms and rotates queries and keys in place and writes keys and values to cache rows `slots`; the
     value columns of proj are written when the values are the keys."""
     T = proj.shape[0]
     if not proj.is_cuda:
@@ -109,20 +129,24 @@ def prepare(proj: torch.Tensor, s: WindowShape, q_norm, k_norm, eps: float, cs: 
         if s.values_are_keys:
             proj[:, s.q_width + kw:s.q_width + s.kv_width] = qk[:, s.q_width:]
         q, k = qk[:, :s.q_width].view(T, s.heads, s.dim), qk[:, s.q_width:].view(T, s.kv_heads, s.dim)
-        proj[:, :s.q_width] = _norm_rotate(q, q_norm, eps, cs, s).reshape(T, -1)
+        q = _norm_rotate(q, q_norm, eps, cs, s)
+        if s.temperature is not None:
+            coef, every = s.temperature
+            q = q * (1 + coef * torch.log((pos + 1).div(every, rounding_mode="floor") + 1.0))[:, None, None]
+        proj[:, :s.q_width] = q.reshape(T, -1)
         proj[:, s.q_width:s.q_width + kw] = _norm_rotate(k, k_norm, eps, cs, s).reshape(T, -1)
         cache.view(-1, s.row_width)[slots, :s.kv_width] = proj[:, s.q_width:s.q_width + s.kv_width]
         return
+    coef, every = s.temperature or (0.0, 0)
     rc = _lib.load("window").ts_window_prep(
         _lib.ptr(proj), _ll(proj.stride(0)), _lib.ptr(bias), _lib.ptr(q_norm), _lib.ptr(k_norm), _f(eps), _lib.ptr(cs),
         _lib.ptr(slots), _lib.ptr(cache), T, s.heads, s.kv_heads, s.dim, s.vdim, s.rot, int(s.pairs), int(s.values_are_keys),
-        s.row_width, int(proj.dtype == torch.float32),
-        _lib.stream_ptr())
+        _lib.ptr(pos if every else None), _f(coef), every, s.row_width, int(proj.dtype == torch.float32), _lib.stream_ptr())
     _lib.check(rc, "ts_window_prep")
 
 
 def attend_rows(proj: torch.Tensor, s: WindowShape, cache, block_table, row_seq, row_len, max_len: int, out: torch.Tensor,
-                out_scale: float = 1.0, gate: torch.Tensor | None = None) -> None:
+                out_scale: float = 1.0, gate: torch.Tensor | None = None, bias: ScoreBias = NO_BIAS) -> None:
     """out [T, out_width] = out_scale * attention of the query rows proj[:, :q_width]; row r belongs to row `row_seq[r]` of
     the block table and sees the keys before row_len[r] that the mask leaves.  `gate` ([T, heads] or [T, out_width]): the
     result is multiplied by its sigmoid."""
@@ -136,7 +160,12 @@ def attend_rows(proj: torch.Tensor, s: WindowShape, cache, block_table, row_seq,
             q = proj[t, :s.q_width].float().view(s.kv_heads, -1, s.dim)
             k = rows[:, :kw].view(-1, s.kv_heads, s.dim)
             v = rows[:, kw:s.kv_width].view(-1, s.kv_heads, s.vdim)
-            w = torch.softmax(torch.einsum("ghd,jgd->ghj", q, k) * s.scale, -1)
+            sc = torch.einsum("ghd,jgd->ghj", q, k) * s.scale
+            if bias.slopes is not None:
+                sc = sc - bias.slopes.view(s.kv_heads, -1, 1) * (int(row_len[t]) - 1 - j).float()
+            if bias.add is not None:
+                sc = sc + bias.add.view(s.kv_heads, -1, 1)
+            w = torch.sigmoid(sc) if s.sigmoid else torch.softmax(sc, -1)
             o = (torch.einsum("ghj,jgv->ghv", w, v) * out_scale).reshape(s.heads, s.vdim)
             if gate is not None:
                 o = o * torch.sigmoid(gate[t].float()).view(s.heads, -1)
@@ -154,13 +183,13 @@ def attend_rows(proj: torch.Tensor, s: WindowShape, cache, block_table, row_seq,
     rc = lib.ts_window_attend(
         _lib.ptr(proj), _ll(proj.stride(0)), _lib.ptr(cache), _lib.ptr(block_table), block_table.shape[1], _lib.ptr(row_seq),
         _lib.ptr(row_len), _lib.ptr(out), _ll(out.stride(0)), _lib.ptr(po), _lib.ptr(pl), T, s.heads, s.kv_heads, s.dim,
-        s.vdim, s.row_width, bs, s.window, s.keep, int(s.chunked), keys, splits, _f(s.scale), _f(out_scale), gp, gld, mode, fp32,
-        _lib.stream_ptr())
+        s.vdim, s.row_width, bs, s.window, s.keep, int(s.chunked), keys, splits, _f(s.scale), _f(out_scale), _lib.ptr(bias.slopes),
+        _lib.ptr(bias.add), int(s.sigmoid), gp, gld, mode, fp32, _lib.stream_ptr())
     _lib.check(rc, "ts_window_attend")
 
 
 def attend_portions(proj: torch.Tensor, s: WindowShape, rows: torch.Tensor | None, cu_q, cu_k, max_q: int, out: torch.Tensor,
-                    out_scale: float = 1.0, gate: torch.Tensor | None = None) -> None:
+                    out_scale: float = 1.0, gate: torch.Tensor | None = None, bias: ScoreBias = NO_BIAS) -> None:
     """Portions of prompts, bf16: queries proj[:, :q_width]; keys and values of every sequence, in key order, in `rows`
     [Tk, row_width] (None: exactly the portions' own, beside the queries).  cu_q / cu_k int32 offsets of every sequence
     (its queries are the last of its keys): the kept first positions, if they are not part of the window's run, then the
@@ -172,5 +201,5 @@ def attend_portions(proj: torch.Tensor, s: WindowShape, rows: torch.Tensor | Non
         _lib.ptr(proj), _ll(proj.stride(0)), _ll(proj.shape[0]), ctypes.c_void_p(at),
         ctypes.c_void_p(at + s.kv_heads * s.dim * proj.element_size()), _ll(src.stride(0)), _ll(src.shape[0]), _lib.ptr(cu_q),
         _lib.ptr(cu_k), cu_q.numel() - 1, max_q, s.heads, s.kv_heads, s.dim, s.vdim, s.window, s.keep, int(s.chunked),
-        _f(s.scale), _f(out_scale), gp, gld, mode, _lib.ptr(out), _ll(out.stride(0)), _lib.stream_ptr())
+        _f(s.scale), _f(out_scale), _lib.ptr(bias.slopes), _lib.ptr(bias.add), int(s.sigmoid), gp, gld, mode, _lib.ptr(out), _ll(out.stride(0)), _lib.stream_ptr())
     _lib.check(rc, "ts_window_prefill")

@@ -417,6 +417,9 @@ register_models_from_meta([
     ModelInfo("kabulix", "trainscale", ("3B",), "KabulixForCausalLM", attention="sliding window with sinks, latent, chunked",
               mlp="dense (gelu glu), moe (silu glu, grouped sigmoid router, shared expert)", norm="rmsnorm (offset weight)",
               notes="serving only: models/kabulix.py; window, chunk and latent caches"),
+    ModelInfo("lovurax", "trainscale", ("2B",), "LovuraxForCausalLM", attention="retention, sigmoid with distance slopes, latent",
+              mlp="dense (xIELU)", norm="rmsnorm",
+              notes="serving only: models/lovurax.py; key/value and latent caches, matrix state per sequence"),
     ModelInfo("llava", "llava-hf", ("7B", "13B"), "LlavaForConditionalGeneration", supported=False, notes="vision tower not covered"),
 ])
 
