@@ -317,7 +317,7 @@ def main():
     ap.add_argument("--serve", nargs="*", default=None, metavar="SIZE",
                     help="instead: prefill / decode throughput of a served design beside the closest model at these "
                          "sizes (default all), with per-op roofline fractions; one GPU")
-    ap.add_argument("--serve-model", default="mezilix", choices=["mezilix", "vibepel", "kabulix"], help="design that --serve measures")
+    ap.add_argument("--serve-model", default="mezilix", choices=["mezilix", "vibepel", "kabulix", "lovurax"], help="design that --serve measures")
     args = ap.parse_args()
     if args.serve is not None:
         return run_serving(args)

@@ -1133,7 +1133,8 @@ struct RetentionParams {
   const void* proj;            // rows [q H x D | k H x D | v H x V | gate H x V]
   long long ld;
   const float* angles;         // [rows][cos (rot / 2) | sin (rot / 2)]
-  const float* powers;         // [H][RT_POWERS] g^0, g^1, ...
+  const float* powers;         // [H][powers_ld] g^0, g^1, ... (BS_BLOCK + 1 of them at least)
+  int powers_ld;
   float k_scale, eps;
   float* state;
   long long state_ld;
@@ -1145,8 +1146,6 @@ struct RetentionParams {
   long long out_ld;
   int rows, H, D, V, rot;
 };
-constexpr int RT_POWERS = BS_BLOCK + 1;
-
 // coordinate c of a head whose projected row is x, rotated (halves) and scaled
 template <typename T>
 __device__ __forceinline__ float rotated(const T* x, int c, int rot, const float* cs, float scale) {
@@ -1168,7 +1167,7 @@ __global__ void __launch_bounds__(256) retention_scan_kernel(RetentionParams p) 
   const int row0 = p.cu[blockIdx.z], n = p.cu[blockIdx.z + 1] - row0, D = p.D, V = p.V;
   if (n <= 0) return;
   const int prev = p.row_prev[row0], next = p.row_next[row0 + n - 1];
-  const float g = p.powers[h * RT_POWERS + 1];
+  const float g = p.powers[h * p.powers_ld + 1];
   const long long head = static_cast<long long>(h) * D * V;
   float S[NR];
 #pragma unroll
@@ -1234,7 +1233,7 @@ __global__ void __launch_bounds__(128) retention_blocks_kernel(RetentionParams p
   const int D = p.D, ds = D + 1;
   float* qs = smf + warp * 2 * BS_BLOCK * ds;
   float* ks = qs + BS_BLOCK * ds;
-  const float* pw = p.powers + h * RT_POWERS;
+  const float* pw = p.powers + h * p.powers_ld;
   const long long at = (first_block(p.cu, z) + blockIdx.x) * p.H + h;
   for (int c = lane; c < D; c += 32) {
 #pragma unroll
@@ -1285,7 +1284,7 @@ __global__ void __launch_bounds__(RTS_THREADS) retention_step_kernel(RetentionPa
   const long long head = static_cast<long long>(h) * D * V;
   const float* S = prev >= 0 ? p.state + prev * p.state_ld + head : nullptr;
   float* N = next >= 0 ? p.state + next * p.state_ld + head : nullptr;
-  const float g = p.powers[h * RT_POWERS + 1];
+  const float g = p.powers[h * p.powers_ld + 1];
   for (int c = tid; c < D; c += RTS_THREADS) {
     qs[c] = rotated(x + h * D, c, p.rot, cs, 1.f);
     ks[c] = rotated(x + (p.H + h) * D, c, p.rot, cs, p.k_scale);
@@ -1851,28 +1850,25 @@ extern "C" int ts_wkv_step(const void* rkvg, long long ld, const float* w_raw, c
   return (int)cudaGetLastError();
 }
 
-static int retention_params(RetentionParams& p, const void* proj, long long ld, const float* angles, const float* powers,
+static int retention_params(RetentionParams& p, const void* proj, long long ld, const float* angles, const float* powers, int powers_ld,
                             float k_scale, float* state, long long state_ld, const int* row_prev, const int* row_next, int H, int D,
                             int V, int rot) {
   if (H <= 0 || H > 65535 || D <= 0 || D > 256 || V <= 0 || V > 512 || rot < 0 || rot > D || rot % 2 ||
-      state_ld < static_cast<long long>(H) * D * V)
+      powers_ld <= BS_BLOCK || state_ld < static_cast<long long>(H) * D * V)
     return -10;
   p = {};
-  p.proj = proj; p.ld = ld; p.angles = angles; p.powers = powers; p.k_scale = k_scale; p.state = state; p.state_ld = state_ld;
+  p.proj = proj; p.ld = ld; p.angles = angles; p.powers = powers; p.powers_ld = powers_ld; p.k_scale = k_scale; p.state = state; p.state_ld = state_ld;
   p.row_prev = row_prev; p.row_next = row_next; p.H = H; p.D = D; p.V = V; p.rot = rot;
   return 0;
 }
 
-// Length of a head's row of powers of its decay, from g^0 on.
-extern "C" int ts_retention_powers() { return RT_POWERS; }
-
 // Single rows of retention: projection -> out [rows][out_ld] = norm * silu(gate), state advanced.
-extern "C" int ts_retention_step(const void* proj, long long ld, const float* angles, const float* powers, float k_scale, float eps,
+extern "C" int ts_retention_step(const void* proj, long long ld, const float* angles, const float* powers, int powers_ld, float k_scale, float eps,
                                  float* state, long long state_ld, const int* row_prev, const int* row_next, void* out,
                                  long long out_ld, int rows, int H, int D, int V, int rot, int fp32, void* stream) {
   if (rows <= 0) return 0;
   RetentionParams p;
-  if (int e = retention_params(p, proj, ld, angles, powers, k_scale, state, state_ld, row_prev, row_next, H, D, V, rot)) return e;
+  if (int e = retention_params(p, proj, ld, angles, powers, powers_ld, k_scale, state, state_ld, row_prev, row_next, H, D, V, rot)) return e;
   p.eps = eps; p.out = out; p.out_ld = out_ld; p.rows = rows;
   const bool vec = V % 4 == 0 && state_ld % 4 == 0;
   const int nvec = vec ? V / 4 : V, groups = RTS_THREADS / (nvec < RTS_THREADS ? nvec : RTS_THREADS);
@@ -1898,12 +1894,12 @@ template <typename T> static int dispatch_retention_scan(const RetentionParams& 
 }
 
 // Portions of retention: o [rows][H V] of the recurrence, the last state of every portion to its state row.  fp32 arithmetic.
-extern "C" int ts_retention_scan(const void* proj, long long ld, const float* angles, const float* powers, float k_scale,
+extern "C" int ts_retention_scan(const void* proj, long long ld, const float* angles, const float* powers, int powers_ld, float k_scale,
                                  float* state, long long state_ld, const int* row_prev, const int* row_next, const int* cu,
                                  int portions, float* o, int H, int D, int V, int rot, int fp32, void* stream) {
   if (portions <= 0) return 0;
   RetentionParams p;
-  if (int e = retention_params(p, proj, ld, angles, powers, k_scale, state, state_ld, row_prev, row_next, H, D, V, rot)) return e;
+  if (int e = retention_params(p, proj, ld, angles, powers, powers_ld, k_scale, state, state_ld, row_prev, row_next, H, D, V, rot)) return e;
   if (portions > 65535) return -10;
   p.cu = cu; p.o = o;
   return fp32 ? dispatch_retention_scan<float>(p, portions, ST(stream)) : dispatch_retention_scan<__nv_bfloat16>(p, portions, ST(stream));
@@ -1911,13 +1907,13 @@ extern "C" int ts_retention_scan(const void* proj, long long ld, const float* an
 
 // Portions of retention in bf16 models: as ts_retention_scan, on the tensor cores.  Workspaces: rt, kt [rows][H D], coef
 // [blocks][H][BS_COEF_RET].
-extern "C" int ts_retention_block_scan(const void* proj, long long ld, const float* angles, const float* powers, float k_scale,
+extern "C" int ts_retention_block_scan(const void* proj, long long ld, const float* angles, const float* powers, int powers_ld, float k_scale,
                                        float* rt, float* kt, float* coef, float* state, long long state_ld, const int* row_prev,
                                        const int* row_next, const int* cu, int portions, int max_rows, float* o, int H, int D,
                                        int V, int rot, void* stream) {
   if (portions <= 0) return 0;
   RetentionParams r;
-  if (int e = retention_params(r, proj, ld, angles, powers, k_scale, state, state_ld, row_prev, row_next, H, D, V, rot)) return e;
+  if (int e = retention_params(r, proj, ld, angles, powers, powers_ld, k_scale, state, state_ld, row_prev, row_next, H, D, V, rot)) return e;
   if (!blocked_ok(D, V) || portions > 65535 || max_rows <= 0 || ld % 8 || (reinterpret_cast<uintptr_t>(proj) & 15u)) return -10;
   r.cu = cu;
   const size_t smem = 4 * 2 * BS_BLOCK * (D + 1) * sizeof(float);

@@ -16,7 +16,7 @@ from typing import Callable
 
 import torch
 
-from ..ops.masks import KeyMask
+from ..ops.masks import UNBOUNDED, KeyMask
 from .batch import HostBatch, StepEntry
 from .engine import EngineConfig, EngineCore
 
@@ -42,6 +42,12 @@ KABULIX_SIZES = {
                experts=32, top=4, groups=8, kept=4, ff=1536),
     "4k": dict(layers=8, width=4096, heads=32, kv=8, dim=128, window=4096, keep=4, chunk=4096, ldim=128, lrot=64, lvdim=128, rank=512,
                experts=64, top=6, groups=8, kept=4, ff=1536),
+}
+# layers take turns: retention, sigmoid attention, retention, latent attention
+LOVURAX_SIZES = {
+    "1k": dict(layers=12, width=1024, heads=8, kv=2, dim=128, rheads=4, rdim=128, rvdim=256, ldim=64, lvdim=64, rank=256, ff=4096),
+    "2k": dict(layers=16, width=2048, heads=16, kv=4, dim=128, rheads=8, rdim=128, rvdim=256, ldim=128, lvdim=128, rank=512, ff=8192),
+    "4k": dict(layers=8, width=4096, heads=32, kv=8, dim=128, rheads=16, rdim=128, rvdim=256, ldim=128, lvdim=128, rank=512, ff=16384),
 }
 VOCAB = 32000
 FP32_TFLOPS = 74.4            # nominal: 148 SMs x 128 lanes x 2 x 1.965 GHz
@@ -93,6 +99,15 @@ def build_kabulix(z: dict):
                                       latent_rot=z["lrot"], latent_vdim=z["lvdim"], rank=z["rank"], latent_window=z["window"],
                                       ff=ff * (z["top"] + 1), experts=z["experts"], top=z["top"], expert_ff=ff, shared_ff=ff,
                                       groups=z["groups"], keep_groups=z["kept"], rot_dims=z["dim"] // 2),
+                       torch.bfloat16, "cuda", seed=0)
+
+
+def build_lovurax(z: dict):
+    from ..models.lovurax import build_model, pattern_config
+    kinds = ("rarl" * z["layers"])[:z["layers"]]
+    return build_model(pattern_config(kinds, vocab=VOCAB, width=z["width"], heads=z["heads"], kv_heads=z["kv"], dim=z["dim"],
+                                      ret_heads=z["rheads"], ret_dim=z["rdim"], ret_vdim=z["rvdim"], latent_dim=z["ldim"],
+                                      latent_vdim=z["lvdim"], rank=z["rank"], ff=z["ff"]),
                        torch.bfloat16, "cuda", seed=0)
 
 
@@ -350,10 +365,54 @@ def kabulix_table(z: dict, rows: int, lengths: list[tuple[int, int]]) -> list[tu
     ]
 
 
+def lovurax_table(z: dict, rows: int, lengths: list[tuple[int, int]]) -> list[tuple]:
+    from ..ops import gemm, grouped, latent_attention as latent, recurrent, stream, window_attention as window
+    W = z["width"]
+    keys, pairs = _seen(lengths, KeyMask(UNBOUNDED))
+
+    def boundary(a, k, out):
+        final = isinstance(out, torch.Tensor)                  # last boundary: only the wanted rows
+        T = (out if final else out[0]).shape[0]
+        return (4 + 2 + 2 + (0 if final else 4) + 2) * T * W, 0.0
+
+    return [
+        (stream, "prenorm_embed", "embedding, norm", lambda a, k, o: (a[0].shape[0] * W * (2 + 4 + 2), 0.0)),
+        (stream, "prenorm", "gated sum, norm", boundary),
+        (stream, "prenorm_final", "last norm", boundary),
+        (gemm, "serve_linear", _linear_name("gemm"), _linear_cost),
+        (gemm, "matmul_nt", _linear_name("gemm"), _linear_cost),
+        (window, "prepare", "head norms, temperature, cache write",
+         lambda a, k, o: (a[0].shape[0] * 2 * (2 * (a[1].q_width + a[1].kv_heads * a[1].dim) + a[1].kv_heads * a[1].vdim +
+                                               a[1].kv_width), 0.0)),
+        (latent, "prepare", "latent norm, cache write",
+         lambda a, k, o: (a[0].shape[0] * 2 * (a[1].rank + a[1].row_width * (2 if o is not None else 1)), 0.0)),
+        (latent, "gather_rows", "key gather", lambda a, k, o: (2 * _bytes(o), 0.0)),
+        (window, "attend_rows", "attention (sigmoid, rows)",
+         lambda a, k, o: (keys * a[1].kv_width * 2 + a[0].shape[0] * (a[1].q_width + 2 * a[1].out_width) * 2,
+                          2.0 * pairs * a[1].heads * (a[1].dim + a[1].vdim))),
+        (window, "attend_portions", "attention (sigmoid, portions)",
+         lambda a, k, o: (a[0].shape[0] * (a[1].q_width + a[1].kv_width + 2 * a[1].out_width) * 2,
+                          2.0 * pairs * a[1].heads * (a[1].dim + a[1].vdim))),
+        (latent, "attend_latent", "attention (latent space)",
+         lambda a, k, o: (keys * a[2].row_width * 2 + 2 * _bytes(a[0]), 4.0 * pairs * a[2].heads * a[2].rank)),
+        (latent, "attend_expanded", "attention (latent, portions)",
+         lambda a, k, o: (_bytes(a[1], a[7]) + a[0].shape[0] * a[3].q_width * 2,
+                          2.0 * pairs * a[3].heads * (a[3].dim + a[3].vdim))),
+        (grouped, "head_linear", lambda a, o: f"per-head projection {a[1].shape[1]}x{a[1].shape[2]}",
+         lambda a, k, o: (_bytes(a[0], a[1], o), 2.0 * a[0].shape[0] * a[1].numel())),
+        (recurrent, "retention_step", "retention step",
+         lambda a, k, o: (a[0].shape[0] * ((a[1].proj_width + a[1].out_width) * 2 + 2 * 4 * a[1].state_width), 0.0)),
+        # two fp32 products of every state element per token
+        (recurrent, "retention_scan", "retention scan",
+         lambda a, k, o: (a[0].shape[0] * (2 * a[1].qk_width + a[1].out_width) * 2 + _bytes(o), 0.0, 4.0 * o.numel() * a[1].dim)),
+        (recurrent, "gated_norm", "gated norm", lambda a, k, o: (_bytes(a[0]) + 2 * _bytes(a[4]), 0.0)),
+    ]
+
+
 def closest_table(z: dict, rows: int, lengths: list[tuple[int, int]], runner) -> list[tuple]:
     from ..ops import activation, gemm, moe, norm, rope
     W, H, D = z["width"], z["heads"], z.get("vdim") or z["dim"]
-    keys, pairs = _seen(lengths, KeyMask(1 << 30))
+    keys, pairs = _seen(lengths, KeyMask(UNBOUNDED))
     hkv = z.get("kv") or max(1, H // 4)
 
     def grouped_cost(a, k, out):
@@ -386,7 +445,8 @@ class Design:
 
 DESIGNS = {"mezilix": Design(SIZES, build_mezilix, build_closest, mezilix_table),
            "vibepel": Design(VIBEPEL_SIZES, build_vibepel, build_closest_dense, vibepel_table),
-           "kabulix": Design(KABULIX_SIZES, build_kabulix, build_closest, kabulix_table)}
+           "kabulix": Design(KABULIX_SIZES, build_kabulix, build_closest, kabulix_table),
+           "lovurax": Design(LOVURAX_SIZES, build_lovurax, build_closest_dense, lovurax_table)}
 
 
 def measure(design: str, name: str, peaks: dict, prompts: int = 2, prompt_len: int = 4096, batches=(8, 64), context: int = 2048,

@@ -363,7 +363,7 @@ class LovuraxLayer(nn.Module):
 
 
 class LovuraxForCausalLM(ServedDecoder):
-    LIBRARIES = ("stream", "window", "recurrent", "latent", "latent_prefill", "skinny", "gemm")
+    LIBRARIES = ("stream", "window", "recurrent", "retention", "latent", "latent_prefill", "skinny", "gemm")
 
     def __init__(self, cfg: LovuraxConfig):
         super().__init__()

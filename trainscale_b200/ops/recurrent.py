@@ -1,5 +1,5 @@
 """Recurrent mixers with an fp32 matrix state per head: the gated delta rule (with short convolutions in front), WKV time
-mixing and retention (csrc/recurrent.cu).
+mixing (csrc/recurrent.cu) and retention (csrc/recurrent.cu; csrc/retention.cu for long portions).
 
 All run over a flattened batch whose first rows are single tokens (decoding: one launch from projection to gated norm) and
 whose other rows are portions of prompts (a scan).  A sequence's state row holds [convolution inputs or token-shift row, if any |
@@ -21,6 +21,7 @@ from .stream import StreamRows
 _ll, _f = ctypes.c_longlong, ctypes.c_float
 MAX_HEAD = 256           # largest key or value size of a head
 MAX_RETENTION_VALUE = 512  # retention: largest value size
+RETENTION_CHUNK = 128      # tokens of a chunk of csrc/retention.cu
 SCAN_WKV, SCAN_DELTA, SCAN_RETENTION = 0, 1, 2
 
 
@@ -103,10 +104,10 @@ class RetentionShape:
     def state_width(self) -> int:
         return _up4(self.heads * self.dim * self.vdim)
 
-    def powers(self, n: int = 9) -> torch.Tensor:
-        """fp32 [heads, n] g^0 .. g^(n - 1) of the decays as fp32 numbers."""
+    def powers(self) -> torch.Tensor:
+        """fp32 [heads, RETENTION_CHUNK + 1] g^0, g^1, ... of the decays as fp32 numbers."""
         g = torch.tensor(self.decay, dtype=torch.float32).double()
-        return (g[:, None] ** torch.arange(n, dtype=torch.float64)).float()
+        return (g[:, None] ** torch.arange(RETENTION_CHUNK + 1, dtype=torch.float64)).float()
 
 
 @dataclass
@@ -347,16 +348,37 @@ def retention(proj: torch.Tensor, s: RetentionShape, powers: torch.Tensor, eps: 
         retention_step(proj[:n_single], s, powers, eps, cs, rows, state, out[:n_single])
     if n_single < T:
         tail = StreamRows(rows.prev[n_single:], rows.next[n_single:])
-        part = proj[n_single:]
-        o = retention_scan(part, s, powers, cs[n_single:], tail, state, portions, proj.dtype == torch.bfloat16)
+        part, bf16 = proj[n_single:], proj.dtype == torch.bfloat16
+        if bf16 and portions.longest >= CHUNKS_FROM and _chunked(s.dim, s.vdim) and part.stride(0) % 8 == 0:
+            return retention_chunks(part, s, powers, eps, cs[n_single:], tail, state, portions, out[n_single:])
+        o = retention_scan(part, s, powers, cs[n_single:], tail, state, portions, bf16)
         gate = part[:, 2 * s.qk_width + s.out_width:s.proj_width]
         gated_norm(o, None, 0, gate, out[n_single:], s.heads, s.vdim, eps)
+
+
+CHUNKS_FROM = 64         # tokens of the longest portion from which chunks side by side beat one block after another
+
+
+@functools.lru_cache(maxsize=None)
+def _chunked(dim: int, vdim: int) -> bool:
+    return bool(_lib.load("retention").ts_retention_chunks_supported(dim, vdim))
+
+
+def retention_chunks(proj, s: RetentionShape, powers, eps: float, cs, rows: StreamRows, state, portions, out) -> None:
+    """Portions, bf16: from projection to gated norm, all chunks of a portion side by side."""
+    lib, T = _lib.load("retention"), proj.shape[0]
+    chunks = torch.empty(lib.ts_retention_chunks_count(T, portions.count), s.heads, s.dim, s.vdim, dtype=torch.float32, device=proj.device)
+    rc = lib.ts_retention_chunks(
+        _lib.ptr(proj), _ll(proj.stride(0)), _ll(T), _lib.ptr(cs), _lib.ptr(powers), powers.shape[1], _f(s.dim ** -0.5), _f(eps),
+        _lib.ptr(chunks), _lib.ptr(state), _ll(state.stride(0)), _lib.ptr(rows.prev), _lib.ptr(rows.next), _lib.ptr(portions.cu),
+        portions.count, portions.longest, _lib.ptr(out), _ll(out.stride(0)), s.heads, s.dim, s.vdim, s.rot, _lib.stream_ptr())
+    _lib.check(rc, "ts_retention_chunks")
 
 
 def retention_step(proj, s: RetentionShape, powers, eps: float, cs, rows: StreamRows, state, out) -> None:
     """Single rows: rotation, state update, norm and gate."""
     rc = _lib.load("recurrent").ts_retention_step(
-        _lib.ptr(proj), _ll(proj.stride(0)), _lib.ptr(cs), _lib.ptr(powers), _f(s.dim ** -0.5), _f(eps), _lib.ptr(state),
+        _lib.ptr(proj), _ll(proj.stride(0)), _lib.ptr(cs), _lib.ptr(powers), powers.shape[1], _f(s.dim ** -0.5), _f(eps), _lib.ptr(state),
         _ll(state.stride(0)), _lib.ptr(rows.prev), _lib.ptr(rows.next), _lib.ptr(out), _ll(out.stride(0)), proj.shape[0], s.heads,
         s.dim, s.vdim, s.rot, int(proj.dtype == torch.float32), _lib.stream_ptr())
     _lib.check(rc, "ts_retention_step")
@@ -371,13 +393,13 @@ def retention_scan(proj, s: RetentionShape, powers, cs, rows: StreamRows, state,
         rt, kt = (torch.empty(T, s.qk_width, dtype=torch.float32, device=dev) for _ in range(2))
         coef = _workspace(T, portions, SCAN_RETENTION, s.heads, device=dev)
         rc = lib.ts_retention_block_scan(
-            _lib.ptr(proj), _ll(proj.stride(0)), _lib.ptr(cs), _lib.ptr(powers), _f(s.dim ** -0.5), _lib.ptr(rt), _lib.ptr(kt),
+            _lib.ptr(proj), _ll(proj.stride(0)), _lib.ptr(cs), _lib.ptr(powers), powers.shape[1], _f(s.dim ** -0.5), _lib.ptr(rt), _lib.ptr(kt),
             _lib.ptr(coef), _lib.ptr(state), _ll(state.stride(0)), _lib.ptr(rows.prev), _lib.ptr(rows.next), _lib.ptr(portions.cu),
             portions.count, portions.longest, _lib.ptr(o), s.heads, s.dim, s.vdim, s.rot, _lib.stream_ptr())
         _lib.check(rc, "ts_retention_block_scan")
         return o
     rc = lib.ts_retention_scan(
-        _lib.ptr(proj), _ll(proj.stride(0)), _lib.ptr(cs), _lib.ptr(powers), _f(s.dim ** -0.5), _lib.ptr(state),
+        _lib.ptr(proj), _ll(proj.stride(0)), _lib.ptr(cs), _lib.ptr(powers), powers.shape[1], _f(s.dim ** -0.5), _lib.ptr(state),
         _ll(state.stride(0)), _lib.ptr(rows.prev), _lib.ptr(rows.next), _lib.ptr(portions.cu), portions.count, _lib.ptr(o), s.heads,
         s.dim, s.vdim, s.rot, int(proj.dtype == torch.float32), _lib.stream_ptr())
     _lib.check(rc, "ts_retention_scan")
