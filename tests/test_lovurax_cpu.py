@@ -377,7 +377,7 @@ def test_cache_spec_presets_and_registry():
     assert all(torch.equal(x, y) for x, y in zip(a.parameters(), b.parameters()))
     assert torch.isfinite(a(torch.tensor([tokens(20, 1)]))).all()
     spec = a.cache_spec()
-    assert spec.has_state and spec.bytes_per_token(2) == 2 * (2 * 128 + 96) and spec.bytes_per_sequence() == 2 * 4 * 2 * 4 * 32 * 64
+    assert spec.has_state and spec.bytes_per_token(2) == 2 * (2 * 128 + 96) and spec.bytes_per_sequence() == 2 * 4 * 2 * 2 * 64 * 128
     assert math.isclose(a.config.layers[0].mixer.shape.decay[0], 1 - 2.0 ** -5)
 
 

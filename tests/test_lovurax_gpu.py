@@ -256,6 +256,43 @@ def test_attend_portions_with_sigmoid_weights(H, G, D, V, sloped, added, size, k
     assert out[:, s.out_width:].abs().sum() == 0
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,G,D,V", [(8, 2, 64, 64), (5, 1, 96, 40), (1, 1, 32, 128), (24, 3, 16, 16)])
+@pytest.mark.parametrize("shift", [-6.0, 30.0])
+def test_sigmoid_weights_that_fade_with_the_distance(dtype, H, G, D, V, shift):
+    """With the scores' bound known, far keys are left out: the result stays that of all keys.  One key stands out as far as the
+    bound allows, just where its weight is still large."""
+    from trainscale_b200.ops import window_attention as wa
+    from trainscale_b200.ops.masks import UNBOUNDED
+    n, bs = 1500, 16
+    s = wa.WindowShape(H, G, D, V, 0, UNBOUNDED, D ** -0.5, sigmoid=True)
+    q, kv = rnd(n, s.q_width, seed=1, dtype=dtype), rnd(n + 4, s.row_width, seed=2, dtype=dtype)
+    slopes, add = wa.distance_slopes(H).cuda(), rnd(H, seed=3) + shift
+    for h in range(H):
+        reach = min(n - 1, int((30.0 + add[h].item()) / slopes[h].item()))          # a score of 30 there has a weight of about one half
+        if reach >= 0:
+            g = h // (H // G)
+            u = q[n - 1, h * D:(h + 1) * D].float()
+            kv[n - 1 - reach, g * D:(g + 1) * D] = (u * (30.0 / (s.scale * u.pow(2).sum()))).to(dtype)
+    k, v = kv[:n, :G * D].double().view(n, G, D), kv[:n, G * D:s.kv_width].double().view(n, G, V)
+    rows = [n - 1, n - 2, 700, 100, 1, 0]
+    i, j = torch.tensor(rows, device="cuda")[:, None], torch.arange(n, device="cuda")[None]
+    products = torch.stack([q[:, h * D:(h + 1) * D].double() @ k[:, h // (H // G)].t() for h in range(H)]).max().item() * s.scale
+    bias = wa.ScoreBias(slopes, add, products * 1.001)
+    assert H == 1 or min(wa.sigmoid_reach(bias.limit, a, b) for a, b in zip(add.tolist(), slopes.tolist())) < 700
+    want = attend(q[rows].double().view(len(rows), H, D), k, v, s.scale, (i - j).double(), j <= i, slopes, add, True).reshape(len(rows), -1)
+    out = torch.zeros(len(rows), s.out_width, dtype=dtype, device="cuda")
+    table = torch.arange((n + 4) // bs, dtype=torch.int32, device="cuda")[None]
+    wa.attend_rows(q[rows].contiguous(), s, kv.view(-1, bs, s.row_width), table, i32(*[0] * len(rows)), i32(*[r + 1 for r in rows]), n, out, bias=bias)
+    assert rel(out, want) < tol(dtype, 1.5) and all(rel(out[x], want[x]) < tol(dtype, 2.0) for x in range(len(rows)))
+    if dtype == BF:
+        whole = torch.zeros(n, s.out_width, dtype=BF, device="cuda")
+        wa.attend_portions(torch.cat([q, kv[:n]], 1), s, None, i32(0, n), i32(0, n), n, whole, bias=bias)
+        assert rel(whole[rows], want) < tol(BF)
+        wa.attend_portions(q[900:].contiguous(), s, kv[:n].contiguous(), i32(0, n - 900), i32(0, n), n - 900, whole, bias=bias)
+        assert rel(whole[[n - 901, n - 902]], want[:2]) < tol(BF)
+
+
 def test_sigmoid_weights_far_below_and_above_one():
     """Scores of hundreds either way: weights of zero and one, no overflow where two of them share a reciprocal."""
     from trainscale_b200.ops import window_attention as wa
@@ -277,7 +314,7 @@ def test_sigmoid_weights_far_below_and_above_one():
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("heads,dim,vdim,rank", [(3, 24, 16, 48), (2, 12, 20, 33), (5, 64, 80, 64), (17, 40, 24, 272)])
+@pytest.mark.parametrize("heads,dim,vdim,rank", [(3, 24, 16, 48), (2, 12, 20, 33), (5, 64, 72, 80), (17, 40, 24, 272)])
 def test_latent_attention_without_positions(dtype, heads, dim, vdim, rank):
     """No rotated part and no window: cache rows, the latent form of single rows and, where it runs, the expanded form of portions."""
     from trainscale_b200.ops import latent_attention as L
@@ -316,7 +353,7 @@ def test_latent_attention_without_positions(dtype, heads, dim, vdim, rank):
 
 
 # ---------------------------------------------------------------------------------------------- retention
-RETENTION = [(4, 32, 64, 32), (2, 64, 64, 16), (3, 128, 256, 128), (2, 128, 128, 64), (5, 8, 8, 4), (2, 24, 40, 16), (3, 20, 36, 6), (1, 17, 9, 2),
+RETENTION = [(5, 32, 64, 32), (2, 64, 64, 16), (3, 128, 256, 128), (2, 128, 128, 64), (5, 8, 8, 4), (2, 24, 40, 16), (3, 20, 36, 6), (1, 17, 9, 2),
              (2, 256, 128, 64), (2, 96, 200, 96), (2, 64, 512, 64), (2, 40, 72, 0), (1, 72, 320, 48), (3, 80, 16, 10)]      # H, D, V, rotated
 DECAYS = (0.97, 0.9995, 0.5, 0.995, 1.0)
 
@@ -388,7 +425,7 @@ def test_retention_portions(dtype, H, D, V, rot, lens):
     assert torch.equal(state[:20], before[:20]) and torch.equal(state[20 + len(lens):], before[20 + len(lens):]) and out[:, s.out_width:].abs().sum() == 0
 
 
-@pytest.mark.parametrize("D,V", [(128, 256), (64, 64), (32, 64), (128, 128)])
+@pytest.mark.parametrize("D,V", [(128, 256), (64, 64), (48, 64), (128, 128)])
 def test_retention_chunks_keep_fp32_accuracy(D, V):
     """What the chunks add up, before it is rounded to bf16: against fp64, with large queries and keys, far below bf16 rounding."""
     from trainscale_b200.ops import recurrent

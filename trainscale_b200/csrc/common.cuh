@@ -123,6 +123,13 @@ __device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)
 // Factor sigmoid(gate) of an attention result: one gate per head or one per element.
 constexpr int GATE_HEAD = 1, GATE_ELEMENT = 2;
 
+// Distance up to which a key can have a sigmoid weight of 2^-48 or more, if no product of query and key exceeds `limit` and
+// `slope` per position is taken off `limit + add`.
+__device__ __forceinline__ int sigmoid_reach(float limit, float add, float slope) {
+  const float d = (limit + add + 33.28f) / slope;                  // 48 ln 2; infinite without a slope or a limit
+  return d < 1073741824.f ? max(0, static_cast<int>(d) + 1) : 1 << 30;
+}
+
 // Gated products: act 6 is silu(g) * u, act 7 the tanh form of gelu(g) * u, both written as g * sigmoid(y) * u.  `FAST`:
 // for results that are rounded to 16 bits.  Their weights interleave GLU_BLOCK gate rows with the GLU_BLOCK up rows of
 // the same outputs.
@@ -445,6 +452,17 @@ __device__ __forceinline__ uint32_t cluster_ctarank() {
 }
 __device__ __forceinline__ void cluster_sync_all() {
   asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+// write to the same smem offset in CTA `cta` of this cluster
+__device__ __forceinline__ void st_shared_cluster(float* p, uint32_t cta, float v) {
+  asm volatile(
+      "{\n\t"
+      ".reg .b32 ra;\n\t"
+      "mapa.shared::cluster.u32 ra, %0, %1;\n\t"
+      "st.shared::cluster.f32 [ra], %2;\n\t"
+      "}\n" ::"r"(smem_u32(p)),
+      "r"(cta), "f"(v)
+      : "memory");
 }
 // arrive on the barrier at the same smem offset in CTA `cta` of this cluster
 __device__ __forceinline__ void mbar_arrive_cluster(uint64_t* bar, uint32_t cta) {

@@ -75,6 +75,54 @@ latent_prep_kernel(T* __restrict__ proj, long long ld, int H, int dim, int rot, 
   }
 }
 
+// The same for bf16 rows without a rotated part, rank and row_width multiples of eight: one warp per token, 16-byte vectors.
+constexpr int LPV_WARPS = 4;
+__global__ void __launch_bounds__(LPV_WARPS * 32)
+latent_norm_vec_kernel(const __nv_bfloat16* __restrict__ down, long long ld, int rank, const float* __restrict__ norm_w, float eps,
+                       const long long* __restrict__ slots, __nv_bfloat16* __restrict__ cache, __nv_bfloat16* __restrict__ flat,
+                       int row_width, int rows) {
+  constexpr int NV = 4;                            // vectors of a lane: rank up to 1024
+  const int t = blockIdx.x * LPV_WARPS + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (t >= rows) return;
+  const uint4* src = reinterpret_cast<const uint4*>(down + t * ld);
+  const int vecs = rank / 8;
+  uint4 raw[NV];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) raw[i] = i * 32 + lane < vecs ? src[i * 32 + lane] : make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const uint32_t r[4] = {raw[i].x, raw[i].y, raw[i].z, raw[i].w};
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float2 f = unpack_bf16x2(r[j]);
+      ss += f.x * f.x + f.y * f.y;
+    }
+  }
+  const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(rank) + eps);
+  uint4* crow = reinterpret_cast<uint4*>(cache + slots[t] * row_width);
+  uint4* frow = flat ? reinterpret_cast<uint4*>(flat + static_cast<long long>(t) * row_width) : nullptr;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = i * 32 + lane;
+    if (c >= row_width / 8) continue;
+    uint32_t o[4] = {0u, 0u, 0u, 0u};              // columns past the latent pad the row
+    if (c < vecs) {
+      const uint32_t r[4] = {raw[i].x, raw[i].y, raw[i].z, raw[i].w};
+      const float4 wa = reinterpret_cast<const float4*>(norm_w)[2 * c], wb = reinterpret_cast<const float4*>(norm_w)[2 * c + 1];
+      const float w[8] = {wa.x, wa.y, wa.z, wa.w, wb.x, wb.y, wb.z, wb.w};
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float2 f = unpack_bf16x2(r[j]);
+        o[j] = pack_bf16x2(f.x * inv * w[2 * j], f.y * inv * w[2 * j + 1]);
+      }
+    }
+    const uint4 v = make_uint4(o[0], o[1], o[2], o[3]);
+    crow[c] = v;
+    if (frow) frow[c] = v;
+  }
+}
+
 __global__ void latent_gather_kernel(const uint4* __restrict__ cache, const long long* __restrict__ slots,
                                      uint4* __restrict__ out, long long rows, int vec) {
   const long long total = rows * vec;
@@ -431,6 +479,14 @@ extern "C" int ts_latent_prep(void* proj, long long ld, int H, int dim, int rot,
                               int row_width, int rows, int fp32, void* stream) {
   if (rows <= 0) return 0;
   if (H <= 0 || rank <= 0 || rot < 0 || rot % 2 || row_width < rank + rot) return -10;
+  const __nv_bfloat16* down = (const __nv_bfloat16*)proj + H * dim;
+  if (!fp32 && rot == 0 && rank % 8 == 0 && row_width % 8 == 0 && row_width <= 1024 && ld % 8 == 0 &&
+      ((reinterpret_cast<uintptr_t>(down) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(flat) |
+        reinterpret_cast<uintptr_t>(norm_w)) & 15u) == 0) {
+    latent_norm_vec_kernel<<<(rows + LPV_WARPS - 1) / LPV_WARPS, LPV_WARPS * 32, 0, ST(stream)>>>(
+        down, ld, rank, norm_w, eps, slots, (__nv_bfloat16*)cache, (__nv_bfloat16*)flat, row_width, rows);
+    return (int)cudaGetLastError();
+  }
   const size_t sm = sizeof(float) * (rot > 0 ? rot : 2);
   if (fp32)
     latent_prep_kernel<float><<<rows, 128, sm, ST(stream)>>>((float*)proj, ld, H, dim, rot, rank, norm_w, eps, inv_freq,

@@ -13,7 +13,7 @@
 //   warp 1       MMA issuer: S_t = Q_t K^T over the unrotated, then the rotated columns; O_t += P_t V, P_t from TMEM
 //   warps 2..9   softmax: one thread per query row; scores, running max and sum in fp32.  Or (`SIG`) weights that are not
 //                normalized: sigmoid(score + a number per head - a slope per head times the distance), so there is no running
-//                maximum, no rescaling and no sum
+//                maximum, no rescaling and no sum; with a slope the key tiles begin where a weight can reach 2^-48
 // Queries are the LAST Lq of the sequence's Lk keys.  A query sees the `window` keys up to its own, or those of its chunk of
 // `window` keys (the first key row then lies on a chunk's border), and besides the first `keep` key rows; these are the
 // sequence's first positions, which a portion's caller may have put right in front of its window.  Key tiles that no row
@@ -74,6 +74,7 @@ struct LatentPrefillParams {
   int gate_mode;                         // GATE_HEAD: column h, GATE_ELEMENT: column h * vdim + c
   const float* slopes;                   // SIG: [H] (nullptr: zeros)
   const float* add;                      // SIG: [H] (nullptr: zeros)
+  float limit;                           // SIG: no (q . k) * scale exceeds it
   float scale_log2;
   float o_scale;                         // factor of the result
   __nv_bfloat16* o;                      // [rows][o_stride], head h at column h * vdim
@@ -81,8 +82,8 @@ struct LatentPrefillParams {
 };
 
 // first key row of the window or chunk of the query at key row c
-__device__ __forceinline__ int window_first(const LatentPrefillParams& p, int c) {
-  return p.chunked ? c / p.window * p.window : max(0, c - p.window + 1);
+__device__ __forceinline__ int window_first(const LatentPrefillParams& p, int window, int c) {
+  return p.chunked ? c / window * window : max(0, c - window + 1);
 }
 
 template <bool SIG>
@@ -118,15 +119,18 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
   if ((int)blockIdx.y >= n_qblocks) return;
   const int qb = n_qblocks - 1 - blockIdx.y;
   const int off = Lk - Lq;
+  // sigmoid weights that fade with the distance: keys behind the last one that can count are not looked at
+  const int window = SIG && !p.chunked && p.slopes
+                         ? min(p.window, sigmoid_reach(p.limit, p.add ? p.add[h] : 0.f, p.slopes[h]) + 1) : p.window;
   // the block's key tiles: those of the kept rows left of its first window, then the windows' (kb_lo on).  Query tile t works
   // on [0, held[t]), which hold kept rows (also where they are among the windows'), and on [first[t], nkv[t])
   int r0[2], held[2], first[2], nkv[2];
   const int keep_tiles = (p.keep + 127) / 128;
-  const int kb_lo = window_first(p, qb * 256 + off) / 128, kept = min(keep_tiles, kb_lo);
+  const int kb_lo = window_first(p, window, qb * 256 + off) / 128, kept = min(keep_tiles, kb_lo);
 #pragma unroll
   for (int t = 0; t < 2; ++t) {
     r0[t] = qb * 256 + t * 128;
-    first[t] = kept + window_first(p, r0[t] + off) / 128 - kb_lo;
+    first[t] = kept + window_first(p, window, r0[t] + off) / 128 - kb_lo;
     held[t] = min(keep_tiles, first[t]);
     nkv[t] = r0[t] >= Lq ? 0 : max(0, kept + (min(Lk, r0[t] + 128 + off) + 127) / 128 - kb_lo);
   }
@@ -246,8 +250,8 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
     const int nt = nkv[t];
     const float sc = p.scale_log2;
     const int limit = min(Lk - 1, row + off);          // last visible key
-    const int lo = window_first(p, row + off);         // first key of the window
-    const int lo_last = window_first(p, r0[t] + 127 + off);
+    const int lo = window_first(p, window, row + off);         // first key of the window
+    const int lo_last = window_first(p, window, r0[t] + 127 + off);
     constexpr float LOG2E = 1.4426950408889634f;
     const float slope = SIG && p.slopes ? p.slopes[h] * LOG2E : 0.f, add = SIG && p.add ? p.add[h] * LOG2E : 0.f;
     for (int i = 0; i < nt && alive; ++i) {
@@ -513,11 +517,11 @@ extern "C" int ts_latent_prefill(const void* q, long long q_ld, long long q_rows
 // q: rows [q_rows][q_ld], head h at column h * dim.  k / v: rows [k_rows][kv_ld], key/value head g at columns g * dim and
 // g * vdim.  cu_q / cu_k: [sequences + 1].  window, keep, chunked: which keys a query sees (top of the file).
 // sigmoid: weights sigmoid(score + add[h] - slopes[h] * distance), not normalized (add and slopes: nullptr for zeros; without
-// sigmoid there are none).  out: [q_rows][o_stride] = o_scale * attention (* sigmoid(gate)).
+// sigmoid there are none); no (q . k) * scale may exceed `limit` (infinity: unknown).  out: [q_rows][o_stride] = o_scale * attention (* sigmoid(gate)).
 extern "C" int ts_window_prefill(const void* q, long long q_ld, long long q_rows, const void* k, const void* v,
                                  long long kv_ld, long long k_rows, const int* cu_q, const int* cu_k, int sequences,
                                  int max_q, int H, int G, int dim, int vdim, int window, int keep, int chunked, float scale,
-                                 float o_scale, const float* slopes, const float* add, int sigmoid, const void* gate,
+                                 float o_scale, const float* slopes, const float* add, int sigmoid, float limit, const void* gate,
                                  long long gate_ld, int gate_mode, void* out, long long o_stride, void* stream) {
   if (sequences <= 0 || max_q <= 0) return 0;
   LatentPrefillPlan pl;
@@ -539,7 +543,7 @@ extern "C" int ts_window_prefill(const void* q, long long q_ld, long long q_rows
   p.gate = reinterpret_cast<const __nv_bfloat16*>(gate); p.gate_ld = gate_ld; p.gate_mode = gate_mode;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.o = reinterpret_cast<__nv_bfloat16*>(out); p.o_stride = o_stride;
-  p.slopes = slopes; p.add = add;
+  p.slopes = slopes; p.add = add; p.limit = limit;
   return sigmoid ? launch_prefill<true>(tQ, tQ, tK, tK, tV, pl, p, dim, 0, vdim, sequences, max_q, stream)
                  : launch_prefill<false>(tQ, tQ, tK, tK, tV, pl, p, dim, 0, vdim, sequences, max_q, stream);
 }

@@ -1266,22 +1266,24 @@ __global__ void __launch_bounds__(128) retention_blocks_kernel(RetentionParams p
   if (lane == 0) out[64] = pw[n];
 }
 
-// Single rows: projection -> gated norm, state advanced.  One CTA per (row, head).
+// Single rows: projection -> gated norm, state advanced.  A cluster of CTAs per (row, head), each with its share of the value
+// columns; their sums of squares meet in every CTA's shared memory.  grid (rows, H, shares), cluster (1, 1, shares).
 constexpr int RTS_THREADS = 256;
+constexpr int RTS_SHARES = 8;
 template <typename T, int VEC>
 __global__ void __launch_bounds__(RTS_THREADS) retention_step_kernel(RetentionParams p) {
   extern __shared__ __align__(16) float smf[];
-  __shared__ float scratch[32];
-  const int row = blockIdx.x, h = blockIdx.y, D = p.D, V = p.V, tid = threadIdx.x;
+  __shared__ float scratch[32], sums[RTS_SHARES];
+  const int row = blockIdx.x, h = blockIdx.y, shares = gridDim.z, D = p.D, V = p.V / shares, v0 = blockIdx.z * V, tid = threadIdx.x;
   const int nvec = V / VEC, span = min(nvec, RTS_THREADS), groups = RTS_THREADS / span;
-  float* vs = smf;                               // [V]
+  float* vs = smf;                               // [V] this CTA's columns
   float* part = vs + (V + 3) / 4 * 4;            // [groups][V]
   float* qs = part + (groups * V + 3) / 4 * 4;   // [D]
   float* ks = qs + D;                            // [D]
   const int prev = p.row_prev[row], next = p.row_next[row];
   const T* x = reinterpret_cast<const T*>(p.proj) + row * p.ld;
   const float* cs = p.angles + static_cast<long long>(row) * p.rot;
-  const long long head = static_cast<long long>(h) * D * V;
+  const long long head = static_cast<long long>(h) * D * p.V + v0;
   const float* S = prev >= 0 ? p.state + prev * p.state_ld + head : nullptr;
   float* N = next >= 0 ? p.state + next * p.state_ld + head : nullptr;
   const float g = p.powers[h * p.powers_ld + 1];
@@ -1289,7 +1291,7 @@ __global__ void __launch_bounds__(RTS_THREADS) retention_step_kernel(RetentionPa
     qs[c] = rotated(x + h * D, c, p.rot, cs, 1.f);
     ks[c] = rotated(x + (p.H + h) * D, c, p.rot, cs, p.k_scale);
   }
-  for (int c = tid; c < V; c += RTS_THREADS) vs[c] = to_f32(x[2 * p.H * D + h * V + c]);
+  for (int c = tid; c < V; c += RTS_THREADS) vs[c] = to_f32(x[2 * p.H * D + h * p.V + v0 + c]);
   __syncthreads();
   const int grp = tid / span;
   for (int base = 0; base < nvec; base += span) {
@@ -1304,14 +1306,14 @@ __global__ void __launch_bounds__(RTS_THREADS) retention_step_kernel(RetentionPa
       float st[VEC];
 #pragma unroll
       for (int e = 0; e < VEC; ++e) st[e] = 0.f;
-      if (S) load_vec<VEC>(S + static_cast<long long>(r) * V + cv, st);
+      if (S) load_vec<VEC>(S + static_cast<long long>(r) * p.V + cv, st);
       const float k = ks[r], q = qs[r];
 #pragma unroll
       for (int e = 0; e < VEC; ++e) {
         st[e] = g * st[e] + k * v[e];
         acc[e] += st[e] * q;
       }
-      if (N) store_vec<VEC>(N + static_cast<long long>(r) * V + cv, st);
+      if (N) store_vec<VEC>(N + static_cast<long long>(r) * p.V + cv, st);
     }
     store_vec<VEC>(part + grp * V + cv, acc);
   }
@@ -1324,9 +1326,15 @@ __global__ void __launch_bounds__(RTS_THREADS) retention_step_kernel(RetentionPa
     ss += s * s;
   }
   ss = block_sum(ss, scratch);
-  const float inv = 1.f / sqrtf(ss / static_cast<float>(V) + p.eps);
-  const T* gate = x + 2 * p.H * D + (p.H + h) * V;
-  T* out = reinterpret_cast<T*>(p.out) + row * p.out_ld + h * V;
+  if (shares > 1) {
+    if (tid < shares) st_shared_cluster(&sums[blockIdx.z], tid, ss);
+    cluster_sync_all();
+    ss = 0.f;
+    for (int i = 0; i < shares; ++i) ss += sums[i];
+  }
+  const float inv = 1.f / sqrtf(ss / static_cast<float>(p.V) + p.eps);
+  const T* gate = x + 2 * p.H * D + (p.H + h) * p.V + v0;
+  T* out = reinterpret_cast<T*>(p.out) + row * p.out_ld + h * p.V + v0;
   for (int c = tid; c < V; c += RTS_THREADS) out[c] = from_f32<T>(vs[c] * inv * silu(to_f32(gate[c])));
 }
 
@@ -1862,6 +1870,28 @@ static int retention_params(RetentionParams& p, const void* proj, long long ld, 
   return 0;
 }
 
+// Shares of the value columns: enough CTAs for two per SM, at least 32 columns each.
+template <typename T, int VEC> static int launch_retention_step(const RetentionParams& p, cudaStream_t st) {
+  int shares = 1;
+  while (VEC == 4 && shares < RTS_SHARES && p.V % (shares * 2 * 4) == 0 && p.V / (shares * 2) >= 32 &&
+         static_cast<long long>(p.rows) * p.H * shares < 2 * sm_count())
+    shares *= 2;
+  const int V = p.V / shares, nvec = V / VEC, groups = RTS_THREADS / (nvec < RTS_THREADS ? nvec : RTS_THREADS);
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(p.rows, p.H, shares);
+  cfg.blockDim = dim3(RTS_THREADS);
+  cfg.dynamicSmemBytes = ((V + 3) / 4 * 4 + (groups * V + 3) / 4 * 4 + 2 * p.D) * sizeof(float);
+  cfg.stream = st;
+  cudaLaunchAttribute at[1];
+  at[0].id = cudaLaunchAttributeClusterDimension;
+  at[0].val.clusterDim.x = 1;
+  at[0].val.clusterDim.y = 1;
+  at[0].val.clusterDim.z = shares;
+  cfg.attrs = at;
+  cfg.numAttrs = 1;
+  return (int)cudaLaunchKernelEx(&cfg, retention_step_kernel<T, VEC>, p);
+}
+
 // Single rows of retention: projection -> out [rows][out_ld] = norm * silu(gate), state advanced.
 extern "C" int ts_retention_step(const void* proj, long long ld, const float* angles, const float* powers, int powers_ld, float k_scale, float eps,
                                  float* state, long long state_ld, const int* row_prev, const int* row_next, void* out,
@@ -1871,17 +1901,8 @@ extern "C" int ts_retention_step(const void* proj, long long ld, const float* an
   if (int e = retention_params(p, proj, ld, angles, powers, powers_ld, k_scale, state, state_ld, row_prev, row_next, H, D, V, rot)) return e;
   p.eps = eps; p.out = out; p.out_ld = out_ld; p.rows = rows;
   const bool vec = V % 4 == 0 && state_ld % 4 == 0;
-  const int nvec = vec ? V / 4 : V, groups = RTS_THREADS / (nvec < RTS_THREADS ? nvec : RTS_THREADS);
-  const size_t smem = ((V + 3) / 4 * 4 + (groups * V + 3) / 4 * 4 + 2 * D) * sizeof(float);
-  const dim3 grid(rows, H);
-  if (fp32) {
-    if (vec) retention_step_kernel<float, 4><<<grid, RTS_THREADS, smem, ST(stream)>>>(p);
-    else retention_step_kernel<float, 1><<<grid, RTS_THREADS, smem, ST(stream)>>>(p);
-  } else {
-    if (vec) retention_step_kernel<__nv_bfloat16, 4><<<grid, RTS_THREADS, smem, ST(stream)>>>(p);
-    else retention_step_kernel<__nv_bfloat16, 1><<<grid, RTS_THREADS, smem, ST(stream)>>>(p);
-  }
-  return (int)cudaGetLastError();
+  if (fp32) return vec ? launch_retention_step<float, 4>(p, ST(stream)) : launch_retention_step<float, 1>(p, ST(stream));
+  return vec ? launch_retention_step<__nv_bfloat16, 4>(p, ST(stream)) : launch_retention_step<__nv_bfloat16, 1>(p, ST(stream));
 }
 
 template <typename T> static int dispatch_retention_scan(const RetentionParams& p, int portions, cudaStream_t st) {

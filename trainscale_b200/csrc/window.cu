@@ -13,7 +13,8 @@
 //                     cache; the result may be multiplied by the sigmoid of a gate per head or per element
 //
 // Scores are (q . k) * scale, plus a number per head, minus a slope per head times the distance of query and key (either may be
-// absent).  Weights are their softmax over the visible keys or, without any normalization, their sigmoids.
+// absent).  Weights are their softmax over the visible keys or, without any normalization, their sigmoids.  With a bound of the
+// products and a slope, sigmoids fade below 2^-48 at a distance that is known beforehand; keys beyond it are not read.
 // Portions of prompts: ts_window_prefill (latent_prefill.cu).
 //
 // Decoding reads every cached key and value in the window once per key/value head.  `window_attend_mma_kernel` (bf16): the
@@ -257,6 +258,7 @@ struct WindowAttendParams {
   const float* slopes;         // [H] subtracted from a score per position of distance (nullptr: none)
   const float* add;            // [H] added to every score (nullptr: none)
   int sigmoid;                 // weights: sigmoid(score), not normalized
+  float limit;                 // no (q . k) * scale exceeds it: sigmoid weights that fade with the distance end at some key
   int rows, H, G, dim, vdim, row_width, max_blocks, block_size, window, keep, chunked, chunk, splits;
   float scale, o_scale;
 };
@@ -264,8 +266,8 @@ struct WindowAttendParams {
 // A row's visible keys, numbered 0 .. count - 1 in key order: the kept first positions, then those from `lo` on.
 struct VisibleKeys {
   int lo, kept, count;
-  __device__ VisibleKeys(const WindowAttendParams& p, int len) {
-    lo = p.chunked ? (len - 1) / p.window * p.window : max(0, len - p.window);
+  __device__ VisibleKeys(const WindowAttendParams& p, int len, int reach) {
+    lo = p.chunked ? (len - 1) / p.window * p.window : max(0, len - min(p.window, reach));
     kept = min(p.keep, lo);
     count = len - lo + kept;
   }
@@ -304,7 +306,7 @@ __global__ void __launch_bounds__(128) window_attend_simt_kernel(WindowAttendPar
   for (int i = threadIdx.x; i < p.vdim; i += blockDim.x) acc[i] = 0.f;
   float m = p.sigmoid ? 0.f : -INFINITY, l = 0.f;
   const float slope = p.slopes ? p.slopes[h] : 0.f, add = p.add ? p.add[h] : 0.f;
-  const VisibleKeys vis(p, len);
+  const VisibleKeys vis(p, len, p.sigmoid ? sigmoid_reach(p.limit, add, slope) : 1 << 30);
   auto key_row = [&](int i) {
     const int j = vis.position(i);
     return cache + (static_cast<long long>(bt[j / p.block_size]) * p.block_size + j % p.block_size) * p.row_width;
@@ -390,8 +392,14 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attend_mma_kernel(Window
   const int nh = min(16, (g + 1) * group - h0);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
   const int len = p.row_len[row];
-  const VisibleKeys vis(p, len);
-  const int j0 = split * p.chunk, j1 = min(vis.count, j0 + p.chunk);       // this CTA's share of them
+  int reach = 1 << 30;                     // of the farthest-reaching head
+  if (SIG && p.slopes) {
+    reach = 0;
+    for (int i = 0; i < nh; ++i) reach = max(reach, sigmoid_reach(p.limit, p.add ? p.add[h0 + i] : 0.f, p.slopes[h0 + i]));
+  }
+  const VisibleKeys vis(p, len, reach);
+  const int chunk = SIG ? ((vis.count + p.splits - 1) / p.splits + WA_KT - 1) / WA_KT * WA_KT : p.chunk;
+  const int j0 = split * chunk, j1 = min(vis.count, j0 + chunk);           // this CTA's share of them
   const int* bt = p.block_table + static_cast<long long>(p.row_seq[row]) * p.max_blocks;
   const __nv_bfloat16* kc = reinterpret_cast<const __nv_bfloat16*>(p.cache) + g * p.dim;
   const __nv_bfloat16* vc = reinterpret_cast<const __nv_bfloat16*>(p.cache) + p.G * p.dim + g * p.vdim;
@@ -685,12 +693,12 @@ extern "C" int ts_window_splits(int rows, int H, int G, int dim, int vdim, int k
   return s < 1 ? 1 : s;
 }
 
-// window, keep, chunked: which keys a row sees; slopes, add, sigmoid: their weights (top of the file).  `keys`: upper bound of their number; `splits` of ts_window_splits with the workspaces it needs (splits > 1).
+// window, keep, chunked: which keys a row sees; slopes, add, sigmoid, limit: their weights (top of the file).  `keys`: upper bound of their number; `splits` of ts_window_splits with the workspaces it needs (splits > 1).
 extern "C" int ts_window_attend(const void* q, long long q_ld, const void* cache, const int* block_table, int max_blocks,
                                 const int* row_seq, const int* row_len, void* out, long long out_ld, float* part_out,
                                 float* part_lse, int rows, int H, int G, int dim, int vdim, int row_width, int block_size,
                                 int window, int keep, int chunked, int keys, int splits, float scale, float o_scale,
-                                const float* slopes, const float* add, int sigmoid, const void* gate, long long gate_ld,
+                                const float* slopes, const float* add, int sigmoid, float limit, const void* gate, long long gate_ld,
                                 int gate_mode, int fp32, void* stream) {
   if (rows <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G || dim <= 0 || vdim <= 0 || window <= 0 || keep < 0 || keys <= 0 || splits < 1 ||
@@ -700,7 +708,7 @@ extern "C" int ts_window_attend(const void* q, long long q_ld, const void* cache
   p.q = q; p.q_ld = q_ld; p.cache = cache; p.block_table = block_table; p.row_seq = row_seq; p.row_len = row_len; p.out = out;
   p.out_ld = out_ld; p.part_out = part_out; p.part_lse = part_lse; p.rows = rows; p.H = H; p.G = G; p.dim = dim;
   p.vdim = vdim; p.row_width = row_width; p.max_blocks = max_blocks; p.block_size = block_size; p.window = window;
-  p.keep = keep; p.chunked = chunked; p.slopes = slopes; p.add = add; p.sigmoid = sigmoid; p.gate = gate; p.gate_ld = gate_ld; p.gate_mode = gate_mode;
+  p.keep = keep; p.chunked = chunked; p.slopes = slopes; p.add = add; p.sigmoid = sigmoid; p.limit = limit; p.gate = gate; p.gate_ld = gate_ld; p.gate_mode = gate_mode;
   p.splits = splits; p.chunk = ((keys + splits - 1) / splits + 15) / 16 * 16; p.scale = scale; p.o_scale = o_scale;
   const bool vec = window_mma_ok(dim, vdim, fp32) && scale > 0.f && q_ld % 8 == 0 && row_width % 8 == 0 &&
                    (reinterpret_cast<uintptr_t>(q) & 15u) == 0 && (reinterpret_cast<uintptr_t>(cache) & 15u) == 0;

@@ -370,6 +370,15 @@ def lovurax_table(z: dict, rows: int, lengths: list[tuple[int, int]]) -> list[tu
     W = z["width"]
     keys, pairs = _seen(lengths, KeyMask(UNBOUNDED))
 
+    # key rows per key/value head, and (query, key, head) triples, whose sigmoid weights can count: head norms of ones, scores' addend
+    # and temperature of the random model
+    from ..models.lovurax import RANDOM_SCORE_ADD
+    H, group, longest = z["heads"], z["heads"] // z["kv"], max(start + n for start, n in lengths)
+    limit = 1.02 * z["dim"] ** 0.5 * (1.0 + 0.1 * math.log(longest // 4096 + 1))
+    seen = [_seen(lengths, KeyMask(window.sigmoid_reach(limit, RANDOM_SCORE_ADD, slope) + 1)) for slope in window.distance_slopes(H).tolist()]
+    near_keys = sum(max(k for k, _ in seen[g:g + group]) for g in range(0, H, group)) / z["kv"]
+    near_pairs = sum(n for _, n in seen)
+
     def boundary(a, k, out):
         final = isinstance(out, torch.Tensor)                  # last boundary: only the wanted rows
         T = (out if final else out[0]).shape[0]
@@ -388,11 +397,11 @@ def lovurax_table(z: dict, rows: int, lengths: list[tuple[int, int]]) -> list[tu
          lambda a, k, o: (a[0].shape[0] * 2 * (a[1].rank + a[1].row_width * (2 if o is not None else 1)), 0.0)),
         (latent, "gather_rows", "key gather", lambda a, k, o: (2 * _bytes(o), 0.0)),
         (window, "attend_rows", "attention (sigmoid, rows)",
-         lambda a, k, o: (keys * a[1].kv_width * 2 + a[0].shape[0] * (a[1].q_width + 2 * a[1].out_width) * 2,
-                          2.0 * pairs * a[1].heads * (a[1].dim + a[1].vdim))),
+         lambda a, k, o: (near_keys * a[1].kv_width * 2 + a[0].shape[0] * (a[1].q_width + 2 * a[1].out_width) * 2,
+                          2.0 * near_pairs * (a[1].dim + a[1].vdim))),
         (window, "attend_portions", "attention (sigmoid, portions)",
          lambda a, k, o: (a[0].shape[0] * (a[1].q_width + a[1].kv_width + 2 * a[1].out_width) * 2,
-                          2.0 * pairs * a[1].heads * (a[1].dim + a[1].vdim))),
+                          2.0 * near_pairs * (a[1].dim + a[1].vdim))),
         (latent, "attend_latent", "attention (latent space)",
          lambda a, k, o: (keys * a[2].row_width * 2 + 2 * _bytes(a[0]), 4.0 * pairs * a[2].heads * a[2].rank)),
         (latent, "attend_expanded", "attention (latent, portions)",
@@ -405,6 +414,8 @@ def lovurax_table(z: dict, rows: int, lengths: list[tuple[int, int]]) -> list[tu
         # two fp32 products of every state element per token
         (recurrent, "retention_scan", "retention scan",
          lambda a, k, o: (a[0].shape[0] * (2 * a[1].qk_width + a[1].out_width) * 2 + _bytes(o), 0.0, 4.0 * o.numel() * a[1].dim)),
+        (recurrent, "retention_chunks", "retention (chunks, norm, gate)",
+         lambda a, k, o: (a[0].shape[0] * (a[1].proj_width + a[1].out_width) * 2, 0.0, 4.0 * a[0].shape[0] * a[1].out_width * a[1].dim)),
         (recurrent, "gated_norm", "gated norm", lambda a, k, o: (_bytes(a[0]) + 2 * _bytes(a[4]), 0.0)),
     ]
 

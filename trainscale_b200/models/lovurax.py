@@ -34,6 +34,8 @@ from ..ops.stream import ElementGate
 from ..ops.window_attention import ScoreBias, WindowShape
 from .served import ServedDecoder, fp32_param, require, up8, weight_param
 
+RANDOM_SCORE_ADD = -4.0        # of a randomly initialised attention mixer
+
 
 @dataclass(frozen=True)
 class RetentionConfig:
@@ -139,7 +141,7 @@ def pattern_config(kinds: str, vocab: int, width: int, heads: int, kv_heads: int
 
 
 PRESETS: dict[str, LovuraxConfig] = {
-    "lovurax-tiny": pattern_config("rarl", vocab=32000, width=320, heads=4, kv_heads=2, dim=64, ret_heads=4, ret_dim=32, ret_vdim=64,
+    "lovurax-tiny": pattern_config("rarl", vocab=32000, width=256, heads=4, kv_heads=2, dim=64, ret_heads=2, ret_dim=64, ret_vdim=128,
                                    latent_dim=64, latent_vdim=64, rank=96, ff=640, temperature=(0.2, 64)),
     "lovurax-2b": pattern_config("rarl" * 5, vocab=64000, width=2048, heads=16, kv_heads=4, dim=128, ret_heads=8, ret_dim=128,
                                  ret_vdim=256, latent_dim=128, latent_vdim=128, rank=512, ff=8192, rope_base=500000.0),
@@ -240,6 +242,7 @@ class AttentionMixer(Mixer):
         self.cfg = cfg
         self.q_norm, self.k_norm, self.score_add = fp32_param(s.dim), fp32_param(s.dim), fp32_param(s.heads)
         self.register_buffer("slopes", window.distance_slopes(s.heads).to(self.q_norm.device), persistent=False)
+        self.limit = math.inf                     # of a score before its temperature and bias
 
     def tensors(self):
         s = self.cfg.shape
@@ -249,13 +252,23 @@ class AttentionMixer(Mixer):
         yield "pb", self.score_add
         yield "o", self.w_o[:, :s.out_width]
 
+    def finalize(self) -> None:
+        """A normed head has at most dim in its square sum, so the norms' largest weights bound every product (2% for rounding)."""
+        s = self.cfg.shape
+        self.limit = 1.02 * abs(s.scale) * s.dim * float(self.q_norm.abs().max() * self.k_norm.abs().max())
+
+    def score_bias(self, longest: int) -> ScoreBias:
+        """For sequences of up to `longest` tokens; the temperature is one at the first token and moves one way from there."""
+        coef, every = self.cfg.shape.temperature
+        return ScoreBias(self.slopes, self.score_add, self.limit * max(1.0, abs(1.0 + coef * math.log(longest // every + 1))))
+
     def cache_entry(self) -> dict[str, tuple[int, ...]]:
         return {"kv": (self.cfg.shape.row_width,)}
 
     def mix(self, proj, out, batch, cache, state, ctx: StepContext) -> None:
         s, T, rows_cache = self.cfg.shape, proj.shape[0], cache["kv"]
         window.prepare(proj, s, self.q_norm, self.k_norm, self.eps, None, batch.slots, rows_cache, pos=batch.positions)
-        gate, bias = proj[:, s.in_width:s.in_width + s.out_width], ScoreBias(self.slopes, self.score_add)
+        gate, bias = proj[:, s.in_width:s.in_width + s.out_width], self.score_bias(batch.max_len)
         tensor_cores = proj.is_cuda and proj.dtype == torch.bfloat16 and window.portions_supported(s)
         nd = batch.n_single if tensor_cores else T
         if nd > 0:
@@ -397,7 +410,7 @@ class LovuraxForCausalLM(ServedDecoder):
             elif leaf in ("b", "act"):
                 t.zero_()
             elif leaf == "pb":
-                t.fill_(-4.0)
+                t.fill_(RANDOM_SCORE_ADD)
             else:
                 t.normal_(0.0, 1.0 / math.sqrt(t.shape[-1]), generator=gen)
         self.finalize()

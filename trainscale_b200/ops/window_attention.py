@@ -11,13 +11,14 @@ from __future__ import annotations
 
 import ctypes
 import functools
+import math
 from dataclasses import dataclass
 
 import torch
 
 from . import _lib
 from .latent_attention import gate_args
-from .masks import KeyMask
+from .masks import UNBOUNDED, KeyMask
 
 _ll, _f = ctypes.c_longlong, ctypes.c_float
 
@@ -71,6 +72,8 @@ class ScoreBias:
     """Terms of a head's scores besides q . k * scale, fp32 [heads]; either may be None."""
     slopes: torch.Tensor | None = None    # times the distance of query and key, taken off
     add: torch.Tensor | None = None
+    limit: float = math.inf               # no q . k * scale exceeds it; then sigmoid weights that fade with the distance are left
+                                          # out where they are below 2^-48
 
 
 NO_BIAS = ScoreBias()
@@ -79,6 +82,11 @@ NO_BIAS = ScoreBias()
 def distance_slopes(heads: int) -> torch.Tensor:
     """Slopes 2^(-8 (h + 1) / heads), a geometric series over the heads that ends at 2^-8."""
     return torch.tensor([2.0 ** (-8.0 * (h + 1) / heads) for h in range(heads)], dtype=torch.float32)
+
+
+def sigmoid_reach(limit: float, add: float, slope: float) -> int:
+    """Distance up to which a sigmoid weight can be 2^-48 or more, as the kernels compute it."""
+    return UNBOUNDED if math.isinf(limit) or slope <= 0 else max(0, min(UNBOUNDED, int((limit + add + 33.28) / slope) + 1))
 
 
 @functools.lru_cache(maxsize=None)
@@ -184,7 +192,7 @@ def attend_rows(proj: torch.Tensor, s: WindowShape, cache, block_table, row_seq,
         _lib.ptr(proj), _ll(proj.stride(0)), _lib.ptr(cache), _lib.ptr(block_table), block_table.shape[1], _lib.ptr(row_seq),
         _lib.ptr(row_len), _lib.ptr(out), _ll(out.stride(0)), _lib.ptr(po), _lib.ptr(pl), T, s.heads, s.kv_heads, s.dim,
         s.vdim, s.row_width, bs, s.window, s.keep, int(s.chunked), keys, splits, _f(s.scale), _f(out_scale), _lib.ptr(bias.slopes),
-        _lib.ptr(bias.add), int(s.sigmoid), gp, gld, mode, fp32, _lib.stream_ptr())
+        _lib.ptr(bias.add), int(s.sigmoid), _f(bias.limit), gp, gld, mode, fp32, _lib.stream_ptr())
     _lib.check(rc, "ts_window_attend")
 
 
@@ -201,5 +209,6 @@ def attend_portions(proj: torch.Tensor, s: WindowShape, rows: torch.Tensor | Non
         _lib.ptr(proj), _ll(proj.stride(0)), _ll(proj.shape[0]), ctypes.c_void_p(at),
         ctypes.c_void_p(at + s.kv_heads * s.dim * proj.element_size()), _ll(src.stride(0)), _ll(src.shape[0]), _lib.ptr(cu_q),
         _lib.ptr(cu_k), cu_q.numel() - 1, max_q, s.heads, s.kv_heads, s.dim, s.vdim, s.window, s.keep, int(s.chunked),
-        _f(s.scale), _f(out_scale), _lib.ptr(bias.slopes), _lib.ptr(bias.add), int(s.sigmoid), gp, gld, mode, _lib.ptr(out), _ll(out.stride(0)), _lib.stream_ptr())
+        _f(s.scale), _f(out_scale), _lib.ptr(bias.slopes), _lib.ptr(bias.add), int(s.sigmoid), _f(bias.limit), gp, gld, mode,
+        _lib.ptr(out), _ll(out.stride(0)), _lib.stream_ptr())
     _lib.check(rc, "ts_window_prefill")
