@@ -94,19 +94,59 @@ __device__ __forceinline__ float2 unpack_bf16x2(uint32_t v) {
   return __bfloat1622float2(b);
 }
 
+// two fp32 lanes in one instruction
+__device__ __forceinline__ uint64_t pack_f32x2(float lo, float hi) {
+  uint64_t d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+  return d;
+}
+__device__ __forceinline__ float2 unpack_f32x2(uint64_t v) {
+  float2 d;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(d.x), "=f"(d.y) : "l"(v));
+  return d;
+}
+__device__ __forceinline__ uint64_t fma_f32x2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ uint64_t add_f32x2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ uint64_t mul_f32x2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+
 // a v^2 + v / 2 for v > 0, b (e^v - 1 - v) + v / 2 for v <= 0.  Near zero the bracket is a power series: the difference
 // would cancel.
-template <bool FAST> __device__ __forceinline__ float xielu(float v, float a, float b) {
+__device__ __forceinline__ float xielu(float v, float a, float b) {
   const float n = fminf(v, 0.f);
   const float series = n * n * (0.5f + n * (1.f / 6.f + n * (1.f / 24.f + n * (1.f / 120.f + n * (1.f / 720.f)))));
-  const float left = n > -0.25f ? series : (FAST ? __expf(n) : expf(n)) - 1.f - n;
+  const float left = n > -0.25f ? series : expf(n) - 1.f - n;
   const float p = fmaxf(v, 0.f);
   return a * p * p + b * left + 0.5f * v;
 }
 
+// The same of two values, for results that are rounded to 16 bits (close to zero the linear term hides what the shorter series
+// and the difference lose).
+__device__ __forceinline__ float2 xielu_pair(float x, float y, float a, float b) {
+  const uint64_t v = pack_f32x2(x, y), minus = pack_f32x2(-1.f, -1.f), half = pack_f32x2(0.5f, 0.5f);
+  const float nx = fminf(x, 0.f), ny = fminf(y, 0.f);
+  const uint64_t n = pack_f32x2(nx, ny), p = fma_f32x2(n, minus, v);
+  const float2 l = unpack_f32x2(mul_f32x2(n, pack_f32x2(1.4426950408889634f, 1.4426950408889634f)));
+  const float2 e = unpack_f32x2(fma_f32x2(n, minus, add_f32x2(pack_f32x2(fast_ex2(l.x), fast_ex2(l.y)), minus)));
+  const float2 s = unpack_f32x2(mul_f32x2(mul_f32x2(n, n), fma_f32x2(n, pack_f32x2(1.f / 6.f, 1.f / 6.f), half)));
+  const uint64_t left = pack_f32x2(nx > -0.00390625f ? s.x : e.x, ny > -0.00390625f ? s.y : e.y);
+  return unpack_f32x2(fma_f32x2(pack_f32x2(b, b), left, fma_f32x2(mul_f32x2(pack_f32x2(a, a), p), p, mul_f32x2(v, half))));
+}
+
 // Activations that a product may apply to its result: 1 squared ReLU, 2 tanh, 3 soft cap a * tanh(v / a), 4 a * v,
-// 5 xielu(v; a, b).  `FAST`: for results that are rounded to 16 bits.
-template <bool FAST> __device__ __forceinline__ float product_act(float v, int act, float a, float b) {
+// 5 xielu(v; a, b).
+__device__ __forceinline__ float product_act(float v, int act, float a, float b) {
   if (act == 1) {
     v = fmaxf(v, 0.f);
     return v * v;
@@ -114,7 +154,7 @@ template <bool FAST> __device__ __forceinline__ float product_act(float v, int a
   if (act == 2) return tanhf(v);
   if (act == 3) return a * tanhf(v / a);
   if (act == 4) return a * v;
-  if (act == 5) return xielu<FAST>(v, a, b);
+  if (act == 5) return xielu(v, a, b);
   return v;
 }
 

@@ -65,13 +65,17 @@ __device__ __forceinline__ void gemm_activate(const GemmParams& p, uint32_t* r, 
   const float a = p.act_a;
   if (p.act == 1) {
 #pragma unroll
-    for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(product_act<true>(__uint_as_float(r[j]), 1, a, 0.f));
+    for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(product_act(__uint_as_float(r[j]), 1, a, 0.f));
   } else if (p.act == 4) {
 #pragma unroll
     for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(a * __uint_as_float(r[j]));
   } else if (p.act == 5) {
 #pragma unroll
-    for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(xielu<true>(__uint_as_float(r[j]), a, p.act_b));
+    for (int j = 0; j < 32; j += 2) {
+      const float2 y = xielu_pair(__uint_as_float(r[j]), __uint_as_float(r[j + 1]), a, p.act_b);
+      r[j] = __float_as_uint(y.x);
+      r[j + 1] = __float_as_uint(y.y);
+    }
   } else {
 #pragma unroll
     for (int j = 0; j < 32; ++j) {

@@ -157,7 +157,7 @@ skinny_gemm_kernel(SkinnyParams p) {
           for (int w = 0; w < KW; ++w) f += red[tile * KW + w][n + 8][tk];
           v = glu_act<true>(v, f, p.act);
         } else {
-          if (nn < p.act_cols) v = product_act<false>(v, p.act, p.act_a, p.act_b);
+          if (nn < p.act_cols) v = product_act(v, p.act, p.act_a, p.act_b);
         }
         skinny_store<__nv_bfloat16>(p, g, p.order ? p.order[first + base + tk] : base + tk, nn, v);
       }
@@ -203,7 +203,7 @@ __global__ void __launch_bounds__(256) grouped_simt_kernel(SkinnyParams p) {
     for (int t = 0; t < TM; ++t) {
       float v = warp_sum(acc[t]);
       if (glu) v = glu_act<false>(v, warp_sum(fac[t]), p.act);
-      else if (n < p.act_cols) v = product_act<false>(v, p.act, p.act_a, p.act_b);
+      else if (n < p.act_cols) v = product_act(v, p.act, p.act_a, p.act_b);
       if (lane == 0 && base + t < m_total) skinny_store<T>(p, g, slot[t], n, v);
     }
   }
